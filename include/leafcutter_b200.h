@@ -41,7 +41,8 @@ typedef enum lc_status {
 /* ggml tensor type codes: rust/src/model/quant.rs:45-76 */
 enum {
     LC_TYPE_F32 = 0, LC_TYPE_F16 = 1, LC_TYPE_Q4_0 = 2, LC_TYPE_Q8_0 = 8,
-    LC_TYPE_Q4_K = 12, LC_TYPE_Q5_K = 13, LC_TYPE_Q6_K = 14, LC_TYPE_IQ4_NL = 20
+    LC_TYPE_Q4_K = 12, LC_TYPE_Q5_K = 13, LC_TYPE_Q6_K = 14, LC_TYPE_IQ4_NL = 20,
+    LC_TYPE_BF16 = 30
 };
 
 const char* lc_last_error(void);
@@ -177,7 +178,8 @@ typedef struct lc_model_config {
     int32_t device;           /* CUDA device ordinal */
     int32_t tp_size;          /* model-parallel ranks the model is cut into; 0 or 1 = whole model; 0 after lc_dist_init = that world */
     int32_t tp_rank;          /* which of them this handle holds (0 after lc_dist_init = that rank) */
-    int32_t reserved[5];
+    int32_t compute_f32;      /* checkpoint-directory designs: 0 = bf16 activations and cache; 1 = everything in true 32-bit */
+    int32_t reserved[4];
 } lc_model_config;
 
 /* ---- Model parallelism (no counterpart in the reference, which runs on one device) ----
@@ -254,6 +256,17 @@ int32_t lc_model_destroy(lc_model* m);
  * read the config keys (loader.rs:106-133), upload every tensor, finalize. */
 int32_t lc_model_load_gguf(const char* path, const lc_model_config* overrides, lc_model** out);
 int32_t lc_model_get_config(const lc_model* m, lc_model_config* out);
+
+/* ---- Checkpoint directories (no counterpart in the reference) ----
+ * A folder with config.json and model.safetensors.  The config's "architecture" selects the design from the library's
+ * registry and gives every size and constant; the weights are bf16.  The handle serves the same calls as a GGUF model
+ * (batches, generation, decode loop, sampling), with a paged cache for the layers that attend and one recurrent state per
+ * sequence slot for the layers that do not.  Of `overrides` (may be NULL) these are read: max_seq_len (0 -> 4096), max_seqs,
+ * kv_page_tokens, kv_pool_tokens, device, compute_f32.
+ * lc_model_create_json takes the config's text; the tensors follow through lc_model_set_tensor / lc_model_synth_tensor under
+ * their checkpoint names, then lc_model_finalize. */
+int32_t lc_model_create_json(const char* config_json, const lc_model_config* overrides, lc_model** out);
+int32_t lc_model_load_dir(const char* dir, const lc_model_config* overrides, lc_model** out);
 
 /* ---- Pre-flight checks of a GGUF file: capability report + corruption scan ----
  * lc_scan_blocks / lc_scan_blocks_dev: the per-tensor body of scan_for_corruption (rust/src/model/loader.rs:301-422) on the
@@ -332,6 +345,15 @@ int32_t lc_forward(lc_model* m, const int64_t* tokens, int32_t n, float* logits_
  * greedy token of each sequence (may be NULL). */
 int32_t lc_forward_batch(lc_model* m, int32_t n_seqs, const int32_t* seq_ids, const int64_t* tokens,
                          const int32_t* n_tokens, float* logits_out, int64_t* next_out);
+
+/* lc_forward_batch with a choice of rows: sequence i wants the logits of n_want[i] places (0-based among its tokens of this
+ * call, ascending; possibly none), listed in `want` one sequence after the other.  logits_out is [sum of n_want, vocab],
+ * next_out the greedy picks of the same rows (both may be NULL). */
+int32_t lc_step(lc_model* m, int32_t n_seqs, const int32_t* seq_ids, const int64_t* tokens, const int32_t* n_tokens,
+                const int32_t* n_want, const int32_t* want, float* logits_out, int64_t* next_out);
+/* Admission: a free sequence slot, empty (LC_ERR_KV_FULL when all max_seqs are taken); and its return with everything it holds. */
+int32_t lc_seq_open(lc_model* m, int32_t* seq_id);
+int32_t lc_seq_close(lc_model* m, int32_t seq_id);
 
 /* sampler::sample_top_p (rust/src/inference/sampler.rs:6-50) on the GPU with the uniform draw u in [0, 1) supplied by the
  * caller (the reference's `rng.gen::<f32>()`, :39): logits / temperature, softmax, stable descending sort, the shortest

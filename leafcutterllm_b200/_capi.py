@@ -13,9 +13,10 @@ STATUS_NAMES = {0: "LC_OK", -1: "LC_ERR_INVALID", -2: "LC_ERR_UNSUPPORTED", -3: 
                 -5: "LC_ERR_KV_FULL", -6: "LC_ERR_MISSING", -7: "LC_ERR_STATE"}
 
 TYPE_F32, TYPE_F16, TYPE_Q4_0, TYPE_Q8_0, TYPE_Q4_K, TYPE_Q5_K, TYPE_Q6_K, TYPE_IQ4_NL = 0, 1, 2, 8, 12, 13, 14, 20
+TYPE_BF16 = 30
 # (elements per block, bytes per block): rust/src/model/quant.rs:186-262
 QUANT_GEOMETRY = {TYPE_F32: (1, 4), TYPE_F16: (1, 2), TYPE_Q4_0: (32, 18), TYPE_Q8_0: (32, 34), TYPE_Q4_K: (256, 144),
-                  TYPE_Q5_K: (256, 176), TYPE_Q6_K: (256, 210), TYPE_IQ4_NL: (32, 18)}
+                  TYPE_Q5_K: (256, 176), TYPE_Q6_K: (256, 210), TYPE_IQ4_NL: (32, 18), TYPE_BF16: (1, 2)}
 
 
 class ModelConfig(C.Structure):
@@ -24,7 +25,8 @@ class ModelConfig(C.Structure):
                 ("vocab_size", C.c_int32), ("rope_theta", C.c_float), ("rms_eps", C.c_float),
                 ("kv_dtype", C.c_int32), ("rope_mode", C.c_int32), ("n_experts", C.c_int32), ("top_k", C.c_int32),
                 ("max_seqs", C.c_int32), ("kv_page_tokens", C.c_int32), ("kv_pool_tokens", C.c_int64),
-                ("device", C.c_int32), ("tp_size", C.c_int32), ("tp_rank", C.c_int32), ("reserved", C.c_int32 * 5)]
+                ("device", C.c_int32), ("tp_size", C.c_int32), ("tp_rank", C.c_int32), ("compute_f32", C.c_int32),
+                ("reserved", C.c_int32 * 4)]
 
 
 class Counters(C.Structure):
@@ -99,6 +101,11 @@ SIGNATURES = {
     "lc_model_finalize": (_i32, [_vp]),
     "lc_model_destroy": (_i32, [_vp]),
     "lc_model_load_gguf": (_i32, [C.c_char_p, C.POINTER(ModelConfig), C.POINTER(_vp)]),
+    "lc_model_create_json": (_i32, [C.c_char_p, C.POINTER(ModelConfig), C.POINTER(_vp)]),
+    "lc_model_load_dir": (_i32, [C.c_char_p, C.POINTER(ModelConfig), C.POINTER(_vp)]),
+    "lc_step": (_i32, [_vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
+    "lc_seq_open": (_i32, [_vp, C.POINTER(_i32)]),
+    "lc_seq_close": (_i32, [_vp, _i32]),
     "lc_model_get_config": (_i32, [_vp, C.POINTER(ModelConfig)]),
     "lc_sample_top_p": (_i32, [_vp, _sz, C.c_float, C.c_float, C.c_float, C.POINTER(C.c_int64)]),
     "lc_model_set_seed": (_i32, [_vp, _u64]),

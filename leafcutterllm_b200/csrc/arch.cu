@@ -1,0 +1,225 @@
+// Registry of the checkpoint-directory designs and the loader of such directories: config.json names the design and gives
+// every size and constant, model.safetensors holds the weights (an 8-byte little-endian header length, a JSON header of
+// name -> dtype, shape, data_offsets, then the data).
+#include <cmath>
+#include <cstring>
+#include "lc_arch.h"
+#include "lc_json.h"
+#include "lc_model.h"
+
+namespace lc {
+
+void rotary_frequencies(const RotarySpec& r, std::vector<double>* freq, double* magnitude) {
+    const int n = r.dims / 2;
+    freq->assign((size_t)n, 0.0);
+    *magnitude = 1.0;
+    for (int i = 0; i < n; i++) (*freq)[i] = std::pow(r.base, -2.0 * i / r.dims);
+    if (!r.yarn) return;
+    const double pi = 3.14159265358979323846;
+    auto pair_at = [&](double turns) { return r.dims * std::log(r.original / (2.0 * pi * turns)) / (2.0 * std::log(r.base)); };
+    const double lo = std::fmax(std::floor(pair_at(r.fast)), 0.0), hi = std::fmin(std::ceil(pair_at(r.slow)), r.dims - 1.0);
+    for (int i = 0; i < n; i++) {
+        const double ramp = std::fmin(std::fmax((i - lo) / std::fmax(hi - lo, 0.001), 0.0), 1.0);
+        (*freq)[i] = (*freq)[i] / r.factor * ramp + (*freq)[i] * (1.0 - ramp);
+    }
+    *magnitude = 0.1 * std::log(r.factor) + 1.0;
+}
+
+namespace {
+
+// Typed access to one JSON object; the first problem is kept as the error text.
+struct Fields {
+    const JValue* o;
+    std::string where;
+    const JValue* need(const char* key, JValue::Kind kind) const {
+        const JValue* v = o ? o->get(key) : nullptr;
+        if (!v || v->kind != kind) { set_error("config: %s lacks '%s' or it has the wrong type", where.c_str(), key); return nullptr; }
+        return v;
+    }
+    int32_t integer(const char* key, int* out, int lo) const {
+        const JValue* v = need(key, JValue::NUM);
+        if (!v) return LC_ERR_INVALID;
+        LC_CHECK(v->num == std::floor(v->num) && v->num >= lo && v->num < 2147483648.0, LC_ERR_INVALID, "config: %s: '%s' = %g is out of range", where.c_str(), key, v->num);
+        *out = (int)v->num;
+        return LC_OK;
+    }
+    int32_t real(const char* key, double* out) const {
+        const JValue* v = need(key, JValue::NUM);
+        if (!v) return LC_ERR_INVALID;
+        *out = v->num;
+        return LC_OK;
+    }
+    int32_t real(const char* key, float* out) const {
+        double d = 0;
+        LC_TRY(real(key, &d));
+        *out = (float)d;
+        return LC_OK;
+    }
+    bool has(const char* key) const { const JValue* v = o->get(key); return v && v->kind != JValue::NUL; }
+};
+
+int32_t parse_rotary(const JValue& v, const std::string& where, RotarySpec* out) {
+    Fields f{&v, where + ".rot"};
+    LC_TRY(f.integer("dims", &out->dims, 2));
+    LC_CHECK(out->dims % 2 == 0, LC_ERR_INVALID, "config: %s: an odd number of rotated dimensions", f.where.c_str());
+    LC_TRY(f.real("base", &out->base));
+    if (f.has("scaling")) {
+        const JValue* sv = f.need("scaling", JValue::OBJ);
+        if (!sv) return LC_ERR_INVALID;
+        Fields s{sv, f.where + ".scaling"};
+        out->yarn = true;
+        LC_TRY(s.real("factor", &out->factor));
+        LC_TRY(s.real("original", &out->original));
+        LC_TRY(s.real("fast", &out->fast));
+        LC_TRY(s.real("slow", &out->slow));
+    }
+    return LC_OK;
+}
+
+int32_t parse_layer(const JValue& v, int index, LayerSpec* out) {
+    Fields f{&v, "layer " + std::to_string(index)};
+    const JValue *type = f.need("type", JValue::STR), *mixer = f.need("mixer", JValue::OBJ);
+    if (!type || !mixer) return LC_ERR_INVALID;
+    Fields m{mixer, f.where + ".mixer"};
+    LC_TRY(m.integer("heads", &out->heads, 1));
+    LC_TRY(m.integer("dim", &out->dim, 1));
+    LC_TRY(m.integer("vdim", &out->vdim, 1));
+    if (type->str == "channel_delta") {
+        out->mixer = MixerKind::ChannelDelta;
+        LC_TRY(m.integer("kv_heads", &out->kv_heads, 1));
+        LC_TRY(m.integer("conv", &out->conv_taps, 1));
+        LC_CHECK(out->heads % out->kv_heads == 0, LC_ERR_INVALID, "config: %s: %d heads over %d key heads", m.where.c_str(), out->heads, out->kv_heads);
+    } else if (type->str == "latent_attention") {
+        out->mixer = MixerKind::LatentAttention;
+        LC_TRY(m.integer("kv_rank", &out->kv_rank, 1));
+        LC_TRY(m.integer("rot_dim", &out->rot_dim, 2));
+        if (m.has("q_rank")) LC_TRY(m.integer("q_rank", &out->q_rank, 1));
+        LC_TRY(m.real("scale", &out->scale));
+        const JValue* rot = m.need("rot", JValue::OBJ);
+        if (!rot) return LC_ERR_INVALID;
+        LC_TRY(parse_rotary(*rot, m.where, &out->rot));
+        LC_CHECK(out->rot.dims <= out->rot_dim, LC_ERR_INVALID, "config: %s: %d of %d dimensions rotated", m.where.c_str(), out->rot.dims, out->rot_dim);
+    } else {
+        set_error("config: %s: unknown mixer type '%s'", f.where.c_str(), type->str.c_str());
+        return LC_ERR_UNSUPPORTED;
+    }
+    if (f.has("mlp")) {
+        const JValue* mlp = f.need("mlp", JValue::OBJ);
+        if (!mlp) return LC_ERR_INVALID;
+        Fields p{mlp, f.where + ".mlp"};
+        const JValue* kind = p.need("kind", JValue::STR);
+        if (!kind) return LC_ERR_INVALID;
+        LC_CHECK(kind->str == "dense", LC_ERR_UNSUPPORTED, "config: %s: unknown kind '%s'", p.where.c_str(), kind->str.c_str());
+        out->ffn = FfnKind::Relu2;
+        LC_TRY(p.integer("ff", &out->ff, 1));
+    }
+    return LC_OK;
+}
+
+// Varasun: a free mix of gated-delta-rule layers and latent-attention layers, listed one by one.
+int32_t parse_varasun(const JValue& cfg, ArchSpec* out) {
+    Fields f{&cfg, "the model"};
+    LC_TRY(f.integer("width", &out->width, 1));
+    LC_TRY(f.integer("vocab", &out->vocab, 1));
+    LC_TRY(f.real("logit_scale", &out->logit_scale));
+    LC_TRY(f.real("logit_softcap", &out->logit_softcap));
+    const JValue* norm = f.need("norm", JValue::OBJ);
+    if (!norm) return LC_ERR_INVALID;
+    LC_TRY((Fields{norm, "norm"}.real("eps", &out->eps)));
+    const JValue* layers = f.need("layers", JValue::ARR);
+    if (!layers) return LC_ERR_INVALID;
+    LC_CHECK(!layers->arr.empty(), LC_ERR_INVALID, "config: no layers");
+    for (size_t i = 0; i < layers->arr.size(); i++) {
+        LayerSpec ly;
+        LC_TRY(parse_layer(layers->arr[i], (int)i, &ly));
+        out->layers.push_back(ly);
+    }
+    return LC_OK;
+}
+
+struct ArchEntry { const char* name; int32_t (*parse)(const JValue&, ArchSpec*); };
+const ArchEntry kRegistry[] = {{"Varasun", parse_varasun}};
+
+uint32_t safetensors_type(const std::string& dtype) {
+    if (dtype == "BF16") return LC_TYPE_BF16;
+    if (dtype == "F16") return LC_TYPE_F16;
+    if (dtype == "F32") return LC_TYPE_F32;
+    return ~0u;
+}
+
+int32_t load_safetensors(lc_model* m, const std::string& path) {
+    Mapping file;
+    LC_TRY(file.open_file(path));
+    const uint8_t* base = (const uint8_t*)file.base;
+    LC_CHECK(file.size >= 8, LC_ERR_INVALID, "%s: too short", path.c_str());
+    uint64_t hlen = 0;
+    for (int i = 0; i < 8; i++) hlen |= (uint64_t)base[i] << (8 * i);
+    LC_CHECK(hlen <= file.size - 8, LC_ERR_INVALID, "%s: the header reaches past the end of the file", path.c_str());
+    const std::string text((const char*)base + 8, (size_t)hlen);  // a copy that ends in 0: the reader's number parsing may look one character ahead
+    JReader jr{text.c_str(), text.c_str() + text.size()};
+    const JValue head = jr.value();
+    LC_CHECK(jr.ok && head.kind == JValue::OBJ, LC_ERR_INVALID, "%s: the header is not a JSON object", path.c_str());
+    const uint8_t* data = base + 8 + hlen;
+    const size_t room = file.size - 8 - (size_t)hlen;
+    for (auto& kv : head.obj) {
+        if (kv.first == "__metadata__") continue;
+        const JValue *dtype = kv.second.get("dtype"), *shape = kv.second.get("shape"), *off = kv.second.get("data_offsets");
+        LC_CHECK(dtype && shape && off && shape->kind == JValue::ARR && off->kind == JValue::ARR && off->arr.size() == 2, LC_ERR_INVALID,
+                 "%s: tensor %s has a malformed entry", path.c_str(), kv.first.c_str());
+        const uint32_t typ = safetensors_type(dtype->str);
+        LC_CHECK(typ != ~0u, LC_ERR_UNSUPPORTED, "%s: tensor %s has dtype %s", path.c_str(), kv.first.c_str(), dtype->str.c_str());
+        std::vector<uint64_t> dims;  // fastest first
+        uint64_t count = 1;
+        for (size_t i = shape->arr.size(); i > 0; i--) { dims.push_back((uint64_t)shape->arr[i - 1].num); count *= dims.back(); }
+        if (dims.empty()) dims.push_back(1);
+        LC_CHECK(dims.size() <= 4 && count > 0, LC_ERR_UNSUPPORTED, "%s: tensor %s has an unsupported shape", path.c_str(), kv.first.c_str());
+        const double b = off->arr[0].num, e = off->arr[1].num;
+        LC_CHECK(b >= 0 && e >= b && e <= (double)room && (uint64_t)(e - b) == lc_tensor_bytes(typ, count), LC_ERR_INVALID,
+                 "%s: tensor %s: its offsets do not match its shape or the file", path.c_str(), kv.first.c_str());
+        LC_TRY(lc_model_set_tensor(m, kv.first.c_str(), typ, dims.data(), (int32_t)dims.size(), data + (size_t)b, (size_t)(e - b)));
+    }
+    return LC_OK;
+}
+
+}  // namespace
+
+int32_t arch_from_json(const char* text, size_t len, ArchSpec* out) {
+    const std::string copy(text, len);
+    JReader jr{copy.c_str(), copy.c_str() + copy.size()};
+    const JValue cfg = jr.value();
+    LC_CHECK(jr.ok && cfg.kind == JValue::OBJ, LC_ERR_INVALID, "config: not a JSON object");
+    const JValue* name = cfg.get("architecture");
+    LC_CHECK(name && name->kind == JValue::STR, LC_ERR_INVALID, "config: no 'architecture'");
+    for (const ArchEntry& a : kRegistry)
+        if (name->str == a.name) {
+            out->name = a.name;
+            return a.parse(cfg, out);
+        }
+    set_error("config: architecture '%s' is not known to this library", name->str.c_str());
+    return LC_ERR_UNSUPPORTED;
+}
+
+}  // namespace lc
+
+extern "C" int32_t lc_model_load_dir(const char* dir, const lc_model_config* overrides, lc_model** out) {
+    LC_CHECK(dir && out, LC_ERR_INVALID, "lc_model_load_dir: null argument");
+    *out = nullptr;
+    std::string text;
+    {
+        Mapping cfg;
+        LC_TRY(cfg.open_file(std::string(dir) + "/config.json"));
+        text.assign((const char*)cfg.base, cfg.size);
+    }
+    lc_model* m = nullptr;
+    LC_TRY(lc_model_create_json(text.c_str(), overrides, &m));
+    int32_t st = load_safetensors(m, std::string(dir) + "/model.safetensors");
+    if (st == LC_OK) st = lc_model_finalize(m);
+    if (st != LC_OK) {
+        const std::string keep = get_error();
+        lc_model_destroy(m);
+        set_error("%s", keep.c_str());
+        return st;
+    }
+    *out = m;
+    return LC_OK;
+}

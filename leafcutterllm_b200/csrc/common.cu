@@ -83,6 +83,7 @@ bool quant_geom(uint32_t typ, QuantGeom* g) {
         case LC_TYPE_Q5_K: *g = {256, 176}; return true;
         case LC_TYPE_Q6_K: *g = {256, 210}; return true;
         case LC_TYPE_IQ4_NL: *g = {32, 18}; return true;
+        case LC_TYPE_BF16: *g = {1, 2}; return true;
         default: return false;
     }
 }

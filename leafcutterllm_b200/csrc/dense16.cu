@@ -1,0 +1,361 @@
+// Products over bf16 weight matrices, y[t, r] = sum_k x[t, k] w[r, k], for any number of tokens.
+//
+// bf16 activations: dense_umma_kernel, tcgen05.mma kind::f16 with f32 accumulators in tensor memory.  The WEIGHT rows are the
+// M of the instruction (128 per tile) and the tokens its N (16 .. 256), so the same kernel streams the weights of a
+// one-token decode step at memory speed and multiplies prefill chunks at tensor-core speed:
+//   warp 0   one thread requests TMA boxes of 64 elements of k x 128 weight rows and x N tokens (128-byte swizzle) into a
+//            ring of stages; the first weight boxes leave before the kernel waits for its predecessor;
+//   warp 1   one thread issues the products of a stage (four K = 16 steps) and commits them to the stage's "empty" barrier;
+//   warps 4-7  read finished accumulators (two sets, so the next tile's products overlap), apply the epilogue and store;
+//            lane = weight row, so a warp's store of one token is contiguous.
+// Few tiles: k is cut into shares over several CTAs; each leaves its partial tile in scratch and takes a ticket, the last one
+// adds the shares in share order (the result does not depend on which CTA that is) and runs the epilogue.
+// Work items are dealt round robin to a grid of at most one CTA per SM.  Every wait is bounded: one that runs out raises the
+// library's device error flag and the CTA winds down (copies awaited, tensor memory freed).
+//
+// f32 activations: dense_f32_kernel, plain f32 FMAs (64 x 64 tiles), for models that run in true 32-bit.
+#include <cstdlib>
+#include "lc_mixers.h"
+#include "lc_tma.cuh"
+#include "lc_umma.cuh"
+
+namespace lc {
+
+namespace {
+
+constexpr int kM = 128;          // weight rows per tile
+constexpr int kKB = 64;          // elements of k per stage
+constexpr int kABytes = kM * kKB * 2;
+constexpr int kThreads = 256;
+
+struct DenseParams {
+    void* out;
+    float* partial;
+    unsigned* tickets;
+    int* error_flag;
+    const float *e0, *e1;
+    size_t out_batch;
+    int n, T, ldo, kblocks, mt, nt, batch, shares, items, stages;
+    int out_f32, epi, e_div;
+    float scale, cap;
+};
+
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float dense_epilogue(const DenseParams& p, int row, float y) {
+    switch (p.epi) {
+        case DENSE_RELU2: { const float r = fmaxf(y, 0.0f); return r * r; }
+        case DENSE_LOG_DECAY: return -p.e0[row / p.e_div] * softplus_f(y + p.e1[row]);
+        case DENSE_LOGITS: { const float v = y * p.scale; return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v; }
+        default: return y;
+    }
+}
+// 16 accumulators of weight row `row`, tokens t0 .. t0 + 15
+__device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int row, int t0, const float (&v)[16]) {
+    if (row >= p.n) return;
+    const size_t at = (size_t)b * p.out_batch + (size_t)t0 * p.ldo + row;
+    const int m = min(16, p.T - t0);
+    if (p.out_f32) {
+        float* o = (float*)p.out + at;
+#pragma unroll
+        for (int j = 0; j < 16; j++)
+            if (j < m) o[(size_t)j * p.ldo] = dense_epilogue(p, row, v[j]);
+    } else {
+        __nv_bfloat16* o = (__nv_bfloat16*)p.out + at;
+#pragma unroll
+        for (int j = 0; j < 16; j++)
+            if (j < m) o[(size_t)j * p.ldo] = __float2bfloat16_rn(dense_epilogue(p, row, v[j]));
+    }
+}
+
+template <int NT>
+__global__ void __launch_bounds__(kThreads, 1)
+dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx, const DenseParams p) {
+    constexpr int kBBytes = NT * kKB * 2, kStage = kABytes + kBBytes;
+    constexpr uint32_t kCols = NT < 32 ? 32 : NT;  // tensor-memory columns of one accumulator set
+    constexpr uint32_t kAlloc = 2 * kCols;
+    extern __shared__ unsigned char smem_raw[];
+    unsigned char* smem = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+    uint64_t* full = (uint64_t*)(smem + (size_t)p.stages * kStage);
+    uint64_t *empty = full + p.stages, *acc_full = empty + p.stages, *acc_empty = acc_full + 2;
+    uint32_t* tmem_slot = (uint32_t*)(acc_empty + 2);
+    volatile int* stop = (volatile int*)(tmem_slot + 1);
+    unsigned* last_share = (unsigned*)(tmem_slot + 2);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < p.stages; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], 1); }
+        for (int i = 0; i < 2; i++) { mbar_init(&acc_full[i], 1); mbar_init(&acc_empty[i], 128); }
+        *stop = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    }
+    if (warp == 2) tmem_alloc(tmem_slot, kAlloc);
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = *tmem_slot;
+    pdl_launch_dependents();
+
+    // item -> (weight tile fastest over shares, then token tiles): consecutive CTAs share a weight tile's rows
+    struct Item { int b, m, n, share, k0, k1; };
+    auto item_of = [&](int it) {
+        Item r;
+        r.share = it % p.shares; it /= p.shares;
+        r.n = it % p.nt; it /= p.nt;
+        r.m = it % p.mt; r.b = it / p.mt;
+        r.k0 = (int)((long long)p.kblocks * r.share / p.shares);
+        r.k1 = (int)((long long)p.kblocks * (r.share + 1) / p.shares);
+        return r;
+    };
+    if (warp == 0 && lane == 0) {
+        int issued = 0;
+        bool ok = true;
+        // weight boxes of the first stages, before the activations exist
+        int pre = 0;
+        {
+            const Item r = item_of(blockIdx.x);
+            for (; pre < p.stages && r.k0 + pre < r.k1; pre++) {
+                mbar_expect_tx(&full[pre], kStage);
+                tma_load_3d(smem + (size_t)pre * kStage, &tw, (r.k0 + pre) * kKB, r.m * kM, r.b, &full[pre]);
+            }
+        }
+        pdl_wait();
+        for (int it = blockIdx.x; it < p.items && ok; it += gridDim.x) {
+            const Item r = item_of(it);
+            for (int kb = r.k0; kb < r.k1; kb++) {
+                const int st = issued % p.stages, round = issued / p.stages;
+                unsigned char* a = smem + (size_t)st * kStage;
+                if (issued >= pre) {
+                    if (round > 0 && !mbar_wait(&empty[st], (uint32_t)(round - 1) & 1)) { ok = false; break; }
+                    mbar_expect_tx(&full[st], kStage);
+                    tma_load_3d(a, &tw, kb * kKB, r.m * kM, r.b, &full[st]);
+                }
+                tma_load_3d(a + kABytes, &tx, kb * kKB, r.b, r.n * NT, &full[st]);
+                issued++;
+                if (*stop) { ok = false; break; }
+            }
+        }
+        if (!ok) {
+            *stop = 1;
+            atomicExch(p.error_flag, 11);
+            for (int i = max(0, issued - p.stages); i < issued; i++) mbar_wait(&full[i % p.stages], (uint32_t)(i / p.stages) & 1);
+        }
+    } else if (warp == 1 && lane == 0) {
+        const uint32_t idesc = idesc_bf16(kM, NT);
+        int used = 0, tile = 0;
+        bool ok = true;
+        for (int it = blockIdx.x; it < p.items && ok; it += gridDim.x, tile++) {
+            const Item r = item_of(it);
+            const int set = tile & 1;
+            if (tile >= 2 && !mbar_wait(&acc_empty[set], (uint32_t)(tile / 2 - 1) & 1)) { ok = false; break; }
+            tc_fence_after();
+            for (int kb = r.k0; kb < r.k1; kb++, used++) {
+                const int st = used % p.stages;
+                if (!mbar_wait(&full[st], (uint32_t)(used / p.stages) & 1)) { ok = false; break; }
+                tc_fence_after();
+                const uint32_t a = smem_u32(smem + (size_t)st * kStage);
+                const uint64_t da = umma_desc_sw128(a), db = umma_desc_sw128(a + kABytes);
+#pragma unroll
+                for (int k = 0; k < 4; k++) umma_f16_ss(tmem + (uint32_t)set * kCols, da + 2 * k, db + 2 * k, idesc, kb > r.k0 || k > 0);
+                umma_commit(&empty[st]);
+            }
+            if (ok) umma_commit(&acc_full[set]);
+        }
+        if (!ok) { *stop = 1; atomicExch(p.error_flag, 12); }
+    } else if (warp >= 4) {
+        pdl_wait();  // earlier kernels may still read what this one overwrites
+        const int ew = warp - 4, row_in = ew * 32 + lane;
+        int tile = 0;
+        for (int it = blockIdx.x; it < p.items; it += gridDim.x, tile++) {
+            const Item r = item_of(it);
+            const int set = tile & 1;
+            if (!mbar_wait(&acc_full[set], (uint32_t)(tile / 2) & 1)) { *stop = 1; if (lane == 0) atomicExch(p.error_flag, 13); break; }
+            tc_fence_after();
+            const uint32_t base = tmem + (uint32_t)set * kCols + ((uint32_t)(ew * 32) << 16);
+            const int row = r.m * kM + row_in, t0 = r.n * NT;
+            const size_t plane = (size_t)NT * kM;
+            const int cell = (r.b * p.mt + r.m) * p.nt + r.n;
+            float* part = p.shares > 1 ? p.partial + (size_t)cell * p.shares * plane : nullptr;
+#pragma unroll 1
+            for (int c = 0; c < NT; c += 16) {
+                if (t0 + c >= p.T) break;
+                uint32_t raw[16];
+                tmem_ld16(base + c, raw);
+                asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                float v[16];
+#pragma unroll
+                for (int j = 0; j < 16; j++) v[j] = __uint_as_float(raw[j]);
+                if (part) {
+#pragma unroll
+                    for (int j = 0; j < 16; j++) part[(size_t)r.share * plane + (size_t)(c + j) * kM + row_in] = v[j];
+                } else {
+                    dense_store16(p, r.b, row, t0 + c, v);
+                }
+            }
+            tc_fence_before();
+            mbar_arrive(&acc_empty[set]);
+            if (part) {
+                __threadfence();
+                asm volatile("bar.sync 1, 128;" ::: "memory");
+                if (threadIdx.x == 128) {
+                    const unsigned t = atomicAdd(&p.tickets[cell], 1u);
+                    *last_share = t == (unsigned)(p.shares - 1);
+                    if (*last_share) p.tickets[cell] = 0;
+                    __threadfence();
+                }
+                asm volatile("bar.sync 1, 128;" ::: "memory");
+                const bool mine = *last_share != 0;
+                asm volatile("bar.sync 1, 128;" ::: "memory");
+                if (mine) {
+#pragma unroll 1
+                    for (int c = 0; c < NT; c += 16) {
+                        if (t0 + c >= p.T) break;
+                        float v[16];
+#pragma unroll
+                        for (int j = 0; j < 16; j++) v[j] = 0.0f;
+                        for (int sh = 0; sh < p.shares; sh++)
+#pragma unroll
+                            for (int j = 0; j < 16; j++) v[j] += __ldcg(part + (size_t)sh * plane + (size_t)(c + j) * kM + row_in);
+                        dense_store16(p, r.b, row, t0 + c, v);
+                    }
+                }
+            }
+        }
+    } else {
+        pdl_wait();
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    if (warp == 2) tmem_free(tmem, kAlloc);
+}
+
+// True 32-bit: 64 weight rows x 64 tokens per CTA, 4 x 4 outputs per thread.
+__global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __restrict__ w, int ldw, size_t w_batch, const float* __restrict__ x, int ldx,
+                                                        size_t x_batch, int k, const DenseParams p) {
+    constexpr int KT = 16;
+    __shared__ float ws[KT][64 + 4], xs[KT][64 + 4];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r0 = blockIdx.x * 64, t0 = blockIdx.y * 64, b = blockIdx.z;
+    w += (size_t)b * w_batch;
+    x += (size_t)b * x_batch;
+    const int tr = threadIdx.x & 15, tt = threadIdx.x >> 4;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < k; k0 += KT) {
+        for (int i = threadIdx.x; i < 64 * KT; i += 256) {
+            const int r = i / KT, c = i % KT, kk = k0 + c;
+            ws[c][r] = (r0 + r < p.n && kk < k) ? __bfloat162float(w[(size_t)(r0 + r) * ldw + kk]) : 0.0f;
+            xs[c][r] = (t0 + r < p.T && kk < k) ? x[(size_t)(t0 + r) * ldx + kk] : 0.0f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int c = 0; c < KT; c++) {
+            float a[4], q[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) { a[i] = ws[c][tr + 16 * i]; q[i] = xs[c][tt + 16 * i]; }
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(q[i], a[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int t = t0 + tt + 16 * i;
+        if (t >= p.T) continue;
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int row = r0 + tr + 16 * j;
+            if (row < p.n) ((float*)p.out)[(size_t)b * p.out_batch + (size_t)t * p.ldo + row] = dense_epilogue(p, row, acc[i][j]);
+        }
+    }
+}
+
+template <int NT>
+int32_t launch_umma(const DenseArgs& a, const CUtensorMap& tx, DenseParams p, cudaStream_t s) {
+    const size_t stage = kABytes + (size_t)NT * kKB * 2, fixed = 1024 + 512;
+    p.stages = (int)std::min<size_t>(12, (kMaxSmem - fixed) / stage);
+    const size_t smem = fixed + (size_t)p.stages * stage;
+    LC_CUDA(ensure_smem_limit((const void*)dense_umma_kernel<NT>, smem));
+    const int grid = std::min(p.items, sm_count());
+    LC_CUDA(launch_pdl(dense_umma_kernel<NT>, dim3((unsigned)grid), dim3(kThreads), smem, s, *(const CUtensorMap*)a.w->tmap, tx, p));
+    return LC_OK;
+}
+
+constexpr size_t kPartialBytes = (size_t)64 << 20;
+constexpr int kMaxTickets = 4096;
+
+}  // namespace
+
+int32_t dense_weight_init(DenseWeight* w, const __nv_bfloat16* data, int n, int k, int ld, int batch, size_t batch_stride) {
+    w->data = data; w->n = n; w->k = k; w->ld = ld; w->batch = batch; w->batch_stride = batch_stride;
+    LC_CHECK(n > 0 && k > 0 && ld >= k && ld % 8 == 0 && batch >= 1 && batch_stride % 8 == 0 && (uintptr_t)data % 16 == 0, LC_ERR_INVALID,
+             "dense weight [%d x %d], rows %d apart: layout", n, k, ld);
+    w->has_tmap = make_bf16_tmap_3d(w->tmap, data, (uint64_t)k, (uint64_t)n, (uint64_t)batch, (uint64_t)ld, batch > 1 ? batch_stride : (uint64_t)ld * n, kKB, kM, 1);
+    LC_CHECK(w->has_tmap, LC_ERR_CUDA, "dense weight [%d x %d]: no tensor map", n, k);
+    return LC_OK;
+}
+
+int32_t dense_workspace_alloc(DenseWorkspace* ws) {
+    LC_CUDA(cudaMalloc((void**)&ws->partial, kPartialBytes));
+    ws->partial_bytes = kPartialBytes;
+    LC_CUDA(cudaMalloc((void**)&ws->tickets, kMaxTickets * sizeof(unsigned)));
+    LC_CUDA(cudaMemset(ws->tickets, 0, kMaxTickets * sizeof(unsigned)));
+    ws->max_tickets = kMaxTickets;
+    return LC_OK;
+}
+void dense_workspace_free(DenseWorkspace* ws) {
+    if (ws->partial) cudaFree(ws->partial);
+    if (ws->tickets) cudaFree(ws->tickets);
+    ws->partial = nullptr;
+    ws->tickets = nullptr;
+    ws->maps.clear();
+}
+
+int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
+    if (a.T <= 0) return LC_OK;
+    const DenseWeight& w = *a.w;
+    DenseParams p{};
+    p.out = a.out; p.e0 = a.e0; p.e1 = a.e1; p.out_batch = a.out_batch;
+    p.n = w.n; p.T = a.T; p.ldo = a.ldo; p.batch = w.batch;
+    p.out_f32 = a.out_f32 || a.f32; p.epi = a.epi; p.e_div = a.e_div; p.scale = a.scale; p.cap = a.cap;
+    p.error_flag = gemv_error_flag_dev();
+    if (a.f32) {
+        LC_CUDA(launch_pdl(dense_f32_kernel, dim3((unsigned)((w.n + 63) / 64), (unsigned)((a.T + 63) / 64), (unsigned)w.batch), dim3(256), 0, s, w.data,
+                           w.ld, w.batch_stride, (const float*)a.x, a.ldx, a.x_batch, w.k, p));
+        return LC_OK;
+    }
+    const int NT = a.T <= 16 ? 16 : a.T <= 32 ? 32 : a.T <= 64 ? 64 : a.T <= 128 ? 128 : 256;
+    p.kblocks = (w.k + kKB - 1) / kKB;
+    p.mt = (w.n + kM - 1) / kM;
+    p.nt = (a.T + NT - 1) / NT;
+    const int cells = p.mt * p.nt * w.batch, sms = sm_count();
+    p.shares = 1;
+    if (cells * 4 < sms * 3 && cells <= ws.max_tickets) {  // fewer tiles than three quarters of the SMs: cut k
+        p.shares = std::max(1, std::min(std::min(p.kblocks / 2, 16), sms / cells));
+        while (p.shares > 1 && (size_t)cells * p.shares * NT * kM * sizeof(float) > ws.partial_bytes) p.shares--;
+    }
+    p.items = cells * p.shares;
+    p.partial = ws.partial; p.tickets = ws.tickets;
+    LC_CHECK((uintptr_t)a.x % 16 == 0 && a.ldx % 8 == 0 && a.x_batch % 8 == 0 && a.x_rows >= a.T, LC_ERR_INVALID, "dense product: activation layout");
+    const std::vector<uint64_t> key = {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_batch, (uint64_t)w.batch, (uint64_t)a.x_rows, (uint64_t)NT};
+    std::unique_ptr<DenseWorkspace::Map>& mp = ws.maps[key];
+    if (!mp) {
+        mp.reset(new DenseWorkspace::Map);
+        // order (k, matrix, token): a token tile is one box
+        const bool ok = make_bf16_tmap_3d(mp->b, a.x, (uint64_t)w.k, (uint64_t)w.batch, (uint64_t)a.x_rows, w.batch > 1 ? a.x_batch : (uint64_t)a.ldx, (uint64_t)a.ldx, kKB, 1, (uint32_t)NT);
+        if (!ok) ws.maps.erase(key);
+        LC_CHECK(ok, LC_ERR_CUDA, "dense product: no tensor map over the activations");
+    }
+    const CUtensorMap& tx = *(const CUtensorMap*)mp->b;
+    switch (NT) {
+        case 16: return launch_umma<16>(a, tx, p, s);
+        case 32: return launch_umma<32>(a, tx, p, s);
+        case 64: return launch_umma<64>(a, tx, p, s);
+        case 128: return launch_umma<128>(a, tx, p, s);
+        default: return launch_umma<256>(a, tx, p, s);
+    }
+}
+
+}  // namespace lc

@@ -14,131 +14,11 @@
 #include <map>
 #include <string>
 #include <vector>
-#include "lc_kernels.h"
+#include "lc_model.h"
 #include "lc_synth.h"
 #include "lc_tma.cuh"
 
 using namespace lc;
-
-namespace {
-
-struct DevTensor {
-    uint32_t typ = 0;
-    std::vector<uint64_t> dims;
-    void* dev = nullptr;   // owning pointer (null when the bytes live inside a fused buffer)
-    void* view = nullptr;  // where the bytes are
-    size_t nbytes = 0;
-    size_t rows = 0, cols = 0;
-};
-
-struct LayerW {
-    QWeight qkv, o, gate, up, down;
-    QWeight q, k, v;  // used when the three cannot be fused
-    bool fused_qkv = false;
-    const float* attn_norm = nullptr;
-    const float* ffn_norm = nullptr;
-    void* fused_buf = nullptr;
-    // mixture-of-experts FFN (no counterpart in the reference): f32 router [n_experts, H], the experts' three matrices,
-    // and -- when every expert is Q4_K with a tensor map -- device arrays of those maps for the one-launch grouped product
-    const float* router = nullptr;
-    std::vector<QWeight> egate, eup, edown;
-    void *tm_gate = nullptr, *tm_up = nullptr, *tm_down = nullptr;
-    bool grouped_ok = false;
-};
-
-constexpr int kPrefillChunk = 512;
-constexpr int kTokTile = 8;
-constexpr int kMoeGroupedTokens = 64;  // calls of at most this many tokens run the experts as one grouped launch
-
-}  // namespace
-
-struct lc_model {
-    lc_model_config cfg{};
-    int device = 0;
-    cudaStream_t stream = nullptr;
-    std::map<std::string, DevTensor> tensors;
-    bool finalized = false;
-    std::vector<LayerW> layers;
-    QWeight head;
-    const DevTensor* embed = nullptr;
-    const float* final_norm = nullptr;
-    std::vector<void*> owned;  // f32 copies of norm gains etc.
-
-    // geometry: H, L, hd are the model's; nh, nkv, F, V, nqkv are THIS RANK'S part when the model is cut across ranks
-    // (tp > 1: heads, kv heads, FFN rows and vocabulary rows divided by tp; experts e0 .. e0 + El - 1 of a mixture layer)
-    int H = 0, L = 0, nh = 0, nkv = 0, hd = 0, F = 0, V = 0, nqkv = 0;
-    int tp = 1, rank = 0, v0 = 0, e0 = 0, El = 0;
-    bool use_dist = false;               // the ranks are other processes (lc_dist_init); else members lists them, or tp == 1
-    std::vector<lc_model*> members;      // rank 0 of an in-process group: every rank's handle in rank order (itself first)
-    lc_model* leader = nullptr;          // a rank > 0 of such a group
-    float* d_part = nullptr;             // where the column-cut products leave their partial rows for the sum over the ranks
-    long long* d_key = nullptr;          // greedy pick of the local vocabulary slice as (total-order key << 32 | global index)
-    long long* d_key_max = nullptr;
-    float* d_logits_all = nullptr;       // dist: the ranks' logit slices gathered for the host
-    PrefillTile* d_tiles = nullptr;      // the call's tokens as runs of up to 64 consecutive positions of one sequence
-    int n_tiles = 0;
-    float* pending_dst = nullptr;        // where the next sum over the ranks has to land
-    bool pending_pushed = false;         // ... and whether the product already sent its rows to the ranks
-    GemvPush push_desc;
-    int page_tokens = 16, pages_per_seq = 0, pages_total = 0, max_seqs = 1, t_cap = 0;
-    size_t kv_elt = 2;
-
-    // KV cache
-    std::vector<void*> k_pools, v_pools;  // per layer
-    struct alignas(64) TmapBytes { unsigned char b[128]; };
-    std::vector<TmapBytes> k_tmaps, v_tmaps;  // per layer: tensor maps over the key and value pools (f16 pools of 128-dim heads)
-    bool k_tmaps_ok = false;
-    std::vector<int> free_pages;
-    std::vector<std::vector<int>> seq_pages;
-    std::vector<int> seq_len;
-    int32_t* d_page_table = nullptr;
-    std::vector<int32_t> h_page_table;
-    bool page_table_dirty = true;
-
-    // step buffers
-    int64_t* d_tokens = nullptr;
-    int32_t *d_tok_seq = nullptr, *d_tok_pos = nullptr, *d_tok_rope = nullptr, *d_last_idx = nullptr;
-    float *d_hidden = nullptr, *d_hidden2 = nullptr, *d_qkv = nullptr, *d_attn = nullptr, *d_ffn = nullptr;
-    float *d_last = nullptr, *d_logits = nullptr;
-    bool seeded = false;          // lc_model_set_seed: stochastic sampling allowed, draws from seeded_uniform(seed, draws++)
-    uint64_t seed = 0, draws = 0;
-    int64_t* d_next = nullptr;
-    int64_t* d_out_tokens = nullptr;
-    size_t out_tokens_cap = 0;
-    int32_t* d_step_ctr = nullptr;
-    unsigned long long* d_stream_slots = nullptr;  // cross-CTA merge slots of the single-token attention kernel (zero between launches)
-    // mixture-of-experts scratch: the router's picks and weights per token, per-expert slot counts and lists, the slots'
-    // FFN hidden rows and outputs (calls of up to kMoeGroupedTokens tokens), every expert's output plane (larger calls)
-    int32_t *d_moe_sel = nullptr, *d_moe_cnt = nullptr, *d_moe_lists = nullptr;
-    float *d_moe_w = nullptr, *d_moe_h = nullptr, *d_moe_y = nullptr, *d_moe_yall = nullptr;
-    GemvPlanes moe_planes_x, moe_planes_h;  // fixed-point activations of the grouped launches: the layer's input per token, the experts' hidden rows per slot
-    unsigned long long* d_moe_touched = nullptr;  // experts that received a token, summed over layers and steps since the last read
-    uint64_t expert_bytes_each = 0, expert_bytes_all = 0;
-    double touched_per_step = 0.0;
-    void* d_attn_scratch = nullptr;
-    GemmWorkspace gemm_ws;  // f16 activation halves for the many-token tensor-core product
-    bool any_unfused_qkv = false;  // some layer's q/k/v differ in type
-    float* d_qkv_parts = nullptr;  // then: [T][nq] | [T][nkv hd] | [T][nkv hd] before they are interleaved into d_qkv
-    int* d_attn_counters = nullptr;
-    size_t attn_scratch_bytes = 0;
-    unsigned long long* d_sanity = nullptr;
-
-    std::map<int, cudaGraphExec_t> decode_graphs;
-    int graph_nodes = 0;
-    cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-
-    lc_counters ctr{};
-    uint64_t launches_in_call = 0;
-
-    // What the device-side per-token metadata currently describes (a decode step for these sequences at
-    // these cache positions), so that consecutive one-token calls only have to send the token ids.
-    bool meta_valid = false;
-    std::vector<int> meta_seqs, meta_pos;
-    // pinned staging for the per-step host <-> device traffic
-    int64_t* pin_tokens = nullptr;
-    int64_t* pin_next = nullptr;
-    float* pin_logits = nullptr;
-};
 
 namespace {
 
@@ -204,28 +84,6 @@ int32_t shard_plan(const lc_model_config& c, int tp, int rank, const std::string
         pl.kind = SHARD_COLS; pl.count = dims[0] / tp; pl.first = pl.count * rank;
     }
     *out = pl;
-    return LC_OK;
-}
-
-struct DeviceGuard {
-    int prev = 0;
-    bool ok = false;
-    explicit DeviceGuard(int dev) {
-        if (cudaGetDevice(&prev) == cudaSuccess && cudaSetDevice(dev) == cudaSuccess) ok = true;
-    }
-    ~DeviceGuard() { if (ok) cudaSetDevice(prev); }
-};
-
-template <typename T>
-int32_t dalloc(T** p, size_t count) {
-    void* q = nullptr;
-    cudaError_t e = cudaMalloc(&q, std::max<size_t>(count * sizeof(T), 16));
-    if (e != cudaSuccess) {
-        (void)cudaGetLastError();
-        set_error("device allocation of %zu bytes failed: %s", count * sizeof(T), cudaGetErrorString(e));
-        return LC_ERR_OOM;
-    }
-    *p = (T*)q;
     return LC_OK;
 }
 
@@ -519,6 +377,7 @@ int32_t reduce_ranks(lc_model* lead, size_t count) {
 
 // The transformer layers (engine.rs:95-116) on T tokens described by d_tokens / d_tok_*, for every rank of the model.
 int32_t run_layers(lc_model* lead, int T, bool decode_step) {
+    if (lead->stack) return stack_run_layers(lead, T, decode_step);
     std::vector<lc_model*> R = ranks_of(lead);
     for (lc_model* m : R) {
         LC_TRY(launch_embed(m->embed->typ, m->embed->view, m->embed->rows, m->embed->cols, m->d_tokens, T, m->d_hidden, m->stream));
@@ -537,8 +396,13 @@ int32_t run_layers(lc_model* lead, int T, bool decode_step) {
 // Engine::forward (engine.rs:78-132): layers, then final norm + head on n_last rows.  identity_last:
 // every token is the last of its sequence (a decode step), so no gather is needed; otherwise the rows
 // listed in d_last_idx are gathered.  Logits (of this rank's vocabulary rows) land in d_logits rows row0.., greedy picks in d_next.
-int32_t forward_tokens(lc_model* lead, int T, int n_last, bool identity_last, int row0) {
-    LC_TRY(run_layers(lead, T, identity_last));
+int32_t head_tokens(lc_model* lead, int n_last, bool identity_last, int row0) {
+    if (lead->stack) {
+        LC_TRY(stack_head(lead, n_last, identity_last ? nullptr : lead->d_last_idx, lead->d_logits + (size_t)row0 * lead->V));
+        LC_TRY(launch_argmax(lead->d_logits + (size_t)row0 * lead->V, lead->V, n_last, lead->d_next + row0, lead->stream));
+        lead->launches_in_call += 1;
+        return LC_OK;
+    }
     std::vector<lc_model*> R = ranks_of(lead);
     for (lc_model* m : R) {
         const float* last = m->d_hidden;
@@ -577,15 +441,24 @@ int32_t forward_tokens(lc_model* lead, int T, int n_last, bool identity_last, in
     return LC_OK;
 }
 
+int32_t forward_tokens(lc_model* lead, int T, int n_last, bool identity_last, int row0) {
+    LC_TRY(run_layers(lead, T, identity_last));
+    return head_tokens(lead, n_last, identity_last, row0);
+}
+
 uint64_t algo_bytes_step(const lc_model* m, const std::vector<int>& ctx_lens) {
     uint64_t b = m->ctr.weight_bytes;  // every matrix and gain once
     if (m->cfg.n_experts > 0)          // ... but only the experts that received a token (average per layer of the last steps)
         b = b - m->expert_bytes_all + (uint64_t)(m->touched_per_step * (double)m->expert_bytes_each);
     // the embedding table is not streamed: one row per token instead
     if (m->embed) {
-        bool tied = m->tensors.find("output.weight") == m->tensors.end();
+        bool tied = !m->stack && m->tensors.find("output.weight") == m->tensors.end();
         if (!tied) b -= m->embed->nbytes;
         b += (uint64_t)ctx_lens.size() * (m->embed->nbytes / std::max<size_t>(m->embed->rows, 1));
+    }
+    if (m->stack) {  // latents of the context read, one token's written; recurrent state read and written
+        for (int c : ctx_lens) b += m->stack->cache_bytes_per_token * ((uint64_t)c + 1) + 2 * m->stack->state_bytes_per_seq;
+        return b;
     }
     uint64_t per_tok = (uint64_t)m->L * 2 * m->nkv * m->hd * m->kv_elt;
     for (int c : ctx_lens) b += per_tok * (uint64_t)c + per_tok;  // read the context, write one token
@@ -607,6 +480,16 @@ int32_t upload_meta(lc_model* m, const std::vector<int64_t>& tok, const std::vec
         if (tiles.empty() || tiles.back().n == 64 || seq[i] != seq[i - 1] || pos[i] != pos[i - 1] + 1) tiles.push_back(PrefillTile{(int32_t)i, 0, seq[i], pos[i]});
         tiles.back().n++;
     }
+    if (m->stack) {  // the same runs uncut
+        std::vector<SeqRun> runs;
+        for (size_t i = 0; i < T; i++) {
+            if (runs.empty() || seq[i] != seq[i - 1] || pos[i] != pos[i - 1] + 1) runs.push_back(SeqRun{(int32_t)i, 0, seq[i], pos[i]});
+            runs.back().n++;
+        }
+        m->stack->n_runs = (int)runs.size();
+        LC_CUDA(cudaMemcpyAsync(m->stack->d_runs, runs.data(), runs.size() * sizeof(SeqRun), cudaMemcpyHostToDevice, m->stream));
+        LC_CUDA(cudaStreamSynchronize(m->stream));
+    }
     m->n_tiles = (int)tiles.size();
     if (!tiles.empty()) LC_CUDA(cudaMemcpyAsync(m->d_tiles, tiles.data(), tiles.size() * sizeof(PrefillTile), cudaMemcpyHostToDevice, m->stream));
     // the copies read pageable host vectors that die with the caller's frame
@@ -626,13 +509,13 @@ void finish_call(lc_model* m) {
 // round trip of its own; flag_result() looks at what arrived.
 static int32_t queue_flag_read(lc_model* m) {
     int* f = gemv_error_flag_dev();
-    int* dst = reinterpret_cast<int*>(m->pin_next + m->max_seqs);
+    int* dst = reinterpret_cast<int*>(m->pin_next + m->head_rows);
     *dst = 0;
     if (f) LC_CUDA(cudaMemcpyAsync(dst, f, sizeof(int), cudaMemcpyDeviceToHost, m->stream));
     return LC_OK;
 }
 static int32_t flag_result(lc_model* m) {
-    const int v = *reinterpret_cast<const int*>(m->pin_next + m->max_seqs);
+    const int v = *reinterpret_cast<const int*>(m->pin_next + m->head_rows);
     if (v != 0) {
         cudaMemsetAsync(gemv_error_flag_dev(), 0, sizeof(int), m->stream);
         set_error("a device-side check failed (code %d: %s); the results of this call are not valid", v,
@@ -664,19 +547,8 @@ static int32_t reserve_out_tokens(lc_model* m, size_t need);
 static int32_t stage_decode_meta(lc_model* m, int n_seqs, const int32_t* seq_ids, const int64_t* toks);
 static void after_decode_steps(lc_model* m, int n_seqs, const int32_t* seq_ids, int steps);
 
-int32_t lc_model_create(const lc_model_config* cfg, lc_model** out) {
-    LC_CHECK(cfg && out, LC_ERR_INVALID, "lc_model_create: null argument");
-    LC_CHECK(cfg->hidden_size > 0 && cfg->num_layers > 0 && cfg->num_heads > 0 && cfg->num_kv_heads > 0 &&
-                 cfg->intermediate_size > 0 && cfg->vocab_size > 0 && cfg->max_seq_len > 0,
-             LC_ERR_INVALID, "lc_model_create: non-positive dimension");
-    LC_CHECK(cfg->hidden_size % cfg->num_heads == 0, LC_ERR_INVALID, "hidden_size %d is not a multiple of num_heads %d",
-             cfg->hidden_size, cfg->num_heads);
-    LC_CHECK(cfg->num_heads % cfg->num_kv_heads == 0, LC_ERR_INVALID, "num_heads %d is not a multiple of num_kv_heads %d",
-             cfg->num_heads, cfg->num_kv_heads);
-    LC_CHECK(cfg->n_experts >= 0 && cfg->n_experts <= kMaxExperts, LC_ERR_INVALID, "n_experts %d outside 0..%d", cfg->n_experts, kMaxExperts);
-    if (cfg->n_experts > 0)
-        LC_CHECK(cfg->top_k >= 1 && cfg->top_k <= kMaxTopK && cfg->top_k <= cfg->n_experts, LC_ERR_INVALID,
-                 "top_k %d outside 1..min(%d, n_experts = %d)", cfg->top_k, kMaxTopK, cfg->n_experts);
+// A handle from a checked config; `stack` set: its layers are those of a checkpoint-directory design.
+static int32_t create_handle(const lc_model_config* cfg, std::unique_ptr<LayerStack> stack, lc_model** out) {
     if (!have_device()) return LC_ERR_CUDA;
     LC_CHECK(cfg->device >= 0 && cfg->device < lc_device_count(), LC_ERR_INVALID, "device %d not present", cfg->device);
     DeviceGuard dg(cfg->device);
@@ -700,6 +572,7 @@ int32_t lc_model_create(const lc_model_config* cfg, lc_model** out) {
     m->tp = tp; m->rank = rk;
     m->cfg.tp_size = tp; m->cfg.tp_rank = rk;
     m->use_dist = tp > 1 && dist_active() && dist_world() == tp && dist_rank() == rk;
+    m->stack = std::move(stack);
     m->H = cfg->hidden_size; m->L = cfg->num_layers; m->nh = cfg->num_heads / tp; m->nkv = cfg->num_kv_heads / tp;
     m->hd = m->H / cfg->num_heads; m->F = experts ? cfg->intermediate_size : cfg->intermediate_size / tp; m->V = cfg->vocab_size / tp;
     m->v0 = m->V * rk;
@@ -711,11 +584,47 @@ int32_t lc_model_create(const lc_model_config* cfg, lc_model** out) {
     int64_t pool = m->cfg.kv_pool_tokens > 0 ? m->cfg.kv_pool_tokens : (int64_t)m->max_seqs * m->pages_per_seq * m->page_tokens;
     m->pages_total = (int)((pool + m->page_tokens - 1) / m->page_tokens);
     m->kv_elt = m->cfg.kv_dtype ? 4 : 2;
-    m->t_cap = std::max(kPrefillChunk, m->max_seqs);
+    m->t_cap = std::max(m->stack ? kStackChunk : kPrefillChunk, m->max_seqs);
+    m->head_rows = std::max(16, m->max_seqs);
+    m->seq_open.assign(m->max_seqs, 0);
     m->stream = lc::stream();
     if (!m->stream) { delete m; set_error("could not create a CUDA stream"); return LC_ERR_CUDA; }
     *out = m;
     return LC_OK;
+}
+
+int32_t lc_model_create(const lc_model_config* cfg, lc_model** out) {
+    LC_CHECK(cfg && out, LC_ERR_INVALID, "lc_model_create: null argument");
+    LC_CHECK(cfg->hidden_size > 0 && cfg->num_layers > 0 && cfg->num_heads > 0 && cfg->num_kv_heads > 0 &&
+                 cfg->intermediate_size > 0 && cfg->vocab_size > 0 && cfg->max_seq_len > 0,
+             LC_ERR_INVALID, "lc_model_create: non-positive dimension");
+    LC_CHECK(cfg->hidden_size % cfg->num_heads == 0, LC_ERR_INVALID, "hidden_size %d is not a multiple of num_heads %d",
+             cfg->hidden_size, cfg->num_heads);
+    LC_CHECK(cfg->num_heads % cfg->num_kv_heads == 0, LC_ERR_INVALID, "num_heads %d is not a multiple of num_kv_heads %d",
+             cfg->num_heads, cfg->num_kv_heads);
+    LC_CHECK(cfg->n_experts >= 0 && cfg->n_experts <= kMaxExperts, LC_ERR_INVALID, "n_experts %d outside 0..%d", cfg->n_experts, kMaxExperts);
+    if (cfg->n_experts > 0)
+        LC_CHECK(cfg->top_k >= 1 && cfg->top_k <= kMaxTopK && cfg->top_k <= cfg->n_experts, LC_ERR_INVALID,
+                 "top_k %d outside 1..min(%d, n_experts = %d)", cfg->top_k, kMaxTopK, cfg->n_experts);
+    return create_handle(cfg, nullptr, out);
+}
+
+int32_t lc_model_create_json(const char* config_json, const lc_model_config* overrides, lc_model** out) {
+    LC_CHECK(config_json && out, LC_ERR_INVALID, "lc_model_create_json: null argument");
+    std::unique_ptr<LayerStack> stack(new LayerStack);
+    LC_TRY(arch_from_json(config_json, strlen(config_json), &stack->spec));
+    lc_model_config c{};
+    if (overrides) c = *overrides;
+    LC_CHECK(c.tp_size <= 1 && !dist_active(), LC_ERR_UNSUPPORTED, "%s: models of this design are not cut across ranks", stack->spec.name.c_str());
+    c.tp_size = 1; c.tp_rank = 0;
+    c.hidden_size = stack->spec.width; c.vocab_size = stack->spec.vocab; c.num_layers = (int32_t)stack->spec.layers.size();
+    c.rms_eps = stack->spec.eps; c.rope_mode = 1; c.n_experts = 0; c.top_k = 0;
+    c.num_heads = c.num_kv_heads = 1; c.intermediate_size = 1;
+    for (const LayerSpec& L : stack->spec.layers) { c.num_heads = std::max(c.num_heads, L.heads); c.intermediate_size = std::max(c.intermediate_size, L.ff); }
+    if (c.max_seq_len <= 0) c.max_seq_len = 4096;
+    stack->f32 = c.compute_f32 != 0;
+    c.kv_dtype = stack->f32 ? 1 : 0;
+    return create_handle(&c, std::move(stack), out);
 }
 
 // Registers a tensor given by its WHOLE dims and allocates this rank's part of it.  *out_t = null when the rank keeps
@@ -813,7 +722,8 @@ int32_t lc_model_get_tensor(lc_model* m, const char* name, void* out_bytes, size
 }
 
 // A gain vector as f32 on the device (norm weights are F32 in GGUF files; F16 is widened).
-static int32_t gain_f32(lc_model* m, const std::string& name, int expect, const float** out) {
+}  // extern "C"
+int32_t lc::model_gain_f32(lc_model* m, const std::string& name, int expect, const float** out) {
     auto it = m->tensors.find(name);
     LC_CHECK(it != m->tensors.end(), LC_ERR_MISSING, "missing tensor %s", name.c_str());
     DevTensor& t = it->second;
@@ -827,6 +737,7 @@ static int32_t gain_f32(lc_model* m, const std::string& name, int expect, const 
     *out = p;
     return LC_OK;
 }
+extern "C" {
 
 static int32_t weight_of(lc_model* m, const std::string& name, int n, int k, QWeight* w, DevTensor** tt) {
     auto it = m->tensors.find(name);
@@ -860,7 +771,7 @@ static int32_t finalize_experts(lc_model* m, int l) {
     LayerW& w = m->layers[l];
     const int E = m->cfg.n_experts, H = m->H, F = m->F;
     const std::string p = "blk." + std::to_string(l) + ".";
-    LC_TRY(gain_f32(m, p + "ffn_gate_inp.weight", E * H, &w.router));
+    LC_TRY(model_gain_f32(m, p + "ffn_gate_inp.weight", E * H, &w.router));
     const int El = m->El;  // the experts this rank holds: e0 .. e0 + El - 1, stored at 0 .. El - 1
     w.egate.resize(El); w.eup.resize(El); w.edown.resize(El);
     bool q4k = true;
@@ -892,10 +803,8 @@ static int32_t finalize_experts(lc_model* m, int l) {
     return LC_OK;
 }
 
-int32_t lc_model_finalize(lc_model* m) {
-    LC_TRY(check_model(m, false));
-    LC_CHECK(!m->finalized, LC_ERR_STATE, "model already finalized");
-    DeviceGuard dg(m->device);
+// The Llama family: nine tensors per layer, embedding, final norm, head.
+static int32_t bind_blocks(lc_model* m) {
     const int H = m->H, F = m->F, V = m->V, nq = m->nh * m->hd, nkvd = m->nkv * m->hd;
     m->layers.resize(m->L);
     for (int l = 0; l < m->L; l++) {
@@ -933,8 +842,8 @@ int32_t lc_model_finalize(lc_model* m) {
             LC_CHECK(tg->typ == tu->typ, LC_ERR_UNSUPPORTED, "layer %d: gate/up projections have different quant types", l);
             LC_TRY(weight_of(m, p + "ffn_down.weight", H, F, &w.down, nullptr));
         }
-        LC_TRY(gain_f32(m, p + "attn_norm.weight", H, &w.attn_norm));
-        LC_TRY(gain_f32(m, p + "ffn_norm.weight", H, &w.ffn_norm));
+        LC_TRY(model_gain_f32(m, p + "attn_norm.weight", H, &w.attn_norm));
+        LC_TRY(model_gain_f32(m, p + "ffn_norm.weight", H, &w.ffn_norm));
     }
     {
         auto it = m->tensors.find("token_embd.weight");
@@ -942,7 +851,7 @@ int32_t lc_model_finalize(lc_model* m) {
         LC_CHECK((int)it->second.cols == H, LC_ERR_INVALID, "token_embd.weight rows are %zu wide, hidden size is %d", it->second.cols, H);
         m->embed = &it->second;
     }
-    LC_TRY(gain_f32(m, "output_norm.weight", H, &m->final_norm));
+    LC_TRY(model_gain_f32(m, "output_norm.weight", H, &m->final_norm));
     // loader.rs:192-199: tied head when output.weight is absent
     if (m->tensors.count("output.weight")) {
         LC_TRY(weight_of(m, "output.weight", V, H, &m->head, nullptr));
@@ -952,23 +861,11 @@ int32_t lc_model_finalize(lc_model* m) {
         const size_t row_bytes = e.nbytes / e.rows;
         LC_TRY(qweight_init(&m->head, e.typ, (const uint8_t*)e.view + (size_t)m->v0 * row_bytes, V, H));
     }
+    return LC_OK;
+}
 
-    // weight sanity scan (loader.rs:241-249) and resident byte count
-    LC_TRY(dalloc(&m->d_sanity, 1));
-    LC_CUDA(cudaMemsetAsync(m->d_sanity, 0, 8, m->stream));
-    uint64_t wbytes = 0;
-    for (auto& kv : m->tensors) {
-        DevTensor& t = kv.second;
-        wbytes += t.nbytes;
-        LC_TRY(launch_sanity_scan(t.typ, t.view, t.rows * t.cols, m->d_sanity, m->stream));
-    }
-    unsigned long long bad = 0;
-    LC_CUDA(cudaMemcpyAsync(&bad, m->d_sanity, 8, cudaMemcpyDeviceToHost, m->stream));
-    LC_CUDA(cudaStreamSynchronize(m->stream));
-    m->ctr.sanitize_hits = bad;
-    m->ctr.weight_bytes = wbytes;
-
-    // KV pools and the page table
+// Key and value pools of every layer, their tensor maps, the merge slots of the single-token attention kernel.
+static int32_t alloc_block_pools(lc_model* m) {
     size_t page_elems = (size_t)m->nkv * m->page_tokens * m->hd;
     m->k_pools.resize(m->L); m->v_pools.resize(m->L);
     for (int l = 0; l < m->L; l++) {
@@ -991,19 +888,12 @@ int32_t lc_model_finalize(lc_model* m) {
             LC_CUDA(cudaMemsetAsync(m->d_stream_slots, 0, slot_bytes, m->stream));
         }
     }
-    m->free_pages.resize(m->pages_total);
-    for (int i = 0; i < m->pages_total; i++) m->free_pages[i] = m->pages_total - 1 - i;
-    m->seq_pages.assign(m->max_seqs, {});
-    m->seq_len.assign(m->max_seqs, 0);
-    m->h_page_table.assign((size_t)m->max_seqs * m->pages_per_seq, 0);
-    LC_TRY(dalloc(&m->d_page_table, m->h_page_table.size()));
-    m->ctr.kv_pages_total = m->pages_total;
+    return LC_OK;
+}
 
-    // step buffers
-    int T = m->t_cap;
-    LC_TRY(dalloc(&m->d_tokens, T)); LC_TRY(dalloc(&m->d_tok_seq, T)); LC_TRY(dalloc(&m->d_tok_pos, T));
-    LC_TRY(dalloc(&m->d_tok_rope, T)); LC_TRY(dalloc(&m->d_last_idx, T)); LC_TRY(dalloc(&m->d_tiles, T));
-    LC_TRY(dalloc(&m->d_hidden, (size_t)T * H)); LC_TRY(dalloc(&m->d_hidden2, (size_t)T * H));
+static int32_t alloc_block_buffers(lc_model* m) {
+    const int T = m->t_cap, H = m->H, F = m->F, nq = m->nh * m->hd;
+    LC_TRY(dalloc(&m->d_hidden2, (size_t)T * H));
     LC_TRY(dalloc(&m->d_qkv, (size_t)T * m->nqkv)); LC_TRY(dalloc(&m->d_attn, (size_t)T * nq));
     LC_TRY(dalloc(&m->d_ffn, (size_t)T * F));
     LC_TRY(qgemm_workspace_alloc(&m->gemm_ws, T, std::max(std::max(H, F), nq)));
@@ -1026,28 +916,69 @@ int32_t lc_model_finalize(lc_model* m) {
         LC_TRY(dalloc(&m->d_moe_touched, 1));
         LC_CUDA(cudaMemsetAsync(m->d_moe_touched, 0, 8, m->stream));
     }
-    LC_TRY(dalloc(&m->d_last, (size_t)m->max_seqs * H)); LC_TRY(dalloc(&m->d_logits, (size_t)m->max_seqs * V));
-    LC_TRY(dalloc(&m->d_next, m->max_seqs)); LC_TRY(dalloc(&m->d_step_ctr, 1));
-    if (m->tp > 1) {
-        // partial rows of the column-cut products and the greedy-pick keys: in the buffers the other ranks can read when the
-        // ranks are processes (a collective call: every rank finalizes its model at the same point), else plain memory
-        LC_TRY(dalloc(&m->d_key_max, (size_t)m->max_seqs));
-        LC_TRY(dalloc(&m->d_key, (size_t)m->max_seqs));
-        LC_TRY(dalloc(&m->d_part, (size_t)T * H));
-        if (m->use_dist) {  // a collective call: every rank finalizes its model at the same point
-            LC_TRY(dist_setup());
-            LC_TRY(dalloc(&m->d_logits_all, (size_t)m->max_seqs * m->cfg.vocab_size));
-        }
-    }
     size_t sc = 16;
     for (int t = 1; t <= T; t++) sc = std::max(sc, attention_scratch_bytes(t, m->nh, m->hd, m->cfg.max_seq_len));
     m->attn_scratch_bytes = sc;
     LC_TRY(dalloc((uint8_t**)&m->d_attn_scratch, sc));
     LC_TRY(dalloc(&m->d_attn_counters, (size_t)T * m->nh));
     LC_CUDA(cudaMemsetAsync(m->d_attn_counters, 0, (size_t)T * m->nh * sizeof(int), m->stream));
+    return LC_OK;
+}
+
+int32_t lc_model_finalize(lc_model* m) {
+    LC_TRY(check_model(m, false));
+    LC_CHECK(!m->finalized, LC_ERR_STATE, "model already finalized");
+    DeviceGuard dg(m->device);
+    LC_TRY(m->stack ? stack_bind(m) : bind_blocks(m));
+    const int H = m->H, V = m->V;
+
+    // weight sanity scan (loader.rs:241-249) and resident byte count
+    LC_TRY(dalloc(&m->d_sanity, 1));
+    LC_CUDA(cudaMemsetAsync(m->d_sanity, 0, 8, m->stream));
+    uint64_t wbytes = 0;
+    for (auto& kv : m->tensors) {
+        DevTensor& t = kv.second;
+        wbytes += t.nbytes;
+        LC_TRY(launch_sanity_scan(t.typ, t.view, t.rows * t.cols, m->d_sanity, m->stream));
+    }
+    unsigned long long bad = 0;
+    LC_CUDA(cudaMemcpyAsync(&bad, m->d_sanity, 8, cudaMemcpyDeviceToHost, m->stream));
+    LC_CUDA(cudaStreamSynchronize(m->stream));
+    m->ctr.sanitize_hits = bad;
+    m->ctr.weight_bytes = wbytes;
+
+    // KV pools and the page table
+    if (!m->stack) LC_TRY(alloc_block_pools(m));
+    m->free_pages.resize(m->pages_total);
+    for (int i = 0; i < m->pages_total; i++) m->free_pages[i] = m->pages_total - 1 - i;
+    m->seq_pages.assign(m->max_seqs, {});
+    m->seq_len.assign(m->max_seqs, 0);
+    m->h_page_table.assign((size_t)m->max_seqs * m->pages_per_seq, 0);
+    LC_TRY(dalloc(&m->d_page_table, m->h_page_table.size()));
+    m->ctr.kv_pages_total = m->pages_total;
+
+    // step buffers
+    int T = m->t_cap;
+    LC_TRY(dalloc(&m->d_tokens, T)); LC_TRY(dalloc(&m->d_tok_seq, T)); LC_TRY(dalloc(&m->d_tok_pos, T));
+    LC_TRY(dalloc(&m->d_tok_rope, T)); LC_TRY(dalloc(&m->d_last_idx, T)); LC_TRY(dalloc(&m->d_tiles, T));
+    LC_TRY(dalloc(&m->d_hidden, (size_t)T * H));
+    LC_TRY(m->stack ? stack_alloc(m) : alloc_block_buffers(m));
+    LC_TRY(dalloc(&m->d_last, (size_t)m->head_rows * H)); LC_TRY(dalloc(&m->d_logits, (size_t)m->head_rows * V));
+    LC_TRY(dalloc(&m->d_next, m->head_rows)); LC_TRY(dalloc(&m->d_step_ctr, 1));
+    if (m->tp > 1) {
+        // partial rows of the column-cut products and the greedy-pick keys: in the buffers the other ranks can read when the
+        // ranks are processes (a collective call: every rank finalizes its model at the same point), else plain memory
+        LC_TRY(dalloc(&m->d_key_max, (size_t)m->head_rows));
+        LC_TRY(dalloc(&m->d_key, (size_t)m->head_rows));
+        LC_TRY(dalloc(&m->d_part, (size_t)T * H));
+        if (m->use_dist) {  // a collective call: every rank finalizes its model at the same point
+            LC_TRY(dist_setup());
+            LC_TRY(dalloc(&m->d_logits_all, (size_t)m->head_rows * m->cfg.vocab_size));
+        }
+    }
     LC_CUDA(cudaHostAlloc((void**)&m->pin_tokens, (size_t)m->max_seqs * 8, cudaHostAllocDefault));
-    LC_CUDA(cudaHostAlloc((void**)&m->pin_next, ((size_t)m->max_seqs + 1) * 8, cudaHostAllocDefault));  // + one word: the device error flag of a call
-    LC_CUDA(cudaHostAlloc((void**)&m->pin_logits, (size_t)m->max_seqs * m->cfg.vocab_size * 4, cudaHostAllocDefault));
+    LC_CUDA(cudaHostAlloc((void**)&m->pin_next, ((size_t)m->head_rows + 1) * 8, cudaHostAllocDefault));  // + one word: the device error flag of a call
+    LC_CUDA(cudaHostAlloc((void**)&m->pin_logits, (size_t)m->head_rows * m->cfg.vocab_size * 4, cudaHostAllocDefault));
     LC_TRY(reserve_out_tokens(m, (size_t)1024 * m->max_seqs));
     LC_CUDA(cudaEventCreate(&m->ev0));
     LC_CUDA(cudaEventCreate(&m->ev1));
@@ -1064,6 +995,7 @@ int32_t lc_model_destroy(lc_model* m) {
     for (auto& kv : m->tensors) if (kv.second.dev) cudaFree(kv.second.dev);
     for (auto& w : m->layers) if (w.fused_buf) cudaFree(w.fused_buf);
     for (void* p : m->owned) cudaFree(p);
+    stack_free(m);
     for (void* p : m->k_pools) cudaFree(p);
     for (void* p : m->v_pools) cudaFree(p);
     if (m->leader) {  // leaving a group: the leader must not drive this handle any more
@@ -1147,6 +1079,12 @@ int32_t lc_kv_memory_bytes(const lc_model* m, uint64_t* out) {
     LC_CHECK(out, LC_ERR_INVALID, "null output");
     uint64_t tokens = 0;
     for (int v : m->seq_len) tokens += v;
+    if (m->stack) {
+        uint64_t live = 0;
+        for (int v : m->seq_len) live += v > 0;
+        *out = tokens * m->stack->cache_bytes_per_token + live * m->stack->state_bytes_per_seq;
+        return LC_OK;
+    }
     *out = tokens * (uint64_t)m->L * 2 * m->cfg.num_kv_heads * m->hd * m->kv_elt;  // cache/mod.rs:80-84, over all ranks
     return LC_OK;
 }
@@ -1186,22 +1124,38 @@ static int32_t fetch_logits(lc_model* lead, int n_rows, float* host_out) {
     return LC_OK;
 }
 
-int32_t lc_forward_batch(lc_model* lead, int32_t n_seqs, const int32_t* seq_ids, const int64_t* tokens, const int32_t* n_tokens,
-                         float* logits_out, int64_t* next_out) {
+// One step over a ragged batch: the new tokens of every listed sequence run together, in chunks of t_cap tokens that may
+// hold parts of several sequences.  The head runs on the wanted rows (place want[j] among the sequence's tokens of this
+// call, ascending per sequence), head_rows at a time.
+static int32_t run_step(lc_model* lead, int32_t n_seqs, const int32_t* seq_ids, const int64_t* tokens, const int32_t* n_tokens, const int32_t* n_want,
+                        const int32_t* want, float* logits_out, int64_t* next_out) {
     LC_TRY(check_model(lead, true));
     LC_TRY(check_drivable(lead));
-    LC_CHECK(n_seqs >= 1 && n_seqs <= lead->max_seqs && seq_ids && tokens && n_tokens, LC_ERR_INVALID, "forward_batch: bad argument");
+    LC_CHECK(n_seqs >= 1 && n_seqs <= lead->max_seqs && seq_ids && tokens && n_tokens, LC_ERR_INVALID, "step: bad argument");
     DeviceGuard dg(lead->device);
     std::vector<lc_model*> R = ranks_of(lead);
     int total = 0, longest = 0;
+    std::vector<int> rows;  // wanted rows as indices into the call's tokens
+    bool each_wanted = true;
+    size_t w_at = 0;
     for (int i = 0; i < n_seqs; i++) {
         LC_CHECK(seq_ids[i] >= 0 && seq_ids[i] < lead->max_seqs, LC_ERR_INVALID, "sequence id %d outside 0..%d", seq_ids[i], lead->max_seqs - 1);
         for (int j = 0; j < i; j++) LC_CHECK(seq_ids[j] != seq_ids[i], LC_ERR_INVALID, "sequence id %d listed twice", seq_ids[i]);
         LC_CHECK(n_tokens[i] >= 1, LC_ERR_INVALID, "sequence %d has no tokens in this call", seq_ids[i]);
-        for (lc_model* m : R) LC_TRY(ensure_pages(m, seq_ids[i], m->seq_len[seq_ids[i]] + n_tokens[i]));
+        const int nw = n_want ? n_want[i] : 1;
+        LC_CHECK(nw >= 0 && (nw == 0 || !n_want || want), LC_ERR_INVALID, "step: bad list of wanted places");
+        for (int j = 0; j < nw; j++, w_at++) {
+            const int place = n_want ? want[w_at] : n_tokens[i] - 1;
+            LC_CHECK(place >= 0 && place < n_tokens[i] && (j == 0 || total + place > rows.back()), LC_ERR_INVALID,
+                     "sequence %d: wanted place %d outside its %d tokens or out of order", seq_ids[i], place, n_tokens[i]);
+            rows.push_back(total + place);
+        }
+        each_wanted = each_wanted && nw == 1;
         total += n_tokens[i];
         longest = std::max(longest, n_tokens[i]);
     }
+    for (int i = 0; i < n_seqs; i++)
+        for (lc_model* m : R) LC_TRY(ensure_pages(m, seq_ids[i], m->seq_len[seq_ids[i]] + n_tokens[i]));
     for (lc_model* m : R) LC_TRY(sync_page_table(m));
     if (longest == 1) {
         // a decode step: token ids in (pinned staging), graph replay, picks and logits out
@@ -1213,53 +1167,62 @@ int32_t lc_forward_batch(lc_model* lead, int32_t n_seqs, const int32_t* seq_ids,
         LC_TRY(run_decode_steps(lead, n_seqs, 1));
         if (next_out) LC_CUDA(cudaMemcpyAsync(lead->pin_next, lead->d_next, (size_t)n_seqs * 8, cudaMemcpyDeviceToHost, lead->stream));
         LC_TRY(queue_flag_read(lead));
-        if (logits_out) LC_TRY(fetch_logits(lead, n_seqs, logits_out));
+        std::vector<float> all;  // some rows are not wanted: fetch all, keep the others
+        if (logits_out && !rows.empty()) {
+            if (!each_wanted) all.resize((size_t)n_seqs * lead->cfg.vocab_size);
+            LC_TRY(fetch_logits(lead, n_seqs, each_wanted ? logits_out : all.data()));
+        }
         LC_CUDA(cudaStreamSynchronize(lead->stream));
-        if (next_out) memcpy(next_out, lead->pin_next, (size_t)n_seqs * 8);
+        for (size_t j = 0; j < rows.size(); j++) {
+            if (!all.empty()) memcpy(logits_out + j * lead->cfg.vocab_size, all.data() + (size_t)rows[j] * lead->cfg.vocab_size, (size_t)lead->cfg.vocab_size * 4);
+            if (next_out) next_out[j] = lead->pin_next[rows[j]];
+        }
         for (lc_model* m : R) { after_decode_steps(m, n_seqs, seq_ids, 1); finish_call(m); }
         return flag_result(lead);
     }
     for (lc_model* m : R) m->meta_valid = false;
     // Rotary index = position inside the CALL (reference mode, attention.rs:13-21) or the cache position.
-    if (total <= lead->t_cap) {
-        std::vector<int64_t> tok; std::vector<int32_t> seq, pos, rope, last;
-        int off = 0;
-        for (int i = 0; i < n_seqs; i++) {
-            for (int t = 0; t < n_tokens[i]; t++) {
-                int p = lead->seq_len[seq_ids[i]] + t;
-                tok.push_back(tokens[off + t]); seq.push_back(seq_ids[i]); pos.push_back(p);
-                rope.push_back(lead->cfg.rope_mode ? p : t);
-            }
-            off += n_tokens[i];
-            last.push_back(off - 1);
+    std::vector<int64_t> tok(tokens, tokens + total);
+    std::vector<int32_t> seq, pos, rope;
+    for (int i = 0; i < n_seqs; i++)
+        for (int t = 0; t < n_tokens[i]; t++) {
+            const int p = lead->seq_len[seq_ids[i]] + t;
+            seq.push_back(seq_ids[i]); pos.push_back(p); rope.push_back(lead->cfg.rope_mode ? p : t);
         }
-        for (lc_model* m : R) LC_TRY(upload_meta(m, tok, seq, pos, rope, last));
-        LC_TRY(forward_tokens(lead, total, n_seqs, total == n_seqs, 0));
-    } else {
-        // long prompts: one sequence after the other, each in chunks of t_cap tokens over its growing cache
-        int off = 0;
-        for (int i = 0; i < n_seqs; i++) {
-            for (int c0 = 0; c0 < n_tokens[i]; c0 += lead->t_cap) {
-                int T = std::min(lead->t_cap, n_tokens[i] - c0);
-                std::vector<int64_t> tok(T); std::vector<int32_t> seq(T, seq_ids[i]), pos(T), rope(T), last(1, T - 1);
-                for (int t = 0; t < T; t++) {
-                    tok[t] = tokens[off + c0 + t];
-                    pos[t] = lead->seq_len[seq_ids[i]] + c0 + t;
-                    rope[t] = lead->cfg.rope_mode ? pos[t] : (c0 + t);
-                }
-                for (lc_model* m : R) LC_TRY(upload_meta(m, tok, seq, pos, rope, last));
-                if (c0 + T == n_tokens[i]) LC_TRY(forward_tokens(lead, T, 1, T == 1, i));
-                else LC_TRY(run_layers(lead, T, false));
+    size_t done = 0, held = 0;  // wanted rows that are on the host; rows in d_logits behind them
+    auto flush = [&]() -> int32_t {
+        if (held == 0) return LC_OK;
+        if (next_out) LC_CUDA(cudaMemcpyAsync(lead->pin_next, lead->d_next, held * 8, cudaMemcpyDeviceToHost, lead->stream));
+        if (logits_out) LC_TRY(fetch_logits(lead, (int)held, logits_out + done * lead->cfg.vocab_size));
+        LC_CUDA(cudaStreamSynchronize(lead->stream));
+        if (next_out) memcpy(next_out + done, lead->pin_next, held * 8);
+        done += held;
+        held = 0;
+        return LC_OK;
+    };
+    size_t next_row = 0;
+    for (int c0 = 0; c0 < total; c0 += lead->t_cap) {
+        const int T = std::min(lead->t_cap, total - c0);
+        auto part = [&](auto& v) { return typename std::remove_reference<decltype(v)>::type(v.begin() + c0, v.begin() + c0 + T); };
+        for (lc_model* m : R) LC_TRY(upload_meta(m, part(tok), part(seq), part(pos), part(rope), {}));
+        const bool all_last = total == n_seqs;
+        LC_TRY(run_layers(lead, T, all_last));
+        while (next_row < rows.size() && rows[next_row] < c0 + T) {
+            std::vector<int32_t> idx;
+            while (next_row < rows.size() && rows[next_row] < c0 + T && held + idx.size() < (size_t)lead->head_rows) idx.push_back(rows[next_row++] - c0);
+            for (lc_model* m : R) {
+                LC_CUDA(cudaMemcpyAsync(m->d_last_idx, idx.data(), idx.size() * 4, cudaMemcpyHostToDevice, m->stream));
+                LC_CUDA(cudaStreamSynchronize(m->stream));
             }
-            off += n_tokens[i];
+            LC_TRY(head_tokens(lead, (int)idx.size(), false, (int)held));
+            held += idx.size();
+            if (held == (size_t)lead->head_rows) LC_TRY(flush());
         }
     }
+    LC_TRY(flush());
+    LC_CUDA(cudaStreamSynchronize(lead->stream));
     for (lc_model* m : R)
         for (int i = 0; i < n_seqs; i++) m->seq_len[seq_ids[i]] += n_tokens[i];
-    if (next_out) LC_CUDA(cudaMemcpyAsync(lead->pin_next, lead->d_next, (size_t)n_seqs * 8, cudaMemcpyDeviceToHost, lead->stream));
-    if (logits_out) LC_TRY(fetch_logits(lead, n_seqs, logits_out));
-    LC_CUDA(cudaStreamSynchronize(lead->stream));
-    if (next_out) memcpy(next_out, lead->pin_next, (size_t)n_seqs * 8);
     for (lc_model* m : R) {
         m->ctr.forward_calls += 1;
         m->ctr.tokens_prefilled += total;
@@ -1269,6 +1232,40 @@ int32_t lc_forward_batch(lc_model* lead, int32_t n_seqs, const int32_t* seq_ids,
         finish_call(m);
     }
     return check_device_flag(lead);
+}
+
+int32_t lc_forward_batch(lc_model* m, int32_t n_seqs, const int32_t* seq_ids, const int64_t* tokens, const int32_t* n_tokens, float* logits_out,
+                         int64_t* next_out) {
+    return run_step(m, n_seqs, seq_ids, tokens, n_tokens, nullptr, nullptr, logits_out, next_out);
+}
+
+int32_t lc_step(lc_model* m, int32_t n_seqs, const int32_t* seq_ids, const int64_t* tokens, const int32_t* n_tokens, const int32_t* n_want,
+                const int32_t* want, float* logits_out, int64_t* next_out) {
+    LC_CHECK(n_want, LC_ERR_INVALID, "lc_step: null argument");
+    return run_step(m, n_seqs, seq_ids, tokens, n_tokens, n_want, want, logits_out, next_out);
+}
+
+int32_t lc_seq_open(lc_model* m, int32_t* seq_id) {
+    LC_TRY(check_model(m, true));
+    LC_TRY(check_drivable(m));
+    LC_CHECK(seq_id, LC_ERR_INVALID, "lc_seq_open: null output");
+    for (int i = 0; i < m->max_seqs; i++)
+        if (!m->seq_open[i]) {
+            LC_TRY(lc_kv_clear(m, i));
+            m->seq_open[i] = 1;
+            *seq_id = i;
+            return LC_OK;
+        }
+    set_error("all %d sequence slots are in use", m->max_seqs);
+    return LC_ERR_KV_FULL;
+}
+
+int32_t lc_seq_close(lc_model* m, int32_t seq_id) {
+    LC_TRY(check_model(m, true));
+    LC_CHECK(seq_id >= 0 && seq_id < m->max_seqs && m->seq_open[seq_id], LC_ERR_INVALID, "lc_seq_close: slot %d is not open", seq_id);
+    LC_TRY(lc_kv_clear(m, seq_id));
+    m->seq_open[seq_id] = 0;
+    return LC_OK;
 }
 
 int32_t lc_forward(lc_model* m, const int64_t* tokens, int32_t n, float* logits_out) {
@@ -1511,8 +1508,10 @@ int32_t lc_probe_attention(lc_model* m, int32_t layer, const float* normed, int3
     DeviceGuard dg(m->device);
     LC_TRY(probe_meta(m, seq));
     LC_CUDA(cudaMemcpyAsync(m->d_hidden, normed, (size_t)seq * m->H * 4, cudaMemcpyHostToDevice, m->stream));
-    LC_TRY(attention_block(m, layer, m->d_hidden, nullptr, seq, nullptr, m->d_hidden2, false));
-    LC_CUDA(cudaMemcpyAsync(out, m->d_hidden2, (size_t)seq * m->H * 4, cudaMemcpyDeviceToHost, m->stream));
+    float* res = m->d_hidden2;
+    if (m->stack) LC_TRY(stack_probe(m, layer, seq, false, &res));
+    else LC_TRY(attention_block(m, layer, m->d_hidden, nullptr, seq, nullptr, m->d_hidden2, false));
+    LC_CUDA(cudaMemcpyAsync(out, res, (size_t)seq * m->H * 4, cudaMemcpyDeviceToHost, m->stream));
     LC_CUDA(cudaStreamSynchronize(m->stream));
     m->seq_len[0] += seq;
     finish_call(m);
@@ -1524,8 +1523,10 @@ int32_t lc_probe_ffn(lc_model* m, int32_t layer, const float* x, int32_t seq, fl
     LC_CHECK(layer >= 0 && layer < m->L && x && out && seq >= 1 && seq <= m->t_cap, LC_ERR_INVALID, "probe_ffn: bad argument");
     DeviceGuard dg(m->device);
     LC_CUDA(cudaMemcpyAsync(m->d_hidden, x, (size_t)seq * m->H * 4, cudaMemcpyHostToDevice, m->stream));
-    LC_TRY(ffn_block(m, layer, m->d_hidden, nullptr, seq, nullptr, m->d_hidden2, false));
-    LC_CUDA(cudaMemcpyAsync(out, m->d_hidden2, (size_t)seq * m->H * 4, cudaMemcpyDeviceToHost, m->stream));
+    float* res = m->d_hidden2;
+    if (m->stack) LC_TRY(stack_probe(m, layer, seq, true, &res));
+    else LC_TRY(ffn_block(m, layer, m->d_hidden, nullptr, seq, nullptr, m->d_hidden2, false));
+    LC_CUDA(cudaMemcpyAsync(out, res, (size_t)seq * m->H * 4, cudaMemcpyDeviceToHost, m->stream));
     LC_CUDA(cudaStreamSynchronize(m->stream));
     finish_call(m);
     return LC_OK;

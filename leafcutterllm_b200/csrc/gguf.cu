@@ -300,7 +300,7 @@ extern "C" int32_t lc_gguf_inspect(const char* path, int32_t scan, lc_gguf_repor
         if (!known) continue;
         report->tensors_by_type[t.typ]++;
         QuantGeom g;
-        if (!quant_geom(t.typ, &g)) report->unsupported_types |= 1u << t.typ;  // quant.rs:243-254: the same eight types
+        if (t.typ == LC_TYPE_BF16 || !quant_geom(t.typ, &g)) report->unsupported_types |= 1u << t.typ;  // quant.rs:243-254: the same eight types
     }
 
     // missing tensors of the first layers, unrecognised blk.* tensors (loader.rs:59-89)

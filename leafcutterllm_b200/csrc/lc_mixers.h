@@ -1,0 +1,173 @@
+// Launch interface of the layers that checkpoint-directory designs are made of (bf16 weights; activations bf16, or f32 when
+// the model runs in true 32-bit), and what a model of such layers keeps on the device.
+#pragma once
+#include <cuda_bf16.h>
+#include <map>
+#include <memory>
+#include <vector>
+#include "lc_arch.h"
+#include "lc_common.cuh"
+
+namespace lc {
+
+inline int round8(int v) { return (v + 7) & ~7; }
+
+// ---- dense16.cu: y = x W^T over bf16 weights -----------------------------------------------------------------------------
+// `batch` matrices of n rows and k columns (one per head in the batched products), rows ld elements apart (ld % 8 == 0).
+struct DenseWeight {
+    const __nv_bfloat16* data = nullptr;
+    int n = 0, k = 0, ld = 0, batch = 1;
+    size_t batch_stride = 0;
+    alignas(64) unsigned char tmap[128];
+    bool has_tmap = false;
+};
+int32_t dense_weight_init(DenseWeight* w, const __nv_bfloat16* data, int n, int k, int ld, int batch = 1, size_t batch_stride = 0);
+
+enum DenseEpilogue {
+    DENSE_STORE = 0,
+    DENSE_RELU2 = 1,      // max(y, 0)^2
+    DENSE_LOG_DECAY = 2,  // -e0[row / e_div] * softplus(y + e1[row]), 32-bit
+    DENSE_LOGITS = 3      // y * scale, then cap * tanh(. / cap) when cap > 0
+};
+struct DenseArgs {
+    const DenseWeight* w = nullptr;
+    const void* x = nullptr;      // [x_rows][..] activations, bf16 or (f32 = true) float; row t of matrix b at x + b * x_batch + t * ldx
+    int ldx = 0, x_rows = 0;      // x_rows: rows the buffer has (>= T)
+    size_t x_batch = 0;
+    int T = 0;
+    void* out = nullptr;          // row t of matrix b at out + b * out_batch + t * ldo
+    int ldo = 0;
+    size_t out_batch = 0;
+    bool out_f32 = false;         // otherwise the activations' type
+    DenseEpilogue epi = DENSE_STORE;
+    const float* e0 = nullptr;
+    const float* e1 = nullptr;
+    int e_div = 1;
+    float scale = 1.0f, cap = 0.0f;
+    bool f32 = false;
+};
+// Scratch of the shares of k that several CTAs sum, and the tensor maps over activation buffers seen so far.
+struct DenseWorkspace {
+    float* partial = nullptr;
+    size_t partial_bytes = 0;
+    unsigned* tickets = nullptr;
+    int max_tickets = 0;
+    struct Map { alignas(64) unsigned char b[128]; };
+    std::map<std::vector<uint64_t>, std::unique_ptr<Map>> maps;
+};
+int32_t dense_workspace_alloc(DenseWorkspace* ws);
+void dense_workspace_free(DenseWorkspace* ws);
+int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s);
+
+// ---- mixers.cu -------------------------------------------------------------------------------------------------------
+// Consecutive tokens of one sequence inside a call: rows tok0 .. tok0 + n - 1, the first at position pos0.
+struct SeqRun { int32_t tok0, n, seq, pos0; };
+
+// Copies a weight into a padded layout: element (r, c) of [rows, cols] goes to row map(r), column map(c), where a map sends
+// index i of groups of `len` to group * stride + i, entries from `split` on moved up by `shift`; `transpose` swaps rows and
+// columns inside each row group (dst row = group * stride + column, dst column = index inside the group).
+struct PackMap { int len = 0, stride = 0, split = 0, shift = 0; };
+int32_t launch_pack(const __nv_bfloat16* src, int rows, int cols, __nv_bfloat16* dst, int ld, PackMap row, PackMap col, bool transpose, cudaStream_t s);
+
+// x[t] = embed[ids[t]] in f32 and, act != null, as bf16 (rows ld_act apart); ids outside the table give zero rows
+int32_t launch_embed_rows(const __nv_bfloat16* table, int rows, int width, const int64_t* ids, int T, float* x, void* act, int ld_act, cudaStream_t s);
+// act[t] = bf16(x[t])
+int32_t launch_act_rows(const float* x, int width, int T, void* act, int ld_act, cudaStream_t s);
+// x[t] += rms_norm(y[t]) * w; act != null: also the sum as bf16
+int32_t launch_norm_residual(const float* y, const float* w, float eps, int width, int T, float* x, void* act, int ld_act, cudaStream_t s);
+// out[i] = rms_norm(x[idx ? idx[i] : i]) * w as activations
+int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, float eps, int width, int n, void* out, int ldo, bool f32, cudaStream_t s);
+
+// Gated delta rule with one decay per key channel.  `proj` rows hold q | k | v | ... | beta logits as projected; the inputs of
+// the short convolutions of the last `taps` positions live in `ring` [slot][taps][channels], entry position % taps.
+struct DeltaShape { int heads, kv_heads, dim, vdim, taps, ld, off_k, off_v, off_b, channels; float unit_eps, eps; };
+struct DeltaArgs {
+    DeltaShape g;
+    const void* proj = nullptr;
+    const float* conv = nullptr;       // [channels][taps], the last column weighs the current token
+    void* ring = nullptr;
+    float* state = nullptr;            // [slot][heads][dim][vdim]
+    const int32_t *tok_seq = nullptr, *tok_pos = nullptr;
+    int T = 0;
+    float* qk = nullptr;               // [T][2][kv_heads * dim] unit vectors, q scaled by dim^-1/2
+    float* v = nullptr;                // [T][heads * vdim]
+    const float* log_decay = nullptr;  // [T][heads * dim]
+    float* o = nullptr;                // [T][heads * vdim]
+    const SeqRun* runs = nullptr;
+    int n_runs = 0;
+    const float* norm_w = nullptr;     // [vdim]
+    const void* gate = nullptr;        // [T][heads * vdim] before the sigmoid
+    void* out = nullptr;               // [T][ldo] activations
+    int ldo = 0;
+    bool f32 = false;
+};
+int32_t launch_delta_prep(const DeltaArgs& a, cudaStream_t s);   // convolutions, silu, unit vectors
+int32_t launch_delta_scan(const DeltaArgs& a, cudaStream_t s);   // the recurrence over every run; leaves state and ring for the next call
+int32_t launch_delta_output(const DeltaArgs& a, cudaStream_t s); // per-head norm, gate
+int32_t launch_delta_step(const DeltaArgs& a, cudaStream_t s);   // the three for one new token per sequence (rows of tok_seq / tok_pos)
+
+// Cache of latent attention: per page page_tokens rows [kv_rank | pad | rot_dim | pad] of the activations' type.
+struct LatentShape { int heads, dim, rot, rank, ld_q, dp, cp, rp, rot_pairs; float scale; };  // dp, cp, rp: dim, rank, rot rounded up to 8
+struct LatentArgs {
+    LatentShape g;
+    const float* proj = nullptr;       // [T][ld_proj]: query latent | kv latent | rotated key part
+    int ld_proj = 0, q_rank = 0, off_c = 0, off_r = 0;
+    const float *q_norm = nullptr, *c_norm = nullptr;
+    float eps = 1e-6f;
+    const float2* rot = nullptr;       // [position][rot_pairs] (cos, sin)
+    void* cq = nullptr;                // [T][ld_cq]
+    int ld_cq = 0;
+    void* cache = nullptr;
+    int page_tokens = 16;
+    const int32_t *page_table = nullptr, *tok_seq = nullptr, *tok_pos = nullptr;
+    int pages_per_seq = 0, T = 0;
+    const void* q = nullptr;           // [T][heads][ld_q]: unrotated part at 0, part to rotate at dp
+    const void* q_abs = nullptr;       // [T][heads][cp]: the unrotated part carried through the key projection
+    void* o = nullptr;                 // [T][heads][cp]: weighted sums of latents
+    bool f32 = false;
+};
+int32_t launch_latent_prep(const LatentArgs& a, cudaStream_t s);
+int32_t launch_rot_table(const double* freq_dev, int pairs, double magnitude, int positions, float2* out, cudaStream_t s);
+// ---- latent_attention.cu ---------------------------------------------------------------------------------------------
+int32_t launch_latent_attention(const LatentArgs& a, cudaStream_t s);
+
+// ---- a stack of such layers (layers.cu) --------------------------------------------------------------------------------
+struct StackLayer {
+    LayerSpec s;
+    const float *norm1 = nullptr, *norm2 = nullptr;
+    DenseWeight in, out, up, down;
+    // ChannelDelta: `in` = q | k | v | a1 | g1 | b
+    DenseWeight a2, g2;
+    DeltaShape dg{};
+    int off_a = 0, off_g = 0;
+    const float *conv = nullptr, *a_exp = nullptr, *dt_bias = nullptr, *o_norm = nullptr;
+    float* state = nullptr;
+    void* ring = nullptr;
+    // LatentAttention: `in` = dq | dkv
+    DenseWeight uq, uk_t, uv;
+    LatentShape lg{};
+    int off_r = 0, off_c = 0, ep = 0;
+    const float *q_norm = nullptr, *c_norm = nullptr;
+    const float2* rot = nullptr;
+    void* cache = nullptr;
+};
+struct LayerStack {
+    ArchSpec spec;
+    bool f32 = false;                  // true 32-bit activations and cache
+    std::vector<StackLayer> layers;
+    DenseWeight head;
+    const __nv_bfloat16* embed = nullptr;
+    const float* final_norm = nullptr;
+    DenseWorkspace ws;
+    std::vector<void*> owned;
+    std::vector<std::pair<RotarySpec, const float2*>> rot_tables;
+    uint64_t cache_bytes_per_token = 0, state_bytes_per_seq = 0;
+    // step buffers for t_cap tokens
+    int width_p = 0;
+    void *xa = nullptr, *proj = nullptr, *gate = nullptr, *mixed = nullptr, *cq = nullptr, *q = nullptr, *q_abs = nullptr, *o_lat = nullptr, *ffn = nullptr, *last = nullptr;
+    float *y = nullptr, *projf = nullptr, *log_decay = nullptr, *qk = nullptr, *v = nullptr, *o = nullptr;
+    SeqRun* d_runs = nullptr;
+    int n_runs = 0;
+};
+
+}  // namespace lc

@@ -96,6 +96,7 @@ __device__ __forceinline__ float dequant_elem(uint32_t typ, const uint8_t* base,
     switch (typ) {
         case LC_TYPE_F32: return ((const float*)base)[idx];
         case LC_TYPE_F16: return h2f(((const uint16_t*)base)[idx]);
+        case LC_TYPE_BF16: return __uint_as_float((uint32_t)((const uint16_t*)base)[idx] << 16);
         case LC_TYPE_Q4_0: return dequant_elem_q4_0(base + (idx >> 5) * 18, (int)(idx & 31));
         case LC_TYPE_Q8_0: return dequant_elem_q8_0(base + (idx >> 5) * 34, (int)(idx & 31));
         case LC_TYPE_Q4_K: return dequant_elem_q4_k(base + (idx >> 8) * 144, (int)(idx & 255));

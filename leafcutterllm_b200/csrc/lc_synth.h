@@ -363,6 +363,7 @@ LCS_HD void lcs_quantize_q6_k_block(const float* x, uint8_t* out) {
 // ggml type codes used here (rust/src/model/quant.rs:45-76).
 #define LCS_TYPE_F32 0
 #define LCS_TYPE_F16 1
+#define LCS_TYPE_BF16 30
 #define LCS_TYPE_Q4_0 2
 #define LCS_TYPE_Q8_0 8
 #define LCS_TYPE_Q4_K 12
@@ -392,6 +393,11 @@ LCS_HD void lcs_synth_block(uint32_t typ, uint64_t seed, uint64_t name_hash, flo
     } else if (typ == LCS_TYPE_F16) {
         uint16_t h = lcs_f32_to_f16(lcs_normal(seed, name_hash, blk, sigma));
         out[0] = (uint8_t)(h & 0xFF); out[1] = (uint8_t)(h >> 8);
+    } else if (typ == LCS_TYPE_BF16) {  // round to nearest, ties to even (the values are finite)
+        union { float f; uint32_t u; } v;
+        v.f = lcs_normal(seed, name_hash, blk, sigma);
+        uint32_t b = (v.u + 0x7FFFu + ((v.u >> 16) & 1u)) >> 16;
+        out[0] = (uint8_t)(b & 0xFF); out[1] = (uint8_t)(b >> 8);
     } else {  // F32
         union { float f; uint32_t u; } v;
         v.f = lcs_normal(seed, name_hash, blk, sigma);

@@ -1,0 +1,537 @@
+// The kernels of the checkpoint-directory layers around their products: embedding, norms and residual sums, the gated delta
+// rule with its short convolutions, the preparation of latent attention.  Template parameter A = type of the activations
+// (bf16, or float when a model runs in true 32-bit); norms, decays, step sizes, unit vectors, the recurrence and its state,
+// rotation angles and residual sums are f32 in both.
+#include <cmath>
+#include "lc_mixers.h"
+#include "lc_tma.cuh"
+
+namespace lc {
+
+namespace {
+
+template <typename A> __device__ __forceinline__ float act_f(A v);
+template <> __device__ __forceinline__ float act_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float act_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename A> __device__ __forceinline__ A to_act(float v);
+template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 to_act<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+__device__ __forceinline__ int mapped(const PackMap& m, int i) {
+    if (m.len == 0) return i;
+    const int g = i / m.len, r = i - g * m.len;
+    return g * m.stride + r + (m.shift && r >= m.split ? m.shift : 0);
+}
+__global__ void pack_kernel(const __nv_bfloat16* __restrict__ src, int rows, int cols, __nv_bfloat16* __restrict__ dst, int ld, PackMap rm, PackMap cm, int transpose) {
+    const size_t n = (size_t)rows * cols;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+        const int r = (int)(i / cols), c = (int)(i % cols);
+        if (transpose) {
+            const int g = r / rm.len, q = r - g * rm.len;
+            dst[((size_t)g * rm.stride + c) * ld + q] = src[i];
+        } else {
+            dst[(size_t)mapped(rm, r) * ld + mapped(cm, c)] = src[i];
+        }
+    }
+}
+
+__global__ void __launch_bounds__(256) embed_rows_kernel(const __nv_bfloat16* __restrict__ table, int rows, int width, const int64_t* __restrict__ ids,
+                                                         float* __restrict__ x, __nv_bfloat16* __restrict__ act, int ld_act) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int64_t id = ids[t];
+    const bool ok = id >= 0 && id < rows;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        const __nv_bfloat16 v = ok ? table[(size_t)id * width + c] : __float2bfloat16_rn(0.0f);
+        x[(size_t)t * width + c] = __bfloat162float(v);
+        if (act) act[(size_t)t * ld_act + c] = v;
+    }
+}
+
+__global__ void __launch_bounds__(256) act_rows_kernel(const float* __restrict__ x, int width, __nv_bfloat16* __restrict__ act, int ld_act) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (int c = threadIdx.x; c < width; c += blockDim.x) act[(size_t)blockIdx.x * ld_act + c] = __float2bfloat16_rn(x[(size_t)blockIdx.x * width + c]);
+}
+
+__global__ void __launch_bounds__(512) norm_residual_kernel(const float* __restrict__ y, const float* __restrict__ w, float eps, int width, float* __restrict__ x,
+                                                            __nv_bfloat16* __restrict__ act, int ld_act) {
+    __shared__ float sh[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const float* yr = y + t * width;
+    float* xr = x + t * width;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) { const float v = yr[c]; ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, sh);
+    const float r = 1.0f / sqrtf(ss / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        const float v = xr[c] + yr[c] * r * w[c];
+        xr[c] = v;
+        if (act) act[t * ld_act + c] = __float2bfloat16_rn(v);
+    }
+}
+
+template <typename A>
+__global__ void __launch_bounds__(512) norm_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ idx, const float* __restrict__ w, float eps, int width,
+                                                        A* __restrict__ out, int ldo) {
+    __shared__ float sh[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const float* xr = x + (size_t)(idx ? idx[blockIdx.x] : (int)blockIdx.x) * width;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) { const float v = xr[c]; ss = fmaf(v, v, ss); }
+    ss = block_sum(ss, sh);
+    const float r = 1.0f / sqrtf(ss / (float)width + eps);
+    A* o = out + (size_t)blockIdx.x * ldo;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) o[c] = to_act<A>(xr[c] * r * w[c]);
+}
+
+// ---- gated delta rule ------------------------------------------------------------------------------------------------
+// The convolution of one channel at token t: the inputs of earlier positions come from the call's rows as far as they belong
+// to the same sequence's run, from the ring before that, and are zero before the sequence's start.
+template <typename A>
+__device__ __forceinline__ float conv_at(const DeltaShape& g, const A* proj, const A* ring, const float* w, const int32_t* tok_seq, const int32_t* tok_pos, int t,
+                                         int seq, int pos, int channel, int column) {
+    float acc = 0.0f;
+    for (int j = g.taps - 1; j >= 0; j--) {  // j tokens back
+        float v = 0.0f;
+        if (pos - j >= 0) {
+            const int tt = t - j;
+            if (tt >= 0 && tok_seq[tt] == seq && tok_pos[tt] == pos - j) v = act_f<A>(proj[(size_t)tt * g.ld + column]);
+            else v = act_f<A>(ring[((size_t)seq * g.taps + (pos - j) % g.taps) * g.channels + channel]);
+        }
+        acc = fmaf(w[channel * g.taps + (g.taps - 1 - j)], v, acc);
+    }
+    return acc;
+}
+__device__ __forceinline__ float silu32(float v) { return v * sigmoid_f(v); }
+
+// One warp per (token, head unit): kv_heads units of q, kv_heads of k, heads of v.
+template <typename A>
+__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const DeltaShape& g = a.g;
+    const int t = blockIdx.x, unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (unit >= 2 * g.kv_heads + g.heads) return;
+    const A* proj = (const A*)a.proj;
+    const A* ring = (const A*)a.ring;
+    const int seq = a.tok_seq[t], pos = a.tok_pos[t];
+    if (unit >= 2 * g.kv_heads) {
+        const int h = unit - 2 * g.kv_heads, c0 = 2 * g.kv_heads * g.dim + h * g.vdim;
+        for (int i = lane; i < g.vdim; i += 32)
+            a.v[(size_t)t * g.heads * g.vdim + h * g.vdim + i] = silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, g.off_v + h * g.vdim + i));
+        return;
+    }
+    const bool is_k = unit >= g.kv_heads;
+    const int h = is_k ? unit - g.kv_heads : unit, c0 = unit * g.dim, col0 = (is_k ? g.off_k : 0) + h * g.dim;
+    float* o = a.qk + ((size_t)t * 2 + (is_k ? 1 : 0)) * g.kv_heads * g.dim + h * g.dim;
+    float ss = 0.0f, v[8];
+    int n = 0;
+    for (int i = lane; i < g.dim; i += 32, n++) {
+        const float s = silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, col0 + i));
+        ss = fmaf(s, s, ss);
+        if (n < 8) v[n] = s;
+    }
+    ss = warp_sum(ss);
+    float r = 1.0f / sqrtf(ss + g.unit_eps);
+    if (!is_k) r *= 1.0f / sqrtf((float)g.dim);
+    n = 0;
+    for (int i = lane; i < g.dim; i += 32, n++) o[i] = v[n] * r;
+}
+
+// The recurrence, token by token in f32.  A CTA of four warps owns 32 value columns of one head of one run; four lanes share
+// a column's `dim` state entries (DPL each: float4 groups dealt round robin), eight columns per warp.
+constexpr int kScanTok = 16;  // tokens staged in shared memory at a time
+template <typename A, int DPL>
+__global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaArgs a) {
+    constexpr int DP = DPL * 4;
+    extern __shared__ float sm[];
+    float *s_q = sm, *s_k = s_q + kScanTok * DP, *s_g = s_k + kScanTok * DP, *s_v = s_g + kScanTok * DP, *s_b = s_v + kScanTok * 32;
+    pdl_launch_dependents();
+    pdl_wait();
+    const DeltaShape& g = a.g;
+    const SeqRun run = a.runs[blockIdx.x];
+    const int h = blockIdx.y, rep = g.heads / g.kv_heads, kh = h / rep;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r4 = lane & 3, col = warp * 8 + (lane >> 2), e = blockIdx.z * 32 + col;
+    float* st = a.state + ((size_t)run.seq * g.heads + h) * g.dim * g.vdim;
+    const A* proj = (const A*)a.proj;
+    float S[DPL];
+#pragma unroll
+    for (int i = 0; i < DPL; i++) {
+        const int d = (i >> 2) * 16 + r4 * 4 + (i & 3);
+        S[i] = (run.pos0 > 0 && d < g.dim && e < g.vdim) ? st[(size_t)d * g.vdim + e] : 0.0f;
+    }
+    for (int c0 = 0; c0 < run.n; c0 += kScanTok) {
+        const int m = min(kScanTok, run.n - c0);
+        __syncthreads();
+        for (int i = threadIdx.x; i < m * DP; i += 128) {
+            const int t = i / DP, d = i - t * DP;
+            const size_t tok = (size_t)(run.tok0 + c0 + t);
+            float q = 0.0f, k = 0.0f, gg = 0.0f;
+            if (d < g.dim) {
+                q = a.qk[tok * 2 * g.kv_heads * g.dim + kh * g.dim + d];
+                k = a.qk[(tok * 2 + 1) * g.kv_heads * g.dim + kh * g.dim + d];
+                gg = expf(a.log_decay[tok * g.heads * g.dim + h * g.dim + d]);
+            }
+            s_q[i] = q; s_k[i] = k; s_g[i] = gg;
+        }
+        for (int i = threadIdx.x; i < m * 32; i += 128) {
+            const int t = i >> 5, c = blockIdx.z * 32 + (i & 31);
+            s_v[i] = c < g.vdim ? a.v[(size_t)(run.tok0 + c0 + t) * g.heads * g.vdim + h * g.vdim + c] : 0.0f;
+        }
+        if (threadIdx.x < m) s_b[threadIdx.x] = sigmoid_f(act_f<A>(proj[(size_t)(run.tok0 + c0 + threadIdx.x) * g.ld + g.off_b + h]));
+        __syncthreads();
+        for (int t = 0; t < m; t++) {
+            const float4 *q4 = (const float4*)(s_q + t * DP), *k4 = (const float4*)(s_k + t * DP), *g4 = (const float4*)(s_g + t * DP);
+            float kk[DPL], dot = 0.0f;
+#pragma unroll
+            for (int i = 0; i < DPL / 4; i++) {
+                const float4 kv = k4[i * 4 + r4], gv = g4[i * 4 + r4];
+                kk[4 * i] = kv.x; kk[4 * i + 1] = kv.y; kk[4 * i + 2] = kv.z; kk[4 * i + 3] = kv.w;
+                S[4 * i] *= gv.x; S[4 * i + 1] *= gv.y; S[4 * i + 2] *= gv.z; S[4 * i + 3] *= gv.w;
+#pragma unroll
+                for (int j = 0; j < 4; j++) dot = fmaf(S[4 * i + j], kk[4 * i + j], dot);
+            }
+            dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+            dot += __shfl_xor_sync(0xffffffffu, dot, 2);
+            const float u = s_b[t] * (s_v[t * 32 + col] - dot);
+            float o = 0.0f;
+#pragma unroll
+            for (int i = 0; i < DPL / 4; i++) {
+                const float4 qv = q4[i * 4 + r4];
+                const float qq[4] = {qv.x, qv.y, qv.z, qv.w};
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    S[4 * i + j] = fmaf(kk[4 * i + j], u, S[4 * i + j]);
+                    o = fmaf(S[4 * i + j], qq[j], o);
+                }
+            }
+            o += __shfl_xor_sync(0xffffffffu, o, 1);
+            o += __shfl_xor_sync(0xffffffffu, o, 2);
+            if (r4 == 0 && e < g.vdim) a.o[(size_t)(run.tok0 + c0 + t) * g.heads * g.vdim + h * g.vdim + e] = o;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < DPL; i++) {
+        const int d = (i >> 2) * 16 + r4 * 4 + (i & 3);
+        if (d < g.dim && e < g.vdim) st[(size_t)d * g.vdim + e] = S[i];
+    }
+    // the inputs of the last `taps` positions, for the convolutions of the next call (this head's v channels, and the q and k
+    // channels of its key head once)
+    if (blockIdx.z == 0) {
+        A* ring = (A*)a.ring + (size_t)run.seq * g.taps * g.channels;
+        const int m = min(run.n, g.taps), qk = h % rep == 0 ? 2 * g.dim : 0;
+        for (int i = threadIdx.x; i < m * (g.vdim + qk); i += 128) {
+            const int j = i / (g.vdim + qk), c = i - j * (g.vdim + qk);
+            int column, channel;
+            if (c < g.vdim) { column = g.off_v + h * g.vdim + c; channel = 2 * g.kv_heads * g.dim + h * g.vdim + c; }
+            else if (c < g.vdim + g.dim) { column = kh * g.dim + c - g.vdim; channel = column; }
+            else { column = g.off_k + kh * g.dim + c - g.vdim - g.dim; channel = g.kv_heads * g.dim + kh * g.dim + c - g.vdim - g.dim; }
+            const int t = run.n - 1 - j;
+            ring[(size_t)((run.pos0 + t) % g.taps) * g.channels + channel] = proj[(size_t)(run.tok0 + t) * g.ld + column];
+        }
+    }
+}
+
+// One warp per (token, head): o / rms(o) * norm * sigmoid(gate)
+template <typename A>
+__global__ void __launch_bounds__(256) delta_output_kernel(const DeltaArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const DeltaShape& g = a.g;
+    const int t = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (h >= g.heads) return;
+    const float* o = a.o + ((size_t)t * g.heads + h) * g.vdim;
+    const A* gate = (const A*)a.gate + ((size_t)t * g.heads + h) * g.vdim;
+    float ss = 0.0f;
+    for (int i = lane; i < g.vdim; i += 32) ss = fmaf(o[i], o[i], ss);
+    ss = warp_sum(ss);
+    const float r = 1.0f / sqrtf(ss / (float)g.vdim + g.eps);
+    A* dst = (A*)a.out + (size_t)t * a.ldo + h * g.vdim;
+    for (int i = lane; i < g.vdim; i += 32) dst[i] = to_act<A>(o[i] * r * a.norm_w[i] * sigmoid_f(act_f<A>(gate[i])));
+}
+
+// One new token of every sequence: convolutions, unit vectors, recurrence, norm and gate of one head of one token per CTA.
+// With G = diag(g):  dot = (G S)^T k,  u = beta (v - dot),  S' = G S + k u^T,  o = S'^T q = (G S)^T q + u (k . q), so the state
+// is walked once; a thread owns VEC neighbouring value columns and every `groups`-th key row, kept in registers (ROWS of
+// them; 0: re-read for the update).  The ring entry written here is not one that any head reads in this step.
+template <typename A, int VEC, int ROWS>
+__global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
+    extern __shared__ float sm[];
+    __shared__ float red[32], s_norm[3];
+    pdl_launch_dependents();
+    pdl_wait();
+    const DeltaShape& g = a.g;
+    const int h = blockIdx.x, t = blockIdx.y, rep = g.heads / g.kv_heads, kh = h / rep, seq = a.tok_seq[t], pos = a.tok_pos[t];
+    const int cols = g.vdim / VEC, groups = 256 / cols;
+    float *s_q = sm, *s_k = s_q + g.dim, *s_g = s_k + g.dim, *s_v = s_g + g.dim, *s_dk = s_v + g.vdim, *s_dq = s_dk + groups * g.vdim;
+    const A* proj = (const A*)a.proj + (size_t)t * g.ld;
+    A* ring = (A*)a.ring + (size_t)seq * g.taps * g.channels;
+    const int c = threadIdx.x % cols, gr = threadIdx.x / cols;
+    float* st = a.state + ((size_t)seq * g.heads + h) * g.dim * g.vdim + c * VEC;
+    const bool live = pos > 0, mine = gr < groups;
+    float S[ROWS > 0 ? ROWS : 1][VEC];
+    if (ROWS > 0 && mine) {  // the state's reads travel while the convolutions run
+#pragma unroll
+        for (int i = 0; i < ROWS; i++) {
+            const int d = gr + i * groups;
+#pragma unroll
+            for (int j = 0; j < VEC; j++) S[i][j] = 0.0f;
+            if (d < g.dim && live) {
+                if constexpr (VEC == 4) { const float4 v = *(const float4*)(st + (size_t)d * g.vdim); S[i][0] = v.x; S[i][1] = v.y; S[i][2] = v.z; S[i][3] = v.w; }
+                else S[i][0] = st[(size_t)d * g.vdim];
+            }
+        }
+    }
+    const int now = pos % g.taps;
+    for (int i = threadIdx.x; i < 2 * g.dim + g.vdim; i += 256) {
+        int column, channel;
+        bool owner = true;
+        float* dst;
+        if (i < 2 * g.dim) {
+            const bool is_k = i >= g.dim;
+            const int d = is_k ? i - g.dim : i;
+            column = (is_k ? g.off_k : 0) + kh * g.dim + d;
+            channel = (is_k ? g.kv_heads * g.dim : 0) + kh * g.dim + d;
+            owner = h % rep == 0;
+            dst = (is_k ? s_k : s_q) + d;
+        } else {
+            const int d = i - 2 * g.dim;
+            column = g.off_v + h * g.vdim + d;
+            channel = 2 * g.kv_heads * g.dim + h * g.vdim + d;
+            dst = s_v + d;
+        }
+        const A cur = proj[column];
+        float acc = 0.0f;
+        for (int j = g.taps - 1; j > 0; j--)
+            if (pos - j >= 0) acc = fmaf(a.conv[channel * g.taps + g.taps - 1 - j], act_f<A>(ring[(size_t)((pos - j) % g.taps) * g.channels + channel]), acc);
+        acc = fmaf(a.conv[channel * g.taps + g.taps - 1], act_f<A>(cur), acc);
+        *dst = silu32(acc);
+        if (owner) ring[(size_t)now * g.channels + channel] = cur;
+    }
+    for (int d = threadIdx.x; d < g.dim; d += 256) s_g[d] = expf(a.log_decay[(size_t)t * g.heads * g.dim + h * g.dim + d]);
+    __syncthreads();
+    if (threadIdx.x < 96) {  // |q|^2, |k|^2, q . k
+        const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
+        const float *x = w == 1 ? s_k : s_q, *y = w == 0 ? s_q : s_k;
+        float v = 0.0f;
+        for (int d = lane; d < g.dim; d += 32) v = fmaf(x[d], y[d], v);
+        v = warp_sum(v);
+        if (lane == 0) s_norm[w] = v;
+    }
+    __syncthreads();
+    const float rq = 1.0f / sqrtf(s_norm[0] + g.unit_eps) * (1.0f / sqrtf((float)g.dim)), rk = 1.0f / sqrtf(s_norm[1] + g.unit_eps), qk = s_norm[2] * rq * rk;
+    const float beta = sigmoid_f(act_f<A>(proj[g.off_b + h]));
+    float dk[VEC], dq[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; j++) dk[j] = dq[j] = 0.0f;
+    auto load = [&](int d, float (&v)[VEC]) {
+#pragma unroll
+        for (int j = 0; j < VEC; j++) v[j] = live ? st[(size_t)d * g.vdim + j] : 0.0f;
+    };
+    if (mine) {
+        if constexpr (ROWS > 0) {
+#pragma unroll
+            for (int i = 0; i < ROWS; i++) {
+                const int d = gr + i * groups;
+                if (d < g.dim) {
+                    const float gg = s_g[d], k = s_k[d] * rk, q = s_q[d] * rq;
+#pragma unroll
+                    for (int j = 0; j < VEC; j++) { S[i][j] *= gg; dk[j] = fmaf(S[i][j], k, dk[j]); dq[j] = fmaf(S[i][j], q, dq[j]); }
+                }
+            }
+        } else {
+            for (int d = gr; d < g.dim; d += groups) {
+                const float gg = s_g[d], k = s_k[d] * rk, q = s_q[d] * rq;
+                float v[VEC];
+                load(d, v);
+#pragma unroll
+                for (int j = 0; j < VEC; j++) { v[j] *= gg; dk[j] = fmaf(v[j], k, dk[j]); dq[j] = fmaf(v[j], q, dq[j]); }
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < VEC; j++) { s_dk[gr * g.vdim + c * VEC + j] = dk[j]; s_dq[gr * g.vdim + c * VEC + j] = dq[j]; }
+    }
+    __syncthreads();
+    float ss = 0.0f;
+    for (int e = threadIdx.x; e < g.vdim; e += 256) {  // u replaces v, the read-out replaces the first partial row
+        float sk = 0.0f, sq = 0.0f;
+        for (int i = 0; i < groups; i++) { sk += s_dk[i * g.vdim + e]; sq += s_dq[i * g.vdim + e]; }
+        const float u = beta * (s_v[e] - sk), o = fmaf(u, qk, sq);
+        s_v[e] = u;
+        s_dq[e] = o;
+        ss = fmaf(o, o, ss);
+    }
+    ss = block_sum(ss, red);  // also publishes u and o
+    if (mine) {
+        float u[VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; j++) u[j] = s_v[c * VEC + j];
+        if constexpr (ROWS > 0) {
+#pragma unroll
+            for (int i = 0; i < ROWS; i++) {
+                const int d = gr + i * groups;
+                if (d < g.dim) {
+                    const float k = s_k[d] * rk;
+#pragma unroll
+                    for (int j = 0; j < VEC; j++) S[i][j] = fmaf(k, u[j], S[i][j]);
+                    if constexpr (VEC == 4) *(float4*)(st + (size_t)d * g.vdim) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+                    else st[(size_t)d * g.vdim] = S[i][0];
+                }
+            }
+        } else {
+            for (int d = gr; d < g.dim; d += groups) {
+                float v[VEC];
+                load(d, v);
+#pragma unroll
+                for (int j = 0; j < VEC; j++) st[(size_t)d * g.vdim + j] = fmaf(s_k[d] * rk, u[j], v[j] * s_g[d]);
+            }
+        }
+    }
+    const float r = 1.0f / sqrtf(ss / (float)g.vdim + g.eps);
+    const A* gate = (const A*)a.gate + ((size_t)t * g.heads + h) * g.vdim;
+    A* dst = (A*)a.out + (size_t)t * a.ldo + h * g.vdim;
+    for (int e = threadIdx.x; e < g.vdim; e += 256) dst[e] = to_act<A>(s_dq[e] * r * a.norm_w[e] * sigmoid_f(act_f<A>(gate[e])));
+}
+
+// ---- latent attention: norms of the two latents, rotation of the shared key part, cache append -------------------------------
+__global__ void rot_table_kernel(const double* __restrict__ freq, int pairs, double magnitude, int positions, float2* __restrict__ out) {
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= positions * pairs) return;
+    const int p = i / pairs;
+    double s, c;
+    sincos((double)p * freq[i - p * pairs], &s, &c);
+    out[i] = make_float2((float)(c * magnitude), (float)(s * magnitude));
+}
+
+template <typename A>
+__global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a) {
+    __shared__ float sh[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const LatentShape& g = a.g;
+    const int t = blockIdx.x, seq = a.tok_seq[t], pos = a.tok_pos[t];
+    const float* p = a.proj + (size_t)t * a.ld_proj;
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) ss = fmaf(p[i], p[i], ss);
+    ss = block_sum(ss, sh);
+    float r = 1.0f / sqrtf(ss / (float)a.q_rank + a.eps);
+    A* cq = (A*)a.cq + (size_t)t * a.ld_cq;
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) cq[i] = to_act<A>(p[i] * r * a.q_norm[i]);
+    __syncthreads();
+    const float* c = p + a.off_c;
+    ss = 0.0f;
+    for (int i = threadIdx.x; i < g.rank; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
+    ss = block_sum(ss, sh);
+    r = 1.0f / sqrtf(ss / (float)g.rank + a.eps);
+    const int page = a.page_table[(size_t)seq * a.pages_per_seq + pos / a.page_tokens];
+    A* row = (A*)a.cache + ((size_t)page * a.page_tokens + pos % a.page_tokens) * (g.cp + g.rp);
+    for (int i = threadIdx.x; i < g.cp; i += blockDim.x) row[i] = to_act<A>(i < g.rank ? c[i] * r * a.c_norm[i] : 0.0f);
+    const float* kr = p + a.off_r;
+    for (int i = threadIdx.x; i < g.rp; i += blockDim.x) {
+        float v = i < g.rot ? kr[i] : 0.0f;
+        if (i < 2 * g.rot_pairs) {
+            const float2 cs = a.rot[(size_t)pos * g.rot_pairs + i / 2];
+            const float u = kr[i & ~1], w = kr[i | 1];
+            v = (i & 1) ? w * cs.x + u * cs.y : u * cs.x - w * cs.y;
+        }
+        row[g.cp + i] = to_act<A>(v);
+    }
+}
+
+int norm_threads(int width) { return width >= 2048 ? 512 : width >= 512 ? 256 : 128; }
+
+template <typename A>
+int32_t scan_dispatch(const DeltaArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)a.n_runs, (unsigned)a.g.heads, (unsigned)((a.g.vdim + 31) / 32));
+    const int dpl = a.g.dim <= 32 ? 8 : a.g.dim <= 64 ? 16 : a.g.dim <= 128 ? 32 : 64;
+    const size_t smem = (size_t)kScanTok * (3 * 4 * dpl + 32 + 1) * sizeof(float);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+        LC_CUDA(launch_pdl(kern, grid, dim3(128), smem, s, a));
+        return LC_OK;
+    };
+    switch (dpl) {
+        case 8: return go(delta_scan_kernel<A, 8>);
+        case 16: return go(delta_scan_kernel<A, 16>);
+        case 32: return go(delta_scan_kernel<A, 32>);
+        default: return go(delta_scan_kernel<A, 64>);
+    }
+}
+
+template <typename A>
+int32_t step_dispatch(const DeltaArgs& a, cudaStream_t s) {
+    const int vec = a.g.vdim % 4 == 0 ? 4 : 1, cols = a.g.vdim / vec;
+    LC_CHECK(cols <= 256, LC_ERR_UNSUPPORTED, "delta rule: %d value dimensions per head", a.g.vdim);
+    const int groups = 256 / cols, rows = (a.g.dim + groups - 1) / groups;
+    const size_t smem = (size_t)(3 * a.g.dim + a.g.vdim + 2 * groups * a.g.vdim) * sizeof(float);
+    const dim3 grid((unsigned)a.g.heads, (unsigned)a.T);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+        LC_CUDA(launch_pdl(kern, grid, dim3(256), smem, s, a));
+        return LC_OK;
+    };
+    if (vec == 4) return rows <= 4 ? go(delta_step_kernel<A, 4, 4>) : rows <= 16 ? go(delta_step_kernel<A, 4, 16>) : go(delta_step_kernel<A, 4, 0>);
+    return rows <= 16 ? go(delta_step_kernel<A, 1, 16>) : go(delta_step_kernel<A, 1, 0>);
+}
+
+}  // namespace
+
+int32_t launch_pack(const __nv_bfloat16* src, int rows, int cols, __nv_bfloat16* dst, int ld, PackMap row, PackMap col, bool transpose, cudaStream_t s) {
+    const size_t n = (size_t)rows * cols, blocks = (n + 255) / 256;
+    pack_kernel<<<(unsigned)std::min<size_t>(blocks, (size_t)sm_count() * 16), 256, 0, s>>>(src, rows, cols, dst, ld, row, col, transpose ? 1 : 0);
+    LC_CUDA(cudaGetLastError());
+    return LC_OK;
+}
+int32_t launch_embed_rows(const __nv_bfloat16* table, int rows, int width, const int64_t* ids, int T, float* x, void* act, int ld_act, cudaStream_t s) {
+    LC_CUDA(launch_pdl(embed_rows_kernel, dim3((unsigned)T), dim3(256), 0, s, table, rows, width, ids, x, (__nv_bfloat16*)act, ld_act));
+    return LC_OK;
+}
+int32_t launch_act_rows(const float* x, int width, int T, void* act, int ld_act, cudaStream_t s) {
+    LC_CUDA(launch_pdl(act_rows_kernel, dim3((unsigned)T), dim3(256), 0, s, x, width, (__nv_bfloat16*)act, ld_act));
+    return LC_OK;
+}
+int32_t launch_norm_residual(const float* y, const float* w, float eps, int width, int T, float* x, void* act, int ld_act, cudaStream_t s) {
+    LC_CUDA(launch_pdl(norm_residual_kernel, dim3((unsigned)T), dim3((unsigned)norm_threads(width)), 0, s, y, w, eps, width, x, (__nv_bfloat16*)act, ld_act));
+    return LC_OK;
+}
+int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, float eps, int width, int n, void* out, int ldo, bool f32, cudaStream_t s) {
+    const dim3 grid((unsigned)n), block((unsigned)norm_threads(width));
+    if (f32) LC_CUDA(launch_pdl(norm_rows_kernel<float>, grid, block, 0, s, x, idx, w, eps, width, (float*)out, ldo));
+    else LC_CUDA(launch_pdl(norm_rows_kernel<__nv_bfloat16>, grid, block, 0, s, x, idx, w, eps, width, (__nv_bfloat16*)out, ldo));
+    return LC_OK;
+}
+int32_t launch_delta_prep(const DeltaArgs& a, cudaStream_t s) {
+    LC_CHECK(a.g.dim <= 256, LC_ERR_UNSUPPORTED, "delta rule: %d key dimensions per head (at most 256)", a.g.dim);
+    const dim3 grid((unsigned)a.T, (unsigned)((2 * a.g.kv_heads + a.g.heads + 7) / 8));
+    if (a.f32) LC_CUDA(launch_pdl(delta_prep_kernel<float>, grid, dim3(256), 0, s, a));
+    else LC_CUDA(launch_pdl(delta_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, a));
+    return LC_OK;
+}
+int32_t launch_delta_scan(const DeltaArgs& a, cudaStream_t s) { return a.f32 ? scan_dispatch<float>(a, s) : scan_dispatch<__nv_bfloat16>(a, s); }
+int32_t launch_delta_step(const DeltaArgs& a, cudaStream_t s) { return a.f32 ? step_dispatch<float>(a, s) : step_dispatch<__nv_bfloat16>(a, s); }
+int32_t launch_delta_output(const DeltaArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)a.T, (unsigned)((a.g.heads + 7) / 8));
+    if (a.f32) LC_CUDA(launch_pdl(delta_output_kernel<float>, grid, dim3(256), 0, s, a));
+    else LC_CUDA(launch_pdl(delta_output_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, a));
+    return LC_OK;
+}
+int32_t launch_latent_prep(const LatentArgs& a, cudaStream_t s) {
+    if (a.f32) LC_CUDA(launch_pdl(latent_prep_kernel<float>, dim3((unsigned)a.T), dim3(256), 0, s, a));
+    else LC_CUDA(launch_pdl(latent_prep_kernel<__nv_bfloat16>, dim3((unsigned)a.T), dim3(256), 0, s, a));
+    return LC_OK;
+}
+int32_t launch_rot_table(const double* freq_dev, int pairs, double magnitude, int positions, float2* out, cudaStream_t s) {
+    const size_t n = (size_t)pairs * positions;
+    LC_CHECK(n < ((size_t)1 << 31), LC_ERR_UNSUPPORTED, "rotation table of %zu entries", n);
+    rot_table_kernel<<<(unsigned)((n + 255) / 256), 256, 0, s>>>(freq_dev, pairs, magnitude, positions, out);
+    LC_CUDA(cudaGetLastError());
+    return LC_OK;
+}
+
+}  // namespace lc

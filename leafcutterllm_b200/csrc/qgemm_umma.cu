@@ -43,6 +43,7 @@
 #include "lc_kernels.h"
 #include "lc_quant.cuh"
 #include "lc_tma.cuh"
+#include "lc_umma.cuh"
 
 namespace lc {
 
@@ -81,16 +82,6 @@ struct GemmParams {
 };
 
 // ---- tcgen05 wrappers -------------------------------------------------------------------------------------------------
-// Shared-memory operand descriptor, K-major, 128-byte swizzle: start address and the byte distance between 8-row groups
-// in 16-byte units, descriptor version 1, layout code 2.
-__device__ __forceinline__ uint64_t umma_desc_sw128(uint32_t saddr) {
-    uint64_t d = (uint64_t)((saddr >> 4) & 0x3FFFu);
-    d |= (uint64_t)1 << 16;                 // leading byte offset: unused with a swizzled K-major tile
-    d |= (uint64_t)(1024u >> 4) << 32;      // stride byte offset: 8 rows x 128 B
-    d |= (uint64_t)1 << 46;
-    d |= (uint64_t)2 << 61;
-    return d;
-}
 // f32 accumulate, f16 x f16, both K-major, M = 128
 __host__ __device__ constexpr uint32_t idesc_f16(int n_tok) {
     return (1u << 4) | (0u << 7) | (0u << 10) | ((uint32_t)(n_tok >> 3) << 17) | ((uint32_t)(kRows >> 4) << 24);
@@ -110,22 +101,6 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* r) {
         "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
         : "memory");
 }
-__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t* r) {
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
-        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
-          "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-        : "r"(taddr));
-}
-__device__ __forceinline__ void umma_commit(uint64_t* bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
-    asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-
 // ---- unpacking ---------------------------------------------------------------------------------------------------------
 struct HdrQ4K { float d, dmin; uint32_t sc_lo, sc_hi, mn_lo, mn_hi; };
 __device__ __forceinline__ void load_hdr(const unsigned char* rp, HdrQ4K& h) {

@@ -21,6 +21,7 @@
 #include "lc_kernels.h"
 #include "lc_quant.cuh"
 #include "lc_tma.cuh"
+#include "lc_umma.cuh"
 
 namespace lc {
 
@@ -98,6 +99,18 @@ bool make_key_pool_tmap(void* out128, const void* pool, uint64_t rows) {
     cuuint32_t box[2] = {64, 16};
     cuuint32_t estr[2] = {1, 1};
     CUresult r = encode_fn()((CUtensorMap*)out128, CU_TENSOR_MAP_DATA_TYPE_UINT16, 2, (void*)pool, dims, strides, box, estr,
+                             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r == CUDA_SUCCESS;
+}
+
+bool make_bf16_tmap_3d(void* out128, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1, uint64_t s2, uint32_t b0, uint32_t b1, uint32_t b2) {
+    if (!encode_fn() || ((uintptr_t)base % 16) != 0 || s1 % 8 != 0 || s2 % 8 != 0 || b0 * 2 != 128 || b1 > 256 || b2 > 256) return false;
+    cuuint64_t dims[3] = {d0, d1, d2};
+    cuuint64_t strides[2] = {s1 * 2, s2 * 2};
+    cuuint32_t box[3] = {b0, b1, b2};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = encode_fn()((CUtensorMap*)out128, CU_TENSOR_MAP_DATA_TYPE_UINT16, 3, (void*)base, dims, strides, box, estr,
                              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
                              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     return r == CUDA_SUCCESS;

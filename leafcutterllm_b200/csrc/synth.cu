@@ -8,7 +8,7 @@
 namespace lc {
 
 static bool synth_has_quantiser(uint32_t typ) {
-    return typ == LC_TYPE_F32 || typ == LC_TYPE_F16 || typ == LC_TYPE_Q4_0 || typ == LC_TYPE_Q8_0 || typ == LC_TYPE_Q4_K || typ == LC_TYPE_Q5_K ||
+    return typ == LC_TYPE_F32 || typ == LC_TYPE_F16 || typ == LC_TYPE_BF16 || typ == LC_TYPE_Q4_0 || typ == LC_TYPE_Q8_0 || typ == LC_TYPE_Q4_K || typ == LC_TYPE_Q5_K ||
            typ == LC_TYPE_Q6_K;
 }
 

@@ -7,6 +7,7 @@ and sized (rust/src/cache/mod.rs).  Weights arrive as raw GGUF blocks and stay o
 from __future__ import annotations
 
 import ctypes as C
+import json
 from typing import Callable, Iterable, Optional, Sequence
 
 import numpy as np
@@ -58,6 +59,44 @@ class Engine:
         self.vocab_size = cfg.vocab_size
         self.max_seqs = max(1, cfg.max_seqs)
         return self
+
+    @classmethod
+    def _adopt(cls, handle, max_seqs: int) -> "Engine":
+        self = cls.__new__(cls)
+        self._h = handle
+        cfg = ModelConfig()
+        check(load().lc_model_get_config(handle, C.byref(cfg)))
+        self.cfg = cfg
+        self.vocab_size = cfg.vocab_size
+        self.max_seqs = max(1, max_seqs)
+        return self
+
+    @staticmethod
+    def _stack_overrides(max_seq_len, max_seqs, kv_page_tokens, kv_pool_tokens, device, dtype) -> ModelConfig:
+        over = ModelConfig()
+        over.max_seq_len, over.max_seqs, over.kv_page_tokens = max_seq_len, max_seqs, kv_page_tokens
+        over.kv_pool_tokens, over.device = kv_pool_tokens, device
+        over.compute_f32 = {"bfloat16": 0, "float32": 1}[dtype]
+        return over
+
+    @classmethod
+    def load_dir(cls, path: str, max_seq_len: int = 0, max_seqs: int = 1, kv_page_tokens: int = 16, kv_pool_tokens: int = 0,
+                 device: int = 0, dtype: str = "bfloat16") -> "Engine":
+        """A checkpoint directory (config.json + model.safetensors); the config's "architecture" selects the design.
+        dtype "float32" runs activations, cache and products in true 32-bit."""
+        over = cls._stack_overrides(max_seq_len, max_seqs, kv_page_tokens, kv_pool_tokens, device, dtype)
+        h = C.c_void_p()
+        check(load().lc_model_load_dir(str(path).encode(), C.byref(over), C.byref(h)))
+        return cls._adopt(h, max_seqs)
+
+    @classmethod
+    def from_config(cls, config: dict, max_seq_len: int = 0, max_seqs: int = 1, kv_page_tokens: int = 16, kv_pool_tokens: int = 0,
+                    device: int = 0, dtype: str = "bfloat16") -> "Engine":
+        """The same from a parsed config.json; the tensors follow (set_tensor / synth_tensor), then finalize()."""
+        over = cls._stack_overrides(max_seq_len, max_seqs, kv_page_tokens, kv_pool_tokens, device, dtype)
+        h = C.c_void_p()
+        check(load().lc_model_create_json(json.dumps(config).encode(), C.byref(over), C.byref(h)))
+        return cls._adopt(h, max_seqs)
 
     @staticmethod
     def group(engines: Sequence["Engine"]) -> "Engine":
@@ -117,6 +156,30 @@ class Engine:
         logits = np.empty((n, self.vocab_size), np.float32) if want_logits else None
         nxt = np.empty(n, np.int64)
         check(load().lc_forward_batch(self._h, n, _p(ids), _p(flat), _p(counts), _p(logits) if want_logits else None, _p(nxt)))
+        return logits, nxt
+
+    # ---- batches of sequences that come and go ------------------------------
+    def open_sequence(self) -> int:
+        """A free sequence slot; raises LeafcutterError (LC_ERR_KV_FULL) when all are taken."""
+        out = C.c_int32()
+        check(load().lc_seq_open(self._h, C.byref(out)))
+        return out.value
+
+    def close_sequence(self, seq_id: int) -> None:
+        """Gives back the slot with its cache pages and state."""
+        check(load().lc_seq_close(self._h, seq_id))
+
+    def step(self, seq_ids: Sequence[int], token_lists: Sequence[Sequence[int]], want: Sequence[Sequence[int]]):
+        """The next tokens of several sequences as one batch; logits (and greedy picks) at the wanted places of each list."""
+        ids = np.ascontiguousarray(seq_ids, dtype=np.int32)
+        counts = np.ascontiguousarray([len(t) for t in token_lists], dtype=np.int32)
+        flat = np.ascontiguousarray([x for t in token_lists for x in t], dtype=np.int64)
+        n_want = np.ascontiguousarray([len(w) for w in want], dtype=np.int32)
+        places = np.ascontiguousarray([x for w in want for x in w] + [0], dtype=np.int32)
+        rows = int(n_want.sum())
+        logits = np.empty((rows, self.vocab_size), np.float32)
+        nxt = np.empty(rows, np.int64)
+        check(load().lc_step(self._h, len(seq_ids), _p(ids), _p(flat), _p(counts), _p(n_want), _p(places), _p(logits), _p(nxt)))
         return logits, nxt
 
     def generate(self, tokens: Iterable[int], max_tokens: int, temperature: float = 0.0, top_p: float = 1.0,
