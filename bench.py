@@ -299,6 +299,57 @@ def moe_decode(lc, synth, local: int, n_seqs: int = 16, prompt_len: int = 1024, 
     return out
 
 
+def layered_leg(lc, synth, local: int, sizes=("1b", "7b"), prompt_len: int = PROMPT_LEN, steps: int = 32, batches=(1, 16, 64), llama: bool = True, pattern: str = "") -> dict:
+    """Varasun-shaped models (gated delta rule and latent attention layers, bf16, random weights) beside Llama-shaped models of
+    the same width, depth, heads and FFN width (16-bit and Q4_K weights): prefill of one prompt and decode steps at several
+    batch sizes, all contexts of prompt_len tokens.  The weights of a step exceed L2, so nothing is flushed between steps."""
+    peak, which = measured_peaks()
+    shapes = {"1b": dict(width=2048, heads=16, ff=5632, q_rank=768), "7b": dict(width=4096, heads=32, ff=11008, q_rank=1536)}
+    pattern = pattern or "dddaddda"
+    out = {"prompt_len": prompt_len, "pattern": pattern, "peak_gbs": peak, "peak_source": which}
+
+    def measure(build, vocab):
+        r = {}
+        for b in batches:
+            eng = build(b)
+            ctr0 = None
+            first = []
+            for s_ in range(b):  # the first prompt pays for kernel images: with one sequence it runs twice
+                prompt = synth.prompt_tokens(prompt_len, vocab, s_).tolist()
+                if s_ == 0:
+                    eng.forward_batch([0], [prompt], want_logits=False)
+                    eng.kv_clear(0)
+                    lc._capi.check(lc.load().lc_timer_begin())
+                _, nxt = eng.forward_batch([s_], [prompt], want_logits=False)
+                if s_ == 0:
+                    import ctypes as C
+                    ms = C.c_float()
+                    lc._capi.check(lc.load().lc_timer_end(C.byref(ms)))
+                    r.setdefault("prefill_tok_s", round(prompt_len / (ms.value * 1e-3), 1))
+                first.append(int(nxt[0]))
+            ids = list(range(b))
+            toks, _ = eng.decode_loop(ids, first, 3)
+            eng.reset_counters()
+            toks, ms = eng.decode_loop(ids, toks[-1].tolist(), steps)
+            ctr0 = eng.counters()
+            eng.close()
+            gbs = ctr0["algo_bytes_last_step"] / (ms / steps * 1e-3) / 1e9
+            r[f"decode_b{b}"] = {"ms_per_step": round(ms / steps, 4), "tok_s": round(b * steps / (ms * 1e-3), 1), "gbs": round(gbs, 1), "frac": round(gbs / peak, 3),
+                                 "launches_per_step": round(ctr0["kernel_launches"] / steps, 1)}
+        return r
+
+    cap = prompt_len + steps + 16
+    for size in sizes:
+        sh = shapes[size]
+        spec = synth.layered_spec(size, sh["width"], pattern, sh["ff"], 32000, sh["heads"], q_rank=sh["q_rank"])
+        out[size] = {"varasun": measure(lambda b: synth.build_layered_engine(spec, max_seq_len=cap, max_seqs=b, device=local), 32000)}
+        if llama:
+            for tag, typ in (("llama_f16", lc.TYPE_F16), ("llama_q4k", lc.TYPE_Q4_K)):
+                ls = synth.ModelSpec(size + tag, len(pattern), sh["width"], sh["heads"], sh["heads"], sh["ff"], 32000, 10000.0, typ, typ, typ)
+                out[size][tag] = measure(lambda b: synth.build_engine(ls, cap, on_device=True, device=local, max_seqs=b, rope_mode="absolute"), 32000)
+    return out
+
+
 def gemv_sweep(lc) -> dict:
     """Q4_K GEMV (one token) timed alone for a range of row counts: back-to-back launches over >= 600 MB of distinct
     weights per shape, CUDA events on the library's stream.  Shows the streaming rate and the fixed cost per launch."""
@@ -800,9 +851,13 @@ def main():
     ap.add_argument("--no-bs64", action="store_true", help="skip the 64-sequence continuous-batching leg (configs[2])")
     ap.add_argument("--no-extra", action="store_true", help="skip the legs after the metric: configs[0], configs[3] (one GPU), the cut 70B / mixture models (several GPUs)")
     ap.add_argument("--ref-context", type=int, default=64, help="--impl reference: context of the sampled CPU run (the oracle's prefill is slow)")
-    ap.add_argument("--only", default="", choices=["", "gemv", "attn", "gemv-sweep", "gemv-types", "gemm", "gemm-small", "bs64", "moe", "tiny", "q4km", "tp-ranks", "tcgen05-probe"], help="gemv / attn: run just the isolated GEMV or decode-attention loop (small cases for profilers); gemv-sweep: GEMV time against row count; tp-ranks: the ranks of a cut 70B-shape model as one in-process group on one GPU (what each rank's kernels cost)")
+    ap.add_argument("--only", default="", choices=["", "gemv", "attn", "gemv-sweep", "gemv-types", "gemm", "gemm-small", "bs64", "moe", "tiny", "q4km", "tp-ranks", "tcgen05-probe", "layered"], help="gemv / attn: run just the isolated GEMV or decode-attention loop (small cases for profilers); gemv-sweep: GEMV time against row count; layered: Varasun-shaped models beside Llama-shaped ones of equal size; tp-ranks: the ranks of a cut 70B-shape model as one in-process group on one GPU (what each rank's kernels cost)")
     ap.add_argument("--gemm-shapes", default="", help="--only gemm: k x n pairs instead of the 7B layer shapes, e.g. 1024x12288,8192x12288")
     ap.add_argument("--gemm-tokens", default="", help="--only gemm: token counts instead of 64,512")
+    ap.add_argument("--layered-sizes", default="1b,7b", help="--only layered: which sizes")
+    ap.add_argument("--layered-batches", default="1,16,64", help="--only layered: sequences per decode step")
+    ap.add_argument("--layered-pattern", default="", help="--only layered: one letter per layer (d = gated delta rule, a = latent attention)")
+    ap.add_argument("--no-llama", action="store_true", help="--only layered: skip the Llama-shaped models")
     ap.add_argument("--tp", type=int, default=8, help="--only tp-ranks: ranks the model is cut over")
     ap.add_argument("--profile-range", action="store_true", help="bracket the timed decode loop with cudaProfilerStart/Stop")
     ap.add_argument("--layers", type=int, default=0, help="profiling only: keep this many of the 32 layers (the printed number is then not the metric)")
@@ -840,6 +895,12 @@ def main():
         shapes = [tuple(int(v) for v in sh.split("x")) for sh in args.gemm_shapes.split(",")] if args.gemm_shapes else None
         tokens = tuple(int(v) for v in args.gemm_tokens.split(",")) if args.gemm_tokens else ((64,) if args.only == "gemm-small" else (64, 512))
         print(json.dumps(gemm_microbench(lc, tokens=tokens, small=args.only == "gemm-small", shapes=shapes)))
+    elif args.only == "layered":
+        import leafcutterllm_b200 as lc
+        from leafcutterllm_b200 import synth
+        lc._capi.check(lc.load().lc_set_device(0))
+        print(json.dumps(layered_leg(lc, synth, 0, sizes=tuple(args.layered_sizes.split(",")), prompt_len=args.prompt_len, steps=min(args.steps, 32),
+                                     batches=tuple(int(v) for v in args.layered_batches.split(",")), llama=not args.no_llama, pattern=args.layered_pattern)))
     elif args.only == "tcgen05-probe":
         import ctypes as C
         import leafcutterllm_b200 as lc

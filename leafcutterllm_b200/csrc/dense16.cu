@@ -6,7 +6,7 @@
 //   warp 0   one thread requests TMA boxes of 64 elements of k x 128 weight rows and x N tokens (128-byte swizzle) into a
 //            ring of stages; the first weight boxes leave before the kernel waits for its predecessor;
 //   warp 1   one thread issues the products of a stage (four K = 16 steps) and commits them to the stage's "empty" barrier;
-//   warps 4-7  read finished accumulators (two sets, so the next tile's products overlap), apply the epilogue and store;
+//   warps 4-11  read finished accumulators (two sets, so the next tile's products overlap), apply the epilogue and store;
 //            lane = weight row, so a warp's store of one token is contiguous.
 // Few tiles: k is cut into shares over several CTAs; each leaves its partial tile in scratch and takes a ticket, the last one
 // adds the shares in share order (the result does not depend on which CTA that is) and runs the epilogue.
@@ -26,7 +26,8 @@ namespace {
 constexpr int kM = 128;          // weight rows per tile
 constexpr int kKB = 64;          // elements of k per stage
 constexpr int kABytes = kM * kKB * 2;
-constexpr int kThreads = 256;
+constexpr int kEpiWarps = 8;     // warps 4 .. 11: two per quarter of the rows, each with half of the tokens
+constexpr int kThreads = 128 + 32 * kEpiWarps;
 
 struct DenseParams {
     void* out;
@@ -41,34 +42,52 @@ struct DenseParams {
 };
 
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
-__device__ __forceinline__ float dense_epilogue(const DenseParams& p, int row, float y) {
+// ea, eb: the row's constants of the epilogue
+__device__ __forceinline__ float dense_epilogue(const DenseParams& p, float ea, float eb, float y) {
     switch (p.epi) {
         case DENSE_RELU2: { const float r = fmaxf(y, 0.0f); return r * r; }
-        case DENSE_LOG_DECAY: return -p.e0[row / p.e_div] * softplus_f(y + p.e1[row]);
+        case DENSE_LOG_DECAY: return -ea * softplus_f(y + eb);
         case DENSE_LOGITS: { const float v = y * p.scale; return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v; }
         default: return y;
     }
 }
-// 16 accumulators of weight row `row`, tokens t0 .. t0 + 15
-__device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int row, int t0, const float (&v)[16]) {
-    if (row >= p.n) return;
+__device__ __forceinline__ void dense_row_constants(const DenseParams& p, int row, float& ea, float& eb) {
+    ea = eb = 0.0f;
+    if (p.epi == DENSE_LOG_DECAY && row < p.n) { ea = p.e0[row / p.e_div]; eb = p.e1[row]; }
+}
+// 16 accumulators of weight row `row`, tokens t0 .. t0 + 15, for a whole warp (lane = row).  bf16: lane pairs swap halves, so
+// a lane stores two rows of every other token.
+__device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int row, int t0, const float (&v)[16], float ea, float eb) {
     const size_t at = (size_t)b * p.out_batch + (size_t)t0 * p.ldo + row;
     const int m = min(16, p.T - t0);
     if (p.out_f32) {
+        if (row >= p.n) return;
         float* o = (float*)p.out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * p.ldo] = dense_epilogue(p, row, v[j]);
+            if (j < m) o[(size_t)j * p.ldo] = dense_epilogue(p, ea, eb, v[j]);
+    } else if ((p.n & 1) == 0 && (p.ldo & 1) == 0) {  // row pairs stay inside the matrix and 4-byte aligned
+        const bool odd = row & 1;
+        __nv_bfloat16* o = (__nv_bfloat16*)p.out + at - (odd ? 1 : 0);
+#pragma unroll
+        for (int j = 0; j < 16; j += 2) {
+            const float x = dense_epilogue(p, ea, eb, v[j]), y = dense_epilogue(p, ea, eb, v[j + 1]);
+            const float other = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
+            const __nv_bfloat162 pr = odd ? __floats2bfloat162_rn(other, y) : __floats2bfloat162_rn(x, other);
+            const int jj = j + (odd ? 1 : 0);
+            if (jj < m && row < p.n) *(__nv_bfloat162*)(o + (size_t)jj * p.ldo) = pr;
+        }
     } else {
+        if (row >= p.n) return;
         __nv_bfloat16* o = (__nv_bfloat16*)p.out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * p.ldo] = __float2bfloat16_rn(dense_epilogue(p, row, v[j]));
+            if (j < m) o[(size_t)j * p.ldo] = __float2bfloat16_rn(dense_epilogue(p, ea, eb, v[j]));
     }
 }
 
 template <int NT>
-__global__ void __launch_bounds__(kThreads, 1)
+__global__ void __launch_bounds__(kThreads, NT <= 64 ? 2 : 1)
 dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx, const DenseParams p) {
     constexpr int kBBytes = NT * kKB * 2, kStage = kABytes + kBBytes;
     constexpr uint32_t kCols = NT < 32 ? 32 : NT;  // tensor-memory columns of one accumulator set
@@ -83,7 +102,7 @@ dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant_
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
         for (int i = 0; i < p.stages; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], 1); }
-        for (int i = 0; i < 2; i++) { mbar_init(&acc_full[i], 1); mbar_init(&acc_empty[i], 128); }
+        for (int i = 0; i < 2; i++) { mbar_init(&acc_full[i], 1); mbar_init(&acc_empty[i], 32 * kEpiWarps); }
         *stop = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
@@ -163,20 +182,23 @@ dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant_
         if (!ok) { *stop = 1; atomicExch(p.error_flag, 12); }
     } else if (warp >= 4) {
         pdl_wait();  // earlier kernels may still read what this one overwrites
-        const int ew = warp - 4, row_in = ew * 32 + lane;
+        constexpr int kHalf = NT >= 32 ? NT / 2 : NT;  // tokens of one warp; a 16-token tile leaves the second half idle
+        const int quarter = warp & 3, half = (warp - 4) >> 2, row_in = quarter * 32 + lane, c_lo = half * kHalf, c_hi = c_lo < NT ? c_lo + kHalf : c_lo;
         int tile = 0;
         for (int it = blockIdx.x; it < p.items; it += gridDim.x, tile++) {
             const Item r = item_of(it);
             const int set = tile & 1;
+            const int row = r.m * kM + row_in, t0 = r.n * NT;
+            float ea, eb;
+            dense_row_constants(p, row, ea, eb);
             if (!mbar_wait(&acc_full[set], (uint32_t)(tile / 2) & 1)) { *stop = 1; if (lane == 0) atomicExch(p.error_flag, 13); break; }
             tc_fence_after();
-            const uint32_t base = tmem + (uint32_t)set * kCols + ((uint32_t)(ew * 32) << 16);
-            const int row = r.m * kM + row_in, t0 = r.n * NT;
+            const uint32_t base = tmem + (uint32_t)set * kCols + ((uint32_t)(quarter * 32) << 16);
             const size_t plane = (size_t)NT * kM;
             const int cell = (r.b * p.mt + r.m) * p.nt + r.n;
             float* part = p.shares > 1 ? p.partial + (size_t)cell * p.shares * plane : nullptr;
 #pragma unroll 1
-            for (int c = 0; c < NT; c += 16) {
+            for (int c = c_lo; c < c_hi; c += 16) {
                 if (t0 + c >= p.T) break;
                 uint32_t raw[16];
                 tmem_ld16(base + c, raw);
@@ -185,37 +207,42 @@ dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant_
 #pragma unroll
                 for (int j = 0; j < 16; j++) v[j] = __uint_as_float(raw[j]);
                 if (part) {
+                    const int m = p.T - t0 - c;
 #pragma unroll
-                    for (int j = 0; j < 16; j++) part[(size_t)r.share * plane + (size_t)(c + j) * kM + row_in] = v[j];
+                    for (int j = 0; j < 16; j++)
+                        if (j < m) part[(size_t)r.share * plane + (size_t)(c + j) * kM + row_in] = v[j];
                 } else {
-                    dense_store16(p, r.b, row, t0 + c, v);
+                    dense_store16(p, r.b, row, t0 + c, v, ea, eb);
                 }
             }
             tc_fence_before();
             mbar_arrive(&acc_empty[set]);
             if (part) {
                 __threadfence();
-                asm volatile("bar.sync 1, 128;" ::: "memory");
+                asm volatile("bar.sync 1, %0;" ::"n"(32 * kEpiWarps) : "memory");
                 if (threadIdx.x == 128) {
                     const unsigned t = atomicAdd(&p.tickets[cell], 1u);
                     *last_share = t == (unsigned)(p.shares - 1);
                     if (*last_share) p.tickets[cell] = 0;
                     __threadfence();
                 }
-                asm volatile("bar.sync 1, 128;" ::: "memory");
+                asm volatile("bar.sync 1, %0;" ::"n"(32 * kEpiWarps) : "memory");
                 const bool mine = *last_share != 0;
-                asm volatile("bar.sync 1, 128;" ::: "memory");
+                asm volatile("bar.sync 1, %0;" ::"n"(32 * kEpiWarps) : "memory");
                 if (mine) {
 #pragma unroll 1
-                    for (int c = 0; c < NT; c += 16) {
+                    for (int c = c_lo; c < c_hi; c += 16) {
                         if (t0 + c >= p.T) break;
                         float v[16];
+                        const int m = p.T - t0 - c;
 #pragma unroll
-                        for (int j = 0; j < 16; j++) v[j] = 0.0f;
-                        for (int sh = 0; sh < p.shares; sh++)
-#pragma unroll
-                            for (int j = 0; j < 16; j++) v[j] += __ldcg(part + (size_t)sh * plane + (size_t)(c + j) * kM + row_in);
-                        dense_store16(p, r.b, row, t0 + c, v);
+                        for (int j = 0; j < 16; j++) {
+                            v[j] = 0.0f;
+                            if (j < m)
+#pragma unroll 4
+                                for (int sh = 0; sh < p.shares; sh++) v[j] += __ldcg(part + (size_t)sh * plane + (size_t)(c + j) * kM + row_in);
+                        }
+                        dense_store16(p, r.b, row, t0 + c, v, ea, eb);
                     }
                 }
             }
@@ -267,7 +294,11 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int row = r0 + tr + 16 * j;
-            if (row < p.n) ((float*)p.out)[(size_t)b * p.out_batch + (size_t)t * p.ldo + row] = dense_epilogue(p, row, acc[i][j]);
+            if (row < p.n) {
+                float ea, eb;
+                dense_row_constants(p, row, ea, eb);
+                ((float*)p.out)[(size_t)b * p.out_batch + (size_t)t * p.ldo + row] = dense_epilogue(p, ea, eb, acc[i][j]);
+            }
         }
     }
 }
@@ -275,7 +306,8 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
 template <int NT>
 int32_t launch_umma(const DenseArgs& a, const CUtensorMap& tx, DenseParams p, cudaStream_t s) {
     const size_t stage = kABytes + (size_t)NT * kKB * 2, fixed = 1024 + 512;
-    p.stages = (int)std::min<size_t>(12, (kMaxSmem - fixed) / stage);
+    // few tokens: half of the shared memory, so that the next kernel's first weight boxes travel while this one drains
+    p.stages = (int)((NT <= 64 ? kMaxSmem / 2 - 1024 : kMaxSmem) - fixed) / (int)stage;
     const size_t smem = fixed + (size_t)p.stages * stage;
     LC_CUDA(ensure_smem_limit((const void*)dense_umma_kernel<NT>, smem));
     const int grid = std::min(p.items, sm_count());
@@ -332,9 +364,13 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     p.nt = (a.T + NT - 1) / NT;
     const int cells = p.mt * p.nt * w.batch, sms = sm_count();
     p.shares = 1;
-    if (cells * 4 < sms * 3 && cells <= ws.max_tickets) {  // fewer tiles than three quarters of the SMs: cut k
-        p.shares = std::max(1, std::min(std::min(p.kblocks / 2, 16), sms / cells));
-        while (p.shares > 1 && (size_t)cells * p.shares * NT * kM * sizeof(float) > ws.partial_bytes) p.shares--;
+    if (NT <= 64 && cells <= ws.max_tickets) {  // cut k where that evens out the CTAs' work: k blocks of the busiest CTA, plus two per item
+        long best = -1;
+        for (int c = 1; c <= std::min(16, p.kblocks / 2); c++) {
+            if ((size_t)cells * c * NT * kM * sizeof(float) > ws.partial_bytes) break;
+            const long waves = ((long)cells * c + sms - 1) / sms, cost = waves * (((p.kblocks + c - 1) / c) + 2) + (c > 1 ? 3 : 0);
+            if (best < 0 || cost < best) { best = cost; p.shares = c; }
+        }
     }
     p.items = cells * p.shares;
     p.partial = ws.partial; p.tickets = ws.tickets;

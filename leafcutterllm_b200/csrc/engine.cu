@@ -480,16 +480,7 @@ int32_t upload_meta(lc_model* m, const std::vector<int64_t>& tok, const std::vec
         if (tiles.empty() || tiles.back().n == 64 || seq[i] != seq[i - 1] || pos[i] != pos[i - 1] + 1) tiles.push_back(PrefillTile{(int32_t)i, 0, seq[i], pos[i]});
         tiles.back().n++;
     }
-    if (m->stack) {  // the same runs uncut
-        std::vector<SeqRun> runs;
-        for (size_t i = 0; i < T; i++) {
-            if (runs.empty() || seq[i] != seq[i - 1] || pos[i] != pos[i - 1] + 1) runs.push_back(SeqRun{(int32_t)i, 0, seq[i], pos[i]});
-            runs.back().n++;
-        }
-        m->stack->n_runs = (int)runs.size();
-        LC_CUDA(cudaMemcpyAsync(m->stack->d_runs, runs.data(), runs.size() * sizeof(SeqRun), cudaMemcpyHostToDevice, m->stream));
-        LC_CUDA(cudaStreamSynchronize(m->stream));
-    }
+    if (m->stack) LC_TRY(stack_upload_runs(m, seq, pos));
     m->n_tiles = (int)tiles.size();
     if (!tiles.empty()) LC_CUDA(cudaMemcpyAsync(m->d_tiles, tiles.data(), tiles.size() * sizeof(PrefillTile), cudaMemcpyHostToDevice, m->stream));
     // the copies read pageable host vectors that die with the caller's frame
@@ -1182,20 +1173,37 @@ static int32_t run_step(lc_model* lead, int32_t n_seqs, const int32_t* seq_ids, 
     }
     for (lc_model* m : R) m->meta_valid = false;
     // Rotary index = position inside the CALL (reference mode, attention.rs:13-21) or the cache position.
-    std::vector<int64_t> tok(tokens, tokens + total);
+    // Sequences that bring few tokens run ahead of the others (the layers treat the two kinds differently); `rows` follows.
+    std::vector<int64_t> tok;
     std::vector<int32_t> seq, pos, rope;
-    for (int i = 0; i < n_seqs; i++)
-        for (int t = 0; t < n_tokens[i]; t++) {
-            const int p = lead->seq_len[seq_ids[i]] + t;
-            seq.push_back(seq_ids[i]); pos.push_back(p); rope.push_back(lead->cfg.rope_mode ? p : t);
+    std::vector<std::pair<int, int>> picks;  // (row of the reordered call, place in the caller's output), ascending by row
+    for (int pass = 0; pass < 2; pass++)
+        for (int i = 0, off = 0, w0 = 0; i < n_seqs; off += n_tokens[i], w0 += n_want ? n_want[i] : 1, i++) {
+            if ((n_tokens[i] >= kTileRun) != (pass == 1)) continue;
+            const int shift = (int)tok.size() - off, nw = n_want ? n_want[i] : 1;
+            for (int j = 0; j < nw; j++) picks.push_back({rows[w0 + j] + shift, w0 + j});
+            for (int t = 0; t < n_tokens[i]; t++) {
+                const int p = lead->seq_len[seq_ids[i]] + t;
+                tok.push_back(tokens[off + t]); seq.push_back(seq_ids[i]); pos.push_back(p); rope.push_back(lead->cfg.rope_mode ? p : t);
+            }
         }
-    size_t done = 0, held = 0;  // wanted rows that are on the host; rows in d_logits behind them
+    size_t done = 0, held = 0;  // picks that are on the host; rows in d_logits behind them
+    const size_t V = (size_t)lead->cfg.vocab_size;
+    std::vector<float> stage;
     auto flush = [&]() -> int32_t {
         if (held == 0) return LC_OK;
+        bool in_order = true;
+        for (size_t j = 1; j < held; j++) in_order = in_order && picks[done + j].second == picks[done].second + (int)j;
         if (next_out) LC_CUDA(cudaMemcpyAsync(lead->pin_next, lead->d_next, held * 8, cudaMemcpyDeviceToHost, lead->stream));
-        if (logits_out) LC_TRY(fetch_logits(lead, (int)held, logits_out + done * lead->cfg.vocab_size));
+        if (logits_out) {
+            if (!in_order) stage.resize(held * V);
+            LC_TRY(fetch_logits(lead, (int)held, in_order ? logits_out + (size_t)picks[done].second * V : stage.data()));
+        }
         LC_CUDA(cudaStreamSynchronize(lead->stream));
-        if (next_out) memcpy(next_out + done, lead->pin_next, held * 8);
+        for (size_t j = 0; j < held; j++) {
+            if (next_out) next_out[picks[done + j].second] = lead->pin_next[j];
+            if (logits_out && !in_order) memcpy(logits_out + (size_t)picks[done + j].second * V, stage.data() + j * V, V * 4);
+        }
         done += held;
         held = 0;
         return LC_OK;
@@ -1205,11 +1213,10 @@ static int32_t run_step(lc_model* lead, int32_t n_seqs, const int32_t* seq_ids, 
         const int T = std::min(lead->t_cap, total - c0);
         auto part = [&](auto& v) { return typename std::remove_reference<decltype(v)>::type(v.begin() + c0, v.begin() + c0 + T); };
         for (lc_model* m : R) LC_TRY(upload_meta(m, part(tok), part(seq), part(pos), part(rope), {}));
-        const bool all_last = total == n_seqs;
-        LC_TRY(run_layers(lead, T, all_last));
-        while (next_row < rows.size() && rows[next_row] < c0 + T) {
+        LC_TRY(run_layers(lead, T, false));
+        while (next_row < picks.size() && picks[next_row].first < c0 + T) {
             std::vector<int32_t> idx;
-            while (next_row < rows.size() && rows[next_row] < c0 + T && held + idx.size() < (size_t)lead->head_rows) idx.push_back(rows[next_row++] - c0);
+            while (next_row < picks.size() && picks[next_row].first < c0 + T && held + idx.size() < (size_t)lead->head_rows) idx.push_back(picks[next_row++].first - c0);
             for (lc_model* m : R) {
                 LC_CUDA(cudaMemcpyAsync(m->d_last_idx, idx.data(), idx.size() * 4, cudaMemcpyHostToDevice, m->stream));
                 LC_CUDA(cudaStreamSynchronize(m->stream));

@@ -1,7 +1,10 @@
 // Latent attention: every head's key is the projection of ONE cached latent per token (plus a rotated part all heads share) and
 // its value another projection of the same latent.  The key projection is moved onto the query and the value projection behind
-// the weighted sum, so the kernels here attend with `heads` queries per token over rows [latent | rotated part] of the paged
-// cache and return, per head, the weighted sum of latents.
+// the weighted sum, so for FEW tokens the kernels attend with `heads` queries per token over rows [latent | rotated part] of
+// the paged cache and return, per head, the weighted sum of latents.  For MANY tokens of a sequence that costs more than
+// projecting the context once: the latents are gathered, keys and values of all heads projected by two ordinary products, and
+// the prefill kernel attends over those.
+#include <algorithm>
 #include <cmath>
 #include "lc_mixers.h"
 #include "lc_tma.cuh"
@@ -73,20 +76,513 @@ __global__ void __launch_bounds__(kPlainThreads) latent_attention_plain_kernel(c
     for (int i = threadIdx.x; i < g.cp; i += kPlainThreads) out[i] = to_act<A>(s_o[i] / l);
 }
 
-}  // namespace
+// ---- tensor-core forms (bf16) -------------------------------------------------------------------------------------------
+typedef __nv_bfloat16 bf16;
+__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, int src_bytes) {  // src_bytes 0: zeros
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
+}
+__device__ __forceinline__ uint32_t pack2(float a, float b) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+// (a, b) as a bf16 pair and the pair of what that rounding lost: the weights keep 16 bits of mantissa in the two products
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = pack2(a - __low2float(h), b - __high2float(h));
+}
+// element i of a rotated part whose row starts at r
+__device__ __forceinline__ float rotated(const bf16* r, const float2* tab, int pairs, int n, int i) {
+    if (i >= n) return 0.0f;
+    if (i >= 2 * pairs) return __bfloat162float(r[i]);
+    const float2 cs = tab[i / 2];
+    const float u = __bfloat162float(r[i & ~1]), w = __bfloat162float(r[i | 1]);
+    return (i & 1) ? w * cs.x + u * cs.y : u * cs.x - w * cs.y;
+}
+constexpr int kKeys = 64;  // keys per tile
 
-int32_t launch_latent_attention(const LatentArgs& a, cudaStream_t s) {
+// Few tokens per sequence: the queries of 16 * MT heads of ONE token are the rows of the products, the cached rows (latent |
+// rotated part) the keys and, without the rotated part, the values.  Eight warps: for the scores each takes one row tile and
+// 8 * MT keys, for the weighted sum all rows and 8 * NCT latent columns.  The context is cut into gridDim.z pieces.
+struct LatentPieces { float *o, *ml; };  // [token][piece][heads][cp] sums, [token][piece][heads][2] maximum (log2 units) and weight sum
+template <int MT, int NCT>
+__global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, const LatentPieces pc) {
+    constexpr int KG = 8 / MT, ROWS = 16 * MT;
+    extern __shared__ __align__(128) unsigned char smem[];
+    const LatentShape& g = a.g;
+    const int d = g.cp + g.rp, d32 = (d + 31) & ~31, pitch = d32 + 8, row_bytes = pitch * 2;
+    bf16 *s_q = (bf16*)smem, *s_k = s_q + ROWS * pitch, *s_ph = s_k + 2 * kKeys * pitch, *s_pl = s_ph + ROWS * (kKeys + 8);
+    float *s_wmax = (float*)(s_pl + ROWS * (kKeys + 8)), *s_wsum = s_wmax + ROWS * KG, *s_m = s_wsum + ROWS * KG, *s_l = s_m + 2 * ROWS;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+    const int t = blockIdx.x, h0 = blockIdx.y * ROWS, nh = min(ROWS, g.heads - h0);
+    pdl_launch_dependents();
+    pdl_wait();
+    const int seq = a.tok_seq[t], pos = a.tok_pos[t], pieces = gridDim.z;
+    const int tiles = pos / kKeys + 1, per = (tiles + pieces - 1) / pieces, kt0 = blockIdx.z * per, kt1 = min(tiles, kt0 + per);
+    const size_t out_row = ((size_t)t * pieces + blockIdx.z) * g.heads;
+    if (kt0 >= kt1) {
+        for (int i = tid; i < nh; i += 256) { pc.ml[(out_row + h0 + i) * 2] = -INFINITY; pc.ml[(out_row + h0 + i) * 2 + 1] = 0.0f; }
+        return;
+    }
+    const int32_t* pt = a.page_table + (size_t)seq * a.pages_per_seq;
+    const bf16* cache = (const bf16*)a.cache;
+    const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), ph_sm = smem_u32(s_ph), pl_sm = smem_u32(s_pl);
+    const int chunks = d / 8;
+    auto load = [&](int kt, int buf) {
+        for (int key = warp; key < kKeys; key += 8) {
+            const int kp = kt * kKeys + key;
+            const bool ok = kp <= pos;
+            const bf16* src = cache + ((size_t)(ok ? pt[kp / a.page_tokens] : 0) * a.page_tokens + kp % a.page_tokens) * d;
+            for (int c = lane; c < chunks; c += 32) cp16(k_sm + (uint32_t)((buf * kKeys + key) * row_bytes + c * 16), ok ? src + c * 8 : cache, ok ? 16 : 0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    load(kt0, 0);
+    for (int i = tid; i < 2 * kKeys * (pitch - d); i += 256) s_k[(i / (pitch - d)) * pitch + d + i % (pitch - d)] = __float2bfloat16_rn(0.0f);
+    for (int i = tid; i < ROWS * pitch; i += 256) {
+        const int r = i / pitch, c = i - r * pitch;
+        bf16 v = __float2bfloat16_rn(0.0f);
+        if (r < nh) {
+            const size_t th = (size_t)t * g.heads + h0 + r;
+            if (c < g.rank) v = ((const bf16*)a.q_abs)[th * g.cp + c];
+            else if (c >= g.cp && c < d) v = __float2bfloat16_rn(rotated((const bf16*)a.q + th * g.ld_q + g.dp, a.rot + (size_t)pos * g.rot_pairs, g.rot_pairs, g.rot, c - g.cp));
+        }
+        s_q[i] = v;
+    }
+    if (tid < ROWS) { s_m[tid] = -INFINITY; s_l[tid] = 0.0f; }
+    float o[MT][NCT][4];
+#pragma unroll
+    for (int i = 0; i < MT; i++)
+#pragma unroll
+        for (int j = 0; j < NCT; j++) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.0f;
+    const float sc = g.scale * 1.4426950408889634f;
+    const int mt = warp % MT, kg = warp / MT, row0 = mt * 16;
+    int par = 0;
+    for (int kt = kt0; kt < kt1; kt++, par ^= 1) {
+        const int buf = (kt - kt0) & 1;
+        if (kt + 1 < kt1) { load(kt + 1, buf ^ 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        const uint32_t kb = k_sm + (uint32_t)(buf * kKeys * row_bytes);
+        // scores of rows row0 .. + 15 with keys kg * 8 MT ..
+        float s[MT][4];
+#pragma unroll
+        for (int i = 0; i < MT; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+        const uint32_t qa = q_sm + (uint32_t)((row0 + (lane & 15)) * row_bytes + (lane >> 4) * 16);
+        const uint32_t ka = kb + (uint32_t)((kg * 8 * MT + (lane & 7)) * row_bytes + (lane >> 3) * 16);
+        for (int k = 0; k < d32; k += 32) {
+            uint32_t a0[4], a1[4];
+            ldsm4(qa + k * 2, a0);
+            ldsm4(qa + k * 2 + 32, a1);
+#pragma unroll
+            for (int i = 0; i < MT; i++) {
+                uint32_t b[4];
+                ldsm4(ka + (uint32_t)(8 * i * row_bytes + k * 2), b);
+                mma_bf16(s[i], a0, b[0], b[1]);
+                mma_bf16(s[i], a1, b[2], b[3]);
+            }
+        }
+        float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const int key = kt * kKeys + kg * 8 * MT + 8 * i + 2 * t4 + (j & 1);
+                s[i][j] = key <= pos ? s[i][j] * sc : -INFINITY;
+                mx[j >> 1] = fmaxf(mx[j >> 1], s[i][j]);
+            }
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+            if (t4 == 0) s_wmax[(row0 + g8 + 8 * r) * KG + kg] = mx[r];
+        }
+        __syncthreads();
+        auto new_max = [&](int row) {
+            float v = s_m[par * ROWS + row];
+#pragma unroll
+            for (int i = 0; i < KG; i++) v = fmaxf(v, s_wmax[row * KG + i]);
+            return v;
+        };
+        float sum[2] = {0.0f, 0.0f};
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int row = row0 + g8 + 8 * r;
+            const float m = new_max(row);
+            if (kg == 0 && t4 == 0) s_m[(par ^ 1) * ROWS + row] = m;
+#pragma unroll
+            for (int i = 0; i < MT; i++) {
+                const float p0 = exp2f(s[i][2 * r] - m), p1 = exp2f(s[i][2 * r + 1] - m);
+                sum[r] += p0 + p1;
+                uint32_t hi, lo;
+                split2(p0, p1, hi, lo);
+                const int at = row * (kKeys + 8) + kg * 8 * MT + 8 * i + 2 * t4;
+                *(uint32_t*)(s_ph + at) = hi;
+                *(uint32_t*)(s_pl + at) = lo;
+            }
+            sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 1);
+            sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 2);
+            if (t4 == 0) s_wsum[row * KG + kg] = sum[r];
+        }
+        __syncthreads();
+        if (tid < ROWS) {
+            float l = s_l[tid] * exp2f(s_m[par * ROWS + tid] - s_m[(par ^ 1) * ROWS + tid]);
+#pragma unroll
+            for (int i = 0; i < KG; i++) l += s_wsum[tid * KG + i];
+            s_l[tid] = l;
+        }
+        // weighted sum of this warp's latent columns
+        const int c0 = warp * NCT * 8;
+        if (c0 < g.cp) {
+#pragma unroll
+            for (int i = 0; i < MT; i++) {
+                const float f0 = exp2f(s_m[par * ROWS + 16 * i + g8] - s_m[(par ^ 1) * ROWS + 16 * i + g8]);
+                const float f1 = exp2f(s_m[par * ROWS + 16 * i + g8 + 8] - s_m[(par ^ 1) * ROWS + 16 * i + g8 + 8]);
+#pragma unroll
+                for (int j = 0; j < NCT; j++) { o[i][j][0] *= f0; o[i][j][1] *= f0; o[i][j][2] *= f1; o[i][j][3] *= f1; }
+            }
+#pragma unroll
+            for (int ks = 0; ks < kKeys / 16; ks++) {
+                uint32_t ph[MT][4], pl[MT][4];
+#pragma unroll
+                for (int i = 0; i < MT; i++) {
+                    const uint32_t off = (uint32_t)((16 * i + (lane & 15)) * (kKeys + 8) + 16 * ks + (lane >> 4) * 8) * 2;
+                    ldsm4(ph_sm + off, ph[i]);
+                    ldsm4(pl_sm + off, pl[i]);
+                }
+#pragma unroll
+                for (int j = 0; j < NCT; j += 2) {
+                    if (c0 + 8 * j >= g.cp) break;
+                    uint32_t b[4];
+                    ldsm4t(kb + (uint32_t)((16 * ks + (lane & 15)) * row_bytes + (c0 + 8 * j + (lane >> 4) * 8) * 2), b);
+#pragma unroll
+                    for (int i = 0; i < MT; i++) {
+                        mma_bf16(o[i][j], ph[i], b[0], b[1]);
+                        mma_bf16(o[i][j], pl[i], b[0], b[1]);
+                        mma_bf16(o[i][j + 1], ph[i], b[2], b[3]);
+                        mma_bf16(o[i][j + 1], pl[i], b[2], b[3]);
+                    }
+                }
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < MT; i++)
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int row = 16 * i + g8 + 8 * r;
+            if (row >= nh) continue;
+            const float inv = 1.0f / s_l[row];
+#pragma unroll
+            for (int j = 0; j < NCT; j++) {
+                const int c = (warp * NCT + j) * 8 + 2 * t4;
+                if (c >= g.cp) continue;
+                if (pieces == 1) *(uint32_t*)((bf16*)a.o + ((size_t)t * g.heads + h0 + row) * g.cp + c) = pack2(o[i][j][2 * r] * inv, o[i][j][2 * r + 1] * inv);
+                else *(float2*)(pc.o + (out_row + h0 + row) * g.cp + c) = make_float2(o[i][j][2 * r], o[i][j][2 * r + 1]);
+            }
+        }
+    if (pieces > 1 && tid < nh) {
+        pc.ml[(out_row + h0 + tid) * 2] = s_m[par * ROWS + tid];
+        pc.ml[(out_row + h0 + tid) * 2 + 1] = s_l[tid];
+    }
+}
+
+constexpr int kMaxPieces = 64;
+__global__ void __launch_bounds__(128) latent_merge_kernel(LatentPieces pc, int pieces, int heads, int cp, bf16* __restrict__ out) {
+    __shared__ float s_w[kMaxPieces];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int h = blockIdx.x, t = blockIdx.y;
+    const size_t base = (size_t)t * pieces * heads + h;
+    if (threadIdx.x < 32) {
+        float m = -INFINITY, l = 0.0f;
+        for (int i = threadIdx.x; i < pieces; i += 32) m = fmaxf(m, pc.ml[(base + (size_t)i * heads) * 2]);
+        m = warp_max(m);
+        for (int i = threadIdx.x; i < pieces; i += 32) {
+            const float w = exp2f(pc.ml[(base + (size_t)i * heads) * 2] - m);
+            s_w[i] = w;
+            l += w * pc.ml[(base + (size_t)i * heads) * 2 + 1];
+        }
+        l = warp_sum(l);
+        __syncwarp();
+        for (int i = threadIdx.x; i < pieces; i += 32) s_w[i] /= l;
+    }
+    __syncthreads();
+    for (int c = threadIdx.x * 2; c < cp; c += 256) {
+        float x = 0.0f, y = 0.0f;
+#pragma unroll 4
+        for (int i = 0; i < pieces; i++) {
+            if (s_w[i] == 0.0f) continue;  // an empty piece has written no sums
+            const float2 v = *(const float2*)(pc.o + (base + (size_t)i * heads) * cp + c);
+            x = fmaf(s_w[i], v.x, x);
+            y = fmaf(s_w[i], v.y, y);
+        }
+        *(uint32_t*)(out + ((size_t)t * heads + h) * cp + c) = pack2(x, y);
+    }
+}
+
+// The cached rows of a context, in order: row row0 + i of out = position i of the sequence.
+__global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* __restrict__ cache, int row16, int page_tokens, const int32_t* __restrict__ page_table,
+                                                            int pages_per_seq, const LatentContext* __restrict__ ctx, uint4* __restrict__ out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const LatentContext c = ctx[blockIdx.y];
+    const int n = c.len * row16;
+    for (int i = blockIdx.x * 256 + threadIdx.x; i < n; i += gridDim.x * 256) {
+        const int p = i / row16, w = i - p * row16;
+        const int page = page_table[(size_t)c.seq * pages_per_seq + p / page_tokens];
+        out[(size_t)(c.row0 + p) * row16 + w] = cache[((size_t)page * page_tokens + p % page_tokens) * row16 + w];
+    }
+}
+
+// Many tokens of a sequence: keys and values of every head have been projected from the gathered latents; a CTA of four warps
+// takes 64 consecutive queries of one head, tiles of 64 keys, online softmax in log2 units.
+template <int NV>
+__global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentArgs a, const LatentPrefill p) {
+    extern __shared__ __align__(128) unsigned char smem[];
+    const LatentShape& g = a.g;
+    const int d = g.dp + g.rp, d32 = (d + 31) & ~31, pitch = d32 + 8, rb = pitch * 2;
+    constexpr int kVP = NV * 8 + 8, kVB = kVP * 2;
+    bf16 *s_q = (bf16*)smem, *s_k = s_q + 64 * pitch, *s_v = s_k + 2 * kKeys * pitch;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+    pdl_launch_dependents();
+    pdl_wait();
+    const LatentTile tl = p.tiles[gridDim.x - 1 - blockIdx.x];  // the tiles with the longest contexts first
+    const int h = blockIdx.y, ld_c = g.cp + g.rp, ldk = g.heads * g.dp, ldv = g.heads * p.ep;
+    const int ctx_end = tl.pos0 + tl.n, n_kt = (ctx_end + kKeys - 1) / kKeys;
+    const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), v_sm = smem_u32(s_v);
+    const bf16 *kc = (const bf16*)p.k + (size_t)tl.row0 * ldk + h * g.dp, *rc = (const bf16*)p.c + (size_t)tl.row0 * ld_c + g.cp,
+               *vc = (const bf16*)p.v + (size_t)tl.row0 * ldv + h * p.ep;
+    const int kch = g.dp / 8, rch = g.rp / 8, vch = p.ep / 8, per_key = kch + rch + vch;
+    auto load = [&](int kt, int buf) {
+        for (int i = tid; i < kKeys * per_key; i += 128) {
+            const int key = i / per_key, c = i - key * per_key, kp = kt * kKeys + key;
+            const bool ok = kp < ctx_end;
+            const bf16* src;
+            uint32_t dst;
+            if (c < kch) { src = kc + (size_t)kp * ldk + c * 8; dst = k_sm + (uint32_t)((buf * kKeys + key) * rb + c * 16); }
+            else if (c < kch + rch) { src = rc + (size_t)kp * ld_c + (c - kch) * 8; dst = k_sm + (uint32_t)((buf * kKeys + key) * rb + c * 16); }
+            else { src = vc + (size_t)kp * ldv + (c - kch - rch) * 8; dst = v_sm + (uint32_t)((buf * kKeys + key) * kVB + (c - kch - rch) * 16); }
+            cp16(dst, ok ? src : kc, ok ? 16 : 0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    load(0, 0);
+    const bf16 zero = __float2bfloat16_rn(0.0f);
+    for (int i = tid; i < 2 * kKeys * (pitch - d); i += 128) s_k[(i / (pitch - d)) * pitch + d + i % (pitch - d)] = zero;
+    if (kVP > p.ep)
+        for (int i = tid; i < 2 * kKeys * (kVP - p.ep); i += 128) s_v[(i / (kVP - p.ep)) * kVP + p.ep + i % (kVP - p.ep)] = zero;
+    for (int i = tid; i < 64 * (pitch / 8); i += 128) {
+        const int r = i / (pitch / 8), c = (i - r * (pitch / 8)) * 8;
+        const size_t th = (size_t)(tl.tok0 + r) * g.heads + h;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (r < tl.n && c < d) {
+            const bf16* row = (const bf16*)a.q + th * g.ld_q;
+            if (c < g.dp) v = *(const uint4*)(row + c);
+            else {
+                const float2* tab = a.rot + (size_t)(tl.pos0 + r) * g.rot_pairs;
+                uint32_t w[4];
+#pragma unroll
+                for (int j = 0; j < 4; j++) w[j] = pack2(rotated(row + g.dp, tab, g.rot_pairs, g.rot, c - g.dp + 2 * j), rotated(row + g.dp, tab, g.rot_pairs, g.rot, c - g.dp + 2 * j + 1));
+                v = make_uint4(w[0], w[1], w[2], w[3]);
+            }
+        }
+        *(uint4*)(s_q + r * pitch + c) = v;
+    }
+    float o[NV][4];
+#pragma unroll
+    for (int i = 0; i < NV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
+    const float sc = g.scale * 1.4426950408889634f;
+    const int q0 = warp * 16, qpos[2] = {tl.pos0 + q0 + g8, tl.pos0 + q0 + g8 + 8};
+    const int last_kt = min(n_kt - 1, (tl.pos0 + q0 + 15) / kKeys);
+    for (int kt = 0; kt < n_kt; kt++) {
+        const int buf = kt & 1;
+        if (kt + 1 < n_kt) { load(kt + 1, buf ^ 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (kt <= last_kt) {
+            const uint32_t kb = k_sm + (uint32_t)(buf * kKeys * rb), vb = v_sm + (uint32_t)(buf * kKeys * kVB);
+            float s[8][4];
+#pragma unroll
+            for (int i = 0; i < 8; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+            const uint32_t qa = q_sm + (uint32_t)((q0 + (lane & 15)) * rb + (lane >> 4) * 16), ka = kb + (uint32_t)((lane & 7) * rb + (lane >> 3) * 16);
+            for (int k = 0; k < d32; k += 32) {
+                uint32_t a0[4], a1[4];
+                ldsm4(qa + k * 2, a0);
+                ldsm4(qa + k * 2 + 32, a1);
+#pragma unroll
+                for (int nt = 0; nt < 8; nt++) {
+                    uint32_t b[4];
+                    ldsm4(ka + (uint32_t)(8 * nt * rb + k * 2), b);
+                    mma_bf16(s[nt], a0, b[0], b[1]);
+                    mma_bf16(s[nt], a1, b[2], b[3]);
+                }
+            }
+            float mx[2] = {-INFINITY, -INFINITY};
+            const bool edge = kt * kKeys + kKeys - 1 > tl.pos0 + q0;
+#pragma unroll
+            for (int nt = 0; nt < 8; nt++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    float v = s[nt][i] * sc;
+                    if (edge && kt * kKeys + 8 * nt + 2 * t4 + (i & 1) > qpos[i >> 1]) v = -INFINITY;
+                    s[nt][i] = v;
+                    mx[i >> 1] = fmaxf(mx[i >> 1], v);
+                }
+            float corr[2];
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+                const float m = fmaxf(m_run[r], mx[r]);  // finite: key 0 is never past a query's position
+                corr[r] = exp2f(m_run[r] - m);
+                m_run[r] = m;
+            }
+            float ps[2] = {0.0f, 0.0f};
+            uint32_t ph[4][4], pl[4][4];
+#pragma unroll
+            for (int nt = 0; nt < 8; nt++) {
+                float pv[4];
+#pragma unroll
+                for (int i = 0; i < 4; i++) { pv[i] = exp2f(s[nt][i] - m_run[i >> 1]); ps[i >> 1] += pv[i]; }
+                const int ks = nt >> 1, hs = (nt & 1) * 2;
+                split2(pv[0], pv[1], ph[ks][hs], pl[ks][hs]);
+                split2(pv[2], pv[3], ph[ks][hs + 1], pl[ks][hs + 1]);
+            }
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                ps[r] += __shfl_xor_sync(0xffffffffu, ps[r], 1);
+                ps[r] += __shfl_xor_sync(0xffffffffu, ps[r], 2);
+                l_run[r] = l_run[r] * corr[r] + ps[r];
+            }
+#pragma unroll
+            for (int i = 0; i < NV; i++) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+#pragma unroll
+            for (int ks = 0; ks < 4; ks++)
+#pragma unroll
+                for (int np = 0; np < NV / 2; np++) {
+                    uint32_t b[4];
+                    ldsm4t(vb + (uint32_t)((16 * ks + (lane & 15)) * kVB + (16 * np + (lane >> 4) * 8) * 2), b);
+                    mma_bf16(o[2 * np], ph[ks], b[0], b[1]);
+                    mma_bf16(o[2 * np], pl[ks], b[0], b[1]);
+                    mma_bf16(o[2 * np + 1], ph[ks], b[2], b[3]);
+                    mma_bf16(o[2 * np + 1], pl[ks], b[2], b[3]);
+                }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        const int row = q0 + g8 + 8 * r;
+        if (row >= tl.n) continue;
+        const float inv = 1.0f / l_run[r];
+        bf16* dst = (bf16*)p.out + (size_t)(tl.tok0 + row) * ldv + h * p.ep + 2 * t4;
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+            if (8 * i + 2 * t4 < p.ep) *(uint32_t*)(dst + 8 * i) = pack2(o[i][2 * r] * inv, o[i][2 * r + 1] * inv);
+    }
+}
+
+size_t decode_smem(const LatentShape& g, int mt) {
+    const size_t pitch = ((g.cp + g.rp + 31) & ~31) + 8, rows = 16 * (size_t)mt;
+    return (rows + 2 * kKeys) * pitch * 2 + 2 * rows * (kKeys + 8) * 2 + (2 * rows * (8 / mt) + 3 * rows) * 4;
+}
+size_t prefill_smem(const LatentShape& g, int nv) {
+    const size_t pitch = ((g.dp + g.rp + 31) & ~31) + 8;
+    return (64 + 2 * kKeys) * pitch * 2 + 2 * kKeys * ((size_t)nv * 8 + 8) * 2;
+}
+int value_tiles(int ep) { return ep <= 32 ? 4 : ep <= 64 ? 8 : ep <= 128 ? 16 : 32; }
+
+int32_t launch_plain(const LatentArgs& a, cudaStream_t s) {
     const size_t smem = (size_t)(2 * a.g.cp + a.g.rp + 2 * kPlainThreads) * 4;
-    LC_CHECK(smem <= 100 * 1024, LC_ERR_UNSUPPORTED, "latent attention: rank %d", a.g.rank);
+    LC_CHECK(smem <= kMaxSmem, LC_ERR_UNSUPPORTED, "latent attention: rank %d", a.g.rank);
     const dim3 grid((unsigned)a.g.heads, (unsigned)a.T);
     if (a.f32) {
         LC_CUDA(ensure_smem_limit((const void*)latent_attention_plain_kernel<float>, smem));
         LC_CUDA(launch_pdl(latent_attention_plain_kernel<float>, grid, dim3(kPlainThreads), smem, s, a));
     } else {
-        LC_CUDA(ensure_smem_limit((const void*)latent_attention_plain_kernel<__nv_bfloat16>, smem));
-        LC_CUDA(launch_pdl(latent_attention_plain_kernel<__nv_bfloat16>, grid, dim3(kPlainThreads), smem, s, a));
+        LC_CUDA(ensure_smem_limit((const void*)latent_attention_plain_kernel<bf16>, smem));
+        LC_CUDA(launch_pdl(latent_attention_plain_kernel<bf16>, grid, dim3(kPlainThreads), smem, s, a));
     }
     return LC_OK;
+}
+
+}  // namespace
+
+size_t latent_pieces_bytes(const LatentShape& g, int tokens) {
+    // pieces * tokens * row blocks stays near twice the SM count, so the scratch is bounded by that many row blocks
+    const size_t blocks = std::max<size_t>((size_t)4 * sm_count(), (size_t)tokens * ((g.heads + 15) / 16));
+    return blocks * 32 * ((size_t)g.cp + 2) * sizeof(float) * 2;
+}
+
+int32_t launch_latent_attention(const LatentArgs& a, void* scratch, size_t scratch_bytes, int* launches, cudaStream_t s) {
+    const LatentShape& g = a.g;
+    const int mt = g.heads <= 16 ? 1 : 2;
+    *launches = 1;
+    if (a.T <= 0) return LC_OK;
+    if (a.f32 || g.cp > 512 || decode_smem(g, mt) > kMaxSmem) return launch_plain(a, s);
+    const int blocks = (g.heads + 16 * mt - 1) / (16 * mt);
+    int pieces = std::max(1, std::min(kMaxPieces, 2 * sm_count() / (a.T * blocks)));
+    pieces = std::min(pieces, (a.pages_per_seq * a.page_tokens + kKeys - 1) / kKeys);
+    auto need = [&](int n) { return (size_t)a.T * n * g.heads * ((size_t)g.cp + 2) * sizeof(float); };
+    while (pieces > 1 && need(pieces) > scratch_bytes) pieces--;
+    LatentPieces pc;
+    pc.o = (float*)scratch;
+    pc.ml = pc.o + (size_t)a.T * pieces * g.heads * g.cp;
+    const size_t smem = decode_smem(g, mt);
+    const dim3 grid((unsigned)a.T, (unsigned)blocks, (unsigned)pieces);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+        LC_CUDA(launch_pdl(kern, grid, dim3(256), smem, s, a, pc));
+        return LC_OK;
+    };
+    const int nct = g.cp <= 128 ? 2 : g.cp <= 256 ? 4 : 8;
+    if (mt == 1) LC_TRY(nct == 2 ? go(latent_decode_kernel<1, 2>) : nct == 4 ? go(latent_decode_kernel<1, 4>) : go(latent_decode_kernel<1, 8>));
+    else LC_TRY(nct == 2 ? go(latent_decode_kernel<2, 2>) : nct == 4 ? go(latent_decode_kernel<2, 4>) : go(latent_decode_kernel<2, 8>));
+    if (pieces > 1) {
+        LC_CUDA(launch_pdl(latent_merge_kernel, dim3((unsigned)g.heads, (unsigned)a.T), dim3(128), 0, s, pc, pieces, g.heads, g.cp, (bf16*)a.o));
+        *launches = 2;
+    }
+    return LC_OK;
+}
+
+bool latent_prefill_applies(const LatentShape& g, int ep, bool f32) { return !f32 && ep <= 256 && prefill_smem(g, value_tiles(ep)) <= kMaxSmem; }
+
+int32_t launch_latent_gather(const LatentArgs& a, const LatentContext* ctx, int n_ctx, int longest, void* out, cudaStream_t s) {
+    const int row16 = (a.g.cp + a.g.rp) / 8;
+    const int gx = std::max(1, std::min((int)(((size_t)longest * row16 + 255) / 256), 4 * sm_count()));
+    LC_CUDA(launch_pdl(latent_gather_kernel, dim3((unsigned)gx, (unsigned)n_ctx), dim3(256), 0, s, (const uint4*)a.cache, row16, a.page_tokens, a.page_table,
+                       a.pages_per_seq, ctx, (uint4*)out));
+    return LC_OK;
+}
+
+int32_t launch_latent_prefill(const LatentArgs& a, const LatentPrefill& p, int n_tiles, cudaStream_t s) {
+    const int nv = value_tiles(p.ep);
+    const size_t smem = prefill_smem(a.g, nv);
+    const dim3 grid((unsigned)n_tiles, (unsigned)a.g.heads);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+        LC_CUDA(launch_pdl(kern, grid, dim3(128), smem, s, a, p));
+        return LC_OK;
+    };
+    switch (nv) {
+        case 4: return go(latent_prefill_kernel<4>);
+        case 8: return go(latent_prefill_kernel<8>);
+        case 16: return go(latent_prefill_kernel<16>);
+        default: return go(latent_prefill_kernel<32>);
+    }
 }
 
 }  // namespace lc

@@ -15,6 +15,7 @@ namespace lc {
 namespace {
 
 typedef __nv_bfloat16 bf16;
+constexpr int kContextRows = 16384;  // rows of projected keys and values at a time (one longer context is taken whole)
 
 int32_t zalloc(LayerStack& st, void** p, size_t bytes) {
     uint8_t* q = nullptr;
@@ -184,6 +185,20 @@ int32_t bind_latent(lc_model* m, StackLayer& L, const std::string& p) {
     }
     LC_TRY(dense_weight_init(&L.uv, uv, s.vdim, s.kv_rank, g.cp, s.heads, (size_t)s.vdim * g.cp));
     L.ep = round8(s.vdim);
+    // the same two projections for whole contexts
+    if (latent_prefill_applies(g, L.ep, st.f32)) {
+        auto all_heads = [&](const char* name, int per, int per_p, DenseWeight* w) -> int32_t {
+            DevTensor* wt = nullptr;
+            LC_TRY(matrix(m, p + name, s.heads * per, s.kv_rank, &wt));
+            if (per == per_p && g.cp == s.kv_rank) return dense_weight_init(w, (const bf16*)wt->view, s.heads * per, s.kv_rank, s.kv_rank);
+            void* q = nullptr;
+            LC_TRY(zalloc(st, &q, (size_t)s.heads * per_p * g.cp * 2));
+            LC_TRY(launch_pack((const bf16*)wt->view, s.heads * per, s.kv_rank, (bf16*)q, g.cp, PackMap{per, per_p, 0, 0}, PackMap(), false, m->stream));
+            return dense_weight_init(w, (const bf16*)q, s.heads * per_p, s.kv_rank, g.cp);
+        };
+        LC_TRY(all_heads("uk", s.dim, g.dp, &L.uk_all));
+        LC_TRY(all_heads("uv", s.vdim, L.ep, &L.uv_all));
+    }
     LC_TRY(plain_weight(m, p + "o", W, s.heads * s.vdim, &L.out, PackMap{s.vdim, L.ep, 0, 0}, s.heads * L.ep));
     LC_TRY(model_gain_f32(m, p + "dq.norm", qr, &L.q_norm));
     LC_TRY(model_gain_f32(m, p + "dkv.norm", s.kv_rank, &L.c_norm));
@@ -227,7 +242,7 @@ int32_t delta_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, b
     return product(m, L.out, st.mixed, d.ldo, T, st.y, st.spec.width, true);
 }
 
-int32_t latent_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T) {
+int32_t latent_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bool decode_step) {
     LayerStack& st = *m->stack;
     const LatentShape& g = L.lg;
     LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in.n, true));
@@ -239,13 +254,30 @@ int32_t latent_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T) 
     m->launches_in_call += 1;
     const int ldq = g.heads * g.ld_q, ldc = g.heads * g.cp, lde = g.heads * L.ep;
     LC_TRY(product(m, L.uq, st.cq, a.ld_cq, T, st.q, ldq));
-    DenseArgs b;
-    b.x_batch = (size_t)g.ld_q; b.out_batch = (size_t)g.cp;
-    LC_TRY(product(m, L.uk_t, st.q, ldq, T, st.q_abs, ldc, false, DENSE_STORE, b));
-    LC_TRY(launch_latent_attention(a, m->stream));
-    m->launches_in_call += 1;
-    b.x_batch = (size_t)g.cp; b.out_batch = (size_t)L.ep;
-    LC_TRY(product(m, L.uv, st.o_lat, ldc, T, st.mixed, lde, false, DENSE_STORE, b));
+    const int few = decode_step || !st.prefill_tiles ? T : st.n_short;
+    if (few > 0) {
+        DenseArgs b;
+        b.x_batch = (size_t)g.ld_q; b.out_batch = (size_t)g.cp;
+        LC_TRY(product(m, L.uk_t, st.q, ldq, few, st.q_abs, ldc, false, DENSE_STORE, b));
+        a.T = few;
+        int launches = 0;
+        LC_TRY(launch_latent_attention(a, st.pieces, st.pieces_bytes, &launches, m->stream));
+        m->launches_in_call += launches;
+        b.x_batch = (size_t)g.cp; b.out_batch = (size_t)L.ep;
+        LC_TRY(product(m, L.uv, st.o_lat, ldc, few, st.mixed, lde, false, DENSE_STORE, b));
+    }
+    if (few < T)
+        for (const LayerStack::Group& gr : st.groups) {
+            LC_TRY(launch_latent_gather(a, st.d_lat_ctx + gr.ctx0, gr.n_ctx, gr.longest, st.ctx_c.p, m->stream));
+            DenseArgs c;
+            c.x_rows = gr.rows;
+            LC_TRY(product(m, L.uk_all, st.ctx_c.p, g.cp + g.rp, gr.rows, st.ctx_k.p, g.heads * g.dp, false, DENSE_STORE, c));
+            LC_TRY(product(m, L.uv_all, st.ctx_c.p, g.cp + g.rp, gr.rows, st.ctx_v.p, lde, false, DENSE_STORE, c));
+            LatentPrefill p;
+            p.tiles = st.d_lat_tiles + gr.tile0; p.c = st.ctx_c.p; p.k = st.ctx_k.p; p.v = st.ctx_v.p; p.out = st.mixed; p.ep = L.ep;
+            LC_TRY(launch_latent_prefill(a, p, gr.n_tiles, m->stream));
+            m->launches_in_call += 2;
+        }
     return product(m, L.out, st.mixed, lde, T, st.y, st.spec.width, true);
 }
 
@@ -297,6 +329,7 @@ int32_t stack_alloc(lc_model* m) {
     LayerStack& st = *m->stack;
     const size_t T = (size_t)m->t_cap, e = elt(st);
     st.width_p = round8(st.spec.width);
+    st.prefill_tiles = !st.f32;
     size_t proj = 8, projf = 8, gate = 8, mixed = 8, cq = 8, q = 8, qa = 8, ffn = 8, ld = 8, qk = 8, v = 8;
     for (StackLayer& L : st.layers) {
         const LayerSpec& s = L.s;
@@ -319,6 +352,11 @@ int32_t stack_alloc(lc_model* m) {
             qa = std::max(qa, (size_t)g.heads * g.cp);
             mixed = std::max(mixed, (size_t)g.heads * L.ep);
             const size_t row = (size_t)(g.cp + g.rp) * e;
+            st.prefill_tiles = st.prefill_tiles && latent_prefill_applies(g, L.ep, st.f32);
+            st.ctx_c_row = std::max(st.ctx_c_row, (size_t)(g.cp + g.rp));
+            st.ctx_k_row = std::max(st.ctx_k_row, (size_t)g.heads * g.dp);
+            st.ctx_v_row = std::max(st.ctx_v_row, (size_t)g.heads * L.ep);
+            st.pieces_bytes = std::max(st.pieces_bytes, latent_pieces_bytes(g, m->max_seqs));
             LC_TRY(zalloc(st, &L.cache, (size_t)m->pages_total * m->page_tokens * row));
             st.cache_bytes_per_token += row;
         }
@@ -333,18 +371,64 @@ int32_t stack_alloc(lc_model* m) {
     LC_TRY(zalloc(st, (void**)&st.y, T * st.spec.width * 4)); LC_TRY(zalloc(st, (void**)&st.log_decay, T * ld * 4));
     LC_TRY(zalloc(st, (void**)&st.qk, T * qk * 4)); LC_TRY(zalloc(st, (void**)&st.v, T * v * 4)); LC_TRY(zalloc(st, (void**)&st.o, T * v * 4));
     LC_TRY(zalloc(st, (void**)&st.d_runs, T * sizeof(SeqRun)));
+    LC_TRY(zalloc(st, (void**)&st.d_lat_tiles, T * sizeof(LatentTile))); LC_TRY(zalloc(st, (void**)&st.d_lat_ctx, T * sizeof(LatentContext)));
+    if (st.pieces_bytes) LC_TRY(zalloc(st, &st.pieces, st.pieces_bytes));
     return LC_OK;
 }
 
 void stack_free(lc_model* m) {
     if (!m->stack) return;
     for (void* p : m->stack->owned) cudaFree(p);
+    for (DevBuf* b : {&m->stack->ctx_c, &m->stack->ctx_k, &m->stack->ctx_v}) b->release();
     dense_workspace_free(&m->stack->ws);
+}
+
+// What a call's tokens mean to the layers: runs of consecutive positions, those of at least kTileRun tokens also as tiles
+// over contexts of their own.  The caller orders the runs so that the short ones come first.
+int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const std::vector<int32_t>& pos) {
+    LayerStack& st = *m->stack;
+    std::vector<SeqRun> runs;
+    for (size_t i = 0; i < seq.size(); i++) {
+        if (runs.empty() || seq[i] != seq[i - 1] || pos[i] != pos[i - 1] + 1) runs.push_back(SeqRun{(int32_t)i, 0, seq[i], pos[i]});
+        runs.back().n++;
+    }
+    st.n_runs = (int)runs.size();
+    LC_CUDA(cudaMemcpyAsync(st.d_runs, runs.data(), runs.size() * sizeof(SeqRun), cudaMemcpyHostToDevice, m->stream));
+    st.groups.clear();
+    st.n_short = (int)seq.size();
+    std::vector<LatentTile> tiles;
+    std::vector<LatentContext> ctx;
+    size_t first = 0;
+    while (first < runs.size() && runs[first].n < kTileRun) first++;
+    if (st.prefill_tiles && first < runs.size()) {
+        st.n_short = runs[first].tok0;
+        int most = 0;
+        for (size_t i = first; i < runs.size(); i++) {
+            const SeqRun& r = runs[i];
+            const int len = r.pos0 + r.n;
+            if (st.groups.empty() || st.groups.back().rows + len > kContextRows) st.groups.push_back({(int)tiles.size(), 0, (int)ctx.size(), 0, 0, 0});
+            LayerStack::Group& gr = st.groups.back();
+            for (int t = 0; t < r.n; t += 64) { tiles.push_back(LatentTile{r.tok0 + t, std::min(64, r.n - t), r.pos0 + t, gr.rows}); gr.n_tiles++; }
+            ctx.push_back(LatentContext{r.seq, len, gr.rows});
+            gr.n_ctx++;
+            gr.rows += len;
+            gr.longest = std::max(gr.longest, len);
+            most = std::max(most, gr.rows);
+        }
+        LC_CUDA(cudaMemcpyAsync(st.d_lat_tiles, tiles.data(), tiles.size() * sizeof(LatentTile), cudaMemcpyHostToDevice, m->stream));
+        LC_CUDA(cudaMemcpyAsync(st.d_lat_ctx, ctx.data(), ctx.size() * sizeof(LatentContext), cudaMemcpyHostToDevice, m->stream));
+        const size_t rows = (size_t)std::max(most, std::min(kContextRows, m->t_cap));
+        LC_TRY(st.ctx_c.reserve(rows * st.ctx_c_row * 2));
+        LC_TRY(st.ctx_k.reserve(rows * st.ctx_k_row * 2));
+        LC_TRY(st.ctx_v.reserve(rows * st.ctx_v_row * 2));
+    }
+    LC_CUDA(cudaStreamSynchronize(m->stream));  // the copies read vectors that die with this frame
+    return LC_OK;
 }
 
 int32_t stack_mixer(lc_model* m, int l, const void* x, int ldx, int T, bool decode_step) {
     StackLayer& L = m->stack->layers[l];
-    return L.s.mixer == MixerKind::ChannelDelta ? delta_block(m, L, x, ldx, T, decode_step) : latent_block(m, L, x, ldx, T);
+    return L.s.mixer == MixerKind::ChannelDelta ? delta_block(m, L, x, ldx, T, decode_step) : latent_block(m, L, x, ldx, T, decode_step);
 }
 int32_t stack_ffn(lc_model* m, int l, const void* x, int ldx, int T) { return relu2_block(m, m->stack->layers[l], x, ldx, T); }
 

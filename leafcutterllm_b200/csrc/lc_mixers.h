@@ -129,7 +129,22 @@ struct LatentArgs {
 int32_t launch_latent_prep(const LatentArgs& a, cudaStream_t s);
 int32_t launch_rot_table(const double* freq_dev, int pairs, double magnitude, int positions, float2* out, cudaStream_t s);
 // ---- latent_attention.cu ---------------------------------------------------------------------------------------------
-int32_t launch_latent_attention(const LatentArgs& a, cudaStream_t s);
+// Tokens 0 .. T - 1 of `a`, each over its own context through q_abs / q, into o.  scratch: partial sums of context pieces.
+size_t latent_pieces_bytes(const LatentShape& g, int tokens);
+int32_t launch_latent_attention(const LatentArgs& a, void* scratch, size_t scratch_bytes, int* launches, cudaStream_t s);
+// Runs of many tokens: up to 64 consecutive tokens (rows tok0 .. of the call, first position pos0) whose sequence's gathered
+// context starts at row row0 of c / k / v.
+struct LatentTile { int32_t tok0, n, pos0, row0; };
+struct LatentContext { int32_t seq, len, row0; };
+struct LatentPrefill {
+    const LatentTile* tiles = nullptr;
+    const void *c = nullptr, *k = nullptr, *v = nullptr;  // [rows][cp + rp], [rows][heads * dp], [rows][heads * ep]
+    void* out = nullptr;                                  // [T][heads * ep]
+    int ep = 0;
+};
+bool latent_prefill_applies(const LatentShape& g, int ep, bool f32);
+int32_t launch_latent_gather(const LatentArgs& a, const LatentContext* ctx, int n_ctx, int longest, void* out, cudaStream_t s);
+int32_t launch_latent_prefill(const LatentArgs& a, const LatentPrefill& p, int n_tiles, cudaStream_t s);
 
 // ---- a stack of such layers (layers.cu) --------------------------------------------------------------------------------
 struct StackLayer {
@@ -144,7 +159,8 @@ struct StackLayer {
     float* state = nullptr;
     void* ring = nullptr;
     // LatentAttention: `in` = dq | dkv
-    DenseWeight uq, uk_t, uv;
+    DenseWeight uq, uk_t, uv;       // one token at a time: key projection transposed per head, value projection per head
+    DenseWeight uk_all, uv_all;     // whole contexts: all heads at once
     LatentShape lg{};
     int off_r = 0, off_c = 0, ep = 0;
     const float *q_norm = nullptr, *c_norm = nullptr;
@@ -168,6 +184,18 @@ struct LayerStack {
     float *y = nullptr, *projf = nullptr, *log_decay = nullptr, *qk = nullptr, *v = nullptr, *o = nullptr;
     SeqRun* d_runs = nullptr;
     int n_runs = 0;
+    // latent attention of the call: its first n_short tokens attend one by one, the others in tiles over projected contexts,
+    // in groups whose contexts fit the context buffers
+    struct Group { int tile0, n_tiles, ctx0, n_ctx, rows, longest; };
+    int n_short = 0;
+    std::vector<Group> groups;
+    LatentTile* d_lat_tiles = nullptr;
+    LatentContext* d_lat_ctx = nullptr;
+    void* pieces = nullptr;
+    size_t pieces_bytes = 0;
+    bool prefill_tiles = false;        // every latent layer has a tile form
+    size_t ctx_c_row = 0, ctx_k_row = 0, ctx_v_row = 0;  // widest rows of the context buffers, in elements
+    DevBuf ctx_c, ctx_k, ctx_v;
 };
 
 }  // namespace lc

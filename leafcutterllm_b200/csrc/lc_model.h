@@ -37,6 +37,7 @@ struct LayerW {
 };
 
 constexpr int kPrefillChunk = 512;
+constexpr int kTileRun = 16;             // runs of fewer tokens attend token by token
 constexpr int kStackChunk = 2048;      // tokens per pass of a checkpoint-directory design
 constexpr int kTokTile = 8;
 constexpr int kMoeGroupedTokens = 64;  // calls of at most this many tokens run the experts as one grouped launch
@@ -167,6 +168,7 @@ int32_t model_gain_f32(lc_model* m, const std::string& name, int expect, const f
 int32_t stack_bind(lc_model* m);   // weights
 int32_t stack_alloc(lc_model* m);  // cache, state and step buffers, sized by the handle's pool and slots
 void stack_free(lc_model* m);
+int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const std::vector<int32_t>& pos);
 int32_t stack_run_layers(lc_model* m, int T, bool decode_step);
 int32_t stack_head(lc_model* m, int n, const int32_t* idx, float* logits);  // logits of rows idx (null: rows 0 .. n - 1)
 int32_t stack_probe(lc_model* m, int l, int T, bool ffn, float** y);

@@ -2,6 +2,7 @@
 // rule with its short convolutions, the preparation of latent attention.  Template parameter A = type of the activations
 // (bf16, or float when a model runs in true 32-bit); norms, decays, step sizes, unit vectors, the recurrence and its state,
 // rotation angles and residual sums are f32 in both.
+#include <algorithm>
 #include <cmath>
 #include "lc_mixers.h"
 #include "lc_tma.cuh"
@@ -43,6 +44,17 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const __nv_bfloat16* __
     const int t = blockIdx.x;
     const int64_t id = ids[t];
     const bool ok = id >= 0 && id < rows;
+    if (width % 8 == 0) {
+        for (int c = threadIdx.x * 8; c < width; c += blockDim.x * 8) {
+            const uint4 v = ok ? *(const uint4*)(table + (size_t)id * width + c) : make_uint4(0u, 0u, 0u, 0u);
+            const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+            float4* o = (float4*)(x + (size_t)t * width + c);
+            o[0] = make_float4(__uint_as_float(u[0] << 16), __uint_as_float(u[0] & 0xFFFF0000u), __uint_as_float(u[1] << 16), __uint_as_float(u[1] & 0xFFFF0000u));
+            o[1] = make_float4(__uint_as_float(u[2] << 16), __uint_as_float(u[2] & 0xFFFF0000u), __uint_as_float(u[3] << 16), __uint_as_float(u[3] & 0xFFFF0000u));
+            if (act) *(uint4*)(act + (size_t)t * ld_act + c) = v;
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         const __nv_bfloat16 v = ok ? table[(size_t)id * width + c] : __float2bfloat16_rn(0.0f);
         x[(size_t)t * width + c] = __bfloat162float(v);
@@ -56,22 +68,58 @@ __global__ void __launch_bounds__(256) act_rows_kernel(const float* __restrict__
     for (int c = threadIdx.x; c < width; c += blockDim.x) act[(size_t)blockIdx.x * ld_act + c] = __float2bfloat16_rn(x[(size_t)blockIdx.x * width + c]);
 }
 
+// VEC = 4: rows of a multiple of four elements; a row of up to 4096 elements stays in registers between its two passes.
+template <int VEC>
 __global__ void __launch_bounds__(512) norm_residual_kernel(const float* __restrict__ y, const float* __restrict__ w, float eps, int width, float* __restrict__ x,
                                                             __nv_bfloat16* __restrict__ act, int ld_act) {
+    constexpr int kHeld = 4;
     __shared__ float sh[32];
     pdl_launch_dependents();
     pdl_wait();
     const size_t t = blockIdx.x;
     const float* yr = y + t * width;
     float* xr = x + t * width;
+    __nv_bfloat16* ar = act ? act + t * ld_act : nullptr;
     float ss = 0.0f;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) { const float v = yr[c]; ss = fmaf(v, v, ss); }
-    ss = block_sum(ss, sh);
-    const float r = 1.0f / sqrtf(ss / (float)width + eps);
-    for (int c = threadIdx.x; c < width; c += blockDim.x) {
-        const float v = xr[c] + yr[c] * r * w[c];
-        xr[c] = v;
-        if (act) act[t * ld_act + c] = __float2bfloat16_rn(v);
+    if constexpr (VEC == 4) {
+        float4 yv[kHeld], xv[kHeld];
+#pragma unroll
+        for (int i = 0; i < kHeld; i++) {
+            const int c = (threadIdx.x + i * blockDim.x) * 4;
+            if (c < width) { yv[i] = *(const float4*)(yr + c); xv[i] = *(const float4*)(xr + c); }
+            else yv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            ss = fmaf(yv[i].x, yv[i].x, fmaf(yv[i].y, yv[i].y, fmaf(yv[i].z, yv[i].z, fmaf(yv[i].w, yv[i].w, ss))));
+        }
+        for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < width; c += blockDim.x * 4) {
+            const float4 v = *(const float4*)(yr + c);
+            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+        }
+        ss = block_sum(ss, sh);
+        const float r = 1.0f / sqrtf(ss / (float)width + eps);
+        auto put = [&](int c, float4 yy, float4 xx) {
+            const float4 g = *(const float4*)(w + c);
+            xx.x += yy.x * r * g.x; xx.y += yy.y * r * g.y; xx.z += yy.z * r * g.z; xx.w += yy.w * r * g.w;
+            *(float4*)(xr + c) = xx;
+            if (ar) {
+                *(__nv_bfloat162*)(ar + c) = __floats2bfloat162_rn(xx.x, xx.y);
+                *(__nv_bfloat162*)(ar + c + 2) = __floats2bfloat162_rn(xx.z, xx.w);
+            }
+        };
+#pragma unroll
+        for (int i = 0; i < kHeld; i++) {
+            const int c = (threadIdx.x + i * blockDim.x) * 4;
+            if (c < width) put(c, yv[i], xv[i]);
+        }
+        for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < width; c += blockDim.x * 4) put(c, *(const float4*)(yr + c), *(const float4*)(xr + c));
+    } else {
+        for (int c = threadIdx.x; c < width; c += blockDim.x) { const float v = yr[c]; ss = fmaf(v, v, ss); }
+        ss = block_sum(ss, sh);
+        const float r = 1.0f / sqrtf(ss / (float)width + eps);
+        for (int c = threadIdx.x; c < width; c += blockDim.x) {
+            const float v = xr[c] + yr[c] * r * w[c];
+            xr[c] = v;
+            if (ar) ar[c] = __float2bfloat16_rn(v);
+        }
     }
 }
 
@@ -110,38 +158,84 @@ __device__ __forceinline__ float conv_at(const DeltaShape& g, const A* proj, con
 }
 __device__ __forceinline__ float silu32(float v) { return v * sigmoid_f(v); }
 
-// One warp per (token, head unit): kv_heads units of q, kv_heads of k, heads of v.
-template <typename A>
+// One warp per (stretch of kPrepTok tokens, head unit): kv_heads units of q, kv_heads of k, heads of v; a lane owns every 32nd
+// channel and keeps its last inputs in registers while it walks the stretch (TAPS of them; 0: any number, re-read).
+constexpr int kPrepTok = 16;
+template <typename A, int TAPS, int CPL>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const DeltaShape& g = a.g;
-    const int t = blockIdx.x, unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (unit >= 2 * g.kv_heads + g.heads) return;
     const A* proj = (const A*)a.proj;
     const A* ring = (const A*)a.ring;
-    const int seq = a.tok_seq[t], pos = a.tok_pos[t];
-    if (unit >= 2 * g.kv_heads) {
-        const int h = unit - 2 * g.kv_heads, c0 = 2 * g.kv_heads * g.dim + h * g.vdim;
-        for (int i = lane; i < g.vdim; i += 32)
-            a.v[(size_t)t * g.heads * g.vdim + h * g.vdim + i] = silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, g.off_v + h * g.vdim + i));
-        return;
+    const bool is_v = unit >= 2 * g.kv_heads, is_k = !is_v && unit >= g.kv_heads;
+    const int h = is_v ? unit - 2 * g.kv_heads : is_k ? unit - g.kv_heads : unit, n = is_v ? g.vdim : g.dim;
+    const int c0 = is_v ? 2 * g.kv_heads * g.dim + h * g.vdim : unit * g.dim, col0 = is_v ? g.off_v + h * g.vdim : (is_k ? g.off_k : 0) + h * g.dim;
+    const int t0 = blockIdx.x * kPrepTok, t1 = min(a.T, t0 + kPrepTok);
+    float w[CPL][TAPS > 0 ? TAPS : 1], win[CPL][TAPS > 0 ? TAPS : 1];  // win[.][j]: the input j + 1 tokens back
+    if constexpr (TAPS > 0)
+#pragma unroll
+        for (int c = 0; c < CPL; c++)
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) w[c][j] = lane + 32 * c < n ? a.conv[(c0 + lane + 32 * c) * TAPS + j] : 0.0f;
+    int prev_seq = -1, prev_pos = -1;
+    for (int t = t0; t < t1; t++) {
+        const int seq = a.tok_seq[t], pos = a.tok_pos[t];
+        float y[CPL], ss = 0.0f;
+        if constexpr (TAPS > 0) {
+            const bool follows = seq == prev_seq && pos == prev_pos + 1;
+#pragma unroll
+            for (int c = 0; c < CPL; c++) {
+                const int i = lane + 32 * c;
+                y[c] = 0.0f;
+                if (i >= n) continue;
+                if (!follows) {  // first token of the stretch or of a run: earlier inputs from the call's rows, the ring, or none
+#pragma unroll
+                    for (int j = 1; j < TAPS; j++) {
+                        float v = 0.0f;
+                        if (pos - j >= 0) {
+                            const int tt = t - j;
+                            if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) v = act_f<A>(proj[(size_t)tt * g.ld + col0 + i]);
+                            else v = act_f<A>(ring[((size_t)seq * TAPS + (pos - j) % TAPS) * g.channels + c0 + i]);
+                        }
+                        win[c][j - 1] = v;
+                    }
+                }
+                const float cur = act_f<A>(proj[(size_t)t * g.ld + col0 + i]);
+                float acc = 0.0f;
+#pragma unroll
+                for (int j = TAPS - 1; j > 0; j--) acc = fmaf(w[c][TAPS - 1 - j], win[c][j - 1], acc);
+                acc = fmaf(w[c][TAPS - 1], cur, acc);
+#pragma unroll
+                for (int j = TAPS - 1; j > 0; j--) win[c][j] = win[c][j - 1];
+                win[c][0] = cur;
+                y[c] = silu32(acc);
+                ss = fmaf(y[c], y[c], ss);
+            }
+            prev_seq = seq; prev_pos = pos;
+        } else {
+#pragma unroll
+            for (int c = 0; c < CPL; c++) {
+                const int i = lane + 32 * c;
+                y[c] = i < n ? silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, col0 + i)) : 0.0f;
+                ss = fmaf(y[c], y[c], ss);
+            }
+        }
+        float r = 1.0f;
+        float* o;
+        if (is_v) {
+            o = a.v + (size_t)t * g.heads * g.vdim + h * g.vdim;
+        } else {
+            o = a.qk + ((size_t)t * 2 + (is_k ? 1 : 0)) * g.kv_heads * g.dim + h * g.dim;
+            r = 1.0f / sqrtf(warp_sum(ss) + g.unit_eps);
+            if (!is_k) r *= 1.0f / sqrtf((float)g.dim);
+        }
+#pragma unroll
+        for (int c = 0; c < CPL; c++)
+            if (lane + 32 * c < n) o[lane + 32 * c] = y[c] * r;
     }
-    const bool is_k = unit >= g.kv_heads;
-    const int h = is_k ? unit - g.kv_heads : unit, c0 = unit * g.dim, col0 = (is_k ? g.off_k : 0) + h * g.dim;
-    float* o = a.qk + ((size_t)t * 2 + (is_k ? 1 : 0)) * g.kv_heads * g.dim + h * g.dim;
-    float ss = 0.0f, v[8];
-    int n = 0;
-    for (int i = lane; i < g.dim; i += 32, n++) {
-        const float s = silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, col0 + i));
-        ss = fmaf(s, s, ss);
-        if (n < 8) v[n] = s;
-    }
-    ss = warp_sum(ss);
-    float r = 1.0f / sqrtf(ss + g.unit_eps);
-    if (!is_k) r *= 1.0f / sqrtf((float)g.dim);
-    n = 0;
-    for (int i = lane; i < g.dim; i += 32, n++) o[i] = v[n] * r;
 }
 
 // The recurrence, token by token in f32.  A CTA of four warps owns 32 value columns of one head of one run; four lanes share
@@ -444,7 +538,25 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a) {
     }
 }
 
-int norm_threads(int width) { return width >= 2048 ? 512 : width >= 512 ? 256 : 128; }
+int norm_threads(int width) { return width >= 4096 ? 512 : width >= 1024 ? 256 : 128; }
+
+template <typename A>
+int32_t prep_dispatch(const DeltaArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)((a.T + kPrepTok - 1) / kPrepTok), (unsigned)((2 * a.g.kv_heads + a.g.heads + 7) / 8));
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(launch_pdl(kern, grid, dim3(256), 0, s, a));
+        return LC_OK;
+    };
+    const int widest = std::max(a.g.dim, a.g.vdim);
+    LC_CHECK(widest <= 512, LC_ERR_UNSUPPORTED, "delta rule: %d dimensions per head", widest);
+    if (widest > 128) return go(delta_prep_kernel<A, 0, 16>);
+    switch (a.g.taps) {
+        case 2: return go(delta_prep_kernel<A, 2, 4>);
+        case 3: return go(delta_prep_kernel<A, 3, 4>);
+        case 4: return go(delta_prep_kernel<A, 4, 4>);
+        default: return go(delta_prep_kernel<A, 0, 4>);
+    }
+}
 
 template <typename A>
 int32_t scan_dispatch(const DeltaArgs& a, cudaStream_t s) {
@@ -497,7 +609,9 @@ int32_t launch_act_rows(const float* x, int width, int T, void* act, int ld_act,
     return LC_OK;
 }
 int32_t launch_norm_residual(const float* y, const float* w, float eps, int width, int T, float* x, void* act, int ld_act, cudaStream_t s) {
-    LC_CUDA(launch_pdl(norm_residual_kernel, dim3((unsigned)T), dim3((unsigned)norm_threads(width)), 0, s, y, w, eps, width, x, (__nv_bfloat16*)act, ld_act));
+    const dim3 grid((unsigned)T), block((unsigned)norm_threads(width));
+    if (width % 4 == 0 && (uintptr_t)w % 16 == 0) LC_CUDA(launch_pdl(norm_residual_kernel<4>, grid, block, 0, s, y, w, eps, width, x, (__nv_bfloat16*)act, ld_act));
+    else LC_CUDA(launch_pdl(norm_residual_kernel<1>, grid, block, 0, s, y, w, eps, width, x, (__nv_bfloat16*)act, ld_act));
     return LC_OK;
 }
 int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, float eps, int width, int n, void* out, int ldo, bool f32, cudaStream_t s) {
@@ -508,10 +622,7 @@ int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, flo
 }
 int32_t launch_delta_prep(const DeltaArgs& a, cudaStream_t s) {
     LC_CHECK(a.g.dim <= 256, LC_ERR_UNSUPPORTED, "delta rule: %d key dimensions per head (at most 256)", a.g.dim);
-    const dim3 grid((unsigned)a.T, (unsigned)((2 * a.g.kv_heads + a.g.heads + 7) / 8));
-    if (a.f32) LC_CUDA(launch_pdl(delta_prep_kernel<float>, grid, dim3(256), 0, s, a));
-    else LC_CUDA(launch_pdl(delta_prep_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, a));
-    return LC_OK;
+    return a.f32 ? prep_dispatch<float>(a, s) : prep_dispatch<__nv_bfloat16>(a, s);
 }
 int32_t launch_delta_scan(const DeltaArgs& a, cudaStream_t s) { return a.f32 ? scan_dispatch<float>(a, s) : scan_dispatch<__nv_bfloat16>(a, s); }
 int32_t launch_delta_step(const DeltaArgs& a, cudaStream_t s) { return a.f32 ? step_dispatch<float>(a, s) : step_dispatch<__nv_bfloat16>(a, s); }

@@ -13,7 +13,7 @@ from typing import Iterator, Tuple
 
 import numpy as np
 
-from ._capi import TYPE_F32, TYPE_Q4_0, TYPE_Q4_K, TYPE_Q6_K, TYPE_Q8_0, check, load
+from ._capi import TYPE_BF16, TYPE_F16, TYPE_F32, TYPE_Q4_0, TYPE_Q4_K, TYPE_Q6_K, TYPE_Q8_0, check, load
 
 SIGMA = 0.02
 WEIGHT_SEED = 1234
@@ -97,6 +97,91 @@ LLAMA7B_Q4KM = ModelSpec("llama2-7b-shape-q4_k_m", 32, 4096, 32, 32, 11008, 3200
 MIXTRAL = ModelSpec("mixtral-8x7b-shape-q4_k", 32, 4096, 32, 8, 14336, 32000, 10000.0, TYPE_Q4_K, TYPE_Q4_K, TYPE_Q4_K, n_experts=8, top_k=2)
 # Llama-3-70B shape, Q4_K.
 LLAMA70B = ModelSpec("llama3-70b-shape-q4_k", 80, 8192, 64, 8, 28672, 128256, 500000.0, TYPE_Q4_K, TYPE_Q4_K, TYPE_Q4_K)
+
+
+@dataclass
+class LayeredSpec:
+    """A checkpoint-directory model: the parsed config.json (architecture "Varasun") with the ranks that only the tensors'
+    shapes give (decay_rank, gate_rank), for random weights."""
+    name: str
+    config: dict
+    decay_rank: int
+    gate_rank: int
+
+    @property
+    def vocab_size(self) -> int:
+        return self.config["vocab"]
+
+    def tensors(self) -> Iterator[Tuple[str, int, Tuple[int, ...], str]]:
+        """(checkpoint name, ggml type, dims fastest-first, 'normal' | 'ones')"""
+        c = self.config
+        W = c["width"]
+        def mat(name, rows, cols):
+            return name, TYPE_BF16, (cols, rows), "normal"
+        def vec(name, n, kind="ones"):
+            return name, TYPE_BF16, (n,), kind
+        yield mat("embed", c["vocab"], W)
+        for i, ly in enumerate(c["layers"]):
+            m, p = ly["mixer"], f"l{i}.mix."
+            H, D, E = m["heads"], m["dim"], m["vdim"]
+            yield vec(f"l{i}.norm1", W)
+            if ly["type"] == "channel_delta":
+                nk = m["kv_heads"] * D
+                for t, n in (("q", nk), ("k", nk), ("v", H * E)):
+                    yield mat(p + t, n, W)
+                    yield mat(p + t + ".conv", n, m["conv"])
+                yield mat(p + "b", H, W)
+                yield vec(p + "A_log", H, "normal")
+                yield vec(p + "norm", E)
+                yield mat(p + "a1", self.decay_rank, W)
+                yield mat(p + "a2", H * D, self.decay_rank)
+                yield vec(p + "dt_bias", H * D, "normal")
+                yield mat(p + "g1", self.gate_rank, W)
+                yield mat(p + "g2", H * E, self.gate_rank)
+                yield mat(p + "o", W, H * E)
+            else:
+                C_, R, Q = m["kv_rank"], m["rot_dim"], m["q_rank"]
+                yield mat(p + "dq", Q, W)
+                yield vec(p + "dq.norm", Q)
+                yield mat(p + "uq", H * (D + R), Q)
+                yield mat(p + "dkv", C_ + R, W)
+                yield vec(p + "dkv.norm", C_)
+                yield mat(p + "uk", H * D, C_)
+                yield mat(p + "uv", H * E, C_)
+                yield mat(p + "o", W, H * E)
+            if ly["mlp"] is not None:
+                F = ly["mlp"]["ff"]
+                yield vec(f"l{i}.norm2", W)
+                yield mat(f"l{i}.mlp.up", F, W)
+                yield mat(f"l{i}.mlp.down", W, F)
+        yield vec("final.norm", W)
+        yield mat("head", c["vocab"], W)
+
+
+def layered_spec(name: str, width: int, pattern: str, ff: int, vocab: int, heads: int, head_dim: int = 128, q_rank: int = 1536, kv_rank: int = 512,
+                 rot_dim: int = 64, low_rank: int = 128) -> LayeredSpec:
+    """pattern: one letter per layer, d = gated delta rule, a = latent attention, each with a feed-forward of `ff`."""
+    delta = {"heads": heads, "kv_heads": heads, "dim": head_dim, "vdim": head_dim, "conv": 4}
+    latent = {"heads": heads, "dim": head_dim, "rot_dim": rot_dim, "vdim": head_dim, "kv_rank": kv_rank, "q_rank": q_rank,
+              "scale": (head_dim + rot_dim) ** -0.5,
+              "rot": {"dims": rot_dim, "base": 10000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    layers = [{"type": "channel_delta" if ch == "d" else "latent_attention", "mixer": dict(delta if ch == "d" else latent),
+               "mlp": {"kind": "dense", "ff": ff}} for ch in pattern]
+    config = {"architecture": "Varasun", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "logit_softcap": 30.0, "layers": layers}
+    return LayeredSpec(name, config, low_rank, low_rank)
+
+
+def build_layered_engine(spec: LayeredSpec, seed: int = WEIGHT_SEED, **engine_kwargs):
+    """An `Engine` holding the synthetic model, every tensor synthesised on the device."""
+    from .engine import Engine
+    eng = Engine.from_config(spec.config, **engine_kwargs)
+    for name, typ, dims, kind in spec.tensors():
+        if kind == "ones":
+            eng.set_tensor(name, TYPE_F32, dims, np.ones(int(np.prod(dims)), np.float32))
+        else:
+            eng.synth_tensor(name, typ, dims, seed, SIGMA)
+    eng.finalize()
+    return eng
 
 
 def host_tensor(typ: int, seed: int, name: str, n_elems: int, sigma: float = SIGMA) -> np.ndarray:
