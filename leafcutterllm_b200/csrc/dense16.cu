@@ -3,8 +3,9 @@
 // bf16 activations: dense_umma_kernel, tcgen05.mma kind::f16 with f32 accumulators in tensor memory.  The WEIGHT rows are the
 // M of the instruction (128 per tile) and the tokens its N (16 .. 256), so the same kernel streams the weights of a
 // one-token decode step at memory speed and multiplies prefill chunks at tensor-core speed:
-//   warp 0   one thread requests TMA boxes of 64 elements of k x 128 weight rows and x N tokens (128-byte swizzle) into a
-//            ring of stages; the first weight boxes leave before the kernel waits for its predecessor;
+//   warp 0   one thread fills a ring of stages: per 64 elements of k one bulk copy of a 128-row weight block, which lies
+//            contiguous and ready swizzled in memory, and one TMA box of N tokens (128-byte swizzle); the first weight
+//            blocks leave before the kernel waits for its predecessor;
 //   warp 1   one thread issues the products of a stage (four K = 16 steps) and commits them to the stage's "empty" barrier;
 //   warps 4-11  read finished accumulators (two sets, so the next tile's products overlap), apply the epilogue and store;
 //            lane = weight row, so a warp's store of one token is contiguous.
@@ -36,7 +37,7 @@ struct DenseParams {
     int* error_flag;
     const float *e0, *e1;
     size_t out_batch;
-    int n, T, ldo, kblocks, mt, nt, batch, shares, items, stages;
+    int n, T, ldo, kblocks, mt, nt, batch, shares, items, stages, stage_tx;
     int out_f32, epi, e_div;
     float scale, cap;
 };
@@ -88,7 +89,7 @@ __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int r
 
 template <int NT>
 __global__ void __launch_bounds__(kThreads, NT <= 64 ? 2 : 1)
-dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant__ CUtensorMap tx, const DenseParams p) {
+dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ CUtensorMap tx, const DenseParams p) {
     constexpr int kBBytes = NT * kKB * 2, kStage = kABytes + kBBytes;
     constexpr uint32_t kCols = NT < 32 ? 32 : NT;  // tensor-memory columns of one accumulator set
     constexpr uint32_t kAlloc = 2 * kCols;
@@ -125,6 +126,7 @@ dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant_
         r.k1 = (int)((long long)p.kblocks * (r.share + 1) / p.shares);
         return r;
     };
+    auto block = [&](const Item& r, int kb) { return w + (((size_t)r.b * p.mt + r.m) * p.kblocks + kb) * kABytes; };
     if (warp == 0 && lane == 0) {
         int issued = 0;
         bool ok = true;
@@ -133,24 +135,26 @@ dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant_
         {
             const Item r = item_of(blockIdx.x);
             for (; pre < p.stages && r.k0 + pre < r.k1; pre++) {
-                mbar_expect_tx(&full[pre], kStage);
-                tma_load_3d(smem + (size_t)pre * kStage, &tw, (r.k0 + pre) * kKB, r.m * kM, r.b, &full[pre]);
+                mbar_expect_tx(&full[pre], p.stage_tx);
+                bulk_load(smem + (size_t)pre * kStage, block(r, r.k0 + pre), kABytes, &full[pre]);
             }
         }
         pdl_wait();
+        int st = 0;
+        uint32_t phase = 1;  // parity of the "empty" phase to wait for; the first round finds every stage free
         for (int it = blockIdx.x; it < p.items && ok; it += gridDim.x) {
             const Item r = item_of(it);
-            for (int kb = r.k0; kb < r.k1; kb++) {
-                const int st = issued % p.stages, round = issued / p.stages;
+            const unsigned char* wb = block(r, r.k0);
+            for (int kb = r.k0; kb < r.k1; kb++, wb += kABytes) {
                 unsigned char* a = smem + (size_t)st * kStage;
                 if (issued >= pre) {
-                    if (round > 0 && !mbar_wait(&empty[st], (uint32_t)(round - 1) & 1)) { ok = false; break; }
-                    mbar_expect_tx(&full[st], kStage);
-                    tma_load_3d(a, &tw, kb * kKB, r.m * kM, r.b, &full[st]);
+                    if (issued >= p.stages && !mbar_wait(&empty[st], phase)) { ok = false; break; }
+                    mbar_expect_tx(&full[st], p.stage_tx);
+                    bulk_load(a, wb, kABytes, &full[st]);
                 }
                 tma_load_3d(a + kABytes, &tx, kb * kKB, r.b, r.n * NT, &full[st]);
                 issued++;
-                if (*stop) { ok = false; break; }
+                if (++st == p.stages) { st = 0; phase ^= 1; }
             }
         }
         if (!ok) {
@@ -160,22 +164,24 @@ dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant_
         }
     } else if (warp == 1 && lane == 0) {
         const uint32_t idesc = idesc_bf16(kM, NT);
-        int used = 0, tile = 0;
+        const uint64_t desc0 = umma_desc_sw128(smem_u32(smem));  // a start address below 256 KB: adding to the descriptor moves it
+        int tile = 0, st = 0;
+        uint32_t phase = 0;
         bool ok = true;
         for (int it = blockIdx.x; it < p.items && ok; it += gridDim.x, tile++) {
             const Item r = item_of(it);
             const int set = tile & 1;
             if (tile >= 2 && !mbar_wait(&acc_empty[set], (uint32_t)(tile / 2 - 1) & 1)) { ok = false; break; }
             tc_fence_after();
-            for (int kb = r.k0; kb < r.k1; kb++, used++) {
-                const int st = used % p.stages;
-                if (!mbar_wait(&full[st], (uint32_t)(used / p.stages) & 1)) { ok = false; break; }
+            const uint32_t d = tmem + (uint32_t)set * kCols;
+            for (int kb = r.k0; kb < r.k1; kb++) {
+                if (!mbar_wait(&full[st], phase)) { ok = false; break; }
                 tc_fence_after();
-                const uint32_t a = smem_u32(smem + (size_t)st * kStage);
-                const uint64_t da = umma_desc_sw128(a), db = umma_desc_sw128(a + kABytes);
+                const uint64_t da = desc0 + (uint64_t)st * (kStage / 16), db = da + kABytes / 16;
 #pragma unroll
-                for (int k = 0; k < 4; k++) umma_f16_ss(tmem + (uint32_t)set * kCols, da + 2 * k, db + 2 * k, idesc, kb > r.k0 || k > 0);
+                for (int k = 0; k < 4; k++) umma_f16_ss(d, da + 2 * k, db + 2 * k, idesc, kb > r.k0 || k > 0);
                 umma_commit(&empty[st]);
+                if (++st == p.stages) { st = 0; phase ^= 1; }
             }
             if (ok) umma_commit(&acc_full[set]);
         }
@@ -236,12 +242,13 @@ dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant_
                         float v[16];
                         const int m = p.T - t0 - c;
 #pragma unroll
-                        for (int j = 0; j < 16; j++) {
-                            v[j] = 0.0f;
-                            if (j < m)
-#pragma unroll 4
-                                for (int sh = 0; sh < p.shares; sh++) v[j] += __ldcg(part + (size_t)sh * plane + (size_t)(c + j) * kM + row_in);
-                        }
+                        for (int j = 0; j < 16; j++) v[j] = 0.0f;
+                        const float* ps = part + (size_t)c * kM + row_in;
+#pragma unroll 2
+                        for (int sh = 0; sh < p.shares; sh++, ps += plane)
+#pragma unroll
+                            for (int j = 0; j < 16; j++)
+                                if (j < m) v[j] += __ldcg(ps + j * kM);
                         dense_store16(p, r.b, row, t0 + c, v, ea, eb);
                     }
                 }
@@ -254,6 +261,23 @@ dense_umma_kernel(const __grid_constant__ CUtensorMap tw, const __grid_constant_
     __syncthreads();
     tc_fence_after();
     if (warp == 2) tmem_free(tmem, kAlloc);
+}
+
+// One 16-byte chunk (eight elements of k of one row) per thread and turn; chunk c of row r of a block sits at c ^ (r & 7).
+__global__ void tile_kernel(const __nv_bfloat16* __restrict__ src, int n, int k, int ld, size_t batch_stride, size_t chunks, uint4* __restrict__ dst) {
+    const int mt = (n + kM - 1) / kM, kblocks = (k + kKB - 1) / kKB;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < chunks; i += (size_t)gridDim.x * blockDim.x) {
+        const int c = (int)(i & 7) ^ (int)((i >> 3) & 7), r_in = (int)(i >> 3) & (kM - 1);
+        size_t b = i >> 10;
+        const int kb = (int)(b % kblocks);
+        b /= kblocks;
+        const int row = (int)(b % mt) * kM + r_in, k0 = kb * kKB + c * 8;
+        b /= mt;
+        alignas(16) __nv_bfloat16 v[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) v[j] = row < n && k0 + j < k ? src[b * batch_stride + (size_t)row * ld + k0 + j] : __float2bfloat16_rn(0.0f);
+        dst[i] = *(const uint4*)v;
+    }
 }
 
 // True 32-bit: 64 weight rows x 64 tokens per CTA, 4 x 4 outputs per thread.
@@ -311,7 +335,7 @@ int32_t launch_umma(const DenseArgs& a, const CUtensorMap& tx, DenseParams p, cu
     const size_t smem = fixed + (size_t)p.stages * stage;
     LC_CUDA(ensure_smem_limit((const void*)dense_umma_kernel<NT>, smem));
     const int grid = std::min(p.items, sm_count());
-    LC_CUDA(launch_pdl(dense_umma_kernel<NT>, dim3((unsigned)grid), dim3(kThreads), smem, s, *(const CUtensorMap*)a.w->tmap, tx, p));
+    LC_CUDA(launch_pdl(dense_umma_kernel<NT>, dim3((unsigned)grid), dim3(kThreads), smem, s, a.w->tiles, tx, p));
     return LC_OK;
 }
 
@@ -324,8 +348,18 @@ int32_t dense_weight_init(DenseWeight* w, const __nv_bfloat16* data, int n, int 
     w->data = data; w->n = n; w->k = k; w->ld = ld; w->batch = batch; w->batch_stride = batch_stride;
     LC_CHECK(n > 0 && k > 0 && ld >= k && ld % 8 == 0 && batch >= 1 && batch_stride % 8 == 0 && (uintptr_t)data % 16 == 0, LC_ERR_INVALID,
              "dense weight [%d x %d], rows %d apart: layout", n, k, ld);
-    w->has_tmap = make_bf16_tmap_3d(w->tmap, data, (uint64_t)k, (uint64_t)n, (uint64_t)batch, (uint64_t)ld, batch > 1 ? batch_stride : (uint64_t)ld * n, kKB, kM, 1);
-    LC_CHECK(w->has_tmap, LC_ERR_CUDA, "dense weight [%d x %d]: no tensor map", n, k);
+    w->tiles = nullptr;
+    return LC_OK;
+}
+
+size_t dense_tile_bytes(const DenseWeight& w) { return (size_t)w.batch * ((w.n + kM - 1) / kM) * ((w.k + kKB - 1) / kKB) * kABytes; }
+
+int32_t dense_weight_tile(DenseWeight* w, void* dst, cudaStream_t s) {
+    const size_t chunks = dense_tile_bytes(*w) / 16;
+    tile_kernel<<<(unsigned)std::min<size_t>((chunks + 255) / 256, (size_t)sm_count() * 32), 256, 0, s>>>(w->data, w->n, w->k, w->ld, w->batch_stride, chunks, (uint4*)dst);
+    LC_CUDA(cudaGetLastError());
+    w->tiles = (const unsigned char*)dst;
+    w->data = nullptr;
     return LC_OK;
 }
 
@@ -333,7 +367,7 @@ int32_t dense_workspace_alloc(DenseWorkspace* ws) {
     LC_CUDA(cudaMalloc((void**)&ws->partial, kPartialBytes));
     ws->partial_bytes = kPartialBytes;
     LC_CUDA(cudaMalloc((void**)&ws->tickets, kMaxTickets * sizeof(unsigned)));
-    LC_CUDA(cudaMemset(ws->tickets, 0, kMaxTickets * sizeof(unsigned)));
+    LC_CUDA(cudaMemsetAsync(ws->tickets, 0, kMaxTickets * sizeof(unsigned), stream()));
     ws->max_tickets = kMaxTickets;
     return LC_OK;
 }
@@ -353,34 +387,49 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     p.n = w.n; p.T = a.T; p.ldo = a.ldo; p.batch = w.batch;
     p.out_f32 = a.out_f32 || a.f32; p.epi = a.epi; p.e_div = a.e_div; p.scale = a.scale; p.cap = a.cap;
     p.error_flag = gemv_error_flag_dev();
+    LC_CHECK(a.f32 ? w.data != nullptr : w.tiles != nullptr, LC_ERR_STATE, "dense product: the weight is not in the form this product reads");
     if (a.f32) {
         LC_CUDA(launch_pdl(dense_f32_kernel, dim3((unsigned)((w.n + 63) / 64), (unsigned)((a.T + 63) / 64), (unsigned)w.batch), dim3(256), 0, s, w.data,
                            w.ld, w.batch_stride, (const float*)a.x, a.ldx, a.x_batch, w.k, p));
         return LC_OK;
     }
-    const int NT = a.T <= 16 ? 16 : a.T <= 32 ? 32 : a.T <= 64 ? 64 : a.T <= 128 ? 128 : 256;
+    const int sms = sm_count();
     p.kblocks = (w.k + kKB - 1) / kKB;
     p.mt = (w.n + kM - 1) / kM;
+    // tokens per tile: what finishes first at the measured time of one block of k (in hundredths of a microsecond)
+    static const struct { int nt, t; } kSizes[] = {{16, 17}, {32, 17}, {64, 19}, {128, 24}, {256, 36}};
+    int NT = 16;
+    long best_nt = -1;
+    for (const auto& z : kSizes) {
+        const long tiles = (long)p.mt * ((a.T + z.nt - 1) / z.nt) * w.batch, cost = (tiles + sms - 1) / sms * z.t;
+        if (a.T <= 64 ? z.nt >= a.T && best_nt < 0 : z.nt >= 64 && (best_nt < 0 || cost < best_nt)) { best_nt = cost; NT = z.nt; }
+    }
     p.nt = (a.T + NT - 1) / NT;
-    const int cells = p.mt * p.nt * w.batch, sms = sm_count();
+    const int cells = p.mt * p.nt * w.batch;
     p.shares = 1;
-    if (NT <= 64 && cells <= ws.max_tickets) {  // cut k where that evens out the CTAs' work: k blocks of the busiest CTA, plus two per item
+    if (NT <= 64 && cells <= ws.max_tickets) {  // cut k where that evens out the CTAs' work: k blocks of the busiest CTA, plus what an item
+        // and the summing of the shares cost
         long best = -1;
         for (int c = 1; c <= std::min(16, p.kblocks / 2); c++) {
             if ((size_t)cells * c * NT * kM * sizeof(float) > ws.partial_bytes) break;
-            const long waves = ((long)cells * c + sms - 1) / sms, cost = waves * (((p.kblocks + c - 1) / c) + 2) + (c > 1 ? 3 : 0);
+            const long waves = ((long)cells * c + sms - 1) / sms;
+            const long cost = waves * (((p.kblocks + c - 1) / c) + 2 + (c > 1 ? NT / 16 : 0)) + (c > 1 ? 3 + c * NT / 32 : 0);
             if (best < 0 || cost < best) { best = cost; p.shares = c; }
         }
     }
     p.items = cells * p.shares;
     p.partial = ws.partial; p.tickets = ws.tickets;
     LC_CHECK((uintptr_t)a.x % 16 == 0 && a.ldx % 8 == 0 && a.x_batch % 8 == 0 && a.x_rows >= a.T, LC_ERR_INVALID, "dense product: activation layout");
-    const std::vector<uint64_t> key = {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_batch, (uint64_t)w.batch, (uint64_t)a.x_rows, (uint64_t)NT};
+    // a single tile of fewer tokens than NT brings only those: what the other rows of the operand hold reaches columns that
+    // are never read
+    const int box = std::min(NT, a.T);
+    p.stage_tx = kABytes + box * kKB * 2;
+    const std::vector<uint64_t> key = {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_batch, (uint64_t)w.batch, (uint64_t)a.x_rows, (uint64_t)box};
     std::unique_ptr<DenseWorkspace::Map>& mp = ws.maps[key];
     if (!mp) {
         mp.reset(new DenseWorkspace::Map);
         // order (k, matrix, token): a token tile is one box
-        const bool ok = make_bf16_tmap_3d(mp->b, a.x, (uint64_t)w.k, (uint64_t)w.batch, (uint64_t)a.x_rows, w.batch > 1 ? a.x_batch : (uint64_t)a.ldx, (uint64_t)a.ldx, kKB, 1, (uint32_t)NT);
+        const bool ok = make_bf16_tmap_3d(mp->b, a.x, (uint64_t)w.k, (uint64_t)w.batch, (uint64_t)a.x_rows, w.batch > 1 ? a.x_batch : (uint64_t)a.ldx, (uint64_t)a.ldx, kKB, 1, (uint32_t)box);
         if (!ok) ws.maps.erase(key);
         LC_CHECK(ok, LC_ERR_CUDA, "dense product: no tensor map over the activations");
     }

@@ -706,6 +706,7 @@ int32_t lc_model_get_tensor(lc_model* m, const char* name, void* out_bytes, size
     LC_CHECK(name && out_bytes, LC_ERR_INVALID, "get_tensor: null argument");
     auto it = m->tensors.find(canonical_name(name));
     LC_CHECK(it != m->tensors.end(), LC_ERR_MISSING, "tensor %s was never set", name);
+    LC_CHECK(it->second.view != nullptr, LC_ERR_STATE, "tensor %s lives on in another layout only", name);
     LC_CHECK(it->second.nbytes == nbytes, LC_ERR_INVALID, "tensor %s holds %zu bytes, %zu requested", name, it->second.nbytes, nbytes);
     LC_CUDA(cudaMemcpyAsync(out_bytes, it->second.view, nbytes, cudaMemcpyDeviceToHost, m->stream));
     LC_CUDA(cudaStreamSynchronize(m->stream));
@@ -920,7 +921,7 @@ int32_t lc_model_finalize(lc_model* m) {
     LC_TRY(check_model(m, false));
     LC_CHECK(!m->finalized, LC_ERR_STATE, "model already finalized");
     DeviceGuard dg(m->device);
-    LC_TRY(m->stack ? stack_bind(m) : bind_blocks(m));
+    if (!m->stack) LC_TRY(bind_blocks(m));
     const int H = m->H, V = m->V;
 
     // weight sanity scan (loader.rs:241-249) and resident byte count
@@ -937,6 +938,7 @@ int32_t lc_model_finalize(lc_model* m) {
     LC_CUDA(cudaStreamSynchronize(m->stream));
     m->ctr.sanitize_hits = bad;
     m->ctr.weight_bytes = wbytes;
+    if (m->stack) LC_TRY(stack_bind(m));  // rewrites the weights, so behind the scan
 
     // KV pools and the page table
     if (!m->stack) LC_TRY(alloc_block_pools(m));

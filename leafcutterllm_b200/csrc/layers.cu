@@ -21,8 +21,44 @@ int32_t zalloc(LayerStack& st, void** p, size_t bytes) {
     uint8_t* q = nullptr;
     LC_TRY(dalloc(&q, bytes));
     st.owned.push_back(q);
-    LC_CUDA(cudaMemset(q, 0, std::max<size_t>(bytes, 16)));
+    LC_CUDA(cudaMemsetAsync(q, 0, std::max<size_t>(bytes, 16), stream()));
     *p = q;
+    return LC_OK;
+}
+
+// The same for a plain copy of a weight.
+int32_t talloc(LayerStack& st, void** p, size_t bytes) {
+    LC_TRY(zalloc(st, p, bytes));
+    st.temps.push_back(st.owned.back());
+    st.owned.pop_back();
+    return LC_OK;
+}
+
+// bf16 products read weights in blocks: builds them for `ws`, then drops the plain copies and the checkpoint's tensors they
+// came from.  A model in true 32-bit keeps the plain forms.
+int32_t block_weights(lc_model* m, std::vector<DenseWeight*> ws) {
+    LayerStack& st = *m->stack;
+    if (st.f32) {
+        st.owned.insert(st.owned.end(), st.temps.begin(), st.temps.end());
+        st.temps.clear();
+        return LC_OK;
+    }
+    for (DenseWeight* w : ws) {
+        if (!w->data) continue;
+        uint8_t* p = nullptr;
+        LC_TRY(dalloc(&p, dense_tile_bytes(*w)));
+        st.owned.push_back(p);
+        LC_TRY(dense_weight_tile(w, p, m->stream));
+    }
+    LC_CUDA(cudaStreamSynchronize(m->stream));
+    for (void* p : st.temps) cudaFree(p);
+    st.temps.clear();
+    for (const std::string& name : st.packed) {
+        DevTensor& t = m->tensors[name];
+        if (t.dev) cudaFree(t.dev);
+        t.dev = t.view = nullptr;
+    }
+    st.packed.clear();
     return LC_OK;
 }
 
@@ -35,6 +71,7 @@ int32_t matrix(lc_model* m, const std::string& name, int rows, int cols, DevTens
     LC_CHECK((rows == 0 || (int)t.rows == rows) && (cols == 0 || (int)t.cols == cols), LC_ERR_INVALID, "tensor %s is [%zu x %zu], expected [%d x %d]", name.c_str(),
              t.rows, t.cols, rows, cols);
     *out = &t;
+    m->stack->packed.push_back(name);
     return LC_OK;
 }
 
@@ -47,30 +84,23 @@ int32_t plain_weight(lc_model* m, const std::string& name, int n, int k, DenseWe
     if (k_out == k && k % 8 == 0) return dense_weight_init(w, (const bf16*)t->view, n, k, k);
     void* p = nullptr;
     const int ld = round8(k_out);
-    LC_TRY(zalloc(*m->stack, &p, (size_t)n * ld * 2));
+    LC_TRY(talloc(*m->stack, &p, (size_t)n * ld * 2));
     LC_TRY(launch_pack((const bf16*)t->view, n, k, (bf16*)p, ld, PackMap(), col, false, m->stream));
     return dense_weight_init(w, (const bf16*)p, n, k_out, ld);
 }
 
 // Several matrices over the same input as one, each part's rows starting at a multiple of eight; `offs` receives the starts.
-// Parts whose rows are copied as they are keep being readable under their names, without a second copy.
 int32_t fused_weight(lc_model* m, const std::vector<std::string>& names, const std::vector<int>& rows, int k, DenseWeight* w, std::vector<int>* offs) {
     int total = 0;
     for (int r : rows) { offs->push_back(total); total += round8(r); }
     const int ld = round8(k);
     void* p = nullptr;
-    LC_TRY(zalloc(*m->stack, &p, (size_t)total * ld * 2));
+    LC_TRY(talloc(*m->stack, &p, (size_t)total * ld * 2));
     for (size_t i = 0; i < names.size(); i++) {
         DevTensor* t = nullptr;
         LC_TRY(matrix(m, names[i], rows[i], k, &t));
         bf16* dst = (bf16*)p + (size_t)(*offs)[i] * ld;
         LC_TRY(launch_pack((const bf16*)t->view, rows[i], k, dst, ld, PackMap(), PackMap(), false, m->stream));
-        if (ld == k && t->dev) {
-            LC_CUDA(cudaStreamSynchronize(m->stream));
-            cudaFree(t->dev);
-            t->dev = nullptr;
-            t->view = dst;
-        }
     }
     return dense_weight_init(w, (const bf16*)p, total, k, ld);
 }
@@ -115,7 +145,8 @@ int32_t bind_delta(lc_model* m, StackLayer& L, const std::string& p) {
     for (float& v : h) v = std::exp(v);
     void* ae = nullptr;
     LC_TRY(zalloc(st, &ae, h.size() * 4));
-    LC_CUDA(cudaMemcpy(ae, h.data(), h.size() * 4, cudaMemcpyHostToDevice));
+    LC_CUDA(cudaMemcpyAsync(ae, h.data(), h.size() * 4, cudaMemcpyHostToDevice, m->stream));
+    LC_CUDA(cudaStreamSynchronize(m->stream));
     L.a_exp = (const float*)ae;
     LC_TRY(model_gain_f32(m, p + "dt_bias", nd, &L.dt_bias));
     LC_TRY(model_gain_f32(m, p + "norm", s.vdim, &L.o_norm));
@@ -131,7 +162,7 @@ int32_t rot_table(lc_model* m, const RotarySpec& r, const float2** out) {
     rotary_frequencies(r, &freq, &mag);
     void *d = nullptr, *tab = nullptr;
     LC_TRY(zalloc(st, &d, freq.size() * 8));
-    LC_CUDA(cudaMemcpy(d, freq.data(), freq.size() * 8, cudaMemcpyHostToDevice));
+    LC_CUDA(cudaMemcpyAsync(d, freq.data(), freq.size() * 8, cudaMemcpyHostToDevice, m->stream));
     LC_TRY(zalloc(st, &tab, freq.size() * (size_t)m->cfg.max_seq_len * sizeof(float2)));
     LC_TRY(launch_rot_table((const double*)d, (int)freq.size(), mag, m->cfg.max_seq_len, (float2*)tab, m->stream));
     LC_CUDA(cudaStreamSynchronize(m->stream));
@@ -164,7 +195,7 @@ int32_t bind_latent(lc_model* m, StackLayer& L, const std::string& p) {
     } else {
         void* u = nullptr;
         const int ld = round8(qr);
-        LC_TRY(zalloc(st, &u, (size_t)s.heads * g.ld_q * ld * 2));
+        LC_TRY(talloc(st, &u, (size_t)s.heads * g.ld_q * ld * 2));
         LC_TRY(launch_pack((const bf16*)t->view, s.heads * (s.dim + s.rot_dim), qr, (bf16*)u, ld, PackMap{s.dim + s.rot_dim, g.ld_q, s.dim, g.dp - s.dim}, PackMap(),
                            false, m->stream));
         LC_TRY(dense_weight_init(&L.uq, (const bf16*)u, s.heads * g.ld_q, qr, ld));
@@ -172,14 +203,14 @@ int32_t bind_latent(lc_model* m, StackLayer& L, const std::string& p) {
     // key projection, transposed per head: [heads][rank][dim]
     LC_TRY(matrix(m, p + "uk", s.heads * s.dim, s.kv_rank, &t));
     void* kt = nullptr;
-    LC_TRY(zalloc(st, &kt, (size_t)s.heads * s.kv_rank * g.dp * 2));
+    LC_TRY(talloc(st, &kt, (size_t)s.heads * s.kv_rank * g.dp * 2));
     LC_TRY(launch_pack((const bf16*)t->view, s.heads * s.dim, s.kv_rank, (bf16*)kt, g.dp, PackMap{s.dim, s.kv_rank, 0, 0}, PackMap(), true, m->stream));
     LC_TRY(dense_weight_init(&L.uk_t, (const bf16*)kt, s.kv_rank, s.dim, g.dp, s.heads, (size_t)s.kv_rank * g.dp));
     LC_TRY(matrix(m, p + "uv", s.heads * s.vdim, s.kv_rank, &t));
     const bf16* uv = (const bf16*)t->view;
     if (g.cp != s.kv_rank) {
         void* v = nullptr;
-        LC_TRY(zalloc(st, &v, (size_t)s.heads * s.vdim * g.cp * 2));
+        LC_TRY(talloc(st, &v, (size_t)s.heads * s.vdim * g.cp * 2));
         LC_TRY(launch_pack(uv, s.heads * s.vdim, s.kv_rank, (bf16*)v, g.cp, PackMap(), PackMap(), false, m->stream));
         uv = (const bf16*)v;
     }
@@ -192,7 +223,7 @@ int32_t bind_latent(lc_model* m, StackLayer& L, const std::string& p) {
             LC_TRY(matrix(m, p + name, s.heads * per, s.kv_rank, &wt));
             if (per == per_p && g.cp == s.kv_rank) return dense_weight_init(w, (const bf16*)wt->view, s.heads * per, s.kv_rank, s.kv_rank);
             void* q = nullptr;
-            LC_TRY(zalloc(st, &q, (size_t)s.heads * per_p * g.cp * 2));
+            LC_TRY(talloc(st, &q, (size_t)s.heads * per_p * g.cp * 2));
             LC_TRY(launch_pack((const bf16*)wt->view, s.heads * per, s.kv_rank, (bf16*)q, g.cp, PackMap{per, per_p, 0, 0}, PackMap(), false, m->stream));
             return dense_weight_init(w, (const bf16*)q, s.heads * per_p, s.kv_rank, g.cp);
         };
@@ -314,15 +345,16 @@ int32_t stack_bind(lc_model* m) {
             LC_TRY(plain_weight(m, p + "mlp.down", sp.width, L.s.ff, &L.down));
             LC_TRY(model_gain_f32(m, p + "norm2", sp.width, &L.norm2));
         }
+        LC_TRY(block_weights(m, {&L.in, &L.out, &L.up, &L.down, &L.a2, &L.g2, &L.uq, &L.uk_t, &L.uv, &L.uk_all, &L.uv_all}));
     }
     DevTensor* e = nullptr;
     LC_TRY(matrix(m, "embed", sp.vocab, sp.width, &e));
     st.embed = (const bf16*)e->view;
+    st.packed.clear();  // the embedding table is read as it is
     m->embed = e;
     LC_TRY(model_gain_f32(m, "final.norm", sp.width, &st.final_norm));
     LC_TRY(plain_weight(m, "head", sp.vocab, sp.width, &st.head));
-    LC_CUDA(cudaStreamSynchronize(m->stream));
-    return LC_OK;
+    return block_weights(m, {&st.head});
 }
 
 int32_t stack_alloc(lc_model* m) {
@@ -379,6 +411,7 @@ int32_t stack_alloc(lc_model* m) {
 void stack_free(lc_model* m) {
     if (!m->stack) return;
     for (void* p : m->stack->owned) cudaFree(p);
+    for (void* p : m->stack->temps) cudaFree(p);
     for (DevBuf* b : {&m->stack->ctx_c, &m->stack->ctx_k, &m->stack->ctx_v}) b->release();
     dense_workspace_free(&m->stack->ws);
 }

@@ -18,10 +18,12 @@ struct DenseWeight {
     const __nv_bfloat16* data = nullptr;
     int n = 0, k = 0, ld = 0, batch = 1;
     size_t batch_stride = 0;
-    alignas(64) unsigned char tmap[128];
-    bool has_tmap = false;
+    const unsigned char* tiles = nullptr;  // the tensor-core form: [matrix][n / 128][k / 64] blocks of 128 rows x 128 bytes, swizzled, zero-padded
 };
 int32_t dense_weight_init(DenseWeight* w, const __nv_bfloat16* data, int n, int k, int ld, int batch = 1, size_t batch_stride = 0);
+// Rewrites the plain matrix into blocks at dst (dense_tile_bytes of them), after which `data` is no longer read.
+size_t dense_tile_bytes(const DenseWeight& w);
+int32_t dense_weight_tile(DenseWeight* w, void* dst, cudaStream_t s);
 
 enum DenseEpilogue {
     DENSE_STORE = 0,
@@ -176,6 +178,8 @@ struct LayerStack {
     const float* final_norm = nullptr;
     DenseWorkspace ws;
     std::vector<void*> owned;
+    std::vector<void*> temps;          // plain copies of weights, dropped once their blocks exist
+    std::vector<std::string> packed;   // checkpoint tensors whose bytes live on in blocks only
     std::vector<std::pair<RotarySpec, const float2*>> rot_tables;
     uint64_t cache_bytes_per_token = 0, state_bytes_per_seq = 0;
     // step buffers for t_cap tokens

@@ -181,60 +181,76 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
 #pragma unroll
             for (int j = 0; j < TAPS; j++) w[c][j] = lane + 32 * c < n ? a.conv[(c0 + lane + 32 * c) * TAPS + j] : 0.0f;
     int prev_seq = -1, prev_pos = -1;
-    for (int t = t0; t < t1; t++) {
-        const int seq = a.tok_seq[t], pos = a.tok_pos[t];
-        float y[CPL], ss = 0.0f;
-        if constexpr (TAPS > 0) {
-            const bool follows = seq == prev_seq && pos == prev_pos + 1;
+    constexpr int kAhead = 4;
+    float ahead[kAhead][CPL];
+    int seq_a[kAhead], pos_a[kAhead];
+    for (int tb = t0; tb < t1; tb += kAhead) {
 #pragma unroll
-            for (int c = 0; c < CPL; c++) {
-                const int i = lane + 32 * c;
-                y[c] = 0.0f;
-                if (i >= n) continue;
-                if (!follows) {  // first token of the stretch or of a run: earlier inputs from the call's rows, the ring, or none
+        for (int u = 0; u < kAhead; u++) {
+            const int t = min(tb + u, t1 - 1);
+            seq_a[u] = a.tok_seq[t]; pos_a[u] = a.tok_pos[t];
+            if constexpr (TAPS > 0)
 #pragma unroll
-                    for (int j = 1; j < TAPS; j++) {
-                        float v = 0.0f;
-                        if (pos - j >= 0) {
-                            const int tt = t - j;
-                            if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) v = act_f<A>(proj[(size_t)tt * g.ld + col0 + i]);
-                            else v = act_f<A>(ring[((size_t)seq * TAPS + (pos - j) % TAPS) * g.channels + c0 + i]);
+                for (int c = 0; c < CPL; c++) ahead[u][c] = lane + 32 * c < n ? act_f<A>(proj[(size_t)t * g.ld + col0 + lane + 32 * c]) : 0.0f;
+        }
+#pragma unroll
+        for (int u = 0; u < kAhead; u++) {
+            const int t = tb + u;
+            if (t >= t1) break;
+            const int seq = seq_a[u], pos = pos_a[u];
+            float y[CPL], ss = 0.0f;
+            if constexpr (TAPS > 0) {
+                const bool follows = seq == prev_seq && pos == prev_pos + 1;
+#pragma unroll
+                for (int c = 0; c < CPL; c++) {
+                    const int i = lane + 32 * c;
+                    y[c] = 0.0f;
+                    if (i >= n) continue;
+                    if (!follows) {  // first token of the stretch or of a run: earlier inputs from the call's rows, the ring, or none
+#pragma unroll
+                        for (int j = 1; j < TAPS; j++) {
+                            float v = 0.0f;
+                            if (pos - j >= 0) {
+                                const int tt = t - j;
+                                if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) v = act_f<A>(proj[(size_t)tt * g.ld + col0 + i]);
+                                else v = act_f<A>(ring[((size_t)seq * TAPS + (pos - j) % TAPS) * g.channels + c0 + i]);
+                            }
+                            win[c][j - 1] = v;
                         }
-                        win[c][j - 1] = v;
                     }
+                    const float cur = ahead[u][c];
+                    float acc = 0.0f;
+#pragma unroll
+                    for (int j = TAPS - 1; j > 0; j--) acc = fmaf(w[c][TAPS - 1 - j], win[c][j - 1], acc);
+                    acc = fmaf(w[c][TAPS - 1], cur, acc);
+#pragma unroll
+                    for (int j = TAPS - 1; j > 0; j--) win[c][j] = win[c][j - 1];
+                    win[c][0] = cur;
+                    y[c] = silu32(acc);
+                    ss = fmaf(y[c], y[c], ss);
                 }
-                const float cur = act_f<A>(proj[(size_t)t * g.ld + col0 + i]);
-                float acc = 0.0f;
+                prev_seq = seq; prev_pos = pos;
+            } else {
 #pragma unroll
-                for (int j = TAPS - 1; j > 0; j--) acc = fmaf(w[c][TAPS - 1 - j], win[c][j - 1], acc);
-                acc = fmaf(w[c][TAPS - 1], cur, acc);
-#pragma unroll
-                for (int j = TAPS - 1; j > 0; j--) win[c][j] = win[c][j - 1];
-                win[c][0] = cur;
-                y[c] = silu32(acc);
-                ss = fmaf(y[c], y[c], ss);
+                for (int c = 0; c < CPL; c++) {
+                    const int i = lane + 32 * c;
+                    y[c] = i < n ? silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, col0 + i)) : 0.0f;
+                    ss = fmaf(y[c], y[c], ss);
+                }
             }
-            prev_seq = seq; prev_pos = pos;
-        } else {
-#pragma unroll
-            for (int c = 0; c < CPL; c++) {
-                const int i = lane + 32 * c;
-                y[c] = i < n ? silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, col0 + i)) : 0.0f;
-                ss = fmaf(y[c], y[c], ss);
+            float r = 1.0f;
+            float* o;
+            if (is_v) {
+                o = a.v + (size_t)t * g.heads * g.vdim + h * g.vdim;
+            } else {
+                o = a.qk + ((size_t)t * 2 + (is_k ? 1 : 0)) * g.kv_heads * g.dim + h * g.dim;
+                r = 1.0f / sqrtf(warp_sum(ss) + g.unit_eps);
+                if (!is_k) r *= 1.0f / sqrtf((float)g.dim);
             }
-        }
-        float r = 1.0f;
-        float* o;
-        if (is_v) {
-            o = a.v + (size_t)t * g.heads * g.vdim + h * g.vdim;
-        } else {
-            o = a.qk + ((size_t)t * 2 + (is_k ? 1 : 0)) * g.kv_heads * g.dim + h * g.dim;
-            r = 1.0f / sqrtf(warp_sum(ss) + g.unit_eps);
-            if (!is_k) r *= 1.0f / sqrtf((float)g.dim);
-        }
 #pragma unroll
-        for (int c = 0; c < CPL; c++)
-            if (lane + 32 * c < n) o[lane + 32 * c] = y[c] * r;
+            for (int c = 0; c < CPL; c++)
+                if (lane + 32 * c < n) o[lane + 32 * c] = y[c] * r;
+        }
     }
 }
 
