@@ -259,16 +259,19 @@ int32_t delta_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, b
     LC_TRY(product(m, L.g2, at(st, st.proj, (size_t)L.off_g), L.in.n, T, st.gate, nv));
     DeltaArgs d;
     d.g = L.dg; d.proj = st.proj; d.conv = L.conv; d.ring = L.ring; d.state = L.state; d.tok_seq = m->d_tok_seq; d.tok_pos = m->d_tok_pos; d.T = T;
-    d.qk = st.qk; d.v = st.v; d.log_decay = st.log_decay; d.o = st.o; d.runs = st.d_runs; d.n_runs = st.n_runs; d.norm_w = L.o_norm; d.gate = st.gate;
+    d.qk = st.qk; d.v = st.v; d.log_decay = st.log_decay; d.o = st.o; d.norm_w = L.o_norm; d.gate = st.gate;
     d.out = st.mixed; d.ldo = round8(nv); d.f32 = st.f32;
     if (decode_step) {
         LC_TRY(launch_delta_step(d, m->stream));
         m->launches_in_call += 1;
     } else {
         LC_TRY(launch_delta_prep(d, m->stream));
-        LC_TRY(launch_delta_scan(d, m->stream));
+        d.runs = st.d_short_runs; d.n_runs = st.n_short_runs;
+        d.chunks = st.d_chunks; d.n_chunks = st.n_chunks; d.chunk_runs = st.d_chunk_runs; d.n_chunk_runs = st.n_chunk_runs;
+        if (d.n_runs) LC_TRY(launch_delta_scan(d, m->stream));
+        if (d.n_chunk_runs) LC_TRY(launch_delta_chunks(d, (float*)st.chunk_scratch.p, m->stream));
         LC_TRY(launch_delta_output(d, m->stream));
-        m->launches_in_call += 3;
+        m->launches_in_call += 2 + (d.n_runs ? 1 : 0) + (d.n_chunk_runs ? 2 : 0);
     }
     return product(m, L.out, st.mixed, d.ldo, T, st.y, st.spec.width, true);
 }
@@ -361,7 +364,7 @@ int32_t stack_alloc(lc_model* m) {
     LayerStack& st = *m->stack;
     const size_t T = (size_t)m->t_cap, e = elt(st);
     st.width_p = round8(st.spec.width);
-    st.prefill_tiles = !st.f32;
+    st.prefill_tiles = st.delta_chunks = !st.f32;
     size_t proj = 8, projf = 8, gate = 8, mixed = 8, cq = 8, q = 8, qa = 8, ffn = 8, ld = 8, qk = 8, v = 8;
     for (StackLayer& L : st.layers) {
         const LayerSpec& s = L.s;
@@ -375,6 +378,8 @@ int32_t stack_alloc(lc_model* m) {
             v = std::max(v, nv);
             LC_TRY(zalloc(st, (void**)&L.state, (size_t)m->max_seqs * S * 4));
             LC_TRY(zalloc(st, &L.ring, (size_t)m->max_seqs * ring * e));
+            st.delta_chunks = st.delta_chunks && delta_chunks_apply(L.dg, st.f32);
+            st.chunk_bytes = std::max(st.chunk_bytes, delta_chunk_bytes(L.dg));
             st.state_bytes_per_seq += S * 4 + ring * e;
         } else {
             const LatentShape& g = L.lg;
@@ -403,6 +408,8 @@ int32_t stack_alloc(lc_model* m) {
     LC_TRY(zalloc(st, (void**)&st.y, T * st.spec.width * 4)); LC_TRY(zalloc(st, (void**)&st.log_decay, T * ld * 4));
     LC_TRY(zalloc(st, (void**)&st.qk, T * qk * 4)); LC_TRY(zalloc(st, (void**)&st.v, T * v * 4)); LC_TRY(zalloc(st, (void**)&st.o, T * v * 4));
     LC_TRY(zalloc(st, (void**)&st.d_runs, T * sizeof(SeqRun)));
+    LC_TRY(zalloc(st, (void**)&st.d_short_runs, T * sizeof(SeqRun))); LC_TRY(zalloc(st, (void**)&st.d_chunks, T * sizeof(DeltaChunk)));
+    LC_TRY(zalloc(st, (void**)&st.d_chunk_runs, T * sizeof(DeltaChunkRun)));
     LC_TRY(zalloc(st, (void**)&st.d_lat_tiles, T * sizeof(LatentTile))); LC_TRY(zalloc(st, (void**)&st.d_lat_ctx, T * sizeof(LatentContext)));
     if (st.pieces_bytes) LC_TRY(zalloc(st, &st.pieces, st.pieces_bytes));
     return LC_OK;
@@ -412,7 +419,7 @@ void stack_free(lc_model* m) {
     if (!m->stack) return;
     for (void* p : m->stack->owned) cudaFree(p);
     for (void* p : m->stack->temps) cudaFree(p);
-    for (DevBuf* b : {&m->stack->ctx_c, &m->stack->ctx_k, &m->stack->ctx_v}) b->release();
+    for (DevBuf* b : {&m->stack->ctx_c, &m->stack->ctx_k, &m->stack->ctx_v, &m->stack->chunk_scratch}) b->release();
     dense_workspace_free(&m->stack->ws);
 }
 
@@ -427,6 +434,21 @@ int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const st
     }
     st.n_runs = (int)runs.size();
     LC_CUDA(cudaMemcpyAsync(st.d_runs, runs.data(), runs.size() * sizeof(SeqRun), cudaMemcpyHostToDevice, m->stream));
+    std::vector<SeqRun> shorts;
+    std::vector<DeltaChunk> chunks;
+    std::vector<DeltaChunkRun> chunk_runs;
+    for (const SeqRun& r : runs) {
+        if (!st.delta_chunks || r.n < kChunkRun) { shorts.push_back(r); continue; }
+        chunk_runs.push_back(DeltaChunkRun{r, (int32_t)chunks.size(), (r.n + kDeltaChunk - 1) / kDeltaChunk});
+        for (int t = 0; t < r.n; t += kDeltaChunk) chunks.push_back(DeltaChunk{r.tok0 + t, std::min(kDeltaChunk, r.n - t)});
+    }
+    st.n_short_runs = (int)shorts.size(); st.n_chunks = (int)chunks.size(); st.n_chunk_runs = (int)chunk_runs.size();
+    if (!shorts.empty()) LC_CUDA(cudaMemcpyAsync(st.d_short_runs, shorts.data(), shorts.size() * sizeof(SeqRun), cudaMemcpyHostToDevice, m->stream));
+    if (!chunks.empty()) {
+        LC_CUDA(cudaMemcpyAsync(st.d_chunks, chunks.data(), chunks.size() * sizeof(DeltaChunk), cudaMemcpyHostToDevice, m->stream));
+        LC_CUDA(cudaMemcpyAsync(st.d_chunk_runs, chunk_runs.data(), chunk_runs.size() * sizeof(DeltaChunkRun), cudaMemcpyHostToDevice, m->stream));
+        LC_TRY(st.chunk_scratch.reserve(std::max(chunks.size(), (size_t)m->t_cap / kDeltaChunk) * st.chunk_bytes));
+    }
     st.groups.clear();
     st.n_short = (int)seq.size();
     std::vector<LatentTile> tiles;

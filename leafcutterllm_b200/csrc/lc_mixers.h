@@ -83,6 +83,9 @@ int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, flo
 // Gated delta rule with one decay per key channel.  `proj` rows hold q | k | v | ... | beta logits as projected; the inputs of
 // the short convolutions of the last `taps` positions live in `ring` [slot][taps][channels], entry position % taps.
 struct DeltaShape { int heads, kv_heads, dim, vdim, taps, ld, off_k, off_v, off_b, channels; float unit_eps, eps; };
+constexpr int kDeltaChunk = 64;
+struct DeltaChunk { int32_t tok0, n; };                       // up to kDeltaChunk consecutive tokens of a run
+struct DeltaChunkRun { SeqRun run; int32_t chunk0, n_chunks; };
 struct DeltaArgs {
     DeltaShape g;
     const void* proj = nullptr;
@@ -95,8 +98,11 @@ struct DeltaArgs {
     float* v = nullptr;                // [T][heads * vdim]
     const float* log_decay = nullptr;  // [T][heads * dim]
     float* o = nullptr;                // [T][heads * vdim]
-    const SeqRun* runs = nullptr;
+    const SeqRun* runs = nullptr;      // walked token by token
     int n_runs = 0;
+    const DeltaChunk* chunks = nullptr;         // longer runs (delta_chunk.cu)
+    const DeltaChunkRun* chunk_runs = nullptr;
+    int n_chunks = 0, n_chunk_runs = 0;
     const float* norm_w = nullptr;     // [vdim]
     const void* gate = nullptr;        // [T][heads * vdim] before the sigmoid
     void* out = nullptr;               // [T][ldo] activations
@@ -107,6 +113,33 @@ int32_t launch_delta_prep(const DeltaArgs& a, cudaStream_t s);   // convolutions
 int32_t launch_delta_scan(const DeltaArgs& a, cudaStream_t s);   // the recurrence over every run; leaves state and ring for the next call
 int32_t launch_delta_output(const DeltaArgs& a, cudaStream_t s); // per-head norm, gate
 int32_t launch_delta_step(const DeltaArgs& a, cudaStream_t s);   // the three for one new token per sequence (rows of tok_seq / tok_pos)
+
+// delta_chunk.cu: the recurrence over `chunk_runs`, in chunks; scratch of delta_chunk_bytes per chunk
+bool delta_chunks_apply(const DeltaShape& g, bool f32);
+size_t delta_chunk_bytes(const DeltaShape& g);
+int32_t launch_delta_chunks(const DeltaArgs& a, float* scratch, cudaStream_t s);
+
+#ifdef __CUDACC__
+// The inputs of a run's last `taps` positions, for the convolutions of the next call: head h's v channels, and the q and k
+// channels of its key head once per group.
+template <typename A>
+__device__ __forceinline__ void delta_keep_inputs(const DeltaArgs& a, const SeqRun& run, int h, int tid, int threads) {
+    const DeltaShape& g = a.g;
+    const int rep = g.heads / g.kv_heads, kh = h / rep;
+    A* ring = (A*)a.ring + (size_t)run.seq * g.taps * g.channels;
+    const A* proj = (const A*)a.proj;
+    const int m = run.n < g.taps ? run.n : g.taps, per = g.vdim + (h % rep == 0 ? 2 * g.dim : 0);
+    for (int i = tid; i < m * per; i += threads) {
+        const int j = i / per, c = i - j * per;
+        int column, channel;
+        if (c < g.vdim) { column = g.off_v + h * g.vdim + c; channel = 2 * g.kv_heads * g.dim + h * g.vdim + c; }
+        else if (c < g.vdim + g.dim) { column = kh * g.dim + c - g.vdim; channel = column; }
+        else { column = g.off_k + kh * g.dim + c - g.vdim - g.dim; channel = g.kv_heads * g.dim + kh * g.dim + c - g.vdim - g.dim; }
+        const int t = run.n - 1 - j;
+        ring[(size_t)((run.pos0 + t) % g.taps) * g.channels + channel] = proj[(size_t)(run.tok0 + t) * g.ld + column];
+    }
+}
+#endif
 
 // Cache of latent attention: per page page_tokens rows [kv_rank | pad | rot_dim | pad] of the activations' type.
 struct LatentShape { int heads, dim, rot, rank, ld_q, dp, cp, rp, rot_pairs; float scale; };  // dp, cp, rp: dim, rank, rot rounded up to 8
@@ -188,6 +221,14 @@ struct LayerStack {
     float *y = nullptr, *projf = nullptr, *log_decay = nullptr, *qk = nullptr, *v = nullptr, *o = nullptr;
     SeqRun* d_runs = nullptr;
     int n_runs = 0;
+    // gated delta rule of the call: short runs walk token by token, long ones in chunks (when every such layer has that form)
+    bool delta_chunks = false;
+    SeqRun* d_short_runs = nullptr;
+    DeltaChunk* d_chunks = nullptr;
+    DeltaChunkRun* d_chunk_runs = nullptr;
+    int n_short_runs = 0, n_chunks = 0, n_chunk_runs = 0;
+    size_t chunk_bytes = 0;            // scratch per chunk, widest layer
+    DevBuf chunk_scratch;
     // latent attention of the call: its first n_short tokens attend one by one, the others in tiles over projected contexts,
     // in groups whose contexts fit the context buffers
     struct Group { int tile0, n_tiles, ctx0, n_ctx, rows, longest; };

@@ -38,6 +38,7 @@ struct LayerW {
 
 constexpr int kPrefillChunk = 512;
 constexpr int kTileRun = 16;             // runs of fewer tokens attend token by token
+constexpr int kChunkRun = 32;            // runs of fewer tokens walk the gated delta rule token by token
 constexpr int kStackChunk = 2048;      // tokens per pass of a checkpoint-directory design
 constexpr int kTokTile = 8;
 constexpr int kMoeGroupedTokens = 64;  // calls of at most this many tokens run the experts as one grouped launch

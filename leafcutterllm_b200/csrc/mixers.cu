@@ -331,21 +331,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaArgs a) {
         const int d = (i >> 2) * 16 + r4 * 4 + (i & 3);
         if (d < g.dim && e < g.vdim) st[(size_t)d * g.vdim + e] = S[i];
     }
-    // the inputs of the last `taps` positions, for the convolutions of the next call (this head's v channels, and the q and k
-    // channels of its key head once)
-    if (blockIdx.z == 0) {
-        A* ring = (A*)a.ring + (size_t)run.seq * g.taps * g.channels;
-        const int m = min(run.n, g.taps), qk = h % rep == 0 ? 2 * g.dim : 0;
-        for (int i = threadIdx.x; i < m * (g.vdim + qk); i += 128) {
-            const int j = i / (g.vdim + qk), c = i - j * (g.vdim + qk);
-            int column, channel;
-            if (c < g.vdim) { column = g.off_v + h * g.vdim + c; channel = 2 * g.kv_heads * g.dim + h * g.vdim + c; }
-            else if (c < g.vdim + g.dim) { column = kh * g.dim + c - g.vdim; channel = column; }
-            else { column = g.off_k + kh * g.dim + c - g.vdim - g.dim; channel = g.kv_heads * g.dim + kh * g.dim + c - g.vdim - g.dim; }
-            const int t = run.n - 1 - j;
-            ring[(size_t)((run.pos0 + t) % g.taps) * g.channels + channel] = proj[(size_t)(run.tok0 + t) * g.ld + column];
-        }
-    }
+    if (blockIdx.z == 0) delta_keep_inputs<A>(a, run, h, threadIdx.x, 128);
 }
 
 // One warp per (token, head): o / rms(o) * norm * sigmoid(gate)
