@@ -42,9 +42,10 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf
 
 constexpr int kChunkThreads = 288;  // 136 lower tiles of 4 x 4 pairs, each in two halves of the channels: 272
 template <int DP>
-__global__ void __launch_bounds__(kChunkThreads) delta_chunk_kernel(const DeltaArgs a, float* __restrict__ scratch) {
+__global__ void __launch_bounds__(kChunkThreads, 2) delta_chunk_kernel(const DeltaArgs a, float* __restrict__ scratch) {
     extern __shared__ __align__(16) float sm[];
-    float *s_k = sm, *s_q = s_k + DP * kP, *s_G = s_q + DP * kP, *s_A = s_G + DP * kP, *s_B = s_A + kC * kC, *s_b = s_B + kC * kC;
+    float *s_k = sm, *s_q = s_k + DP * kP, *s_G = s_q + DP * kP, *s_b = s_G + DP * kP;
+    float* s_A = DP * kP >= kC * kC ? s_q : s_b + kC;  // takes the place of q once q has been used
     pdl_launch_dependents();
     pdl_wait();
     const DeltaShape& g = a.g;
@@ -53,20 +54,36 @@ __global__ void __launch_bounds__(kChunkThreads) delta_chunk_kernel(const DeltaA
     const ChunkLayout L{DP, padded_cols(g.vdim)};
     float* out = scratch + ((size_t)blockIdx.x * g.heads + h) * L.size();
     // channel-major copies; rows past the chunk's tokens and channels past dim are zero (no key, no decay)
-    for (int i = tid; i < kC * DP; i += kChunkThreads) {
-        const int t = i & (kC - 1), d = i / kC;
-        float q = 0.0f, k = 0.0f, l = 0.0f;
-        if (t < ck.n && d < g.dim) {
-            const size_t tok = (size_t)(ck.tok0 + t);
-            q = a.qk[tok * 2 * g.kv_heads * g.dim + kh * g.dim + d];
-            k = a.qk[(tok * 2 + 1) * g.kv_heads * g.dim + kh * g.dim + d];
-            l = a.log_decay[tok * g.heads * g.dim + h * g.dim + d] * kLog2e;
+    const int nk = g.kv_heads * g.dim;
+    if (g.dim % 4 == 0) {
+        for (int i = tid; i < kC * DP / 4; i += kChunkThreads) {
+            const int t = i & (kC - 1), d = i / kC * 4;
+            float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q, l = q;
+            if (t < ck.n && d < g.dim) {
+                const size_t tok = (size_t)(ck.tok0 + t);
+                q = *(const float4*)(a.qk + tok * 2 * nk + kh * g.dim + d);
+                k = *(const float4*)(a.qk + (tok * 2 + 1) * nk + kh * g.dim + d);
+                l = *(const float4*)(a.log_decay + tok * g.heads * g.dim + h * g.dim + d);
+            }
+            const float qq[4] = {q.x, q.y, q.z, q.w}, kk[4] = {k.x, k.y, k.z, k.w}, ll[4] = {l.x, l.y, l.z, l.w};
+#pragma unroll
+            for (int j = 0; j < 4; j++) { s_q[(d + j) * kP + t] = qq[j]; s_k[(d + j) * kP + t] = kk[j]; s_G[(d + j) * kP + t] = ll[j] * kLog2e; }
         }
-        s_q[d * kP + t] = q; s_k[d * kP + t] = k; s_G[d * kP + t] = l;
+    } else {
+        for (int i = tid; i < kC * DP; i += kChunkThreads) {
+            const int t = i & (kC - 1), d = i / kC;
+            float q = 0.0f, k = 0.0f, l = 0.0f;
+            if (t < ck.n && d < g.dim) {
+                const size_t tok = (size_t)(ck.tok0 + t);
+                q = a.qk[tok * 2 * nk + kh * g.dim + d];
+                k = a.qk[(tok * 2 + 1) * nk + kh * g.dim + d];
+                l = a.log_decay[tok * g.heads * g.dim + h * g.dim + d] * kLog2e;
+            }
+            s_q[d * kP + t] = q; s_k[d * kP + t] = k; s_G[d * kP + t] = l;
+        }
     }
     for (int i = tid; i < kC; i += kChunkThreads)
         s_b[i] = i < ck.n ? sigmoid_f(__bfloat162float(((const __nv_bfloat16*)a.proj)[(size_t)(ck.tok0 + i) * g.ld + g.off_b + h])) : 0.0f;
-    for (int i = tid; i < 2 * kC * kC; i += kChunkThreads) s_A[i] = 0.0f;  // and B behind it
     __syncthreads();
     for (int d = tid; d < DP; d += kChunkThreads) {
         float sum = 0.0f;
@@ -121,47 +138,57 @@ __global__ void __launch_bounds__(kChunkThreads) delta_chunk_kernel(const DeltaA
                 ta[i][j] += __shfl_xor_sync(m, ta[i][j], 1);
                 tb[i][j] += __shfl_xor_sync(m, tb[i][j], 1);
             }
-        if ((tid & 1) == 0) {
+        // B goes out as [s][t] with zeros above the diagonal: one half writes the tile, the other the tile across the diagonal
+        float* bt = out + L.bt();
 #pragma unroll
-            for (int i = 0; i < 4; i++)
-#pragma unroll
-                for (int j = 0; j < 4; j++) {
-                    s_A[(4 * ti + i) * kC + 4 * tj + j] = ta[i][j];
-                    s_B[(4 * tj + j) * kC + 4 * ti + i] = tb[i][j];  // [s][t]
-                }
+        for (int j = 0; j < 4; j++) {
+            if ((tid & 1) == 0) *(float4*)(bt + (4 * tj + j) * kC + 4 * ti) = make_float4(tb[0][j], tb[1][j], tb[2][j], tb[3][j]);
+            else if (ti != tj) *(float4*)(bt + (4 * ti + j) * kC + 4 * tj) = make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
-    __syncthreads();
-    for (int i = tid; i < kC * kC / 4; i += kChunkThreads) ((float4*)(out + L.bt()))[i] = ((const float4*)s_B)[i];
     for (int i = tid; i < kC * DP; i += kChunkThreads) {
         const int d = i % DP, t = i / DP;
         out[L.kh() + i] = s_k[d * kP + t] * exp2f(s_G[d * kP + kC - 1] - s_G[d * kP + t]);
     }
-    for (int i = tid; i < DP * kC; i += kChunkThreads) {
-        const int t = i & (kC - 1), d = i / kC;
-        out[L.wq() + (size_t)d * 128 + 64 + t] = s_q[d * kP + t] * exp2f(s_G[d * kP + t]);
+    for (int i = tid; i < DP * kC / 4; i += kChunkThreads) {
+        const int t = (i & (kC / 4 - 1)) * 4, d = i / (kC / 4);
+        const float4 q = *(const float4*)(s_q + d * kP + t), e = *(const float4*)(s_G + d * kP + t);
+        *(float4*)(out + L.wq() + (size_t)d * 128 + 64 + t) = make_float4(q.x * exp2f(e.x), q.y * exp2f(e.y), q.z * exp2f(e.z), q.w * exp2f(e.w));
     }
     for (int d = tid; d < DP; d += kChunkThreads) out[L.ge() + d] = exp2f(s_G[d * kP + kC - 1]);
-    // forward substitution, one column of the right-hand sides per thread
+    __syncthreads();  // q has been used
+    if (tile && (tid & 1) == 0)
+#pragma unroll
+        for (int i = 0; i < 4; i++) *(float4*)(s_A + (4 * ti + i) * kC + 4 * tj) = make_float4(ta[i][0], ta[i][1], ta[i][2], ta[i][3]);
+    __syncthreads();
+    // forward substitution, one column of the right-hand sides per thread; entries of A on and above the diagonal are not used
     for (int c = tid; c < DP + L.e; c += kChunkThreads) {
         float x[kC];
         const bool is_w = c < DP;
         const int col = is_w ? c : c - DP;
+        if (is_w) {
+#pragma unroll
+            for (int t = 0; t < kC; t += 4) {
+                const float4 k = *(const float4*)(s_k + col * kP + t), e = *(const float4*)(s_G + col * kP + t);
+                x[t] = k.x * exp2f(e.x); x[t + 1] = k.y * exp2f(e.y); x[t + 2] = k.z * exp2f(e.z); x[t + 3] = k.w * exp2f(e.w);
+            }
+        } else {
+            const float* v = a.v + (size_t)ck.tok0 * g.heads * g.vdim + h * g.vdim + col;
+#pragma unroll
+            for (int t = 0; t < kC; t++) x[t] = t < ck.n && col < g.vdim ? v[(size_t)t * g.heads * g.vdim] : 0.0f;
+        }
 #pragma unroll
         for (int t = 0; t < kC; t++) {
-            float r;
-            if (is_w) r = s_k[col * kP + t] * exp2f(s_G[col * kP + t]);
-            else r = t < ck.n && col < g.vdim ? a.v[(size_t)(ck.tok0 + t) * g.heads * g.vdim + h * g.vdim + col] : 0.0f;
             float p[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
-            for (int s = 0; s < t; s += 4) {  // entries on and above the diagonal are zero
+            for (int s = 0; s < t; s += 4) {
                 const float4 row = *(const float4*)(s_A + t * kC + s);
                 p[0] = fmaf(row.x, x[s], p[0]);
                 if (s + 1 < t) p[1] = fmaf(row.y, x[s + 1], p[1]);
                 if (s + 2 < t) p[2] = fmaf(row.z, x[s + 2], p[2]);
                 if (s + 3 < t) p[3] = fmaf(row.w, x[s + 3], p[3]);
             }
-            x[t] = s_b[t] * (r - ((p[0] + p[1]) + (p[2] + p[3])));
+            x[t] = s_b[t] * (x[t] - ((p[0] + p[1]) + (p[2] + p[3])));
         }
         if (is_w) {
 #pragma unroll
@@ -289,7 +316,7 @@ __global__ void __launch_bounds__(kCarryThreads) delta_carry_kernel(const DeltaA
 }
 
 int padded_dim(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : 128; }
-size_t chunk_smem(int dp) { return ((size_t)3 * dp * kP + 2 * kC * kC + kC) * sizeof(float); }
+size_t chunk_smem(int dp) { return ((size_t)3 * dp * kP + kC + (dp * kP >= kC * kC ? 0 : kC * kC)) * sizeof(float); }
 size_t carry_smem(int dp) { return ((size_t)2 * dp * 128 + kC * dp + kC * kC + 2 * kC * kCols + dp * kCols + dp) * sizeof(float); }
 
 }  // namespace

@@ -156,7 +156,7 @@ __device__ __forceinline__ float conv_at(const DeltaShape& g, const A* proj, con
     }
     return acc;
 }
-__device__ __forceinline__ float silu32(float v) { return v * sigmoid_f(v); }
+__device__ __forceinline__ float silu32(float v) { return __fdividef(v, 1.0f + __expf(-v)); }
 
 // One warp per (stretch of kPrepTok tokens, head unit): kv_heads units of q, kv_heads of k, heads of v; a lane owns every 32nd
 // channel and keeps its last inputs in registers while it walks the stretch (TAPS of them; 0: any number, re-read).
