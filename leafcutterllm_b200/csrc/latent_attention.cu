@@ -147,17 +147,18 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
+    // queries: the part carried through the key projection as it is, the other part rotated; both arrive with the first tile
+    for (int i = tid; i < ROWS * (g.cp / 8); i += 256) {
+        const int r = i / (g.cp / 8), c = i - r * (g.cp / 8);
+        cp16(q_sm + (uint32_t)(r * row_bytes + c * 16), (const bf16*)a.q_abs + ((size_t)t * g.heads + h0 + min(r, nh - 1)) * g.cp + c * 8, r < nh ? 16 : 0);
+    }
     load(kt0, 0);
-    for (int i = tid; i < 2 * kKeys * (pitch - d); i += 256) s_k[(i / (pitch - d)) * pitch + d + i % (pitch - d)] = __float2bfloat16_rn(0.0f);
-    for (int i = tid; i < ROWS * pitch; i += 256) {
-        const int r = i / pitch, c = i - r * pitch;
-        bf16 v = __float2bfloat16_rn(0.0f);
-        if (r < nh) {
-            const size_t th = (size_t)t * g.heads + h0 + r;
-            if (c < g.rank) v = ((const bf16*)a.q_abs)[th * g.cp + c];
-            else if (c >= g.cp && c < d) v = __float2bfloat16_rn(rotated((const bf16*)a.q + th * g.ld_q + g.dp, a.rot + (size_t)pos * g.rot_pairs, g.rot_pairs, g.rot, c - g.cp));
-        }
-        s_q[i] = v;
+    const bf16 zero = __float2bfloat16_rn(0.0f);
+    for (int i = tid; i < 2 * kKeys * (pitch - d); i += 256) s_k[(i / (pitch - d)) * pitch + d + i % (pitch - d)] = zero;
+    const float2* tab = a.rot + (size_t)pos * g.rot_pairs;
+    for (int i = tid; i < ROWS * (pitch - g.cp); i += 256) {
+        const int r = i / (pitch - g.cp), c = i - r * (pitch - g.cp);
+        s_q[r * pitch + g.cp + c] = r < nh && c < g.rp ? __float2bfloat16_rn(rotated((const bf16*)a.q + ((size_t)t * g.heads + h0 + r) * g.ld_q + g.dp, tab, g.rot_pairs, g.rot, c)) : zero;
     }
     if (tid < ROWS) { s_m[tid] = -INFINITY; s_l[tid] = 0.0f; }
     float o[MT][NCT][4];

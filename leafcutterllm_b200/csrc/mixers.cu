@@ -181,17 +181,24 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
 #pragma unroll
             for (int j = 0; j < TAPS; j++) w[c][j] = lane + 32 * c < n ? a.conv[(c0 + lane + 32 * c) * TAPS + j] : 0.0f;
     int prev_seq = -1, prev_pos = -1;
-    constexpr int kAhead = 4;
-    float ahead[kAhead][CPL];
-    int seq_a[kAhead], pos_a[kAhead];
+    const A* in = proj + col0 + lane;
+    bool ok[CPL];
+#pragma unroll
+    for (int c = 0; c < CPL; c++) ok[c] = lane + 32 * c < n;
+    float* o = (is_v ? a.v + (size_t)h * g.vdim : a.qk + (is_k ? g.kv_heads * g.dim : 0) + (size_t)h * g.dim) + lane;
+    const unsigned ld_o = is_v ? g.heads * g.vdim : 2 * g.kv_heads * g.dim, ld = g.ld;
+    const float q_scale = is_v || is_k ? 1.0f : 1.0f / sqrtf((float)g.dim);
+    constexpr int kAhead = TAPS > 0 ? 4 : 1;  // tokens whose inputs are fetched together
     for (int tb = t0; tb < t1; tb += kAhead) {
+        float ahead[kAhead][CPL];
+        int seq_a[kAhead], pos_a[kAhead];
 #pragma unroll
         for (int u = 0; u < kAhead; u++) {
-            const int t = min(tb + u, t1 - 1);
+            const unsigned t = min(tb + u, t1 - 1);
             seq_a[u] = a.tok_seq[t]; pos_a[u] = a.tok_pos[t];
             if constexpr (TAPS > 0)
 #pragma unroll
-                for (int c = 0; c < CPL; c++) ahead[u][c] = lane + 32 * c < n ? act_f<A>(proj[(size_t)t * g.ld + col0 + lane + 32 * c]) : 0.0f;
+                for (int c = 0; c < CPL; c++) ahead[u][c] = ok[c] ? act_f<A>(in[(size_t)(t * ld) + 32 * c]) : 0.0f;
         }
 #pragma unroll
         for (int u = 0; u < kAhead; u++) {
@@ -200,33 +207,30 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
             const int seq = seq_a[u], pos = pos_a[u];
             float y[CPL], ss = 0.0f;
             if constexpr (TAPS > 0) {
-                const bool follows = seq == prev_seq && pos == prev_pos + 1;
+                if (seq != prev_seq || pos != prev_pos + 1) {  // first token of the stretch or of a run: earlier inputs from the call's rows, the ring, or none
 #pragma unroll
-                for (int c = 0; c < CPL; c++) {
-                    const int i = lane + 32 * c;
-                    y[c] = 0.0f;
-                    if (i >= n) continue;
-                    if (!follows) {  // first token of the stretch or of a run: earlier inputs from the call's rows, the ring, or none
+                    for (int j = 1; j < TAPS; j++) {
+                        const int tt = t - j;
+                        const bool here = tt >= 0 && pos - j >= 0 && a.tok_seq[max(tt, 0)] == seq && a.tok_pos[max(tt, 0)] == pos - j;
 #pragma unroll
-                        for (int j = 1; j < TAPS; j++) {
-                            float v = 0.0f;
-                            if (pos - j >= 0) {
-                                const int tt = t - j;
-                                if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) v = act_f<A>(proj[(size_t)tt * g.ld + col0 + i]);
-                                else v = act_f<A>(ring[((size_t)seq * TAPS + (pos - j) % TAPS) * g.channels + c0 + i]);
-                            }
-                            win[c][j - 1] = v;
+                        for (int c = 0; c < CPL; c++) {
+                            win[c][j - 1] = 0.0f;
+                            if (!ok[c] || pos - j < 0) continue;
+                            win[c][j - 1] = here ? act_f<A>(in[(size_t)((unsigned)tt * ld) + 32 * c])
+                                                 : act_f<A>(ring[((size_t)seq * TAPS + (pos - j) % TAPS) * g.channels + c0 + lane + 32 * c]);
                         }
                     }
-                    const float cur = ahead[u][c];
+                }
+#pragma unroll
+                for (int c = 0; c < CPL; c++) {
                     float acc = 0.0f;
 #pragma unroll
                     for (int j = TAPS - 1; j > 0; j--) acc = fmaf(w[c][TAPS - 1 - j], win[c][j - 1], acc);
-                    acc = fmaf(w[c][TAPS - 1], cur, acc);
+                    acc = fmaf(w[c][TAPS - 1], ahead[u][c], acc);
 #pragma unroll
                     for (int j = TAPS - 1; j > 0; j--) win[c][j] = win[c][j - 1];
-                    win[c][0] = cur;
-                    y[c] = silu32(acc);
+                    win[c][0] = ahead[u][c];
+                    y[c] = silu32(acc);  // channels past n: zero weights, zero inputs
                     ss = fmaf(y[c], y[c], ss);
                 }
                 prev_seq = seq; prev_pos = pos;
@@ -234,22 +238,14 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
 #pragma unroll
                 for (int c = 0; c < CPL; c++) {
                     const int i = lane + 32 * c;
-                    y[c] = i < n ? silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, col0 + i)) : 0.0f;
+                    y[c] = ok[c] ? silu32(conv_at<A>(g, proj, ring, a.conv, a.tok_seq, a.tok_pos, t, seq, pos, c0 + i, col0 + i)) : 0.0f;
                     ss = fmaf(y[c], y[c], ss);
                 }
             }
-            float r = 1.0f;
-            float* o;
-            if (is_v) {
-                o = a.v + (size_t)t * g.heads * g.vdim + h * g.vdim;
-            } else {
-                o = a.qk + ((size_t)t * 2 + (is_k ? 1 : 0)) * g.kv_heads * g.dim + h * g.dim;
-                r = 1.0f / sqrtf(warp_sum(ss) + g.unit_eps);
-                if (!is_k) r *= 1.0f / sqrtf((float)g.dim);
-            }
+            const float r = is_v ? 1.0f : q_scale / sqrtf(warp_sum(ss) + g.unit_eps);
 #pragma unroll
             for (int c = 0; c < CPL; c++)
-                if (lane + 32 * c < n) o[lane + 32 * c] = y[c] * r;
+                if (ok[c]) o[(size_t)((unsigned)t * ld_o) + 32 * c] = y[c] * r;
         }
     }
 }
