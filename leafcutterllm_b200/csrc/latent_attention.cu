@@ -112,12 +112,12 @@ __device__ __forceinline__ float rotated(const bf16* r, const float2* tab, int p
 constexpr int kKeys = 64;  // keys per tile
 
 // Few tokens per sequence: the queries of 16 * MT heads of ONE token are the rows of the products, the cached rows (latent |
-// rotated part) the keys and, without the rotated part, the values.  Eight warps: for the scores each takes one row tile and
-// 8 * MT keys, for the weighted sum all rows and 8 * NCT latent columns.  The context is cut into gridDim.z pieces.
+// rotated part) the keys and, without the rotated part, the values.  8 * MT warps: for the scores each takes one row tile and
+// eight keys, for the weighted sum all rows and 8 * NCT latent columns.  The context is cut into gridDim.z pieces.
 struct LatentPieces { float *o, *ml; };  // [token][piece][heads][cp] sums, [token][piece][heads][2] maximum (log2 units) and weight sum
 template <int MT, int NCT>
-__global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, const LatentPieces pc) {
-    constexpr int KG = 8 / MT, ROWS = 16 * MT;
+__global__ void __launch_bounds__(256 * MT) latent_decode_kernel(const LatentArgs a, const LatentPieces pc) {
+    constexpr int KG = 8, ROWS = 16 * MT, THREADS = 256 * MT, WARPS = THREADS / 32;
     extern __shared__ __align__(128) unsigned char smem[];
     const LatentShape& g = a.g;
     const int d = g.cp + g.rp, d32 = (d + 31) & ~31, pitch = d32 + 8, row_bytes = pitch * 2;
@@ -131,7 +131,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     const int tiles = pos / kKeys + 1, per = (tiles + pieces - 1) / pieces, kt0 = blockIdx.z * per, kt1 = min(tiles, kt0 + per);
     const size_t out_row = ((size_t)t * pieces + blockIdx.z) * g.heads;
     if (kt0 >= kt1) {
-        for (int i = tid; i < nh; i += 256) { pc.ml[(out_row + h0 + i) * 2] = -INFINITY; pc.ml[(out_row + h0 + i) * 2 + 1] = 0.0f; }
+        for (int i = tid; i < nh; i += THREADS) { pc.ml[(out_row + h0 + i) * 2] = -INFINITY; pc.ml[(out_row + h0 + i) * 2 + 1] = 0.0f; }
         return;
     }
     const int32_t* pt = a.page_table + (size_t)seq * a.pages_per_seq;
@@ -139,7 +139,8 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
     const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), ph_sm = smem_u32(s_ph), pl_sm = smem_u32(s_pl);
     const int chunks = d / 8;
     auto load = [&](int kt, int buf) {
-        for (int key = warp; key < kKeys; key += 8) {
+        #pragma unroll
+        for (int key = warp; key < kKeys; key += WARPS) {
             const int kp = kt * kKeys + key;
             const bool ok = kp <= pos;
             const bf16* src = cache + ((size_t)(ok ? pt[kp / a.page_tokens] : 0) * a.page_tokens + kp % a.page_tokens) * d;
@@ -148,15 +149,15 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     // queries: the part carried through the key projection as it is, the other part rotated; both arrive with the first tile
-    for (int i = tid; i < ROWS * (g.cp / 8); i += 256) {
+    for (int i = tid; i < ROWS * (g.cp / 8); i += THREADS) {
         const int r = i / (g.cp / 8), c = i - r * (g.cp / 8);
         cp16(q_sm + (uint32_t)(r * row_bytes + c * 16), (const bf16*)a.q_abs + ((size_t)t * g.heads + h0 + min(r, nh - 1)) * g.cp + c * 8, r < nh ? 16 : 0);
     }
     load(kt0, 0);
     const bf16 zero = __float2bfloat16_rn(0.0f);
-    for (int i = tid; i < 2 * kKeys * (pitch - d); i += 256) s_k[(i / (pitch - d)) * pitch + d + i % (pitch - d)] = zero;
+    for (int i = tid; i < 2 * kKeys * (pitch - d); i += THREADS) s_k[(i / (pitch - d)) * pitch + d + i % (pitch - d)] = zero;
     const float2* tab = a.rot + (size_t)pos * g.rot_pairs;
-    for (int i = tid; i < ROWS * (pitch - g.cp); i += 256) {
+    for (int i = tid; i < ROWS * (pitch - g.cp); i += THREADS) {
         const int r = i / (pitch - g.cp), c = i - r * (pitch - g.cp);
         s_q[r * pitch + g.cp + c] = r < nh && c < g.rp ? __float2bfloat16_rn(rotated((const bf16*)a.q + ((size_t)t * g.heads + h0 + r) * g.ld_q + g.dp, tab, g.rot_pairs, g.rot, c)) : zero;
     }
@@ -175,33 +176,26 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
         else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         const uint32_t kb = k_sm + (uint32_t)(buf * kKeys * row_bytes);
-        // scores of rows row0 .. + 15 with keys kg * 8 MT ..
-        float s[MT][4];
-#pragma unroll
-        for (int i = 0; i < MT; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+        // scores of rows row0 .. + 15 with keys 8 kg .. + 7, two sums that take turns
+        float s[4] = {0.0f, 0.0f, 0.0f, 0.0f}, s2[4] = {0.0f, 0.0f, 0.0f, 0.0f};
         const uint32_t qa = q_sm + (uint32_t)((row0 + (lane & 15)) * row_bytes + (lane >> 4) * 16);
-        const uint32_t ka = kb + (uint32_t)((kg * 8 * MT + (lane & 7)) * row_bytes + (lane >> 3) * 16);
+        const uint32_t ka = kb + (uint32_t)((kg * 8 + (lane & 7)) * row_bytes + (lane >> 3) * 16);
+#pragma unroll 3
         for (int k = 0; k < d32; k += 32) {
-            uint32_t a0[4], a1[4];
+            uint32_t a0[4], a1[4], b[4];
             ldsm4(qa + k * 2, a0);
             ldsm4(qa + k * 2 + 32, a1);
-#pragma unroll
-            for (int i = 0; i < MT; i++) {
-                uint32_t b[4];
-                ldsm4(ka + (uint32_t)(8 * i * row_bytes + k * 2), b);
-                mma_bf16(s[i], a0, b[0], b[1]);
-                mma_bf16(s[i], a1, b[2], b[3]);
-            }
+            ldsm4(ka + k * 2, b);
+            mma_bf16(s, a0, b[0], b[1]);
+            mma_bf16(s2, a1, b[2], b[3]);
         }
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-        for (int i = 0; i < MT; i++)
-#pragma unroll
-            for (int j = 0; j < 4; j++) {
-                const int key = kt * kKeys + kg * 8 * MT + 8 * i + 2 * t4 + (j & 1);
-                s[i][j] = key <= pos ? s[i][j] * sc : -INFINITY;
-                mx[j >> 1] = fmaxf(mx[j >> 1], s[i][j]);
-            }
+        for (int j = 0; j < 4; j++) {
+            const int key = kt * kKeys + kg * 8 + 2 * t4 + (j & 1);
+            s[j] = key <= pos ? (s[j] + s2[j]) * sc : -INFINITY;
+            mx[j >> 1] = fmaxf(mx[j >> 1], s[j]);
+        }
 #pragma unroll
         for (int r = 0; r < 2; r++) {
             mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
@@ -221,16 +215,13 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const LatentArgs a, 
             const int row = row0 + g8 + 8 * r;
             const float m = new_max(row);
             if (kg == 0 && t4 == 0) s_m[(par ^ 1) * ROWS + row] = m;
-#pragma unroll
-            for (int i = 0; i < MT; i++) {
-                const float p0 = exp2f(s[i][2 * r] - m), p1 = exp2f(s[i][2 * r + 1] - m);
-                sum[r] += p0 + p1;
-                uint32_t hi, lo;
-                split2(p0, p1, hi, lo);
-                const int at = row * (kKeys + 8) + kg * 8 * MT + 8 * i + 2 * t4;
-                *(uint32_t*)(s_ph + at) = hi;
-                *(uint32_t*)(s_pl + at) = lo;
-            }
+            const float p0 = exp2f(s[2 * r] - m), p1 = exp2f(s[2 * r + 1] - m);
+            sum[r] = p0 + p1;
+            uint32_t hi, lo;
+            split2(p0, p1, hi, lo);
+            const int at = row * (kKeys + 8) + kg * 8 + 2 * t4;
+            *(uint32_t*)(s_ph + at) = hi;
+            *(uint32_t*)(s_pl + at) = lo;
             sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 1);
             sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 2);
             if (t4 == 0) s_wsum[row * KG + kg] = sum[r];
@@ -498,7 +489,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentArgs a,
 
 size_t decode_smem(const LatentShape& g, int mt) {
     const size_t pitch = ((g.cp + g.rp + 31) & ~31) + 8, rows = 16 * (size_t)mt;
-    return (rows + 2 * kKeys) * pitch * 2 + 2 * rows * (kKeys + 8) * 2 + (2 * rows * (8 / mt) + 3 * rows) * 4;
+    return (rows + 2 * kKeys) * pitch * 2 + 2 * rows * (kKeys + 8) * 2 + (2 * rows * 8 + 3 * rows) * 4;
 }
 size_t prefill_smem(const LatentShape& g, int nv) {
     const size_t pitch = ((g.dp + g.rp + 31) & ~31) + 8;
@@ -523,8 +514,8 @@ int32_t launch_plain(const LatentArgs& a, cudaStream_t s) {
 }  // namespace
 
 size_t latent_pieces_bytes(const LatentShape& g, int tokens) {
-    // pieces * tokens * row blocks stays near twice the SM count, so the scratch is bounded by that many row blocks
-    const size_t blocks = std::max<size_t>((size_t)4 * sm_count(), (size_t)tokens * ((g.heads + 15) / 16));
+    // pieces * tokens * row blocks stays within the SM count, so the scratch is bounded by that many row blocks
+    const size_t blocks = std::max<size_t>((size_t)sm_count(), (size_t)tokens * ((g.heads + 15) / 16));
     return blocks * 32 * ((size_t)g.cp + 2) * sizeof(float) * 2;
 }
 
@@ -535,7 +526,7 @@ int32_t launch_latent_attention(const LatentArgs& a, void* scratch, size_t scrat
     if (a.T <= 0) return LC_OK;
     if (a.f32 || g.cp > 512 || decode_smem(g, mt) > kMaxSmem) return launch_plain(a, s);
     const int blocks = (g.heads + 16 * mt - 1) / (16 * mt);
-    int pieces = std::max(1, std::min(kMaxPieces, 2 * sm_count() / (a.T * blocks)));
+    int pieces = std::max(1, std::min(kMaxPieces, sm_count() / (a.T * blocks)));
     pieces = std::min(pieces, (a.pages_per_seq * a.page_tokens + kKeys - 1) / kKeys);
     auto need = [&](int n) { return (size_t)a.T * n * g.heads * ((size_t)g.cp + 2) * sizeof(float); };
     while (pieces > 1 && need(pieces) > scratch_bytes) pieces--;
@@ -546,12 +537,12 @@ int32_t launch_latent_attention(const LatentArgs& a, void* scratch, size_t scrat
     const dim3 grid((unsigned)a.T, (unsigned)blocks, (unsigned)pieces);
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(ensure_smem_limit((const void*)kern, smem));
-        LC_CUDA(launch_pdl(kern, grid, dim3(256), smem, s, a, pc));
+        LC_CUDA(launch_pdl(kern, grid, dim3((unsigned)(256 * mt)), smem, s, a, pc));
         return LC_OK;
     };
-    const int nct = g.cp <= 128 ? 2 : g.cp <= 256 ? 4 : 8;
+    const int nct = g.cp <= 128 * mt ? 2 : g.cp <= 256 * mt ? 4 : 8;  // latent columns of a warp, in eights
     if (mt == 1) LC_TRY(nct == 2 ? go(latent_decode_kernel<1, 2>) : nct == 4 ? go(latent_decode_kernel<1, 4>) : go(latent_decode_kernel<1, 8>));
-    else LC_TRY(nct == 2 ? go(latent_decode_kernel<2, 2>) : nct == 4 ? go(latent_decode_kernel<2, 4>) : go(latent_decode_kernel<2, 8>));
+    else LC_TRY(nct == 2 ? go(latent_decode_kernel<2, 2>) : go(latent_decode_kernel<2, 4>));
     if (pieces > 1) {
         LC_CUDA(launch_pdl(latent_merge_kernel, dim3((unsigned)g.heads, (unsigned)a.T), dim3(128), 0, s, pc, pieces, g.heads, g.cp, (bf16*)a.o));
         *launches = 2;
