@@ -45,7 +45,8 @@ pub struct LcModelConfig {
     pub device: i32,
     pub tp_size: i32,
     pub tp_rank: i32,
-    pub reserved: [i32; 5],
+    pub compute_f32: i32,
+    pub reserved: [i32; 4],
 }
 
 #[repr(C)]

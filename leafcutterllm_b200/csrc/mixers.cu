@@ -352,15 +352,15 @@ __global__ void __launch_bounds__(256) delta_output_kernel(const DeltaArgs a) {
 // With G = diag(g):  dot = (G S)^T k,  u = beta (v - dot),  S' = G S + k u^T,  o = S'^T q = (G S)^T q + u (k . q), so the state
 // is walked once; a thread owns VEC neighbouring value columns and every `groups`-th key row, kept in registers (ROWS of
 // them; 0: re-read for the update).  The ring entry written here is not one that any head reads in this step.
-template <typename A, int VEC, int ROWS>
-__global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
+template <typename A, int VEC, int ROWS, int THREADS>
+__global__ void __launch_bounds__(THREADS) delta_step_kernel(const DeltaArgs a) {
     extern __shared__ float sm[];
     __shared__ float red[32], s_norm[3];
     pdl_launch_dependents();
     pdl_wait();
     const DeltaShape& g = a.g;
     const int h = blockIdx.x, t = blockIdx.y, rep = g.heads / g.kv_heads, kh = h / rep, seq = a.tok_seq[t], pos = a.tok_pos[t];
-    const int cols = g.vdim / VEC, groups = 256 / cols;
+    const int cols = g.vdim / VEC, groups = THREADS / cols;
     float *s_q = sm, *s_k = s_q + g.dim, *s_g = s_k + g.dim, *s_v = s_g + g.dim, *s_dk = s_v + g.vdim, *s_dq = s_dk + groups * g.vdim;
     const A* proj = (const A*)a.proj + (size_t)t * g.ld;
     A* ring = (A*)a.ring + (size_t)seq * g.taps * g.channels;
@@ -380,8 +380,20 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
             }
         }
     }
+    // what the later phases need travels with the state
+    constexpr int kHold = 2;
+    const A* gate = (const A*)a.gate + ((size_t)t * g.heads + h) * g.vdim;
+    float gate_r[kHold], norm_r[kHold], decay_r[kHold];
+#pragma unroll
+    for (int i = 0; i < kHold; i++) {
+        const int e = threadIdx.x + i * THREADS;
+        gate_r[i] = e < g.vdim ? act_f<A>(gate[e]) : 0.0f;
+        norm_r[i] = e < g.vdim ? a.norm_w[e] : 0.0f;
+        decay_r[i] = e < g.dim ? a.log_decay[(size_t)t * g.heads * g.dim + h * g.dim + e] : 0.0f;
+    }
+    const float beta_in = act_f<A>(proj[g.off_b + h]);
     const int now = pos % g.taps;
-    for (int i = threadIdx.x; i < 2 * g.dim + g.vdim; i += 256) {
+    for (int i = threadIdx.x; i < 2 * g.dim + g.vdim; i += THREADS) {
         int column, channel;
         bool owner = true;
         float* dst;
@@ -406,7 +418,9 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
         *dst = silu32(acc);
         if (owner) ring[(size_t)now * g.channels + channel] = cur;
     }
-    for (int d = threadIdx.x; d < g.dim; d += 256) s_g[d] = expf(a.log_decay[(size_t)t * g.heads * g.dim + h * g.dim + d]);
+#pragma unroll
+    for (int i = 0; i < kHold; i++)
+        if (threadIdx.x + i * THREADS < g.dim) s_g[threadIdx.x + i * THREADS] = expf(decay_r[i]);
     __syncthreads();
     if (threadIdx.x < 96) {  // |q|^2, |k|^2, q . k
         const int w = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -418,7 +432,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
     }
     __syncthreads();
     const float rq = 1.0f / sqrtf(s_norm[0] + g.unit_eps) * (1.0f / sqrtf((float)g.dim)), rk = 1.0f / sqrtf(s_norm[1] + g.unit_eps), qk = s_norm[2] * rq * rk;
-    const float beta = sigmoid_f(act_f<A>(proj[g.off_b + h]));
+    const float beta = sigmoid_f(beta_in);
     float dk[VEC], dq[VEC];
 #pragma unroll
     for (int j = 0; j < VEC; j++) dk[j] = dq[j] = 0.0f;
@@ -451,7 +465,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
     }
     __syncthreads();
     float ss = 0.0f;
-    for (int e = threadIdx.x; e < g.vdim; e += 256) {  // u replaces v, the read-out replaces the first partial row
+    for (int e = threadIdx.x; e < g.vdim; e += THREADS) {  // u replaces v, the read-out replaces the first partial row
         float sk = 0.0f, sq = 0.0f;
         for (int i = 0; i < groups; i++) { sk += s_dk[i * g.vdim + e]; sq += s_dq[i * g.vdim + e]; }
         const float u = beta * (s_v[e] - sk), o = fmaf(u, qk, sq);
@@ -486,9 +500,12 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaArgs a) {
         }
     }
     const float r = 1.0f / sqrtf(ss / (float)g.vdim + g.eps);
-    const A* gate = (const A*)a.gate + ((size_t)t * g.heads + h) * g.vdim;
     A* dst = (A*)a.out + (size_t)t * a.ldo + h * g.vdim;
-    for (int e = threadIdx.x; e < g.vdim; e += 256) dst[e] = to_act<A>(s_dq[e] * r * a.norm_w[e] * sigmoid_f(act_f<A>(gate[e])));
+#pragma unroll
+    for (int i = 0; i < kHold; i++) {
+        const int e = threadIdx.x + i * THREADS;
+        if (e < g.vdim) dst[e] = to_act<A>(s_dq[e] * r * norm_r[i] * sigmoid_f(gate_r[i]));
+    }
 }
 
 // ---- latent attention: norms of the two latents, rotation of the shared key part, cache append -------------------------------
@@ -576,18 +593,19 @@ int32_t scan_dispatch(const DeltaArgs& a, cudaStream_t s) {
 
 template <typename A>
 int32_t step_dispatch(const DeltaArgs& a, cudaStream_t s) {
-    const int vec = a.g.vdim % 4 == 0 ? 4 : 1, cols = a.g.vdim / vec;
-    LC_CHECK(cols <= 256, LC_ERR_UNSUPPORTED, "delta rule: %d value dimensions per head", a.g.vdim);
-    const int groups = 256 / cols, rows = (a.g.dim + groups - 1) / groups;
+    const int vec = a.g.vdim % 4 == 0 ? 4 : 1, cols = a.g.vdim / vec, threads = vec == 4 && a.g.dim * a.g.vdim >= 8192 ? 512 : 256;
+    LC_CHECK(cols <= threads && a.g.vdim <= 512, LC_ERR_UNSUPPORTED, "delta rule: %d value dimensions per head", a.g.vdim);
+    const int groups = threads / cols, rows = (a.g.dim + groups - 1) / groups;
     const size_t smem = (size_t)(3 * a.g.dim + a.g.vdim + 2 * groups * a.g.vdim) * sizeof(float);
     const dim3 grid((unsigned)a.g.heads, (unsigned)a.T);
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(ensure_smem_limit((const void*)kern, smem));
-        LC_CUDA(launch_pdl(kern, grid, dim3(256), smem, s, a));
+        LC_CUDA(launch_pdl(kern, grid, dim3((unsigned)threads), smem, s, a));
         return LC_OK;
     };
-    if (vec == 4) return rows <= 4 ? go(delta_step_kernel<A, 4, 4>) : rows <= 16 ? go(delta_step_kernel<A, 4, 16>) : go(delta_step_kernel<A, 4, 0>);
-    return rows <= 16 ? go(delta_step_kernel<A, 1, 16>) : go(delta_step_kernel<A, 1, 0>);
+    if (threads == 512) return rows <= 4 ? go(delta_step_kernel<A, 4, 4, 512>) : rows <= 8 ? go(delta_step_kernel<A, 4, 8, 512>) : go(delta_step_kernel<A, 4, 0, 512>);
+    if (vec == 4) return rows <= 4 ? go(delta_step_kernel<A, 4, 4, 256>) : rows <= 16 ? go(delta_step_kernel<A, 4, 16, 256>) : go(delta_step_kernel<A, 4, 0, 256>);
+    return rows <= 16 ? go(delta_step_kernel<A, 1, 16, 256>) : go(delta_step_kernel<A, 1, 0, 256>);
 }
 
 }  // namespace

@@ -102,3 +102,14 @@ def test_bf16_tensors_from_the_generator(lc):
     f = synth.host_tensor(lc.TYPE_F32, 7, "t", 4096).view(np.float32)
     b = synth.host_tensor(lc.TYPE_BF16, 7, "t", 4096).view(np.uint16)
     assert np.array_equal(b, U.bf16_bytes(f))
+
+
+def test_command_line_inspects_a_checkpoint_directory(lc, tmp_path, capsys):
+    from leafcutterllm_b200.__main__ import main
+    cfg = mixed_config()
+    U.write_checkpoint(tmp_path, cfg, U.weights(cfg))
+    assert main(["inspect", "--model", str(tmp_path)]) == 0
+    import json
+    assert json.loads(capsys.readouterr().out) == {"architecture": "Varasun", "width": 104, "vocab": 131, "layers": {"channel_delta": 2, "latent_attention": 2}}
+    assert main(["generate", "--model", str(tmp_path / "nothing"), "--tokens", "1,2"]) == 1
+    assert "error" in capsys.readouterr().err

@@ -248,6 +248,14 @@ def test_checkpoint_directory_and_trace_runner(gpu, model, tmp_path, monkeypatch
     want = m.forward(toks, m.new_state())
     U.check(eng.forward(toks)[None], want[-1:], dtype)
     eng.close()
+    from leafcutterllm_b200.__main__ import main
+    st, picks = m.new_state(), []
+    line = m.forward(toks, st)[-1]
+    for _ in range(4):
+        picks.append(int(line.argmax()))
+        line = m.forward(picks[-1:], st)[-1]
+    assert main(["generate", "--model", str(tmp_path), "--tokens", ",".join(map(str, toks)), "--max-tokens", "4", "--dtype", "float32", "--keep-going"]) == 0
+    assert [int(t) for t in capsys.readouterr().out.split()] == picks
     steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:20], "want": [19, 3]}, {"id": "y", "tokens": toks[:1], "want": []}], "end": []},
              {"step": 1, "entries": [{"id": "y", "tokens": toks[1:3], "want": []}], "end": ["y"]},
              {"step": 2, "entries": [{"id": "z", "tokens": toks, "want": [32]}, {"id": "x", "tokens": toks[20:21], "want": [0]}], "end": ["x", "z"]}]
