@@ -110,19 +110,21 @@ __device__ __forceinline__ float rotated(const bf16* r, const float2* tab, int p
     return (i & 1) ? w * cs.x + u * cs.y : u * cs.x - w * cs.y;
 }
 constexpr int kKeys = 64;  // keys per tile
+constexpr int kPartPitch = kKeys + 4;
 
 // Few tokens per sequence: the queries of 16 * MT heads of ONE token are the rows of the products, the cached rows (latent |
-// rotated part) the keys and, without the rotated part, the values.  8 * MT warps: for the scores each takes one row tile and
-// eight keys, for the weighted sum all rows and 8 * NCT latent columns.  The context is cut into gridDim.z pieces.
+// rotated part) the keys and, without the rotated part, the values.  8 * MT warps: for the scores each takes all rows,
+// sixteen keys and 1 / (2 MT) of the row's elements (partial scores meet in shared memory); for the softmax sixteen threads
+// share a row; for the weighted sum a warp takes all rows and 8 * NCT latent columns.  The context is cut into gridDim.z pieces.
 struct LatentPieces { float *o, *ml; };  // [token][piece][heads][cp] sums, [token][piece][heads][2] maximum (log2 units) and weight sum
 template <int MT, int NCT>
 __global__ void __launch_bounds__(256 * MT) latent_decode_kernel(const LatentArgs a, const LatentPieces pc) {
-    constexpr int KG = 8, ROWS = 16 * MT, THREADS = 256 * MT, WARPS = THREADS / 32;
+    constexpr int KQ = 2 * MT, ROWS = 16 * MT, THREADS = 256 * MT, WARPS = THREADS / 32;
     extern __shared__ __align__(128) unsigned char smem[];
     const LatentShape& g = a.g;
     const int d = g.cp + g.rp, d32 = (d + 31) & ~31, pitch = d32 + 8, row_bytes = pitch * 2;
     bf16 *s_q = (bf16*)smem, *s_k = s_q + ROWS * pitch, *s_ph = s_k + 2 * kKeys * pitch, *s_pl = s_ph + ROWS * (kKeys + 8);
-    float *s_wmax = (float*)(s_pl + ROWS * (kKeys + 8)), *s_wsum = s_wmax + ROWS * KG, *s_m = s_wsum + ROWS * KG, *s_l = s_m + 2 * ROWS;
+    float *s_part = (float*)(s_pl + ROWS * (kKeys + 8)), *s_corr = s_part + KQ * ROWS * kPartPitch;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
     const int t = blockIdx.x, h0 = blockIdx.y * ROWS, nh = min(ROWS, g.heads - h0);
     pdl_launch_dependents();
@@ -139,12 +141,15 @@ __global__ void __launch_bounds__(256 * MT) latent_decode_kernel(const LatentArg
     const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), ph_sm = smem_u32(s_ph), pl_sm = smem_u32(s_pl);
     const int chunks = d / 8;
     auto load = [&](int kt, int buf) {
-        #pragma unroll
-        for (int key = warp; key < kKeys; key += WARPS) {
-            const int kp = kt * kKeys + key;
-            const bool ok = kp <= pos;
-            const bf16* src = cache + ((size_t)(ok ? pt[kp / a.page_tokens] : 0) * a.page_tokens + kp % a.page_tokens) * d;
-            for (int c = lane; c < chunks; c += 32) cp16(k_sm + (uint32_t)((buf * kKeys + key) * row_bytes + c * 16), ok ? src + c * 8 : cache, ok ? 16 : 0);
+        // lane j finds the cached row of the warp's j-th key
+        const int kp = kt * kKeys + warp + (lane % (kKeys / WARPS)) * WARPS;
+        const int row = kp <= pos ? pt[kp / a.page_tokens] * a.page_tokens + kp % a.page_tokens : -1;
+#pragma unroll
+        for (int j = 0; j < kKeys / WARPS; j++) {
+            const int rj = __shfl_sync(0xffffffffu, row, j);
+            const bf16* src = cache + (size_t)max(rj, 0) * d;
+            const uint32_t dst = k_sm + (uint32_t)((buf * kKeys + warp + j * WARPS) * row_bytes);
+            for (int c = lane; c < chunks; c += 32) cp16(dst + c * 16, src + c * 8, rj >= 0 ? 16 : 0);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -161,85 +166,85 @@ __global__ void __launch_bounds__(256 * MT) latent_decode_kernel(const LatentArg
         const int r = i / (pitch - g.cp), c = i - r * (pitch - g.cp);
         s_q[r * pitch + g.cp + c] = r < nh && c < g.rp ? __float2bfloat16_rn(rotated((const bf16*)a.q + ((size_t)t * g.heads + h0 + r) * g.ld_q + g.dp, tab, g.rot_pairs, g.rot, c)) : zero;
     }
-    if (tid < ROWS) { s_m[tid] = -INFINITY; s_l[tid] = 0.0f; }
     float o[MT][NCT][4];
 #pragma unroll
     for (int i = 0; i < MT; i++)
 #pragma unroll
         for (int j = 0; j < NCT; j++) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.0f;
     const float sc = g.scale * 1.4426950408889634f;
-    const int mt = warp % MT, kg = warp / MT, row0 = mt * 16;
-    int par = 0;
-    for (int kt = kt0; kt < kt1; kt++, par ^= 1) {
+    const int kg = warp & 3, kq = warp >> 2, steps = d32 / 16, st0 = steps * kq / KQ, st1 = steps * (kq + 1) / KQ;
+    const int srow = tid >> 4, skey = (tid & 15) * 4;  // the softmax's row and its first key of this thread
+    float m_run = -INFINITY, l_run = 0.0f;
+    for (int kt = kt0; kt < kt1; kt++) {
         const int buf = (kt - kt0) & 1;
         if (kt + 1 < kt1) { load(kt + 1, buf ^ 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
         else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         const uint32_t kb = k_sm + (uint32_t)(buf * kKeys * row_bytes);
-        // scores of rows row0 .. + 15 with keys 8 kg .. + 7, two sums that take turns
-        float s[4] = {0.0f, 0.0f, 0.0f, 0.0f}, s2[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-        const uint32_t qa = q_sm + (uint32_t)((row0 + (lane & 15)) * row_bytes + (lane >> 4) * 16);
-        const uint32_t ka = kb + (uint32_t)((kg * 8 + (lane & 7)) * row_bytes + (lane >> 3) * 16);
+        float s[MT][2][4];
+#pragma unroll
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int j = 0; j < 2; j++) s[i][j][0] = s[i][j][1] = s[i][j][2] = s[i][j][3] = 0.0f;
+        const uint32_t qa = q_sm + (uint32_t)((lane & 15) * row_bytes + (lane >> 4) * 16);
+        const uint32_t ka = kb + (uint32_t)((kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * row_bytes + ((lane >> 3) & 1) * 16);
 #pragma unroll 3
-        for (int k = 0; k < d32; k += 32) {
-            uint32_t a0[4], a1[4], b[4];
-            ldsm4(qa + k * 2, a0);
-            ldsm4(qa + k * 2 + 32, a1);
-            ldsm4(ka + k * 2, b);
-            mma_bf16(s, a0, b[0], b[1]);
-            mma_bf16(s2, a1, b[2], b[3]);
-        }
-        float mx[2] = {-INFINITY, -INFINITY};
+        for (int st = st0; st < st1; st++) {
+            uint32_t b[4];
+            ldsm4(ka + st * 32, b);
 #pragma unroll
-        for (int j = 0; j < 4; j++) {
-            const int key = kt * kKeys + kg * 8 + 2 * t4 + (j & 1);
-            s[j] = key <= pos ? (s[j] + s2[j]) * sc : -INFINITY;
-            mx[j >> 1] = fmaxf(mx[j >> 1], s[j]);
+            for (int i = 0; i < MT; i++) {
+                uint32_t aq[4];
+                ldsm4(qa + (uint32_t)(16 * i * row_bytes) + st * 32, aq);
+                mma_bf16(s[i][0], aq, b[0], b[1]);
+                mma_bf16(s[i][1], aq, b[2], b[3]);
+            }
         }
 #pragma unroll
-        for (int r = 0; r < 2; r++) {
-            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-            if (t4 == 0) s_wmax[(row0 + g8 + 8 * r) * KG + kg] = mx[r];
+        for (int i = 0; i < MT; i++)
+#pragma unroll
+            for (int j = 0; j < 2; j++)
+#pragma unroll
+                for (int r = 0; r < 2; r++)
+                    *(float2*)(s_part + (kq * ROWS + 16 * i + g8 + 8 * r) * kPartPitch + kg * 16 + 8 * j + 2 * t4) = make_float2(s[i][j][2 * r], s[i][j][2 * r + 1]);
+        __syncthreads();
+        {
+            float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+            for (int q = 0; q < KQ; q++) {
+                const float4 x = *(const float4*)(s_part + (q * ROWS + srow) * kPartPitch + skey);
+                v[0] += x.x; v[1] += x.y; v[2] += x.z; v[3] += x.w;
+            }
+            float mx = m_run;
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                v[j] = kt * kKeys + skey + j <= pos ? v[j] * sc : -INFINITY;
+                mx = fmaxf(mx, v[j]);
+            }
+#pragma unroll
+            for (int w = 1; w < 16; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
+            const float corr = exp2f(m_run - mx);  // mx is finite: a tile starts at or before the token's position
+            m_run = mx;
+            float sum = 0.0f;
+#pragma unroll
+            for (int j = 0; j < 4; j++) { v[j] = exp2f(v[j] - mx); sum += v[j]; }
+#pragma unroll
+            for (int w = 1; w < 16; w <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, w);
+            l_run = l_run * corr + sum;
+            if ((tid & 15) == 0) s_corr[srow] = corr;
+            uint32_t h0, l0, h1, l1;
+            split2(v[0], v[1], h0, l0);
+            split2(v[2], v[3], h1, l1);
+            *(uint2*)(s_ph + srow * (kKeys + 8) + skey) = make_uint2(h0, h1);
+            *(uint2*)(s_pl + srow * (kKeys + 8) + skey) = make_uint2(l0, l1);
         }
         __syncthreads();
-        auto new_max = [&](int row) {
-            float v = s_m[par * ROWS + row];
-#pragma unroll
-            for (int i = 0; i < KG; i++) v = fmaxf(v, s_wmax[row * KG + i]);
-            return v;
-        };
-        float sum[2] = {0.0f, 0.0f};
-#pragma unroll
-        for (int r = 0; r < 2; r++) {
-            const int row = row0 + g8 + 8 * r;
-            const float m = new_max(row);
-            if (kg == 0 && t4 == 0) s_m[(par ^ 1) * ROWS + row] = m;
-            const float p0 = exp2f(s[2 * r] - m), p1 = exp2f(s[2 * r + 1] - m);
-            sum[r] = p0 + p1;
-            uint32_t hi, lo;
-            split2(p0, p1, hi, lo);
-            const int at = row * (kKeys + 8) + kg * 8 + 2 * t4;
-            *(uint32_t*)(s_ph + at) = hi;
-            *(uint32_t*)(s_pl + at) = lo;
-            sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 1);
-            sum[r] += __shfl_xor_sync(0xffffffffu, sum[r], 2);
-            if (t4 == 0) s_wsum[row * KG + kg] = sum[r];
-        }
-        __syncthreads();
-        if (tid < ROWS) {
-            float l = s_l[tid] * exp2f(s_m[par * ROWS + tid] - s_m[(par ^ 1) * ROWS + tid]);
-#pragma unroll
-            for (int i = 0; i < KG; i++) l += s_wsum[tid * KG + i];
-            s_l[tid] = l;
-        }
         // weighted sum of this warp's latent columns
         const int c0 = warp * NCT * 8;
         if (c0 < g.cp) {
 #pragma unroll
             for (int i = 0; i < MT; i++) {
-                const float f0 = exp2f(s_m[par * ROWS + 16 * i + g8] - s_m[(par ^ 1) * ROWS + 16 * i + g8]);
-                const float f1 = exp2f(s_m[par * ROWS + 16 * i + g8 + 8] - s_m[(par ^ 1) * ROWS + 16 * i + g8 + 8]);
+                const float f0 = s_corr[16 * i + g8], f1 = s_corr[16 * i + g8 + 8];
 #pragma unroll
                 for (int j = 0; j < NCT; j++) { o[i][j][0] *= f0; o[i][j][1] *= f0; o[i][j][2] *= f1; o[i][j][3] *= f1; }
             }
@@ -269,13 +274,19 @@ __global__ void __launch_bounds__(256 * MT) latent_decode_kernel(const LatentArg
         }
         __syncthreads();
     }
+    // the rows' weight sums, where the loop's corrections were (every warp is past them)
+    if ((tid & 15) == 0) {
+        s_corr[srow] = l_run;
+        if (pieces > 1 && srow < nh) { pc.ml[(out_row + h0 + srow) * 2] = m_run; pc.ml[(out_row + h0 + srow) * 2 + 1] = l_run; }
+    }
+    __syncthreads();
 #pragma unroll
     for (int i = 0; i < MT; i++)
 #pragma unroll
         for (int r = 0; r < 2; r++) {
             const int row = 16 * i + g8 + 8 * r;
             if (row >= nh) continue;
-            const float inv = 1.0f / s_l[row];
+            const float inv = 1.0f / s_corr[row];
 #pragma unroll
             for (int j = 0; j < NCT; j++) {
                 const int c = (warp * NCT + j) * 8 + 2 * t4;
@@ -284,10 +295,6 @@ __global__ void __launch_bounds__(256 * MT) latent_decode_kernel(const LatentArg
                 else *(float2*)(pc.o + (out_row + h0 + row) * g.cp + c) = make_float2(o[i][j][2 * r], o[i][j][2 * r + 1]);
             }
         }
-    if (pieces > 1 && tid < nh) {
-        pc.ml[(out_row + h0 + tid) * 2] = s_m[par * ROWS + tid];
-        pc.ml[(out_row + h0 + tid) * 2 + 1] = s_l[tid];
-    }
 }
 
 constexpr int kMaxPieces = 64;
@@ -489,7 +496,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentArgs a,
 
 size_t decode_smem(const LatentShape& g, int mt) {
     const size_t pitch = ((g.cp + g.rp + 31) & ~31) + 8, rows = 16 * (size_t)mt;
-    return (rows + 2 * kKeys) * pitch * 2 + 2 * rows * (kKeys + 8) * 2 + (2 * rows * 8 + 3 * rows) * 4;
+    return (rows + 2 * kKeys) * pitch * 2 + 2 * rows * (kKeys + 8) * 2 + ((size_t)2 * mt * rows * kPartPitch + rows) * 4;
 }
 size_t prefill_smem(const LatentShape& g, int nv) {
     const size_t pitch = ((g.dp + g.rp + 31) & ~31) + 8;
