@@ -140,13 +140,17 @@ __global__ void __launch_bounds__(256 * MT) latent_decode_kernel(const LatentArg
     const bf16* cache = (const bf16*)a.cache;
     const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), ph_sm = smem_u32(s_ph), pl_sm = smem_u32(s_pl);
     const int chunks = d / 8;
-    auto load = [&](int kt, int buf) {
-        // lane j finds the cached row of the warp's j-th key
+    auto row_of = [&](int kt) {  // lane j finds the cached row of the warp's j-th key
         const int kp = kt * kKeys + warp + (lane % (kKeys / WARPS)) * WARPS;
-        const int row = kp <= pos ? pt[kp / a.page_tokens] * a.page_tokens + kp % a.page_tokens : -1;
+        return kp <= pos ? pt[kp / a.page_tokens] * a.page_tokens + kp % a.page_tokens : -1;
+    };
+    int rows_next = row_of(kt0);  // of the tile that is loaded next: looked up one tile ahead
+    auto load = [&](int kt, int buf) {
+        const int rows = rows_next;
+        rows_next = row_of(kt + 1);
 #pragma unroll
         for (int j = 0; j < kKeys / WARPS; j++) {
-            const int rj = __shfl_sync(0xffffffffu, row, j);
+            const int rj = __shfl_sync(0xffffffffu, rows, j);
             const bf16* src = cache + (size_t)max(rj, 0) * d;
             const uint32_t dst = k_sm + (uint32_t)((buf * kKeys + warp + j * WARPS) * row_bytes);
             for (int c = lane; c < chunks; c += 32) cp16(dst + c * 16, src + c * 8, rj >= 0 ? 16 : 0);

@@ -162,7 +162,7 @@ __device__ __forceinline__ float silu32(float v) { return __fdividef(v, 1.0f + _
 // channel and keeps its last inputs in registers while it walks the stretch (TAPS of them; 0: any number, re-read).
 constexpr int kPrepTok = 16;
 template <typename A, int TAPS, int CPL>
-__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaArgs a) {
+__global__ void __launch_bounds__(256, CPL > 4 ? 2 : 3) delta_prep_kernel(const DeltaArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const DeltaShape& g = a.g;
