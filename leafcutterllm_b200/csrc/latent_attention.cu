@@ -322,16 +322,16 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(LatentPieces pc, int 
         for (int i = threadIdx.x; i < pieces; i += 32) s_w[i] /= l;
     }
     __syncthreads();
-    for (int c = threadIdx.x * 2; c < cp; c += 256) {
-        float x = 0.0f, y = 0.0f;
-#pragma unroll 4
+    for (int c = threadIdx.x * 4; c < cp; c += 512) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float* src = pc.o + base * cp + c;
+#pragma unroll 8
         for (int i = 0; i < pieces; i++) {
-            if (s_w[i] == 0.0f) continue;  // an empty piece has written no sums
-            const float2 v = *(const float2*)(pc.o + (base + (size_t)i * heads) * cp + c);
-            x = fmaf(s_w[i], v.x, x);
-            y = fmaf(s_w[i], v.y, y);
+            const float w = s_w[i];  // 0: an empty piece, which has written no sums
+            const float4 v = w != 0.0f ? *(const float4*)(src + (size_t)i * heads * cp) : make_float4(0.f, 0.f, 0.f, 0.f);
+            x.x = fmaf(w, v.x, x.x); x.y = fmaf(w, v.y, x.y); x.z = fmaf(w, v.z, x.z); x.w = fmaf(w, v.w, x.w);
         }
-        *(uint32_t*)(out + ((size_t)t * heads + h) * cp + c) = pack2(x, y);
+        *(uint2*)(out + ((size_t)t * heads + h) * cp + c) = make_uint2(pack2(x.x, x.y), pack2(x.z, x.w));
     }
 }
 

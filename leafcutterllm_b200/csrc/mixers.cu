@@ -130,12 +130,24 @@ __global__ void __launch_bounds__(512) norm_rows_kernel(const float* __restrict_
     pdl_launch_dependents();
     pdl_wait();
     const float* xr = x + (size_t)(idx ? idx[blockIdx.x] : (int)blockIdx.x) * width;
-    float ss = 0.0f;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) { const float v = xr[c]; ss = fmaf(v, v, ss); }
+    constexpr int kHeld = 8;  // elements of a thread that stay in registers between the passes
+    float v[kHeld], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kHeld; i++) {
+        const int c = threadIdx.x + i * blockDim.x;
+        v[i] = c < width ? xr[c] : 0.0f;
+        ss = fmaf(v[i], v[i], ss);
+    }
+    for (int c = threadIdx.x + kHeld * blockDim.x; c < width; c += blockDim.x) ss = fmaf(xr[c], xr[c], ss);
     ss = block_sum(ss, sh);
     const float r = 1.0f / sqrtf(ss / (float)width + eps);
     A* o = out + (size_t)blockIdx.x * ldo;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) o[c] = to_act<A>(xr[c] * r * w[c]);
+#pragma unroll
+    for (int i = 0; i < kHeld; i++) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < width) o[c] = to_act<A>(v[i] * r * w[c]);
+    }
+    for (int c = threadIdx.x + kHeld * blockDim.x; c < width; c += blockDim.x) o[c] = to_act<A>(xr[c] * r * w[c]);
 }
 
 // ---- gated delta rule ------------------------------------------------------------------------------------------------
@@ -520,25 +532,25 @@ __global__ void rot_table_kernel(const double* __restrict__ freq, int pairs, dou
 
 template <typename A>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const LatentArgs a) {
-    __shared__ float sh[32];
+    __shared__ float sh[32], sh2[32];
     pdl_launch_dependents();
     pdl_wait();
     const LatentShape& g = a.g;
     const int t = blockIdx.x, seq = a.tok_seq[t], pos = a.tok_pos[t];
     const float* p = a.proj + (size_t)t * a.ld_proj;
-    float ss = 0.0f;
-    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) ss = fmaf(p[i], p[i], ss);
-    ss = block_sum(ss, sh);
-    float r = 1.0f / sqrtf(ss / (float)a.q_rank + a.eps);
-    A* cq = (A*)a.cq + (size_t)t * a.ld_cq;
-    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) cq[i] = to_act<A>(p[i] * r * a.q_norm[i]);
-    __syncthreads();
     const float* c = p + a.off_c;
-    ss = 0.0f;
-    for (int i = threadIdx.x; i < g.rank; i += blockDim.x) ss = fmaf(c[i], c[i], ss);
-    ss = block_sum(ss, sh);
-    r = 1.0f / sqrtf(ss / (float)g.rank + a.eps);
+    float sq = 0.0f, sc = 0.0f;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) sq = fmaf(p[i], p[i], sq);
+#pragma unroll 4
+    for (int i = threadIdx.x; i < g.rank; i += blockDim.x) sc = fmaf(c[i], c[i], sc);
     const int page = a.page_table[(size_t)seq * a.pages_per_seq + pos / a.page_tokens];
+    sq = block_sum(sq, sh);
+    sc = block_sum(sc, sh2);
+    const float rq = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps), r = 1.0f / sqrtf(sc / (float)g.rank + a.eps);
+    A* cq = (A*)a.cq + (size_t)t * a.ld_cq;
+#pragma unroll 4
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) cq[i] = to_act<A>(p[i] * rq * a.q_norm[i]);
     A* row = (A*)a.cache + ((size_t)page * a.page_tokens + pos % a.page_tokens) * (g.cp + g.rp);
     for (int i = threadIdx.x; i < g.cp; i += blockDim.x) row[i] = to_act<A>(i < g.rank ? c[i] * r * a.c_norm[i] : 0.0f);
     const float* kr = p + a.off_r;
