@@ -402,7 +402,8 @@ int32_t lc_reset_counters(lc_model* m);
 
 /* Layer-level probes for parity tests: run one sub-block of layer `layer` on host activations
  * through the same kernels lc_forward uses.  attention_forward (attention.rs:37-118) appends to
- * the KV cache of slot 0; ffn_forward (engine.rs:146-164). */
+ * the KV cache of slot 0; ffn_forward (engine.rs:146-164).  For a checkpoint-directory design: the layer's mixer (whatever its kind) and
+ * feed-forward on the residual rows given, before the sublayer's output norm. */
 int32_t lc_probe_attention(lc_model* m, int32_t layer, const float* normed, int32_t seq, float* out);
 int32_t lc_probe_ffn(lc_model* m, int32_t layer, const float* x, int32_t seq, float* out);
 
