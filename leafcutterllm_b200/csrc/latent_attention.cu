@@ -8,6 +8,7 @@
 #include <cmath>
 #include "lc_mixers.h"
 #include "lc_tma.cuh"
+#include "lc_umma.cuh"
 
 namespace lc {
 
@@ -109,196 +110,224 @@ __device__ __forceinline__ float rotated(const bf16* r, const float2* tab, int p
     const float u = __bfloat162float(r[i & ~1]), w = __bfloat162float(r[i | 1]);
     return (i & 1) ? w * cs.x + u * cs.y : u * cs.x - w * cs.y;
 }
-constexpr int kKeys = 64;  // keys per tile
-constexpr int kPartPitch = kKeys + 4;
+constexpr int kKeys = 64;  // keys per tile of the prefill kernel
 
 // Few tokens per sequence: the queries of 16 * MT heads of ONE token are the rows of the products, the cached rows (latent |
-// rotated part) the keys and, without the rotated part, the values.  8 * MT warps: for the scores each takes all rows,
-// sixteen keys and 1 / (2 MT) of the row's elements (partial scores meet in shared memory); for the softmax sixteen threads
-// share a row; for the weighted sum a warp takes all rows and 8 * NCT latent columns.  The context is cut into gridDim.z pieces.
+// rotated part) the keys and, without the rotated part, the values.  The context is cut into gridDim.z pieces and walked in
+// tiles of 32 keys by three kinds of warps:
+//   producer (1)   a lane per key: looks up the cached row and requests it with one bulk copy, four tiles in flight; keys past
+//                  the token's position repeat its own row (their weight is zero, but the row has to be finite);
+//   scores (8)     a warp takes all rows, sixteen keys and a quarter of the rows' elements; the partial scores meet in shared
+//                  memory, then a few threads per row do the online softmax and write the weights, high and low halves;
+//   sums (8)       a warp takes all rows and 8 * NCT latent columns, one tile behind the scores.
+// Waits are bounded; one that runs out raises the library's device error flag (every loop has a fixed count and goes on).
 struct LatentPieces { float *o, *ml; };  // [token][piece][heads][cp] sums, [token][piece][heads][2] maximum (log2 units) and weight sum
+constexpr int kDecodeKeys = 32, kDecodeTiles = 4, kDecodeThreads = 17 * 32, kPPitch = kDecodeKeys + 8, kPartPitch = kDecodeKeys + 4;
 template <int MT, int NCT>
-__global__ void __launch_bounds__(256 * MT) latent_decode_kernel(const LatentArgs a, const LatentPieces pc) {
-    constexpr int KQ = 2 * MT, ROWS = 16 * MT, THREADS = 256 * MT, WARPS = THREADS / 32;
+__global__ void __launch_bounds__(kDecodeThreads, 1) latent_decode_kernel(const LatentArgs a, const LatentPieces pc, int* error_flag) {
+    constexpr int ROWS = 16 * MT, KQ = 4;
+    constexpr int KPT = ROWS * kDecodeKeys / 256, TPR = kDecodeKeys / KPT;  // keys per softmax thread, threads per row
     extern __shared__ __align__(128) unsigned char smem[];
     const LatentShape& g = a.g;
     const int d = g.cp + g.rp, d32 = (d + 31) & ~31, pitch = d32 + 8, row_bytes = pitch * 2;
-    bf16 *s_q = (bf16*)smem, *s_k = s_q + ROWS * pitch, *s_ph = s_k + 2 * kKeys * pitch, *s_pl = s_ph + ROWS * (kKeys + 8);
-    float *s_part = (float*)(s_pl + ROWS * (kKeys + 8)), *s_corr = s_part + KQ * ROWS * kPartPitch;
+    bf16 *s_q = (bf16*)smem, *s_k = s_q + ROWS * pitch, *s_p = s_k + kDecodeTiles * kDecodeKeys * pitch;  // s_p: [2 tiles][high, low][ROWS][kPPitch]
+    float *s_part = (float*)(s_p + 4 * ROWS * kPPitch), *s_corr = s_part + KQ * ROWS * kPartPitch, *s_l = s_corr + 2 * ROWS;
+    uint64_t *full = (uint64_t*)(s_l + ROWS), *empty = full + kDecodeTiles, *p_full = empty + kDecodeTiles, *p_empty = p_full + 2;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
     const int t = blockIdx.x, h0 = blockIdx.y * ROWS, nh = min(ROWS, g.heads - h0);
+    if (tid == 0) {
+        for (int i = 0; i < kDecodeTiles; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], 8); }
+        for (int i = 0; i < 2; i++) { mbar_init(&p_full[i], 8); mbar_init(&p_empty[i], 8); }
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    }
     pdl_launch_dependents();
     pdl_wait();
     const int seq = a.tok_seq[t], pos = a.tok_pos[t], pieces = gridDim.z;
-    const int tiles = pos / kKeys + 1, per = (tiles + pieces - 1) / pieces, kt0 = blockIdx.z * per, kt1 = min(tiles, kt0 + per);
+    const int tiles = pos / kDecodeKeys + 1, per = (tiles + pieces - 1) / pieces, kt0 = blockIdx.z * per, n = min(tiles, kt0 + per) - kt0;
     const size_t out_row = ((size_t)t * pieces + blockIdx.z) * g.heads;
-    if (kt0 >= kt1) {
-        for (int i = tid; i < nh; i += THREADS) { pc.ml[(out_row + h0 + i) * 2] = -INFINITY; pc.ml[(out_row + h0 + i) * 2 + 1] = 0.0f; }
+    if (n <= 0) {
+        for (int i = tid; i < nh; i += kDecodeThreads) { pc.ml[(out_row + h0 + i) * 2] = -INFINITY; pc.ml[(out_row + h0 + i) * 2 + 1] = 0.0f; }
         return;
     }
-    const int32_t* pt = a.page_table + (size_t)seq * a.pages_per_seq;
-    const bf16* cache = (const bf16*)a.cache;
-    const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), ph_sm = smem_u32(s_ph), pl_sm = smem_u32(s_pl);
-    const int chunks = d / 8;
-    auto row_of = [&](int kt) {  // lane j finds the cached row of the warp's j-th key
-        const int kp = kt * kKeys + warp + (lane % (kKeys / WARPS)) * WARPS;
-        return kp <= pos ? pt[kp / a.page_tokens] * a.page_tokens + kp % a.page_tokens : -1;
-    };
-    int rows_next = row_of(kt0);  // of the tile that is loaded next: looked up one tile ahead
-    auto load = [&](int kt, int buf) {
-        const int rows = rows_next;
-        rows_next = row_of(kt + 1);
-#pragma unroll
-        for (int j = 0; j < kKeys / WARPS; j++) {
-            const int rj = __shfl_sync(0xffffffffu, rows, j);
-            const bf16* src = cache + (size_t)max(rj, 0) * d;
-            const uint32_t dst = k_sm + (uint32_t)((buf * kKeys + warp + j * WARPS) * row_bytes);
-            for (int c = lane; c < chunks; c += 32) cp16(dst + c * 16, src + c * 8, rj >= 0 ? 16 : 0);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    // queries: the part carried through the key projection as it is, the other part rotated; both arrive with the first tile
-    for (int i = tid; i < ROWS * (g.cp / 8); i += THREADS) {
+    auto wait = [&](uint64_t* bar, int phase) { if (!mbar_wait(bar, (uint32_t)phase & 1)) atomicExch(error_flag, 14); };
+    const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), p_sm = smem_u32(s_p);
+    // queries: the part carried through the key projection as it is, the other part rotated; zeros behind every row
+    for (int i = tid; i < ROWS * (g.cp / 8); i += kDecodeThreads) {
         const int r = i / (g.cp / 8), c = i - r * (g.cp / 8);
         cp16(q_sm + (uint32_t)(r * row_bytes + c * 16), (const bf16*)a.q_abs + ((size_t)t * g.heads + h0 + min(r, nh - 1)) * g.cp + c * 8, r < nh ? 16 : 0);
     }
-    load(kt0, 0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
     const bf16 zero = __float2bfloat16_rn(0.0f);
-    for (int i = tid; i < 2 * kKeys * (pitch - d); i += THREADS) s_k[(i / (pitch - d)) * pitch + d + i % (pitch - d)] = zero;
+    for (int i = tid; i < kDecodeTiles * kDecodeKeys * (pitch - d); i += kDecodeThreads) s_k[(i / (pitch - d)) * pitch + d + i % (pitch - d)] = zero;
     const float2* tab = a.rot + (size_t)pos * g.rot_pairs;
-    for (int i = tid; i < ROWS * (pitch - g.cp); i += THREADS) {
+    for (int i = tid; i < ROWS * (pitch - g.cp); i += kDecodeThreads) {
         const int r = i / (pitch - g.cp), c = i - r * (pitch - g.cp);
         s_q[r * pitch + g.cp + c] = r < nh && c < g.rp ? __float2bfloat16_rn(rotated((const bf16*)a.q + ((size_t)t * g.heads + h0 + r) * g.ld_q + g.dp, tab, g.rot_pairs, g.rot, c)) : zero;
     }
-    float o[MT][NCT][4];
-#pragma unroll
-    for (int i = 0; i < MT; i++)
-#pragma unroll
-        for (int j = 0; j < NCT; j++) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.0f;
-    const float sc = g.scale * 1.4426950408889634f;
-    const int kg = warp & 3, kq = warp >> 2, steps = d32 / 16, st0 = steps * kq / KQ, st1 = steps * (kq + 1) / KQ;
-    const int srow = tid >> 4, skey = (tid & 15) * 4;  // the softmax's row and its first key of this thread
-    float m_run = -INFINITY, l_run = 0.0f;
-    for (int kt = kt0; kt < kt1; kt++) {
-        const int buf = (kt - kt0) & 1;
-        if (kt + 1 < kt1) { load(kt + 1, buf ^ 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
-        else asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();
-        const uint32_t kb = k_sm + (uint32_t)(buf * kKeys * row_bytes);
-        float s[MT][2][4];
-#pragma unroll
-        for (int i = 0; i < MT; i++)
-#pragma unroll
-            for (int j = 0; j < 2; j++) s[i][j][0] = s[i][j][1] = s[i][j][2] = s[i][j][3] = 0.0f;
-        const uint32_t qa = q_sm + (uint32_t)((lane & 15) * row_bytes + (lane >> 4) * 16);
-        const uint32_t ka = kb + (uint32_t)((kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * row_bytes + ((lane >> 3) & 1) * 16);
-#pragma unroll 3
-        for (int st = st0; st < st1; st++) {
-            uint32_t b[4];
-            ldsm4(ka + st * 32, b);
-#pragma unroll
-            for (int i = 0; i < MT; i++) {
-                uint32_t aq[4];
-                ldsm4(qa + (uint32_t)(16 * i * row_bytes) + st * 32, aq);
-                mma_bf16(s[i][0], aq, b[0], b[1]);
-                mma_bf16(s[i][1], aq, b[2], b[3]);
-            }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+
+    if (warp == 16) {
+        const int32_t* pt = a.page_table + (size_t)seq * a.pages_per_seq;
+        auto row_of = [&](int i) {
+            const int kp = min((kt0 + i) * kDecodeKeys + lane, pos);
+            return (size_t)pt[kp / a.page_tokens] * a.page_tokens + kp % a.page_tokens;
+        };
+        size_t row = row_of(0);
+        for (int i = 0; i < n; i++) {
+            const size_t cur = row;
+            row = row_of(i + 1);
+            const int b = i % kDecodeTiles;
+            if (i >= kDecodeTiles) wait(&empty[b], i / kDecodeTiles - 1);
+            if (lane == 0) mbar_expect_tx(&full[b], (uint32_t)(kDecodeKeys * d * 2));
+            __syncwarp();
+            bulk_load(s_k + (size_t)(b * kDecodeKeys + lane) * pitch, (const bf16*)a.cache + cur * d, (uint32_t)(d * 2), &full[b]);
         }
+    } else if (warp < 8) {
+        const int kg = warp & 1, kq = warp >> 1, steps = d32 / 16, st0 = steps * kq / KQ, st1 = steps * (kq + 1) / KQ;
+        const int srow = tid / TPR, skey = (tid % TPR) * KPT;
+        const float sc = g.scale * 1.4426950408889634f;
+        float m_run = -INFINITY, l_run = 0.0f;
+        const uint32_t qa = q_sm + (uint32_t)((lane & 15) * row_bytes + (lane >> 4) * 16);
+        for (int i = 0; i < n; i++) {
+            const int b = i % kDecodeTiles;
+            wait(&full[b], i / kDecodeTiles);
+            float s[MT][2][4];
 #pragma unroll
-        for (int i = 0; i < MT; i++)
+            for (int m = 0; m < MT; m++)
 #pragma unroll
-            for (int j = 0; j < 2; j++)
+                for (int j = 0; j < 2; j++) s[m][j][0] = s[m][j][1] = s[m][j][2] = s[m][j][3] = 0.0f;
+            const uint32_t ka = k_sm + (uint32_t)((b * kDecodeKeys + kg * 16 + (lane & 7) + ((lane >> 4) << 3)) * row_bytes + ((lane >> 3) & 1) * 16);
+#pragma unroll 3
+            for (int st = st0; st < st1; st++) {
+                uint32_t kb[4];
+                ldsm4(ka + st * 32, kb);
 #pragma unroll
-                for (int r = 0; r < 2; r++)
-                    *(float2*)(s_part + (kq * ROWS + 16 * i + g8 + 8 * r) * kPartPitch + kg * 16 + 8 * j + 2 * t4) = make_float2(s[i][j][2 * r], s[i][j][2 * r + 1]);
-        __syncthreads();
-        {
-            float v[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-            for (int q = 0; q < KQ; q++) {
-                const float4 x = *(const float4*)(s_part + (q * ROWS + srow) * kPartPitch + skey);
-                v[0] += x.x; v[1] += x.y; v[2] += x.z; v[3] += x.w;
+                for (int m = 0; m < MT; m++) {
+                    uint32_t aq[4];
+                    ldsm4(qa + (uint32_t)(16 * m * row_bytes) + st * 32, aq);
+                    mma_bf16(s[m][0], aq, kb[0], kb[1]);
+                    mma_bf16(s[m][1], aq, kb[2], kb[3]);
+                }
             }
+            asm volatile("bar.sync 1, 256;" ::: "memory");  // the previous tile's partial scores have been read
+#pragma unroll
+            for (int m = 0; m < MT; m++)
+#pragma unroll
+                for (int j = 0; j < 2; j++)
+#pragma unroll
+                    for (int r = 0; r < 2; r++)
+                        *(float2*)(s_part + (kq * ROWS + 16 * m + g8 + 8 * r) * kPartPitch + kg * 16 + 8 * j + 2 * t4) = make_float2(s[m][j][2 * r], s[m][j][2 * r + 1]);
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            float v[KPT];
+#pragma unroll
+            for (int j = 0; j < KPT; j++) v[j] = 0.0f;
+#pragma unroll
+            for (int q = 0; q < KQ; q++)
+#pragma unroll
+                for (int j = 0; j < KPT; j += 2) {
+                    const float2 x = *(const float2*)(s_part + (q * ROWS + srow) * kPartPitch + skey + j);
+                    v[j] += x.x; v[j + 1] += x.y;
+                }
             float mx = m_run;
 #pragma unroll
-            for (int j = 0; j < 4; j++) {
-                v[j] = kt * kKeys + skey + j <= pos ? v[j] * sc : -INFINITY;
+            for (int j = 0; j < KPT; j++) {
+                v[j] = (kt0 + i) * kDecodeKeys + skey + j <= pos ? v[j] * sc : -INFINITY;
                 mx = fmaxf(mx, v[j]);
             }
 #pragma unroll
-            for (int w = 1; w < 16; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
+            for (int w = 1; w < TPR; w <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, w));
             const float corr = exp2f(m_run - mx);  // mx is finite: a tile starts at or before the token's position
             m_run = mx;
             float sum = 0.0f;
 #pragma unroll
-            for (int j = 0; j < 4; j++) { v[j] = exp2f(v[j] - mx); sum += v[j]; }
+            for (int j = 0; j < KPT; j++) { v[j] = exp2f(v[j] - mx); sum += v[j]; }
 #pragma unroll
-            for (int w = 1; w < 16; w <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, w);
+            for (int w = 1; w < TPR; w <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, w);
             l_run = l_run * corr + sum;
-            if ((tid & 15) == 0) s_corr[srow] = corr;
-            uint32_t h0, l0, h1, l1;
-            split2(v[0], v[1], h0, l0);
-            split2(v[2], v[3], h1, l1);
-            *(uint2*)(s_ph + srow * (kKeys + 8) + skey) = make_uint2(h0, h1);
-            *(uint2*)(s_pl + srow * (kKeys + 8) + skey) = make_uint2(l0, l1);
-        }
-        __syncthreads();
-        // weighted sum of this warp's latent columns
-        const int c0 = warp * NCT * 8;
-        if (c0 < g.cp) {
+            const int pb = i & 1;
+            if (i >= 2) wait(&p_empty[pb], i / 2 - 1);
+            if (tid % TPR == 0) s_corr[pb * ROWS + srow] = corr;
+            bf16* ph = s_p + (size_t)(2 * pb) * ROWS * kPPitch + srow * kPPitch + skey;
 #pragma unroll
-            for (int i = 0; i < MT; i++) {
-                const float f0 = s_corr[16 * i + g8], f1 = s_corr[16 * i + g8 + 8];
-#pragma unroll
-                for (int j = 0; j < NCT; j++) { o[i][j][0] *= f0; o[i][j][1] *= f0; o[i][j][2] *= f1; o[i][j][3] *= f1; }
+            for (int j = 0; j < KPT; j += 2) {
+                uint32_t hi, lo;
+                split2(v[j], v[j + 1], hi, lo);
+                *(uint32_t*)(ph + j) = hi;
+                *(uint32_t*)(ph + ROWS * kPPitch + j) = lo;
             }
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&p_full[pb]);
+        }
+        if (tid % TPR == 0) {
+            s_l[srow] = l_run;
+            if (pieces > 1 && srow < nh) { pc.ml[(out_row + h0 + srow) * 2] = m_run; pc.ml[(out_row + h0 + srow) * 2 + 1] = l_run; }
+        }
+        asm volatile("bar.sync 2, 512;" ::: "memory");
+    } else {
+        const int c0 = (warp - 8) * NCT * 8;
+        float o[MT][NCT][4];
 #pragma unroll
-            for (int ks = 0; ks < kKeys / 16; ks++) {
-                uint32_t ph[MT][4], pl[MT][4];
+        for (int m = 0; m < MT; m++)
 #pragma unroll
-                for (int i = 0; i < MT; i++) {
-                    const uint32_t off = (uint32_t)((16 * i + (lane & 15)) * (kKeys + 8) + 16 * ks + (lane >> 4) * 8) * 2;
-                    ldsm4(ph_sm + off, ph[i]);
-                    ldsm4(pl_sm + off, pl[i]);
+            for (int j = 0; j < NCT; j++) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.0f;
+        for (int i = 0; i < n; i++) {
+            const int b = i % kDecodeTiles, pb = i & 1;
+            wait(&p_full[pb], i / 2);
+            wait(&full[b], i / kDecodeTiles);
+            if (c0 < g.cp) {
+#pragma unroll
+                for (int m = 0; m < MT; m++) {
+                    const float f0 = s_corr[pb * ROWS + 16 * m + g8], f1 = s_corr[pb * ROWS + 16 * m + g8 + 8];
+#pragma unroll
+                    for (int j = 0; j < NCT; j++) { o[m][j][0] *= f0; o[m][j][1] *= f0; o[m][j][2] *= f1; o[m][j][3] *= f1; }
                 }
+                const uint32_t vb = k_sm + (uint32_t)((b * kDecodeKeys + (lane & 15)) * row_bytes + (c0 + (lane >> 4) * 8) * 2);
 #pragma unroll
-                for (int j = 0; j < NCT; j += 2) {
-                    if (c0 + 8 * j >= g.cp) break;
-                    uint32_t b[4];
-                    ldsm4t(kb + (uint32_t)((16 * ks + (lane & 15)) * row_bytes + (c0 + 8 * j + (lane >> 4) * 8) * 2), b);
+                for (int ks = 0; ks < kDecodeKeys / 16; ks++) {
+                    uint32_t ph[MT][4], pl[MT][4];
 #pragma unroll
-                    for (int i = 0; i < MT; i++) {
-                        mma_bf16(o[i][j], ph[i], b[0], b[1]);
-                        mma_bf16(o[i][j], pl[i], b[0], b[1]);
-                        mma_bf16(o[i][j + 1], ph[i], b[2], b[3]);
-                        mma_bf16(o[i][j + 1], pl[i], b[2], b[3]);
+                    for (int m = 0; m < MT; m++) {
+                        const uint32_t at = p_sm + (uint32_t)(((2 * pb) * ROWS + 16 * m + (lane & 15)) * kPPitch + 16 * ks + (lane >> 4) * 8) * 2;
+                        ldsm4(at, ph[m]);
+                        ldsm4(at + ROWS * kPPitch * 2, pl[m]);
+                    }
+#pragma unroll
+                    for (int j = 0; j < NCT; j += 2) {
+                        if (c0 + 8 * j >= g.cp) break;
+                        uint32_t v[4];
+                        ldsm4t(vb + (uint32_t)(16 * ks * row_bytes + 16 * j), v);
+#pragma unroll
+                        for (int m = 0; m < MT; m++) {
+                            mma_bf16(o[m][j], ph[m], v[0], v[1]);
+                            mma_bf16(o[m][j + 1], ph[m], v[2], v[3]);
+                            mma_bf16(o[m][j], pl[m], v[0], v[1]);
+                            mma_bf16(o[m][j + 1], pl[m], v[2], v[3]);
+                        }
                     }
                 }
             }
+            __syncwarp();
+            if (lane == 0) { mbar_arrive(&empty[b]); mbar_arrive(&p_empty[pb]); }
         }
-        __syncthreads();
-    }
-    // the rows' weight sums, where the loop's corrections were (every warp is past them)
-    if ((tid & 15) == 0) {
-        s_corr[srow] = l_run;
-        if (pieces > 1 && srow < nh) { pc.ml[(out_row + h0 + srow) * 2] = m_run; pc.ml[(out_row + h0 + srow) * 2 + 1] = l_run; }
-    }
-    __syncthreads();
+        asm volatile("bar.sync 2, 512;" ::: "memory");
 #pragma unroll
-    for (int i = 0; i < MT; i++)
+        for (int m = 0; m < MT; m++)
 #pragma unroll
-        for (int r = 0; r < 2; r++) {
-            const int row = 16 * i + g8 + 8 * r;
-            if (row >= nh) continue;
-            const float inv = 1.0f / s_corr[row];
+            for (int r = 0; r < 2; r++) {
+                const int row = 16 * m + g8 + 8 * r;
+                if (row >= nh) continue;
+                const float inv = 1.0f / s_l[row];
 #pragma unroll
-            for (int j = 0; j < NCT; j++) {
-                const int c = (warp * NCT + j) * 8 + 2 * t4;
-                if (c >= g.cp) continue;
-                if (pieces == 1) *(uint32_t*)((bf16*)a.o + ((size_t)t * g.heads + h0 + row) * g.cp + c) = pack2(o[i][j][2 * r] * inv, o[i][j][2 * r + 1] * inv);
-                else *(float2*)(pc.o + (out_row + h0 + row) * g.cp + c) = make_float2(o[i][j][2 * r], o[i][j][2 * r + 1]);
+                for (int j = 0; j < NCT; j++) {
+                    const int c = c0 + 8 * j + 2 * t4;
+                    if (c >= g.cp) continue;
+                    if (pieces == 1) *(uint32_t*)((bf16*)a.o + ((size_t)t * g.heads + h0 + row) * g.cp + c) = pack2(o[m][j][2 * r] * inv, o[m][j][2 * r + 1] * inv);
+                    else *(float2*)(pc.o + (out_row + h0 + row) * g.cp + c) = make_float2(o[m][j][2 * r], o[m][j][2 * r + 1]);
+                }
             }
-        }
+    }
 }
 
 constexpr int kMaxPieces = 64;
@@ -500,7 +529,7 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const LatentArgs a,
 
 size_t decode_smem(const LatentShape& g, int mt) {
     const size_t pitch = ((g.cp + g.rp + 31) & ~31) + 8, rows = 16 * (size_t)mt;
-    return (rows + 2 * kKeys) * pitch * 2 + 2 * rows * (kKeys + 8) * 2 + ((size_t)2 * mt * rows * kPartPitch + rows) * 4;
+    return (rows + kDecodeTiles * kDecodeKeys) * pitch * 2 + 4 * rows * kPPitch * 2 + (4 * rows * kPartPitch + 3 * rows) * 4 + (2 * kDecodeTiles + 4) * 8;
 }
 size_t prefill_smem(const LatentShape& g, int nv) {
     const size_t pitch = ((g.dp + g.rp + 31) & ~31) + 8;
@@ -538,7 +567,7 @@ int32_t launch_latent_attention(const LatentArgs& a, void* scratch, size_t scrat
     if (a.f32 || g.cp > 512 || decode_smem(g, mt) > kMaxSmem) return launch_plain(a, s);
     const int blocks = (g.heads + 16 * mt - 1) / (16 * mt);
     int pieces = std::max(1, std::min(kMaxPieces, sm_count() / (a.T * blocks)));
-    pieces = std::min(pieces, (a.pages_per_seq * a.page_tokens + kKeys - 1) / kKeys);
+    pieces = std::min(pieces, (a.pages_per_seq * a.page_tokens + kDecodeKeys - 1) / kDecodeKeys);
     auto need = [&](int n) { return (size_t)a.T * n * g.heads * ((size_t)g.cp + 2) * sizeof(float); };
     while (pieces > 1 && need(pieces) > scratch_bytes) pieces--;
     LatentPieces pc;
@@ -548,12 +577,12 @@ int32_t launch_latent_attention(const LatentArgs& a, void* scratch, size_t scrat
     const dim3 grid((unsigned)a.T, (unsigned)blocks, (unsigned)pieces);
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(ensure_smem_limit((const void*)kern, smem));
-        LC_CUDA(launch_pdl(kern, grid, dim3((unsigned)(256 * mt)), smem, s, a, pc));
+        LC_CUDA(launch_pdl(kern, grid, dim3(kDecodeThreads), smem, s, a, pc, gemv_error_flag_dev()));
         return LC_OK;
     };
-    const int nct = g.cp <= 128 * mt ? 2 : g.cp <= 256 * mt ? 4 : 8;  // latent columns of a warp, in eights
+    const int nct = g.cp <= 128 ? 2 : g.cp <= 256 ? 4 : 8;  // latent columns of a warp, in eights
     if (mt == 1) LC_TRY(nct == 2 ? go(latent_decode_kernel<1, 2>) : nct == 4 ? go(latent_decode_kernel<1, 4>) : go(latent_decode_kernel<1, 8>));
-    else LC_TRY(nct == 2 ? go(latent_decode_kernel<2, 2>) : go(latent_decode_kernel<2, 4>));
+    else LC_TRY(nct == 2 ? go(latent_decode_kernel<2, 2>) : nct == 4 ? go(latent_decode_kernel<2, 4>) : go(latent_decode_kernel<2, 8>));
     if (pieces > 1) {
         LC_CUDA(launch_pdl(latent_merge_kernel, dim3((unsigned)g.heads, (unsigned)a.T), dim3(128), 0, s, pc, pieces, g.heads, g.cp, (bf16*)a.o));
         *launches = 2;
