@@ -3,11 +3,16 @@
 // name -> dtype, shape, data_offsets, then the data).
 #include <cmath>
 #include <cstring>
+#include <initializer_list>
 #include "lc_arch.h"
 #include "lc_json.h"
 #include "lc_model.h"
 
 namespace lc {
+
+const char* mixer_name(MixerKind k) {
+    return k == MixerKind::ChannelDelta ? "channel_delta" : k == MixerKind::LatentAttention ? "latent_attention" : "attention";
+}
 
 void rotary_frequencies(const RotarySpec& r, std::vector<double>* freq, double* magnitude) {
     const int n = r.dims / 2;
@@ -29,7 +34,7 @@ namespace {
 
 // Typed access to one JSON object; the first problem is kept as the error text.
 struct Fields {
-    const JValue* o;
+    const JValue* o = nullptr;
     std::string where;
     const JValue* need(const char* key, JValue::Kind kind) const {
         const JValue* v = o ? o->get(key) : nullptr;
@@ -55,6 +60,11 @@ struct Fields {
         *out = (float)d;
         return LC_OK;
     }
+    int32_t child(const char* key, Fields* out) const {
+        out->o = need(key, JValue::OBJ);
+        out->where = where + "." + key;
+        return out->o ? LC_OK : LC_ERR_INVALID;
+    }
     bool has(const char* key) const { const JValue* v = o->get(key); return v && v->kind != JValue::NUL; }
 };
 
@@ -76,21 +86,75 @@ int32_t parse_rotary(const JValue& v, const std::string& where, RotarySpec* out)
     return LC_OK;
 }
 
-int32_t parse_layer(const JValue& v, int index, LayerSpec* out) {
+// The constants of plain attention: heads over shared key/value heads, rotation, window, the layer whose cache it reads.
+int32_t parse_attention(const Fields& m, int index, LayerSpec* out) {
+    LC_TRY(m.integer("kv_heads", &out->kv_heads, 1));
+    LC_CHECK(out->heads % out->kv_heads == 0, LC_ERR_INVALID, "config: %s: %d heads over %d key heads", m.where.c_str(), out->heads, out->kv_heads);
+    LC_TRY(m.real("scale", &out->scale));
+    if (m.has("rot")) {
+        const JValue* rot = m.need("rot", JValue::OBJ);
+        if (!rot) return LC_ERR_INVALID;
+        LC_TRY(parse_rotary(*rot, m.where, &out->rot));
+        LC_CHECK(out->rot.dims <= out->dim, LC_ERR_INVALID, "config: %s: %d of %d dimensions rotated", m.where.c_str(), out->rot.dims, out->dim);
+    }
+    if (m.has("mask")) {
+        Fields k;
+        LC_TRY(m.child("mask", &k));
+        LC_TRY(k.integer("size", &out->mask.size, 1));
+        if (k.has("keep_first")) LC_TRY(k.integer("keep_first", &out->mask.keep_first, 0));
+    }
+    if (m.has("kv_from")) {
+        LC_TRY(m.integer("kv_from", &out->kv_from, 0));
+        LC_CHECK(out->kv_from < index, LC_ERR_INVALID, "config: %s: 'kv_from' %d is not an earlier layer", m.where.c_str(), out->kv_from);
+    }
+    return LC_OK;
+}
+
+int32_t parse_moe(const Fields& p, MoeSpec* out) {
+    Fields expert, router;
+    LC_TRY(p.child("expert", &expert));
+    LC_TRY(expert.integer("ff", &out->ff, 1));
+    LC_TRY(p.child("router", &router));
+    LC_TRY(router.integer("experts", &out->experts, 1));
+    LC_TRY(router.integer("top", &out->top, 1));
+    if (router.has("identity")) LC_TRY(router.integer("identity", &out->identity, 0));
+    if (router.has("groups")) {
+        Fields g;
+        LC_TRY(router.child("groups", &g));
+        LC_TRY(g.integer("count", &out->groups, 1));
+        LC_TRY(g.integer("keep", &out->keep, 1));
+    }
+    if (p.has("shared")) {
+        Fields sh;
+        LC_TRY(p.child("shared", &sh));
+        LC_TRY(sh.integer("ff", &out->shared_ff, 1));
+    }
+    const int n = out->outputs();
+    LC_CHECK(n % out->groups == 0 && out->keep <= out->groups, LC_ERR_INVALID, "config: %s: %d router outputs in %d groups, %d kept", router.where.c_str(), n, out->groups, out->keep);
+    LC_CHECK(out->top <= n / out->groups * out->keep, LC_ERR_INVALID, "config: %s: 'top' %d of at most %d", router.where.c_str(), out->top, n / out->groups * out->keep);
+    LC_CHECK(n <= kMaxRouterOutputs && out->top <= kMaxChoices, LC_ERR_UNSUPPORTED, "config: %s: %d router outputs, top %d (at most %d, %d)", router.where.c_str(), n, out->top,
+             kMaxRouterOutputs, kMaxChoices);
+    return LC_OK;
+}
+
+// dense: what "kind": "dense" means in the design
+int32_t parse_layer(const JValue& v, int index, FfnKind dense, std::initializer_list<MixerKind> mixers, LayerSpec* out) {
     Fields f{&v, "layer " + std::to_string(index)};
     const JValue *type = f.need("type", JValue::STR), *mixer = f.need("mixer", JValue::OBJ);
     if (!type || !mixer) return LC_ERR_INVALID;
     Fields m{mixer, f.where + ".mixer"};
+    bool known = false;
+    for (MixerKind k : mixers)
+        if (type->str == mixer_name(k)) { out->mixer = k; known = true; }
+    LC_CHECK(known, LC_ERR_UNSUPPORTED, "config: %s: unknown mixer type '%s'", f.where.c_str(), type->str.c_str());
     LC_TRY(m.integer("heads", &out->heads, 1));
     LC_TRY(m.integer("dim", &out->dim, 1));
     LC_TRY(m.integer("vdim", &out->vdim, 1));
-    if (type->str == "channel_delta") {
-        out->mixer = MixerKind::ChannelDelta;
+    if (out->mixer == MixerKind::ChannelDelta) {
         LC_TRY(m.integer("kv_heads", &out->kv_heads, 1));
         LC_TRY(m.integer("conv", &out->conv_taps, 1));
         LC_CHECK(out->heads % out->kv_heads == 0, LC_ERR_INVALID, "config: %s: %d heads over %d key heads", m.where.c_str(), out->heads, out->kv_heads);
-    } else if (type->str == "latent_attention") {
-        out->mixer = MixerKind::LatentAttention;
+    } else if (out->mixer == MixerKind::LatentAttention) {
         LC_TRY(m.integer("kv_rank", &out->kv_rank, 1));
         LC_TRY(m.integer("rot_dim", &out->rot_dim, 2));
         if (m.has("q_rank")) LC_TRY(m.integer("q_rank", &out->q_rank, 1));
@@ -100,29 +164,30 @@ int32_t parse_layer(const JValue& v, int index, LayerSpec* out) {
         LC_TRY(parse_rotary(*rot, m.where, &out->rot));
         LC_CHECK(out->rot.dims <= out->rot_dim, LC_ERR_INVALID, "config: %s: %d of %d dimensions rotated", m.where.c_str(), out->rot.dims, out->rot_dim);
     } else {
-        set_error("config: %s: unknown mixer type '%s'", f.where.c_str(), type->str.c_str());
-        return LC_ERR_UNSUPPORTED;
+        LC_TRY(parse_attention(m, index, out));
     }
     if (f.has("mlp")) {
-        const JValue* mlp = f.need("mlp", JValue::OBJ);
-        if (!mlp) return LC_ERR_INVALID;
-        Fields p{mlp, f.where + ".mlp"};
+        Fields p;
+        LC_TRY(f.child("mlp", &p));
         const JValue* kind = p.need("kind", JValue::STR);
         if (!kind) return LC_ERR_INVALID;
-        LC_CHECK(kind->str == "dense", LC_ERR_UNSUPPORTED, "config: %s: unknown kind '%s'", p.where.c_str(), kind->str.c_str());
-        out->ffn = FfnKind::Relu2;
-        LC_TRY(p.integer("ff", &out->ff, 1));
+        if (kind->str == "dense") {
+            out->ffn = dense;
+            LC_TRY(p.integer("ff", &out->ff, 1));
+        } else if (kind->str == "moe" && dense == FfnKind::GatedSilu) {
+            out->ffn = FfnKind::Moe;
+            LC_TRY(parse_moe(p, &out->moe));
+        } else {
+            set_error("config: %s: unknown kind '%s'", p.where.c_str(), kind->str.c_str());
+            return LC_ERR_UNSUPPORTED;
+        }
     }
     return LC_OK;
 }
 
-// Varasun: a free mix of gated-delta-rule layers and latent-attention layers, listed one by one.
-int32_t parse_varasun(const JValue& cfg, ArchSpec* out) {
-    Fields f{&cfg, "the model"};
+int32_t parse_stack(const Fields& f, FfnKind dense, std::initializer_list<MixerKind> mixers, ArchSpec* out) {
     LC_TRY(f.integer("width", &out->width, 1));
     LC_TRY(f.integer("vocab", &out->vocab, 1));
-    LC_TRY(f.real("logit_scale", &out->logit_scale));
-    LC_TRY(f.real("logit_softcap", &out->logit_softcap));
     const JValue* norm = f.need("norm", JValue::OBJ);
     if (!norm) return LC_ERR_INVALID;
     LC_TRY((Fields{norm, "norm"}.real("eps", &out->eps)));
@@ -131,14 +196,37 @@ int32_t parse_varasun(const JValue& cfg, ArchSpec* out) {
     LC_CHECK(!layers->arr.empty(), LC_ERR_INVALID, "config: no layers");
     for (size_t i = 0; i < layers->arr.size(); i++) {
         LayerSpec ly;
-        LC_TRY(parse_layer(layers->arr[i], (int)i, &ly));
+        LC_TRY(parse_layer(layers->arr[i], (int)i, dense, mixers, &ly));
+        if (ly.kv_from >= 0) {
+            const LayerSpec& src = out->layers[(size_t)ly.kv_from];
+            LC_CHECK(src.mixer == MixerKind::Attention && src.kv_from < 0 && src.kv_heads == ly.kv_heads && src.dim == ly.dim && src.vdim == ly.vdim, LC_ERR_INVALID,
+                     "config: layer %d cannot read the keys and values of layer %d", (int)i, ly.kv_from);
+        }
         out->layers.push_back(ly);
     }
     return LC_OK;
 }
 
+// Varasun: a free mix of gated-delta-rule layers and latent-attention layers, listed one by one.
+int32_t parse_varasun(const JValue& cfg, ArchSpec* out) {
+    Fields f{&cfg, "the model"};
+    LC_TRY(f.real("logit_scale", &out->logit_scale));
+    LC_TRY(f.real("logit_softcap", &out->logit_softcap));
+    return parse_stack(f, FfnKind::Relu2, {MixerKind::ChannelDelta, MixerKind::LatentAttention}, out);
+}
+
+// Tenetar: windowed attention layers, some of which read an earlier layer's keys and values, with gated or mixture
+// feed-forwards; norms on both sides of every sublayer.
+int32_t parse_tenetar(const JValue& cfg, ArchSpec* out) {
+    Fields f{&cfg, "the model"}, e;
+    LC_TRY(f.child("embedding", &e));
+    LC_TRY(e.real("scale", &out->embed_scale));
+    out->norm_inputs = true;
+    return parse_stack(f, FfnKind::GatedSilu, {MixerKind::Attention}, out);
+}
+
 struct ArchEntry { const char* name; int32_t (*parse)(const JValue&, ArchSpec*); };
-const ArchEntry kRegistry[] = {{"Varasun", parse_varasun}};
+const ArchEntry kRegistry[] = {{"Varasun", parse_varasun}, {"Tenetar", parse_tenetar}};
 
 uint32_t safetensors_type(const std::string& dtype) {
     if (dtype == "BF16") return LC_TYPE_BF16;

@@ -11,6 +11,8 @@
 //            lane = weight row, so a warp's store of one token is contiguous.
 // Few tiles: k is cut into shares over several CTAs; each leaves its partial tile in scratch and takes a ticket, the last one
 // adds the shares in share order (the result does not depend on which CTA that is) and runs the epilogue.
+// Grouped form (one matrix per expert): the tokens come as tiles of rows that share a matrix, found on the device.  Their
+// activations are gathered four rows at a time (TMA gather), the instruction's N follows the tile's rows.
 // Work items are dealt round robin to a grid of at most one CTA per SM.  Every wait is bounded: one that runs out raises the
 // library's device error flag and the CTA winds down (copies awaited, tensor memory freed).
 //
@@ -40,12 +42,19 @@ struct DenseParams {
     int n, T, ldo, kblocks, mt, nt, batch, shares, items, stages, stage_tx;
     int out_f32, epi, e_div;
     float scale, cap;
+    void* out2;
+    int ldo2, split;
+    // grouped form
+    const ExpertTile* tiles;
+    const int32_t *n_tiles, *lists, *off;
+    int list_stride;
 };
 
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // ea, eb: the row's constants of the epilogue
-__device__ __forceinline__ float dense_epilogue(const DenseParams& p, float ea, float eb, float y) {
+__device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool second, float ea, float eb, float y) {
     switch (p.epi) {
+        case DENSE_SPLIT_RELU2: if (!second) return y;  // fall through
         case DENSE_RELU2: { const float r = fmaxf(y, 0.0f); return r * r; }
         case DENSE_LOG_DECAY: return -ea * softplus_f(y + eb);
         case DENSE_LOGITS: { const float v = y * p.scale; return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v; }
@@ -56,38 +65,56 @@ __device__ __forceinline__ void dense_row_constants(const DenseParams& p, int ro
     ea = eb = 0.0f;
     if (p.epi == DENSE_LOG_DECAY && row < p.n) { ea = p.e0[row / p.e_div]; eb = p.e1[row]; }
 }
-// 16 accumulators of weight row `row`, tokens t0 .. t0 + 15, for a whole warp (lane = row).  bf16: lane pairs swap halves, so
-// a lane stores two rows of every other token.
-__device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int row, int t0, const float (&v)[16], float ea, float eb) {
-    const size_t at = (size_t)b * p.out_batch + (size_t)t0 * p.ldo + row;
-    const int m = min(16, p.T - t0);
-    if (p.out_f32) {
-        if (row >= p.n) return;
-        float* o = (float*)p.out + at;
-#pragma unroll
-        for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * p.ldo] = dense_epilogue(p, ea, eb, v[j]);
-    } else if ((p.n & 1) == 0 && (p.ldo & 1) == 0) {  // row pairs stay inside the matrix and 4-byte aligned
+__device__ __forceinline__ float silu_of(float g) { return g / (1.0f + expf(-g)); }
+// 16 accumulators of weight row `row`, tokens t0 .. t0 + m - 1 (m may exceed 16), for a whole warp (lane = row).  bf16: lane
+// pairs swap halves, so a lane stores two rows of every other token.
+__device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int row, int t0, int m, const float (&v)[16], float ea, float eb) {
+    if (p.epi == DENSE_GATED_SILU) {  // even lanes hold gates, odd ones the matching values; each makes every other token's output
         const bool odd = row & 1;
-        __nv_bfloat16* o = (__nv_bfloat16*)p.out + at - (odd ? 1 : 0);
+        const size_t at = (size_t)b * p.out_batch + (size_t)t0 * p.ldo + (row >> 1);
 #pragma unroll
         for (int j = 0; j < 16; j += 2) {
-            const float x = dense_epilogue(p, ea, eb, v[j]), y = dense_epilogue(p, ea, eb, v[j + 1]);
+            const float other = __shfl_xor_sync(0xffffffffu, odd ? v[j] : v[j + 1], 1);
+            const float y = odd ? silu_of(other) * v[j + 1] : silu_of(v[j]) * other;
+            const int jj = j + (odd ? 1 : 0);
+            if (jj >= m || row >= p.n) continue;
+            if (p.out_f32) ((float*)p.out)[at + (size_t)jj * p.ldo] = y;
+            else ((__nv_bfloat16*)p.out)[at + (size_t)jj * p.ldo] = __float2bfloat16_rn(y);
+        }
+        return;
+    }
+    // a warp's 32 rows lie on one side of a split
+    const bool second = p.epi == DENSE_SPLIT_RELU2 && row >= p.split;
+    const int ldo = second ? p.ldo2 : p.ldo, r = second ? row - p.split : row;
+    void* out = second ? p.out2 : p.out;
+    const size_t at = (size_t)b * p.out_batch + (size_t)t0 * ldo + r;
+    if (p.epi == DENSE_SPLIT_RELU2 ? !second : p.out_f32) {
+        if (row >= p.n) return;
+        float* o = (float*)out + at;
+#pragma unroll
+        for (int j = 0; j < 16; j++)
+            if (j < m) o[(size_t)j * ldo] = dense_epilogue(p, second, ea, eb, v[j]);
+    } else if ((p.n & 1) == 0 && (ldo & 1) == 0) {  // row pairs stay inside the matrix and 4-byte aligned
+        const bool odd = row & 1;
+        __nv_bfloat16* o = (__nv_bfloat16*)out + at - (odd ? 1 : 0);
+#pragma unroll
+        for (int j = 0; j < 16; j += 2) {
+            const float x = dense_epilogue(p, second, ea, eb, v[j]), y = dense_epilogue(p, second, ea, eb, v[j + 1]);
             const float other = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
             const __nv_bfloat162 pr = odd ? __floats2bfloat162_rn(other, y) : __floats2bfloat162_rn(x, other);
             const int jj = j + (odd ? 1 : 0);
-            if (jj < m && row < p.n) *(__nv_bfloat162*)(o + (size_t)jj * p.ldo) = pr;
+            if (jj < m && row < p.n) *(__nv_bfloat162*)(o + (size_t)jj * ldo) = pr;
         }
     } else {
         if (row >= p.n) return;
-        __nv_bfloat16* o = (__nv_bfloat16*)p.out + at;
+        __nv_bfloat16* o = (__nv_bfloat16*)out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * p.ldo] = __float2bfloat16_rn(dense_epilogue(p, ea, eb, v[j]));
+            if (j < m) o[(size_t)j * ldo] = __float2bfloat16_rn(dense_epilogue(p, second, ea, eb, v[j]));
     }
 }
 
-template <int NT>
+template <int NT, bool GROUPED>
 __global__ void __launch_bounds__(kThreads, NT <= 64 ? 2 : 1)
 dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ CUtensorMap tx, const DenseParams p) {
     constexpr int kBBytes = NT * kKB * 2, kStage = kABytes + kBBytes;
@@ -116,18 +143,67 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
     pdl_launch_dependents();
 
     // item -> (weight tile fastest over shares, then token tiles): consecutive CTAs share a weight tile's rows
-    struct Item { int b, m, n, share, k0, k1; };
+    struct Item { int b, m, n, share, k0, k1, t0, rows, first; };
     auto item_of = [&](int it) {
         Item r;
         r.share = it % p.shares; it /= p.shares;
-        r.n = it % p.nt; it /= p.nt;
-        r.m = it % p.mt; r.b = it / p.mt;
+        if constexpr (GROUPED) {  // neighbours share a tile's activations, then an expert's matrix
+            r.m = it % p.mt; r.n = it / p.mt;
+            const ExpertTile tl = p.tiles[r.n];
+            r.b = tl.expert; r.t0 = tl.row0; r.rows = tl.rows; r.first = tl.first;
+        } else {
+            r.n = it % p.nt; it /= p.nt;
+            r.m = it % p.mt; r.b = it / p.mt;
+            r.t0 = r.n * NT; r.rows = p.T - r.t0; r.first = 0;
+        }
         r.k0 = (int)((long long)p.kblocks * r.share / p.shares);
         r.k1 = (int)((long long)p.kblocks * (r.share + 1) / p.shares);
         return r;
     };
     auto block = [&](const Item& r, int kb) { return w + (((size_t)r.b * p.mt + r.m) * p.kblocks + kb) * kABytes; };
-    if (warp == 0 && lane == 0) {
+    if (GROUPED && warp == 0) {
+        pdl_wait();
+        const int items = *p.n_tiles * p.mt * p.shares;
+        int issued = 0, st = 0;
+        uint32_t phase = 1;
+        bool ok = true;
+        for (int it = blockIdx.x; it < items && ok; it += gridDim.x) {
+            const Item r = item_of(it);
+            const unsigned char* wb = block(r, r.k0);
+            const int fours = (r.rows + 3) / 4;
+            int4 rows[2];  // of the gathers lane and lane + 32
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                int* q = &rows[i].x;
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    const int at = min((lane + 32 * i) * 4 + j, r.rows - 1);
+                    q[j] = p.lists ? p.lists[(size_t)r.b * p.list_stride + r.first + at] : r.t0 + at;
+                }
+            }
+            for (int kb = r.k0; kb < r.k1; kb++, wb += kABytes) {
+                unsigned char* a = smem + (size_t)st * kStage;
+                const bool free = issued < p.stages || mbar_wait(&empty[st], phase);
+                if (!__all_sync(0xffffffffu, free)) { ok = false; break; }
+                if (lane == 0) {
+                    mbar_expect_tx(&full[st], kABytes + fours * 512);
+                    bulk_load(a, wb, kABytes, &full[st]);
+                }
+                __syncwarp();
+#pragma unroll
+                for (int i = 0; i < 2; i++)
+                    if (lane + 32 * i < fours) tma_gather4(a + kABytes + (lane + 32 * i) * 512, &tx, kb * kKB, rows[i], &full[st]);
+                issued++;
+                if (++st == p.stages) { st = 0; phase ^= 1; }
+            }
+        }
+        if (!ok && lane == 0) {
+            *stop = 1;
+            atomicExch(p.error_flag, 11);
+            for (int i = max(0, issued - p.stages); i < issued; i++) mbar_wait(&full[i % p.stages], (uint32_t)(i / p.stages) & 1);
+        }
+        __syncwarp();
+    } else if (warp == 0 && lane == 0) {
         int issued = 0;
         bool ok = true;
         // weight boxes of the first stages, before the activations exist
@@ -163,14 +239,17 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
             for (int i = max(0, issued - p.stages); i < issued; i++) mbar_wait(&full[i % p.stages], (uint32_t)(i / p.stages) & 1);
         }
     } else if (warp == 1 && lane == 0) {
-        const uint32_t idesc = idesc_bf16(kM, NT);
+        uint32_t idesc = idesc_bf16(kM, NT);
+        if constexpr (GROUPED) pdl_wait();
+        const int items = GROUPED ? *p.n_tiles * p.mt * p.shares : p.items;
         const uint64_t desc0 = umma_desc_sw128(smem_u32(smem));  // a start address below 256 KB: adding to the descriptor moves it
         int tile = 0, st = 0;
         uint32_t phase = 0;
         bool ok = true;
-        for (int it = blockIdx.x; it < p.items && ok; it += gridDim.x, tile++) {
+        for (int it = blockIdx.x; it < items && ok; it += gridDim.x, tile++) {
             const Item r = item_of(it);
             const int set = tile & 1;
+            if constexpr (GROUPED) idesc = idesc_bf16(kM, (r.rows + 15) & ~15);
             if (tile >= 2 && !mbar_wait(&acc_empty[set], (uint32_t)(tile / 2 - 1) & 1)) { ok = false; break; }
             tc_fence_after();
             const uint32_t d = tmem + (uint32_t)set * kCols;
@@ -190,22 +269,23 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
         pdl_wait();  // earlier kernels may still read what this one overwrites
         constexpr int kHalf = NT >= 32 ? NT / 2 : NT;  // tokens of one warp; a 16-token tile leaves the second half idle
         const int quarter = warp & 3, half = (warp - 4) >> 2, row_in = quarter * 32 + lane, c_lo = half * kHalf, c_hi = c_lo < NT ? c_lo + kHalf : c_lo;
+        const int items = GROUPED ? *p.n_tiles * p.mt * p.shares : p.items;
         int tile = 0;
-        for (int it = blockIdx.x; it < p.items; it += gridDim.x, tile++) {
+        for (int it = blockIdx.x; it < items; it += gridDim.x, tile++) {
             const Item r = item_of(it);
             const int set = tile & 1;
-            const int row = r.m * kM + row_in, t0 = r.n * NT;
+            const int row = r.m * kM + row_in, t0 = r.t0, ob = GROUPED ? 0 : r.b;
             float ea, eb;
             dense_row_constants(p, row, ea, eb);
             if (!mbar_wait(&acc_full[set], (uint32_t)(tile / 2) & 1)) { *stop = 1; if (lane == 0) atomicExch(p.error_flag, 13); break; }
             tc_fence_after();
             const uint32_t base = tmem + (uint32_t)set * kCols + ((uint32_t)(quarter * 32) << 16);
             const size_t plane = (size_t)NT * kM;
-            const int cell = (r.b * p.mt + r.m) * p.nt + r.n;
+            const int cell = GROUPED ? r.n * p.mt + r.m : (r.b * p.mt + r.m) * p.nt + r.n;
             float* part = p.shares > 1 ? p.partial + (size_t)cell * p.shares * plane : nullptr;
 #pragma unroll 1
             for (int c = c_lo; c < c_hi; c += 16) {
-                if (t0 + c >= p.T) break;
+                if (c >= r.rows) break;
                 uint32_t raw[16];
                 tmem_ld16(base + c, raw);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -213,12 +293,12 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
 #pragma unroll
                 for (int j = 0; j < 16; j++) v[j] = __uint_as_float(raw[j]);
                 if (part) {
-                    const int m = p.T - t0 - c;
+                    const int m = r.rows - c;
 #pragma unroll
                     for (int j = 0; j < 16; j++)
                         if (j < m) part[(size_t)r.share * plane + (size_t)(c + j) * kM + row_in] = v[j];
                 } else {
-                    dense_store16(p, r.b, row, t0 + c, v, ea, eb);
+                    dense_store16(p, ob, row, t0 + c, r.rows - c, v, ea, eb);
                 }
             }
             tc_fence_before();
@@ -238,9 +318,9 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
                 if (mine) {
 #pragma unroll 1
                     for (int c = c_lo; c < c_hi; c += 16) {
-                        if (t0 + c >= p.T) break;
+                        if (c >= r.rows) break;
                         float v[16];
-                        const int m = p.T - t0 - c;
+                        const int m = r.rows - c;
 #pragma unroll
                         for (int j = 0; j < 16; j++) v[j] = 0.0f;
                         const float* ps = part + (size_t)c * kM + row_in;
@@ -249,7 +329,7 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
 #pragma unroll
                             for (int j = 0; j < 16; j++)
                                 if (j < m) v[j] += __ldcg(ps + j * kM);
-                        dense_store16(p, r.b, row, t0 + c, v, ea, eb);
+                        dense_store16(p, ob, row, t0 + c, r.rows - c, v, ea, eb);
                     }
                 }
             }
@@ -280,23 +360,32 @@ __global__ void tile_kernel(const __nv_bfloat16* __restrict__ src, int n, int k,
     }
 }
 
-// True 32-bit: 64 weight rows x 64 tokens per CTA, 4 x 4 outputs per thread.
+// True 32-bit: 64 weight rows x 64 tokens per CTA, 4 x 4 outputs per thread.  Grouped (p.off): blockIdx.z is the expert, the
+// tokens are the rows of its list.
 __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __restrict__ w, int ldw, size_t w_batch, const float* __restrict__ x, int ldx,
                                                         size_t x_batch, int k, const DenseParams p) {
     constexpr int KT = 16;
     __shared__ float ws[KT][64 + 4], xs[KT][64 + 4];
+    __shared__ int x_row[64];
     pdl_launch_dependents();
     pdl_wait();
     const int r0 = blockIdx.x * 64, t0 = blockIdx.y * 64, b = blockIdx.z;
+    const int row0 = p.off ? p.off[b] : 0, T = p.off ? p.off[b + 1] - row0 : p.T;
+    if (t0 >= T) return;
     w += (size_t)b * w_batch;
-    x += (size_t)b * x_batch;
+    if (!p.off) x += (size_t)b * x_batch;
+    if (threadIdx.x < 64) {
+        const int t = min(t0 + (int)threadIdx.x, T - 1);
+        x_row[threadIdx.x] = p.lists ? p.lists[(size_t)b * p.list_stride + t] : row0 + t;
+    }
+    __syncthreads();
     const int tr = threadIdx.x & 15, tt = threadIdx.x >> 4;
     float acc[4][4] = {};
     for (int k0 = 0; k0 < k; k0 += KT) {
         for (int i = threadIdx.x; i < 64 * KT; i += 256) {
             const int r = i / KT, c = i % KT, kk = k0 + c;
             ws[c][r] = (r0 + r < p.n && kk < k) ? __bfloat162float(w[(size_t)(r0 + r) * ldw + kk]) : 0.0f;
-            xs[c][r] = (t0 + r < p.T && kk < k) ? x[(size_t)(t0 + r) * ldx + kk] : 0.0f;
+            xs[c][r] = (t0 + r < T && kk < k) ? x[(size_t)x_row[r] * ldx + kk] : 0.0f;
         }
         __syncthreads();
 #pragma unroll
@@ -314,28 +403,32 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int t = t0 + tt + 16 * i;
-        if (t >= p.T) continue;
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int row = r0 + tr + 16 * j;
-            if (row < p.n) {
-                float ea, eb;
-                dense_row_constants(p, row, ea, eb);
-                ((float*)p.out)[(size_t)b * p.out_batch + (size_t)t * p.ldo + row] = dense_epilogue(p, ea, eb, acc[i][j]);
+            if (p.epi == DENSE_GATED_SILU) {
+                const float up = __shfl_xor_sync(0xffffffffu, acc[i][j], 1);
+                if (t < T && row < p.n && (row & 1) == 0) ((float*)p.out)[(size_t)(row0 + t) * p.ldo + (row >> 1)] = silu_of(acc[i][j]) * up;
+                continue;
             }
+            if (t >= T || row >= p.n) continue;
+            float ea, eb;
+            dense_row_constants(p, row, ea, eb);
+            if (p.epi == DENSE_SPLIT_RELU2 && row >= p.split) ((float*)p.out2)[(size_t)t * p.ldo2 + row - p.split] = dense_epilogue(p, true, ea, eb, acc[i][j]);
+            else ((float*)p.out)[(p.off ? 0 : (size_t)b * p.out_batch) + (size_t)(row0 + t) * p.ldo + row] = dense_epilogue(p, false, ea, eb, acc[i][j]);
         }
     }
 }
 
-template <int NT>
+template <int NT, bool GROUPED>
 int32_t launch_umma(const DenseArgs& a, const CUtensorMap& tx, DenseParams p, cudaStream_t s) {
     const size_t stage = kABytes + (size_t)NT * kKB * 2, fixed = 1024 + 512;
     // few tokens: half of the shared memory, so that the next kernel's first weight boxes travel while this one drains
     p.stages = (int)((NT <= 64 ? kMaxSmem / 2 - 1024 : kMaxSmem) - fixed) / (int)stage;
     const size_t smem = fixed + (size_t)p.stages * stage;
-    LC_CUDA(ensure_smem_limit((const void*)dense_umma_kernel<NT>, smem));
+    LC_CUDA(ensure_smem_limit((const void*)dense_umma_kernel<NT, GROUPED>, smem));
     const int grid = std::min(p.items, sm_count());
-    LC_CUDA(launch_pdl(dense_umma_kernel<NT>, dim3((unsigned)grid), dim3(kThreads), smem, s, a.w->tiles, tx, p));
+    LC_CUDA(launch_pdl(dense_umma_kernel<NT, GROUPED>, dim3((unsigned)grid), dim3(kThreads), smem, s, a.w->tiles, tx, p));
     return LC_OK;
 }
 
@@ -379,6 +472,57 @@ void dense_workspace_free(DenseWorkspace* ws) {
     ws->maps.clear();
 }
 
+namespace {
+// Shares of k, where cutting it evens out the CTAs' work: k blocks of the busiest CTA, plus what an item and the summing of
+// the shares cost.  `cells` are expected tiles, `room` the most there can be.
+int choose_shares(const DenseParams& p, const DenseWorkspace& ws, int NT, int cells, int room) {
+    int shares = 1;
+    if (NT > 64 || room > ws.max_tickets) return shares;
+    const int sms = sm_count();
+    long best = -1;
+    for (int c = 1; c <= std::min(16, p.kblocks / 2); c++) {
+        if ((size_t)room * c * NT * kM * sizeof(float) > ws.partial_bytes) break;
+        const long waves = ((long)cells * c + sms - 1) / sms;
+        const long cost = waves * (((p.kblocks + c - 1) / c) + 2 + (c > 1 ? NT / 16 : 0)) + (c > 1 ? 3 + c * NT / 32 : 0);
+        if (best < 0 || cost < best) { best = cost; shares = c; }
+    }
+    return shares;
+}
+
+// The tensor map for `key`, made by `make` when it is new.
+template <typename Make>
+int32_t map_of(DenseWorkspace& ws, const std::vector<uint64_t>& key, Make make, const CUtensorMap** out) {
+    std::unique_ptr<DenseWorkspace::Map>& mp = ws.maps[key];
+    if (!mp) {
+        mp.reset(new DenseWorkspace::Map);
+        const bool ok = make(mp->b);
+        if (!ok) ws.maps.erase(key);
+        LC_CHECK(ok, LC_ERR_CUDA, "dense product: no tensor map over the activations");
+    }
+    *out = (const CUtensorMap*)mp->b;
+    return LC_OK;
+}
+
+int32_t launch_grouped(const DenseArgs& a, DenseWorkspace& ws, DenseParams p, cudaStream_t s) {
+    const ExpertPlan& g = *a.plan;
+    const DenseWeight& w = *a.w;
+    const int room = p.mt * g.most_tiles;
+    p.nt = 1;
+    p.shares = choose_shares(p, ws, g.tile_rows, p.mt * std::min(g.most_tiles, std::min(w.batch, g.most_rows)), room);
+    p.items = room * p.shares;
+    const CUtensorMap* tx = nullptr;
+    LC_TRY(map_of(ws, {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_rows, 1, 4},
+                  [&](void* b) { return make_bf16_tmap_rows(b, a.x, (uint64_t)w.k, (uint64_t)a.x_rows, (uint64_t)a.ldx); }, &tx));
+    switch (g.tile_rows) {
+        case 16: return launch_umma<16, true>(a, *tx, p, s);
+        case 32: return launch_umma<32, true>(a, *tx, p, s);
+        case 64: return launch_umma<64, true>(a, *tx, p, s);
+        case 128: return launch_umma<128, true>(a, *tx, p, s);
+        default: return launch_umma<256, true>(a, *tx, p, s);
+    }
+}
+}  // namespace
+
 int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     if (a.T <= 0) return LC_OK;
     const DenseWeight& w = *a.w;
@@ -387,6 +531,9 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     p.n = w.n; p.T = a.T; p.ldo = a.ldo; p.batch = w.batch;
     p.out_f32 = a.out_f32 || a.f32; p.epi = a.epi; p.e_div = a.e_div; p.scale = a.scale; p.cap = a.cap;
     p.error_flag = gemv_error_flag_dev();
+    p.out2 = a.out2; p.ldo2 = a.ldo2; p.split = a.split;
+    if (a.plan) { p.tiles = a.plan->tiles; p.n_tiles = a.plan->n_tiles; p.off = a.plan->off; p.lists = a.gather ? a.plan->lists : nullptr; p.list_stride = a.plan->list_stride; }
+    LC_CHECK((a.epi != DENSE_GATED_SILU || w.n % 2 == 0) && (a.epi != DENSE_SPLIT_RELU2 || (a.split % 32 == 0 && w.batch == 1)), LC_ERR_INVALID, "dense product: epilogue layout");
     LC_CHECK(a.f32 ? w.data != nullptr : w.tiles != nullptr, LC_ERR_STATE, "dense product: the weight is not in the form this product reads");
     if (a.f32) {
         LC_CUDA(launch_pdl(dense_f32_kernel, dim3((unsigned)((w.n + 63) / 64), (unsigned)((a.T + 63) / 64), (unsigned)w.batch), dim3(256), 0, s, w.data,
@@ -396,6 +543,9 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     const int sms = sm_count();
     p.kblocks = (w.k + kKB - 1) / kKB;
     p.mt = (w.n + kM - 1) / kM;
+    p.partial = ws.partial; p.tickets = ws.tickets;
+    LC_CHECK((uintptr_t)a.x % 16 == 0 && a.ldx % 8 == 0 && a.x_batch % 8 == 0 && a.x_rows >= a.T, LC_ERR_INVALID, "dense product: activation layout");
+    if (a.plan) return launch_grouped(a, ws, p, s);
     // tokens per tile: what finishes first at the measured time of one block of k (in hundredths of a microsecond)
     static const struct { int nt, t; } kSizes[] = {{16, 17}, {32, 17}, {64, 19}, {128, 24}, {256, 36}};
     int NT = 16;
@@ -406,40 +556,22 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     }
     p.nt = (a.T + NT - 1) / NT;
     const int cells = p.mt * p.nt * w.batch;
-    p.shares = 1;
-    if (NT <= 64 && cells <= ws.max_tickets) {  // cut k where that evens out the CTAs' work: k blocks of the busiest CTA, plus what an item
-        // and the summing of the shares cost
-        long best = -1;
-        for (int c = 1; c <= std::min(16, p.kblocks / 2); c++) {
-            if ((size_t)cells * c * NT * kM * sizeof(float) > ws.partial_bytes) break;
-            const long waves = ((long)cells * c + sms - 1) / sms;
-            const long cost = waves * (((p.kblocks + c - 1) / c) + 2 + (c > 1 ? NT / 16 : 0)) + (c > 1 ? 3 + c * NT / 32 : 0);
-            if (best < 0 || cost < best) { best = cost; p.shares = c; }
-        }
-    }
+    p.shares = choose_shares(p, ws, NT, cells, cells);
     p.items = cells * p.shares;
-    p.partial = ws.partial; p.tickets = ws.tickets;
-    LC_CHECK((uintptr_t)a.x % 16 == 0 && a.ldx % 8 == 0 && a.x_batch % 8 == 0 && a.x_rows >= a.T, LC_ERR_INVALID, "dense product: activation layout");
     // a single tile of fewer tokens than NT brings only those: what the other rows of the operand hold reaches columns that
     // are never read
     const int box = std::min(NT, a.T);
     p.stage_tx = kABytes + box * kKB * 2;
-    const std::vector<uint64_t> key = {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_batch, (uint64_t)w.batch, (uint64_t)a.x_rows, (uint64_t)box};
-    std::unique_ptr<DenseWorkspace::Map>& mp = ws.maps[key];
-    if (!mp) {
-        mp.reset(new DenseWorkspace::Map);
-        // order (k, matrix, token): a token tile is one box
-        const bool ok = make_bf16_tmap_3d(mp->b, a.x, (uint64_t)w.k, (uint64_t)w.batch, (uint64_t)a.x_rows, w.batch > 1 ? a.x_batch : (uint64_t)a.ldx, (uint64_t)a.ldx, kKB, 1, (uint32_t)box);
-        if (!ok) ws.maps.erase(key);
-        LC_CHECK(ok, LC_ERR_CUDA, "dense product: no tensor map over the activations");
-    }
-    const CUtensorMap& tx = *(const CUtensorMap*)mp->b;
+    const CUtensorMap* tx = nullptr;  // order (k, matrix, token): a token tile is one box
+    LC_TRY(map_of(ws, {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_batch, (uint64_t)w.batch, (uint64_t)a.x_rows, (uint64_t)box}, [&](void* b) {
+        return make_bf16_tmap_3d(b, a.x, (uint64_t)w.k, (uint64_t)w.batch, (uint64_t)a.x_rows, w.batch > 1 ? a.x_batch : (uint64_t)a.ldx, (uint64_t)a.ldx, kKB, 1, (uint32_t)box);
+    }, &tx));
     switch (NT) {
-        case 16: return launch_umma<16>(a, tx, p, s);
-        case 32: return launch_umma<32>(a, tx, p, s);
-        case 64: return launch_umma<64>(a, tx, p, s);
-        case 128: return launch_umma<128>(a, tx, p, s);
-        default: return launch_umma<256>(a, tx, p, s);
+        case 16: return launch_umma<16, false>(a, *tx, p, s);
+        case 32: return launch_umma<32, false>(a, *tx, p, s);
+        case 64: return launch_umma<64, false>(a, *tx, p, s);
+        case 128: return launch_umma<128, false>(a, *tx, p, s);
+        default: return launch_umma<256, false>(a, *tx, p, s);
     }
 }
 

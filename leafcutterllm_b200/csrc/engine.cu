@@ -448,7 +448,7 @@ int32_t forward_tokens(lc_model* lead, int T, int n_last, bool identity_last, in
 
 uint64_t algo_bytes_step(const lc_model* m, const std::vector<int>& ctx_lens) {
     uint64_t b = m->ctr.weight_bytes;  // every matrix and gain once
-    if (m->cfg.n_experts > 0)          // ... but only the experts that received a token (average per layer of the last steps)
+    if (m->d_moe_touched)              // ... but only the experts that received a token (average per layer of the last steps)
         b = b - m->expert_bytes_all + (uint64_t)(m->touched_per_step * (double)m->expert_bytes_each);
     // the embedding table is not streamed: one row per token instead
     if (m->embed) {
@@ -456,8 +456,8 @@ uint64_t algo_bytes_step(const lc_model* m, const std::vector<int>& ctx_lens) {
         if (!tied) b -= m->embed->nbytes;
         b += (uint64_t)ctx_lens.size() * (m->embed->nbytes / std::max<size_t>(m->embed->rows, 1));
     }
-    if (m->stack) {  // latents of the context read, one token's written; recurrent state read and written
-        for (int c : ctx_lens) b += m->stack->cache_bytes_per_token * ((uint64_t)c + 1) + 2 * m->stack->state_bytes_per_seq;
+    if (m->stack) {
+        for (int c : ctx_lens) b += stack_step_bytes(m, c);
         return b;
     }
     uint64_t per_tok = (uint64_t)m->L * 2 * m->nkv * m->hd * m->kv_elt;
@@ -1384,7 +1384,7 @@ static void after_decode_steps(lc_model* m, int n_seqs, const int32_t* seq_ids, 
         unsigned long long t = 0;
         if (cudaMemcpyAsync(&t, m->d_moe_touched, 8, cudaMemcpyDeviceToHost, m->stream) == cudaSuccess &&
             cudaMemsetAsync(m->d_moe_touched, 0, 8, m->stream) == cudaSuccess && cudaStreamSynchronize(m->stream) == cudaSuccess)
-            m->touched_per_step = n_seqs <= kMoeGroupedTokens && m->layers[0].grouped_ok ? (double)t / std::max(steps, 1)
+            m->touched_per_step = m->stack || (n_seqs <= kMoeGroupedTokens && m->layers[0].grouped_ok) ? (double)t / std::max(steps, 1)
                                                                                            : (double)m->L * m->El;
     }
     std::vector<int> ctx;

@@ -1,0 +1,602 @@
+// Attention of query heads over shared key/value heads in a paged cache, under a window with kept first tokens (MaskSpec) and
+// with a sink: exp(sink[head]) joins the softmax denominator, without key or value.
+//   attn_prep_kernel    RMS norm over all of a token's q and over all of its k, rotation of halves, cache append
+//   attn_plain_kernel   any shape, f32 arithmetic throughout; models in true 32-bit
+//   attn_tokens_kernel  few tokens per sequence (decode): the query heads of one kv head of one token are the rows of the
+//                       products; every warp walks key tiles of its own
+//   attn_tiles_kernel   runs of many tokens: 64 consecutive queries of one head over key tiles of 64
+// Both tile kernels walk only tiles that hold a visible key: those of the kept first tokens, then those from the window's
+// lower edge on.  Scores, softmax and sums are f32; the weights enter the second product as two bf16 halves.
+// Cache rows hold the key after norm and rotation, so a layer without projections of its own reads another layer's cache.
+#include <algorithm>
+#include <cmath>
+#include "lc_mixers.h"
+#include "lc_mma.cuh"
+#include "lc_tma.cuh"
+
+namespace lc {
+
+namespace {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+// First key of the window and the number of kept keys before it.
+struct Seen { int lo, keep; };
+__device__ __forceinline__ Seen seen_from(const AttnShape& g, int pos) {
+    Seen s;
+    s.lo = g.window > 0 ? max(0, pos - g.window + 1) : 0;
+    s.keep = min(g.keep_first, s.lo);
+    return s;
+}
+// The tiles of `size` keys that hold a visible key, in order: n_first tiles from the start, then from tile `base` on.
+struct Tiles {
+    int n_first, base, n;
+    __device__ __forceinline__ int at(int i) const { return i < n_first ? i : base + i - n_first; }
+};
+__device__ __forceinline__ Tiles tiles_of(const Seen& s, int last, int size) {
+    Tiles t;
+    t.base = s.lo / size;
+    t.n_first = min((s.keep + size - 1) / size, t.base);
+    t.n = t.n_first + last / size - t.base + 1;
+    return t;
+}
+
+template <typename A> __device__ __forceinline__ void put4(A* p, float4 v);
+template <> __device__ __forceinline__ void put4<float>(float* p, float4 v) { *(float4*)p = v; }
+template <> __device__ __forceinline__ void put4<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
+
+// One CTA per token and share of its elements; VEC = 4: dim, vdim and the rotated half are multiples of four.
+template <typename A, int VEC>
+__global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a) {
+    __shared__ float sh[32], sh2[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const AttnShape& g = a.g;
+    const int t = blockIdx.x, seq = a.tok_seq[t], pos = a.tok_pos[t], nq = g.heads * g.dim, nk = g.kv_heads * g.dim, half = g.rot_dims / 2;
+    const bool own = a.off_k >= 0;
+    const float *q = a.proj + (size_t)t * a.ld_proj, *k = q + (own ? a.off_k : 0), *v = q + a.off_v;
+    const int page = a.page_table[(size_t)seq * a.pages_per_seq + pos / a.page_tokens], slot = pos % a.page_tokens;
+    const float2* tab = a.rot + (size_t)pos * half;
+    auto squares = [&](const float* x, int n) {
+        float ss = 0.0f;
+        if constexpr (VEC == 4) {
+#pragma unroll 4
+            for (int i = threadIdx.x * 4; i < n; i += 1024) {
+                const float4 u = *(const float4*)(x + i);
+                ss = fmaf(u.x, u.x, fmaf(u.y, u.y, fmaf(u.z, u.z, fmaf(u.w, u.w, ss))));
+            }
+        } else {
+            for (int i = threadIdx.x; i < n; i += 256) ss = fmaf(x[i], x[i], ss);
+        }
+        return ss;
+    };
+    float sq = squares(q, nq), sk = own ? squares(k, nk) : 0.0f;
+    sq = block_sum(sq, sh);
+    if (own) sk = block_sum(sk, sh2);
+    const float rq = 1.0f / sqrtf(sq / (float)nq + a.eps), rk = own ? 1.0f / sqrtf(sk / (float)nk + a.eps) : 0.0f;
+    // items of a head: VEC pairs of the rotated part, then VEC elements of the rest
+    const int pairs = half / VEC, per = pairs + (g.dim - g.rot_dims) / VEC, start = blockIdx.y * 256 + threadIdx.x, step = gridDim.y * 256;
+    auto item = [&](const float* x, const float* w, float r, A* dst, int i) {
+        if constexpr (VEC == 4) {
+            auto normed = [&](int c) {
+                const float4 u = *(const float4*)(x + c), b = *(const float4*)(w + c);
+                return make_float4(u.x * r * b.x, u.y * r * b.y, u.z * r * b.z, u.w * r * b.w);
+            };
+            if (i < pairs) {
+                const float4 u = normed(4 * i), z = normed(half + 4 * i), cs0 = *(const float4*)(tab + 4 * i), cs1 = *(const float4*)(tab + 4 * i + 2);
+                put4<A>(dst + 4 * i, make_float4(u.x * cs0.x - z.x * cs0.y, u.y * cs0.z - z.y * cs0.w, u.z * cs1.x - z.z * cs1.y, u.w * cs1.z - z.w * cs1.w));
+                put4<A>(dst + half + 4 * i, make_float4(z.x * cs0.x + u.x * cs0.y, z.y * cs0.z + u.y * cs0.w, z.z * cs1.x + u.z * cs1.y, z.w * cs1.z + u.w * cs1.w));
+            } else {
+                const int c = g.rot_dims + 4 * (i - pairs);
+                put4<A>(dst + c, normed(c));
+            }
+        } else {
+            if (i < pairs) {
+                const float u = x[i] * r * w[i], z = x[half + i] * r * w[half + i];
+                const float2 cs = tab[i];
+                dst[i] = to_act<A>(u * cs.x - z * cs.y);
+                dst[half + i] = to_act<A>(z * cs.x + u * cs.y);
+            } else {
+                const int c = g.rot_dims + i - pairs;
+                dst[c] = to_act<A>(x[c] * r * w[c]);
+            }
+        }
+    };
+    A* qo = (A*)a.q + (size_t)t * g.heads * g.dp;
+    for (int i = start; i < g.heads * per; i += step) {
+        const int h = i / per;
+        item(q + h * g.dim, a.q_norm + h * g.dim, rq, qo + h * g.dp, i - h * per);
+    }
+    if (!own) return;
+    const size_t row0 = (size_t)page * g.kv_heads * a.page_tokens + slot;
+    for (int i = start; i < g.kv_heads * per; i += step) {
+        const int h = i / per;
+        item(k + h * g.dim, a.k_norm + h * g.dim, rk, (A*)a.k_cache + (row0 + (size_t)h * a.page_tokens) * g.dp, i - h * per);
+    }
+    const int vper = g.vdim / VEC;
+    for (int i = start; i < g.kv_heads * vper; i += step) {
+        const int h = i / vper, c = (i - h * vper) * VEC;
+        A* dst = (A*)a.v_cache + (row0 + (size_t)h * a.page_tokens) * g.ep + c;
+        if constexpr (VEC == 4) put4<A>(dst, *(const float4*)(v + h * g.vdim + c));
+        else dst[0] = to_act<A>(v[h * g.vdim + c]);
+    }
+}
+
+// One CTA per (head, token), a key per thread.
+constexpr int kPlainThreads = 128;
+template <typename A>
+__global__ void __launch_bounds__(kPlainThreads) attn_plain_kernel(const AttnArgs a) {
+    extern __shared__ float smf[];
+    __shared__ float red[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const AttnShape& g = a.g;
+    const int h = blockIdx.x, t = blockIdx.y, seq = a.tok_seq[t], pos = a.tok_pos[t], kvh = h / (g.heads / g.kv_heads);
+    float *s_q = smf, *s_o = s_q + g.dim, *s_p = s_o + g.vdim;
+    size_t* s_row = (size_t*)(s_p + kPlainThreads + ((g.dim + g.vdim) & 1));
+    const A* q = (const A*)a.q + ((size_t)t * g.heads + h) * g.dp;
+    for (int i = threadIdx.x; i < g.dim; i += kPlainThreads) s_q[i] = act_f<A>(q[i]);
+    for (int i = threadIdx.x; i < g.vdim; i += kPlainThreads) s_o[i] = 0.0f;
+    __syncthreads();
+    const int32_t* pt = a.page_table + (size_t)seq * a.pages_per_seq;
+    const Seen sn = seen_from(g, pos);
+    const int n = sn.keep + pos - sn.lo + 1;  // visible keys: the kept ones, then the window
+    float m = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.0f : 0.0f;
+    for (int k0 = 0; k0 < n; k0 += kPlainThreads) {
+        const int i = k0 + threadIdx.x, key = i < sn.keep ? i : sn.lo + i - sn.keep;
+        float sc = -INFINITY;
+        if (i < n) {
+            const size_t row = ((size_t)pt[key / a.page_tokens] * g.kv_heads + kvh) * a.page_tokens + key % a.page_tokens;
+            s_row[threadIdx.x] = row;
+            const A* kr = (const A*)a.k_cache + row * g.dp;
+            float d = 0.0f;
+            for (int c = 0; c < g.dim; c++) d = fmaf(s_q[c], act_f<A>(kr[c]), d);
+            sc = d * g.scale;
+        }
+        const float mt = fmaxf(m, block_max(sc, red));
+        const float p = i < n ? expf(sc - mt) : 0.0f, corr = expf(m - mt);
+        s_p[threadIdx.x] = p;
+        l = l * corr + block_sum(p, red);
+        m = mt;
+        const int nk = min(kPlainThreads, n - k0);
+        for (int c = threadIdx.x; c < g.vdim; c += kPlainThreads) {
+            float o = s_o[c] * corr;
+            for (int j = 0; j < nk; j++) o = fmaf(s_p[j], act_f<A>(((const A*)a.v_cache)[s_row[j] * g.ep + c]), o);
+            s_o[c] = o;
+        }
+        __syncthreads();
+    }
+    A* out = (A*)a.out + (size_t)t * a.ldo + (size_t)h * g.ep;
+    for (int c = threadIdx.x; c < g.ep; c += kPlainThreads) out[c] = to_act<A>(c < g.vdim ? s_o[c] / l : 0.0f);
+}
+
+// ---- few tokens per sequence ------------------------------------------------------------------------------------------------
+// A CTA of four warps takes up to 16 query heads of one kv head of one token and a piece of its key tiles (16 keys each); the
+// warps deal the tiles among themselves, each with its own ring of copies in flight and its own running softmax, and meet at
+// the end.  Several pieces: the CTA that finishes last merges them.
+constexpr int kDecKeys = 16, kDecStages = 3, kDecWarps = 4, kMaxPieces = 32;
+struct AttnParts { float *o, *ml; unsigned* tickets; };  // [token][kv head][row block][piece][16][ep], [..][16][2] (log2 units)
+
+template <int NV>
+__global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnArgs a, const AttnParts pt_out) {
+    extern __shared__ __align__(128) unsigned char smem[];
+    __shared__ float s_ml[kDecWarps][16][2], s_scale[kMaxPieces][16];
+    __shared__ int s_last;
+    const AttnShape& g = a.g;
+    const int d16 = (g.dp + 15) & ~15, kp = d16 + 8, rb = kp * 2;
+    constexpr int vp = NV * 8 + 8, vb = vp * 2;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+    const int rep = g.heads / g.kv_heads, blocks = (rep + 15) / 16, t = blockIdx.x, kvh = blockIdx.y / blocks, r0 = (blockIdx.y % blocks) * 16, nh = min(16, rep - r0),
+              h0 = kvh * rep + r0, pieces = gridDim.z;
+    bf16 *s_q = (bf16*)smem, *s_k = s_q + 16 * kp + (size_t)warp * kDecStages * kDecKeys * (kp + vp), *s_v = s_k + kDecStages * kDecKeys * kp;
+    pdl_launch_dependents();
+    const bf16 zero = __float2bfloat16_rn(0.0f);
+    for (int i = lane; i < kDecStages * kDecKeys * (d16 - g.dp); i += 32) s_k[(i / (d16 - g.dp)) * kp + g.dp + i % (d16 - g.dp)] = zero;
+    pdl_wait();
+    const int seq = a.tok_seq[t], pos = a.tok_pos[t];
+    const Seen sn = seen_from(g, pos);
+    const Tiles tl = tiles_of(sn, pos, kDecKeys);
+    const int per = (tl.n + pieces - 1) / pieces, i0 = blockIdx.z * per, i1 = min(tl.n, i0 + per), mine = i1 > i0 + warp ? (i1 - i0 - warp + kDecWarps - 1) / kDecWarps : 0;
+    const int32_t* pt = a.page_table + (size_t)seq * a.pages_per_seq;
+    const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), v_sm = smem_u32(s_v);
+    const int kch = g.dp / 8, vch = g.ep / 8;
+    auto load = [&](int j) {
+        if (j < mine) {
+            const int tile = tl.at(i0 + warp + j * kDecWarps), key = min(tile * kDecKeys + (lane & 15), pos), st = j % kDecStages;
+            const int row = (pt[key / a.page_tokens] * g.kv_heads + kvh) * a.page_tokens + key % a.page_tokens;
+#pragma unroll
+            for (int p = 0; p < 4; p++) {
+                const int ki = p * 4 + (lane >> 3);
+                const size_t r = (size_t)__shfl_sync(0xffffffffu, row, ki);
+                const bf16 *ks = (const bf16*)a.k_cache + r * g.dp, *vs = (const bf16*)a.v_cache + r * g.ep;
+                const uint32_t kd = k_sm + (uint32_t)((st * kDecKeys + ki) * rb), vd = v_sm + (uint32_t)((st * kDecKeys + ki) * vb);
+                for (int c = lane & 7; c < kch; c += 8) cp16(kd + c * 16, ks + c * 8, 16);
+                for (int c = lane & 7; c < vch; c += 8) cp16(vd + c * 16, vs + c * 8, 16);
+            }
+        }
+        cp_commit();
+    };
+    load(0);
+    load(1);
+    for (int i = tid; i < 16 * (d16 / 8); i += 32 * kDecWarps) {
+        const int r = i / (d16 / 8), c = (i - r * (d16 / 8)) * 8;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (r < nh && c < g.dp) v = *(const uint4*)((const bf16*)a.q + ((size_t)t * g.heads + h0 + r) * g.dp + c);
+        *(uint4*)(s_q + r * kp + c) = v;
+    }
+    __syncthreads();
+    float o[NV][4], m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int i = 0; i < NV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    const float sc = g.scale * kLog2e;
+    const uint32_t qa = q_sm + (uint32_t)((lane & 15) * rb + (lane >> 4) * 16);
+    for (int j = 0; j < mine; j++) {
+        load(j + 2);
+        cp_wait<2>();
+        __syncwarp();
+        const int st = j % kDecStages, key0 = tl.at(i0 + warp + j * kDecWarps) * kDecKeys;
+        float s[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+        const uint32_t ka = k_sm + (uint32_t)((st * kDecKeys + (lane & 7) + ((lane >> 4) << 3)) * rb + ((lane >> 3) & 1) * 16);
+#pragma unroll 4
+        for (int k = 0; k < d16 / 16; k++) {
+            uint32_t q4[4], kb[4];
+            ldsm4(qa + k * 32, q4);
+            ldsm4(ka + k * 32, kb);
+            mma_bf16(s[0], q4, kb[0], kb[1]);
+            mma_bf16(s[1], q4, kb[2], kb[3]);
+        }
+        float mx[2] = {m_run[0], m_run[1]};
+#pragma unroll
+        for (int i = 0; i < 2; i++)
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+                const int key = key0 + 8 * i + 2 * t4 + (e & 1);
+                s[i][e] = key <= pos && (key >= sn.lo || key < sn.keep) ? s[i][e] * sc : -INFINITY;
+                mx[e >> 1] = fmaxf(mx[e >> 1], s[i][e]);
+            }
+        float corr[2], sum[2] = {0.0f, 0.0f};
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+            mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));  // finite: every tile holds a visible key
+            corr[r] = exp2f(m_run[r] - mx[r]);
+            m_run[r] = mx[r];
+        }
+        uint32_t ph[4], pl[4];
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            float p[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) { p[e] = exp2f(s[i][e] - m_run[e >> 1]); sum[e >> 1] += p[e]; }
+            split2(p[0], p[1], ph[2 * i], pl[2 * i]);
+            split2(p[2], p[3], ph[2 * i + 1], pl[2 * i + 1]);
+        }
+#pragma unroll
+        for (int r = 0; r < 2; r++) l_run[r] = l_run[r] * corr[r] + sum[r];  // this lane's share of the row
+#pragma unroll
+        for (int i = 0; i < NV; i++) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+        const uint32_t va = v_sm + (uint32_t)((st * kDecKeys + (lane & 15)) * vb + (lane >> 4) * 16);
+#pragma unroll
+        for (int np = 0; np < NV / 2; np++) {
+            if (16 * np >= g.ep) break;
+            uint32_t b[4];
+            ldsm4t(va + np * 32, b);
+            mma_bf16(o[2 * np], ph, b[0], b[1]);
+            mma_bf16(o[2 * np + 1], ph, b[2], b[3]);
+            mma_bf16(o[2 * np], pl, b[0], b[1]);
+            mma_bf16(o[2 * np + 1], pl, b[2], b[3]);
+        }
+        __syncwarp();
+    }
+    cp_wait<0>();
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
+        l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
+    }
+    __syncthreads();  // the copies' buffers become the warps' sums: [warp][16][ep]
+    float* s_o = (float*)(s_q + 16 * kp);
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        const int row = g8 + 8 * r;
+        if (row < nh) {
+            if (t4 == 0) { s_ml[warp][row][0] = m_run[r]; s_ml[warp][row][1] = l_run[r]; }
+#pragma unroll
+            for (int i = 0; i < NV; i++)
+                if (8 * i < g.ep) *(float2*)(s_o + ((size_t)warp * 16 + row) * g.ep + 8 * i + 2 * t4) = make_float2(o[i][2 * r], o[i][2 * r + 1]);
+        }
+    }
+    __syncthreads();
+    auto sink_of = [&](int row) { return a.sink ? a.sink[h0 + row] * kLog2e : -INFINITY; };
+    if (tid < nh) {  // the warps' factors; with one piece also the sink and the division
+        float m = pieces == 1 ? sink_of(tid) : -INFINITY;
+        for (int w = 0; w < kDecWarps; w++) m = fmaxf(m, s_ml[w][tid][0]);
+        float l = pieces == 1 && a.sink ? exp2f(sink_of(tid) - m) : 0.0f, f[kDecWarps];
+        for (int w = 0; w < kDecWarps; w++) {
+            f[w] = m == -INFINITY ? 0.0f : exp2f(s_ml[w][tid][0] - m);
+            l += f[w] * s_ml[w][tid][1];
+        }
+        for (int w = 0; w < kDecWarps; w++) s_scale[w][tid] = pieces == 1 ? f[w] / l : f[w];
+        if (pieces > 1) {
+            float* ml = pt_out.ml + ((((size_t)t * gridDim.y + blockIdx.y) * pieces + blockIdx.z) * 16 + tid) * 2;
+            ml[0] = m; ml[1] = l;
+        }
+    }
+    __syncthreads();
+    const int vec = g.ep / 4;
+    const size_t cell = (size_t)t * gridDim.y + blockIdx.y;
+    for (int i = tid; i < nh * vec; i += 32 * kDecWarps) {
+        const int row = i / vec, c = (i - row * vec) * 4;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int w = 0; w < kDecWarps; w++) {
+            const float f = s_scale[w][row];
+            const float4 v = *(const float4*)(s_o + ((size_t)w * 16 + row) * g.ep + c);
+            x.x = fmaf(f, v.x, x.x); x.y = fmaf(f, v.y, x.y); x.z = fmaf(f, v.z, x.z); x.w = fmaf(f, v.w, x.w);
+        }
+        if (pieces == 1) put4<bf16>((bf16*)a.out + (size_t)t * a.ldo + (size_t)(h0 + row) * g.ep + c, x);
+        else *(float4*)(pt_out.o + ((cell * pieces + blockIdx.z) * 16 + row) * g.ep + c) = x;
+    }
+    if (pieces == 1) return;
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) {
+        s_last = atomicAdd(pt_out.tickets + cell, 1u) == (unsigned)pieces - 1;
+        if (s_last) pt_out.tickets[cell] = 0;
+        __threadfence();
+    }
+    __syncthreads();
+    if (!s_last) return;
+    for (int row = warp; row < nh; row += kDecWarps) {  // a lane per piece
+        const float* ml = pt_out.ml + ((cell * pieces + min(lane, pieces - 1)) * 16 + row) * 2;
+        const float pm = lane < pieces ? __ldcg(ml) : -INFINITY, pl = lane < pieces ? __ldcg(ml + 1) : 0.0f, sk = sink_of(row), m = fmaxf(warp_max(pm), sk);
+        const float f = pm == -INFINITY ? 0.0f : exp2f(pm - m), l = warp_sum(f * pl) + (a.sink ? exp2f(sk - m) : 0.0f);
+        if (lane < pieces) s_scale[lane][row] = f / l;
+    }
+    __syncthreads();
+    for (int i = tid; i < nh * vec; i += 32 * kDecWarps) {
+        const int row = i / vec, c = (i - row * vec) * 4;
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        const float* src = pt_out.o + (cell * pieces * 16 + row) * g.ep + c;
+#pragma unroll 8
+        for (int p = 0; p < pieces; p++) {
+            const float f = s_scale[p][row];
+            const float4 v = __ldcg((const float4*)(src + (size_t)p * 16 * g.ep));
+            x.x = fmaf(f, v.x, x.x); x.y = fmaf(f, v.y, x.y); x.z = fmaf(f, v.z, x.z); x.w = fmaf(f, v.w, x.w);
+        }
+        put4<bf16>((bf16*)a.out + (size_t)t * a.ldo + (size_t)(h0 + row) * g.ep + c, x);
+    }
+}
+
+// ---- runs of many tokens ----------------------------------------------------------------------------------------------------
+constexpr int kKeys = 64;
+template <int NV>
+__global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const AttnTile* __restrict__ tiles) {
+    extern __shared__ __align__(128) unsigned char smem[];
+    const AttnShape& g = a.g;
+    const int d16 = (g.dp + 15) & ~15, kp = d16 + 8, rb = kp * 2;
+    constexpr int vp = NV * 8 + 8, vb = vp * 2;
+    bf16 *s_q = (bf16*)smem, *s_k = s_q + 64 * kp, *s_v = s_k + 2 * kKeys * kp;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+    pdl_launch_dependents();
+    const bf16 zero = __float2bfloat16_rn(0.0f);
+    for (int i = tid; i < 2 * kKeys * (d16 - g.dp); i += 128) s_k[(i / (d16 - g.dp)) * kp + g.dp + i % (d16 - g.dp)] = zero;
+    pdl_wait();
+    const AttnTile tl = tiles[gridDim.x - 1 - blockIdx.x];  // the tiles with the longest contexts first
+    const int h = blockIdx.y, kvh = h / (g.heads / g.kv_heads), last = tl.pos0 + tl.n - 1;
+    const Seen sn = seen_from(g, tl.pos0);  // of the first query: no other sees an earlier window
+    Tiles kt = tiles_of(sn, last, kKeys);
+    kt.n_first = min((g.keep_first + kKeys - 1) / kKeys, kt.base);
+    kt.n = kt.n_first + last / kKeys - kt.base + 1;
+    const int32_t* pt = a.page_table + (size_t)tl.seq * a.pages_per_seq;
+    const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), v_sm = smem_u32(s_v);
+    const int kch = g.dp / 8, vch = g.ep / 8;
+    auto load = [&](int tile, int buf) {
+#pragma unroll
+        for (int p = 0; p < 4; p++) {
+            const int ki = p * 16 + (tid >> 3), key = min(tile * kKeys + ki, last);
+            const size_t r = ((size_t)pt[key / a.page_tokens] * g.kv_heads + kvh) * a.page_tokens + key % a.page_tokens;
+            const bf16 *ks = (const bf16*)a.k_cache + r * g.dp, *vs = (const bf16*)a.v_cache + r * g.ep;
+            const uint32_t kd = k_sm + (uint32_t)((buf * kKeys + ki) * rb), vd = v_sm + (uint32_t)((buf * kKeys + ki) * vb);
+            for (int c = tid & 7; c < kch; c += 8) cp16(kd + c * 16, ks + c * 8, 16);
+            for (int c = tid & 7; c < vch; c += 8) cp16(vd + c * 16, vs + c * 8, 16);
+        }
+        cp_commit();
+    };
+    load(kt.at(0), 0);
+    for (int i = tid; i < 64 * (d16 / 8); i += 128) {
+        const int r = i / (d16 / 8), c = (i - r * (d16 / 8)) * 8;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (r < tl.n && c < g.dp) v = *(const uint4*)((const bf16*)a.q + ((size_t)(tl.tok0 + r) * g.heads + h) * g.dp + c);
+        *(uint4*)(s_q + r * kp + c) = v;
+    }
+    float o[NV][4], m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int i = 0; i < NV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
+    const float sc = g.scale * kLog2e;
+    const int q0 = warp * 16, pa = tl.pos0 + q0, pb = min(pa + 15, last), qpos[2] = {pa + g8, pa + g8 + 8};
+    const int wlo_a = g.window > 0 ? max(0, pa - g.window + 1) : 0, wlo_b = g.window > 0 ? max(0, pb - g.window + 1) : 0;
+    const int qlo[2] = {g.window > 0 ? qpos[0] - g.window + 1 : 0, g.window > 0 ? qpos[1] - g.window + 1 : 0};
+    for (int i = 0; i < kt.n; i++) {
+        const int buf = i & 1, key0 = kt.at(i) * kKeys;
+        if (i + 1 < kt.n) { load(kt.at(i + 1), buf ^ 1); cp_wait<1>(); }
+        else cp_wait<0>();
+        __syncthreads();
+        if (q0 < tl.n && key0 <= pb && (key0 + kKeys > wlo_a || key0 < g.keep_first)) {
+            float s[8][4];
+#pragma unroll
+            for (int n = 0; n < 8; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.0f;
+            const uint32_t qa = q_sm + (uint32_t)((q0 + (lane & 15)) * rb + (lane >> 4) * 16),
+                           ka = k_sm + (uint32_t)((buf * kKeys + (lane & 7) + ((lane >> 4) << 3)) * rb + ((lane >> 3) & 1) * 16);
+#pragma unroll 2
+            for (int k = 0; k < d16 / 16; k++) {
+                uint32_t q4[4];
+                ldsm4(qa + k * 32, q4);
+#pragma unroll
+                for (int n = 0; n < 4; n++) {
+                    uint32_t kb[4];
+                    ldsm4(ka + (uint32_t)(16 * n * rb) + k * 32, kb);
+                    mma_bf16(s[2 * n], q4, kb[0], kb[1]);
+                    mma_bf16(s[2 * n + 1], q4, kb[2], kb[3]);
+                }
+            }
+            const bool edge = key0 + kKeys - 1 > pa || key0 < wlo_b;
+            float mx[2] = {m_run[0], m_run[1]}, base[2], corr[2], sum[2] = {0.0f, 0.0f};
+#pragma unroll
+            for (int n = 0; n < 8; n++)
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    float v = s[n][e] * sc;
+                    if (edge) {
+                        const int key = key0 + 8 * n + 2 * t4 + (e & 1), r = e >> 1;
+                        if (key > qpos[r] || (key < qlo[r] && key >= g.keep_first)) v = -INFINITY;
+                    }
+                    s[n][e] = v;
+                    mx[e >> 1] = fmaxf(mx[e >> 1], v);
+                }
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+                base[r] = mx[r] == -INFINITY ? 0.0f : mx[r];  // a query whose window starts behind this tile has seen no key yet
+                corr[r] = exp2f(m_run[r] - base[r]);
+                m_run[r] = mx[r];
+            }
+            uint32_t ph[4][4], pl[4][4];
+#pragma unroll
+            for (int n = 0; n < 8; n++) {
+                float p[4];
+#pragma unroll
+                for (int e = 0; e < 4; e++) { p[e] = exp2f(s[n][e] - base[e >> 1]); sum[e >> 1] += p[e]; }
+                const int ks = n >> 1, hs = (n & 1) * 2;
+                split2(p[0], p[1], ph[ks][hs], pl[ks][hs]);
+                split2(p[2], p[3], ph[ks][hs + 1], pl[ks][hs + 1]);
+            }
+#pragma unroll
+            for (int r = 0; r < 2; r++) l_run[r] = l_run[r] * corr[r] + sum[r];  // this lane's share of the row
+#pragma unroll
+            for (int n = 0; n < NV; n++) { o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1]; }
+            const uint32_t va = v_sm + (uint32_t)((buf * kKeys + (lane & 15)) * vb + (lane >> 4) * 16);
+#pragma unroll
+            for (int ks = 0; ks < 4; ks++)
+#pragma unroll
+                for (int np = 0; np < NV / 2; np++) {
+                    if (16 * np >= g.ep) break;
+                    uint32_t b[4];
+                    ldsm4t(va + (uint32_t)(16 * ks * vb) + np * 32, b);
+                    mma_bf16(o[2 * np], ph[ks], b[0], b[1]);
+                    mma_bf16(o[2 * np + 1], ph[ks], b[2], b[3]);
+                    mma_bf16(o[2 * np], pl[ks], b[0], b[1]);
+                    mma_bf16(o[2 * np + 1], pl[ks], b[2], b[3]);
+                }
+        }
+        __syncthreads();
+    }
+    const float sink = a.sink ? a.sink[h] * kLog2e : -INFINITY;
+#pragma unroll
+    for (int r = 0; r < 2; r++) {
+        const int row = q0 + g8 + 8 * r;
+        l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
+        l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
+        if (row >= tl.n) continue;
+        const float m = fmaxf(m_run[r], sink), f = exp2f(m_run[r] - m), inv = f / (l_run[r] * f + (a.sink ? exp2f(sink - m) : 0.0f));
+        bf16* dst = (bf16*)a.out + (size_t)(tl.tok0 + row) * a.ldo + (size_t)h * g.ep + 2 * t4;
+#pragma unroll
+        for (int n = 0; n < NV; n++)
+            if (8 * n < g.ep) *(uint32_t*)(dst + 8 * n) = pack2(o[n][2 * r] * inv, o[n][2 * r + 1] * inv);
+    }
+}
+
+int value_tiles(int ep) { return ep <= 32 ? 4 : ep <= 64 ? 8 : ep <= 96 ? 12 : ep <= 128 ? 16 : 32; }
+size_t tokens_smem(const AttnShape& g) {
+    const size_t kp = ((g.dp + 15) & ~15) + 8, vp = value_tiles(g.ep) * 8 + 8;
+    return (16 * kp + (size_t)kDecWarps * std::max((size_t)kDecStages * kDecKeys * (kp + vp), (size_t)16 * g.ep * 2)) * 2;
+}
+size_t tiles_smem(const AttnShape& g) {
+    const size_t kp = ((g.dp + 15) & ~15) + 8, vp = value_tiles(g.ep) * 8 + 8;
+    return (64 * kp + 2 * kKeys * (kp + vp)) * 2;
+}
+bool tensor_form(const AttnShape& g, bool f32) { return !f32 && g.ep <= 256 && tokens_smem(g) <= kMaxSmem - 4096 && tiles_smem(g) <= kMaxSmem; }
+int cells(const AttnShape& g) { return g.kv_heads * ((g.heads / g.kv_heads + 15) / 16); }
+
+}  // namespace
+
+int32_t launch_attn_prep(const AttnArgs& a, cudaStream_t s) {
+    const AttnShape& g = a.g;
+    const bool vec = g.dim % 4 == 0 && g.vdim % 4 == 0 && g.rot_dims % 8 == 0;
+    // few tokens: several CTAs each, all of which sum the whole rows
+    const dim3 grid((unsigned)a.T, (unsigned)(a.T < 32 ? std::max(1, std::min(8, (g.heads + g.kv_heads) * g.dim / 1024)) : 1));
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(launch_pdl(kern, grid, dim3(256), 0, s, a));
+        return LC_OK;
+    };
+    if (a.f32) return vec ? go(attn_prep_kernel<float, 4>) : go(attn_prep_kernel<float, 1>);
+    return vec ? go(attn_prep_kernel<bf16, 4>) : go(attn_prep_kernel<bf16, 1>);
+}
+
+size_t attn_part_bytes(const AttnShape& g) {
+    // pieces are only cut while all CTAs stay within two per SM
+    return (size_t)2 * sm_count() * 16 * ((size_t)g.ep + 2) * sizeof(float);
+}
+
+int32_t launch_attn_tokens(const AttnArgs& a, const AttnScratch& sc, cudaStream_t s) {
+    const AttnShape& g = a.g;
+    if (a.T <= 0) return LC_OK;
+    if (!tensor_form(g, a.f32)) {
+        const size_t smem = (size_t)(g.dim + g.vdim + 2 + kPlainThreads) * 4 + kPlainThreads * sizeof(size_t);
+        LC_CHECK(smem <= kMaxSmem, LC_ERR_UNSUPPORTED, "attention: heads of %d and %d dimensions", g.dim, g.vdim);
+        const dim3 grid((unsigned)g.heads, (unsigned)a.T);
+        auto go = [&](auto kern) -> int32_t {
+            LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+            LC_CUDA(launch_pdl(kern, grid, dim3(kPlainThreads), smem, s, a));
+            return LC_OK;
+        };
+        return a.f32 ? go(attn_plain_kernel<float>) : go(attn_plain_kernel<bf16>);
+    }
+    const int n = cells(g), cap = a.pages_per_seq * a.page_tokens;
+    const int span = g.window > 0 ? std::min(cap, g.window) / kDecKeys + 2 + std::min(cap, g.keep_first) / kDecKeys : (cap + kDecKeys - 1) / kDecKeys;  // most tiles of a token
+    int pieces = std::max(1, std::min(std::min(kMaxPieces, 2 * sm_count() / (a.T * n)), (span + kDecWarps - 1) / kDecWarps));
+    if (a.T * n > sc.n_tickets) pieces = 1;
+    while (pieces > 1 && (size_t)a.T * n * pieces * 16 * ((size_t)g.ep + 2) * sizeof(float) > sc.part_bytes) pieces--;
+    AttnParts p;
+    p.o = sc.part;
+    p.ml = sc.part + (size_t)a.T * n * pieces * 16 * g.ep;
+    p.tickets = sc.tickets;
+    const size_t smem = tokens_smem(g);
+    const dim3 grid((unsigned)a.T, (unsigned)n, (unsigned)pieces);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+        LC_CUDA(launch_pdl(kern, grid, dim3(32 * kDecWarps), smem, s, a, p));
+        return LC_OK;
+    };
+    switch (value_tiles(g.ep)) {
+        case 4: return go(attn_tokens_kernel<4>);
+        case 8: return go(attn_tokens_kernel<8>);
+        case 12: return go(attn_tokens_kernel<12>);
+        case 16: return go(attn_tokens_kernel<16>);
+        default: return go(attn_tokens_kernel<32>);
+    }
+}
+
+bool attn_tiles_apply(const AttnShape& g, bool f32) { return tensor_form(g, f32); }
+
+int32_t launch_attn_tiles(const AttnArgs& a, const AttnTile* tiles, int n_tiles, cudaStream_t s) {
+    const size_t smem = tiles_smem(a.g);
+    const dim3 grid((unsigned)n_tiles, (unsigned)a.g.heads);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+        LC_CUDA(launch_pdl(kern, grid, dim3(128), smem, s, a, tiles));
+        return LC_OK;
+    };
+    switch (value_tiles(a.g.ep)) {
+        case 4: return go(attn_tiles_kernel<4>);
+        case 8: return go(attn_tiles_kernel<8>);
+        case 12: return go(attn_tiles_kernel<12>);
+        case 16: return go(attn_tiles_kernel<16>);
+        default: return go(attn_tiles_kernel<32>);
+    }
+}
+
+}  // namespace lc

@@ -7,19 +7,13 @@
 #include <algorithm>
 #include <cmath>
 #include "lc_mixers.h"
+#include "lc_mma.cuh"
 #include "lc_tma.cuh"
 #include "lc_umma.cuh"
 
 namespace lc {
 
 namespace {
-
-template <typename A> __device__ __forceinline__ float act_f(A v);
-template <> __device__ __forceinline__ float act_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float act_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-template <typename A> __device__ __forceinline__ A to_act(float v);
-template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 to_act<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
 // Any shape, any type, f32 arithmetic throughout: one CTA per (token, head), keys in tiles of one per thread.
 constexpr int kPlainThreads = 128;
@@ -78,30 +72,6 @@ __global__ void __launch_bounds__(kPlainThreads) latent_attention_plain_kernel(c
 }
 
 // ---- tensor-core forms (bf16) -------------------------------------------------------------------------------------------
-typedef __nv_bfloat16 bf16;
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src, int src_bytes) {  // src_bytes 0: zeros
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(src_bytes) : "memory");
-}
-__device__ __forceinline__ uint32_t pack2(float a, float b) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t*>(&h);
-}
-// (a, b) as a bf16 pair and the pair of what that rounding lost: the weights keep 16 bits of mantissa in the two products
-__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    hi = *reinterpret_cast<const uint32_t*>(&h);
-    lo = pack2(a - __low2float(h), b - __high2float(h));
-}
 // element i of a rotated part whose row starts at r
 __device__ __forceinline__ float rotated(const bf16* r, const float2* tab, int pairs, int n, int i) {
     if (i >= n) return 0.0f;

@@ -4,8 +4,13 @@
 //                    vectors -> recurrence -> per-head norm and gate -> out
 //   LatentAttention  in = dq | dkv (one product)  ->  latent norms, key rotation, cache append  ->  uq -> (per head) uk^T
 //                    -> attention over the latents -> (per head) uv -> out
+//   Attention        in = q | k | v (one product)  ->  norms over all heads, rotation, cache append  ->  attention -> out
 //   Relu2            up (squared relu in its epilogue) -> down
-// each followed by x += rms_norm(y) w, which also writes the activations the next product reads.
+//   GatedSilu        gate and up rows in turn (one product, silu(gate) * up in its epilogue) -> down
+//   Moe              router | shared gate | shared up (one product) -> choice, token lists -> experts' up, experts' down
+//                    (grouped products), shared down
+// each followed by x += rms_norm(y) w (for Moe on the weighted sum of the experts' rows), which also writes the activations the
+// next product reads: the sum, or its norm where the design has norms on inputs.
 #include <cmath>
 #include <cstring>
 #include "lc_model.h"
@@ -90,9 +95,14 @@ int32_t plain_weight(lc_model* m, const std::string& name, int n, int k, DenseWe
 }
 
 // Several matrices over the same input as one, each part's rows starting at a multiple of eight; `offs` receives the starts.
-int32_t fused_weight(lc_model* m, const std::vector<std::string>& names, const std::vector<int>& rows, int k, DenseWeight* w, std::vector<int>* offs) {
+// The last part starts at a multiple of `last_align`.
+int32_t fused_weight(lc_model* m, const std::vector<std::string>& names, const std::vector<int>& rows, int k, DenseWeight* w, std::vector<int>* offs, int last_align = 8) {
     int total = 0;
-    for (int r : rows) { offs->push_back(total); total += round8(r); }
+    for (size_t i = 0; i < rows.size(); i++) {
+        if (i + 1 == rows.size()) total = (total + last_align - 1) / last_align * last_align;
+        offs->push_back(total);
+        total += round8(rows[i]);
+    }
     const int ld = round8(k);
     void* p = nullptr;
     LC_TRY(talloc(*m->stack, &p, (size_t)total * ld * 2));
@@ -236,6 +246,81 @@ int32_t bind_latent(lc_model* m, StackLayer& L, const std::string& p) {
     return rot_table(m, s.rot, &L.rot);
 }
 
+int32_t bind_attention(lc_model* m, StackLayer& L, const std::string& p) {
+    LayerStack& st = *m->stack;
+    const LayerSpec& s = L.s;
+    const int W = st.spec.width, nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
+    AttnShape& g = L.ag;
+    g.heads = s.heads; g.kv_heads = s.kv_heads; g.dim = s.dim; g.vdim = s.vdim; g.dp = round8(s.dim); g.ep = round8(s.vdim); g.rot_dims = s.rot.dims;
+    g.scale = s.scale; g.window = s.mask.size; g.keep_first = s.mask.keep_first;
+    L.ep = g.ep;
+    std::vector<int> offs;
+    if (s.kv_from < 0) {
+        LC_TRY(fused_weight(m, {p + "q", p + "k", p + "v"}, {nq, nk, nv}, W, &L.in, &offs));
+        L.off_k = offs[1]; L.off_v = offs[2];
+        LC_TRY(model_gain_f32(m, p + "k.norm", nk, &L.k_norm));
+    } else {
+        LC_TRY(plain_weight(m, p + "q", nq, W, &L.in));
+    }
+    LC_TRY(model_gain_f32(m, p + "q.norm", nq, &L.q_norm));
+    if (m->tensors.count(p + "sink")) LC_TRY(model_gain_f32(m, p + "sink", s.heads, &L.sink));
+    LC_TRY(plain_weight(m, p + "o", W, s.heads * s.vdim, &L.out, PackMap{s.vdim, L.ep, 0, 0}, s.heads * L.ep));
+    return s.rot.dims ? rot_table(m, s.rot, &L.rot) : LC_OK;
+}
+
+// The experts' matrices `which` [n, k] as one batch.
+int32_t expert_weights(lc_model* m, const std::string& p, const char* which, int experts, int n, int k, DenseWeight* w) {
+    const int ld = round8(k);
+    void* d = nullptr;
+    LC_TRY(talloc(*m->stack, &d, (size_t)experts * n * ld * 2));
+    for (int e = 0; e < experts; e++) {
+        DevTensor* t = nullptr;
+        LC_TRY(matrix(m, p + "e" + std::to_string(e) + "." + which, n, k, &t));
+        LC_TRY(launch_pack((const bf16*)t->view, n, k, (bf16*)d + (size_t)e * n * ld, ld, PackMap(), PackMap(), false, m->stream));
+    }
+    return dense_weight_init(w, (const bf16*)d, n, k, ld, experts, (size_t)n * ld);
+}
+
+int32_t bind_ffn(lc_model* m, StackLayer& L, const std::string& p) {
+    LayerStack& st = *m->stack;
+    const LayerSpec& s = L.s;
+    const int W = st.spec.width, ld = round8(W);
+    if (s.ffn == FfnKind::Relu2) {
+        LC_TRY(plain_weight(m, p + "up", s.ff, W, &L.up));
+        return plain_weight(m, p + "down", W, s.ff, &L.down);
+    }
+    if (s.ffn == FfnKind::GatedSilu) {
+        void* d = nullptr;
+        LC_TRY(talloc(st, &d, (size_t)2 * s.ff * ld * 2));
+        const char* part[2] = {"gate", "up"};
+        for (int i = 0; i < 2; i++) {
+            DevTensor* t = nullptr;
+            LC_TRY(matrix(m, p + part[i], s.ff, W, &t));
+            LC_TRY(launch_pack((const bf16*)t->view, s.ff, W, (bf16*)d + (size_t)i * ld, ld, PackMap{1, 2, 0, 0}, PackMap(), false, m->stream));
+        }
+        LC_TRY(dense_weight_init(&L.up, (const bf16*)d, 2 * s.ff, W, ld));
+        return plain_weight(m, p + "down", W, s.ff, &L.down);
+    }
+    const MoeSpec& e = s.moe;
+    std::vector<std::string> names = {p + "router"};
+    std::vector<int> rows = {e.outputs()}, offs;
+    if (e.shared_ff) {
+        names.insert(names.end(), {p + "shared.sg", p + "shared.up"});
+        rows.insert(rows.end(), {1, e.shared_ff});
+        LC_TRY(plain_weight(m, p + "shared.down", W, e.shared_ff, &L.shared_down));
+    }
+    LC_TRY(fused_weight(m, names, rows, W, &L.route, &offs, e.shared_ff ? 32 : 8));
+    L.off_gate = e.shared_ff ? offs[1] : 0;
+    L.route_split = e.shared_ff ? offs[2] : (L.route.n + 31) / 32 * 32;
+    LC_TRY(model_gain_f32(m, p + "correction", e.outputs(), &L.correction));
+    LC_TRY(expert_weights(m, p, "up", e.experts, e.ff, W, &L.up));
+    LC_TRY(expert_weights(m, p, "down", e.experts, W, e.ff, &L.down));
+    L.expert_bytes = (uint64_t)2 * e.ff * W * 2;
+    m->expert_bytes_all += L.expert_bytes * e.experts;
+    m->expert_bytes_each = 1;  // d_moe_touched counts bytes
+    return LC_OK;
+}
+
 size_t elt(const LayerStack& st) { return st.f32 ? 4 : 2; }
 
 int32_t product(lc_model* m, const DenseWeight& w, const void* x, int ldx, int T, void* out, int ldo, bool out_f32 = false, DenseEpilogue epi = DENSE_STORE,
@@ -315,18 +400,78 @@ int32_t latent_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, 
     return product(m, L.out, st.mixed, lde, T, st.y, st.spec.width, true);
 }
 
-int32_t relu2_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T) {
+int32_t attention_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bool decode_step) {
     LayerStack& st = *m->stack;
+    const StackLayer& src = L.s.kv_from < 0 ? L : st.layers[(size_t)L.s.kv_from];
+    LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in.n, true));
+    AttnArgs a;
+    a.g = L.ag; a.proj = st.projf; a.ld_proj = L.in.n; a.off_k = L.off_k; a.off_v = L.off_v; a.q_norm = L.q_norm; a.k_norm = L.k_norm; a.eps = st.spec.eps; a.rot = L.rot;
+    a.q = st.q; a.k_cache = src.k_cache; a.v_cache = src.v_cache; a.page_tokens = m->page_tokens; a.page_table = m->d_page_table; a.tok_seq = m->d_tok_seq;
+    a.tok_pos = m->d_tok_pos; a.pages_per_seq = m->pages_per_seq; a.T = T; a.sink = L.sink; a.out = st.mixed; a.ldo = L.ag.heads * L.ep; a.f32 = st.f32;
+    LC_TRY(launch_attn_prep(a, m->stream));
+    m->launches_in_call += 1;
+    const int few = decode_step || !st.prefill_tiles ? T : st.n_short;
+    a.T = few;
+    if (few > 0) {
+        LC_TRY(launch_attn_tokens(a, st.attn, m->stream));
+        m->launches_in_call += 1;
+    }
+    if (few < T) {
+        LC_TRY(launch_attn_tiles(a, st.d_attn_tiles, st.n_attn_tiles, m->stream));
+        m->launches_in_call += 1;
+    }
+    return product(m, L.out, st.mixed, a.ldo, T, st.y, st.spec.width, true);
+}
+
+// What the residual sum (or a probe) needs to finish the mixture's output.
+MoeSum moe_sum(const LayerStack& st, const StackLayer& L, const void* x, int ldx) {
+    const MoeSpec& e = L.s.moe;
+    MoeSum r;
+    r.rows = st.moe_rows; r.ld_rows = round8(st.spec.width); r.sel = st.moe_sel; r.pos = st.moe_pos; r.off = st.plan.off; r.weight = st.moe_w; r.top = e.top; r.experts = e.experts;
+    r.h = x; r.ld_h = ldx;
+    if (e.shared_ff) { r.gate = st.moe_z + L.off_gate; r.ld_gate = L.route_split; }
+    return r;
+}
+
+int32_t moe_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bool decode_step) {
+    LayerStack& st = *m->stack;
+    const MoeSpec& e = L.s.moe;
+    DenseArgs r;
+    const int ldf = round8(e.ff), lds = round8(e.shared_ff);
+    r.split = L.route_split; r.out2 = st.ffn; r.ldo2 = lds;
+    LC_TRY(product(m, L.route, x, ldx, T, st.moe_z, L.route_split, true, DENSE_SPLIT_RELU2, r));
+    ExpertPlan plan = st.plan;
+    // tiles that hold the usual expert's tokens
+    const int usual = (T * e.top + e.outputs() - 1) / e.outputs();
+    plan.tile_rows = usual <= 12 ? 16 : usual <= 24 ? 32 : usual <= 48 ? 64 : usual <= 96 ? 128 : 256;
+    plan.most_rows = T * e.top;
+    plan.most_tiles = std::min(st.plan_tiles, std::min(plan.most_rows, e.experts + plan.most_rows / plan.tile_rows));
+    ChoiceArgs c;
+    c.m = e; c.z = st.moe_z; c.ld_z = L.route_split; c.T = T; c.correction = L.correction; c.sel = st.moe_sel; c.pos = st.moe_pos; c.weight = st.moe_w; c.counts = st.moe_counts;
+    c.plan = plan; c.touched = decode_step ? m->d_moe_touched : nullptr; c.touched_bytes = L.expert_bytes;
+    LC_TRY(launch_expert_choice(c, m->stream));
+    m->launches_in_call += 1;
+    DenseArgs g;
+    g.plan = &plan; g.gather = true;
+    LC_TRY(product(m, L.up, x, ldx, T, st.moe_up, ldf, false, DENSE_RELU2, g));
+    if (e.shared_ff) LC_TRY(product(m, L.shared_down, st.ffn, lds, T, st.y, st.spec.width, true));
+    g.gather = false; g.x_rows = st.moe_slots;
+    return product(m, L.down, st.moe_up, ldf, T, st.moe_rows, round8(st.spec.width), false, DENSE_STORE, g);
+}
+
+int32_t ffn_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bool decode_step) {
+    LayerStack& st = *m->stack;
+    if (L.s.ffn == FfnKind::Moe) return moe_block(m, L, x, ldx, T, decode_step);
     const int ldf = round8(L.s.ff);
-    LC_TRY(product(m, L.up, x, ldx, T, st.ffn, ldf, false, DENSE_RELU2));
+    LC_TRY(product(m, L.up, x, ldx, T, st.ffn, ldf, false, L.s.ffn == FfnKind::GatedSilu ? DENSE_GATED_SILU : DENSE_RELU2));
     return product(m, L.down, st.ffn, ldf, T, st.y, st.spec.width, true);
 }
 
-// The layers' input: the residual itself in f32, or its bf16 copy.
+// The layers' input: the residual itself in f32 models without norms on inputs, else the activations made from it.
 const void* layer_input(lc_model* m, int* ld) {
     LayerStack& st = *m->stack;
-    *ld = st.f32 ? st.spec.width : st.width_p;
-    return st.f32 ? (const void*)m->d_hidden : st.xa;
+    *ld = st.xa ? st.width_p : st.spec.width;
+    return st.xa ? st.xa : (const void*)m->d_hidden;
 }
 
 }  // namespace
@@ -340,15 +485,21 @@ int32_t stack_bind(lc_model* m) {
         StackLayer& L = st.layers[i];
         L.s = sp.layers[i];
         const std::string p = "l" + std::to_string(i) + ".";
-        if (L.s.mixer == MixerKind::ChannelDelta) LC_TRY(bind_delta(m, L, p + "mix."));
-        else LC_TRY(bind_latent(m, L, p + "mix."));
-        LC_TRY(model_gain_f32(m, p + "norm1", sp.width, &L.norm1));
-        if (L.s.ffn != FfnKind::None) {
-            LC_TRY(plain_weight(m, p + "mlp.up", L.s.ff, sp.width, &L.up));
-            LC_TRY(plain_weight(m, p + "mlp.down", sp.width, L.s.ff, &L.down));
-            LC_TRY(model_gain_f32(m, p + "norm2", sp.width, &L.norm2));
+        switch (L.s.mixer) {
+            case MixerKind::ChannelDelta: LC_TRY(bind_delta(m, L, p + "mix.")); break;
+            case MixerKind::LatentAttention: LC_TRY(bind_latent(m, L, p + "mix.")); break;
+            case MixerKind::Attention: LC_TRY(bind_attention(m, L, p + "mix.")); break;
         }
-        LC_TRY(block_weights(m, {&L.in, &L.out, &L.up, &L.down, &L.a2, &L.g2, &L.uq, &L.uk_t, &L.uv, &L.uk_all, &L.uv_all}));
+        auto norms = [&](const std::string& name, const float** in, const float** out) -> int32_t {
+            if (sp.norm_inputs) LC_TRY(model_gain_f32(m, name, sp.width, in));
+            return model_gain_f32(m, sp.norm_inputs ? name + "b" : name, sp.width, out);
+        };
+        LC_TRY(norms(p + "norm1", &L.norm1_in, &L.norm1_out));
+        if (L.s.ffn != FfnKind::None) {
+            LC_TRY(bind_ffn(m, L, p + "mlp."));
+            LC_TRY(norms(p + "norm2", &L.norm2_in, &L.norm2_out));
+        }
+        LC_TRY(block_weights(m, {&L.in, &L.out, &L.up, &L.down, &L.a2, &L.g2, &L.uq, &L.uk_t, &L.uv, &L.uk_all, &L.uv_all, &L.route, &L.shared_down}));
     }
     DevTensor* e = nullptr;
     LC_TRY(matrix(m, "embed", sp.vocab, sp.width, &e));
@@ -365,6 +516,8 @@ int32_t stack_alloc(lc_model* m) {
     const size_t T = (size_t)m->t_cap, e = elt(st);
     st.width_p = round8(st.spec.width);
     st.prefill_tiles = st.delta_chunks = !st.f32;
+    int experts = 0, top = 0;
+    size_t z = 0, hidden = 8, attn_part = 0;
     size_t proj = 8, projf = 8, gate = 8, mixed = 8, cq = 8, q = 8, qa = 8, ffn = 8, ld = 8, qk = 8, v = 8;
     for (StackLayer& L : st.layers) {
         const LayerSpec& s = L.s;
@@ -381,6 +534,19 @@ int32_t stack_alloc(lc_model* m) {
             st.delta_chunks = st.delta_chunks && delta_chunks_apply(L.dg, st.f32);
             st.chunk_bytes = std::max(st.chunk_bytes, delta_chunk_bytes(L.dg));
             st.state_bytes_per_seq += S * 4 + ring * e;
+        } else if (s.mixer == MixerKind::Attention) {
+            const AttnShape& g = L.ag;
+            projf = std::max(projf, (size_t)L.in.n);
+            q = std::max(q, (size_t)g.heads * g.dp);
+            mixed = std::max(mixed, (size_t)g.heads * g.ep);
+            st.prefill_tiles = st.prefill_tiles && attn_tiles_apply(g, st.f32);
+            attn_part = std::max(attn_part, attn_part_bytes(g));
+            if (s.kv_from < 0) {
+                const size_t rows = (size_t)m->pages_total * m->page_tokens * g.kv_heads;
+                LC_TRY(zalloc(st, &L.k_cache, rows * g.dp * e));
+                LC_TRY(zalloc(st, &L.v_cache, rows * g.ep * e));
+                st.cache_bytes_per_token += (size_t)g.kv_heads * (g.dp + g.ep) * e;
+            }
         } else {
             const LatentShape& g = L.lg;
             projf = std::max(projf, (size_t)L.in.n);
@@ -397,9 +563,33 @@ int32_t stack_alloc(lc_model* m) {
             LC_TRY(zalloc(st, &L.cache, (size_t)m->pages_total * m->page_tokens * row));
             st.cache_bytes_per_token += row;
         }
-        if (s.ffn != FfnKind::None) ffn = std::max(ffn, (size_t)round8(s.ff));
+        if (s.ffn == FfnKind::Moe) {
+            experts = std::max(experts, s.moe.experts); top = std::max(top, s.moe.top);
+            z = std::max(z, (size_t)L.route_split);
+            hidden = std::max(hidden, (size_t)round8(s.moe.ff));
+            ffn = std::max(ffn, (size_t)round8(s.moe.shared_ff));
+        } else if (s.ffn != FfnKind::None) ffn = std::max(ffn, (size_t)round8(s.ff));
     }
-    if (!st.f32) LC_TRY(zalloc(st, &st.xa, T * st.width_p * e));
+    if (experts) {
+        st.moe_slots = (int)T * top;
+        st.plan_tiles = experts + st.moe_slots / 16;
+        LC_TRY(zalloc(st, (void**)&st.moe_z, T * z * 4)); LC_TRY(zalloc(st, (void**)&st.moe_w, T * top * 4));
+        LC_TRY(zalloc(st, (void**)&st.moe_sel, T * top * 4)); LC_TRY(zalloc(st, (void**)&st.moe_pos, T * top * 4));
+        LC_TRY(zalloc(st, (void**)&st.moe_counts, ((size_t)experts + 1) * 4));
+        LC_TRY(zalloc(st, &st.moe_up, (size_t)st.moe_slots * hidden * e)); LC_TRY(zalloc(st, &st.moe_rows, (size_t)st.moe_slots * st.width_p * e));
+        LC_TRY(zalloc(st, (void**)&st.plan.tiles, (size_t)st.plan_tiles * sizeof(ExpertTile))); LC_TRY(zalloc(st, (void**)&st.plan.n_tiles, 4));
+        LC_TRY(zalloc(st, (void**)&st.plan.off, ((size_t)experts + 1) * 4)); LC_TRY(zalloc(st, (void**)&st.plan.lists, (size_t)experts * T * 4));
+        st.plan.list_stride = (int)T;
+        LC_TRY(dalloc(&m->d_moe_touched, 1));
+        LC_CUDA(cudaMemsetAsync(m->d_moe_touched, 0, 8, m->stream));
+    }
+    if (attn_part) {
+        st.attn.part_bytes = attn_part;
+        st.attn.n_tickets = 2 * sm_count();
+        LC_TRY(zalloc(st, (void**)&st.attn.part, attn_part)); LC_TRY(zalloc(st, (void**)&st.attn.tickets, (size_t)st.attn.n_tickets * 4));
+        LC_TRY(zalloc(st, (void**)&st.d_attn_tiles, T * sizeof(AttnTile)));
+    }
+    if (!st.f32 || st.spec.norm_inputs) LC_TRY(zalloc(st, &st.xa, T * st.width_p * e));
     LC_TRY(zalloc(st, &st.proj, T * proj * e)); LC_TRY(zalloc(st, (void**)&st.projf, T * projf * 4));
     LC_TRY(zalloc(st, &st.gate, T * gate * e)); LC_TRY(zalloc(st, &st.mixed, T * mixed * e));
     LC_TRY(zalloc(st, &st.cq, T * cq * e)); LC_TRY(zalloc(st, &st.q, T * q * e));
@@ -421,6 +611,19 @@ void stack_free(lc_model* m) {
     for (void* p : m->stack->temps) cudaFree(p);
     for (DevBuf* b : {&m->stack->ctx_c, &m->stack->ctx_k, &m->stack->ctx_v, &m->stack->chunk_scratch}) b->release();
     dense_workspace_free(&m->stack->ws);
+}
+
+// Cache and state a one-token step at position `ctx` reads and writes.
+uint64_t stack_step_bytes(const lc_model* m, int ctx) {
+    const LayerStack& st = *m->stack;
+    uint64_t b = 2 * st.state_bytes_per_seq;
+    for (const StackLayer& L : st.layers) {
+        if (L.s.mixer == MixerKind::LatentAttention) b += (uint64_t)(ctx + 1) * (L.lg.cp + L.lg.rp) * elt(st);
+        if (L.s.mixer != MixerKind::Attention) continue;
+        const int window = L.ag.window > 0 ? L.ag.window : ctx + 1, lo = std::max(0, ctx + 1 - window), seen = ctx + 1 - lo + std::min(L.ag.keep_first, lo);
+        b += (uint64_t)seen * L.ag.kv_heads * (L.ag.dp + L.ag.ep) * elt(st);
+    }
+    return b;
 }
 
 // What a call's tokens mean to the layers: runs of consecutive positions, those of at least kTileRun tokens also as tiles
@@ -451,12 +654,21 @@ int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const st
     }
     st.groups.clear();
     st.n_short = (int)seq.size();
+    st.n_attn_tiles = 0;
     std::vector<LatentTile> tiles;
     std::vector<LatentContext> ctx;
     size_t first = 0;
     while (first < runs.size() && runs[first].n < kTileRun) first++;
-    if (st.prefill_tiles && first < runs.size()) {
-        st.n_short = runs[first].tok0;
+    if (st.prefill_tiles && first < runs.size()) st.n_short = runs[first].tok0;
+    if (st.prefill_tiles && st.d_attn_tiles && first < runs.size()) {
+        std::vector<AttnTile> at;
+        for (size_t i = first; i < runs.size(); i++)
+            for (int t = 0; t < runs[i].n; t += 64) at.push_back(AttnTile{runs[i].tok0 + t, std::min(64, runs[i].n - t), runs[i].seq, runs[i].pos0 + t});
+        st.n_attn_tiles = (int)at.size();
+        LC_CUDA(cudaMemcpyAsync(st.d_attn_tiles, at.data(), at.size() * sizeof(AttnTile), cudaMemcpyHostToDevice, m->stream));
+        LC_CUDA(cudaStreamSynchronize(m->stream));
+    }
+    if (st.prefill_tiles && st.ctx_c_row && first < runs.size()) {
         int most = 0;
         for (size_t i = first; i < runs.size(); i++) {
             const SeqRun& r = runs[i];
@@ -483,25 +695,38 @@ int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const st
 
 int32_t stack_mixer(lc_model* m, int l, const void* x, int ldx, int T, bool decode_step) {
     StackLayer& L = m->stack->layers[l];
-    return L.s.mixer == MixerKind::ChannelDelta ? delta_block(m, L, x, ldx, T, decode_step) : latent_block(m, L, x, ldx, T, decode_step);
+    switch (L.s.mixer) {
+        case MixerKind::ChannelDelta: return delta_block(m, L, x, ldx, T, decode_step);
+        case MixerKind::LatentAttention: return latent_block(m, L, x, ldx, T, decode_step);
+        default: return attention_block(m, L, x, ldx, T, decode_step);
+    }
 }
-int32_t stack_ffn(lc_model* m, int l, const void* x, int ldx, int T) { return relu2_block(m, m->stack->layers[l], x, ldx, T); }
 
 int32_t stack_run_layers(lc_model* m, int T, bool decode_step) {
     LayerStack& st = *m->stack;
     const int W = st.spec.width;
     int ldx = 0;
     const void* x = layer_input(m, &ldx);
-    LC_TRY(launch_embed_rows(st.embed, st.spec.vocab, W, m->d_tokens, T, m->d_hidden, st.xa, st.width_p, m->stream));
+    LC_TRY(launch_embed_rows(st.embed, st.spec.vocab, W, m->d_tokens, T, st.spec.embed_scale, st.layers[0].norm1_in, st.spec.eps, m->d_hidden, st.xa, st.width_p, st.f32,
+                             m->stream));
     m->launches_in_call += 1;
+    ResidualArgs r;
+    r.y = st.y; r.eps = st.spec.eps; r.width = W; r.T = T; r.x = m->d_hidden; r.ld_act = st.width_p; r.f32 = st.f32;
     for (size_t l = 0; l < st.layers.size(); l++) {
+        StackLayer& L = st.layers[l];
+        const bool ffn = L.s.ffn != FfnKind::None, last = l + 1 == st.layers.size();
+        const float* after = last ? nullptr : st.layers[l + 1].norm1_in;  // the norm ahead of the next layer; the last sum is read in f32
+        auto sum = [&](const float* w, const float* next, bool moe) -> int32_t {
+            r.w = w; r.w_next = next; r.act = st.spec.norm_inputs && !next ? nullptr : st.xa;
+            r.moe = moe ? moe_sum(st, L, x, ldx) : MoeSum();
+            m->launches_in_call += 1;
+            return launch_residual(r, m->stream);
+        };
         LC_TRY(stack_mixer(m, (int)l, x, ldx, T, decode_step));
-        LC_TRY(launch_norm_residual(st.y, st.layers[l].norm1, st.spec.eps, W, T, m->d_hidden, st.xa, st.width_p, m->stream));
-        m->launches_in_call += 1;
-        if (st.layers[l].s.ffn == FfnKind::None) continue;
-        LC_TRY(stack_ffn(m, (int)l, x, ldx, T));
-        LC_TRY(launch_norm_residual(st.y, st.layers[l].norm2, st.spec.eps, W, T, m->d_hidden, st.xa, st.width_p, m->stream));
-        m->launches_in_call += 1;
+        LC_TRY(sum(L.norm1_out, ffn ? L.norm2_in : after, false));
+        if (!ffn) continue;
+        LC_TRY(ffn_block(m, L, x, ldx, T, decode_step));
+        LC_TRY(sum(L.norm2_out, after, L.s.ffn == FfnKind::Moe));
     }
     return LC_OK;
 }
@@ -509,13 +734,22 @@ int32_t stack_run_layers(lc_model* m, int T, bool decode_step) {
 // One sublayer on the f32 rows already in d_hidden (its output, before the norm, in `y`): for layer-level checks.
 int32_t stack_probe(lc_model* m, int l, int T, bool ffn, float** y) {
     LayerStack& st = *m->stack;
-    int ldx = 0;
-    const void* x = layer_input(m, &ldx);
-    if (!st.f32) LC_TRY(launch_act_rows(m->d_hidden, st.spec.width, T, st.xa, st.width_p, m->stream));
+    int ldx = st.spec.width;
+    const void* x = m->d_hidden;
+    if (!st.f32) {
+        x = layer_input(m, &ldx);
+        LC_TRY(launch_act_rows(m->d_hidden, st.spec.width, T, st.xa, st.width_p, m->stream));
+    }
     LC_CHECK(!ffn || st.layers[l].s.ffn != FfnKind::None, LC_ERR_INVALID, "layer %d has no feed-forward", l);
-    LC_TRY(ffn ? stack_ffn(m, l, x, ldx, T) : stack_mixer(m, l, x, ldx, T, false));
     *y = st.y;
-    return LC_OK;
+    if (!ffn) return stack_mixer(m, l, x, ldx, T, false);
+    StackLayer& L = st.layers[l];
+    LC_TRY(ffn_block(m, L, x, ldx, T, false));
+    if (L.s.ffn != FfnKind::Moe) return LC_OK;
+    ResidualArgs r;
+    r.y = st.y; r.width = st.spec.width; r.T = T; r.ld_act = st.width_p; r.f32 = st.f32;
+    r.moe = moe_sum(st, L, x, ldx);
+    return launch_residual(r, m->stream);
 }
 
 int32_t stack_head(lc_model* m, int n, const int32_t* idx, float* logits) {

@@ -29,7 +29,20 @@ enum DenseEpilogue {
     DENSE_STORE = 0,
     DENSE_RELU2 = 1,      // max(y, 0)^2
     DENSE_LOG_DECAY = 2,  // -e0[row / e_div] * softplus(y + e1[row]), 32-bit
-    DENSE_LOGITS = 3      // y * scale, then cap * tanh(. / cap) when cap > 0
+    DENSE_LOGITS = 3,     // y * scale, then cap * tanh(. / cap) when cap > 0
+    DENSE_GATED_SILU = 4, // rows in pairs (2i: gate, 2i + 1: up): out row i = silu(gate) * up
+    DENSE_SPLIT_RELU2 = 5 // rows below `split` as they are, in 32-bit, to `out`; the others squared relu, in the activations' type, to out2
+};
+// A product of one of several matrices per token (experts): the tokens come as tiles of rows that share a matrix.
+struct ExpertTile { int32_t expert, first, rows, row0; };  // rows first .. first + rows - 1 of the expert's list; row0: the first one's row in expert order
+struct ExpertPlan {
+    ExpertTile* tiles = nullptr;
+    int32_t* n_tiles = nullptr;
+    int32_t* off = nullptr;        // [experts + 1] rows of the experts before (expert order)
+    int32_t* lists = nullptr;      // [experts][list_stride] token of every row
+    int list_stride = 0;
+    int tile_rows = 16;            // most rows of a tile: 16, 32, 64, 128 or 256
+    int most_tiles = 0, most_rows = 0;  // bounds of this call (what the device finds is not known to the host)
 };
 struct DenseArgs {
     const DenseWeight* w = nullptr;
@@ -46,6 +59,10 @@ struct DenseArgs {
     const float* e1 = nullptr;
     int e_div = 1;
     float scale = 1.0f, cap = 0.0f;
+    void* out2 = nullptr;         // DENSE_SPLIT_RELU2
+    int ldo2 = 0, split = 0;      // split: a multiple of 32
+    const ExpertPlan* plan = nullptr;  // matrix = expert; output rows in expert order, input rows too unless `gather`
+    bool gather = false;          // input row of a tile's row = its token
     bool f32 = false;
 };
 // Scratch of the shares of k that several CTAs sum, and the tensor maps over activation buffers seen so far.
@@ -71,12 +88,39 @@ struct SeqRun { int32_t tok0, n, seq, pos0; };
 struct PackMap { int len = 0, stride = 0, split = 0, shift = 0; };
 int32_t launch_pack(const __nv_bfloat16* src, int rows, int cols, __nv_bfloat16* dst, int ld, PackMap row, PackMap col, bool transpose, cudaStream_t s);
 
-// x[t] = embed[ids[t]] in f32 and, act != null, as bf16 (rows ld_act apart); ids outside the table give zero rows
-int32_t launch_embed_rows(const __nv_bfloat16* table, int rows, int width, const int64_t* ids, int T, float* x, void* act, int ld_act, cudaStream_t s);
+// x[t] = embed[ids[t]] * scale in f32; act != null: the same as activations, through rms_norm(.) * w when w is given.  ids
+// outside the table give zero rows
+int32_t launch_embed_rows(const __nv_bfloat16* table, int rows, int width, const int64_t* ids, int T, float scale, const float* w, float eps, float* x, void* act, int ld_act,
+                          bool f32, cudaStream_t s);
 // act[t] = bf16(x[t])
 int32_t launch_act_rows(const float* x, int width, int T, void* act, int ld_act, cudaStream_t s);
-// x[t] += rms_norm(y[t]) * w; act != null: also the sum as bf16
-int32_t launch_norm_residual(const float* y, const float* w, float eps, int width, int T, float* x, void* act, int ld_act, cudaStream_t s);
+// The output of a mixture of experts at one token: gate * y + sum over the choices of weight * (expert's row, or the input for
+// identity experts).
+struct MoeSum {
+    const void* rows = nullptr;      // experts' outputs in expert order (activations); null: no mixture
+    int ld_rows = 0;
+    const int32_t *sel = nullptr, *pos = nullptr, *off = nullptr;  // [T][top] expert and place in its list; [experts + 1]
+    const float* weight = nullptr;   // [T][top]
+    int top = 0, experts = 0;
+    const void* h = nullptr;         // [T][ld_h] the mixture's input
+    int ld_h = 0;
+    const float* gate = nullptr;     // [T] rows ld_gate apart, before the sigmoid; null: y is not read
+    int ld_gate = 0;
+};
+// x[t] += rms_norm(y[t]) * w; act != null: the sum as activations, through rms_norm(.) * w_next when that is given.  With a
+// mixture y is first replaced by its output (x null: nothing more happens).
+struct ResidualArgs {
+    float* y = nullptr;
+    const float *w = nullptr, *w_next = nullptr;
+    float eps = 1e-6f;
+    int width = 0, T = 0;
+    float* x = nullptr;
+    void* act = nullptr;
+    int ld_act = 0;
+    bool f32 = false;
+    MoeSum moe;
+};
+int32_t launch_residual(const ResidualArgs& a, cudaStream_t s);
 // out[i] = rms_norm(x[idx ? idx[i] : i]) * w as activations
 int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, float eps, int width, int n, void* out, int ldo, bool f32, cudaStream_t s);
 
@@ -181,11 +225,59 @@ bool latent_prefill_applies(const LatentShape& g, int ep, bool f32);
 int32_t launch_latent_gather(const LatentArgs& a, const LatentContext* ctx, int n_ctx, int longest, void* out, cudaStream_t s);
 int32_t launch_latent_prefill(const LatentArgs& a, const LatentPrefill& p, int n_tiles, cudaStream_t s);
 
+// ---- gqa_attention.cu: attention over the keys and values of a paged cache, [page][kv head][page_tokens][dp] and [..][ep] -----
+struct AttnShape {
+    int heads, kv_heads, dim, vdim, dp, ep, rot_dims;  // dp, ep: dim, vdim rounded up to 8; rotation pairs i with i + rot_dims / 2
+    float scale;
+    int window, keep_first;                            // MaskSpec
+};
+struct AttnArgs {
+    AttnShape g;
+    const float* proj = nullptr;       // [T][ld_proj] q | k | v
+    int ld_proj = 0, off_k = -1, off_v = 0;  // off_k < 0: the layer has no keys and values of its own
+    const float *q_norm = nullptr, *k_norm = nullptr;
+    float eps = 1e-6f;
+    const float2* rot = nullptr;       // [position][rot_dims / 2] (cos, sin)
+    void* q = nullptr;                 // [T][heads][dp]
+    void *k_cache = nullptr, *v_cache = nullptr;
+    int page_tokens = 16;
+    const int32_t *page_table = nullptr, *tok_seq = nullptr, *tok_pos = nullptr;
+    int pages_per_seq = 0, T = 0;
+    const float* sink = nullptr;       // [heads] or null
+    void* out = nullptr;               // [T][ldo], heads ep apart
+    int ldo = 0;
+    bool f32 = false;
+};
+int32_t launch_attn_prep(const AttnArgs& a, cudaStream_t s);   // norms over all of q and of k, rotation, cache append
+struct AttnScratch { float* part = nullptr; size_t part_bytes = 0; unsigned* tickets = nullptr; int n_tickets = 0; };
+size_t attn_part_bytes(const AttnShape& g);
+int32_t launch_attn_tokens(const AttnArgs& a, const AttnScratch& sc, cudaStream_t s);  // tokens 0 .. T - 1, each over its own context
+// up to 64 consecutive tokens (rows tok0 .. of the call, first position pos0)
+struct AttnTile { int32_t tok0, n, seq, pos0; };
+bool attn_tiles_apply(const AttnShape& g, bool f32);
+int32_t launch_attn_tiles(const AttnArgs& a, const AttnTile* tiles, int n_tiles, cudaStream_t s);
+
+// ---- expert_choice.cu: routing ---------------------------------------------------------------------------------------------
+struct ChoiceArgs {
+    MoeSpec m;
+    const float* z = nullptr;          // [T][ld_z] router logits
+    int ld_z = 0, T = 0;
+    const float* correction = nullptr; // [outputs]
+    int32_t *sel = nullptr, *pos = nullptr;  // [T][top] expert, its place in the expert's list (experts with matrices)
+    float* weight = nullptr;           // [T][top]
+    int32_t* counts = nullptr;         // [experts] + one ticket word, zero between launches
+    ExpertPlan plan;
+    unsigned long long* touched = nullptr;  // += touched_bytes for every expert that received a token
+    unsigned long long touched_bytes = 0;
+};
+int32_t launch_expert_choice(const ChoiceArgs& a, cudaStream_t s);
+
 // ---- a stack of such layers (layers.cu) --------------------------------------------------------------------------------
 struct StackLayer {
     LayerSpec s;
-    const float *norm1 = nullptr, *norm2 = nullptr;
-    DenseWeight in, out, up, down;
+    // norms of the sublayers' inputs (null: none) and outputs
+    const float *norm1_in = nullptr, *norm1_out = nullptr, *norm2_in = nullptr, *norm2_out = nullptr;
+    DenseWeight in, out, up, down;     // GatedSilu: `up` = gate and up rows in turn
     // ChannelDelta: `in` = q | k | v | a1 | g1 | b
     DenseWeight a2, g2;
     DeltaShape dg{};
@@ -201,6 +293,16 @@ struct StackLayer {
     const float *q_norm = nullptr, *c_norm = nullptr;
     const float2* rot = nullptr;
     void* cache = nullptr;
+    // Attention: `in` = q | k | v (q alone when another layer's cache is read)
+    AttnShape ag{};
+    int off_k = -1, off_v = 0;
+    const float *k_norm = nullptr, *sink = nullptr;
+    void *k_cache = nullptr, *v_cache = nullptr;
+    // Moe: `up` and `down` of all experts; `route` = router | gate of the shared expert | (from row route_split on) its up
+    DenseWeight route, shared_down;
+    int off_gate = 0, route_split = 0;
+    const float* correction = nullptr;
+    uint64_t expert_bytes = 0;         // one expert's matrices
 };
 struct LayerStack {
     ArchSpec spec;
@@ -236,9 +338,18 @@ struct LayerStack {
     std::vector<Group> groups;
     LatentTile* d_lat_tiles = nullptr;
     LatentContext* d_lat_ctx = nullptr;
+    AttnTile* d_attn_tiles = nullptr;
+    int n_attn_tiles = 0;
+    AttnScratch attn;
+    // mixtures of experts
+    float *moe_z = nullptr, *moe_w = nullptr;
+    int32_t *moe_sel = nullptr, *moe_pos = nullptr, *moe_counts = nullptr;
+    void *moe_up = nullptr, *moe_rows = nullptr;  // the experts' hidden rows and outputs, in expert order
+    ExpertPlan plan;
+    int plan_tiles = 0, moe_slots = 0;  // room of the tile list; rows of moe_up and moe_rows
     void* pieces = nullptr;
     size_t pieces_bytes = 0;
-    bool prefill_tiles = false;        // every latent layer has a tile form
+    bool prefill_tiles = false;        // every attention layer has a tile form
     size_t ctx_c_row = 0, ctx_k_row = 0, ctx_v_row = 0;  // widest rows of the context buffers, in elements
     DevBuf ctx_c, ctx_k, ctx_v;
 };

@@ -67,6 +67,14 @@ __device__ __forceinline__ void tma_load_4d(void* dst, const void* tmap, int x, 
         "l"(tmap), "r"(x), "r"(y), "r"(z), "r"(w), "r"(smem_u32(bar))
         : "memory");
 }
+// four rows of a tensor map whose box is one row high, in a row in shared memory
+__device__ __forceinline__ void tma_gather4(void* dst, const void* tmap, int x, int4 rows, uint64_t* bar) {
+    asm volatile(
+        "cp.async.bulk.tensor.2d.shared::cluster.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5, %6}], [%7];" ::"r"(
+            smem_u32(dst)),
+        "l"(tmap), "r"(x), "r"(rows.x), "r"(rows.y), "r"(rows.z), "r"(rows.w), "r"(smem_u32(bar))
+        : "memory");
+}
 
 // cpu.rs:62-64
 __device__ __forceinline__ float silu_f(float v) { return v * (1.0f / (1.0f + expf(-v))); }

@@ -5,19 +5,12 @@
 #include <algorithm>
 #include <cmath>
 #include "lc_mixers.h"
+#include "lc_mma.cuh"
 #include "lc_tma.cuh"
 
 namespace lc {
 
 namespace {
-
-template <typename A> __device__ __forceinline__ float act_f(A v);
-template <> __device__ __forceinline__ float act_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ float act_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
-template <typename A> __device__ __forceinline__ A to_act(float v);
-template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
-template <> __device__ __forceinline__ __nv_bfloat16 to_act<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
-__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 __device__ __forceinline__ int mapped(const PackMap& m, int i) {
     if (m.len == 0) return i;
@@ -62,64 +55,161 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const __nv_bfloat16* __
     }
 }
 
+// The same with a factor on the row and, w != null, the row's norm as activations.
+template <typename A>
+__global__ void __launch_bounds__(256) embed_norm_kernel(const bf16* __restrict__ table, int rows, int width, const int64_t* __restrict__ ids, float scale,
+                                                         const float* __restrict__ w, float eps, float* __restrict__ x, A* __restrict__ act, int ld_act) {
+    __shared__ float sh[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const int64_t id = ids[t];
+    const bool ok = id >= 0 && id < rows;
+    const bf16* src = table + (size_t)(ok ? id : 0) * width;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        const float v = ok ? __bfloat162float(src[c]) * scale : 0.0f;
+        x[t * width + c] = v;
+        ss = fmaf(v, v, ss);
+    }
+    if (!act) return;
+    float r = 1.0f;
+    if (w) r = 1.0f / sqrtf(block_sum(ss, sh) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        const float v = (ok ? __bfloat162float(src[c]) * scale : 0.0f) * r;
+        act[t * ld_act + c] = to_act<A>(w ? v * w[c] : v);
+    }
+}
+
 __global__ void __launch_bounds__(256) act_rows_kernel(const float* __restrict__ x, int width, __nv_bfloat16* __restrict__ act, int ld_act) {
     pdl_launch_dependents();
     pdl_wait();
     for (int c = threadIdx.x; c < width; c += blockDim.x) act[(size_t)blockIdx.x * ld_act + c] = __float2bfloat16_rn(x[(size_t)blockIdx.x * width + c]);
 }
 
-// VEC = 4: rows of a multiple of four elements; a row of up to 4096 elements stays in registers between its two passes.
-template <int VEC>
-__global__ void __launch_bounds__(512) norm_residual_kernel(const float* __restrict__ y, const float* __restrict__ w, float eps, int width, float* __restrict__ x,
-                                                            __nv_bfloat16* __restrict__ act, int ld_act) {
+template <typename A> __device__ __forceinline__ float4 load4(const A* p);
+template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *(const float4*)p; }
+template <> __device__ __forceinline__ float4 load4<bf16>(const bf16* p) {
+    const uint2 v = *(const uint2*)p;
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
+}
+template <typename A> __device__ __forceinline__ void store4(A* p, float4 v);
+template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { *(float4*)p = v; }
+template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
+__device__ __forceinline__ float sq4(float4 v, float ss) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss)))); }
+__device__ __forceinline__ void add4(float4& y, float w, float4 v) { y.x = fmaf(w, v.x, y.x); y.y = fmaf(w, v.y, y.y); y.z = fmaf(w, v.z, y.z); y.w = fmaf(w, v.w, y.w); }
+
+// VEC = 4: rows of a multiple of four elements; a row of up to 16 elements per thread stays in registers between its passes.
+template <typename A, int VEC, bool MOE>
+__global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
     constexpr int kHeld = 4;
-    __shared__ float sh[32];
+    __shared__ float sh[32], sh2[32];
+    __shared__ long long s_row[kMaxChoices];
+    __shared__ float s_w[kMaxChoices], s_gate;
     pdl_launch_dependents();
     pdl_wait();
     const size_t t = blockIdx.x;
-    const float* yr = y + t * width;
-    float* xr = x + t * width;
-    __nv_bfloat16* ar = act ? act + t * ld_act : nullptr;
+    const int width = a.width;
+    float* yr = a.y + t * width;
+    float* xr = a.x + t * width;
+    const float *w = a.w, *wn = a.w_next;
+    A* ar = a.act ? (A*)a.act + t * a.ld_act : nullptr;
+    const A* hr = MOE ? (const A*)a.moe.h + t * a.moe.ld_h : nullptr;
+    float own = 0.0f, gate = 0.0f;  // weight of the input itself, of y
+    if constexpr (MOE) {
+        if ((int)threadIdx.x < a.moe.top) {
+            const size_t i = t * a.moe.top + threadIdx.x;
+            const int e = a.moe.sel[i];
+            s_row[threadIdx.x] = e < a.moe.experts ? (long long)(a.moe.off[e] + a.moe.pos[i]) * a.moe.ld_rows : -1;
+            s_w[threadIdx.x] = a.moe.weight[i];
+        }
+        if (threadIdx.x == 0) s_gate = a.moe.gate ? sigmoid_f(a.moe.gate[t * a.moe.ld_gate]) : 0.0f;
+        __syncthreads();
+        for (int j = 0; j < a.moe.top; j++) own += s_row[j] < 0 ? s_w[j] : 0.0f;
+        gate = s_gate;
+    }
     float ss = 0.0f;
     if constexpr (VEC == 4) {
         float4 yv[kHeld], xv[kHeld];
-#pragma unroll
-        for (int i = 0; i < kHeld; i++) {
-            const int c = (threadIdx.x + i * blockDim.x) * 4;
-            if (c < width) { yv[i] = *(const float4*)(yr + c); xv[i] = *(const float4*)(xr + c); }
-            else yv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-            ss = fmaf(yv[i].x, yv[i].x, fmaf(yv[i].y, yv[i].y, fmaf(yv[i].z, yv[i].z, fmaf(yv[i].w, yv[i].w, ss))));
-        }
-        for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < width; c += blockDim.x * 4) {
-            const float4 v = *(const float4*)(yr + c);
-            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
-        }
-        ss = block_sum(ss, sh);
-        const float r = 1.0f / sqrtf(ss / (float)width + eps);
-        auto put = [&](int c, float4 yy, float4 xx) {
-            const float4 g = *(const float4*)(w + c);
-            xx.x += yy.x * r * g.x; xx.y += yy.y * r * g.y; xx.z += yy.z * r * g.z; xx.w += yy.w * r * g.w;
-            *(float4*)(xr + c) = xx;
-            if (ar) {
-                *(__nv_bfloat162*)(ar + c) = __floats2bfloat162_rn(xx.x, xx.y);
-                *(__nv_bfloat162*)(ar + c + 2) = __floats2bfloat162_rn(xx.z, xx.w);
-            }
+        auto out_at = [&](int c) {
+            if constexpr (!MOE) return *(const float4*)(yr + c);
+            float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (a.moe.gate) add4(y, gate, *(const float4*)(yr + c));
+            for (int j = 0; j < a.moe.top; j++)
+                if (s_row[j] >= 0) add4(y, s_w[j], load4<A>((const A*)a.moe.rows + s_row[j] + c));
+            if (own != 0.0f) add4(y, own, load4<A>(hr + c));
+            return y;
         };
 #pragma unroll
         for (int i = 0; i < kHeld; i++) {
             const int c = (threadIdx.x + i * blockDim.x) * 4;
-            if (c < width) put(c, yv[i], xv[i]);
+            if (c < width) {
+                yv[i] = out_at(c);
+                if (a.x) xv[i] = *(const float4*)(xr + c);
+                else *(float4*)(yr + c) = yv[i];
+            } else yv[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            ss = sq4(yv[i], ss);
+        }
+        for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < width; c += blockDim.x * 4) {
+            const float4 v = out_at(c);
+            if (MOE) *(float4*)(yr + c) = v;
+            ss = sq4(v, ss);
+        }
+        if (MOE && !a.x) return;
+        ss = block_sum(ss, sh);
+        const float r = 1.0f / sqrtf(ss / (float)width + a.eps);
+        float s2 = 0.0f;
+        auto put = [&](int c, float4 yy, float4 xx) {
+            const float4 g = *(const float4*)(w + c);
+            xx.x += yy.x * r * g.x; xx.y += yy.y * r * g.y; xx.z += yy.z * r * g.z; xx.w += yy.w * r * g.w;
+            *(float4*)(xr + c) = xx;
+            if (ar && !wn) store4<A>(ar + c, xx);
+            s2 = sq4(xx, s2);
+            return xx;
+        };
+#pragma unroll
+        for (int i = 0; i < kHeld; i++) {
+            const int c = (threadIdx.x + i * blockDim.x) * 4;
+            if (c < width) xv[i] = put(c, yv[i], xv[i]);
         }
         for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < width; c += blockDim.x * 4) put(c, *(const float4*)(yr + c), *(const float4*)(xr + c));
+        if (!wn) return;
+        const float r2 = 1.0f / sqrtf(block_sum(s2, sh2) / (float)width + a.eps);
+        auto next = [&](int c, float4 v) {
+            const float4 g = *(const float4*)(wn + c);
+            store4<A>(ar + c, make_float4(v.x * r2 * g.x, v.y * r2 * g.y, v.z * r2 * g.z, v.w * r2 * g.w));
+        };
+#pragma unroll
+        for (int i = 0; i < kHeld; i++) {
+            const int c = (threadIdx.x + i * blockDim.x) * 4;
+            if (c < width) next(c, xv[i]);
+        }
+        for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < width; c += blockDim.x * 4) next(c, *(const float4*)(xr + c));
     } else {
-        for (int c = threadIdx.x; c < width; c += blockDim.x) { const float v = yr[c]; ss = fmaf(v, v, ss); }
+        for (int c = threadIdx.x; c < width; c += blockDim.x) {
+            float v = 0.0f;
+            if constexpr (MOE) {
+                if (a.moe.gate) v = gate * yr[c];
+                for (int j = 0; j < a.moe.top; j++)
+                    if (s_row[j] >= 0) v = fmaf(s_w[j], act_f<A>(((const A*)a.moe.rows)[s_row[j] + c]), v);
+                if (own != 0.0f) v = fmaf(own, act_f<A>(hr[c]), v);
+                yr[c] = v;
+            } else v = yr[c];
+            ss = fmaf(v, v, ss);
+        }
+        if (MOE && !a.x) return;
         ss = block_sum(ss, sh);
-        const float r = 1.0f / sqrtf(ss / (float)width + eps);
+        const float r = 1.0f / sqrtf(ss / (float)width + a.eps);
+        float s2 = 0.0f;
         for (int c = threadIdx.x; c < width; c += blockDim.x) {
             const float v = xr[c] + yr[c] * r * w[c];
             xr[c] = v;
-            if (ar) ar[c] = __float2bfloat16_rn(v);
+            if (ar && !wn) ar[c] = to_act<A>(v);
+            s2 = fmaf(v, v, s2);
         }
+        if (!wn) return;
+        const float r2 = 1.0f / sqrtf(block_sum(s2, sh2) / (float)width + a.eps);
+        for (int c = threadIdx.x; c < width; c += blockDim.x) ar[c] = to_act<A>(xr[c] * r2 * wn[c]);
     }
 }
 
@@ -628,19 +718,33 @@ int32_t launch_pack(const __nv_bfloat16* src, int rows, int cols, __nv_bfloat16*
     LC_CUDA(cudaGetLastError());
     return LC_OK;
 }
-int32_t launch_embed_rows(const __nv_bfloat16* table, int rows, int width, const int64_t* ids, int T, float* x, void* act, int ld_act, cudaStream_t s) {
-    LC_CUDA(launch_pdl(embed_rows_kernel, dim3((unsigned)T), dim3(256), 0, s, table, rows, width, ids, x, (__nv_bfloat16*)act, ld_act));
+int32_t launch_embed_rows(const __nv_bfloat16* table, int rows, int width, const int64_t* ids, int T, float scale, const float* w, float eps, float* x, void* act, int ld_act,
+                          bool f32, cudaStream_t s) {
+    const dim3 grid((unsigned)T), block(256);
+    if (scale == 1.0f && !w && !(f32 && act)) LC_CUDA(launch_pdl(embed_rows_kernel, grid, block, 0, s, table, rows, width, ids, x, (bf16*)act, ld_act));
+    else if (f32) LC_CUDA(launch_pdl(embed_norm_kernel<float>, grid, block, 0, s, table, rows, width, ids, scale, w, eps, x, (float*)act, ld_act));
+    else LC_CUDA(launch_pdl(embed_norm_kernel<bf16>, grid, block, 0, s, table, rows, width, ids, scale, w, eps, x, (bf16*)act, ld_act));
     return LC_OK;
 }
 int32_t launch_act_rows(const float* x, int width, int T, void* act, int ld_act, cudaStream_t s) {
     LC_CUDA(launch_pdl(act_rows_kernel, dim3((unsigned)T), dim3(256), 0, s, x, width, (__nv_bfloat16*)act, ld_act));
     return LC_OK;
 }
-int32_t launch_norm_residual(const float* y, const float* w, float eps, int width, int T, float* x, void* act, int ld_act, cudaStream_t s) {
-    const dim3 grid((unsigned)T), block((unsigned)norm_threads(width));
-    if (width % 4 == 0 && (uintptr_t)w % 16 == 0) LC_CUDA(launch_pdl(norm_residual_kernel<4>, grid, block, 0, s, y, w, eps, width, x, (__nv_bfloat16*)act, ld_act));
-    else LC_CUDA(launch_pdl(norm_residual_kernel<1>, grid, block, 0, s, y, w, eps, width, x, (__nv_bfloat16*)act, ld_act));
-    return LC_OK;
+int32_t launch_residual(const ResidualArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)a.T), block((unsigned)norm_threads(a.width));
+    const bool moe = a.moe.rows != nullptr;
+    const bool vec = a.width % 4 == 0 && (uintptr_t)a.w % 16 == 0 && (uintptr_t)a.w_next % 16 == 0 && (a.moe.ld_rows | a.moe.ld_h | a.ld_act) % 4 == 0;
+    LC_CHECK(a.moe.top <= kMaxChoices && (!a.w_next || a.act), LC_ERR_INVALID, "residual sum: bad argument");
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(launch_pdl(kern, grid, block, 0, s, a));
+        return LC_OK;
+    };
+    if (a.f32) {
+        if (moe) return vec ? go(residual_kernel<float, 4, true>) : go(residual_kernel<float, 1, true>);
+        return vec ? go(residual_kernel<float, 4, false>) : go(residual_kernel<float, 1, false>);
+    }
+    if (moe) return vec ? go(residual_kernel<bf16, 4, true>) : go(residual_kernel<bf16, 1, true>);
+    return vec ? go(residual_kernel<bf16, 4, false>) : go(residual_kernel<bf16, 1, false>);
 }
 int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, float eps, int width, int n, void* out, int ldo, bool f32, cudaStream_t s) {
     const dim3 grid((unsigned)n), block((unsigned)norm_threads(width));

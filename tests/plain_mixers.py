@@ -176,3 +176,119 @@ class PlainModel:
         z = linear(rms_norm(x, self.eps, self.w["final.norm"]), self.w["head"]) * self.c["logit_scale"]
         cap = self.c["logit_softcap"]
         return cap * np.tanh(z / cap)
+
+
+# ---- grouped-query attention under a window with kept first tokens, mixtures with identity experts -----------------------------
+def rotate_halves(x, pos, dims, base):
+    """Dimension i of the first `dims` is paired with i + dims / 2; rows (axis 0) at positions `pos`, heads on axis 1."""
+    half = dims // 2
+    a = np.asarray(pos, np.float64)[:, None] * base ** (-2.0 * np.arange(half) / dims)[None, :]
+    cos, sin = np.cos(a)[:, None], np.sin(a)[:, None]
+    y = np.array(x, np.float64)
+    u, v = x[..., :half], x[..., half:dims]
+    y[..., :half] = u * cos - v * sin
+    y[..., half:dims] = v * cos + u * sin
+    return y
+
+
+def visible(query_pos, keys, size, keep_first):
+    """[queries, keys]: key j is seen from i when j <= i and it is nearer than `size` or one of the first `keep_first`."""
+    i, j = np.asarray(query_pos)[:, None], np.arange(keys)[None, :]
+    return (j <= i) & ((i - j < size) | (j < keep_first))
+
+
+def sink_attention(q, k, v, scale, seen, sink):
+    """q: [T, H, D]; k: [S, G, D]; v: [S, G, E]; seen: [T, S]; sink: [H] logits that take weight and give no value."""
+    T, H, G = q.shape[0], q.shape[1], k.shape[1]
+    out = np.zeros((T, H, v.shape[2]))
+    for h in range(H):
+        g = h // (H // G)
+        s = np.where(seen, q[:, h] @ k[:, g].T * scale, -np.inf)
+        m = np.maximum(s.max(axis=1), sink[h])[:, None]
+        e = np.exp(s - m)
+        out[:, h] = e / (e.sum(axis=1, keepdims=True) + np.exp(sink[h] - m)) @ v[:, g]
+    return out
+
+
+def gated_silu(x, gate, up, down):
+    return linear(silu(linear(x, gate)) * linear(x, up), down)
+
+
+def squared_relu(x, up, down):
+    return linear(np.maximum(linear(x, up), 0.0) ** 2, down)
+
+
+def choose_experts(z, correction, groups, keep, top):
+    """One token's router logits -> [(expert, weight)]: softmax scores, choice by score + correction inside the best groups."""
+    s = np.exp(z - z.max())
+    s /= s.sum()
+    choice = s + correction
+    size = len(z) // groups
+    best = sorted(range(groups), key=lambda g: -choice[g * size : (g + 1) * size].max())[:keep]
+    allowed = [e for e in range(len(z)) if e // size in best]
+    return [(e, s[e]) for e in sorted(allowed, key=lambda e: -choice[e])[:top]]
+
+
+class PlainTenetar:
+    """Norms on both sides of every sublayer; attention layers that may read an earlier layer's keys and values; dense or
+    mixture feed-forwards."""
+
+    def __init__(self, config, w):
+        self.c = config
+        self.w = {n: np.asarray(a, np.float64) for n, a in w.items()}
+        self.eps = config["norm"]["eps"]
+
+    def new_state(self):
+        return {"pos": 0, "layers": [dict() for _ in self.c["layers"]]}
+
+    def attention(self, i, x, layers, first):
+        """`layers`: the states of all layers (this one's keys and values are appended to its own, if it has any)."""
+        mx, p, w, T = self.c["layers"][i]["mixer"], "l%d.mix." % i, self.w, len(x)
+        H, G, D, E, rot = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"], mx["rot"]
+        pos = first + np.arange(T)
+        q = rms_norm(linear(x, w[p + "q"]), self.eps, w[p + "q.norm"]).reshape(T, H, D)
+        q = rotate_halves(q, pos, rot["dims"], rot["base"])
+        src = mx.get("kv_from")
+        st = layers[i if src is None else src]
+        if src is None:
+            k = rms_norm(linear(x, w[p + "k"]), self.eps, w[p + "k.norm"]).reshape(T, G, D)
+            k = rotate_halves(k, pos, rot["dims"], rot["base"])
+            v = linear(x, w[p + "v"]).reshape(T, G, E)
+            st["k"] = np.concatenate([st["k"], k]) if st else k
+            st["v"] = np.concatenate([st["v"], v]) if "v" in st else v
+        seen = visible(pos, len(st["k"]), mx["mask"]["size"], mx["mask"]["keep_first"])
+        o = sink_attention(q, st["k"], st["v"], mx["scale"], seen, w[p + "sink"])
+        return linear(o.reshape(T, H * E), w[p + "o"])
+
+    def mixture(self, p, mlp, x):
+        w, r = self.w, mlp["router"]
+        z = linear(x, w[p + "router"])
+        y = np.zeros((len(x), x.shape[1]))
+        for t in range(len(x)):
+            for e, s in choose_experts(z[t], w[p + "correction"], r["groups"]["count"], r["groups"]["keep"], r["top"]):
+                y[t] += s * (x[t] if e >= r["experts"] else squared_relu(x[t], w[p + "e%d.up" % e], w[p + "e%d.down" % e]))
+        return y + sigmoid(linear(x, w[p + "shared.sg"])) * squared_relu(x, w[p + "shared.up"], w[p + "shared.down"])
+
+    def feed_forward(self, i, x):
+        mlp, p = self.c["layers"][i]["mlp"], "l%d.mlp." % i
+        if mlp["kind"] == "moe":
+            return self.mixture(p, mlp, x)
+        return gated_silu(x, self.w[p + "gate"], self.w[p + "up"], self.w[p + "down"])
+
+    def forward(self, tokens, state, trace=None):
+        first, w = state["pos"], self.w
+        x = w["embed"][np.asarray(tokens)] * self.c["embedding"]["scale"]
+        norm = lambda name, v: rms_norm(v, self.eps, w[name])
+        for i, ly in enumerate(self.c["layers"]):
+            l = "l%d." % i
+            x = x + norm(l + "norm1b", self.attention(i, norm(l + "norm1", x), state["layers"], first))
+            if ly["mlp"] is not None:
+                x = x + norm(l + "norm2b", self.feed_forward(i, norm(l + "norm2", x)))
+            if trace is not None:
+                trace.append(x.copy())
+        state["pos"] = first + len(tokens)
+        return linear(norm("final.norm", x), w["head"])
+
+
+def plain_model(config, w):
+    return {"Varasun": PlainModel, "Tenetar": PlainTenetar}[config["architecture"]](config, w)
