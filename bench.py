@@ -299,12 +299,18 @@ def moe_decode(lc, synth, local: int, n_seqs: int = 16, prompt_len: int = 1024, 
     return out
 
 
-def layered_leg(lc, synth, local: int, sizes=("1b", "7b"), prompt_len: int = PROMPT_LEN, steps: int = 32, batches=(1, 16, 64), llama: bool = True, pattern: str = "") -> dict:
-    """Varasun-shaped models (gated delta rule and latent attention layers, bf16, random weights) beside Llama-shaped models of
-    the same width, depth, heads and FFN width (16-bit and Q4_K weights): prefill of one prompt and decode steps at several
-    batch sizes, all contexts of prompt_len tokens.  The weights of a step exceed L2, so nothing is flushed between steps."""
+def layered_leg(lc, synth, local: int, sizes=("1b", "7b"), prompt_len: int = PROMPT_LEN, steps: int = 32, batches=(1, 16, 64), llama: bool = True, pattern: str = "",
+                designs=("varasun",), tenetar_pattern: str = "") -> dict:
+    """Varasun-shaped models (gated delta rule and latent attention layers, bf16, random weights) and Tenetar-shaped ones (windowed
+    attention with shared caches, mixtures of experts) beside Llama-shaped models of the same width, depth, heads and FFN width
+    (16-bit and Q4_K weights; with Tenetar also a Llama-shaped mixture of the same experts, Q4_K): prefill of one prompt and decode
+    steps at several batch sizes, all contexts of prompt_len tokens.  The weights of a step exceed L2, so nothing is flushed
+    between steps."""
     peak, which = measured_peaks()
     shapes = {"1b": dict(width=2048, heads=16, ff=5632, q_rank=768), "7b": dict(width=4096, heads=32, ff=11008, q_rank=1536)}
+    experts = {"1b": dict(kv_heads=4, experts=64, identity=8, top=6, groups=8, keep=4, expert_ff=1024, shared_ff=2048),
+               "7b": dict(kv_heads=8, experts=64, identity=8, top=8, groups=8, keep=4, expert_ff=1536, shared_ff=3072)}
+    tenetar_pattern = tenetar_pattern or "dmmmmsss"
     pattern = pattern or "dddaddda"
     out = {"prompt_len": prompt_len, "pattern": pattern, "peak_gbs": peak, "peak_source": which}
 
@@ -342,7 +348,17 @@ def layered_leg(lc, synth, local: int, sizes=("1b", "7b"), prompt_len: int = PRO
     for size in sizes:
         sh = shapes[size]
         spec = synth.layered_spec(size, sh["width"], pattern, sh["ff"], 32000, sh["heads"], q_rank=sh["q_rank"])
-        out[size] = {"varasun": measure(lambda b: synth.build_layered_engine(spec, max_seq_len=cap, max_seqs=b, device=local), 32000)}
+        out[size] = {}
+        if "varasun" in designs:
+            out[size]["varasun"] = measure(lambda b: synth.build_layered_engine(spec, max_seq_len=cap, max_seqs=b, device=local), 32000)
+        if "tenetar" in designs:
+            ex = experts[size]
+            ts = synth.tenetar_spec(size, sh["width"], tenetar_pattern, sh["ff"], 32000, sh["heads"], **ex)
+            out[size]["tenetar"] = dict(measure(lambda b: synth.build_layered_engine(ts, max_seq_len=cap, max_seqs=b, device=local), 32000), pattern=tenetar_pattern)
+            if llama:
+                ms = synth.ModelSpec(size + "moe", len(tenetar_pattern), sh["width"], sh["heads"], ex["kv_heads"], ex["expert_ff"], 32000, 10000.0, lc.TYPE_Q4_K,
+                                     lc.TYPE_Q4_K, lc.TYPE_Q4_K, n_experts=ex["experts"], top_k=ex["top"])
+                out[size]["llama_moe_q4k"] = measure(lambda b: synth.build_engine(ms, cap, on_device=True, device=local, max_seqs=b, rope_mode="absolute"), 32000)
         if llama:
             for tag, typ in (("llama_f16", lc.TYPE_F16), ("llama_q4k", lc.TYPE_Q4_K)):
                 ls = synth.ModelSpec(size + tag, len(pattern), sh["width"], sh["heads"], sh["heads"], sh["ff"], 32000, 10000.0, typ, typ, typ)
@@ -857,6 +873,8 @@ def main():
     ap.add_argument("--layered-sizes", default="1b,7b", help="--only layered: which sizes")
     ap.add_argument("--layered-batches", default="1,16,64", help="--only layered: sequences per decode step")
     ap.add_argument("--layered-pattern", default="", help="--only layered: one letter per layer (d = gated delta rule, a = latent attention)")
+    ap.add_argument("--layered-designs", default="varasun", help="--only layered: which designs (varasun,tenetar)")
+    ap.add_argument("--tenetar-pattern", default="", help="--only layered: one letter per Tenetar layer (d = dense feed-forward, m = mixture, s = mixture on the last own cache)")
     ap.add_argument("--no-llama", action="store_true", help="--only layered: skip the Llama-shaped models")
     ap.add_argument("--tp", type=int, default=8, help="--only tp-ranks: ranks the model is cut over")
     ap.add_argument("--profile-range", action="store_true", help="bracket the timed decode loop with cudaProfilerStart/Stop")
@@ -900,7 +918,8 @@ def main():
         from leafcutterllm_b200 import synth
         lc._capi.check(lc.load().lc_set_device(0))
         print(json.dumps(layered_leg(lc, synth, 0, sizes=tuple(args.layered_sizes.split(",")), prompt_len=args.prompt_len, steps=min(args.steps, 32),
-                                     batches=tuple(int(v) for v in args.layered_batches.split(",")), llama=not args.no_llama, pattern=args.layered_pattern)))
+                                     batches=tuple(int(v) for v in args.layered_batches.split(",")), llama=not args.no_llama, pattern=args.layered_pattern,
+                                     designs=tuple(args.layered_designs.split(",")), tenetar_pattern=args.tenetar_pattern)))
     elif args.only == "tcgen05-probe":
         import ctypes as C
         import leafcutterllm_b200 as lc

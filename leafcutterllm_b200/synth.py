@@ -101,12 +101,12 @@ LLAMA70B = ModelSpec("llama3-70b-shape-q4_k", 80, 8192, 64, 8, 28672, 128256, 50
 
 @dataclass
 class LayeredSpec:
-    """A checkpoint-directory model: the parsed config.json (architecture "Varasun") with the ranks that only the tensors'
-    shapes give (decay_rank, gate_rank), for random weights."""
+    """A checkpoint-directory model: the parsed config.json with the ranks that only the tensors' shapes give (Varasun:
+    decay_rank, gate_rank), for random weights."""
     name: str
     config: dict
-    decay_rank: int
-    gate_rank: int
+    decay_rank: int = 0
+    gate_rank: int = 0
 
     @property
     def vocab_size(self) -> int:
@@ -124,8 +124,20 @@ class LayeredSpec:
         for i, ly in enumerate(c["layers"]):
             m, p = ly["mixer"], f"l{i}.mix."
             H, D, E = m["heads"], m["dim"], m["vdim"]
-            yield vec(f"l{i}.norm1", W)
-            if ly["type"] == "channel_delta":
+            both = ("", "b") if c["architecture"] == "Tenetar" else ("",)  # norms on inputs and outputs, or on outputs only
+            for end in both:
+                yield vec(f"l{i}.norm1{end}", W)
+            if ly["type"] == "attention":
+                G = m["kv_heads"]
+                yield mat(p + "q", H * D, W)
+                yield vec(p + "q.norm", H * D)
+                if "kv_from" not in m:
+                    yield mat(p + "k", G * D, W)
+                    yield vec(p + "k.norm", G * D)
+                    yield mat(p + "v", G * E, W)
+                yield vec(p + "sink", H)
+                yield mat(p + "o", W, H * E)
+            elif ly["type"] == "channel_delta":
                 nk = m["kv_heads"] * D
                 for t, n in (("q", nk), ("k", nk), ("v", H * E)):
                     yield mat(p + t, n, W)
@@ -149,11 +161,28 @@ class LayeredSpec:
                 yield mat(p + "uk", H * D, C_)
                 yield mat(p + "uv", H * E, C_)
                 yield mat(p + "o", W, H * E)
-            if ly["mlp"] is not None:
-                F = ly["mlp"]["ff"]
-                yield vec(f"l{i}.norm2", W)
-                yield mat(f"l{i}.mlp.up", F, W)
-                yield mat(f"l{i}.mlp.down", W, F)
+            mlp, p = ly["mlp"], f"l{i}.mlp."
+            if mlp is None:
+                continue
+            for end in both:
+                yield vec(f"l{i}.norm2{end}", W)
+            if mlp["kind"] == "moe":
+                r, F, SF = mlp["router"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+                n = r["experts"] + r["identity"]
+                yield mat(p + "router", n, W)
+                yield vec(p + "correction", n, "normal")
+                for e in range(r["experts"]):
+                    yield mat(f"{p}e{e}.up", F, W)
+                    yield mat(f"{p}e{e}.down", W, F)
+                yield mat(p + "shared.up", SF, W)
+                yield mat(p + "shared.down", W, SF)
+                yield mat(p + "shared.sg", 1, W)
+                continue
+            F = mlp["ff"]
+            if c["architecture"] == "Tenetar":
+                yield mat(p + "gate", F, W)
+            yield mat(p + "up", F, W)
+            yield mat(p + "down", W, F)
         yield vec("final.norm", W)
         yield mat("head", c["vocab"], W)
 
@@ -169,6 +198,24 @@ def layered_spec(name: str, width: int, pattern: str, ff: int, vocab: int, heads
                "mlp": {"kind": "dense", "ff": ff}} for ch in pattern]
     config = {"architecture": "Varasun", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "logit_scale": 1.0, "logit_softcap": 30.0, "layers": layers}
     return LayeredSpec(name, config, low_rank, low_rank)
+
+
+def tenetar_spec(name: str, width: int, pattern: str, ff: int, vocab: int, heads: int, kv_heads: int, experts: int, identity: int, top: int, groups: int,
+                 keep: int, expert_ff: int, shared_ff: int, head_dim: int = 128, window: int = 1024, keep_first: int = 16) -> LayeredSpec:
+    """pattern: one letter per layer, d = dense feed-forward, m = mixture, s = mixture, keys and values of the last layer that has
+    its own."""
+    layers, own = [], 0
+    for i, ch in enumerate(pattern):
+        mixer = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+                 "rot": {"dims": head_dim, "base": 10000.0}, "mask": {"size": window, "keep_first": keep_first}}
+        if ch == "s":
+            mixer["kv_from"] = own
+        else:
+            own = i
+        moe = {"kind": "moe", "expert": {"ff": expert_ff}, "shared": {"ff": shared_ff},
+               "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": groups, "keep": keep}}}
+        layers.append({"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff} if ch == "d" else moe})
+    return LayeredSpec(name, {"architecture": "Tenetar", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5}, "layers": layers})
 
 
 def build_layered_engine(spec: LayeredSpec, seed: int = WEIGHT_SEED, **engine_kwargs):

@@ -37,6 +37,82 @@ def config(layers, width=104, vocab=131, eps=1e-5, logit_scale=0.7, softcap=12.0
             "layers": layers}
 
 
+def attention(heads=6, kv_heads=3, dim=20, vdim=12, rot_dims=8, base=10000.0, scale=0.3, window=37, keep_first=5, kv_from=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "rot": {"dims": rot_dims, "base": base},
+         "mask": {"size": window, "keep_first": keep_first}}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": None}
+
+
+def with_experts(layer, experts=10, identity=2, top=3, groups=3, keep=2, ff=24, shared_ff=20):
+    return dict(layer, mlp={"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared_ff},
+                            "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": groups, "keep": keep}}})
+
+
+def tenetar_config(layers, width=104, vocab=131, eps=1e-5, embed_scale=3.0):
+    return {"architecture": "Tenetar", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": embed_scale}, "layers": layers}
+
+
+def tenetar_weights(cfg, seed=0, fixed_choice=False, correction=0.1):
+    """Random weights, already rounded to bf16.  fixed_choice: corrections far larger than any score, so that the rounding of
+    bf16 activations cannot change which experts are chosen (their weights still follow the token)."""
+    rng = np.random.default_rng(seed)
+    W = cfg["width"]
+    w = {}
+
+    def mat(name, n, k, gain=1.0):
+        w[name] = rng.normal(0, gain / np.sqrt(k), (n, k))
+
+    def gain(name, n):
+        w[name] = rng.normal(1, 0.2, n)
+
+    w["embed"] = rng.normal(0, 0.4, (cfg["vocab"], W))
+    for i, ly in enumerate(cfg["layers"]):
+        m, l, p = ly["mixer"], "l%d." % i, "l%d.mix." % i
+        H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        for n in ("norm1", "norm1b"):
+            gain(l + n, W)
+        mat(p + "q", H * D, W)
+        gain(p + "q.norm", H * D)
+        if m.get("kv_from") is None:
+            mat(p + "k", G * D, W)
+            gain(p + "k.norm", G * D)
+            mat(p + "v", G * E, W)
+        w[p + "sink"] = rng.normal(1.0, 1.0, H)
+        mat(p + "o", W, H * E)
+        mlp, p = ly["mlp"], l + "mlp."
+        if mlp is None:
+            continue
+        for n in ("norm2", "norm2b"):
+            gain(l + n, W)
+        if mlp["kind"] == "dense":
+            mat(p + "gate", mlp["ff"], W)
+            mat(p + "up", mlp["ff"], W)
+            mat(p + "down", W, mlp["ff"])
+            continue
+        r, F, SF = mlp["router"], mlp["expert"]["ff"], mlp["shared"]["ff"]
+        n = r["experts"] + r.get("identity", 0)
+        mat(p + "router", n, W, 1.5)
+        w[p + "correction"] = rng.permutation(n) * 2.0 - n if fixed_choice else rng.normal(-correction, correction, n)
+        for e in range(r["experts"]):
+            mat(p + "e%d.up" % e, F, W, 2.0)
+            mat(p + "e%d.down" % e, W, F, 2.0)
+        mat(p + "shared.up", SF, W)
+        mat(p + "shared.down", W, SF)
+        mat(p + "shared.sg", 1, W)
+    gain("final.norm", W)
+    mat("head", cfg["vocab"], W, 2.0)
+    return {n: bf16_round(a) for n, a in w.items()}
+
+
+def tenetar_mixed():
+    """Windows of several sizes, shared caches (also under a wider window than their owner's), every kind of feed-forward."""
+    return tenetar_config([with_ff(attention(), 40), with_experts(attention(heads=4, kv_heads=1, dim=16, vdim=24, rot_dims=16, window=18, keep_first=0)),
+                           with_experts(attention(heads=8, kv_heads=1, dim=16, vdim=24, rot_dims=16, window=50, keep_first=21, kv_from=1), experts=5, identity=3, top=4, groups=4, keep=3, ff=31),
+                           attention(window=1000, keep_first=0, kv_from=0), with_ff(attention(window=9, keep_first=2, kv_from=0), 17)])
+
+
 def weights(cfg, seed=0, decay_rank=5, gate_rank=7, spread=1.0):
     """Random weights, already rounded to bf16.  Products keep about unit size; decays range from slow to fast."""
     rng = np.random.default_rng(seed)

@@ -64,6 +64,85 @@ def test_yarn_leaves_fast_pairs_and_slows_slow_ones():
     assert (f1 <= f0 + 1e-15).all() and (f1 >= f0 / 4.0 - 1e-15).all()
 
 
+@pytest.mark.parametrize("cuts", [[1] * 60, [2, 5, 1, 9, 6, 37], [58, 2]])
+def test_plain_tenetar_in_portions_equals_the_whole(cuts):
+    cfg = U.tenetar_mixed()
+    m = P.plain_model(cfg, U.tenetar_weights(cfg))
+    toks = U.tokens(60, cfg["vocab"])
+    whole = m.forward(toks, m.new_state())
+    st, parts, at = m.new_state(), [], 0
+    for c in cuts:
+        parts.append(m.forward(toks[at : at + c], st))
+        at += c
+    assert np.abs(np.concatenate(parts) - whole).max() < 1e-10
+
+
+def test_window_and_kept_tokens_by_definition():
+    seen = P.visible([0, 3, 9, 10], 11, 4, 2)
+    assert [np.flatnonzero(r).tolist() for r in seen] == [[0], [0, 1, 2, 3], [0, 1, 6, 7, 8, 9], [0, 1, 7, 8, 9, 10]]
+    assert P.visible([5], 6, 1, 0).sum() == 1 and P.visible([5], 6, 100, 0).all()
+
+
+def test_sink_is_a_key_without_value():
+    """A sink equals one more key whose score is the sink and whose value is zero."""
+    rng = np.random.default_rng(2)
+    q, k, v = rng.normal(size=(3, 2, 4)), rng.normal(size=(5, 1, 4)), rng.normal(size=(5, 1, 6))
+    seen = P.visible([2, 3, 4], 5, 3, 1)
+    got = P.sink_attention(q, k, v, 0.5, seen, np.array([0.3, -1.0]))
+    for h, sink in enumerate([0.3, -1.0]):
+        for t in range(3):
+            s = np.append(np.where(seen[t], k[:, 0] @ q[t, h] * 0.5, -np.inf), sink)
+            p = np.exp(s - s.max())
+            p /= p.sum()
+            assert np.allclose(got[t, h], p[:-1] @ v[:, 0])
+
+
+def test_rotation_of_halves_depends_on_distance_only():
+    rng = np.random.default_rng(6)
+    q, k = rng.normal(size=(1, 1, 10)), rng.normal(size=(1, 1, 10))
+    dots = [float(P.rotate_halves(q, [p + 7], 8, 50.0)[0, 0] @ P.rotate_halves(k, [p], 8, 50.0)[0, 0]) for p in (0, 4, 90)]
+    assert np.allclose(dots, dots[0])
+    r = P.rotate_halves(q, [3], 8, 50.0)[0, 0]
+    assert np.allclose(r[8:], q[0, 0, 8:]) and np.isclose(r[1], q[0, 0, 1] * np.cos(3 * 50.0 ** -0.25) - q[0, 0, 5] * np.sin(3 * 50.0 ** -0.25))
+
+
+def test_choice_of_experts_by_definition():
+    z = np.log(np.array([0.30, 0.02, 0.20, 0.08, 0.25, 0.15]))
+    zero = np.zeros(6)
+    assert [e for e, _ in P.choose_experts(z, zero, 1, 1, 3)] == [0, 4, 2]
+    assert [e for e, _ in P.choose_experts(z, zero, 3, 1, 2)] == [0, 1]
+    picks = P.choose_experts(z, np.array([-0.31, 0, 0, 0, 0, 0]), 1, 1, 2)  # the correction moves the choice, not the weight
+    assert [e for e, _ in picks] == [4, 2] and np.allclose([s for _, s in picks], [0.25, 0.20])
+    low = np.array([-9.0, -9.0, 0, 0, -5.0, -5.0])  # a dropped group loses to negative scores of a kept one
+    assert sorted(e for e, _ in P.choose_experts(z, low, 3, 2, 4)) == [2, 3, 4, 5]
+
+
+def broken_tenetar(change):
+    cfg = copy.deepcopy(U.tenetar_mixed())
+    change(cfg)
+    return cfg
+
+
+@pytest.mark.parametrize("change,text", [
+    (lambda c: c.pop("embedding"), "embedding"),
+    (lambda c: c["layers"][0].update(type="channel_delta"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mixer"].update(kv_heads=4), "key heads"),
+    (lambda c: c["layers"][0]["mixer"]["rot"].update(dims=22), "rotated"),
+    (lambda c: c["layers"][0]["mixer"]["mask"].update(size=0), "size"),
+    (lambda c: c["layers"][2]["mixer"].update(kv_from=2), "earlier"),
+    (lambda c: c["layers"][2]["mixer"].update(kv_from=0), "cannot read"),
+    (lambda c: c["layers"][4]["mixer"].update(kv_from=3), "cannot read"),
+    (lambda c: c["layers"][1]["mlp"]["router"]["groups"].update(count=5), "groups"),
+    (lambda c: c["layers"][1]["mlp"]["router"]["groups"].update(keep=4), "groups"),
+    (lambda c: c["layers"][1]["mlp"]["router"].update(top=9), "top"),
+    (lambda c: c["layers"][1]["mlp"].pop("expert"), "expert"),
+])
+def test_tenetar_config_errors_are_named(lc, change, text):
+    with pytest.raises(lc.LeafcutterError) as e:
+        lc.Engine.from_config(broken_tenetar(change))
+    assert text in str(e.value)
+
+
 def broken(change):
     cfg = copy.deepcopy(mixed_config())
     change(cfg)

@@ -18,11 +18,15 @@ def mixed_config():
                      U.with_ff(U.latent(heads=2, dim=16, rot_dim=8, vdim=24, kv_rank=48, q_rank=20, scaling=None), 56)])
 
 
-@pytest.fixture(scope="module")
-def model():
-    cfg = mixed_config()
-    w = U.weights(cfg, 11)
-    return cfg, w, P.PlainModel(cfg, w)
+@pytest.fixture(scope="module", params=["varasun", "tenetar"])
+def model(request):
+    if request.param == "varasun":
+        cfg = mixed_config()
+        w = U.weights(cfg, 11)
+    else:
+        cfg = U.tenetar_mixed()
+        w = U.tenetar_weights(cfg, 12, fixed_choice=True)
+    return cfg, w, P.plain_model(cfg, w)
 
 
 def run_cut(eng, slot, toks, cuts):
@@ -68,11 +72,17 @@ def test_first_tokens(gpu, model, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_a_call_longer_than_one_pass(gpu, dtype):
+@pytest.mark.parametrize("design", ["varasun", "tenetar"])
+def test_a_call_longer_than_one_pass(gpu, design, dtype):
     """More tokens in one call than a pass takes (2048): the second pass continues from the first one's cache and state."""
-    cfg = U.config([U.delta(heads=1, kv_heads=1, dim=16, vdim=16, conv=4), U.latent(heads=2, dim=8, rot_dim=8, vdim=8, kv_rank=24, q_rank=16)], width=32, vocab=40)
-    w = U.weights(cfg, 3)
-    m = P.PlainModel(cfg, w)
+    if design == "varasun":
+        cfg = U.config([U.delta(heads=1, kv_heads=1, dim=16, vdim=16, conv=4), U.latent(heads=2, dim=8, rot_dim=8, vdim=8, kv_rank=24, q_rank=16)], width=32, vocab=40)
+        w = U.weights(cfg, 3)
+    else:
+        cfg = U.tenetar_config([U.with_experts(U.attention(heads=2, kv_heads=1, dim=8, vdim=8, window=700, keep_first=70), experts=5, identity=1, top=2, groups=2, keep=1),
+                                U.attention(heads=2, kv_heads=1, dim=8, vdim=8, window=3000, keep_first=0, kv_from=0)], width=32, vocab=40)
+        w = U.tenetar_weights(cfg, 3, fixed_choice=True)
+    m = P.plain_model(cfg, w)
     a, b = U.tokens(1500, 40, 1), U.tokens(703, 40, 2)
     eng = U.engine(gpu, cfg, w, dtype, max_seq_len=2304, max_seqs=2)
     got, _ = eng.step([0, 1], [a, b], [[0, 1499], [546, 547, 548, 549, 702]])
@@ -120,6 +130,25 @@ def test_pages_and_slots_are_used_again(gpu, model, dtype):
         toks = U.tokens(n, cfg["vocab"], 200 + i)
         cuts = portions(n, [int(rng.integers(1, 33)), 1, 2])
         U.check(run_cut(eng, s, toks, cuts), m.forward(toks, m.new_state()), dtype)
+    eng.close()
+
+
+@pytest.mark.parametrize("sizes", [[260], [1], [2, 70], [33, 1, 1, 2]])
+def test_choices_that_follow_the_token(gpu, sizes):
+    """Every token its own experts (in 32-bit, where rounding does not move a choice): portions, then other sequences beside it."""
+    cfg = U.tenetar_mixed()
+    w = U.tenetar_weights(cfg, 21)
+    m = P.plain_model(cfg, w)
+    toks = U.tokens(260, cfg["vocab"], 9)
+    want = m.forward(toks, m.new_state())
+    eng = U.engine(gpu, cfg, w, "float32", max_seq_len=272, max_seqs=3)
+    U.check(run_cut(eng, 0, toks, portions(260, sizes)), want, "float32")
+    eng.kv_clear()
+    other = U.tokens(90, cfg["vocab"], 10)
+    beside = m.forward(other, m.new_state())
+    eng.step([1, 2], [other[:40], toks[:100]], [[], []])
+    got, _ = eng.step([2, 1, 0], [toks[100:], other[40:41], toks[:9]], [[0, 159], [0], [8]])
+    U.check(got, np.concatenate([want[[100, 259]], beside[[40]], want[[8]]]), "float32")
     eng.close()
 
 
@@ -222,11 +251,18 @@ def test_long_decoding_and_greedy_generation(gpu, model):
 
 
 @pytest.mark.parametrize("n_seqs", [1, 5, 20, 70])
-def test_decode_batches_of_every_product_form(gpu, n_seqs):
+@pytest.mark.parametrize("design", ["varasun", "tenetar"])
+def test_decode_batches_of_every_product_form(gpu, design, n_seqs):
     """Decode steps whose token count selects different tiles, at contexts on both sides of page and key-tile edges."""
-    cfg = U.config([U.with_ff(U.delta(heads=2, kv_heads=1, dim=64, vdim=64), 136), U.latent(heads=20, dim=32, rot_dim=16, vdim=32, kv_rank=96, q_rank=64)], width=128)
-    w = U.weights(cfg, 4)
-    m = P.PlainModel(cfg, w)
+    if design == "varasun":
+        cfg = U.config([U.with_ff(U.delta(heads=2, kv_heads=1, dim=64, vdim=64), 136), U.latent(heads=20, dim=32, rot_dim=16, vdim=32, kv_rank=96, q_rank=64)], width=128)
+        w = U.weights(cfg, 4)
+    else:
+        cfg = U.tenetar_config([U.with_ff(U.attention(heads=20, kv_heads=2, dim=32, vdim=32, window=64, keep_first=16), 136),
+                                U.with_experts(U.attention(heads=20, kv_heads=2, dim=32, vdim=32, window=150, keep_first=0, kv_from=0), experts=6, identity=2, top=3, groups=4,
+                                               keep=3, ff=130, shared_ff=64)], width=128)
+        w = U.tenetar_weights(cfg, 4, fixed_choice=True)
+    m = P.plain_model(cfg, w)
     eng = U.engine(gpu, cfg, w, "bfloat16", max_seq_len=200, max_seqs=n_seqs)
     lens = [(1, 15, 16, 17, 63, 64, 65, 127, 129)[i % 9] for i in range(n_seqs)]
     toks = [U.tokens(n + 3, cfg["vocab"], 700 + i) for i, n in enumerate(lens)]
@@ -273,12 +309,15 @@ def test_checkpoint_directory_and_trace_runner(gpu, model, tmp_path, monkeypatch
 
 def test_incomplete_models_are_named(gpu, model):
     cfg, w, _ = model
-    for drop, status in (("l1.mix.uk", -6), ("final.norm", -6), ("l0.mix.a1", -6)):
+    tenetar = cfg["architecture"] == "Tenetar"
+    dropped = ("l1.mlp.e3.down", "l2.mlp.correction", "l0.norm1b", "l3.mix.q.norm") if tenetar else ("l1.mix.uk", "l0.mix.a1")
+    for drop, status in [(n, -6) for n in dropped + ("final.norm",)]:
         with pytest.raises(gpu.LeafcutterError) as e:
             U.engine(gpu, cfg, {n: a for n, a in w.items() if n != drop})
         assert e.value.status == status and drop in str(e.value)
     wrong = dict(w)
-    wrong["l1.mix.uv"] = w["l1.mix.uv"][:-1]
+    name = "l2.mlp.e1.up" if tenetar else "l1.mix.uv"
+    wrong[name] = w[name][:-1]
     with pytest.raises(gpu.LeafcutterError) as e:
         U.engine(gpu, cfg, wrong)
-    assert e.value.status == -1 and "l1.mix.uv" in str(e.value)
+    assert e.value.status == -1 and name in str(e.value)
