@@ -12,7 +12,7 @@
 // Few tiles: k is cut into shares over several CTAs; each leaves its partial tile in scratch and takes a ticket, the last one
 // adds the shares in share order (the result does not depend on which CTA that is) and runs the epilogue.
 // Grouped form (one matrix per expert): the tokens come as tiles of rows that share a matrix, found on the device.  Their
-// activations are gathered four rows at a time (TMA gather), the instruction's N follows the tile's rows.
+// activations come in boxes of rows, or are gathered four rows at a time (TMA gather); the instruction's N follows the tile's rows.
 // Work items are dealt round robin to a grid of at most one CTA per SM.  Every wait is bounded: one that runs out raises the
 // library's device error flag and the CTA winds down (copies awaited, tensor memory freed).
 //
@@ -31,6 +31,7 @@ constexpr int kKB = 64;          // elements of k per stage
 constexpr int kABytes = kM * kKB * 2;
 constexpr int kEpiWarps = 8;     // warps 4 .. 11: two per quarter of the rows, each with half of the tokens
 constexpr int kThreads = 128 + 32 * kEpiWarps;
+constexpr int kGatherShare = 24;  // gathers of four rows per stage and issuing warp: a third of 64, rounded up
 
 struct DenseParams {
     void* out;
@@ -51,15 +52,20 @@ struct DenseParams {
 };
 
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
-// ea, eb: the row's constants of the epilogue
+// The epilogue is a template parameter of the kernels; kEpiAny stands for the rarer elementwise ones, told apart at run time.
+constexpr int kEpiAny = -1;
+constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS ? kEpiAny : epi; }
+// ea, eb: the row's constants; `second`: behind the split of DENSE_SPLIT_RELU2
+template <int EPI>
 __device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool second, float ea, float eb, float y) {
-    switch (p.epi) {
-        case DENSE_SPLIT_RELU2: if (!second) return y;  // fall through
-        case DENSE_RELU2: { const float r = fmaxf(y, 0.0f); return r * r; }
-        case DENSE_LOG_DECAY: return -ea * softplus_f(y + eb);
-        case DENSE_LOGITS: { const float v = y * p.scale; return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v; }
-        default: return y;
-    }
+    const float r = fmaxf(y, 0.0f);
+    if constexpr (EPI == DENSE_RELU2) return r * r;
+    else if constexpr (EPI == DENSE_SPLIT_RELU2) return second ? r * r : y;
+    else if constexpr (EPI == kEpiAny) {
+        if (p.epi == DENSE_LOG_DECAY) return -ea * softplus_f(y + eb);
+        const float v = y * p.scale;
+        return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v;
+    } else return y;
 }
 __device__ __forceinline__ void dense_row_constants(const DenseParams& p, int row, float& ea, float& eb) {
     ea = eb = 0.0f;
@@ -68,8 +74,9 @@ __device__ __forceinline__ void dense_row_constants(const DenseParams& p, int ro
 __device__ __forceinline__ float silu_of(float g) { return g / (1.0f + expf(-g)); }
 // 16 accumulators of weight row `row`, tokens t0 .. t0 + m - 1 (m may exceed 16), for a whole warp (lane = row).  bf16: lane
 // pairs swap halves, so a lane stores two rows of every other token.
+template <int EPI>
 __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int row, int t0, int m, const float (&v)[16], float ea, float eb) {
-    if (p.epi == DENSE_GATED_SILU) {  // even lanes hold gates, odd ones the matching values; each makes every other token's output
+    if constexpr (EPI == DENSE_GATED_SILU) {  // even lanes hold gates, odd ones the matching values; each makes every other token's output
         const bool odd = row & 1;
         const size_t at = (size_t)b * p.out_batch + (size_t)t0 * p.ldo + (row >> 1);
 #pragma unroll
@@ -84,22 +91,22 @@ __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int r
         return;
     }
     // a warp's 32 rows lie on one side of a split
-    const bool second = p.epi == DENSE_SPLIT_RELU2 && row >= p.split;
+    const bool second = EPI == DENSE_SPLIT_RELU2 && row >= p.split;
     const int ldo = second ? p.ldo2 : p.ldo, r = second ? row - p.split : row;
     void* out = second ? p.out2 : p.out;
     const size_t at = (size_t)b * p.out_batch + (size_t)t0 * ldo + r;
-    if (p.epi == DENSE_SPLIT_RELU2 ? !second : p.out_f32) {
+    if (EPI == DENSE_SPLIT_RELU2 ? !second : p.out_f32 != 0) {
         if (row >= p.n) return;
         float* o = (float*)out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * ldo] = dense_epilogue(p, second, ea, eb, v[j]);
+            if (j < m) o[(size_t)j * ldo] = dense_epilogue<EPI>(p, second, ea, eb, v[j]);
     } else if ((p.n & 1) == 0 && (ldo & 1) == 0) {  // row pairs stay inside the matrix and 4-byte aligned
         const bool odd = row & 1;
         __nv_bfloat16* o = (__nv_bfloat16*)out + at - (odd ? 1 : 0);
 #pragma unroll
         for (int j = 0; j < 16; j += 2) {
-            const float x = dense_epilogue(p, second, ea, eb, v[j]), y = dense_epilogue(p, second, ea, eb, v[j + 1]);
+            const float x = dense_epilogue<EPI>(p, second, ea, eb, v[j]), y = dense_epilogue<EPI>(p, second, ea, eb, v[j + 1]);
             const float other = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
             const __nv_bfloat162 pr = odd ? __floats2bfloat162_rn(other, y) : __floats2bfloat162_rn(x, other);
             const int jj = j + (odd ? 1 : 0);
@@ -110,11 +117,11 @@ __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int r
         __nv_bfloat16* o = (__nv_bfloat16*)out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * ldo] = __float2bfloat16_rn(dense_epilogue(p, second, ea, eb, v[j]));
+            if (j < m) o[(size_t)j * ldo] = __float2bfloat16_rn(dense_epilogue<EPI>(p, second, ea, eb, v[j]));
     }
 }
 
-template <int NT, bool GROUPED>
+template <int NT, bool GROUPED, int EPI>
 __global__ void __launch_bounds__(kThreads, NT <= 64 ? 2 : 1)
 dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ CUtensorMap tx, const DenseParams p) {
     constexpr int kBBytes = NT * kKB * 2, kStage = kABytes + kBBytes;
@@ -161,43 +168,48 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
         return r;
     };
     auto block = [&](const Item& r, int kb) { return w + (((size_t)r.b * p.mt + r.m) * p.kblocks + kb) * kABytes; };
-    if (GROUPED && warp == 0) {
+    if (GROUPED && (warp == 0 || (p.lists && (warp == 2 || warp == 3)))) {
+        // rows that lie together: one thread brings boxes of kBoxRows; rows of a list: three warps deal the gathers of four among
+        // themselves, one thread of each issues them
         pdl_wait();
-        const int items = *p.n_tiles * p.mt * p.shares;
+        constexpr int kBoxRows = NT < 32 ? NT : 32;
+        int4* s_rows = (int4*)(tmem_slot + 4) + (warp == 0 ? 0 : warp - 1) * kGatherShare;
+        const int items = *p.n_tiles * p.mt * p.shares, part = warp == 0 ? 0 : warp - 1;
         int issued = 0, st = 0;
         uint32_t phase = 1;
         bool ok = true;
         for (int it = blockIdx.x; it < items && ok; it += gridDim.x) {
             const Item r = item_of(it);
             const unsigned char* wb = block(r, r.k0);
-            const int fours = (r.rows + 3) / 4;
-            int4 rows[2];  // of the gathers lane and lane + 32
-#pragma unroll
-            for (int i = 0; i < 2; i++) {
-                int* q = &rows[i].x;
-#pragma unroll
-                for (int j = 0; j < 4; j++) {
-                    const int at = min((lane + 32 * i) * 4 + j, r.rows - 1);
-                    q[j] = p.lists ? p.lists[(size_t)r.b * p.list_stride + r.first + at] : r.t0 + at;
+            const int fours = (r.rows + 3) / 4, mine = fours > part ? (fours - part + 2) / 3 : 0;
+            if (p.lists && lane < mine) {
+                const int32_t* list = p.lists + (size_t)r.b * p.list_stride + r.first;
+                const int at = (part + 3 * lane) * 4, last = r.rows - 1;
+                s_rows[lane] = make_int4(list[at], list[min(at + 1, last)], list[min(at + 2, last)], list[min(at + 3, last)]);
+            }
+            __syncwarp();
+            if (lane == 0) {
+                const uint32_t tx_bytes = kABytes + (p.lists ? fours * 512 : (r.rows + kBoxRows - 1) / kBoxRows * (kBoxRows * 128));
+                for (int kb = r.k0; kb < r.k1; kb++, wb += kABytes) {
+                    unsigned char* a = smem + (size_t)st * kStage;
+                    if (issued >= p.stages && !mbar_wait(&empty[st], phase)) { ok = false; break; }
+                    if (warp == 0) {
+                        mbar_expect_tx(&full[st], tx_bytes);
+                        bulk_load(a, wb, kABytes, &full[st]);
+                    }
+                    if (p.lists) {
+#pragma unroll 4
+                        for (int i = 0; i < mine; i++) tma_gather4(a + kABytes + (part + 3 * i) * 512, &tx, kb * kKB, s_rows[i], &full[st]);
+                    } else {
+                        for (int i = 0; i < r.rows; i += kBoxRows) tma_load_2d(a + kABytes + i * 128, &tx, kb * kKB, r.t0 + i, &full[st]);
+                    }
+                    issued++;
+                    if (++st == p.stages) { st = 0; phase ^= 1; }
                 }
             }
-            for (int kb = r.k0; kb < r.k1; kb++, wb += kABytes) {
-                unsigned char* a = smem + (size_t)st * kStage;
-                const bool free = issued < p.stages || mbar_wait(&empty[st], phase);
-                if (!__all_sync(0xffffffffu, free)) { ok = false; break; }
-                if (lane == 0) {
-                    mbar_expect_tx(&full[st], kABytes + fours * 512);
-                    bulk_load(a, wb, kABytes, &full[st]);
-                }
-                __syncwarp();
-#pragma unroll
-                for (int i = 0; i < 2; i++)
-                    if (lane + 32 * i < fours) tma_gather4(a + kABytes + (lane + 32 * i) * 512, &tx, kb * kKB, rows[i], &full[st]);
-                issued++;
-                if (++st == p.stages) { st = 0; phase ^= 1; }
-            }
+            ok = __shfl_sync(0xffffffffu, (int)ok, 0) != 0;
         }
-        if (!ok && lane == 0) {
+        if (!ok && warp == 0 && lane == 0) {
             *stop = 1;
             atomicExch(p.error_flag, 11);
             for (int i = max(0, issued - p.stages); i < issued; i++) mbar_wait(&full[i % p.stages], (uint32_t)(i / p.stages) & 1);
@@ -298,7 +310,7 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
                     for (int j = 0; j < 16; j++)
                         if (j < m) part[(size_t)r.share * plane + (size_t)(c + j) * kM + row_in] = v[j];
                 } else {
-                    dense_store16(p, ob, row, t0 + c, r.rows - c, v, ea, eb);
+                    dense_store16<EPI>(p, ob, row, t0 + c, r.rows - c, v, ea, eb);
                 }
             }
             tc_fence_before();
@@ -324,12 +336,19 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
 #pragma unroll
                         for (int j = 0; j < 16; j++) v[j] = 0.0f;
                         const float* ps = part + (size_t)c * kM + row_in;
+                        if (m >= 16) {
 #pragma unroll 2
-                        for (int sh = 0; sh < p.shares; sh++, ps += plane)
+                            for (int sh = 0; sh < p.shares; sh++, ps += plane)
 #pragma unroll
-                            for (int j = 0; j < 16; j++)
-                                if (j < m) v[j] += __ldcg(ps + j * kM);
-                        dense_store16(p, ob, row, t0 + c, r.rows - c, v, ea, eb);
+                                for (int j = 0; j < 16; j++) v[j] += __ldcg(ps + j * kM);
+                        } else {
+#pragma unroll 2
+                            for (int sh = 0; sh < p.shares; sh++, ps += plane)
+#pragma unroll
+                                for (int j = 0; j < 16; j++)
+                                    if (j < m) v[j] += __ldcg(ps + j * kM);
+                        }
+                        dense_store16<EPI>(p, ob, row, t0 + c, r.rows - c, v, ea, eb);
                     }
                 }
             }
@@ -362,6 +381,7 @@ __global__ void tile_kernel(const __nv_bfloat16* __restrict__ src, int n, int k,
 
 // True 32-bit: 64 weight rows x 64 tokens per CTA, 4 x 4 outputs per thread.  Grouped (p.off): blockIdx.z is the expert, the
 // tokens are the rows of its list.
+template <int EPI>
 __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __restrict__ w, int ldw, size_t w_batch, const float* __restrict__ x, int ldx,
                                                         size_t x_batch, int k, const DenseParams p) {
     constexpr int KT = 16;
@@ -406,7 +426,7 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int row = r0 + tr + 16 * j;
-            if (p.epi == DENSE_GATED_SILU) {
+            if constexpr (EPI == DENSE_GATED_SILU) {
                 const float up = __shfl_xor_sync(0xffffffffu, acc[i][j], 1);
                 if (t < T && row < p.n && (row & 1) == 0) ((float*)p.out)[(size_t)(row0 + t) * p.ldo + (row >> 1)] = silu_of(acc[i][j]) * up;
                 continue;
@@ -414,22 +434,33 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
             if (t >= T || row >= p.n) continue;
             float ea, eb;
             dense_row_constants(p, row, ea, eb);
-            if (p.epi == DENSE_SPLIT_RELU2 && row >= p.split) ((float*)p.out2)[(size_t)t * p.ldo2 + row - p.split] = dense_epilogue(p, true, ea, eb, acc[i][j]);
-            else ((float*)p.out)[(p.off ? 0 : (size_t)b * p.out_batch) + (size_t)(row0 + t) * p.ldo + row] = dense_epilogue(p, false, ea, eb, acc[i][j]);
+            if (EPI == DENSE_SPLIT_RELU2 && row >= p.split) ((float*)p.out2)[(size_t)t * p.ldo2 + row - p.split] = dense_epilogue<EPI>(p, true, ea, eb, acc[i][j]);
+            else ((float*)p.out)[(p.off ? 0 : (size_t)b * p.out_batch) + (size_t)(row0 + t) * p.ldo + row] = dense_epilogue<EPI>(p, false, ea, eb, acc[i][j]);
         }
     }
 }
 
-template <int NT, bool GROUPED>
+template <int NT, bool GROUPED, int EPI>
 int32_t launch_umma(const DenseArgs& a, const CUtensorMap& tx, DenseParams p, cudaStream_t s) {
-    const size_t stage = kABytes + (size_t)NT * kKB * 2, fixed = 1024 + 512;
+    const size_t stage = kABytes + (size_t)NT * kKB * 2, fixed = 1024 + 512 + (GROUPED ? 3 * kGatherShare * 16 : 0);
     // few tokens: half of the shared memory, so that the next kernel's first weight boxes travel while this one drains
     p.stages = (int)((NT <= 64 ? kMaxSmem / 2 - 1024 : kMaxSmem) - fixed) / (int)stage;
     const size_t smem = fixed + (size_t)p.stages * stage;
-    LC_CUDA(ensure_smem_limit((const void*)dense_umma_kernel<NT, GROUPED>, smem));
+    LC_CUDA(ensure_smem_limit((const void*)dense_umma_kernel<NT, GROUPED, EPI>, smem));
     const int grid = std::min(p.items, sm_count());
-    LC_CUDA(launch_pdl(dense_umma_kernel<NT, GROUPED>, dim3((unsigned)grid), dim3(kThreads), smem, s, a.w->tiles, tx, p));
+    LC_CUDA(launch_pdl(dense_umma_kernel<NT, GROUPED, EPI>, dim3((unsigned)grid), dim3(kThreads), smem, s, a.w->tiles, tx, p));
     return LC_OK;
+}
+
+template <bool GROUPED, int EPI>
+int32_t launch_tiles(int NT, const DenseArgs& a, const CUtensorMap& tx, const DenseParams& p, cudaStream_t s) {
+    switch (NT) {
+        case 16: return launch_umma<16, GROUPED, EPI>(a, tx, p, s);
+        case 32: return launch_umma<32, GROUPED, EPI>(a, tx, p, s);
+        case 64: return launch_umma<64, GROUPED, EPI>(a, tx, p, s);
+        case 128: return launch_umma<128, GROUPED, EPI>(a, tx, p, s);
+        default: return launch_umma<256, GROUPED, EPI>(a, tx, p, s);
+    }
 }
 
 constexpr size_t kPartialBytes = (size_t)64 << 20;
@@ -511,15 +542,11 @@ int32_t launch_grouped(const DenseArgs& a, DenseWorkspace& ws, DenseParams p, cu
     p.shares = choose_shares(p, ws, g.tile_rows, p.mt * std::min(g.most_tiles, std::min(w.batch, g.most_rows)), room);
     p.items = room * p.shares;
     const CUtensorMap* tx = nullptr;
-    LC_TRY(map_of(ws, {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_rows, 1, 4},
-                  [&](void* b) { return make_bf16_tmap_rows(b, a.x, (uint64_t)w.k, (uint64_t)a.x_rows, (uint64_t)a.ldx); }, &tx));
-    switch (g.tile_rows) {
-        case 16: return launch_umma<16, true>(a, *tx, p, s);
-        case 32: return launch_umma<32, true>(a, *tx, p, s);
-        case 64: return launch_umma<64, true>(a, *tx, p, s);
-        case 128: return launch_umma<128, true>(a, *tx, p, s);
-        default: return launch_umma<256, true>(a, *tx, p, s);
-    }
+    const uint32_t box = a.gather ? 1 : (uint32_t)std::min(32, g.tile_rows);
+    LC_TRY(map_of(ws, {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_rows, box},
+                  [&](void* b) { return make_bf16_tmap_rows(b, a.x, (uint64_t)w.k, (uint64_t)a.x_rows, (uint64_t)a.ldx, box); }, &tx));
+    LC_CHECK(a.epi == DENSE_STORE || a.epi == DENSE_RELU2, LC_ERR_UNSUPPORTED, "grouped product: epilogue %d", (int)a.epi);
+    return a.epi == DENSE_RELU2 ? launch_tiles<true, DENSE_RELU2>(g.tile_rows, a, *tx, p, s) : launch_tiles<true, DENSE_STORE>(g.tile_rows, a, *tx, p, s);
 }
 }  // namespace
 
@@ -536,9 +563,18 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     LC_CHECK((a.epi != DENSE_GATED_SILU || w.n % 2 == 0) && (a.epi != DENSE_SPLIT_RELU2 || (a.split % 32 == 0 && w.batch == 1)), LC_ERR_INVALID, "dense product: epilogue layout");
     LC_CHECK(a.f32 ? w.data != nullptr : w.tiles != nullptr, LC_ERR_STATE, "dense product: the weight is not in the form this product reads");
     if (a.f32) {
-        LC_CUDA(launch_pdl(dense_f32_kernel, dim3((unsigned)((w.n + 63) / 64), (unsigned)((a.T + 63) / 64), (unsigned)w.batch), dim3(256), 0, s, w.data,
-                           w.ld, w.batch_stride, (const float*)a.x, a.ldx, a.x_batch, w.k, p));
-        return LC_OK;
+        const dim3 grid((unsigned)((w.n + 63) / 64), (unsigned)((a.T + 63) / 64), (unsigned)w.batch);
+        auto go = [&](auto kern) -> int32_t {
+            LC_CUDA(launch_pdl(kern, grid, dim3(256), 0, s, w.data, w.ld, w.batch_stride, (const float*)a.x, a.ldx, a.x_batch, w.k, p));
+            return LC_OK;
+        };
+        switch (epi_class(a.epi)) {
+            case DENSE_STORE: return go(dense_f32_kernel<DENSE_STORE>);
+            case DENSE_RELU2: return go(dense_f32_kernel<DENSE_RELU2>);
+            case DENSE_GATED_SILU: return go(dense_f32_kernel<DENSE_GATED_SILU>);
+            case DENSE_SPLIT_RELU2: return go(dense_f32_kernel<DENSE_SPLIT_RELU2>);
+            default: return go(dense_f32_kernel<kEpiAny>);
+        }
     }
     const int sms = sm_count();
     p.kblocks = (w.k + kKB - 1) / kKB;
@@ -566,12 +602,12 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     LC_TRY(map_of(ws, {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_batch, (uint64_t)w.batch, (uint64_t)a.x_rows, (uint64_t)box}, [&](void* b) {
         return make_bf16_tmap_3d(b, a.x, (uint64_t)w.k, (uint64_t)w.batch, (uint64_t)a.x_rows, w.batch > 1 ? a.x_batch : (uint64_t)a.ldx, (uint64_t)a.ldx, kKB, 1, (uint32_t)box);
     }, &tx));
-    switch (NT) {
-        case 16: return launch_umma<16, false>(a, *tx, p, s);
-        case 32: return launch_umma<32, false>(a, *tx, p, s);
-        case 64: return launch_umma<64, false>(a, *tx, p, s);
-        case 128: return launch_umma<128, false>(a, *tx, p, s);
-        default: return launch_umma<256, false>(a, *tx, p, s);
+    switch (epi_class(a.epi)) {
+        case DENSE_STORE: return launch_tiles<false, DENSE_STORE>(NT, a, *tx, p, s);
+        case DENSE_RELU2: return launch_tiles<false, DENSE_RELU2>(NT, a, *tx, p, s);
+        case DENSE_GATED_SILU: return launch_tiles<false, DENSE_GATED_SILU>(NT, a, *tx, p, s);
+        case DENSE_SPLIT_RELU2: return launch_tiles<false, DENSE_SPLIT_RELU2>(NT, a, *tx, p, s);
+        default: return launch_tiles<false, kEpiAny>(NT, a, *tx, p, s);
     }
 }
 

@@ -7,7 +7,10 @@
 //   attn_tiles_kernel   runs of many tokens: 64 consecutive queries of one head over key tiles of 64
 // Both tile kernels walk only tiles that hold a visible key: those of the kept first tokens, then those from the window's
 // lower edge on.  Scores, softmax and sums are f32; the weights enter the second product as two bf16 halves.
-// Cache rows hold the key after norm and rotation, so a layer without projections of its own reads another layer's cache.
+// Cache rows hold the key after norm and rotation, so a layer without projections of its own reads another layer's cache.  The
+// rows of one page and kv head lie together in the form in which shared memory wants them (ldmatrix without bank conflicts): a
+// row of a multiple of 64 elements has its 16-byte chunks at chunk ^ (position & 7), any other row is padded.  So a tile comes
+// with one bulk copy per page for its keys and one for its values.
 #include <algorithm>
 #include <cmath>
 #include "lc_mixers.h"
@@ -41,6 +44,21 @@ __device__ __forceinline__ Tiles tiles_of(const Seen& s, int last, int size) {
     return t;
 }
 
+// Where element i of the cache row of position `pos` lies (swz: 7 or 0).
+__device__ __forceinline__ int cell_of(int i, int pos, int swz) { return (((i >> 3) ^ (pos & swz)) << 3) + (i & 7); }
+// Requests the keys and values of positions key .. key + n - 1 of one kv head (one thread).
+__device__ __forceinline__ void request_rows(const AttnArgs& a, const int32_t* pt, int kvh, int key, int n, bf16* k_dst, bf16* v_dst, uint64_t* bar) {
+    const AttnShape& g = a.g;
+    while (n > 0) {
+        const int page = key / a.page_tokens, slot = key - page * a.page_tokens, take = min(n, a.page_tokens - slot);
+        const size_t row = ((size_t)pt[page] * g.kv_heads + kvh) * a.page_tokens + slot;
+        bulk_load(k_dst, (const bf16*)a.k_cache + row * g.k_pitch, (uint32_t)(take * g.k_pitch * 2), bar);
+        bulk_load(v_dst, (const bf16*)a.v_cache + row * g.v_pitch, (uint32_t)(take * g.v_pitch * 2), bar);
+        key += take; n -= take;
+        k_dst += take * g.k_pitch; v_dst += take * g.v_pitch;
+    }
+}
+
 template <typename A> __device__ __forceinline__ void put4(A* p, float4 v);
 template <> __device__ __forceinline__ void put4<float>(float* p, float4 v) { *(float4*)p = v; }
 template <> __device__ __forceinline__ void put4<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
@@ -71,12 +89,16 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a) {
         return ss;
     };
     float sq = squares(q, nq), sk = own ? squares(k, nk) : 0.0f;
-    sq = block_sum(sq, sh);
-    if (own) sk = block_sum(sk, sh2);
+    sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) sh2[threadIdx.x >> 5] = sk;
+    sq = block_sum_once(sq, sh);  // its barrier publishes the other warps' shares too
+    sk = 0.0f;
+    for (int w = 0; w < 8; w++) sk += sh2[w];
     const float rq = 1.0f / sqrtf(sq / (float)nq + a.eps), rk = own ? 1.0f / sqrtf(sk / (float)nk + a.eps) : 0.0f;
     // items of a head: VEC pairs of the rotated part, then VEC elements of the rest
     const int pairs = half / VEC, per = pairs + (g.dim - g.rot_dims) / VEC, start = blockIdx.y * 256 + threadIdx.x, step = gridDim.y * 256;
-    auto item = [&](const float* x, const float* w, float r, A* dst, int i) {
+    auto item = [&](const float* x, const float* w, float r, A* row, int swz, int i) {
+        auto dst = [&](int c) { return row + cell_of(c, pos, swz); };
         if constexpr (VEC == 4) {
             auto normed = [&](int c) {
                 const float4 u = *(const float4*)(x + c), b = *(const float4*)(w + c);
@@ -84,39 +106,39 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a) {
             };
             if (i < pairs) {
                 const float4 u = normed(4 * i), z = normed(half + 4 * i), cs0 = *(const float4*)(tab + 4 * i), cs1 = *(const float4*)(tab + 4 * i + 2);
-                put4<A>(dst + 4 * i, make_float4(u.x * cs0.x - z.x * cs0.y, u.y * cs0.z - z.y * cs0.w, u.z * cs1.x - z.z * cs1.y, u.w * cs1.z - z.w * cs1.w));
-                put4<A>(dst + half + 4 * i, make_float4(z.x * cs0.x + u.x * cs0.y, z.y * cs0.z + u.y * cs0.w, z.z * cs1.x + u.z * cs1.y, z.w * cs1.z + u.w * cs1.w));
+                put4<A>(dst(4 * i), make_float4(u.x * cs0.x - z.x * cs0.y, u.y * cs0.z - z.y * cs0.w, u.z * cs1.x - z.z * cs1.y, u.w * cs1.z - z.w * cs1.w));
+                put4<A>(dst(half + 4 * i), make_float4(z.x * cs0.x + u.x * cs0.y, z.y * cs0.z + u.y * cs0.w, z.z * cs1.x + u.z * cs1.y, z.w * cs1.z + u.w * cs1.w));
             } else {
                 const int c = g.rot_dims + 4 * (i - pairs);
-                put4<A>(dst + c, normed(c));
+                put4<A>(dst(c), normed(c));
             }
         } else {
             if (i < pairs) {
                 const float u = x[i] * r * w[i], z = x[half + i] * r * w[half + i];
                 const float2 cs = tab[i];
-                dst[i] = to_act<A>(u * cs.x - z * cs.y);
-                dst[half + i] = to_act<A>(z * cs.x + u * cs.y);
+                *dst(i) = to_act<A>(u * cs.x - z * cs.y);
+                *dst(half + i) = to_act<A>(z * cs.x + u * cs.y);
             } else {
                 const int c = g.rot_dims + i - pairs;
-                dst[c] = to_act<A>(x[c] * r * w[c]);
+                *dst(c) = to_act<A>(x[c] * r * w[c]);
             }
         }
     };
     A* qo = (A*)a.q + (size_t)t * g.heads * g.dp;
     for (int i = start; i < g.heads * per; i += step) {
         const int h = i / per;
-        item(q + h * g.dim, a.q_norm + h * g.dim, rq, qo + h * g.dp, i - h * per);
+        item(q + h * g.dim, a.q_norm + h * g.dim, rq, qo + h * g.dp, 0, i - h * per);
     }
     if (!own) return;
     const size_t row0 = (size_t)page * g.kv_heads * a.page_tokens + slot;
     for (int i = start; i < g.kv_heads * per; i += step) {
         const int h = i / per;
-        item(k + h * g.dim, a.k_norm + h * g.dim, rk, (A*)a.k_cache + (row0 + (size_t)h * a.page_tokens) * g.dp, i - h * per);
+        item(k + h * g.dim, a.k_norm + h * g.dim, rk, (A*)a.k_cache + (row0 + (size_t)h * a.page_tokens) * g.k_pitch, g.k_swz, i - h * per);
     }
     const int vper = g.vdim / VEC;
     for (int i = start; i < g.kv_heads * vper; i += step) {
         const int h = i / vper, c = (i - h * vper) * VEC;
-        A* dst = (A*)a.v_cache + (row0 + (size_t)h * a.page_tokens) * g.ep + c;
+        A* dst = (A*)a.v_cache + (row0 + (size_t)h * a.page_tokens) * g.v_pitch + cell_of(c, pos, g.v_swz);
         if constexpr (VEC == 4) put4<A>(dst, *(const float4*)(v + h * g.vdim + c));
         else dst[0] = to_act<A>(v[h * g.vdim + c]);
     }
@@ -148,9 +170,9 @@ __global__ void __launch_bounds__(kPlainThreads) attn_plain_kernel(const AttnArg
         if (i < n) {
             const size_t row = ((size_t)pt[key / a.page_tokens] * g.kv_heads + kvh) * a.page_tokens + key % a.page_tokens;
             s_row[threadIdx.x] = row;
-            const A* kr = (const A*)a.k_cache + row * g.dp;
+            const A* kr = (const A*)a.k_cache + row * g.k_pitch;
             float d = 0.0f;
-            for (int c = 0; c < g.dim; c++) d = fmaf(s_q[c], act_f<A>(kr[c]), d);
+            for (int c = 0; c < g.dim; c++) d = fmaf(s_q[c], act_f<A>(kr[cell_of(c, key, g.k_swz)]), d);
             sc = d * g.scale;
         }
         const float mt = fmaxf(m, block_max(sc, red));
@@ -161,7 +183,10 @@ __global__ void __launch_bounds__(kPlainThreads) attn_plain_kernel(const AttnArg
         const int nk = min(kPlainThreads, n - k0);
         for (int c = threadIdx.x; c < g.vdim; c += kPlainThreads) {
             float o = s_o[c] * corr;
-            for (int j = 0; j < nk; j++) o = fmaf(s_p[j], act_f<A>(((const A*)a.v_cache)[s_row[j] * g.ep + c]), o);
+            for (int j = 0; j < nk; j++) {
+                const int at = k0 + j, key = at < sn.keep ? at : sn.lo + at - sn.keep;
+                o = fmaf(s_p[j], act_f<A>(((const A*)a.v_cache)[s_row[j] * g.v_pitch + cell_of(c, key, g.v_swz)]), o);
+            }
             s_o[c] = o;
         }
         __syncthreads();
@@ -174,24 +199,30 @@ __global__ void __launch_bounds__(kPlainThreads) attn_plain_kernel(const AttnArg
 // A CTA of four warps takes up to 16 query heads of one kv head of one token and a piece of its key tiles (16 keys each); the
 // warps deal the tiles among themselves, each with its own ring of copies in flight and its own running softmax, and meet at
 // the end.  Several pieces: the CTA that finishes last merges them.
-constexpr int kDecKeys = 16, kDecStages = 3, kDecWarps = 4, kMaxPieces = 32;
+constexpr int kPartCells = 12;  // CTAs per SM whose partial sums there is room for
+constexpr int kDecKeys = 16, kDecStages = 2, kDecWarps = 4, kMaxPieces = 32;
 struct AttnParts { float *o, *ml; unsigned* tickets; };  // [token][kv head][row block][piece][16][ep], [..][16][2] (log2 units)
 
 template <int NV>
-__global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnArgs a, const AttnParts pt_out) {
+__global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnArgs a, const AttnParts pt_out, int* error_flag) {
     extern __shared__ __align__(128) unsigned char smem[];
     __shared__ float s_ml[kDecWarps][16][2], s_scale[kMaxPieces][16];
+    __shared__ uint64_t s_full[kDecWarps][kDecStages];
     __shared__ int s_last;
     const AttnShape& g = a.g;
-    const int d16 = (g.dp + 15) & ~15, kp = d16 + 8, rb = kp * 2;
-    constexpr int vp = NV * 8 + 8, vb = vp * 2;
+    const int d16 = (g.dp + 15) & ~15, qp = d16 + 8, qb = qp * 2, kb_row = g.k_pitch * 2, vb_row = g.v_pitch * 2;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
     const int rep = g.heads / g.kv_heads, blocks = (rep + 15) / 16, t = blockIdx.x, kvh = blockIdx.y / blocks, r0 = (blockIdx.y % blocks) * 16, nh = min(16, rep - r0),
               h0 = kvh * rep + r0, pieces = gridDim.z;
-    bf16 *s_q = (bf16*)smem, *s_k = s_q + 16 * kp + (size_t)warp * kDecStages * kDecKeys * (kp + vp), *s_v = s_k + kDecStages * kDecKeys * kp;
+    bf16 *s_q = (bf16*)smem, *s_k = s_q + 16 * qp + (size_t)warp * kDecStages * kDecKeys * (g.k_pitch + g.v_pitch), *s_v = s_k + kDecStages * kDecKeys * g.k_pitch;
+    uint64_t* full = s_full[warp];
+    if (lane == 0) {
+        for (int i = 0; i < kDecStages; i++) mbar_init(&full[i], 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    }
     pdl_launch_dependents();
-    const bf16 zero = __float2bfloat16_rn(0.0f);
-    for (int i = lane; i < kDecStages * kDecKeys * (d16 - g.dp); i += 32) s_k[(i / (d16 - g.dp)) * kp + g.dp + i % (d16 - g.dp)] = zero;
+    __syncwarp();
     pdl_wait();
     const int seq = a.tok_seq[t], pos = a.tok_pos[t];
     const Seen sn = seen_from(g, pos);
@@ -199,61 +230,57 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
     const int per = (tl.n + pieces - 1) / pieces, i0 = blockIdx.z * per, i1 = min(tl.n, i0 + per), mine = i1 > i0 + warp ? (i1 - i0 - warp + kDecWarps - 1) / kDecWarps : 0;
     const int32_t* pt = a.page_table + (size_t)seq * a.pages_per_seq;
     const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), v_sm = smem_u32(s_v);
-    const int kch = g.dp / 8, vch = g.ep / 8;
     auto load = [&](int j) {
-        if (j < mine) {
-            const int tile = tl.at(i0 + warp + j * kDecWarps), key = min(tile * kDecKeys + (lane & 15), pos), st = j % kDecStages;
-            const int row = (pt[key / a.page_tokens] * g.kv_heads + kvh) * a.page_tokens + key % a.page_tokens;
-#pragma unroll
-            for (int p = 0; p < 4; p++) {
-                const int ki = p * 4 + (lane >> 3);
-                const size_t r = (size_t)__shfl_sync(0xffffffffu, row, ki);
-                const bf16 *ks = (const bf16*)a.k_cache + r * g.dp, *vs = (const bf16*)a.v_cache + r * g.ep;
-                const uint32_t kd = k_sm + (uint32_t)((st * kDecKeys + ki) * rb), vd = v_sm + (uint32_t)((st * kDecKeys + ki) * vb);
-                for (int c = lane & 7; c < kch; c += 8) cp16(kd + c * 16, ks + c * 8, 16);
-                for (int c = lane & 7; c < vch; c += 8) cp16(vd + c * 16, vs + c * 8, 16);
-            }
+        if (lane == 0 && j < mine) {
+            const int st = j % kDecStages, key = tl.at(i0 + warp + j * kDecWarps) * kDecKeys, n = min(kDecKeys, pos + 1 - key);
+            mbar_expect_tx(&full[st], (uint32_t)(n * (g.k_pitch + g.v_pitch) * 2));
+            request_rows(a, pt, kvh, key, n, s_k + st * kDecKeys * g.k_pitch, s_v + st * kDecKeys * g.v_pitch, &full[st]);
         }
-        cp_commit();
     };
-    load(0);
-    load(1);
+    for (int j = 0; j < kDecStages; j++) load(j);
     for (int i = tid; i < 16 * (d16 / 8); i += 32 * kDecWarps) {
         const int r = i / (d16 / 8), c = (i - r * (d16 / 8)) * 8;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
         if (r < nh && c < g.dp) v = *(const uint4*)((const bf16*)a.q + ((size_t)t * g.heads + h0 + r) * g.dp + c);
-        *(uint4*)(s_q + r * kp + c) = v;
+        *(uint4*)(s_q + r * qp + c) = v;
     }
     __syncthreads();
     float o[NV][4], m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
 #pragma unroll
     for (int i = 0; i < NV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     const float sc = g.scale * kLog2e;
-    const uint32_t qa = q_sm + (uint32_t)((lane & 15) * rb + (lane >> 4) * 16);
+    const uint32_t qa = q_sm + (uint32_t)((lane & 15) * qb + (lane >> 4) * 16);
+    const int krow = (lane & 7) + ((lane >> 4) << 3), kx = krow & g.k_swz, kc = (lane >> 3) & 1, vx = lane & 15 & g.v_swz, vc = lane >> 4;
     for (int j = 0; j < mine; j++) {
-        load(j + 2);
-        cp_wait<2>();
-        __syncwarp();
         const int st = j % kDecStages, key0 = tl.at(i0 + warp + j * kDecWarps) * kDecKeys;
+        if (!mbar_wait(&full[st], (uint32_t)(j / kDecStages) & 1)) atomicExch(error_flag, 15);
+        if (key0 + kDecKeys > pos + 1) {  // the rows behind the token: their weights are zero, the values have to be finite
+            for (int i = lane; i < (key0 + kDecKeys - pos - 1) * (g.v_pitch / 8); i += 32) *(uint4*)(s_v + (st * kDecKeys + pos + 1 - key0) * g.v_pitch + i * 8) = make_uint4(0u, 0u, 0u, 0u);
+            __syncwarp();
+        }
         float s[2][4];
 #pragma unroll
         for (int i = 0; i < 2; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
-        const uint32_t ka = k_sm + (uint32_t)((st * kDecKeys + (lane & 7) + ((lane >> 4) << 3)) * rb + ((lane >> 3) & 1) * 16);
+        const uint32_t ka = k_sm + (uint32_t)((st * kDecKeys + krow) * kb_row);
 #pragma unroll 4
         for (int k = 0; k < d16 / 16; k++) {
             uint32_t q4[4], kb[4];
             ldsm4(qa + k * 32, q4);
-            ldsm4(ka + k * 32, kb);
+            ldsm4(ka + (uint32_t)(((2 * k + kc) ^ kx) << 4), kb);
             mma_bf16(s[0], q4, kb[0], kb[1]);
             mma_bf16(s[1], q4, kb[2], kb[3]);
         }
+        const bool edge = key0 + kDecKeys > pos + 1 || key0 < sn.lo;
         float mx[2] = {m_run[0], m_run[1]};
 #pragma unroll
         for (int i = 0; i < 2; i++)
 #pragma unroll
             for (int e = 0; e < 4; e++) {
-                const int key = key0 + 8 * i + 2 * t4 + (e & 1);
-                s[i][e] = key <= pos && (key >= sn.lo || key < sn.keep) ? s[i][e] * sc : -INFINITY;
+                s[i][e] *= sc;
+                if (edge) {
+                    const int key = key0 + 8 * i + 2 * t4 + (e & 1);
+                    if (key > pos || (key < sn.lo && key >= sn.keep)) s[i][e] = -INFINITY;
+                }
                 mx[e >> 1] = fmaxf(mx[e >> 1], s[i][e]);
             }
         float corr[2], sum[2] = {0.0f, 0.0f};
@@ -276,28 +303,31 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
 #pragma unroll
         for (int r = 0; r < 2; r++) l_run[r] = l_run[r] * corr[r] + sum[r];  // this lane's share of the row
 #pragma unroll
-        for (int i = 0; i < NV; i++) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
-        const uint32_t va = v_sm + (uint32_t)((st * kDecKeys + (lane & 15)) * vb + (lane >> 4) * 16);
+        for (int r = 0; r < 2; r++) corr[r] = r == 0 || nh > 8 ? corr[r] : 1.0f;
+        if (__any_sync(0xffffffffu, corr[0] != 1.0f || corr[1] != 1.0f))
+#pragma unroll
+            for (int i = 0; i < NV; i++) { o[i][0] *= corr[0]; o[i][1] *= corr[0]; o[i][2] *= corr[1]; o[i][3] *= corr[1]; }
+        const uint32_t va = v_sm + (uint32_t)((st * kDecKeys + (lane & 15)) * vb_row);
 #pragma unroll
         for (int np = 0; np < NV / 2; np++) {
             if (16 * np >= g.ep) break;
             uint32_t b[4];
-            ldsm4t(va + np * 32, b);
+            ldsm4t(va + (uint32_t)(((2 * np + vc) ^ vx) << 4), b);
             mma_bf16(o[2 * np], ph, b[0], b[1]);
             mma_bf16(o[2 * np + 1], ph, b[2], b[3]);
             mma_bf16(o[2 * np], pl, b[0], b[1]);
             mma_bf16(o[2 * np + 1], pl, b[2], b[3]);
         }
         __syncwarp();
+        load(j + kDecStages);
     }
-    cp_wait<0>();
 #pragma unroll
     for (int r = 0; r < 2; r++) {
         l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
         l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
     }
     __syncthreads();  // the copies' buffers become the warps' sums: [warp][16][ep]
-    float* s_o = (float*)(s_q + 16 * kp);
+    float* s_o = (float*)(s_q + 16 * qp);
 #pragma unroll
     for (int r = 0; r < 2; r++) {
         const int row = g8 + 8 * r;
@@ -373,16 +403,20 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
 // ---- runs of many tokens ----------------------------------------------------------------------------------------------------
 constexpr int kKeys = 64;
 template <int NV>
-__global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const AttnTile* __restrict__ tiles) {
+__global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const AttnTile* __restrict__ tiles, int* error_flag) {
     extern __shared__ __align__(128) unsigned char smem[];
+    __shared__ uint64_t full[2];
     const AttnShape& g = a.g;
-    const int d16 = (g.dp + 15) & ~15, kp = d16 + 8, rb = kp * 2;
-    constexpr int vp = NV * 8 + 8, vb = vp * 2;
-    bf16 *s_q = (bf16*)smem, *s_k = s_q + 64 * kp, *s_v = s_k + 2 * kKeys * kp;
+    const int d16 = (g.dp + 15) & ~15, qp = d16 + 8, qb = qp * 2, kb_row = g.k_pitch * 2, vb_row = g.v_pitch * 2;
+    bf16 *s_q = (bf16*)smem, *s_k = s_q + 64 * qp, *s_v = s_k + 2 * kKeys * g.k_pitch;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+    if (tid == 0) {
+        mbar_init(&full[0], 1);
+        mbar_init(&full[1], 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    }
     pdl_launch_dependents();
-    const bf16 zero = __float2bfloat16_rn(0.0f);
-    for (int i = tid; i < 2 * kKeys * (d16 - g.dp); i += 128) s_k[(i / (d16 - g.dp)) * kp + g.dp + i % (d16 - g.dp)] = zero;
     pdl_wait();
     const AttnTile tl = tiles[gridDim.x - 1 - blockIdx.x];  // the tiles with the longest contexts first
     const int h = blockIdx.y, kvh = h / (g.heads / g.kv_heads), last = tl.pos0 + tl.n - 1;
@@ -392,26 +426,24 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
     kt.n = kt.n_first + last / kKeys - kt.base + 1;
     const int32_t* pt = a.page_table + (size_t)tl.seq * a.pages_per_seq;
     const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), v_sm = smem_u32(s_v);
-    const int kch = g.dp / 8, vch = g.ep / 8;
-    auto load = [&](int tile, int buf) {
-#pragma unroll
-        for (int p = 0; p < 4; p++) {
-            const int ki = p * 16 + (tid >> 3), key = min(tile * kKeys + ki, last);
-            const size_t r = ((size_t)pt[key / a.page_tokens] * g.kv_heads + kvh) * a.page_tokens + key % a.page_tokens;
-            const bf16 *ks = (const bf16*)a.k_cache + r * g.dp, *vs = (const bf16*)a.v_cache + r * g.ep;
-            const uint32_t kd = k_sm + (uint32_t)((buf * kKeys + ki) * rb), vd = v_sm + (uint32_t)((buf * kKeys + ki) * vb);
-            for (int c = tid & 7; c < kch; c += 8) cp16(kd + c * 16, ks + c * 8, 16);
-            for (int c = tid & 7; c < vch; c += 8) cp16(vd + c * 16, vs + c * 8, 16);
-        }
-        cp_commit();
+    auto load = [&](int i) {  // warp 0: a lane per 16 keys
+        if (warp != 0 || i >= kt.n) return;
+        const int key0 = kt.at(i) * kKeys, n = min(kKeys, last + 1 - key0), buf = i & 1;
+        if (lane == 0) mbar_expect_tx(&full[buf], (uint32_t)(n * (g.k_pitch + g.v_pitch) * 2));
+        __syncwarp();
+        if (lane * 16 < n) request_rows(a, pt, kvh, key0 + lane * 16, min(16, n - lane * 16), s_k + (buf * kKeys + lane * 16) * g.k_pitch, s_v + (buf * kKeys + lane * 16) * g.v_pitch, &full[buf]);
+        __syncwarp();
     };
-    load(kt.at(0), 0);
+    __syncwarp();
+    load(0);
+    load(1);
     for (int i = tid; i < 64 * (d16 / 8); i += 128) {
         const int r = i / (d16 / 8), c = (i - r * (d16 / 8)) * 8;
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
         if (r < tl.n && c < g.dp) v = *(const uint4*)((const bf16*)a.q + ((size_t)(tl.tok0 + r) * g.heads + h) * g.dp + c);
-        *(uint4*)(s_q + r * kp + c) = v;
+        *(uint4*)(s_q + r * qp + c) = v;
     }
+    __syncthreads();
     float o[NV][4], m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
 #pragma unroll
     for (int i = 0; i < NV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
@@ -419,17 +451,19 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
     const int q0 = warp * 16, pa = tl.pos0 + q0, pb = min(pa + 15, last), qpos[2] = {pa + g8, pa + g8 + 8};
     const int wlo_a = g.window > 0 ? max(0, pa - g.window + 1) : 0, wlo_b = g.window > 0 ? max(0, pb - g.window + 1) : 0;
     const int qlo[2] = {g.window > 0 ? qpos[0] - g.window + 1 : 0, g.window > 0 ? qpos[1] - g.window + 1 : 0};
+    const int krow = (lane & 7) + ((lane >> 4) << 3), kx = krow & g.k_swz, kc = (lane >> 3) & 1, vx = lane & 15 & g.v_swz, vc = lane >> 4;
     for (int i = 0; i < kt.n; i++) {
         const int buf = i & 1, key0 = kt.at(i) * kKeys;
-        if (i + 1 < kt.n) { load(kt.at(i + 1), buf ^ 1); cp_wait<1>(); }
-        else cp_wait<0>();
-        __syncthreads();
+        if (!mbar_wait(&full[buf], (uint32_t)(i >> 1) & 1)) atomicExch(error_flag, 16);
+        if (key0 + kKeys > last + 1) {  // the rows behind the last query: their weights are zero, the values have to be finite
+            for (int c = tid; c < (key0 + kKeys - last - 1) * (g.v_pitch / 8); c += 128) *(uint4*)(s_v + (buf * kKeys + last + 1 - key0) * g.v_pitch + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+            __syncthreads();
+        }
         if (q0 < tl.n && key0 <= pb && (key0 + kKeys > wlo_a || key0 < g.keep_first)) {
             float s[8][4];
 #pragma unroll
             for (int n = 0; n < 8; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.0f;
-            const uint32_t qa = q_sm + (uint32_t)((q0 + (lane & 15)) * rb + (lane >> 4) * 16),
-                           ka = k_sm + (uint32_t)((buf * kKeys + (lane & 7) + ((lane >> 4) << 3)) * rb + ((lane >> 3) & 1) * 16);
+            const uint32_t qa = q_sm + (uint32_t)((q0 + (lane & 15)) * qb + (lane >> 4) * 16), ka = k_sm + (uint32_t)((buf * kKeys + krow) * kb_row);
 #pragma unroll 2
             for (int k = 0; k < d16 / 16; k++) {
                 uint32_t q4[4];
@@ -437,7 +471,7 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
 #pragma unroll
                 for (int n = 0; n < 4; n++) {
                     uint32_t kb[4];
-                    ldsm4(ka + (uint32_t)(16 * n * rb) + k * 32, kb);
+                    ldsm4(ka + (uint32_t)(16 * n * kb_row + (((2 * k + kc) ^ kx) << 4)), kb);
                     mma_bf16(s[2 * n], q4, kb[0], kb[1]);
                     mma_bf16(s[2 * n + 1], q4, kb[2], kb[3]);
                 }
@@ -478,14 +512,14 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
             for (int r = 0; r < 2; r++) l_run[r] = l_run[r] * corr[r] + sum[r];  // this lane's share of the row
 #pragma unroll
             for (int n = 0; n < NV; n++) { o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1]; }
-            const uint32_t va = v_sm + (uint32_t)((buf * kKeys + (lane & 15)) * vb + (lane >> 4) * 16);
+            const uint32_t va = v_sm + (uint32_t)((buf * kKeys + (lane & 15)) * vb_row);
 #pragma unroll
             for (int ks = 0; ks < 4; ks++)
 #pragma unroll
                 for (int np = 0; np < NV / 2; np++) {
                     if (16 * np >= g.ep) break;
                     uint32_t b[4];
-                    ldsm4t(va + (uint32_t)(16 * ks * vb) + np * 32, b);
+                    ldsm4t(va + (uint32_t)(16 * ks * vb_row + (((2 * np + vc) ^ vx) << 4)), b);
                     mma_bf16(o[2 * np], ph[ks], b[0], b[1]);
                     mma_bf16(o[2 * np + 1], ph[ks], b[2], b[3]);
                     mma_bf16(o[2 * np], pl[ks], b[0], b[1]);
@@ -493,6 +527,7 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
                 }
         }
         __syncthreads();
+        load(i + 2);
     }
     const float sink = a.sink ? a.sink[h] * kLog2e : -INFINITY;
 #pragma unroll
@@ -511,17 +546,28 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
 
 int value_tiles(int ep) { return ep <= 32 ? 4 : ep <= 64 ? 8 : ep <= 96 ? 12 : ep <= 128 ? 16 : 32; }
 size_t tokens_smem(const AttnShape& g) {
-    const size_t kp = ((g.dp + 15) & ~15) + 8, vp = value_tiles(g.ep) * 8 + 8;
-    return (16 * kp + (size_t)kDecWarps * std::max((size_t)kDecStages * kDecKeys * (kp + vp), (size_t)16 * g.ep * 2)) * 2;
+    const size_t qp = ((g.dp + 15) & ~15) + 8;
+    return (16 * qp + (size_t)kDecWarps * std::max((size_t)kDecStages * kDecKeys * (g.k_pitch + g.v_pitch), (size_t)16 * g.ep * 2)) * 2;
 }
 size_t tiles_smem(const AttnShape& g) {
-    const size_t kp = ((g.dp + 15) & ~15) + 8, vp = value_tiles(g.ep) * 8 + 8;
-    return (64 * kp + 2 * kKeys * (kp + vp)) * 2;
+    const size_t qp = ((g.dp + 15) & ~15) + 8;
+    return (64 * qp + 2 * kKeys * ((size_t)g.k_pitch + g.v_pitch)) * 2;
 }
-bool tensor_form(const AttnShape& g, bool f32) { return !f32 && g.ep <= 256 && tokens_smem(g) <= kMaxSmem - 4096 && tiles_smem(g) <= kMaxSmem; }
+int pitch_of(int n8, bool f32, int* swz) {
+    const int chunks = n8 / 8;
+    *swz = !f32 && chunks % 8 == 0 ? 7 : 0;
+    if (f32 || *swz) return n8;
+    return chunks % 2 ? n8 + 16 : n8 + 8;  // an odd number of chunks; an odd row is followed by a chunk of zeros, since products take 16 columns
+}
+bool tensor_form(const AttnShape& g, bool f32) { return !f32 && g.ep <= 256 && tokens_smem(g) <= kMaxSmem - 4096 && tiles_smem(g) <= kMaxSmem - 1024; }
 int cells(const AttnShape& g) { return g.kv_heads * ((g.heads / g.kv_heads + 15) / 16); }
 
 }  // namespace
+
+void attn_cache_layout(AttnShape* g, bool f32) {
+    g->k_pitch = pitch_of(g->dp, f32, &g->k_swz);
+    g->v_pitch = pitch_of(g->ep, f32, &g->v_swz);
+}
 
 int32_t launch_attn_prep(const AttnArgs& a, cudaStream_t s) {
     const AttnShape& g = a.g;
@@ -537,8 +583,7 @@ int32_t launch_attn_prep(const AttnArgs& a, cudaStream_t s) {
 }
 
 size_t attn_part_bytes(const AttnShape& g) {
-    // pieces are only cut while all CTAs stay within two per SM
-    return (size_t)2 * sm_count() * 16 * ((size_t)g.ep + 2) * sizeof(float);
+    return (size_t)kPartCells * sm_count() * 16 * ((size_t)g.ep + 2) * sizeof(float);
 }
 
 int32_t launch_attn_tokens(const AttnArgs& a, const AttnScratch& sc, cudaStream_t s) {
@@ -557,18 +602,24 @@ int32_t launch_attn_tokens(const AttnArgs& a, const AttnScratch& sc, cudaStream_
     }
     const int n = cells(g), cap = a.pages_per_seq * a.page_tokens;
     const int span = g.window > 0 ? std::min(cap, g.window) / kDecKeys + 2 + std::min(cap, g.keep_first) / kDecKeys : (cap + kDecKeys - 1) / kDecKeys;  // most tiles of a token
-    int pieces = std::max(1, std::min(std::min(kMaxPieces, 2 * sm_count() / (a.T * n)), (span + kDecWarps - 1) / kDecWarps));
-    if (a.T * n > sc.n_tickets) pieces = 1;
-    while (pieces > 1 && (size_t)a.T * n * pieces * 16 * ((size_t)g.ep + 2) * sizeof(float) > sc.part_bytes) pieces--;
+    // pieces: fewest turns of a warp over the waves of CTAs (a CTA's start and end cost about four), merging costs a little more
+    const size_t smem = tokens_smem(g);
+    const int resident = sm_count() * std::max(1, (int)std::min<size_t>(4, (kMaxSmem + 1024) / (smem + 4096)));
+    int pieces = 1;
+    long best = -1;
+    for (int c = 1; c <= std::min(kMaxPieces, (span + kDecWarps - 1) / kDecWarps); c++) {
+        if (c > 1 && (a.T * n > sc.n_tickets || (size_t)a.T * n * c * 16 * ((size_t)g.ep + 2) * sizeof(float) > sc.part_bytes)) break;
+        const long waves = ((long)a.T * n * c + resident - 1) / resident, cost = waves * (((span + c - 1) / c + kDecWarps - 1) / kDecWarps + 4) + (c > 1 ? 3 : 0);
+        if (best < 0 || cost < best) { best = cost; pieces = c; }
+    }
     AttnParts p;
     p.o = sc.part;
     p.ml = sc.part + (size_t)a.T * n * pieces * 16 * g.ep;
     p.tickets = sc.tickets;
-    const size_t smem = tokens_smem(g);
     const dim3 grid((unsigned)a.T, (unsigned)n, (unsigned)pieces);
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(ensure_smem_limit((const void*)kern, smem));
-        LC_CUDA(launch_pdl(kern, grid, dim3(32 * kDecWarps), smem, s, a, p));
+        LC_CUDA(launch_pdl(kern, grid, dim3(32 * kDecWarps), smem, s, a, p, gemv_error_flag_dev()));
         return LC_OK;
     };
     switch (value_tiles(g.ep)) {
@@ -587,7 +638,7 @@ int32_t launch_attn_tiles(const AttnArgs& a, const AttnTile* tiles, int n_tiles,
     const dim3 grid((unsigned)n_tiles, (unsigned)a.g.heads);
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(ensure_smem_limit((const void*)kern, smem));
-        LC_CUDA(launch_pdl(kern, grid, dim3(128), smem, s, a, tiles));
+        LC_CUDA(launch_pdl(kern, grid, dim3(128), smem, s, a, tiles, gemv_error_flag_dev()));
         return LC_OK;
     };
     switch (value_tiles(a.g.ep)) {

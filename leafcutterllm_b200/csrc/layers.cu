@@ -20,6 +20,7 @@ namespace lc {
 namespace {
 
 typedef __nv_bfloat16 bf16;
+constexpr int kGatheredRows = 32;    // experts with larger tiles of rows read a copy in expert order (a gather brings about a row per 14 cycles)
 constexpr int kContextRows = 16384;  // rows of projected keys and values at a time (one longer context is taken whole)
 
 int32_t zalloc(LayerStack& st, void** p, size_t bytes) {
@@ -253,6 +254,7 @@ int32_t bind_attention(lc_model* m, StackLayer& L, const std::string& p) {
     AttnShape& g = L.ag;
     g.heads = s.heads; g.kv_heads = s.kv_heads; g.dim = s.dim; g.vdim = s.vdim; g.dp = round8(s.dim); g.ep = round8(s.vdim); g.rot_dims = s.rot.dims;
     g.scale = s.scale; g.window = s.mask.size; g.keep_first = s.mask.keep_first;
+    attn_cache_layout(&g, st.f32);
     L.ep = g.ep;
     std::vector<int> offs;
     if (s.kv_from < 0) {
@@ -453,7 +455,15 @@ int32_t moe_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, boo
     m->launches_in_call += 1;
     DenseArgs g;
     g.plan = &plan; g.gather = true;
-    LC_TRY(product(m, L.up, x, ldx, T, st.moe_up, ldf, false, DENSE_RELU2, g));
+    const void* in = x;
+    int ld_in = ldx;
+    if (!st.f32 && plan.tile_rows > kGatheredRows) {
+        in = st.moe_in; ld_in = st.width_p;
+        LC_TRY(launch_expert_gather(moe_sum(st, L, x, ldx), st.spec.width, T, st.moe_in, ld_in, m->stream));
+        m->launches_in_call += 1;
+        g.gather = false; g.x_rows = st.moe_slots;
+    }
+    LC_TRY(product(m, L.up, in, ld_in, T, st.moe_up, ldf, false, DENSE_RELU2, g));
     if (e.shared_ff) LC_TRY(product(m, L.shared_down, st.ffn, lds, T, st.y, st.spec.width, true));
     g.gather = false; g.x_rows = st.moe_slots;
     return product(m, L.down, st.moe_up, ldf, T, st.moe_rows, round8(st.spec.width), false, DENSE_STORE, g);
@@ -543,9 +553,9 @@ int32_t stack_alloc(lc_model* m) {
             attn_part = std::max(attn_part, attn_part_bytes(g));
             if (s.kv_from < 0) {
                 const size_t rows = (size_t)m->pages_total * m->page_tokens * g.kv_heads;
-                LC_TRY(zalloc(st, &L.k_cache, rows * g.dp * e));
-                LC_TRY(zalloc(st, &L.v_cache, rows * g.ep * e));
-                st.cache_bytes_per_token += (size_t)g.kv_heads * (g.dp + g.ep) * e;
+                LC_TRY(zalloc(st, &L.k_cache, rows * g.k_pitch * e));
+                LC_TRY(zalloc(st, &L.v_cache, rows * g.v_pitch * e));
+                st.cache_bytes_per_token += (size_t)g.kv_heads * (g.k_pitch + g.v_pitch) * e;
             }
         } else {
             const LatentShape& g = L.lg;
@@ -577,6 +587,7 @@ int32_t stack_alloc(lc_model* m) {
         LC_TRY(zalloc(st, (void**)&st.moe_sel, T * top * 4)); LC_TRY(zalloc(st, (void**)&st.moe_pos, T * top * 4));
         LC_TRY(zalloc(st, (void**)&st.moe_counts, ((size_t)experts + 1) * 4));
         LC_TRY(zalloc(st, &st.moe_up, (size_t)st.moe_slots * hidden * e)); LC_TRY(zalloc(st, &st.moe_rows, (size_t)st.moe_slots * st.width_p * e));
+        if (!st.f32) LC_TRY(zalloc(st, &st.moe_in, (size_t)st.moe_slots * st.width_p * e));
         LC_TRY(zalloc(st, (void**)&st.plan.tiles, (size_t)st.plan_tiles * sizeof(ExpertTile))); LC_TRY(zalloc(st, (void**)&st.plan.n_tiles, 4));
         LC_TRY(zalloc(st, (void**)&st.plan.off, ((size_t)experts + 1) * 4)); LC_TRY(zalloc(st, (void**)&st.plan.lists, (size_t)experts * T * 4));
         st.plan.list_stride = (int)T;
@@ -585,7 +596,7 @@ int32_t stack_alloc(lc_model* m) {
     }
     if (attn_part) {
         st.attn.part_bytes = attn_part;
-        st.attn.n_tickets = 2 * sm_count();
+        st.attn.n_tickets = 12 * sm_count();
         LC_TRY(zalloc(st, (void**)&st.attn.part, attn_part)); LC_TRY(zalloc(st, (void**)&st.attn.tickets, (size_t)st.attn.n_tickets * 4));
         LC_TRY(zalloc(st, (void**)&st.d_attn_tiles, T * sizeof(AttnTile)));
     }

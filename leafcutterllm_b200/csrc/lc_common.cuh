@@ -83,6 +83,15 @@ __device__ __forceinline__ float block_sum(float v, float* sh) {
     __syncthreads();
     return sh[0];
 }
+// The same with one barrier, for a `sh` that the block uses once: every thread adds the warps' sums, in order.
+__device__ __forceinline__ float block_sum_once(float v, float* sh) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float r = 0.0f;
+    for (unsigned w = 0; w < (blockDim.x + 31) / 32; w++) r += sh[w];
+    return r;
+}
 __device__ __forceinline__ float block_max(float v, float* sh) {
     v = warp_max(v);
     int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;

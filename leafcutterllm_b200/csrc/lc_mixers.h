@@ -225,12 +225,14 @@ bool latent_prefill_applies(const LatentShape& g, int ep, bool f32);
 int32_t launch_latent_gather(const LatentArgs& a, const LatentContext* ctx, int n_ctx, int longest, void* out, cudaStream_t s);
 int32_t launch_latent_prefill(const LatentArgs& a, const LatentPrefill& p, int n_tiles, cudaStream_t s);
 
-// ---- gqa_attention.cu: attention over the keys and values of a paged cache, [page][kv head][page_tokens][dp] and [..][ep] -----
+// ---- gqa_attention.cu: attention over the keys and values of a paged cache, [page][kv head][page_tokens][pitch] ----------------
 struct AttnShape {
     int heads, kv_heads, dim, vdim, dp, ep, rot_dims;  // dp, ep: dim, vdim rounded up to 8; rotation pairs i with i + rot_dims / 2
     float scale;
     int window, keep_first;                            // MaskSpec
+    int k_pitch, v_pitch, k_swz, v_swz;                // cache rows (attn_cache_layout): elements apart; 7: chunks swizzled by position
 };
+void attn_cache_layout(AttnShape* g, bool f32);
 struct AttnArgs {
     AttnShape g;
     const float* proj = nullptr;       // [T][ld_proj] q | k | v
@@ -271,6 +273,8 @@ struct ChoiceArgs {
     unsigned long long touched_bytes = 0;
 };
 int32_t launch_expert_choice(const ChoiceArgs& a, cudaStream_t s);
+// The bf16 rows m.h of T tokens, each copied to its rows of `out` (expert order, ldo apart).
+int32_t launch_expert_gather(const MoeSum& m, int width, int T, void* out, int ldo, cudaStream_t s);
 
 // ---- a stack of such layers (layers.cu) --------------------------------------------------------------------------------
 struct StackLayer {
@@ -344,7 +348,7 @@ struct LayerStack {
     // mixtures of experts
     float *moe_z = nullptr, *moe_w = nullptr;
     int32_t *moe_sel = nullptr, *moe_pos = nullptr, *moe_counts = nullptr;
-    void *moe_up = nullptr, *moe_rows = nullptr;  // the experts' hidden rows and outputs, in expert order
+    void *moe_up = nullptr, *moe_rows = nullptr, *moe_in = nullptr;  // the experts' hidden rows, outputs and (bf16) inputs, in expert order
     ExpertPlan plan;
     int plan_tiles = 0, moe_slots = 0;  // room of the tile list; rows of moe_up and moe_rows
     void* pieces = nullptr;

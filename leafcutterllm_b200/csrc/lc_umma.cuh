@@ -53,7 +53,7 @@ __device__ __forceinline__ void tmem_free(uint32_t tmem, uint32_t cols) {
 // qgemv.cu: bf16 tensor map of (d0 contiguous elements, d1, d2) with the strides of d1 and d2 in elements, 128-byte swizzle,
 // zero fill; box b0 x b1 x b2 (b0 = 64)
 bool make_bf16_tmap_3d(void* out128, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1, uint64_t s2, uint32_t b0, uint32_t b1, uint32_t b2);
-// the same for rows of k contiguous elements, `stride` apart, box 64 x 1 (for tma_gather4)
-bool make_bf16_tmap_rows(void* out128, const void* base, uint64_t k, uint64_t rows, uint64_t stride);
+// the same for rows of k contiguous elements, `stride` apart, box 64 x box_rows (one row for tma_gather4)
+bool make_bf16_tmap_rows(void* out128, const void* base, uint64_t k, uint64_t rows, uint64_t stride, uint32_t box_rows);
 
 }  // namespace lc

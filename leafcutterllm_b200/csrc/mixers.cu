@@ -74,7 +74,7 @@ __global__ void __launch_bounds__(256) embed_norm_kernel(const bf16* __restrict_
     }
     if (!act) return;
     float r = 1.0f;
-    if (w) r = 1.0f / sqrtf(block_sum(ss, sh) / (float)width + eps);
+    if (w) r = 1.0f / sqrtf(block_sum_once(ss, sh) / (float)width + eps);
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         const float v = (ok ? __bfloat162float(src[c]) * scale : 0.0f) * r;
         act[t * ld_act + c] = to_act<A>(w ? v * w[c] : v);
@@ -156,7 +156,7 @@ __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
             ss = sq4(v, ss);
         }
         if (MOE && !a.x) return;
-        ss = block_sum(ss, sh);
+        ss = block_sum_once(ss, sh);
         const float r = 1.0f / sqrtf(ss / (float)width + a.eps);
         float s2 = 0.0f;
         auto put = [&](int c, float4 yy, float4 xx) {
@@ -174,7 +174,7 @@ __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
         }
         for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < width; c += blockDim.x * 4) put(c, *(const float4*)(yr + c), *(const float4*)(xr + c));
         if (!wn) return;
-        const float r2 = 1.0f / sqrtf(block_sum(s2, sh2) / (float)width + a.eps);
+        const float r2 = 1.0f / sqrtf(block_sum_once(s2, sh2) / (float)width + a.eps);
         auto next = [&](int c, float4 v) {
             const float4 g = *(const float4*)(wn + c);
             store4<A>(ar + c, make_float4(v.x * r2 * g.x, v.y * r2 * g.y, v.z * r2 * g.z, v.w * r2 * g.w));
@@ -198,7 +198,7 @@ __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
             ss = fmaf(v, v, ss);
         }
         if (MOE && !a.x) return;
-        ss = block_sum(ss, sh);
+        ss = block_sum_once(ss, sh);
         const float r = 1.0f / sqrtf(ss / (float)width + a.eps);
         float s2 = 0.0f;
         for (int c = threadIdx.x; c < width; c += blockDim.x) {
@@ -208,7 +208,7 @@ __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
             s2 = fmaf(v, v, s2);
         }
         if (!wn) return;
-        const float r2 = 1.0f / sqrtf(block_sum(s2, sh2) / (float)width + a.eps);
+        const float r2 = 1.0f / sqrtf(block_sum_once(s2, sh2) / (float)width + a.eps);
         for (int c = threadIdx.x; c < width; c += blockDim.x) ar[c] = to_act<A>(xr[c] * r2 * wn[c]);
     }
 }
@@ -229,7 +229,7 @@ __global__ void __launch_bounds__(512) norm_rows_kernel(const float* __restrict_
         ss = fmaf(v[i], v[i], ss);
     }
     for (int c = threadIdx.x + kHeld * blockDim.x; c < width; c += blockDim.x) ss = fmaf(xr[c], xr[c], ss);
-    ss = block_sum(ss, sh);
+    ss = block_sum_once(ss, sh);
     const float r = 1.0f / sqrtf(ss / (float)width + eps);
     A* o = out + (size_t)blockIdx.x * ldo;
 #pragma unroll

@@ -116,11 +116,11 @@ bool make_bf16_tmap_3d(void* out128, const void* base, uint64_t d0, uint64_t d1,
     return r == CUDA_SUCCESS;
 }
 
-bool make_bf16_tmap_rows(void* out128, const void* base, uint64_t k, uint64_t rows, uint64_t stride) {
+bool make_bf16_tmap_rows(void* out128, const void* base, uint64_t k, uint64_t rows, uint64_t stride, uint32_t box_rows) {
     if (!encode_fn() || ((uintptr_t)base % 16) != 0 || stride % 8 != 0) return false;
     cuuint64_t dims[2] = {k, rows};
     cuuint64_t strides[1] = {stride * 2};
-    cuuint32_t box[2] = {64, 1};
+    cuuint32_t box[2] = {64, box_rows};
     cuuint32_t estr[2] = {1, 1};
     CUresult r = encode_fn()((CUtensorMap*)out128, CU_TENSOR_MAP_DATA_TYPE_UINT16, 2, (void*)base, dims, strides, box, estr,
                              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,

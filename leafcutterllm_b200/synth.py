@@ -170,7 +170,7 @@ class LayeredSpec:
                 r, F, SF = mlp["router"], mlp["expert"]["ff"], mlp["shared"]["ff"]
                 n = r["experts"] + r["identity"]
                 yield mat(p + "router", n, W)
-                yield vec(p + "correction", n, "normal")
+                yield vec(p + "correction", n, "zeros")  # random routers are balanced as they are
                 for e in range(r["experts"]):
                     yield mat(f"{p}e{e}.up", F, W)
                     yield mat(f"{p}e{e}.down", W, F)
@@ -223,8 +223,8 @@ def build_layered_engine(spec: LayeredSpec, seed: int = WEIGHT_SEED, **engine_kw
     from .engine import Engine
     eng = Engine.from_config(spec.config, **engine_kwargs)
     for name, typ, dims, kind in spec.tensors():
-        if kind == "ones":
-            eng.set_tensor(name, TYPE_F32, dims, np.ones(int(np.prod(dims)), np.float32))
+        if kind in ("ones", "zeros"):
+            eng.set_tensor(name, TYPE_F32, dims, np.full(int(np.prod(dims)), float(kind == "ones"), np.float32))
         else:
             eng.synth_tensor(name, typ, dims, seed, SIGMA)
     eng.finalize()

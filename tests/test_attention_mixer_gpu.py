@@ -32,9 +32,9 @@ def rows(n, width, seed=0):
     return U.bf16_round(np.random.default_rng(60 + seed).normal(size=(n, width)))
 
 
-def check_portions(gpu, cfg, w, dtype, sizes, slack=1):
+def check_portions(gpu, cfg, w, dtype, sizes, slack=1, page_tokens=16):
     layer, width = cfg["layers"][0], cfg["width"]
-    eng, m = U.engine(gpu, cfg, w, dtype, max_seq_len=512), P.plain_model(cfg, w)
+    eng, m = U.engine(gpu, cfg, w, dtype, max_seq_len=512, kv_page_tokens=page_tokens), P.plain_model(cfg, w)
     x, states, at = rows(sum(sizes), width), [{}], 0
     for n in sizes:
         want = m.attention(0, x[at : at + n].astype(np.float64), states, at)
@@ -48,6 +48,14 @@ def check_portions(gpu, cfg, w, dtype, sizes, slack=1):
 def test_attention_layer(gpu, name, dtype):
     cfg, w = one_layer(*SHAPES[name])
     check_portions(gpu, cfg, w, dtype, (70, 15, 1, 16, 64, 2, 33, 130))  # token by token up to 15 tokens, tiles from 16 on
+
+
+@pytest.mark.parametrize("page_tokens", [1, 5, 8, 24, 64])
+@pytest.mark.parametrize("dims", [(64, 128), (24, 40), (48, 16), (72, 88)])
+def test_pages_and_rows_of_other_sizes(gpu, dims, page_tokens):
+    """Tiles of keys that end inside pages or span several; cache rows that are swizzled, padded or neither."""
+    cfg, w = one_layer(U.attention(heads=4, kv_heads=2, dim=dims[0], vdim=dims[1], rot_dims=16, window=60, keep_first=21, scale=0.1), 64)
+    check_portions(gpu, cfg, w, "bfloat16", (70, 1, 1, 40, 3), page_tokens=page_tokens)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
