@@ -189,6 +189,13 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
             }
             __syncwarp();
             if (lane == 0) {
+                // large tiles leave room for few stages: the weights, which come from memory once, are asked for further ahead
+                constexpr int kAhead = NT >= 128 ? 8 : 0;
+                const bool more = it + (int)gridDim.x < items;
+                const unsigned char* wn = wb;
+                if (kAhead && warp == 0 && more) { const Item q = item_of(it + gridDim.x); wn = block(q, q.k0); }
+                if (kAhead && warp == 0 && it == (int)blockIdx.x)
+                    for (int kb = r.k0 + p.stages; kb < min(r.k0 + kAhead, r.k1); kb++) bulk_prefetch_l2(wb + (size_t)(kb - r.k0) * kABytes, kABytes);
                 const uint32_t tx_bytes = kABytes + (p.lists ? fours * 512 : (r.rows + kBoxRows - 1) / kBoxRows * (kBoxRows * 128));
                 for (int kb = r.k0; kb < r.k1; kb++, wb += kABytes) {
                     unsigned char* a = smem + (size_t)st * kStage;
@@ -196,6 +203,10 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
                     if (warp == 0) {
                         mbar_expect_tx(&full[st], tx_bytes);
                         bulk_load(a, wb, kABytes, &full[st]);
+                        if (kAhead) {
+                            if (kb + kAhead < r.k1) bulk_prefetch_l2(wb + (size_t)kAhead * kABytes, kABytes);
+                            else if (more && kb + kAhead - r.k1 < r.k1 - r.k0) bulk_prefetch_l2(wn + (size_t)(kb + kAhead - r.k1) * kABytes, kABytes);
+                        }
                     }
                     if (p.lists) {
 #pragma unroll 4
@@ -588,7 +599,7 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     long best_nt = -1;
     for (const auto& z : kSizes) {
         const long tiles = (long)p.mt * ((a.T + z.nt - 1) / z.nt) * w.batch, cost = (tiles + sms - 1) / sms * z.t;
-        if (a.T <= 64 ? z.nt >= a.T && best_nt < 0 : z.nt >= 64 && (best_nt < 0 || cost < best_nt)) { best_nt = cost; NT = z.nt; }
+        if (a.T <= 64 ? z.nt >= a.T && best_nt < 0 : z.nt >= 64 && (best_nt < 0 || cost <= best_nt)) { best_nt = cost; NT = z.nt; }
     }
     p.nt = (a.T + NT - 1) / NT;
     const int cells = p.mt * p.nt * w.batch;
