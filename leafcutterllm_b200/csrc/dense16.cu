@@ -31,6 +31,7 @@ constexpr int kKB = 64;          // elements of k per stage
 constexpr int kABytes = kM * kKB * 2;
 constexpr int kEpiWarps = 8;     // warps 4 .. 11: two per quarter of the rows, each with half of the tokens
 constexpr int kThreads = 128 + 32 * kEpiWarps;
+__host__ __device__ constexpr int box_rows(int nt) { return nt > 16 ? nt / 2 : nt; }  // grouped form: rows of a box
 constexpr int kGatherShare = 24;  // gathers of four rows per stage and issuing warp: a third of 64, rounded up
 
 struct DenseParams {
@@ -169,10 +170,10 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
     };
     auto block = [&](const Item& r, int kb) { return w + (((size_t)r.b * p.mt + r.m) * p.kblocks + kb) * kABytes; };
     if (GROUPED && (warp == 0 || (p.lists && (warp == 2 || warp == 3)))) {
-        // rows that lie together: one thread brings boxes of kBoxRows; rows of a list: three warps deal the gathers of four among
+        // rows that lie together: one thread brings one box or two (every copy costs it about a hundred cycles); rows of a list: three warps deal the gathers of four among
         // themselves, one thread of each issues them
         pdl_wait();
-        constexpr int kBoxRows = NT < 32 ? NT : 32;
+        constexpr int kBoxRows = box_rows(NT);
         int4* s_rows = (int4*)(tmem_slot + 4) + (warp == 0 ? 0 : warp - 1) * kGatherShare;
         const int items = *p.n_tiles * p.mt * p.shares, part = warp == 0 ? 0 : warp - 1;
         int issued = 0, st = 0;
@@ -189,30 +190,20 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
             }
             __syncwarp();
             if (lane == 0) {
-                // large tiles leave room for few stages: the weights, which come from memory once, are asked for further ahead
-                constexpr int kAhead = NT >= 128 ? 8 : 0;
-                const bool more = it + (int)gridDim.x < items;
-                const unsigned char* wn = wb;
-                if (kAhead && warp == 0 && more) { const Item q = item_of(it + gridDim.x); wn = block(q, q.k0); }
-                if (kAhead && warp == 0 && it == (int)blockIdx.x)
-                    for (int kb = r.k0 + p.stages; kb < min(r.k0 + kAhead, r.k1); kb++) bulk_prefetch_l2(wb + (size_t)(kb - r.k0) * kABytes, kABytes);
-                const uint32_t tx_bytes = kABytes + (p.lists ? fours * 512 : (r.rows + kBoxRows - 1) / kBoxRows * (kBoxRows * 128));
+                const uint32_t tx_bytes = kABytes + (p.lists ? fours * 512 : (r.rows > kBoxRows ? 2 : 1) * (kBoxRows * 128));
                 for (int kb = r.k0; kb < r.k1; kb++, wb += kABytes) {
                     unsigned char* a = smem + (size_t)st * kStage;
                     if (issued >= p.stages && !mbar_wait(&empty[st], phase)) { ok = false; break; }
                     if (warp == 0) {
                         mbar_expect_tx(&full[st], tx_bytes);
                         bulk_load(a, wb, kABytes, &full[st]);
-                        if (kAhead) {
-                            if (kb + kAhead < r.k1) bulk_prefetch_l2(wb + (size_t)kAhead * kABytes, kABytes);
-                            else if (more && kb + kAhead - r.k1 < r.k1 - r.k0) bulk_prefetch_l2(wn + (size_t)(kb + kAhead - r.k1) * kABytes, kABytes);
-                        }
                     }
                     if (p.lists) {
 #pragma unroll 4
                         for (int i = 0; i < mine; i++) tma_gather4(a + kABytes + (part + 3 * i) * 512, &tx, kb * kKB, s_rows[i], &full[st]);
                     } else {
-                        for (int i = 0; i < r.rows; i += kBoxRows) tma_load_2d(a + kABytes + i * 128, &tx, kb * kKB, r.t0 + i, &full[st]);
+                        tma_load_2d(a + kABytes, &tx, kb * kKB, r.t0, &full[st]);
+                        if (r.rows > kBoxRows) tma_load_2d(a + kABytes + kBoxRows * 128, &tx, kb * kKB, r.t0 + kBoxRows, &full[st]);
                     }
                     issued++;
                     if (++st == p.stages) { st = 0; phase ^= 1; }
@@ -553,7 +544,7 @@ int32_t launch_grouped(const DenseArgs& a, DenseWorkspace& ws, DenseParams p, cu
     p.shares = choose_shares(p, ws, g.tile_rows, p.mt * std::min(g.most_tiles, std::min(w.batch, g.most_rows)), room);
     p.items = room * p.shares;
     const CUtensorMap* tx = nullptr;
-    const uint32_t box = a.gather ? 1 : (uint32_t)std::min(32, g.tile_rows);
+    const uint32_t box = a.gather ? 1 : (uint32_t)box_rows(g.tile_rows);
     LC_TRY(map_of(ws, {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_rows, box},
                   [&](void* b) { return make_bf16_tmap_rows(b, a.x, (uint64_t)w.k, (uint64_t)a.x_rows, (uint64_t)a.ldx, box); }, &tx));
     LC_CHECK(a.epi == DENSE_STORE || a.epi == DENSE_RELU2, LC_ERR_UNSUPPORTED, "grouped product: epilogue %d", (int)a.epi);
