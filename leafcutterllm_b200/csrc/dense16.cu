@@ -170,8 +170,8 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
     };
     auto block = [&](const Item& r, int kb) { return w + (((size_t)r.b * p.mt + r.m) * p.kblocks + kb) * kABytes; };
     if (GROUPED && (warp == 0 || (p.lists && (warp == 2 || warp == 3)))) {
-        // rows that lie together: one thread brings one box or two (every copy costs it about a hundred cycles); rows of a list: three warps deal the gathers of four among
-        // themselves, one thread of each issues them
+        // rows that lie together: one thread brings one box or two (every copy costs it about a hundred cycles); rows of a list:
+        // three warps deal the gathers of four among themselves, one thread of each issues them
         pdl_wait();
         constexpr int kBoxRows = box_rows(NT);
         int4* s_rows = (int4*)(tmem_slot + 4) + (warp == 0 ? 0 : warp - 1) * kGatherShare;
