@@ -73,9 +73,32 @@ def yarn_frequencies(rot):
     return f / sc["factor"] * ramp + f * (1.0 - ramp), 0.1 * math.log(sc["factor"]) + 1.0
 
 
+def wavelength_frequencies(rot):
+    """Per-pair angular frequency when short wavelengths stay, long ones are stretched by `factor`, and those between are blended."""
+    f = rot["base"] ** (-2.0 * np.arange(rot["dims"] // 2) / rot["dims"])
+    sc = rot["scaling"]
+    out = np.zeros_like(f)
+    for i, v in enumerate(f):
+        turns = sc["original"] * v / (2 * math.pi)  # of the pair over the original context
+        if turns > sc["high"]:
+            out[i] = v
+        elif turns < sc["low"]:
+            out[i] = v / sc["factor"]
+        else:
+            keep = (turns - sc["low"]) / (sc["high"] - sc["low"])
+            out[i] = keep * v + (1 - keep) * v / sc["factor"]
+    return out
+
+
+def pair_frequencies(rot):
+    if "high" in rot.get("scaling", {}):
+        return wavelength_frequencies(rot), 1.0
+    return yarn_frequencies(rot)
+
+
 def rotate_pairs(x, pos, rot):
     """Interleaved pairs (2i, 2i + 1) of the first rot.dims entries of the last axis, by the position of the row (axis 0)."""
-    f, mag = yarn_frequencies(rot)
+    f, mag = pair_frequencies(rot)
     a = np.asarray(pos, np.float64)[:, None] * f[None, :]
     cos, sin = np.cos(a) * mag, np.sin(a) * mag
     while cos.ndim < x.ndim:
@@ -290,5 +313,163 @@ class PlainTenetar:
         return linear(norm("final.norm", x), w["head"])
 
 
+# ---- attention beside a linear recurrence, per-layer token inputs, sigmoid-scored mixtures -----------------------------------
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + np.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def capped_attention(q, k, v, scale, first, cap):
+    """Causal softmax attention of H query heads over G key/value heads; scores bounded by cap * tanh(s / cap) unless cap is None."""
+    T, H, G = q.shape[0], q.shape[1], k.shape[1]
+    out = np.zeros((T, H, v.shape[2]))
+    late = np.arange(k.shape[0])[None, :] > (first + np.arange(T))[:, None]
+    for h in range(H):
+        s = q[:, h] @ k[:, h // (H // G)].T * scale
+        if cap is not None:
+            s = cap * np.tanh(s / cap)
+        s[late] = -np.inf
+        e = np.exp(s - s.max(axis=1, keepdims=True))
+        out[:, h] = e / e.sum(axis=1, keepdims=True) @ v[:, h // (H // G)]
+    return out
+
+
+def decayed_sums(q, k, v, decay, state):
+    """One head: state = decay[t] * state + k[t] v[t]^T, read with q[t].  q, k: [T, n]; v: [T, e]; state: [n, e], changed in place."""
+    out = np.zeros_like(v)
+    for t in range(len(v)):
+        state *= decay[t]
+        state += np.outer(k[t], v[t])
+        out[t] = q[t] @ state
+    return out
+
+
+def norm_in_parts(x, parts, eps):
+    """Every one of `parts` equal stretches of a row divided by its own root mean square."""
+    return rms_norm(x.reshape(len(x), parts, -1), eps).reshape(x.shape)
+
+
+def choose_by_sigmoid(z, correction, groups, keep, top):
+    """One token's router logits -> [(expert, weight)]: the groups with the largest sums of two choice scores stay."""
+    s = sigmoid(z)
+    choice = s + correction
+    size = len(z) // groups
+    rank = [np.sort(choice[g * size : (g + 1) * size])[-2:].sum() for g in range(groups)]
+    best = np.argsort(-np.array(rank), kind="stable")[:keep]
+    allowed = [e for e in range(len(z)) if e // size in best]
+    return [(e, s[e]) for e in sorted(allowed, key=lambda e: -choice[e])[:top]]
+
+
+class PlainMunisun:
+    """Layers of two mixers side by side on the same input; norms (weights stored around zero) on both sides of every sublayer; a
+    part of a per-token table joins after the feed-forward."""
+
+    def __init__(self, config, w):
+        self.c = config
+        self.w = {n: np.asarray(a, np.float64) for n, a in w.items()}
+        self.eps = config["norm"]["eps"]
+
+    def new_state(self):
+        return {"pos": 0, "layers": [dict() for _ in self.c["layers"]]}
+
+    def norm(self, name, x):
+        return rms_norm(x, self.eps, 1.0 + self.w[name])
+
+    def attend(self, mx, q, k, v, st, first):
+        st["k"] = np.concatenate([st["k"], k]) if "k" in st else k
+        st["v"] = np.concatenate([st["v"], v]) if "v" in st else v
+        return capped_attention(q, st["k"], st["v"], mx["scale"], first, mx.get("softcap")).reshape(len(q), -1)
+
+    def gated_attention(self, p, mx, x, st, first):
+        """Norms per head ahead of the rotation; an output gate."""
+        T, H, G, D, E, w = len(x), mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"], self.w
+        pos = first + np.arange(T)
+        q = rotate_pairs(rms_norm(linear(x, w[p + "q"]).reshape(T, H, D), self.eps, w[p + "q.norm"]), pos, mx["rot"])
+        k = rotate_pairs(rms_norm(linear(x, w[p + "k"]).reshape(T, G, D), self.eps, w[p + "k.norm"]), pos, mx["rot"])
+        o = self.attend(mx, q, k, linear(x, w[p + "v"]).reshape(T, G, E), st, first)
+        return linear(o * sigmoid(linear(x, w[p + "g"])), w[p + "o"])
+
+    def conv_attention(self, p, mx, x, st, first):
+        """Short convolutions on the projections; norms without weights behind the rotation."""
+        T, H, G, D, E, w = len(x), mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"], self.w
+        pos = first + np.arange(T)
+        u = {}
+        for n in "qkv":
+            y = linear(x, w[p + n])
+            u[n], st["tail." + n] = causal_conv(y, w[p + n + ".conv"], st.get("tail." + n, np.zeros((mx["conv"] - 1, y.shape[1]))))
+        q = rms_norm(rotate_pairs(u["q"].reshape(T, H, D), pos, mx["rot"]), self.eps)
+        k = rms_norm(rotate_pairs(u["k"].reshape(T, G, D), pos, mx["rot"]), self.eps)
+        return linear(self.attend(mx, q, k, u["v"].reshape(T, G, E), st, first), w[p + "o"])
+
+    def state_space(self, p, mx, x, st):
+        T, H, E, N, G, w = len(x), mx["heads"], mx["vdim"], mx["state"], mx["groups"], self.w
+        inner = H * E
+        z = linear(x, w[p + "in"])
+        gate, u, dt = z[:, :inner], z[:, inner : 2 * inner + 2 * G * N], z[:, 2 * inner + 2 * G * N :]
+        if not st:
+            st["tail"], st["S"] = np.zeros((mx["conv"] - 1, u.shape[1])), np.zeros((H, N, E))
+        u, st["tail"] = causal_conv(u, w[p + "conv"], st["tail"])
+        u = silu(u + w[p + "conv.b"])
+        v, b, c = u[:, :inner].reshape(T, H, E), u[:, inner : inner + G * N].reshape(T, G, N), u[:, inner + G * N :].reshape(T, G, N)
+        dt = softplus(dt + w[p + "dt_bias"])
+        y = np.zeros((T, H, E))
+        for h in range(H):
+            g = h // (H // G)
+            decay = np.exp(-np.exp(w[p + "A_log"][h]) * dt[:, h])
+            y[:, h] = decayed_sums(c[:, g], b[:, g], v[:, h] * dt[:, h : h + 1], decay, st["S"][h]) + w[p + "D"][h] * v[:, h]
+        y = norm_in_parts(y.reshape(T, inner) * silu(gate), mx["norm_groups"], self.eps) * w[p + "norm"]
+        return linear(y, w[p + "o"])
+
+    def lightning(self, p, mx, x, st):
+        T, H, D, E, w = len(x), mx["heads"], mx["dim"], mx["vdim"], self.w
+        q, k, v = (silu(linear(x, w[p + n])).reshape(T, H, -1) for n in "qkv")
+        if not st:
+            st["S"] = np.zeros((H, D, E))
+        o = np.zeros((T, H, E))
+        for h in range(H):
+            o[:, h] = decayed_sums(q[:, h], k[:, h], v[:, h], np.full(T, mx["decay"][h]), st["S"][h])
+        o = rms_norm(o.reshape(T, H * E), self.eps, w[p + "norm"]) * sigmoid(linear(x, w[p + "g"]))
+        return linear(o, w[p + "o"])
+
+    def mix(self, i, x, st, first):
+        ly, p, w = self.c["layers"][i], "l%d.mix." % i, self.w
+        m = ly["mixer"]
+        left, right = st.setdefault("left", {}), st.setdefault("right", {})
+        if ly["type"] == "parallel":
+            return m["left_scale"] * self.gated_attention(p + "left.", m["left"], x, left, first) + m["right_scale"] * self.state_space(p + "right.", m["right"], x, right)
+        a, b = self.conv_attention(p + "left.", m["left"], x, left, first), self.lightning(p + "right.", m["right"], x, right)
+        return 0.5 * (rms_norm(a, self.eps, w[p + "left.out"]) + rms_norm(b, self.eps, w[p + "right.out"]))
+
+    def feed_forward(self, i, x):
+        mlp, p, w = self.c["layers"][i]["mlp"], "l%d.mlp." % i, self.w
+        if mlp["kind"] == "dense":
+            return gated_silu(x, w[p + "gate"], w[p + "up"], w[p + "down"])
+        r, y = mlp["router"], np.zeros_like(x)
+        z = linear(x, w[p + "router"])
+        for t in range(len(x)):
+            for e, s in choose_by_sigmoid(z[t], w[p + "correction"], r["groups"]["count"], r["groups"]["keep"], r["top"]):
+                y[t] += s * gated_silu(x[t], w[p + "e%d.gate" % e], w[p + "e%d.up" % e], w[p + "e%d.down" % e])
+        return y
+
+    def token_side(self, i, x, tokens):
+        """What the layer's part of the side table adds to the residual."""
+        p, w, n = "l%d.side." % i, self.w, self.c["token_side"]["dim"]
+        e = w["side.embed"][np.asarray(tokens), i * n : (i + 1) * n]
+        return rms_norm(linear(gelu_tanh(linear(x, w[p + "gate"])) * e, w[p + "proj"]), self.eps, w[p + "norm"])
+
+    def forward(self, tokens, state, trace=None):
+        first, w = state["pos"], self.w
+        x = w["embed"][np.asarray(tokens)] * self.c["embedding"]["scale"]
+        for i, ly in enumerate(self.c["layers"]):
+            l = "l%d." % i
+            x = x + self.norm(l + "norm1b", self.mix(i, self.norm(l + "norm1", x), state["layers"][i], first))
+            if ly["mlp"] is not None:
+                x = x + self.norm(l + "norm2b", self.feed_forward(i, self.norm(l + "norm2", x)))
+            x = x + self.token_side(i, x, tokens)
+            if trace is not None:
+                trace.append(x.copy())
+        state["pos"] = first + len(tokens)
+        return linear(self.norm("final.norm", x), w["head"])
+
+
 def plain_model(config, w):
-    return {"Varasun": PlainModel, "Tenetar": PlainTenetar}[config["architecture"]](config, w)
+    return {"Varasun": PlainModel, "Tenetar": PlainTenetar, "Munisun": PlainMunisun}[config["architecture"]](config, w)
