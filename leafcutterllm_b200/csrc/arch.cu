@@ -11,7 +11,7 @@
 namespace lc {
 
 const char* mixer_name(MixerKind k) {
-    return k == MixerKind::ChannelDelta ? "channel_delta" : k == MixerKind::LatentAttention ? "latent_attention" : "attention";
+    return k == MixerKind::ChannelDelta ? "channel_delta" : k == MixerKind::LatentAttention ? "latent_attention" : k == MixerKind::Attention ? "attention" : "linear_state";
 }
 
 void rotary_frequencies(const RotarySpec& r, std::vector<double>* freq, double* magnitude) {
@@ -19,8 +19,16 @@ void rotary_frequencies(const RotarySpec& r, std::vector<double>* freq, double* 
     freq->assign((size_t)n, 0.0);
     *magnitude = 1.0;
     for (int i = 0; i < n; i++) (*freq)[i] = std::pow(r.base, -2.0 * i / r.dims);
-    if (!r.yarn) return;
     const double pi = 3.14159265358979323846;
+    if (r.scaling == RotaryScaling::None) return;
+    if (r.scaling == RotaryScaling::Wavelength) {
+        for (double& f : *freq) {
+            const double turns = r.original * f / (2.0 * pi);
+            const double keep = turns > r.fast ? 1.0 : turns < r.slow ? 0.0 : (turns - r.slow) / (r.fast - r.slow);
+            f = (1.0 - keep) * f / r.factor + keep * f;
+        }
+        return;
+    }
     auto pair_at = [&](double turns) { return r.dims * std::log(r.original / (2.0 * pi * turns)) / (2.0 * std::log(r.base)); };
     const double lo = std::fmax(std::floor(pair_at(r.fast)), 0.0), hi = std::fmin(std::ceil(pair_at(r.slow)), r.dims - 1.0);
     for (int i = 0; i < n; i++) {
@@ -68,7 +76,8 @@ struct Fields {
     bool has(const char* key) const { const JValue* v = o->get(key); return v && v->kind != JValue::NUL; }
 };
 
-int32_t parse_rotary(const JValue& v, const std::string& where, RotarySpec* out) {
+// scaling: what "scaling" means in the design
+int32_t parse_rotary(const JValue& v, const std::string& where, RotaryScaling scaling, RotarySpec* out) {
     Fields f{&v, where + ".rot"};
     LC_TRY(f.integer("dims", &out->dims, 2));
     LC_CHECK(out->dims % 2 == 0, LC_ERR_INVALID, "config: %s: an odd number of rotated dimensions", f.where.c_str());
@@ -77,24 +86,43 @@ int32_t parse_rotary(const JValue& v, const std::string& where, RotarySpec* out)
         const JValue* sv = f.need("scaling", JValue::OBJ);
         if (!sv) return LC_ERR_INVALID;
         Fields s{sv, f.where + ".scaling"};
-        out->yarn = true;
+        out->scaling = scaling;
+        const bool yarn = scaling == RotaryScaling::Yarn;
         LC_TRY(s.real("factor", &out->factor));
         LC_TRY(s.real("original", &out->original));
-        LC_TRY(s.real("fast", &out->fast));
-        LC_TRY(s.real("slow", &out->slow));
+        LC_TRY(s.real(yarn ? "fast" : "high", &out->fast));
+        LC_TRY(s.real(yarn ? "slow" : "low", &out->slow));
     }
     return LC_OK;
 }
 
-// The constants of plain attention: heads over shared key/value heads, rotation, window, the layer whose cache it reads.
-int32_t parse_attention(const Fields& m, int index, LayerSpec* out) {
-    LC_TRY(m.integer("kv_heads", &out->kv_heads, 1));
+// The sizes that every mixer has.
+int32_t parse_heads(const Fields& m, MixerSpec* out) {
+    LC_TRY(m.integer("heads", &out->heads, 1));
+    LC_TRY(m.integer("vdim", &out->vdim, 1));
+    return LC_OK;
+}
+int32_t parse_sharing(const Fields& m, const char* key, MixerSpec* out) {
+    LC_TRY(m.integer(key, &out->kv_heads, 1));
     LC_CHECK(out->heads % out->kv_heads == 0, LC_ERR_INVALID, "config: %s: %d heads over %d key heads", m.where.c_str(), out->heads, out->kv_heads);
+    return LC_OK;
+}
+
+// The constants of attention: heads over shared key/value heads, rotation, window, the layer whose cache it reads.
+int32_t parse_attention(const Fields& m, int index, RotaryScaling scaling, MixerSpec* out) {
+    out->kind = MixerKind::Attention;
+    LC_TRY(parse_heads(m, out));
+    LC_TRY(m.integer("dim", &out->dim, 1));
+    LC_TRY(parse_sharing(m, "kv_heads", out));
     LC_TRY(m.real("scale", &out->scale));
+    if (m.has("softcap")) {
+        LC_TRY(m.real("softcap", &out->softcap));
+        LC_CHECK(out->softcap > 0.0f, LC_ERR_INVALID, "config: %s: 'softcap' = %g", m.where.c_str(), out->softcap);
+    }
     if (m.has("rot")) {
         const JValue* rot = m.need("rot", JValue::OBJ);
         if (!rot) return LC_ERR_INVALID;
-        LC_TRY(parse_rotary(*rot, m.where, &out->rot));
+        LC_TRY(parse_rotary(*rot, m.where, scaling, &out->rot));
         LC_CHECK(out->rot.dims <= out->dim, LC_ERR_INVALID, "config: %s: %d of %d dimensions rotated", m.where.c_str(), out->rot.dims, out->dim);
     }
     if (m.has("mask")) {
@@ -109,6 +137,88 @@ int32_t parse_attention(const Fields& m, int index, LayerSpec* out) {
     }
     return LC_OK;
 }
+
+int32_t parse_delta(const Fields& m, MixerSpec* out) {
+    out->kind = MixerKind::ChannelDelta;
+    LC_TRY(parse_heads(m, out));
+    LC_TRY(m.integer("dim", &out->dim, 1));
+    LC_TRY(parse_sharing(m, "kv_heads", out));
+    return m.integer("conv", &out->conv_taps, 1);
+}
+
+int32_t parse_latent(const Fields& m, MixerSpec* out) {
+    out->kind = MixerKind::LatentAttention;
+    LC_TRY(parse_heads(m, out));
+    LC_TRY(m.integer("dim", &out->dim, 1));
+    LC_TRY(m.integer("kv_rank", &out->kv_rank, 1));
+    LC_TRY(m.integer("rot_dim", &out->rot_dim, 2));
+    if (m.has("q_rank")) LC_TRY(m.integer("q_rank", &out->q_rank, 1));
+    LC_TRY(m.real("scale", &out->scale));
+    const JValue* rot = m.need("rot", JValue::OBJ);
+    if (!rot) return LC_ERR_INVALID;
+    LC_TRY(parse_rotary(*rot, m.where, RotaryScaling::Yarn, &out->rot));
+    LC_CHECK(out->rot.dims <= out->rot_dim, LC_ERR_INVALID, "config: %s: %d of %d dimensions rotated", m.where.c_str(), out->rot.dims, out->rot_dim);
+    return LC_OK;
+}
+
+int32_t parse_state_space(const Fields& m, MixerSpec* out) {
+    out->kind = MixerKind::LinearState;
+    out->linear = LinearKind::StateSpace;
+    LC_TRY(parse_heads(m, out));
+    LC_TRY(m.integer("state", &out->dim, 1));
+    LC_TRY(parse_sharing(m, "groups", out));
+    LC_TRY(m.integer("conv", &out->conv_taps, 1));
+    LC_TRY(m.integer("norm_groups", &out->norm_parts, 1));
+    LC_CHECK(out->heads * out->vdim % out->norm_parts == 0, LC_ERR_INVALID, "config: %s: %d channels in %d 'norm_groups'", m.where.c_str(), out->heads * out->vdim, out->norm_parts);
+    return LC_OK;
+}
+
+int32_t parse_lightning(const Fields& m, MixerSpec* out) {
+    out->kind = MixerKind::LinearState;
+    out->linear = LinearKind::Constant;
+    LC_TRY(parse_heads(m, out));
+    LC_TRY(m.integer("dim", &out->dim, 1));
+    out->kv_heads = out->heads;
+    const JValue* d = m.need("decay", JValue::ARR);
+    if (!d) return LC_ERR_INVALID;
+    LC_CHECK((int)d->arr.size() == out->heads, LC_ERR_INVALID, "config: %s: %zu values of 'decay' for %d heads", m.where.c_str(), d->arr.size(), out->heads);
+    for (const JValue& v : d->arr) {
+        LC_CHECK(v.kind == JValue::NUM && v.num >= 0.0 && v.num <= 1.0, LC_ERR_INVALID, "config: %s: 'decay' is not in 0 .. 1", m.where.c_str());
+        out->log_decay.push_back((float)std::fmax(std::log(v.num), -1e4));  // far below where exp ends, and still a number
+    }
+    return LC_OK;
+}
+
+// Two mixers side by side; `type` tells which, and how their outputs meet.
+int32_t parse_parallel(const Fields& m, const std::string& type, int index, LayerSpec* out) {
+    Fields left, right;
+    LC_TRY(m.child("left", &left));
+    LC_TRY(m.child("right", &right));
+    MixerSpec& a = out->mix[0];
+    LC_CHECK(!left.has("kv_from"), LC_ERR_UNSUPPORTED, "config: %s: 'kv_from' beside another mixer", left.where.c_str());
+    LC_TRY(parse_attention(left, index, RotaryScaling::Wavelength, &a));
+    a.pairs = AttnPairs::Neighbours;
+    if (type == "parallel") {
+        a.qk_norm = QkNorm::PerHead;
+        a.out_gate = true;
+        LC_TRY(parse_state_space(right, &out->mix[1]));
+        out->combine = Combine::Scaled;
+        LC_TRY(m.real("left_scale", &out->mix_scale[0]));
+        return m.real("right_scale", &out->mix_scale[1]);
+    }
+    a.qk_norm = QkNorm::PerHeadAfter;
+    LC_TRY(left.integer("conv", &a.conv_taps, 1));
+    out->combine = Combine::Normed;
+    return parse_lightning(right, &out->mix[1]);
+}
+
+// What the designs do not share: the types of layers, the kind of feed-forward that "dense" means, how routers work.
+struct Rules {
+    std::initializer_list<const char*> types;
+    FfnKind dense;
+    bool mixtures = false;
+    MoeSpec moe;
+};
 
 int32_t parse_moe(const Fields& p, MoeSpec* out) {
     Fields expert, router;
@@ -125,6 +235,7 @@ int32_t parse_moe(const Fields& p, MoeSpec* out) {
         LC_TRY(g.integer("keep", &out->keep, 1));
     }
     if (p.has("shared")) {
+        LC_CHECK(!out->gated, LC_ERR_UNSUPPORTED, "config: %s: a shared expert beside gated experts", p.where.c_str());
         Fields sh;
         LC_TRY(p.child("shared", &sh));
         LC_TRY(sh.integer("ff", &out->shared_ff, 1));
@@ -137,45 +248,29 @@ int32_t parse_moe(const Fields& p, MoeSpec* out) {
     return LC_OK;
 }
 
-// dense: what "kind": "dense" means in the design
-int32_t parse_layer(const JValue& v, int index, FfnKind dense, std::initializer_list<MixerKind> mixers, LayerSpec* out) {
+int32_t parse_layer(const JValue& v, int index, const Rules& rules, LayerSpec* out) {
     Fields f{&v, "layer " + std::to_string(index)};
     const JValue *type = f.need("type", JValue::STR), *mixer = f.need("mixer", JValue::OBJ);
     if (!type || !mixer) return LC_ERR_INVALID;
-    Fields m{mixer, f.where + ".mixer"};
+    const Fields m{mixer, f.where + ".mixer"};
     bool known = false;
-    for (MixerKind k : mixers)
-        if (type->str == mixer_name(k)) { out->mixer = k; known = true; }
+    for (const char* t : rules.types) known = known || type->str == t;
     LC_CHECK(known, LC_ERR_UNSUPPORTED, "config: %s: unknown mixer type '%s'", f.where.c_str(), type->str.c_str());
-    LC_TRY(m.integer("heads", &out->heads, 1));
-    LC_TRY(m.integer("dim", &out->dim, 1));
-    LC_TRY(m.integer("vdim", &out->vdim, 1));
-    if (out->mixer == MixerKind::ChannelDelta) {
-        LC_TRY(m.integer("kv_heads", &out->kv_heads, 1));
-        LC_TRY(m.integer("conv", &out->conv_taps, 1));
-        LC_CHECK(out->heads % out->kv_heads == 0, LC_ERR_INVALID, "config: %s: %d heads over %d key heads", m.where.c_str(), out->heads, out->kv_heads);
-    } else if (out->mixer == MixerKind::LatentAttention) {
-        LC_TRY(m.integer("kv_rank", &out->kv_rank, 1));
-        LC_TRY(m.integer("rot_dim", &out->rot_dim, 2));
-        if (m.has("q_rank")) LC_TRY(m.integer("q_rank", &out->q_rank, 1));
-        LC_TRY(m.real("scale", &out->scale));
-        const JValue* rot = m.need("rot", JValue::OBJ);
-        if (!rot) return LC_ERR_INVALID;
-        LC_TRY(parse_rotary(*rot, m.where, &out->rot));
-        LC_CHECK(out->rot.dims <= out->rot_dim, LC_ERR_INVALID, "config: %s: %d of %d dimensions rotated", m.where.c_str(), out->rot.dims, out->rot_dim);
-    } else {
-        LC_TRY(parse_attention(m, index, out));
-    }
+    if (type->str == mixer_name(MixerKind::ChannelDelta)) LC_TRY(parse_delta(m, &out->mix[0]));
+    else if (type->str == mixer_name(MixerKind::LatentAttention)) LC_TRY(parse_latent(m, &out->mix[0]));
+    else if (type->str == mixer_name(MixerKind::Attention)) LC_TRY(parse_attention(m, index, RotaryScaling::Yarn, &out->mix[0]));
+    else LC_TRY(parse_parallel(m, type->str, index, out));
     if (f.has("mlp")) {
         Fields p;
         LC_TRY(f.child("mlp", &p));
         const JValue* kind = p.need("kind", JValue::STR);
         if (!kind) return LC_ERR_INVALID;
         if (kind->str == "dense") {
-            out->ffn = dense;
+            out->ffn = rules.dense;
             LC_TRY(p.integer("ff", &out->ff, 1));
-        } else if (kind->str == "moe" && dense == FfnKind::GatedSilu) {
+        } else if (kind->str == "moe" && rules.mixtures) {
             out->ffn = FfnKind::Moe;
+            out->moe = rules.moe;
             LC_TRY(parse_moe(p, &out->moe));
         } else {
             set_error("config: %s: unknown kind '%s'", p.where.c_str(), kind->str.c_str());
@@ -185,7 +280,7 @@ int32_t parse_layer(const JValue& v, int index, FfnKind dense, std::initializer_
     return LC_OK;
 }
 
-int32_t parse_stack(const Fields& f, FfnKind dense, std::initializer_list<MixerKind> mixers, ArchSpec* out) {
+int32_t parse_stack(const Fields& f, const Rules& rules, ArchSpec* out) {
     LC_TRY(f.integer("width", &out->width, 1));
     LC_TRY(f.integer("vocab", &out->vocab, 1));
     const JValue* norm = f.need("norm", JValue::OBJ);
@@ -196,11 +291,12 @@ int32_t parse_stack(const Fields& f, FfnKind dense, std::initializer_list<MixerK
     LC_CHECK(!layers->arr.empty(), LC_ERR_INVALID, "config: no layers");
     for (size_t i = 0; i < layers->arr.size(); i++) {
         LayerSpec ly;
-        LC_TRY(parse_layer(layers->arr[i], (int)i, dense, mixers, &ly));
-        if (ly.kv_from >= 0) {
-            const LayerSpec& src = out->layers[(size_t)ly.kv_from];
-            LC_CHECK(src.mixer == MixerKind::Attention && src.kv_from < 0 && src.kv_heads == ly.kv_heads && src.dim == ly.dim && src.vdim == ly.vdim, LC_ERR_INVALID,
-                     "config: layer %d cannot read the keys and values of layer %d", (int)i, ly.kv_from);
+        LC_TRY(parse_layer(layers->arr[i], (int)i, rules, &ly));
+        const MixerSpec& own = ly.mix[0];
+        if (own.kv_from >= 0) {
+            const MixerSpec& src = out->layers[(size_t)own.kv_from].mix[0];
+            LC_CHECK(src.kind == MixerKind::Attention && src.kv_from < 0 && src.kv_heads == own.kv_heads && src.dim == own.dim && src.vdim == own.vdim, LC_ERR_INVALID,
+                     "config: layer %d cannot read the keys and values of layer %d", (int)i, own.kv_from);
         }
         out->layers.push_back(ly);
     }
@@ -212,7 +308,7 @@ int32_t parse_varasun(const JValue& cfg, ArchSpec* out) {
     Fields f{&cfg, "the model"};
     LC_TRY(f.real("logit_scale", &out->logit_scale));
     LC_TRY(f.real("logit_softcap", &out->logit_softcap));
-    return parse_stack(f, FfnKind::Relu2, {MixerKind::ChannelDelta, MixerKind::LatentAttention}, out);
+    return parse_stack(f, Rules{{"channel_delta", "latent_attention"}, FfnKind::Relu2}, out);
 }
 
 // Tenetar: windowed attention layers, some of which read an earlier layer's keys and values, with gated or mixture
@@ -222,11 +318,27 @@ int32_t parse_tenetar(const JValue& cfg, ArchSpec* out) {
     LC_TRY(f.child("embedding", &e));
     LC_TRY(e.real("scale", &out->embed_scale));
     out->norm_inputs = true;
-    return parse_stack(f, FfnKind::GatedSilu, {MixerKind::Attention}, out);
+    return parse_stack(f, Rules{{"attention"}, FfnKind::GatedSilu, true}, out);
+}
+
+// Munisun: attention and a linear recurrence side by side in every layer, gated or mixture feed-forwards, norms (stored around
+// zero) on both sides of every sublayer, a per-layer input from the token.
+int32_t parse_munisun(const JValue& cfg, ArchSpec* out) {
+    Fields f{&cfg, "the model"}, e, side;
+    LC_TRY(f.child("embedding", &e));
+    LC_TRY(e.real("scale", &out->embed_scale));
+    LC_TRY(f.child("token_side", &side));
+    LC_TRY(side.integer("dim", &out->side_dim, 1));
+    out->norm_inputs = out->norm_one_plus = true;
+    Rules r{{"parallel", "parallel_2"}, FfnKind::GatedSilu, true};
+    r.moe.score = RouterScore::Sigmoid;
+    r.moe.group_top = 2;
+    r.moe.gated = true;
+    return parse_stack(f, r, out);
 }
 
 struct ArchEntry { const char* name; int32_t (*parse)(const JValue&, ArchSpec*); };
-const ArchEntry kRegistry[] = {{"Varasun", parse_varasun}, {"Tenetar", parse_tenetar}};
+const ArchEntry kRegistry[] = {{"Varasun", parse_varasun}, {"Tenetar", parse_tenetar}, {"Munisun", parse_munisun}};
 
 uint32_t safetensors_type(const std::string& dtype) {
     if (dtype == "BF16") return LC_TYPE_BF16;

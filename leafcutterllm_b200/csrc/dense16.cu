@@ -45,7 +45,10 @@ struct DenseParams {
     int out_f32, epi, e_div;
     float scale, cap;
     void* out2;
-    int ldo2, split;
+    int ldo2, split, silu_end;
+    const __nv_bfloat16* table;
+    const int64_t* ids;
+    int table_ld, table_rows;
     // grouped form
     const ExpertTile* tiles;
     const int32_t *n_tiles, *lists, *off;
@@ -55,15 +58,24 @@ struct DenseParams {
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // The epilogue is a template parameter of the kernels; kEpiAny stands for the rarer elementwise ones, told apart at run time.
 constexpr int kEpiAny = -1;
-constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS ? kEpiAny : epi; }
-// ea, eb: the row's constants; `second`: behind the split of DENSE_SPLIT_RELU2
+constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS || epi == DENSE_GELU_TABLE ? kEpiAny : epi; }
+constexpr bool epi_splits(int epi) { return epi == DENSE_SPLIT_RELU2 || epi == DENSE_SPLIT_SILU; }
+__device__ __forceinline__ float silu_of(float g) { return g / (1.0f + expf(-g)); }
+__device__ __forceinline__ float gelu_of(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+// ea, eb: the row's constants; `second`: behind the split of DENSE_SPLIT_*
 template <int EPI>
-__device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool second, float ea, float eb, float y) {
+__device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool second, float ea, float eb, float y, int row, int t) {
     const float r = fmaxf(y, 0.0f);
     if constexpr (EPI == DENSE_RELU2) return r * r;
     else if constexpr (EPI == DENSE_SPLIT_RELU2) return second ? r * r : y;
+    else if constexpr (EPI == DENSE_SPLIT_SILU) return second && row < p.silu_end ? silu_of(y) : y;
     else if constexpr (EPI == kEpiAny) {
         if (p.epi == DENSE_LOG_DECAY) return -ea * softplus_f(y + eb);
+        if (p.epi == DENSE_GELU_TABLE) {
+            if (t >= p.T || row >= p.n) return 0.0f;
+            const int64_t id = p.ids[t];
+            return id >= 0 && id < p.table_rows ? gelu_of(y) * __bfloat162float(p.table[(size_t)id * p.table_ld + row]) : 0.0f;
+        }
         const float v = y * p.scale;
         return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v;
     } else return y;
@@ -72,7 +84,6 @@ __device__ __forceinline__ void dense_row_constants(const DenseParams& p, int ro
     ea = eb = 0.0f;
     if (p.epi == DENSE_LOG_DECAY && row < p.n) { ea = p.e0[row / p.e_div]; eb = p.e1[row]; }
 }
-__device__ __forceinline__ float silu_of(float g) { return g / (1.0f + expf(-g)); }
 // 16 accumulators of weight row `row`, tokens t0 .. t0 + m - 1 (m may exceed 16), for a whole warp (lane = row).  bf16: lane
 // pairs swap halves, so a lane stores two rows of every other token.
 template <int EPI>
@@ -92,22 +103,22 @@ __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int r
         return;
     }
     // a warp's 32 rows lie on one side of a split
-    const bool second = EPI == DENSE_SPLIT_RELU2 && row >= p.split;
+    const bool second = epi_splits(EPI) && row >= p.split;
     const int ldo = second ? p.ldo2 : p.ldo, r = second ? row - p.split : row;
     void* out = second ? p.out2 : p.out;
     const size_t at = (size_t)b * p.out_batch + (size_t)t0 * ldo + r;
-    if (EPI == DENSE_SPLIT_RELU2 ? !second : p.out_f32 != 0) {
+    if (epi_splits(EPI) ? !second : p.out_f32 != 0) {
         if (row >= p.n) return;
         float* o = (float*)out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * ldo] = dense_epilogue<EPI>(p, second, ea, eb, v[j]);
+            if (j < m) o[(size_t)j * ldo] = dense_epilogue<EPI>(p, second, ea, eb, v[j], row, t0 + j);
     } else if ((p.n & 1) == 0 && (ldo & 1) == 0) {  // row pairs stay inside the matrix and 4-byte aligned
         const bool odd = row & 1;
         __nv_bfloat16* o = (__nv_bfloat16*)out + at - (odd ? 1 : 0);
 #pragma unroll
         for (int j = 0; j < 16; j += 2) {
-            const float x = dense_epilogue<EPI>(p, second, ea, eb, v[j]), y = dense_epilogue<EPI>(p, second, ea, eb, v[j + 1]);
+            const float x = dense_epilogue<EPI>(p, second, ea, eb, v[j], row, t0 + j), y = dense_epilogue<EPI>(p, second, ea, eb, v[j + 1], row, t0 + j + 1);
             const float other = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
             const __nv_bfloat162 pr = odd ? __floats2bfloat162_rn(other, y) : __floats2bfloat162_rn(x, other);
             const int jj = j + (odd ? 1 : 0);
@@ -118,7 +129,7 @@ __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int r
         __nv_bfloat16* o = (__nv_bfloat16*)out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * ldo] = __float2bfloat16_rn(dense_epilogue<EPI>(p, second, ea, eb, v[j]));
+            if (j < m) o[(size_t)j * ldo] = __float2bfloat16_rn(dense_epilogue<EPI>(p, second, ea, eb, v[j], row, t0 + j));
     }
 }
 
@@ -436,8 +447,8 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
             if (t >= T || row >= p.n) continue;
             float ea, eb;
             dense_row_constants(p, row, ea, eb);
-            if (EPI == DENSE_SPLIT_RELU2 && row >= p.split) ((float*)p.out2)[(size_t)t * p.ldo2 + row - p.split] = dense_epilogue<EPI>(p, true, ea, eb, acc[i][j]);
-            else ((float*)p.out)[(p.off ? 0 : (size_t)b * p.out_batch) + (size_t)(row0 + t) * p.ldo + row] = dense_epilogue<EPI>(p, false, ea, eb, acc[i][j]);
+            if (epi_splits(EPI) && row >= p.split) ((float*)p.out2)[(size_t)t * p.ldo2 + row - p.split] = dense_epilogue<EPI>(p, true, ea, eb, acc[i][j], row, t);
+            else ((float*)p.out)[(p.off ? 0 : (size_t)b * p.out_batch) + (size_t)(row0 + t) * p.ldo + row] = dense_epilogue<EPI>(p, false, ea, eb, acc[i][j], row, t);
         }
     }
 }
@@ -547,7 +558,8 @@ int32_t launch_grouped(const DenseArgs& a, DenseWorkspace& ws, DenseParams p, cu
     const uint32_t box = a.gather ? 1 : (uint32_t)box_rows(g.tile_rows);
     LC_TRY(map_of(ws, {(uint64_t)(uintptr_t)a.x, (uint64_t)w.k, (uint64_t)a.ldx, (uint64_t)a.x_rows, box},
                   [&](void* b) { return make_bf16_tmap_rows(b, a.x, (uint64_t)w.k, (uint64_t)a.x_rows, (uint64_t)a.ldx, box); }, &tx));
-    LC_CHECK(a.epi == DENSE_STORE || a.epi == DENSE_RELU2, LC_ERR_UNSUPPORTED, "grouped product: epilogue %d", (int)a.epi);
+    LC_CHECK(a.epi == DENSE_STORE || a.epi == DENSE_RELU2 || a.epi == DENSE_GATED_SILU, LC_ERR_UNSUPPORTED, "grouped product: epilogue %d", (int)a.epi);
+    if (a.epi == DENSE_GATED_SILU) return launch_tiles<true, DENSE_GATED_SILU>(g.tile_rows, a, *tx, p, s);
     return a.epi == DENSE_RELU2 ? launch_tiles<true, DENSE_RELU2>(g.tile_rows, a, *tx, p, s) : launch_tiles<true, DENSE_STORE>(g.tile_rows, a, *tx, p, s);
 }
 }  // namespace
@@ -560,9 +572,10 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     p.n = w.n; p.T = a.T; p.ldo = a.ldo; p.batch = w.batch;
     p.out_f32 = a.out_f32 || a.f32; p.epi = a.epi; p.e_div = a.e_div; p.scale = a.scale; p.cap = a.cap;
     p.error_flag = gemv_error_flag_dev();
-    p.out2 = a.out2; p.ldo2 = a.ldo2; p.split = a.split;
+    p.out2 = a.out2; p.ldo2 = a.ldo2; p.split = a.split; p.silu_end = a.silu_end;
+    p.table = a.table; p.table_ld = a.table_ld; p.table_rows = a.table_rows; p.ids = a.ids;
     if (a.plan) { p.tiles = a.plan->tiles; p.n_tiles = a.plan->n_tiles; p.off = a.plan->off; p.lists = a.gather ? a.plan->lists : nullptr; p.list_stride = a.plan->list_stride; }
-    LC_CHECK((a.epi != DENSE_GATED_SILU || w.n % 2 == 0) && (a.epi != DENSE_SPLIT_RELU2 || (a.split % 32 == 0 && w.batch == 1)), LC_ERR_INVALID, "dense product: epilogue layout");
+    LC_CHECK((a.epi != DENSE_GATED_SILU || w.n % 2 == 0) && (!epi_splits(a.epi) || (a.split % 32 == 0 && w.batch == 1)), LC_ERR_INVALID, "dense product: epilogue layout");
     LC_CHECK(a.f32 ? w.data != nullptr : w.tiles != nullptr, LC_ERR_STATE, "dense product: the weight is not in the form this product reads");
     if (a.f32) {
         const dim3 grid((unsigned)((w.n + 63) / 64), (unsigned)((a.T + 63) / 64), (unsigned)w.batch);
@@ -575,6 +588,7 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
             case DENSE_RELU2: return go(dense_f32_kernel<DENSE_RELU2>);
             case DENSE_GATED_SILU: return go(dense_f32_kernel<DENSE_GATED_SILU>);
             case DENSE_SPLIT_RELU2: return go(dense_f32_kernel<DENSE_SPLIT_RELU2>);
+            case DENSE_SPLIT_SILU: return go(dense_f32_kernel<DENSE_SPLIT_SILU>);
             default: return go(dense_f32_kernel<kEpiAny>);
         }
     }
@@ -609,6 +623,7 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
         case DENSE_RELU2: return launch_tiles<false, DENSE_RELU2>(NT, a, *tx, p, s);
         case DENSE_GATED_SILU: return launch_tiles<false, DENSE_GATED_SILU>(NT, a, *tx, p, s);
         case DENSE_SPLIT_RELU2: return launch_tiles<false, DENSE_SPLIT_RELU2>(NT, a, *tx, p, s);
+        case DENSE_SPLIT_SILU: return launch_tiles<false, DENSE_SPLIT_SILU>(NT, a, *tx, p, s);
         default: return launch_tiles<false, kEpiAny>(NT, a, *tx, p, s);
     }
 }

@@ -457,6 +457,7 @@ uint64_t algo_bytes_step(const lc_model* m, const std::vector<int>& ctx_lens) {
         b += (uint64_t)ctx_lens.size() * (m->embed->nbytes / std::max<size_t>(m->embed->rows, 1));
     }
     if (m->stack) {
+        b -= stack_table_bytes(m);  // nor is the side table
         for (int c : ctx_lens) b += stack_step_bytes(m, c);
         return b;
     }
@@ -611,7 +612,7 @@ int32_t lc_model_create_json(const char* config_json, const lc_model_config* ove
     c.hidden_size = stack->spec.width; c.vocab_size = stack->spec.vocab; c.num_layers = (int32_t)stack->spec.layers.size();
     c.rms_eps = stack->spec.eps; c.rope_mode = 1; c.n_experts = 0; c.top_k = 0;
     c.num_heads = c.num_kv_heads = 1; c.intermediate_size = 1;
-    for (const LayerSpec& L : stack->spec.layers) { c.num_heads = std::max(c.num_heads, L.heads); c.intermediate_size = std::max(c.intermediate_size, L.ff); }
+    for (const LayerSpec& L : stack->spec.layers) { c.num_heads = std::max(c.num_heads, L.mix[0].heads); c.intermediate_size = std::max(c.intermediate_size, L.ff); }
     if (c.max_seq_len <= 0) c.max_seq_len = 4096;
     stack->f32 = c.compute_f32 != 0;
     c.kv_dtype = stack->f32 ? 1 : 0;

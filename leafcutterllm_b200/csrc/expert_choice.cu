@@ -1,7 +1,8 @@
 // Routing of a mixture of experts with identity experts and group-limited choice (MoeSpec): from the router's logits to every
 // token's choices and weights, the experts' token lists and the tiles of their grouped products.
-//   s = softmax(z) over all outputs; choice score c = s + correction; the groups (equal runs of outputs) are ranked by their
-//   largest c, the outputs of the best `keep` groups by c, the first `top` of them are chosen and weighted with s.
+//   s = softmax(z) over all outputs, or the sigmoid of each; choice score c = s + correction; the groups (equal runs of outputs)
+//   are ranked by their largest c or the sum of their two largest, the outputs of the best `keep` groups by c, the first `top` of
+//   them are chosen and weighted with s.
 // One warp per token.  The CTA that finishes last (a ticket) turns the experts' counts into offsets and tiles.  The order of
 // tokens inside a list is the order of arrival; nothing that is computed from a list depends on it.
 #include <algorithm>
@@ -37,17 +38,25 @@ __global__ void __launch_bounds__(32 * kWarps) expert_choice_kernel(const Choice
     if (t < a.T) {
         const float* z = a.z + (size_t)t * a.ld_z;
         float mx = -INFINITY, sum = 0.0f;
-        for (int e = lane; e < n; e += 32) { const float v = z[e]; s[e] = v; mx = fmaxf(mx, v); }
-        mx = warp_max(mx);
-        for (int e = lane; e < n; e += 32) { const float v = expf(s[e] - mx); s[e] = v; sum += v; }
-        sum = warp_sum(sum);
-        for (int e = lane; e < n; e += 32) { const float v = s[e] / sum; s[e] = v; c[e] = v + a.correction[e]; }
+        if (m.score == RouterScore::Sigmoid) {
+            for (int e = lane; e < n; e += 32) { const float v = 1.0f / (1.0f + expf(-z[e])); s[e] = v; c[e] = v + a.correction[e]; }
+        } else {
+            for (int e = lane; e < n; e += 32) { const float v = z[e]; s[e] = v; mx = fmaxf(mx, v); }
+            mx = warp_max(mx);
+            for (int e = lane; e < n; e += 32) { const float v = expf(s[e] - mx); s[e] = v; sum += v; }
+            sum = warp_sum(sum);
+            for (int e = lane; e < n; e += 32) { const float v = s[e] / sum; s[e] = v; c[e] = v + a.correction[e]; }
+        }
         __syncwarp();
         if (m.keep < m.groups) {
             for (int g = lane; g < m.groups; g += 32) {
-                float best = -INFINITY;
-                for (int i = 0; i < per; i++) best = fmaxf(best, c[g * per + i]);
-                gs[g] = best;
+                float best = -INFINITY, second = -INFINITY;
+                for (int i = 0; i < per; i++) {
+                    const float v = c[g * per + i];
+                    second = fmaxf(second, fminf(best, v));
+                    best = fmaxf(best, v);
+                }
+                gs[g] = m.group_top == 2 && per > 1 ? best + second : best;
             }
             __syncwarp();
             for (int g = lane; g < m.groups; g += 32) {

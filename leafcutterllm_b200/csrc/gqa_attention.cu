@@ -1,6 +1,7 @@
 // Attention of query heads over shared key/value heads in a paged cache, under a window with kept first tokens (MaskSpec) and
-// with a sink: exp(sink[head]) joins the softmax denominator, without key or value.
+// with a sink: exp(sink[head]) joins the softmax denominator, without key or value.  Scores may be bounded by a tanh, outputs gated.
 //   attn_prep_kernel    RMS norm over all of a token's q and over all of its k, rotation of halves, cache append
+//   attn_head_prep_kernel  the same for norms per head: short convolutions, norm ahead of the rotation or behind it, either pairing
 //   attn_plain_kernel   any shape, f32 arithmetic throughout; models in true 32-bit
 //   attn_tokens_kernel  few tokens per sequence (decode): the query heads of one kv head of one token are the rows of the
 //                       products; every warp walks key tiles of its own
@@ -13,6 +14,7 @@
 // with one bulk copy per page for its keys and one for its values.
 #include <algorithm>
 #include <cmath>
+#include <type_traits>
 #include "lc_mixers.h"
 #include "lc_mma.cuh"
 #include "lc_tma.cuh"
@@ -44,6 +46,19 @@ __device__ __forceinline__ Tiles tiles_of(const Seen& s, int last, int size) {
     return t;
 }
 
+// A score in log2 units, bounded: k.x * tanh(dot * scale / cap) with k = (cap, 2 scale / cap) times log2 e.
+__device__ __forceinline__ float2 cap_constants(const AttnShape& g) { return make_float2(g.cap * kLog2e, g.cap > 0.0f ? 2.0f * g.scale / g.cap * kLog2e : 0.0f); }
+__device__ __forceinline__ float capped(float dot, float2 k) { return k.x - k.x * __fdividef(2.0f, 1.0f + exp2f(dot * k.y)); }
+// The factor on element c of head h of token t's output.
+template <typename A>
+__device__ __forceinline__ float out_factor(const AttnArgs& a, size_t t, int h, int c) {
+    return a.gate && c < a.g.vdim ? a.out_scale * sigmoid_f(act_f<A>(((const A*)a.gate)[t * a.ld_gate + (size_t)h * a.g.vdim + c])) : a.out_scale;
+}
+__device__ __forceinline__ float4 finished(const AttnArgs& a, size_t t, int h, int c, float4 x) {
+    if (!a.gate && a.out_scale == 1.0f) return x;
+    return make_float4(x.x * out_factor<bf16>(a, t, h, c), x.y * out_factor<bf16>(a, t, h, c + 1), x.z * out_factor<bf16>(a, t, h, c + 2), x.w * out_factor<bf16>(a, t, h, c + 3));
+}
+
 // Where element i of the cache row of position `pos` lies (swz: 7 or 0).
 __device__ __forceinline__ int cell_of(int i, int pos, int swz) { return (((i >> 3) ^ (pos & swz)) << 3) + (i & 7); }
 // Requests the keys and values of positions key .. key + n - 1 of one kv head (one thread).
@@ -62,6 +77,9 @@ __device__ __forceinline__ void request_rows(const AttnArgs& a, const int32_t* p
 template <typename A> __device__ __forceinline__ void put4(A* p, float4 v);
 template <> __device__ __forceinline__ void put4<float>(float* p, float4 v) { *(float4*)p = v; }
 template <> __device__ __forceinline__ void put4<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
+template <typename A> __device__ __forceinline__ void put2(A* p, float2 v);
+template <> __device__ __forceinline__ void put2<float>(float* p, float2 v) { *(float2*)p = v; }
+template <> __device__ __forceinline__ void put2<bf16>(bf16* p, float2 v) { *(uint32_t*)p = pack2(v.x, v.y); }
 
 // One CTA per token and share of its elements; VEC = 4: dim, vdim and the rotated half are multiples of four.
 template <typename A, int VEC>
@@ -144,6 +162,157 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a) {
     }
 }
 
+// Norms per head: one warp per (stretch of tokens, head): the heads of q, then of k, then of v.  A lane owns pairs of neighbouring
+// elements, lane + 32 p, and keeps its channels' last inputs while it walks the stretch (TAPS of them; 0: no convolution; -1: any
+// number, re-read).
+template <typename A, int TAPS, int NP>
+__global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, int stretch) {
+    constexpr int kWin = TAPS > 1 ? TAPS - 1 : 1, kTaps = TAPS > 0 ? TAPS : 1;
+    __shared__ float s_x[8][64 * NP];
+    pdl_launch_dependents();
+    pdl_wait();
+    const AttnShape& g = a.g;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.y * 8 + warp;
+    if (unit >= g.heads + 2 * g.kv_heads) return;
+    const bool is_q = unit < g.heads, is_v = unit >= g.heads + g.kv_heads;
+    const int h = is_q ? unit : is_v ? unit - g.heads - g.kv_heads : unit - g.heads, n = is_v ? g.vdim : g.dim, half = g.rot_dims / 2;
+    const int nq = g.heads * g.dim, nk = g.kv_heads * g.dim, channels = nq + nk + g.kv_heads * g.vdim;
+    const int ch0 = (is_q ? 0 : is_v ? nq + nk : nq) + h * n, col0 = (is_q ? 0 : is_v ? a.off_v : a.off_k) + h * n;
+    const int taps = TAPS > 0 ? TAPS : g.taps;
+    const bool even = (n & 1) == 0;  // then pairs are 8-byte aligned
+    auto pair_at = [&](const float* row, int c) {
+        if (c >= n) return make_float2(0.0f, 0.0f);
+        return even ? *(const float2*)(row + c) : make_float2(row[c], c + 1 < n ? row[c + 1] : 0.0f);
+    };
+    const int t0 = blockIdx.x * stretch, t1 = min(a.T, t0 + stretch);
+    float2 w[NP][kTaps], win[NP][kWin], gain[NP];  // win[.][j]: the input j + 1 tokens back
+    const float* gw = is_q ? a.q_norm : a.k_norm;
+#pragma unroll
+    for (int p = 0; p < NP; p++) {
+        const int c = 2 * (lane + 32 * p);
+        if constexpr (TAPS > 0)
+#pragma unroll
+            for (int j = 0; j < TAPS; j++)
+                w[p][j] = make_float2(c < n ? a.conv[(size_t)(ch0 + c) * TAPS + j] : 0.0f, c + 1 < n ? a.conv[(size_t)(ch0 + c + 1) * TAPS + j] : 0.0f);
+        gain[p] = g.norm == QkNorm::PerHead && !is_v ? make_float2(c < n ? gw[c] : 0.0f, c + 1 < n ? gw[c + 1] : 0.0f) : make_float2(1.0f, 1.0f);
+    }
+    int prev_seq = -1, prev_pos = -1;
+    for (int t = t0; t < t1; t++) {
+        const int seq = a.tok_seq[t], pos = a.tok_pos[t];
+        const float* row = a.proj + (size_t)t * a.ld_proj + col0;
+        // the inputs j tokens back: from the call's rows as far as they belong to this run, from the ring before that, zero before the start
+        auto back = [&](int j, int c) {
+            if (pos - j < 0) return make_float2(0.0f, 0.0f);
+            const int tt = t - j;
+            if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) return pair_at(a.proj + (size_t)tt * a.ld_proj + col0, c);
+            return pair_at(a.ring + ((size_t)seq * taps + (pos - j) % taps) * channels + ch0, c);
+        };
+        float2 x[NP];
+        const bool fresh = seq != prev_seq || pos != prev_pos + 1;
+        float ss = 0.0f;
+#pragma unroll
+        for (int p = 0; p < NP; p++) {
+            const int c = 2 * (lane + 32 * p);
+            const float2 u = pair_at(row, c);
+            x[p] = u;
+            if constexpr (TAPS > 0) {
+                if (fresh)
+#pragma unroll
+                    for (int j = 1; j < TAPS; j++) win[p][j - 1] = back(j, c);
+                float2 y = make_float2(0.0f, 0.0f);
+#pragma unroll
+                for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[p][TAPS - 1 - j].x, win[p][j - 1].x, y.x); y.y = fmaf(w[p][TAPS - 1 - j].y, win[p][j - 1].y, y.y); }
+                x[p] = make_float2(fmaf(w[p][TAPS - 1].x, u.x, y.x), fmaf(w[p][TAPS - 1].y, u.y, y.y));
+#pragma unroll
+                for (int j = TAPS - 2; j > 0; j--) win[p][j] = win[p][j - 1];
+                win[p][0] = u;
+            } else if constexpr (TAPS < 0) {
+                float2 y = make_float2(0.0f, 0.0f);
+                if (c < n)
+                    for (int j = taps - 1; j >= 0; j--) {
+                        const float2 v = j == 0 ? u : back(j, c);
+                        const float* cw = a.conv + (size_t)(ch0 + c) * taps + taps - 1 - j;
+                        y.x = fmaf(cw[0], v.x, y.x);
+                        if (c + 1 < n) y.y = fmaf(cw[taps], v.y, y.y);
+                    }
+                x[p] = y;
+            }
+            if (TAPS != 0 && a.one_each && c < n) {
+                float* r = a.ring + ((size_t)seq * taps + pos % taps) * channels + ch0 + c;
+                r[0] = u.x;
+                if (c + 1 < n) r[1] = u.y;
+            }
+            ss = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, ss));
+        }
+        prev_seq = seq; prev_pos = pos;
+        if (!is_v) {
+            if (g.norm == QkNorm::PerHead) {
+                const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
+#pragma unroll
+                for (int p = 0; p < NP; p++) { x[p].x *= r * gain[p].x; x[p].y *= r * gain[p].y; }
+            }
+            const float2* tab = a.rot + (size_t)pos * half;
+            if (g.pairs == AttnPairs::Neighbours) {
+#pragma unroll
+                for (int p = 0; p < NP; p++) {
+                    const int i = lane + 32 * p;
+                    if (i < half) { const float2 cs = tab[i], u = x[p]; x[p] = make_float2(u.x * cs.x - u.y * cs.y, u.y * cs.x + u.x * cs.y); }
+                }
+            } else if (half > 0) {
+                __syncwarp();
+#pragma unroll
+                for (int p = 0; p < NP; p++) *(float2*)(s_x[warp] + 2 * (lane + 32 * p)) = x[p];
+                __syncwarp();
+                auto turned = [&](int c, float v) {
+                    if (c >= 2 * half) return v;
+                    const float2 cs = tab[c < half ? c : c - half];
+                    return c < half ? v * cs.x - s_x[warp][c + half] * cs.y : v * cs.x + s_x[warp][c - half] * cs.y;
+                };
+#pragma unroll
+                for (int p = 0; p < NP; p++) { const int c = 2 * (lane + 32 * p); x[p] = make_float2(turned(c, x[p].x), turned(c + 1, x[p].y)); }
+            }
+            if (g.norm == QkNorm::PerHeadAfter) {
+                ss = 0.0f;
+#pragma unroll
+                for (int p = 0; p < NP; p++) ss = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, ss));
+                const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
+#pragma unroll
+                for (int p = 0; p < NP; p++) { x[p].x *= r; x[p].y *= r; }
+            }
+        }
+        A* dst;
+        int swz = 0;
+        if (is_q) dst = (A*)a.q + ((size_t)t * g.heads + h) * g.dp;
+        else {
+            const int page = a.page_table[(size_t)seq * a.pages_per_seq + pos / a.page_tokens];
+            const size_t at = ((size_t)page * g.kv_heads + h) * a.page_tokens + pos % a.page_tokens;
+            dst = is_v ? (A*)a.v_cache + at * g.v_pitch : (A*)a.k_cache + at * g.k_pitch;
+            swz = is_v ? g.v_swz : g.k_swz;
+        }
+#pragma unroll
+        for (int p = 0; p < NP; p++) {
+            const int c = 2 * (lane + 32 * p);
+            if (c >= n) continue;
+            A* d = dst + cell_of(c, pos, swz);
+            if (c + 1 < n) put2<A>(d, x[p]);
+            else d[0] = to_act<A>(x[p].x);
+        }
+    }
+}
+
+// The inputs of a run's last `taps` positions, for the convolutions of the next call.
+__global__ void __launch_bounds__(256) attn_keep_kernel(const AttnArgs a, const SeqRun* __restrict__ runs) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const AttnShape& g = a.g;
+    const SeqRun run = runs[blockIdx.x];
+    const int nq = g.heads * g.dim, nk = g.kv_heads * g.dim, channels = nq + nk + g.kv_heads * g.vdim, ch = blockIdx.y * 256 + threadIdx.x;
+    if (ch >= channels) return;
+    const int col = ch < nq ? ch : ch < nq + nk ? a.off_k + ch - nq : a.off_v + ch - nq - nk;
+    for (int t = max(0, run.n - g.taps); t < run.n; t++)
+        a.ring[((size_t)run.seq * g.taps + (run.pos0 + t) % g.taps) * channels + ch] = a.proj[(size_t)(run.tok0 + t) * a.ld_proj + col];
+}
+
 // One CTA per (head, token), a key per thread.
 constexpr int kPlainThreads = 128;
 template <typename A>
@@ -174,6 +343,7 @@ __global__ void __launch_bounds__(kPlainThreads) attn_plain_kernel(const AttnArg
             float d = 0.0f;
             for (int c = 0; c < g.dim; c++) d = fmaf(s_q[c], act_f<A>(kr[cell_of(c, key, g.k_swz)]), d);
             sc = d * g.scale;
+            if (g.cap > 0.0f) sc = g.cap * tanhf(sc / g.cap);
         }
         const float mt = fmaxf(m, block_max(sc, red));
         const float p = i < n ? expf(sc - mt) : 0.0f, corr = expf(m - mt);
@@ -192,7 +362,7 @@ __global__ void __launch_bounds__(kPlainThreads) attn_plain_kernel(const AttnArg
         __syncthreads();
     }
     A* out = (A*)a.out + (size_t)t * a.ldo + (size_t)h * g.ep;
-    for (int c = threadIdx.x; c < g.ep; c += kPlainThreads) out[c] = to_act<A>(c < g.vdim ? s_o[c] / l : 0.0f);
+    for (int c = threadIdx.x; c < g.ep; c += kPlainThreads) out[c] = to_act<A>(c < g.vdim ? s_o[c] / l * out_factor<A>(a, t, h, c) : 0.0f);
 }
 
 // ---- few tokens per sequence ------------------------------------------------------------------------------------------------
@@ -203,7 +373,7 @@ constexpr int kPartCells = 12;  // CTAs per SM whose partial sums there is room 
 constexpr int kDecKeys = 16, kDecStages = 2, kDecWarps = 4, kMaxPieces = 32;
 struct AttnParts { float *o, *ml; unsigned* tickets; };  // [token][kv head][row block][piece][16][ep], [..][16][2] (log2 units)
 
-template <int NV>
+template <int NV, bool CAP>
 __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnArgs a, const AttnParts pt_out, int* error_flag) {
     extern __shared__ __align__(128) unsigned char smem[];
     __shared__ float s_ml[kDecWarps][16][2], s_scale[kMaxPieces][16];
@@ -249,6 +419,7 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
 #pragma unroll
     for (int i = 0; i < NV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     const float sc = g.scale * kLog2e;
+    const float2 ck = cap_constants(g);
     const uint32_t qa = q_sm + (uint32_t)((lane & 15) * qb + (lane >> 4) * 16);
     const int krow = (lane & 7) + ((lane >> 4) << 3), kx = krow & g.k_swz, kc = (lane >> 3) & 1, vx = lane & 15 & g.v_swz, vc = lane >> 4;
     for (int j = 0; j < mine; j++) {
@@ -276,7 +447,7 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
         for (int i = 0; i < 2; i++)
 #pragma unroll
             for (int e = 0; e < 4; e++) {
-                s[i][e] *= sc;
+                s[i][e] = CAP ? capped(s[i][e], ck) : s[i][e] * sc;
                 if (edge) {
                     const int key = key0 + 8 * i + 2 * t4 + (e & 1);
                     if (key > pos || (key < sn.lo && key >= sn.keep)) s[i][e] = -INFINITY;
@@ -366,7 +537,7 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
             const float4 v = *(const float4*)(s_o + ((size_t)w * 16 + row) * g.ep + c);
             x.x = fmaf(f, v.x, x.x); x.y = fmaf(f, v.y, x.y); x.z = fmaf(f, v.z, x.z); x.w = fmaf(f, v.w, x.w);
         }
-        if (pieces == 1) put4<bf16>((bf16*)a.out + (size_t)t * a.ldo + (size_t)(h0 + row) * g.ep + c, x);
+        if (pieces == 1) put4<bf16>((bf16*)a.out + (size_t)t * a.ldo + (size_t)(h0 + row) * g.ep + c, finished(a, t, h0 + row, c, x));
         else *(float4*)(pt_out.o + ((cell * pieces + blockIdx.z) * 16 + row) * g.ep + c) = x;
     }
     if (pieces == 1) return;
@@ -396,13 +567,13 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
             const float4 v = __ldcg((const float4*)(src + (size_t)p * 16 * g.ep));
             x.x = fmaf(f, v.x, x.x); x.y = fmaf(f, v.y, x.y); x.z = fmaf(f, v.z, x.z); x.w = fmaf(f, v.w, x.w);
         }
-        put4<bf16>((bf16*)a.out + (size_t)t * a.ldo + (size_t)(h0 + row) * g.ep + c, x);
+        put4<bf16>((bf16*)a.out + (size_t)t * a.ldo + (size_t)(h0 + row) * g.ep + c, finished(a, t, h0 + row, c, x));
     }
 }
 
 // ---- runs of many tokens ----------------------------------------------------------------------------------------------------
 constexpr int kKeys = 64;
-template <int NV>
+template <int NV, bool CAP>
 __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const AttnTile* __restrict__ tiles, int* error_flag) {
     extern __shared__ __align__(128) unsigned char smem[];
     __shared__ uint64_t full[2];
@@ -448,6 +619,7 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
 #pragma unroll
     for (int i = 0; i < NV; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
     const float sc = g.scale * kLog2e;
+    const float2 ck = cap_constants(g);
     const int q0 = warp * 16, pa = tl.pos0 + q0, pb = min(pa + 15, last), qpos[2] = {pa + g8, pa + g8 + 8};
     const int wlo_a = g.window > 0 ? max(0, pa - g.window + 1) : 0, wlo_b = g.window > 0 ? max(0, pb - g.window + 1) : 0;
     const int qlo[2] = {g.window > 0 ? qpos[0] - g.window + 1 : 0, g.window > 0 ? qpos[1] - g.window + 1 : 0};
@@ -482,7 +654,7 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
             for (int n = 0; n < 8; n++)
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
-                    float v = s[n][e] * sc;
+                    float v = CAP ? capped(s[n][e], ck) : s[n][e] * sc;
                     if (edge) {
                         const int key = key0 + 8 * n + 2 * t4 + (e & 1), r = e >> 1;
                         if (key > qpos[r] || (key < qlo[r] && key >= g.keep_first)) v = -INFINITY;
@@ -539,8 +711,16 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
         const float m = fmaxf(m_run[r], sink), f = exp2f(m_run[r] - m), inv = f / (l_run[r] * f + (a.sink ? exp2f(sink - m) : 0.0f));
         bf16* dst = (bf16*)a.out + (size_t)(tl.tok0 + row) * a.ldo + (size_t)h * g.ep + 2 * t4;
 #pragma unroll
-        for (int n = 0; n < NV; n++)
-            if (8 * n < g.ep) *(uint32_t*)(dst + 8 * n) = pack2(o[n][2 * r] * inv, o[n][2 * r + 1] * inv);
+        for (int n = 0; n < NV; n++) {
+            if (8 * n >= g.ep) continue;
+            float2 x = make_float2(o[n][2 * r] * inv, o[n][2 * r + 1] * inv);
+            if (a.gate || a.out_scale != 1.0f) {
+                const int c = 8 * n + 2 * t4;
+                x.x *= out_factor<bf16>(a, tl.tok0 + row, h, c);
+                x.y *= out_factor<bf16>(a, tl.tok0 + row, h, c + 1);
+            }
+            *(uint32_t*)(dst + 8 * n) = pack2(x.x, x.y);
+        }
     }
 }
 
@@ -560,6 +740,29 @@ int pitch_of(int n8, bool f32, int* swz) {
     return chunks % 2 ? n8 + 16 : n8 + 8;  // an odd number of chunks; an odd row is followed by a chunk of zeros, since products take 16 columns
 }
 bool tensor_form(const AttnShape& g, bool f32) { return !f32 && g.ep <= 256 && tokens_smem(g) <= kMaxSmem - 4096 && tiles_smem(g) <= kMaxSmem - 1024; }
+template <typename A, int TAPS>
+int32_t head_prep_pairs(const AttnArgs& a, cudaStream_t s) {
+    const int pairs = (std::max(a.g.dim, a.g.vdim) + 63) / 64, stretch = a.T < 256 ? 1 : 8;
+    const dim3 grid((unsigned)((a.T + stretch - 1) / stretch), (unsigned)((a.g.heads + 2 * a.g.kv_heads + 7) / 8));
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(launch_pdl(kern, grid, dim3(256), 0, s, a, stretch));
+        return LC_OK;
+    };
+    LC_CHECK(pairs <= 8, LC_ERR_UNSUPPORTED, "attention: heads of %d and %d dimensions (at most 512)", a.g.dim, a.g.vdim);
+    return pairs == 1 ? go(attn_head_prep_kernel<A, TAPS, 1>) : pairs == 2 ? go(attn_head_prep_kernel<A, TAPS, 2>) : pairs <= 4 ? go(attn_head_prep_kernel<A, TAPS, 4>)
+                                                                                                                            : go(attn_head_prep_kernel<A, TAPS, 8>);
+}
+template <typename A>
+int32_t head_prep(const AttnArgs& a, cudaStream_t s) {
+    LC_CHECK(a.off_k >= 0, LC_ERR_UNSUPPORTED, "attention: norms per head over another layer's cache");
+    switch (a.g.taps) {
+        case 0: return head_prep_pairs<A, 0>(a, s);
+        case 2: return head_prep_pairs<A, 2>(a, s);
+        case 3: return head_prep_pairs<A, 3>(a, s);
+        case 4: return head_prep_pairs<A, 4>(a, s);
+        default: return head_prep_pairs<A, -1>(a, s);
+    }
+}
 int cells(const AttnShape& g) { return g.kv_heads * ((g.heads / g.kv_heads + 15) / 16); }
 
 }  // namespace
@@ -569,8 +772,16 @@ void attn_cache_layout(AttnShape* g, bool f32) {
     g->v_pitch = pitch_of(g->ep, f32, &g->v_swz);
 }
 
+int32_t launch_attn_keep(const AttnArgs& a, const SeqRun* runs, int n_runs, cudaStream_t s) {
+    const int channels = (a.g.heads + a.g.kv_heads) * a.g.dim + a.g.kv_heads * a.g.vdim;
+    LC_CUDA(launch_pdl(attn_keep_kernel, dim3((unsigned)n_runs, (unsigned)((channels + 255) / 256)), dim3(256), 0, s, a, runs));
+    return LC_OK;
+}
+
 int32_t launch_attn_prep(const AttnArgs& a, cudaStream_t s) {
     const AttnShape& g = a.g;
+    if (g.norm != QkNorm::AllHeads) return a.f32 ? head_prep<float>(a, s) : head_prep<bf16>(a, s);
+    LC_CHECK(g.pairs == AttnPairs::Halves && g.taps == 0, LC_ERR_UNSUPPORTED, "attention: norms over all heads with neighbouring pairs or convolutions");
     const bool vec = g.dim % 4 == 0 && g.vdim % 4 == 0 && g.rot_dims % 8 == 0;
     // few tokens: several CTAs each, all of which sum the whole rows
     const dim3 grid((unsigned)a.T, (unsigned)(a.T < 32 ? std::max(1, std::min(8, (g.heads + g.kv_heads) * g.dim / 1024)) : 1));
@@ -622,12 +833,13 @@ int32_t launch_attn_tokens(const AttnArgs& a, const AttnScratch& sc, cudaStream_
         LC_CUDA(launch_pdl(kern, grid, dim3(32 * kDecWarps), smem, s, a, p, gemv_error_flag_dev()));
         return LC_OK;
     };
+    auto of = [&](auto nv) -> int32_t { return g.cap > 0.0f ? go(attn_tokens_kernel<decltype(nv)::value, true>) : go(attn_tokens_kernel<decltype(nv)::value, false>); };
     switch (value_tiles(g.ep)) {
-        case 4: return go(attn_tokens_kernel<4>);
-        case 8: return go(attn_tokens_kernel<8>);
-        case 12: return go(attn_tokens_kernel<12>);
-        case 16: return go(attn_tokens_kernel<16>);
-        default: return go(attn_tokens_kernel<32>);
+        case 4: return of(std::integral_constant<int, 4>());
+        case 8: return of(std::integral_constant<int, 8>());
+        case 12: return of(std::integral_constant<int, 12>());
+        case 16: return of(std::integral_constant<int, 16>());
+        default: return of(std::integral_constant<int, 32>());
     }
 }
 
@@ -641,12 +853,13 @@ int32_t launch_attn_tiles(const AttnArgs& a, const AttnTile* tiles, int n_tiles,
         LC_CUDA(launch_pdl(kern, grid, dim3(128), smem, s, a, tiles, gemv_error_flag_dev()));
         return LC_OK;
     };
+    auto of = [&](auto nv) -> int32_t { return a.g.cap > 0.0f ? go(attn_tiles_kernel<decltype(nv)::value, true>) : go(attn_tiles_kernel<decltype(nv)::value, false>); };
     switch (value_tiles(a.g.ep)) {
-        case 4: return go(attn_tiles_kernel<4>);
-        case 8: return go(attn_tiles_kernel<8>);
-        case 12: return go(attn_tiles_kernel<12>);
-        case 16: return go(attn_tiles_kernel<16>);
-        default: return go(attn_tiles_kernel<32>);
+        case 4: return of(std::integral_constant<int, 4>());
+        case 8: return of(std::integral_constant<int, 8>());
+        case 12: return of(std::integral_constant<int, 12>());
+        case 16: return of(std::integral_constant<int, 16>());
+        default: return of(std::integral_constant<int, 32>());
     }
 }
 

@@ -5,12 +5,16 @@
 //   LatentAttention  in = dq | dkv (one product)  ->  latent norms, key rotation, cache append  ->  uq -> (per head) uk^T
 //                    -> attention over the latents -> (per head) uv -> out
 //   Attention        in = q | k | v (one product)  ->  norms over all heads, rotation, cache append  ->  attention -> out
+//   Attention and    in = both mixers' projections (one product, silu where a mixer wants it)  ->  convolutions, norms, rotation, cache
+//   LinearState      append -> attention (gated) | convolutions -> recurrence -> norm and gate  ->  out: one product over both outputs side
+//   side by side     by side, or one each where they are normed before they meet
 //   Relu2            up (squared relu in its epilogue) -> down
 //   GatedSilu        gate and up rows in turn (one product, silu(gate) * up in its epilogue) -> down
 //   Moe              router | shared gate | shared up (one product) -> choice, token lists -> experts' up, experts' down
 //                    (grouped products), shared down
+//   token input      gate (gelu times the token's row of a table in its epilogue) -> proj
 // each followed by x += rms_norm(y) w (for Moe on the weighted sum of the experts' rows), which also writes the activations the
-// next product reads: the sum, or its norm where the design has norms on inputs.
+// next product reads: the sum, or its norm where the design has norms on inputs and no token input follows.
 #include <cmath>
 #include <cstring>
 #include "lc_model.h"
@@ -121,9 +125,48 @@ int rows_of(lc_model* m, const std::string& name) {
     return it == m->tensors.end() ? 0 : (int)it->second.rows;
 }
 
-int32_t bind_delta(lc_model* m, StackLayer& L, const std::string& p) {
+// A vector put through `f`, on the host.
+template <typename F>
+int32_t changed_gain(lc_model* m, const std::string& name, int n, F f, const float** out) {
+    const float* g = nullptr;
+    LC_TRY(model_gain_f32(m, name, n, &g));
+    std::vector<float> h((size_t)n);
+    LC_CUDA(cudaMemcpyAsync(h.data(), g, h.size() * 4, cudaMemcpyDeviceToHost, m->stream));
+    LC_CUDA(cudaStreamSynchronize(m->stream));
+    for (float& v : h) v = f(v);
+    void* d = nullptr;
+    LC_TRY(zalloc(*m->stack, &d, h.size() * 4));
+    LC_CUDA(cudaMemcpyAsync(d, h.data(), h.size() * 4, cudaMemcpyHostToDevice, m->stream));
+    LC_CUDA(cudaStreamSynchronize(m->stream));
+    *out = (const float*)d;
+    return LC_OK;
+}
+
+// The weight of one of the model's norms.
+int32_t norm_gain(lc_model* m, const std::string& name, const float** out) {
+    const ArchSpec& sp = m->stack->spec;
+    return sp.norm_one_plus ? changed_gain(m, name, sp.width, [](float v) { return 1.0f + v; }, out) : model_gain_f32(m, name, sp.width, out);
+}
+
+// The taps of the convolutions on q, k and v as one f32 table.
+int32_t conv_table(lc_model* m, const std::string& p, const std::vector<int>& channels, int taps, const float** out) {
+    const char* names[3] = {"q.conv", "k.conv", "v.conv"};
+    void* d = nullptr;
+    LC_TRY(zalloc(*m->stack, &d, (size_t)(channels[0] + channels[1] + channels[2]) * taps * 4));
+    float* at = (float*)d;
+    for (int i = 0; i < 3; i++) {
+        const float* g = nullptr;
+        LC_TRY(model_gain_f32(m, p + names[i], channels[i] * taps, &g));
+        LC_CUDA(cudaMemcpyAsync(at, g, (size_t)channels[i] * taps * 4, cudaMemcpyDeviceToDevice, m->stream));
+        at += (size_t)channels[i] * taps;
+    }
+    *out = (const float*)d;
+    return LC_OK;
+}
+
+int32_t bind_delta(lc_model* m, MixerUnit& L, const std::string& p) {
     LayerStack& st = *m->stack;
-    const LayerSpec& s = L.s;
+    const MixerSpec& s = L.s;
     const int W = st.spec.width, nk = s.kv_heads * s.dim, nv = s.heads * s.vdim, nd = s.heads * s.dim;
     const int ra = rows_of(m, p + "a1"), rg = rows_of(m, p + "g1");
     LC_CHECK(ra > 0 && rg > 0, LC_ERR_MISSING, "missing tensor %sa1 or %sg1", p.c_str(), p.c_str());
@@ -135,30 +178,8 @@ int32_t bind_delta(lc_model* m, StackLayer& L, const std::string& p) {
     LC_TRY(plain_weight(m, p + "a2", nd, ra, &L.a2));
     LC_TRY(plain_weight(m, p + "g2", nv, rg, &L.g2));
     LC_TRY(plain_weight(m, p + "o", W, nv, &L.out));
-    // the three convolutions' taps as one f32 table
-    void* cp = nullptr;
-    LC_TRY(zalloc(st, &cp, (size_t)L.dg.channels * s.conv_taps * 4));
-    const char* cn[3] = {"q.conv", "k.conv", "v.conv"};
-    const int cc[3] = {nk, nk, nv};
-    size_t at = 0;
-    for (int i = 0; i < 3; i++) {
-        const float* g = nullptr;
-        LC_TRY(model_gain_f32(m, p + cn[i], cc[i] * s.conv_taps, &g));
-        LC_CUDA(cudaMemcpyAsync((float*)cp + at, g, (size_t)cc[i] * s.conv_taps * 4, cudaMemcpyDeviceToDevice, m->stream));
-        at += (size_t)cc[i] * s.conv_taps;
-    }
-    L.conv = (const float*)cp;
-    const float* alog = nullptr;
-    LC_TRY(model_gain_f32(m, p + "A_log", s.heads, &alog));
-    std::vector<float> h((size_t)s.heads);
-    LC_CUDA(cudaMemcpyAsync(h.data(), alog, h.size() * 4, cudaMemcpyDeviceToHost, m->stream));
-    LC_CUDA(cudaStreamSynchronize(m->stream));
-    for (float& v : h) v = std::exp(v);
-    void* ae = nullptr;
-    LC_TRY(zalloc(st, &ae, h.size() * 4));
-    LC_CUDA(cudaMemcpyAsync(ae, h.data(), h.size() * 4, cudaMemcpyHostToDevice, m->stream));
-    LC_CUDA(cudaStreamSynchronize(m->stream));
-    L.a_exp = (const float*)ae;
+    LC_TRY(conv_table(m, p, {nk, nk, nv}, s.conv_taps, &L.conv));
+    LC_TRY(changed_gain(m, p + "A_log", s.heads, [](float v) { return std::exp(v); }, &L.a_exp));
     LC_TRY(model_gain_f32(m, p + "dt_bias", nd, &L.dt_bias));
     LC_TRY(model_gain_f32(m, p + "norm", s.vdim, &L.o_norm));
     return LC_OK;
@@ -182,9 +203,9 @@ int32_t rot_table(lc_model* m, const RotarySpec& r, const float2** out) {
     return LC_OK;
 }
 
-int32_t bind_latent(lc_model* m, StackLayer& L, const std::string& p) {
+int32_t bind_latent(lc_model* m, MixerUnit& L, const std::string& p) {
     LayerStack& st = *m->stack;
-    LayerSpec& s = L.s;
+    MixerSpec& s = L.s;
     const int W = st.spec.width, qr = rows_of(m, p + "dq");
     LC_CHECK(qr > 0, LC_ERR_MISSING, "missing tensor %sdq", p.c_str());
     LC_CHECK(s.q_rank == 0 || s.q_rank == qr, LC_ERR_INVALID, "%sdq has %d rows, the config says %d", p.c_str(), qr, s.q_rank);
@@ -247,15 +268,19 @@ int32_t bind_latent(lc_model* m, StackLayer& L, const std::string& p) {
     return rot_table(m, s.rot, &L.rot);
 }
 
-int32_t bind_attention(lc_model* m, StackLayer& L, const std::string& p) {
-    LayerStack& st = *m->stack;
-    const LayerSpec& s = L.s;
-    const int W = st.spec.width, nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
+void attention_shape(const LayerStack& st, MixerUnit& L) {
+    const MixerSpec& s = L.s;
     AttnShape& g = L.ag;
     g.heads = s.heads; g.kv_heads = s.kv_heads; g.dim = s.dim; g.vdim = s.vdim; g.dp = round8(s.dim); g.ep = round8(s.vdim); g.rot_dims = s.rot.dims;
-    g.scale = s.scale; g.window = s.mask.size; g.keep_first = s.mask.keep_first;
+    g.scale = s.scale; g.cap = s.softcap; g.window = s.mask.size; g.keep_first = s.mask.keep_first; g.norm = s.qk_norm; g.pairs = s.pairs; g.taps = s.conv_taps;
     attn_cache_layout(&g, st.f32);
     L.ep = g.ep;
+}
+
+int32_t bind_attention(lc_model* m, MixerUnit& L, const std::string& p) {
+    const MixerSpec& s = L.s;
+    const int W = m->stack->spec.width, nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
+    attention_shape(*m->stack, L);
     std::vector<int> offs;
     if (s.kv_from < 0) {
         LC_TRY(fused_weight(m, {p + "q", p + "k", p + "v"}, {nq, nk, nv}, W, &L.in, &offs));
@@ -270,17 +295,109 @@ int32_t bind_attention(lc_model* m, StackLayer& L, const std::string& p) {
     return s.rot.dims ? rot_table(m, s.rot, &L.rot) : LC_OK;
 }
 
-// The experts' matrices `which` [n, k] as one batch.
-int32_t expert_weights(lc_model* m, const std::string& p, const char* which, int experts, int n, int k, DenseWeight* w) {
-    const int ld = round8(k);
-    void* d = nullptr;
-    LC_TRY(talloc(*m->stack, &d, (size_t)experts * n * ld * 2));
-    for (int e = 0; e < experts; e++) {
-        DevTensor* t = nullptr;
-        LC_TRY(matrix(m, p + "e" + std::to_string(e) + "." + which, n, k, &t));
-        LC_TRY(launch_pack((const bf16*)t->view, n, k, (bf16*)d + (size_t)e * n * ld, ld, PackMap(), PackMap(), false, m->stream));
+// Attention and a linear recurrence side by side.
+int32_t bind_pair(lc_model* m, StackLayer& L, const std::string& p) {
+    LayerStack& st = *m->stack;
+    MixerUnit &a = L.mix[0], &b = L.mix[1];
+    const MixerSpec &sa = a.s, &sb = b.s;
+    const std::string pl = p + "left.", pr = p + "right.";
+    const int W = st.spec.width, nq = sa.heads * sa.dim, nk = sa.kv_heads * sa.dim, nv = sa.kv_heads * sa.vdim, inner = sb.heads * sb.vdim;
+    const bool space = sb.linear == LinearKind::StateSpace;
+    attention_shape(st, a);
+    LinearShape& g = b.ng;
+    g.kind = sb.linear; g.heads = sb.heads; g.groups = sb.kv_heads; g.dim = sb.dim; g.vdim = sb.vdim; g.taps = sb.conv_taps; g.norm_parts = sb.norm_parts; g.eps = st.spec.eps;
+    g.channels = space ? inner + 2 * sb.kv_heads * sb.dim : 0;
+    g.ld_in = round8(g.channels);
+    // rows [row0, row0 + rows) of a tensor of `all` rows; off: where they start
+    struct Part { std::string name; int all, row0, rows; int* off; };
+    std::vector<Part> wide = {{pl + "q", nq, 0, nq, nullptr}, {pl + "k", nk, 0, nk, &a.off_k}, {pl + "v", nv, 0, nv, &a.off_v}}, silu, plain;
+    if (sa.out_gate) plain.push_back({pl + "g", sa.heads * sa.vdim, 0, sa.heads * sa.vdim, &a.off_g});
+    if (space) {
+        const int all = inner + g.channels + sb.heads;
+        wide.push_back({pr + "in", all, inner + g.channels, sb.heads, &g.off_dt});
+        plain.push_back({pr + "in", all, 0, inner, &g.off_g});
+        plain.push_back({pr + "in", all, inner, g.channels, &g.off_v});
+    } else {
+        silu = {{pr + "q", sb.heads * sb.dim, 0, sb.heads * sb.dim, &g.off_q}, {pr + "k", sb.heads * sb.dim, 0, sb.heads * sb.dim, &g.off_k}, {pr + "v", inner, 0, inner, &g.off_v}};
+        plain.push_back({pr + "g", inner, 0, inner, &g.off_g});
     }
-    return dense_weight_init(w, (const bf16*)d, n, k, ld, experts, (size_t)n * ld);
+    auto rows_of_parts = [](const std::vector<Part>& ps) { int n = 0; for (const Part& q : ps) n += round8(q.rows); return n; };
+    L.in_split = (rows_of_parts(wide) + 31) / 32 * 32;
+    L.silu_end = L.in_split + rows_of_parts(silu);
+    const int total = L.silu_end + rows_of_parts(plain), ld = round8(W);
+    void* d = nullptr;
+    LC_TRY(talloc(st, &d, (size_t)total * ld * 2));
+    auto place = [&](const std::vector<Part>& ps, int at, int base) -> int32_t {
+        for (const Part& q : ps) {
+            DevTensor* t = nullptr;
+            LC_TRY(matrix(m, q.name, q.all, W, &t));
+            LC_TRY(launch_pack((const bf16*)t->view + (size_t)q.row0 * W, q.rows, W, (bf16*)d + (size_t)at * ld, ld, PackMap(), PackMap(), false, m->stream));
+            if (q.off) *q.off = at - base;
+            at += round8(q.rows);
+        }
+        return LC_OK;
+    };
+    LC_TRY(place(wide, 0, 0));
+    LC_TRY(place(silu, L.in_split, L.in_split));
+    LC_TRY(place(plain, L.silu_end, L.in_split));
+    LC_TRY(dense_weight_init(&L.in, (const bf16*)d, total, W, ld));
+    g.ld = total - L.in_split;
+    g.ld_dt = L.in_split;
+    if (space) { g.off_k = g.off_v + inner; g.off_q = g.off_k + sb.kv_heads * sb.dim; }
+    // attention
+    if (sa.qk_norm == QkNorm::PerHead) {
+        LC_TRY(model_gain_f32(m, pl + "q.norm", sa.dim, &a.q_norm));
+        LC_TRY(model_gain_f32(m, pl + "k.norm", sa.dim, &a.k_norm));
+    }
+    if (sa.conv_taps) LC_TRY(conv_table(m, pl, {nq, nk, nv}, sa.conv_taps, &a.conv));
+    if (sa.rot.dims) LC_TRY(rot_table(m, sa.rot, &a.rot));
+    // recurrence
+    LC_TRY(model_gain_f32(m, pr + "norm", inner, &b.o_norm));
+    if (space) {
+        LC_TRY(model_gain_f32(m, pr + "conv", g.channels * g.taps, &b.conv));
+        LC_TRY(model_gain_f32(m, pr + "conv.b", g.channels, &b.conv_b));
+        LC_TRY(model_gain_f32(m, pr + "dt_bias", sb.heads, &b.dt_bias));
+        LC_TRY(model_gain_f32(m, pr + "D", sb.heads, &b.skip));
+        LC_TRY(changed_gain(m, pr + "A_log", sb.heads, [](float v) { return std::exp(v); }, &b.a_exp));
+    } else {
+        void* dec = nullptr;
+        LC_TRY(zalloc(st, &dec, (size_t)sb.heads * 4));
+        LC_CUDA(cudaMemcpyAsync(dec, sb.log_decay.data(), (size_t)sb.heads * 4, cudaMemcpyHostToDevice, m->stream));
+        LC_CUDA(cudaStreamSynchronize(m->stream));
+        b.log_decay = (const float*)dec;
+    }
+    // outputs
+    L.mixed_off = sa.heads * a.ep;
+    L.mixed_ld = L.mixed_off + round8(inner);
+    const PackMap heads{sa.vdim, a.ep, 0, 0};
+    if (L.s.combine == Combine::Normed) {
+        LC_TRY(plain_weight(m, pl + "o", W, sa.heads * sa.vdim, &L.out, heads, L.mixed_off));
+        LC_TRY(plain_weight(m, pr + "o", W, inner, &L.out2));
+        LC_TRY(model_gain_f32(m, pl + "out", W, &L.out_norm[0]));
+        return model_gain_f32(m, pr + "out", W, &L.out_norm[1]);
+    }
+    LC_TRY(talloc(st, &d, (size_t)W * L.mixed_ld * 2));
+    DevTensor* t = nullptr;
+    LC_TRY(matrix(m, pl + "o", W, sa.heads * sa.vdim, &t));
+    LC_TRY(launch_pack((const bf16*)t->view, W, sa.heads * sa.vdim, (bf16*)d, L.mixed_ld, PackMap(), heads, false, m->stream));
+    LC_TRY(matrix(m, pr + "o", W, inner, &t));
+    LC_TRY(launch_pack((const bf16*)t->view, W, inner, (bf16*)d + L.mixed_off, L.mixed_ld, PackMap(), PackMap(), false, m->stream));
+    return dense_weight_init(&L.out, (const bf16*)d, W, L.mixed_ld, L.mixed_ld);
+}
+
+// The experts' matrices `parts` [n, k] as one batch; several parts: their rows in turn.
+int32_t expert_weights(lc_model* m, const std::string& p, const std::vector<const char*>& parts, int experts, int n, int k, DenseWeight* w) {
+    const int ld = round8(k), np = (int)parts.size();
+    const size_t each = (size_t)np * n * ld;
+    void* d = nullptr;
+    LC_TRY(talloc(*m->stack, &d, experts * each * 2));
+    for (int e = 0; e < experts; e++)
+        for (int i = 0; i < np; i++) {
+            DevTensor* t = nullptr;
+            LC_TRY(matrix(m, p + "e" + std::to_string(e) + "." + parts[i], n, k, &t));
+            LC_TRY(launch_pack((const bf16*)t->view, n, k, (bf16*)d + e * each + (size_t)i * ld, ld, PackMap{1, np, 0, 0}, PackMap(), false, m->stream));
+        }
+    return dense_weight_init(w, (const bf16*)d, np * n, k, ld, experts, each);
 }
 
 int32_t bind_ffn(lc_model* m, StackLayer& L, const std::string& p) {
@@ -315,9 +432,9 @@ int32_t bind_ffn(lc_model* m, StackLayer& L, const std::string& p) {
     L.off_gate = e.shared_ff ? offs[1] : 0;
     L.route_split = e.shared_ff ? offs[2] : (L.route.n + 31) / 32 * 32;
     LC_TRY(model_gain_f32(m, p + "correction", e.outputs(), &L.correction));
-    LC_TRY(expert_weights(m, p, "up", e.experts, e.ff, W, &L.up));
-    LC_TRY(expert_weights(m, p, "down", e.experts, W, e.ff, &L.down));
-    L.expert_bytes = (uint64_t)2 * e.ff * W * 2;
+    LC_TRY(expert_weights(m, p, e.gated ? std::vector<const char*>{"gate", "up"} : std::vector<const char*>{"up"}, e.experts, e.ff, W, &L.up));
+    LC_TRY(expert_weights(m, p, {"down"}, e.experts, W, e.ff, &L.down));
+    L.expert_bytes = (uint64_t)(e.gated ? 3 : 2) * e.ff * W * 2;
     m->expert_bytes_all += L.expert_bytes * e.experts;
     m->expert_bytes_each = 1;  // d_moe_touched counts bytes
     return LC_OK;
@@ -335,9 +452,9 @@ int32_t product(lc_model* m, const DenseWeight& w, const void* x, int ldx, int T
 }
 const void* at(const LayerStack& st, const void* base, size_t elems) { return (const uint8_t*)base + elems * elt(st); }
 
-int32_t delta_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bool decode_step) {
+int32_t delta_block(lc_model* m, MixerUnit& L, const void* x, int ldx, int T, bool decode_step) {
     LayerStack& st = *m->stack;
-    const LayerSpec& s = L.s;
+    const MixerSpec& s = L.s;
     const int nd = s.heads * s.dim, nv = s.heads * s.vdim;
     LC_TRY(product(m, L.in, x, ldx, T, st.proj, L.in.n));
     DenseArgs e;
@@ -363,7 +480,7 @@ int32_t delta_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, b
     return product(m, L.out, st.mixed, d.ldo, T, st.y, st.spec.width, true);
 }
 
-int32_t latent_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bool decode_step) {
+int32_t latent_block(lc_model* m, MixerUnit& L, const void* x, int ldx, int T, bool decode_step) {
     LayerStack& st = *m->stack;
     const LatentShape& g = L.lg;
     LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in.n, true));
@@ -402,16 +519,19 @@ int32_t latent_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, 
     return product(m, L.out, st.mixed, lde, T, st.y, st.spec.width, true);
 }
 
-int32_t attention_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bool decode_step) {
+// Preparation and attention of `a`'s tokens; the caller has set where they come from and where the output goes.
+int32_t attend(lc_model* m, const MixerUnit& L, const MixerUnit& src, AttnArgs a, int T, bool decode_step) {
     LayerStack& st = *m->stack;
-    const StackLayer& src = L.s.kv_from < 0 ? L : st.layers[(size_t)L.s.kv_from];
-    LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in.n, true));
-    AttnArgs a;
-    a.g = L.ag; a.proj = st.projf; a.ld_proj = L.in.n; a.off_k = L.off_k; a.off_v = L.off_v; a.q_norm = L.q_norm; a.k_norm = L.k_norm; a.eps = st.spec.eps; a.rot = L.rot;
+    a.g = L.ag; a.proj = st.projf; a.off_k = L.off_k; a.off_v = L.off_v; a.q_norm = L.q_norm; a.k_norm = L.k_norm; a.eps = st.spec.eps; a.rot = L.rot;
+    a.conv = L.conv; a.ring = (float*)L.ring; a.one_each = decode_step;
     a.q = st.q; a.k_cache = src.k_cache; a.v_cache = src.v_cache; a.page_tokens = m->page_tokens; a.page_table = m->d_page_table; a.tok_seq = m->d_tok_seq;
-    a.tok_pos = m->d_tok_pos; a.pages_per_seq = m->pages_per_seq; a.T = T; a.sink = L.sink; a.out = st.mixed; a.ldo = L.ag.heads * L.ep; a.f32 = st.f32;
+    a.tok_pos = m->d_tok_pos; a.pages_per_seq = m->pages_per_seq; a.T = T; a.sink = L.sink; a.f32 = st.f32;
     LC_TRY(launch_attn_prep(a, m->stream));
     m->launches_in_call += 1;
+    if (L.ag.taps > 0 && !decode_step) {
+        LC_TRY(launch_attn_keep(a, st.d_runs, st.n_runs, m->stream));
+        m->launches_in_call += 1;
+    }
     const int few = decode_step || !st.prefill_tiles ? T : st.n_short;
     a.T = few;
     if (few > 0) {
@@ -422,7 +542,63 @@ int32_t attention_block(lc_model* m, StackLayer& L, const void* x, int ldx, int 
         LC_TRY(launch_attn_tiles(a, st.d_attn_tiles, st.n_attn_tiles, m->stream));
         m->launches_in_call += 1;
     }
+    return LC_OK;
+}
+
+int32_t attention_block(lc_model* m, MixerUnit& L, const void* x, int ldx, int T, bool decode_step) {
+    LayerStack& st = *m->stack;
+    LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in.n, true));
+    AttnArgs a;
+    a.ld_proj = L.in.n; a.out = st.mixed; a.ldo = L.ag.heads * L.ep;
+    LC_TRY(attend(m, L, L.s.kv_from < 0 ? L : st.layers[(size_t)L.s.kv_from].mix[0], a, T, decode_step));
     return product(m, L.out, st.mixed, a.ldo, T, st.y, st.spec.width, true);
+}
+
+int32_t recur(lc_model* m, const MixerUnit& L, LinearArgs a, int T, bool decode_step) {
+    LayerStack& st = *m->stack;
+    a.g = L.ng; a.proj = st.proj; a.dt = st.projf; a.conv = L.conv; a.conv_b = L.conv_b; a.dt_bias = L.dt_bias; a.a_exp = L.a_exp; a.skip = L.skip; a.log_decay = L.log_decay;
+    a.ring = L.ring; a.in = st.lin; a.state = L.state; a.tok_seq = m->d_tok_seq; a.tok_pos = m->d_tok_pos; a.T = T; a.o = st.o; a.norm_w = L.o_norm; a.f32 = st.f32;
+    int launches = 1;
+    if (decode_step) {
+        LC_TRY(launch_linear_step(a, m->stream));
+        launches++;
+    } else {
+        a.runs = st.d_short_runs; a.n_runs = st.n_short_runs; a.chunk_runs = st.d_chunk_runs; a.n_chunk_runs = st.n_chunk_runs; a.all_runs = st.d_runs; a.n_all_runs = st.n_runs;
+        LC_TRY(launch_linear_runs(a, &launches, m->stream));
+    }
+    LC_TRY(launch_linear_output(a, m->stream));
+    m->launches_in_call += launches;
+    return LC_OK;
+}
+
+// Attention and a linear recurrence side by side; Normed: their outputs in y and y2.
+int32_t pair_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bool decode_step) {
+    LayerStack& st = *m->stack;
+    DenseArgs in;
+    const int ld_act = L.in.n - L.in_split;
+    in.split = L.in_split; in.silu_end = L.silu_end; in.out2 = st.proj; in.ldo2 = ld_act;
+    LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in_split, true, DENSE_SPLIT_SILU, in));
+    const bool normed = L.s.combine == Combine::Normed;
+    AttnArgs a;
+    a.ld_proj = L.in_split; a.out = st.mixed; a.ldo = L.mixed_ld; a.out_scale = normed ? 1.0f : L.s.mix_scale[0];
+    if (L.s.mix[0].out_gate) { a.gate = at(st, st.proj, (size_t)L.mix[0].off_g); a.ld_gate = ld_act; }
+    LC_TRY(attend(m, L.mix[0], L.mix[0], a, T, decode_step));
+    LinearArgs b;
+    b.out = (void*)at(st, st.mixed, (size_t)L.mixed_off); b.ldo = L.mixed_ld; b.out_scale = normed ? 1.0f : L.s.mix_scale[1];
+    LC_TRY(recur(m, L.mix[1], b, T, decode_step));
+    LC_TRY(product(m, L.out, st.mixed, L.mixed_ld, T, st.y, st.spec.width, true));
+    return normed ? product(m, L.out2, b.out, L.mixed_ld, T, st.y2, st.spec.width, true) : LC_OK;
+}
+
+// x += norm(proj(gelu(gate x) * the layer's part of the token's row)): the two products; x as activations is in `xa`.
+int32_t side_block(lc_model* m, int l, int T) {
+    LayerStack& st = *m->stack;
+    const StackLayer& L = st.layers[(size_t)l];
+    const int n = st.spec.side_dim, ld = round8(n);
+    DenseArgs e;
+    e.table = st.side_embed + (size_t)l * n; e.table_ld = (int)st.layers.size() * n; e.table_rows = st.spec.vocab; e.ids = m->d_tokens;
+    LC_TRY(product(m, L.side_gate, st.xa, st.width_p, T, st.side, ld, false, DENSE_GELU_TABLE, e));
+    return product(m, L.side_proj, st.side, ld, T, st.y, st.spec.width, true);
 }
 
 // What the residual sum (or a probe) needs to finish the mixture's output.
@@ -432,6 +608,12 @@ MoeSum moe_sum(const LayerStack& st, const StackLayer& L, const void* x, int ldx
     r.rows = st.moe_rows; r.ld_rows = round8(st.spec.width); r.sel = st.moe_sel; r.pos = st.moe_pos; r.off = st.plan.off; r.weight = st.moe_w; r.top = e.top; r.experts = e.experts;
     r.h = x; r.ld_h = ldx;
     if (e.shared_ff) { r.gate = st.moe_z + L.off_gate; r.ld_gate = L.route_split; }
+    return r;
+}
+
+PairSum pair_sum(const LayerStack& st, const StackLayer& L) {
+    PairSum r;
+    r.y2 = st.y2; r.w0 = L.out_norm[0]; r.w1 = L.out_norm[1];
     return r;
 }
 
@@ -463,7 +645,7 @@ int32_t moe_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, boo
         m->launches_in_call += 1;
         g.gather = false; g.x_rows = st.moe_slots;
     }
-    LC_TRY(product(m, L.up, in, ld_in, T, st.moe_up, ldf, false, DENSE_RELU2, g));
+    LC_TRY(product(m, L.up, in, ld_in, T, st.moe_up, ldf, false, e.gated ? DENSE_GATED_SILU : DENSE_RELU2, g));
     if (e.shared_ff) LC_TRY(product(m, L.shared_down, st.ffn, lds, T, st.y, st.spec.width, true));
     g.gather = false; g.x_rows = st.moe_slots;
     return product(m, L.down, st.moe_up, ldf, T, st.moe_rows, round8(st.spec.width), false, DENSE_STORE, g);
@@ -495,28 +677,39 @@ int32_t stack_bind(lc_model* m) {
         StackLayer& L = st.layers[i];
         L.s = sp.layers[i];
         const std::string p = "l" + std::to_string(i) + ".";
-        switch (L.s.mixer) {
-            case MixerKind::ChannelDelta: LC_TRY(bind_delta(m, L, p + "mix.")); break;
-            case MixerKind::LatentAttention: LC_TRY(bind_latent(m, L, p + "mix.")); break;
-            case MixerKind::Attention: LC_TRY(bind_attention(m, L, p + "mix.")); break;
-        }
+        for (int j = 0; j < L.s.mixers(); j++) L.mix[j].s = L.s.mix[j];
+        MixerUnit& u = L.mix[0];
+        if (L.s.combine != Combine::Single) LC_TRY(bind_pair(m, L, p + "mix."));
+        else if (u.s.kind == MixerKind::ChannelDelta) LC_TRY(bind_delta(m, u, p + "mix."));
+        else if (u.s.kind == MixerKind::LatentAttention) LC_TRY(bind_latent(m, u, p + "mix."));
+        else LC_TRY(bind_attention(m, u, p + "mix."));
         auto norms = [&](const std::string& name, const float** in, const float** out) -> int32_t {
-            if (sp.norm_inputs) LC_TRY(model_gain_f32(m, name, sp.width, in));
-            return model_gain_f32(m, sp.norm_inputs ? name + "b" : name, sp.width, out);
+            if (sp.norm_inputs) LC_TRY(norm_gain(m, name, in));
+            return norm_gain(m, sp.norm_inputs ? name + "b" : name, out);
         };
         LC_TRY(norms(p + "norm1", &L.norm1_in, &L.norm1_out));
         if (L.s.ffn != FfnKind::None) {
             LC_TRY(bind_ffn(m, L, p + "mlp."));
             LC_TRY(norms(p + "norm2", &L.norm2_in, &L.norm2_out));
         }
-        LC_TRY(block_weights(m, {&L.in, &L.out, &L.up, &L.down, &L.a2, &L.g2, &L.uq, &L.uk_t, &L.uv, &L.uk_all, &L.uv_all, &L.route, &L.shared_down}));
+        if (sp.side_dim) {
+            LC_TRY(plain_weight(m, p + "side.gate", sp.side_dim, sp.width, &L.side_gate));
+            LC_TRY(plain_weight(m, p + "side.proj", sp.width, sp.side_dim, &L.side_proj));
+            LC_TRY(model_gain_f32(m, p + "side.norm", sp.width, &L.side_norm));
+        }
+        LC_TRY(block_weights(m, {&u.in, &u.out, &u.a2, &u.g2, &u.uq, &u.uk_t, &u.uv, &u.uk_all, &u.uv_all, &L.in, &L.out, &L.out2, &L.up, &L.down, &L.route, &L.shared_down,
+                                 &L.side_gate, &L.side_proj}));
     }
     DevTensor* e = nullptr;
     LC_TRY(matrix(m, "embed", sp.vocab, sp.width, &e));
     st.embed = (const bf16*)e->view;
-    st.packed.clear();  // the embedding table is read as it is
     m->embed = e;
-    LC_TRY(model_gain_f32(m, "final.norm", sp.width, &st.final_norm));
+    if (sp.side_dim) {
+        LC_TRY(matrix(m, "side.embed", sp.vocab, (int)sp.layers.size() * sp.side_dim, &e));
+        st.side_embed = (const bf16*)e->view;
+    }
+    st.packed.clear();  // the tables are read as they are
+    LC_TRY(norm_gain(m, "final.norm", &st.final_norm));
     LC_TRY(plain_weight(m, "head", sp.vocab, sp.width, &st.head));
     return block_weights(m, {&st.head});
 }
@@ -529,9 +722,10 @@ int32_t stack_alloc(lc_model* m) {
     int experts = 0, top = 0;
     size_t z = 0, hidden = 8, attn_part = 0;
     size_t proj = 8, projf = 8, gate = 8, mixed = 8, cq = 8, q = 8, qa = 8, ffn = 8, ld = 8, qk = 8, v = 8;
-    for (StackLayer& L : st.layers) {
-        const LayerSpec& s = L.s;
-        if (s.mixer == MixerKind::ChannelDelta) {
+    size_t lin = 0;
+    auto alloc_mixer = [&](MixerUnit& L) -> int32_t {
+        const MixerSpec& s = L.s;
+        if (s.kind == MixerKind::ChannelDelta) {
             const size_t nv = (size_t)s.heads * s.vdim, S = (size_t)s.heads * s.dim * s.vdim, ring = (size_t)s.conv_taps * L.dg.channels;
             proj = std::max(proj, (size_t)L.in.n);
             gate = std::max(gate, nv);
@@ -544,19 +738,33 @@ int32_t stack_alloc(lc_model* m) {
             st.delta_chunks = st.delta_chunks && delta_chunks_apply(L.dg, st.f32);
             st.chunk_bytes = std::max(st.chunk_bytes, delta_chunk_bytes(L.dg));
             st.state_bytes_per_seq += S * 4 + ring * e;
-        } else if (s.mixer == MixerKind::Attention) {
+        } else if (s.kind == MixerKind::Attention) {
             const AttnShape& g = L.ag;
             projf = std::max(projf, (size_t)L.in.n);
             q = std::max(q, (size_t)g.heads * g.dp);
             mixed = std::max(mixed, (size_t)g.heads * g.ep);
             st.prefill_tiles = st.prefill_tiles && attn_tiles_apply(g, st.f32);
             attn_part = std::max(attn_part, attn_part_bytes(g));
+            if (g.taps) {
+                const size_t ring = (size_t)g.taps * ((g.heads + g.kv_heads) * g.dim + g.kv_heads * g.vdim);
+                LC_TRY(zalloc(st, &L.ring, (size_t)m->max_seqs * ring * 4));
+                st.state_bytes_per_seq += ring * 4;
+            }
             if (s.kv_from < 0) {
                 const size_t rows = (size_t)m->pages_total * m->page_tokens * g.kv_heads;
                 LC_TRY(zalloc(st, &L.k_cache, rows * g.k_pitch * e));
                 LC_TRY(zalloc(st, &L.v_cache, rows * g.v_pitch * e));
                 st.cache_bytes_per_token += (size_t)g.kv_heads * (g.k_pitch + g.v_pitch) * e;
             }
+        } else if (s.kind == MixerKind::LinearState) {
+            const LinearShape& g = L.ng;
+            const size_t S = (size_t)g.heads * g.dim * g.vdim, ring = (size_t)g.taps * g.channels;
+            v = std::max(v, (size_t)g.heads * g.vdim);
+            lin = std::max(lin, (size_t)g.ld_in);
+            LC_TRY(zalloc(st, (void**)&L.state, (size_t)m->max_seqs * S * 4));
+            if (ring) LC_TRY(zalloc(st, &L.ring, (size_t)m->max_seqs * ring * e));
+            st.delta_chunks = st.delta_chunks && linear_chunks_apply(g, st.f32);
+            st.state_bytes_per_seq += S * 4 + ring * e;
         } else {
             const LatentShape& g = L.lg;
             projf = std::max(projf, (size_t)L.in.n);
@@ -573,12 +781,24 @@ int32_t stack_alloc(lc_model* m) {
             LC_TRY(zalloc(st, &L.cache, (size_t)m->pages_total * m->page_tokens * row));
             st.cache_bytes_per_token += row;
         }
-        if (s.ffn == FfnKind::Moe) {
-            experts = std::max(experts, s.moe.experts); top = std::max(top, s.moe.top);
+        return LC_OK;
+    };
+    bool pairs = false;
+    for (StackLayer& L : st.layers) {
+        const LayerSpec& ls = L.s;
+        for (int j = 0; j < ls.mixers(); j++) LC_TRY(alloc_mixer(L.mix[j]));
+        if (ls.combine != Combine::Single) {
+            proj = std::max(proj, (size_t)(L.in.n - L.in_split));
+            projf = std::max(projf, (size_t)L.in_split);
+            mixed = std::max(mixed, (size_t)L.mixed_ld);
+            pairs = pairs || ls.combine == Combine::Normed;
+        }
+        if (ls.ffn == FfnKind::Moe) {
+            experts = std::max(experts, ls.moe.experts); top = std::max(top, ls.moe.top);
             z = std::max(z, (size_t)L.route_split);
-            hidden = std::max(hidden, (size_t)round8(s.moe.ff));
-            ffn = std::max(ffn, (size_t)round8(s.moe.shared_ff));
-        } else if (s.ffn != FfnKind::None) ffn = std::max(ffn, (size_t)round8(s.ff));
+            hidden = std::max(hidden, (size_t)round8(ls.moe.ff));
+            ffn = std::max(ffn, (size_t)round8(ls.moe.shared_ff));
+        } else if (ls.ffn != FfnKind::None) ffn = std::max(ffn, (size_t)round8(ls.ff));
     }
     if (experts) {
         st.moe_slots = (int)T * top;
@@ -606,6 +826,9 @@ int32_t stack_alloc(lc_model* m) {
     LC_TRY(zalloc(st, &st.cq, T * cq * e)); LC_TRY(zalloc(st, &st.q, T * q * e));
     LC_TRY(zalloc(st, &st.q_abs, T * qa * e)); LC_TRY(zalloc(st, &st.o_lat, T * qa * e));
     LC_TRY(zalloc(st, &st.ffn, T * ffn * e)); LC_TRY(zalloc(st, &st.last, (size_t)m->head_rows * st.width_p * e));
+    if (pairs) LC_TRY(zalloc(st, (void**)&st.y2, T * st.spec.width * 4));
+    if (lin) LC_TRY(zalloc(st, &st.lin, T * lin * e));
+    if (st.spec.side_dim) LC_TRY(zalloc(st, &st.side, T * round8(st.spec.side_dim) * e));
     LC_TRY(zalloc(st, (void**)&st.y, T * st.spec.width * 4)); LC_TRY(zalloc(st, (void**)&st.log_decay, T * ld * 4));
     LC_TRY(zalloc(st, (void**)&st.qk, T * qk * 4)); LC_TRY(zalloc(st, (void**)&st.v, T * v * 4)); LC_TRY(zalloc(st, (void**)&st.o, T * v * 4));
     LC_TRY(zalloc(st, (void**)&st.d_runs, T * sizeof(SeqRun)));
@@ -627,14 +850,20 @@ void stack_free(lc_model* m) {
 // Cache and state a one-token step at position `ctx` reads and writes.
 uint64_t stack_step_bytes(const lc_model* m, int ctx) {
     const LayerStack& st = *m->stack;
-    uint64_t b = 2 * st.state_bytes_per_seq;
-    for (const StackLayer& L : st.layers) {
-        if (L.s.mixer == MixerKind::LatentAttention) b += (uint64_t)(ctx + 1) * (L.lg.cp + L.lg.rp) * elt(st);
-        if (L.s.mixer != MixerKind::Attention) continue;
+    uint64_t b = 2 * st.state_bytes_per_seq + (uint64_t)st.layers.size() * st.spec.side_dim * 2;
+    for (const StackLayer& layer : st.layers) {
+        const MixerUnit& L = layer.mix[0];
+        if (L.s.kind == MixerKind::LatentAttention) b += (uint64_t)(ctx + 1) * (L.lg.cp + L.lg.rp) * elt(st);
+        if (L.s.kind != MixerKind::Attention) continue;
         const int window = L.ag.window > 0 ? L.ag.window : ctx + 1, lo = std::max(0, ctx + 1 - window), seen = ctx + 1 - lo + std::min(L.ag.keep_first, lo);
         b += (uint64_t)seen * L.ag.kv_heads * (L.ag.dp + L.ag.ep) * elt(st);
     }
     return b;
+}
+
+uint64_t stack_table_bytes(const lc_model* m) {
+    const ArchSpec& sp = m->stack->spec;
+    return (uint64_t)sp.vocab * sp.layers.size() * sp.side_dim * 2;
 }
 
 // What a call's tokens mean to the layers: runs of consecutive positions, those of at least kTileRun tokens also as tiles
@@ -661,7 +890,7 @@ int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const st
     if (!chunks.empty()) {
         LC_CUDA(cudaMemcpyAsync(st.d_chunks, chunks.data(), chunks.size() * sizeof(DeltaChunk), cudaMemcpyHostToDevice, m->stream));
         LC_CUDA(cudaMemcpyAsync(st.d_chunk_runs, chunk_runs.data(), chunk_runs.size() * sizeof(DeltaChunkRun), cudaMemcpyHostToDevice, m->stream));
-        LC_TRY(st.chunk_scratch.reserve(std::max(chunks.size(), (size_t)m->t_cap / kDeltaChunk) * st.chunk_bytes));
+        if (st.chunk_bytes) LC_TRY(st.chunk_scratch.reserve(std::max(chunks.size(), (size_t)m->t_cap / kDeltaChunk) * st.chunk_bytes));
     }
     st.groups.clear();
     st.n_short = (int)seq.size();
@@ -706,10 +935,11 @@ int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const st
 
 int32_t stack_mixer(lc_model* m, int l, const void* x, int ldx, int T, bool decode_step) {
     StackLayer& L = m->stack->layers[l];
-    switch (L.s.mixer) {
-        case MixerKind::ChannelDelta: return delta_block(m, L, x, ldx, T, decode_step);
-        case MixerKind::LatentAttention: return latent_block(m, L, x, ldx, T, decode_step);
-        default: return attention_block(m, L, x, ldx, T, decode_step);
+    if (L.s.combine != Combine::Single) return pair_block(m, L, x, ldx, T, decode_step);
+    switch (L.mix[0].s.kind) {
+        case MixerKind::ChannelDelta: return delta_block(m, L.mix[0], x, ldx, T, decode_step);
+        case MixerKind::LatentAttention: return latent_block(m, L.mix[0], x, ldx, T, decode_step);
+        default: return attention_block(m, L.mix[0], x, ldx, T, decode_step);
     }
 }
 
@@ -725,19 +955,25 @@ int32_t stack_run_layers(lc_model* m, int T, bool decode_step) {
     r.y = st.y; r.eps = st.spec.eps; r.width = W; r.T = T; r.x = m->d_hidden; r.ld_act = st.width_p; r.f32 = st.f32;
     for (size_t l = 0; l < st.layers.size(); l++) {
         StackLayer& L = st.layers[l];
-        const bool ffn = L.s.ffn != FfnKind::None, last = l + 1 == st.layers.size();
+        const bool ffn = L.s.ffn != FfnKind::None, last = l + 1 == st.layers.size(), side = st.spec.side_dim > 0;
         const float* after = last ? nullptr : st.layers[l + 1].norm1_in;  // the norm ahead of the next layer; the last sum is read in f32
-        auto sum = [&](const float* w, const float* next, bool moe) -> int32_t {
-            r.w = w; r.w_next = next; r.act = st.spec.norm_inputs && !next ? nullptr : st.xa;
+        // plain_next: the sum itself is read next, not its norm
+        auto sum = [&](const float* w, const float* next, bool moe, bool pair, bool plain_next) -> int32_t {
+            r.w = w; r.w_next = plain_next ? nullptr : next; r.act = st.spec.norm_inputs && !plain_next && !next ? nullptr : st.xa;
             r.moe = moe ? moe_sum(st, L, x, ldx) : MoeSum();
+            r.pair = pair ? pair_sum(st, L) : PairSum();
             m->launches_in_call += 1;
             return launch_residual(r, m->stream);
         };
         LC_TRY(stack_mixer(m, (int)l, x, ldx, T, decode_step));
-        LC_TRY(sum(L.norm1_out, ffn ? L.norm2_in : after, false));
-        if (!ffn) continue;
-        LC_TRY(ffn_block(m, L, x, ldx, T, decode_step));
-        LC_TRY(sum(L.norm2_out, after, L.s.ffn == FfnKind::Moe));
+        LC_TRY(sum(L.norm1_out, ffn ? L.norm2_in : after, false, L.s.combine == Combine::Normed, side && !ffn));
+        if (ffn) {
+            LC_TRY(ffn_block(m, L, x, ldx, T, decode_step));
+            LC_TRY(sum(L.norm2_out, after, L.s.ffn == FfnKind::Moe, false, side));
+        }
+        if (!side) continue;
+        LC_TRY(side_block(m, (int)l, T));
+        LC_TRY(sum(L.side_norm, after, false, false, false));
     }
     return LC_OK;
 }
@@ -753,12 +989,17 @@ int32_t stack_probe(lc_model* m, int l, int T, bool ffn, float** y) {
     }
     LC_CHECK(!ffn || st.layers[l].s.ffn != FfnKind::None, LC_ERR_INVALID, "layer %d has no feed-forward", l);
     *y = st.y;
-    if (!ffn) return stack_mixer(m, l, x, ldx, T, false);
     StackLayer& L = st.layers[l];
+    ResidualArgs r;
+    r.y = st.y; r.eps = st.spec.eps; r.width = st.spec.width; r.T = T; r.ld_act = st.width_p; r.f32 = st.f32;
+    if (!ffn) {
+        LC_TRY(stack_mixer(m, l, x, ldx, T, false));
+        if (L.s.combine != Combine::Normed) return LC_OK;
+        r.pair = pair_sum(st, L);
+        return launch_residual(r, m->stream);
+    }
     LC_TRY(ffn_block(m, L, x, ldx, T, false));
     if (L.s.ffn != FfnKind::Moe) return LC_OK;
-    ResidualArgs r;
-    r.y = st.y; r.width = st.spec.width; r.T = T; r.ld_act = st.width_p; r.f32 = st.f32;
     r.moe = moe_sum(st, L, x, ldx);
     return launch_residual(r, m->stream);
 }

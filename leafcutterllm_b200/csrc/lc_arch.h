@@ -7,20 +7,22 @@
 
 namespace lc {
 
-enum class MixerKind { ChannelDelta, LatentAttention, Attention };
-// Relu2: down(relu(up x)^2).  GatedSilu: down(silu(gate x) * (up x)).  Moe: a mixture of Relu2 experts (MoeSpec).
+enum class MixerKind { ChannelDelta, LatentAttention, Attention, LinearState };
+// Relu2: down(relu(up x)^2).  GatedSilu: down(silu(gate x) * (up x)).  Moe: a mixture of such (MoeSpec).
 enum class FfnKind { None, Relu2, GatedSilu, Moe };
 const char* mixer_name(MixerKind k);
 
-// Rotary embedding, optionally with YaRN's interpolation of the frequencies.  Which dimensions form a pair is the mixer's:
-// neighbours in LatentAttention, halves (i with i + dims / 2) in Attention.
+// Rotary embedding, optionally with scaled frequencies: YaRN's interpolation over pairs, or by wavelength (pairs that turn more
+// than `high` times over the original context keep their frequency, those that turn less than `low` times are slowed by
+// `factor`, linear in the turns between).  Which dimensions form a pair is the mixer's (AttnPairs; neighbours in LatentAttention).
+enum class RotaryScaling { None, Yarn, Wavelength };
 struct RotarySpec {
     int dims = 0;
     double base = 10000.0;
-    bool yarn = false;
-    double factor = 1.0, original = 0.0, fast = 0.0, slow = 0.0;
+    RotaryScaling scaling = RotaryScaling::None;
+    double factor = 1.0, original = 0.0, fast = 0.0, slow = 0.0;  // Wavelength: fast, slow = high, low
     bool operator==(const RotarySpec& o) const {
-        return dims == o.dims && base == o.base && yarn == o.yarn && factor == o.factor && original == o.original && fast == o.fast && slow == o.slow;
+        return dims == o.dims && base == o.base && scaling == o.scaling && factor == o.factor && original == o.original && fast == o.fast && slow == o.slow;
     }
 };
 // Angular frequency of every pair and the factor on cos and sin.
@@ -30,38 +32,74 @@ void rotary_frequencies(const RotarySpec& r, std::vector<double>* freq, double* 
 struct MaskSpec { int size = 0, keep_first = 0; };
 
 constexpr int kMaxRouterOutputs = 1024, kMaxChoices = 32;
-// Router over `experts` feed-forwards and `identity` experts that return their input: softmax scores over all; the `top` largest
-// of score + correction among the best `keep` of `groups` equal groups are chosen and weighted with their scores.
+// Router over `experts` feed-forwards and `identity` experts that return their input.  Scores: softmax over all outputs, or a
+// sigmoid of each.  The `top` largest of score + correction among the best `keep` of `groups` equal groups are chosen and weighted
+// with their scores; a group counts with the sum of its `group_top` (1 or 2) largest.
+enum class RouterScore { Softmax, Sigmoid };
 struct MoeSpec {
     int experts = 0, identity = 0, top = 0, groups = 1, keep = 1, ff = 0;
     int shared_ff = 0;  // 0: no shared expert; otherwise one that runs for every token, times a sigmoid gate
+    RouterScore score = RouterScore::Softmax;
+    int group_top = 1;
+    bool gated = false; // experts are GatedSilu instead of Relu2 (then without a shared one)
     int outputs() const { return experts + identity; }
 };
 
-struct LayerSpec {
-    MixerKind mixer = MixerKind::ChannelDelta;
+// Norms of attention's queries and keys: over all heads together ahead of the rotation (weights of all heads), per head ahead of it
+// (one weight of `dim`), per head behind it (no weight).
+enum class QkNorm { AllHeads, PerHead, PerHeadAfter };
+// The two dimensions of a rotation pair: i and i + dims / 2, or 2i and 2i + 1.
+enum class AttnPairs { Halves, Neighbours };
+// LinearState: S = decay S + step k v^T, read with q, per head.  Constant: decays from the config, q, k and v through silu, the heads
+// normed together, a sigmoid gate on the result.  StateSpace: decay and step from the token, q and k shared by the heads of a
+// group, a convolution with bias ahead of the silu, a skip term, a silu gate ahead of the norm in parts.
+enum class LinearKind { Constant, StateSpace };
+
+struct MixerSpec {
+    MixerKind kind = MixerKind::ChannelDelta;
     int heads = 0, dim = 0, vdim = 0;
-    int kv_heads = 0;                             // ChannelDelta, Attention
-    int conv_taps = 0;                            // ChannelDelta
+    int kv_heads = 0;                             // ChannelDelta, Attention; LinearState: groups that share q and k
+    int conv_taps = 0;                            // ChannelDelta, Attention, LinearState (0: none)
     float unit_eps = 1e-6f;                       // ChannelDelta: inside the root that makes q and k unit vectors
     int q_rank = 0, kv_rank = 0, rot_dim = 0;     // LatentAttention (q_rank 0: the tensor's shape gives it)
     float scale = 1.0f;
     RotarySpec rot;
-    MaskSpec mask;                                // Attention
-    int kv_from = -1;                             // Attention: the layer whose keys and values are read (-1: its own)
+    // Attention
+    MaskSpec mask;
+    int kv_from = -1;                             // the layer whose keys and values are read (-1: its own)
+    QkNorm qk_norm = QkNorm::AllHeads;
+    AttnPairs pairs = AttnPairs::Halves;
+    float softcap = 0.0f;                         // scores through cap * tanh(. / cap); 0: none
+    bool out_gate = false;                        // a sigmoid gate per output element
+    // LinearState
+    LinearKind linear = LinearKind::Constant;
+    int norm_parts = 1;
+    std::vector<float> log_decay;                 // Constant: per head
+};
+
+// Two mixers over one input.  Scaled: scale[0] left + scale[1] right.  Normed: half the sum of the two, each through an RMS norm.
+enum class Combine { Single, Scaled, Normed };
+struct LayerSpec {
+    MixerSpec mix[2];                             // the second one: side by side with the first
+    Combine combine = Combine::Single;
+    float mix_scale[2] = {1.0f, 1.0f};
+    int mixers() const { return combine == Combine::Single ? 1 : 2; }
     FfnKind ffn = FfnKind::None;
     int ff = 0;
     MoeSpec moe;
 };
 
 // A stack of layers with norms on the sublayers' outputs, x += norm1(mixer(x)), x += norm2(ffn(x)); norm_inputs: on their
-// inputs too, x += norm1b(mixer(norm1(x))), x += norm2b(ffn(norm2(x))).
+// inputs too, x += norm1b(mixer(norm1(x))), x += norm2b(ffn(norm2(x))).  side_dim: every layer ends with
+// x += norm(proj(gelu(gate x) * e)), e the layer's part of the token's row in a table of [vocab, layers * side_dim].
 struct ArchSpec {
     std::string name;
     std::vector<LayerSpec> layers;
     int width = 0, vocab = 0;
     float eps = 1e-6f;
     bool norm_inputs = false;
+    bool norm_one_plus = false;  // norm weights stored around zero: 1 + w
+    int side_dim = 0;
     float embed_scale = 1.0f;
     float logit_scale = 1.0f, logit_softcap = 0.0f;  // softcap 0: none
 };

@@ -31,7 +31,9 @@ enum DenseEpilogue {
     DENSE_LOG_DECAY = 2,  // -e0[row / e_div] * softplus(y + e1[row]), 32-bit
     DENSE_LOGITS = 3,     // y * scale, then cap * tanh(. / cap) when cap > 0
     DENSE_GATED_SILU = 4, // rows in pairs (2i: gate, 2i + 1: up): out row i = silu(gate) * up
-    DENSE_SPLIT_RELU2 = 5 // rows below `split` as they are, in 32-bit, to `out`; the others squared relu, in the activations' type, to out2
+    DENSE_SPLIT_RELU2 = 5, // rows below `split` as they are, in 32-bit, to `out`; the others squared relu, in the activations' type, to out2
+    DENSE_SPLIT_SILU = 6,  // the same with silu up to row `silu_end`, and the rest as they are
+    DENSE_GELU_TABLE = 7   // gelu (tanh form) times element `row` of the token's row in a table (0 for ids outside it)
 };
 // A product of one of several matrices per token (experts): the tokens come as tiles of rows that share a matrix.
 struct ExpertTile { int32_t expert, first, rows, row0; };  // rows first .. first + rows - 1 of the expert's list; row0: the first one's row in expert order
@@ -59,8 +61,12 @@ struct DenseArgs {
     const float* e1 = nullptr;
     int e_div = 1;
     float scale = 1.0f, cap = 0.0f;
-    void* out2 = nullptr;         // DENSE_SPLIT_RELU2
+    void* out2 = nullptr;         // DENSE_SPLIT_*
     int ldo2 = 0, split = 0;      // split: a multiple of 32
+    int silu_end = 0;             // DENSE_SPLIT_SILU
+    const __nv_bfloat16* table = nullptr;  // DENSE_GELU_TABLE: rows table_ld apart
+    int table_ld = 0, table_rows = 0;
+    const int64_t* ids = nullptr;
     const ExpertPlan* plan = nullptr;  // matrix = expert; output rows in expert order, input rows too unless `gather`
     bool gather = false;          // input row of a tile's row = its token
     bool f32 = false;
@@ -107,8 +113,12 @@ struct MoeSum {
     const float* gate = nullptr;     // [T] rows ld_gate apart, before the sigmoid; null: y is not read
     int ld_gate = 0;
 };
+// The output of two mixers side by side: (rms_norm(y) * w0 + rms_norm(y2) * w1) / 2.
+struct PairSum {
+    const float *y2 = nullptr, *w0 = nullptr, *w1 = nullptr;  // y2 null: no pair
+};
 // x[t] += rms_norm(y[t]) * w; act != null: the sum as activations, through rms_norm(.) * w_next when that is given.  With a
-// mixture y is first replaced by its output (x null: nothing more happens).
+// mixture or a pair y is first replaced by its output (x null: nothing more happens).
 struct ResidualArgs {
     float* y = nullptr;
     const float *w = nullptr, *w_next = nullptr;
@@ -119,6 +129,7 @@ struct ResidualArgs {
     int ld_act = 0;
     bool f32 = false;
     MoeSum moe;
+    PairSum pair;
 };
 int32_t launch_residual(const ResidualArgs& a, cudaStream_t s);
 // out[i] = rms_norm(x[idx ? idx[i] : i]) * w as activations
@@ -227,9 +238,12 @@ int32_t launch_latent_prefill(const LatentArgs& a, const LatentPrefill& p, int n
 
 // ---- gqa_attention.cu: attention over the keys and values of a paged cache, [page][kv head][page_tokens][pitch] ----------------
 struct AttnShape {
-    int heads, kv_heads, dim, vdim, dp, ep, rot_dims;  // dp, ep: dim, vdim rounded up to 8; rotation pairs i with i + rot_dims / 2
-    float scale;
+    int heads, kv_heads, dim, vdim, dp, ep, rot_dims;  // dp, ep: dim, vdim rounded up to 8
+    float scale, cap;                                  // cap > 0: scores through cap * tanh(. / cap)
     int window, keep_first;                            // MaskSpec
+    QkNorm norm;
+    AttnPairs pairs;
+    int taps;                                          // of the convolutions on q, k and v (0: none; then norm is not AllHeads)
     int k_pitch, v_pitch, k_swz, v_swz;                // cache rows (attn_cache_layout): elements apart; 7: chunks swizzled by position
 };
 void attn_cache_layout(AttnShape* g, bool f32);
@@ -238,6 +252,9 @@ struct AttnArgs {
     const float* proj = nullptr;       // [T][ld_proj] q | k | v
     int ld_proj = 0, off_k = -1, off_v = 0;  // off_k < 0: the layer has no keys and values of its own
     const float *q_norm = nullptr, *k_norm = nullptr;
+    const float* conv = nullptr;       // [channels q | k | v][taps], the last column weighs the current token
+    float* ring = nullptr;             // [slot][taps][channels]: the inputs of the last `taps` positions, entry position % taps
+    bool one_each = false;             // every token is the only one of its sequence: attn_prep also keeps its inputs
     float eps = 1e-6f;
     const float2* rot = nullptr;       // [position][rot_dims / 2] (cos, sin)
     void* q = nullptr;                 // [T][heads][dp]
@@ -246,11 +263,15 @@ struct AttnArgs {
     const int32_t *page_table = nullptr, *tok_seq = nullptr, *tok_pos = nullptr;
     int pages_per_seq = 0, T = 0;
     const float* sink = nullptr;       // [heads] or null
+    const void* gate = nullptr;        // [T][ld_gate] activations, heads vdim apart: sigmoid(gate) on the output; null: none
+    int ld_gate = 0;
+    float out_scale = 1.0f;
     void* out = nullptr;               // [T][ldo], heads ep apart
     int ldo = 0;
     bool f32 = false;
 };
-int32_t launch_attn_prep(const AttnArgs& a, cudaStream_t s);   // norms over all of q and of k, rotation, cache append
+int32_t launch_attn_prep(const AttnArgs& a, cudaStream_t s);   // convolutions, norms of q and k, rotation, cache append
+int32_t launch_attn_keep(const AttnArgs& a, const SeqRun* runs, int n_runs, cudaStream_t s);  // the runs' last inputs, behind attn_prep
 struct AttnScratch { float* part = nullptr; size_t part_bytes = 0; unsigned* tickets = nullptr; int n_tickets = 0; };
 size_t attn_part_bytes(const AttnShape& g);
 int32_t launch_attn_tokens(const AttnArgs& a, const AttnScratch& sc, cudaStream_t s);  // tokens 0 .. T - 1, each over its own context
@@ -258,6 +279,45 @@ int32_t launch_attn_tokens(const AttnArgs& a, const AttnScratch& sc, cudaStream_
 struct AttnTile { int32_t tok0, n, seq, pos0; };
 bool attn_tiles_apply(const AttnShape& g, bool f32);
 int32_t launch_attn_tiles(const AttnArgs& a, const AttnTile* tiles, int n_tiles, cudaStream_t s);
+
+// ---- linear_state.cu: S_t = decay_t S_(t-1) + step_t k_t v_t^T, o_t = S_t^T q_t (+ skip v_t), per head, S in f32 -------------------------
+struct LinearShape {
+    LinearKind kind;
+    int heads, groups, dim, vdim;      // q, k: groups x dim; v: heads x vdim
+    int ld, off_v, off_k, off_q, off_g;  // columns of the projected rows: v, k, q (StateSpace: before the convolution), gate
+    int ld_dt, off_dt;                 // StateSpace: where the steps are projected to
+    int taps, channels, ld_in;         // StateSpace: channels v | k | q, one after the other from off_v on; ld_in: rows of `in`
+    int norm_parts;
+    float eps;
+};
+struct LinearArgs {
+    LinearShape g;
+    const void* proj = nullptr;        // [T][ld] activations
+    const float* dt = nullptr;         // [T][ld_dt] 32-bit part of the projection
+    const float *conv = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_exp = nullptr, *skip = nullptr;  // StateSpace; a_exp = e^A_log
+    const float* log_decay = nullptr;  // Constant: [heads]
+    void* ring = nullptr;              // [slot][taps][channels] activations
+    void* in = nullptr;                // StateSpace: [T][ld_in] v | k | q behind convolution and silu
+    float* state = nullptr;            // [slot][heads][dim][vdim]
+    const int32_t *tok_seq = nullptr, *tok_pos = nullptr;
+    int T = 0;
+    float* o = nullptr;                // [T][heads * vdim]
+    const SeqRun* runs = nullptr;      // walked token by token
+    int n_runs = 0;
+    const DeltaChunkRun* chunk_runs = nullptr;  // in chunks of kDeltaChunk tokens
+    int n_chunk_runs = 0;
+    const SeqRun* all_runs = nullptr;  // all of them, for the inputs that the next call's convolutions need
+    int n_all_runs = 0;
+    const float* norm_w = nullptr;     // [heads * vdim]
+    float out_scale = 1.0f;
+    void* out = nullptr;               // [T][ldo] activations
+    int ldo = 0;
+    bool f32 = false;
+};
+bool linear_chunks_apply(const LinearShape& g, bool f32);
+int32_t launch_linear_runs(const LinearArgs& a, int* launches, cudaStream_t s);  // convolutions, the recurrence over all runs, the kept inputs
+int32_t launch_linear_step(const LinearArgs& a, cudaStream_t s);                 // the same for one token per sequence
+int32_t launch_linear_output(const LinearArgs& a, cudaStream_t s);               // gate and norm
 
 // ---- expert_choice.cu: routing ---------------------------------------------------------------------------------------------
 struct ChoiceArgs {
@@ -277,11 +337,9 @@ int32_t launch_expert_choice(const ChoiceArgs& a, cudaStream_t s);
 int32_t launch_expert_gather(const MoeSum& m, int width, int T, void* out, int ldo, cudaStream_t s);
 
 // ---- a stack of such layers (layers.cu) --------------------------------------------------------------------------------
-struct StackLayer {
-    LayerSpec s;
-    // norms of the sublayers' inputs (null: none) and outputs
-    const float *norm1_in = nullptr, *norm1_out = nullptr, *norm2_in = nullptr, *norm2_out = nullptr;
-    DenseWeight in, out, up, down;     // GatedSilu: `up` = gate and up rows in turn
+struct MixerUnit {
+    MixerSpec s;
+    DenseWeight in, out;            // (two mixers side by side: StackLayer has these)
     // ChannelDelta: `in` = q | k | v | a1 | g1 | b
     DenseWeight a2, g2;
     DeltaShape dg{};
@@ -299,14 +357,33 @@ struct StackLayer {
     void* cache = nullptr;
     // Attention: `in` = q | k | v (q alone when another layer's cache is read)
     AttnShape ag{};
-    int off_k = -1, off_v = 0;
+    int off_k = -1, off_v = 0;      // off_g: the output gate, in the activations' part
     const float *k_norm = nullptr, *sink = nullptr;
     void *k_cache = nullptr, *v_cache = nullptr;
+    // LinearState
+    LinearShape ng{};
+    const float *conv_b = nullptr, *skip = nullptr, *log_decay = nullptr;
+};
+struct StackLayer {
+    LayerSpec s;
+    MixerUnit mix[2];
+    // two mixers side by side: what both read projected by one product, 32-bit rows below in_split, activations behind it (silu up
+    // to row silu_end); their outputs lie side by side in rows of mixed_ld, the second one's from mixed_off on, and leave through
+    // `out` together (Scaled) or through one matrix each (Normed)
+    DenseWeight in, out, out2;
+    int in_split = 0, silu_end = 0, mixed_off = 0, mixed_ld = 0;
+    const float* out_norm[2] = {nullptr, nullptr};
+    // norms of the sublayers' inputs (null: none) and outputs
+    const float *norm1_in = nullptr, *norm1_out = nullptr, *norm2_in = nullptr, *norm2_out = nullptr;
+    DenseWeight up, down;              // GatedSilu: `up` = gate and up rows in turn
     // Moe: `up` and `down` of all experts; `route` = router | gate of the shared expert | (from row route_split on) its up
     DenseWeight route, shared_down;
     int off_gate = 0, route_split = 0;
     const float* correction = nullptr;
     uint64_t expert_bytes = 0;         // one expert's matrices
+    // token input
+    DenseWeight side_gate, side_proj;
+    const float* side_norm = nullptr;
 };
 struct LayerStack {
     ArchSpec spec;
@@ -314,6 +391,7 @@ struct LayerStack {
     std::vector<StackLayer> layers;
     DenseWeight head;
     const __nv_bfloat16* embed = nullptr;
+    const __nv_bfloat16* side_embed = nullptr;
     const float* final_norm = nullptr;
     DenseWorkspace ws;
     std::vector<void*> owned;
@@ -323,8 +401,9 @@ struct LayerStack {
     uint64_t cache_bytes_per_token = 0, state_bytes_per_seq = 0;
     // step buffers for t_cap tokens
     int width_p = 0;
-    void *xa = nullptr, *proj = nullptr, *gate = nullptr, *mixed = nullptr, *cq = nullptr, *q = nullptr, *q_abs = nullptr, *o_lat = nullptr, *ffn = nullptr, *last = nullptr;
-    float *y = nullptr, *projf = nullptr, *log_decay = nullptr, *qk = nullptr, *v = nullptr, *o = nullptr;
+    void *xa = nullptr, *proj = nullptr, *gate = nullptr, *mixed = nullptr, *cq = nullptr, *q = nullptr, *q_abs = nullptr, *o_lat = nullptr, *ffn = nullptr, *last = nullptr,
+         *side = nullptr, *lin = nullptr;
+    float *y = nullptr, *y2 = nullptr, *projf = nullptr, *log_decay = nullptr, *qk = nullptr, *v = nullptr, *o = nullptr;
     SeqRun* d_runs = nullptr;
     int n_runs = 0;
     // gated delta rule of the call: short runs walk token by token, long ones in chunks (when every such layer has that form)

@@ -170,6 +170,7 @@ int32_t stack_bind(lc_model* m);   // weights
 int32_t stack_alloc(lc_model* m);  // cache, state and step buffers, sized by the handle's pool and slots
 void stack_free(lc_model* m);
 uint64_t stack_step_bytes(const lc_model* m, int ctx);
+uint64_t stack_table_bytes(const lc_model* m);  // of tables of which a step reads one row per token (the embedding apart)
 int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const std::vector<int32_t>& pos);
 int32_t stack_run_layers(lc_model* m, int T, bool decode_step);
 int32_t stack_head(lc_model* m, int n, const int32_t* idx, float* logits);  // logits of rows idx (null: rows 0 .. n - 1)

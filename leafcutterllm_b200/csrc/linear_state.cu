@@ -1,0 +1,613 @@
+// Linear recurrences with one decay per head (LinearShape): S_t = e^(l_t) S_(t-1) + b_t k_t v_t^T, o_t = S_t^T q_t + skip v_t.
+// Constant: l from the config, b = 1, q, k, v already through silu (the product's epilogue).  StateSpace: b = softplus(dt + bias),
+// l = -a b, q and k shared by the heads of a group; v, k and q come through a short convolution with bias and silu.
+// S, l, b and all sums are f32; q, k and v are activations (A = bf16, or float when a model runs in true 32-bit).
+//   linear_conv_kernel    convolutions of a call's tokens
+//   linear_scan_kernel    the recurrence token by token: short runs, f32 models
+//   linear_chunk_kernel   long runs, 64 tokens at a time on the tensor cores.  With G_t the sum of l inside the chunk,
+//                           o_t = e^(G_t) S0^T q_t + sum_(s <= t) (q_t . k_s) e^(G_t - G_s) b_s v_s,
+//                           S = e^(G_end) S0 + sum_s k_s (e^(G_end - G_s) b_s v_s)^T;
+//                         q, k and v enter as they are, the f32 factors (weights, scaled values, S0) as two bf16 halves
+//   linear_step_kernel    one token per sequence: convolution, recurrence
+//   linear_output_kernel  gate and norm: Constant rms_norm(o) w sigmoid(gate) over all heads, StateSpace rms_norm(o silu(gate)) w in parts
+#include <algorithm>
+#include <cmath>
+#include "lc_mixers.h"
+#include "lc_mma.cuh"
+#include "lc_tma.cuh"
+
+namespace lc {
+
+namespace {
+
+__device__ __forceinline__ float silu_any(float v) { return v / (1.0f + expf(-v)); }
+__device__ __forceinline__ float softplus_of(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+// (b, l) of head h at token t
+__device__ __forceinline__ float2 step_decay(const LinearArgs& a, size_t t, int h) {
+    if (a.g.kind == LinearKind::Constant) return make_float2(1.0f, a.log_decay[h]);
+    const float b = softplus_of(a.dt[t * a.g.ld_dt + a.g.off_dt + h] + a.dt_bias[h]);
+    return make_float2(b, -a.a_exp[h] * b);
+}
+// Rows of v | k | q that the recurrence reads.
+template <typename A> struct Rows { const A* p; int ld, v, k, q; };
+template <typename A>
+__device__ __forceinline__ Rows<A> rows_of(const LinearArgs& a) {
+    const LinearShape& g = a.g;
+    if (g.kind == LinearKind::Constant) return {(const A*)a.proj, g.ld, g.off_v, g.off_k, g.off_q};
+    return {(const A*)a.in, g.ld_in, 0, g.heads * g.vdim, g.heads * g.vdim + g.groups * g.dim};
+}
+
+template <typename A> __device__ __forceinline__ float2 two(const A* p);
+template <> __device__ __forceinline__ float2 two<float>(const float* p) { return *(const float2*)p; }
+template <> __device__ __forceinline__ float2 two<bf16>(const bf16* p) { return __bfloat1622float2(*(const __nv_bfloat162*)p); }
+template <typename A> __device__ __forceinline__ void put_two(A* p, float2 v);
+template <> __device__ __forceinline__ void put_two<float>(float* p, float2 v) { *(float2*)p = v; }
+template <> __device__ __forceinline__ void put_two<bf16>(bf16* p, float2 v) { *(uint32_t*)p = pack2(v.x, v.y); }
+
+// A thread walks kConvTok tokens of two neighbouring channels and keeps their last inputs in registers (TAPS of them; 0: any
+// number, re-read).  Inputs of earlier positions come from the call's rows as far as they belong to the same run, from the ring
+// before that, and are zero before the sequence's start.
+constexpr int kConvTok = 16;
+template <typename A, int TAPS>
+__global__ void __launch_bounds__(128) linear_conv_kernel(const LinearArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const LinearShape& g = a.g;
+    const int c = (blockIdx.y * 128 + threadIdx.x) * 2;
+    if (c >= g.channels) return;
+    const bool both = c + 1 < g.channels;
+    const int taps = TAPS > 0 ? TAPS : g.taps;
+    constexpr int kT = TAPS > 0 ? TAPS : 1;
+    const A* in = (const A*)a.proj + g.off_v + c;
+    const A* ring = (const A*)a.ring + c;
+    const float2 bias = make_float2(a.conv_b[c], both ? a.conv_b[c + 1] : 0.0f);
+    auto weight = [&](int j) { return make_float2(a.conv[(size_t)c * taps + j], both ? a.conv[(size_t)(c + 1) * taps + j] : 0.0f); };
+    float2 w[kT], win[kT];
+    if constexpr (TAPS > 0)
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) w[j] = weight(j);
+    const int t0 = blockIdx.x * kConvTok, t1 = min(a.T, t0 + kConvTok);
+    int prev_seq = -1, prev_pos = -1;
+    for (int t = t0; t < t1; t++) {
+        const int seq = a.tok_seq[t], pos = a.tok_pos[t];
+        auto back = [&](int j) {
+            if (pos - j < 0) return make_float2(0.0f, 0.0f);
+            const int tt = t - j;
+            if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) return two<A>(in + (size_t)tt * g.ld);
+            const A* r = ring + ((size_t)seq * taps + (pos - j) % taps) * g.channels;
+            return make_float2(act_f<A>(r[0]), both ? act_f<A>(r[1]) : 0.0f);
+        };
+        const float2 u = two<A>(in + (size_t)t * g.ld);
+        float2 y = bias;
+        if constexpr (TAPS > 0) {
+            if (seq != prev_seq || pos != prev_pos + 1)
+#pragma unroll
+                for (int j = 1; j < TAPS; j++) win[j - 1] = back(j);
+#pragma unroll
+            for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[TAPS - 1 - j].x, win[j - 1].x, y.x); y.y = fmaf(w[TAPS - 1 - j].y, win[j - 1].y, y.y); }
+            y.x = fmaf(w[TAPS - 1].x, u.x, y.x); y.y = fmaf(w[TAPS - 1].y, u.y, y.y);
+#pragma unroll
+            for (int j = TAPS - 1; j > 0; j--) win[j] = win[j - 1];
+            win[0] = u;
+            prev_seq = seq; prev_pos = pos;
+        } else {
+            for (int j = taps - 1; j >= 0; j--) {
+                const float2 v = j == 0 ? u : back(j), cw = weight(taps - 1 - j);
+                y.x = fmaf(cw.x, v.x, y.x); y.y = fmaf(cw.y, v.y, y.y);
+            }
+        }
+        put_two<A>((A*)a.in + (size_t)t * g.ld_in + c, make_float2(silu_any(y.x), silu_any(y.y)));
+    }
+}
+
+// The inputs of a run's last `taps` positions, for the convolutions of the next call.
+template <typename A>
+__global__ void __launch_bounds__(256) linear_keep_kernel(const LinearArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const LinearShape& g = a.g;
+    const SeqRun run = a.all_runs[blockIdx.x];
+    const int c = blockIdx.y * 256 + threadIdx.x;
+    if (c >= g.channels) return;
+    for (int t = max(0, run.n - g.taps); t < run.n; t++)
+        ((A*)a.ring)[((size_t)run.seq * g.taps + (run.pos0 + t) % g.taps) * g.channels + c] = ((const A*)a.proj)[(size_t)(run.tok0 + t) * g.ld + g.off_v + c];
+}
+
+// A CTA of four warps owns 32 value columns of one head of one run; four lanes share a column's `dim` state entries (DPL each:
+// float4 groups dealt round robin), eight columns per warp.
+constexpr int kScanTok = 16;  // tokens staged in shared memory at a time
+template <typename A, int DPL>
+__global__ void __launch_bounds__(128) linear_scan_kernel(const LinearArgs a) {
+    constexpr int DP = DPL * 4;
+    extern __shared__ __align__(16) float sm[];
+    float *s_q = sm, *s_k = s_q + kScanTok * DP, *s_v = s_k + kScanTok * DP, *s_b = s_v + kScanTok * 32, *s_g = s_b + kScanTok;
+    pdl_launch_dependents();
+    pdl_wait();
+    const LinearShape& g = a.g;
+    const SeqRun run = a.runs[blockIdx.x];
+    const int h = blockIdx.y, kg = h / (g.heads / g.groups);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r4 = lane & 3, col = warp * 8 + (lane >> 2), e = blockIdx.z * 32 + col;
+    float* st = a.state + ((size_t)run.seq * g.heads + h) * g.dim * g.vdim;
+    const Rows<A> src = rows_of<A>(a);
+    const float skip = a.skip ? a.skip[h] : 0.0f;
+    float S[DPL];
+#pragma unroll
+    for (int i = 0; i < DPL; i++) {
+        const int d = (i >> 2) * 16 + r4 * 4 + (i & 3);
+        S[i] = (run.pos0 > 0 && d < g.dim && e < g.vdim) ? st[(size_t)d * g.vdim + e] : 0.0f;
+    }
+    for (int c0 = 0; c0 < run.n; c0 += kScanTok) {
+        const int m = min(kScanTok, run.n - c0);
+        __syncthreads();
+        for (int i = threadIdx.x; i < m * DP; i += 128) {
+            const int t = i / DP, d = i - t * DP;
+            const A* row = src.p + (size_t)(run.tok0 + c0 + t) * src.ld + kg * g.dim + d;
+            s_q[i] = d < g.dim ? act_f<A>(row[src.q]) : 0.0f;
+            s_k[i] = d < g.dim ? act_f<A>(row[src.k]) : 0.0f;
+        }
+        for (int i = threadIdx.x; i < m * 32; i += 128) {
+            const int t = i >> 5, c = blockIdx.z * 32 + (i & 31);
+            s_v[i] = c < g.vdim ? act_f<A>(src.p[(size_t)(run.tok0 + c0 + t) * src.ld + src.v + h * g.vdim + c]) : 0.0f;
+        }
+        if (threadIdx.x < m) {
+            const float2 bl = step_decay(a, (size_t)(run.tok0 + c0 + threadIdx.x), h);
+            s_b[threadIdx.x] = bl.x;
+            s_g[threadIdx.x] = expf(bl.y);
+        }
+        __syncthreads();
+        for (int t = 0; t < m; t++) {
+            const float4 *q4 = (const float4*)(s_q + t * DP), *k4 = (const float4*)(s_k + t * DP);
+            const float v = s_v[t * 32 + col], u = s_b[t] * v, decay = s_g[t];
+            float o = 0.0f;
+#pragma unroll
+            for (int i = 0; i < DPL / 4; i++) {
+                const float4 kv = k4[i * 4 + r4], qv = q4[i * 4 + r4];
+                const float kk[4] = {kv.x, kv.y, kv.z, kv.w}, qq[4] = {qv.x, qv.y, qv.z, qv.w};
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    S[4 * i + j] = fmaf(kk[j], u, S[4 * i + j] * decay);
+                    o = fmaf(S[4 * i + j], qq[j], o);
+                }
+            }
+            o += __shfl_xor_sync(0xffffffffu, o, 1);
+            o += __shfl_xor_sync(0xffffffffu, o, 2);
+            if (r4 == 0 && e < g.vdim) a.o[(size_t)(run.tok0 + c0 + t) * g.heads * g.vdim + h * g.vdim + e] = fmaf(skip, v, o);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < DPL; i++) {
+        const int d = (i >> 2) * 16 + r4 * 4 + (i & 3);
+        if (d < g.dim && e < g.vdim) st[(size_t)d * g.vdim + e] = S[i];
+    }
+}
+
+// ---- long runs --------------------------------------------------------------------------------------------------------------
+// A CTA of four warps walks the chunks of one run for 32 value columns of one head.  Per chunk a warp owns 16 tokens of the
+// read-outs and a quarter of S's key rows (DP: `dim` padded; few rows: a quarter of the (16 x 8) tiles), which stays in registers
+// as the accumulators of its update; its halves are published for the next chunk's read-outs.
+constexpr int kC = kDeltaChunk, kCols = 32, kVP = kCols + 8;
+__host__ __device__ constexpr size_t chunk_smem(int dp) {
+    return (size_t)(2 * 2 * kC * (dp + 8) + 2 * kC * kVP + 2 * dp * kVP + 2 * kC * kVP) * 2 + 3 * kC * sizeof(float);
+}
+template <int DP>
+__global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
+    constexpr int QP = DP + 8, kMT = DP / 16, kOwnM = kMT >= 4 ? kMT / 4 : 1, kOwnN = kMT >= 4 ? 4 : 2;
+    static_assert(kMT >= 2, "at least two tiles of key rows");
+    extern __shared__ __align__(16) unsigned char smem[];
+    bf16 *s_q = (bf16*)smem, *s_k = s_q + 2 * kC * QP, *s_v = s_k + 2 * kC * QP, *s_S = s_v + 2 * kC * kVP, *s_w = s_S + 2 * DP * kVP;
+    float *s_gh = (float*)(s_w + 2 * kC * kVP), *s_gl = s_gh + kC, *s_b = s_gl + kC;  // G in log2 units as a sum of two floats
+    pdl_launch_dependents();
+    pdl_wait();
+    const LinearShape& g = a.g;
+    const DeltaChunkRun cr = a.chunk_runs[blockIdx.x];
+    const int h = blockIdx.y, kg = h / (g.heads / g.groups), e0 = blockIdx.z * kCols;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+    const Rows<bf16> src = rows_of<bf16>(a);
+    const float skip = a.skip ? a.skip[h] : 0.0f;
+    float* st = a.state + ((size_t)cr.run.seq * g.heads + h) * g.dim * g.vdim;
+    const int m0 = kMT >= 4 ? warp * kOwnM : warp & 1, n0 = kMT >= 4 ? 0 : (warp >> 1) * 2;
+    const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), v_sm = smem_u32(s_v), S_sm = smem_u32(s_S), w_sm = smem_u32(s_w);
+    auto load = [&](int c) {
+        const int buf = c & 1, left = cr.run.n - c * kC;
+        const bf16* row = src.p + (size_t)(cr.run.tok0 + c * kC) * src.ld;
+        for (int i = tid; i < kC * (DP / 8); i += 128) {
+            const int t = i / (DP / 8), d = (i - t * (DP / 8)) * 8;
+            const bool in = t < left && d < g.dim;
+            const bf16* p = row + (in ? (size_t)t * src.ld + kg * g.dim + d : 0);
+            const uint32_t at = (uint32_t)((buf * kC + t) * QP + d) * 2;
+            cp16(q_sm + at, p + (in ? src.q : 0), in ? 16 : 0);
+            cp16(k_sm + at, p + (in ? src.k : 0), in ? 16 : 0);
+        }
+        for (int i = tid; i < kC * (kCols / 8); i += 128) {
+            const int t = i / (kCols / 8), e = (i & (kCols / 8 - 1)) * 8;
+            const bool in = t < left && e0 + e < g.vdim;
+            cp16(v_sm + (uint32_t)((buf * kC + t) * kVP + e) * 2, row + (in ? (size_t)t * src.ld + src.v + h * g.vdim + e0 + e : 0), in ? 16 : 0);
+        }
+        cp_commit();
+    };
+    float2 bl[2];  // warp 0: step and log decay of tokens 2 lane, 2 lane + 1 of the chunk to come; behind the run's end neither
+    auto fetch = [&](int c) {
+        if (warp == 0)
+#pragma unroll
+            for (int j = 0; j < 2; j++) {
+                const int t = c * kC + 2 * lane + j;
+                bl[j] = t < cr.run.n ? step_decay(a, (size_t)(cr.run.tok0 + t), h) : make_float2(0.0f, 0.0f);
+            }
+    };
+    load(0);
+    fetch(0);
+    float S[kOwnM][kOwnN][4];
+#pragma unroll
+    for (int i = 0; i < kOwnM; i++)
+#pragma unroll
+        for (int n = 0; n < kOwnN; n++)
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                const int d = (m0 + i) * 16 + g8 + 8 * r, e = e0 + (n0 + n) * 8 + 2 * t4;
+                float2 v = make_float2(0.0f, 0.0f);
+                if (cr.run.pos0 > 0 && d < g.dim && e < g.vdim) v = *(const float2*)(st + (size_t)d * g.vdim + e);
+                S[i][n][2 * r] = v.x; S[i][n][2 * r + 1] = v.y;
+            }
+    auto publish = [&]() {
+#pragma unroll
+        for (int i = 0; i < kOwnM; i++)
+#pragma unroll
+            for (int n = 0; n < kOwnN; n++)
+#pragma unroll
+                for (int r = 0; r < 2; r++) {
+                    uint32_t hi, lo;
+                    split2(S[i][n][2 * r], S[i][n][2 * r + 1], hi, lo);
+                    bf16* dst = s_S + ((m0 + i) * 16 + g8 + 8 * r) * kVP + (n0 + n) * 8 + 2 * t4;
+                    *(uint32_t*)dst = hi;
+                    *(uint32_t*)(dst + DP * kVP) = lo;
+                }
+    };
+    publish();
+    const int krow = (lane & 7) + ((lane >> 4) << 3), kcol = ((lane >> 3) & 1) * 8, vrow = lane & 15, vcol = (lane >> 4) * 8;
+    for (int c = 0; c < cr.n_chunks; c++) {
+        const int buf = c & 1;
+        if (warp == 0) {
+            const double l0 = (double)bl[0].y * 1.4426950408889634, l1 = (double)bl[1].y * 1.4426950408889634;
+            double sum = l0 + l1;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const double up = __shfl_up_sync(0xffffffffu, sum, o);
+                if (lane >= o) sum += up;
+            }
+            const double at[2] = {sum - l1, sum};
+#pragma unroll
+            for (int j = 0; j < 2; j++) {
+                const float hi = (float)at[j];
+                s_gh[2 * lane + j] = hi;
+                s_gl[2 * lane + j] = (float)(at[j] - (double)hi);
+                s_b[2 * lane + j] = bl[j].x;
+            }
+        }
+        cp_wait<0>();
+        __syncthreads();  // the chunk's rows, G and S are there; nobody reads the other buffers any more
+        if (c + 1 < cr.n_chunks) { load(c + 1); fetch(c + 1); }
+        const float eh = s_gh[kC - 1], el = s_gl[kC - 1], keep = exp2f(eh + el);
+        for (int i = tid; i < kC * (kCols / 2); i += 128) {  // values on their way into S
+            const int t = i / (kCols / 2), e = (i & (kCols / 2 - 1)) * 2;
+            const float f = s_b[t] * exp2f((eh - s_gh[t]) + (el - s_gl[t]));
+            const float2 v = two<bf16>(s_v + (buf * kC + t) * kVP + e);
+            uint32_t hi, lo;
+            split2(v.x * f, v.y * f, hi, lo);
+            *(uint32_t*)(s_w + t * kVP + e) = hi;
+            *(uint32_t*)(s_w + (kC + t) * kVP + e) = lo;
+        }
+        float p[8][4], o[4][4], oi[4][4];
+#pragma unroll
+        for (int n = 0; n < 8; n++) p[n][0] = p[n][1] = p[n][2] = p[n][3] = 0.0f;
+#pragma unroll
+        for (int n = 0; n < 4; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = oi[n][0] = oi[n][1] = oi[n][2] = oi[n][3] = 0.0f;
+#pragma unroll 2
+        for (int kk = 0; kk < DP / 16; kk++) {
+            uint32_t q4[4];
+            ldsm4(q_sm + (uint32_t)((buf * kC + 16 * warp + vrow) * QP + 16 * kk + vcol) * 2, q4);
+#pragma unroll
+            for (int n = 0; n < 4; n++) {
+                if (n > warp) break;
+                uint32_t kb[4];
+                ldsm4(k_sm + (uint32_t)((buf * kC + 16 * n + krow) * QP + 16 * kk + kcol) * 2, kb);
+                mma_bf16(p[2 * n], q4, kb[0], kb[1]);
+                mma_bf16(p[2 * n + 1], q4, kb[2], kb[3]);
+            }
+#pragma unroll
+            for (int n = 0; n < 2; n++)
+#pragma unroll
+                for (int half = 0; half < 2; half++) {
+                    uint32_t sb[4];
+                    ldsm4t(S_sm + (uint32_t)((half * DP + 16 * kk + vrow) * kVP + 16 * n + vcol) * 2, sb);
+                    mma_bf16(oi[2 * n], q4, sb[0], sb[1]);
+                    mma_bf16(oi[2 * n + 1], q4, sb[2], sb[3]);
+                }
+        }
+        const int tr[2] = {16 * warp + g8, 16 * warp + g8 + 8};
+        const float gh[2] = {s_gh[tr[0]], s_gh[tr[1]]}, gl[2] = {s_gl[tr[0]], s_gl[tr[1]]};
+#pragma unroll
+        for (int ks = 0; ks < 4; ks++) {
+            if (ks > warp) break;
+            uint32_t ph[4], pl[4];
+#pragma unroll
+            for (int hs = 0; hs < 2; hs++) {
+                const int s0 = 16 * ks + 8 * hs + 2 * t4;
+                float f[4];
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    const int s = s0 + (j & 1), r = j >> 1;
+                    f[j] = s <= tr[r] ? p[2 * ks + hs][j] * s_b[s] * exp2f((gh[r] - s_gh[s]) + (gl[r] - s_gl[s])) : 0.0f;
+                }
+                split2(f[0], f[1], ph[2 * hs], pl[2 * hs]);
+                split2(f[2], f[3], ph[2 * hs + 1], pl[2 * hs + 1]);
+            }
+#pragma unroll
+            for (int n = 0; n < 2; n++) {
+                uint32_t b[4];
+                ldsm4t(v_sm + (uint32_t)((buf * kC + 16 * ks + vrow) * kVP + 16 * n + vcol) * 2, b);
+                mma_bf16(o[2 * n], ph, b[0], b[1]);
+                mma_bf16(o[2 * n + 1], ph, b[2], b[3]);
+                mma_bf16(o[2 * n], pl, b[0], b[1]);
+                mma_bf16(o[2 * n + 1], pl, b[2], b[3]);
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < 2; r++) {
+            const int t = c * kC + tr[r];
+            if (t >= cr.run.n) continue;
+            const float f = exp2f(gh[r] + gl[r]);
+            float* dst = a.o + (size_t)(cr.run.tok0 + t) * g.heads * g.vdim + h * g.vdim + e0 + 2 * t4;
+#pragma unroll
+            for (int n = 0; n < 4; n++) {
+                if (e0 + 8 * n >= g.vdim) break;
+                const float2 v = two<bf16>(s_v + (buf * kC + tr[r]) * kVP + 8 * n + 2 * t4);
+                *(float2*)(dst + 8 * n) = make_float2(fmaf(f, oi[n][2 * r], o[n][2 * r]) + skip * v.x, fmaf(f, oi[n][2 * r + 1], o[n][2 * r + 1]) + skip * v.y);
+            }
+        }
+        __syncthreads();  // the scaled values are there, S has been read
+#pragma unroll
+        for (int i = 0; i < kOwnM; i++)
+#pragma unroll
+            for (int n = 0; n < kOwnN; n++) { S[i][n][0] *= keep; S[i][n][1] *= keep; S[i][n][2] *= keep; S[i][n][3] *= keep; }
+#pragma unroll
+        for (int ks = 0; ks < 4; ks++) {
+            uint32_t wb[2][kOwnN / 2][4];
+#pragma unroll
+            for (int half = 0; half < 2; half++)
+#pragma unroll
+                for (int n = 0; n < kOwnN / 2; n++) ldsm4t(w_sm + (uint32_t)((half * kC + 16 * ks + vrow) * kVP + n0 * 8 + 16 * n + vcol) * 2, wb[half][n]);
+#pragma unroll
+            for (int i = 0; i < kOwnM; i++) {
+                uint32_t kt[4];  // keys transposed: rows are key dimensions, columns tokens
+                ldsm4t(k_sm + (uint32_t)((buf * kC + 16 * ks + krow) * QP + (m0 + i) * 16 + kcol) * 2, kt);
+#pragma unroll
+                for (int half = 0; half < 2; half++)
+#pragma unroll
+                    for (int n = 0; n < kOwnN / 2; n++) {
+                        mma_bf16(S[i][2 * n], kt, wb[half][n][0], wb[half][n][1]);
+                        mma_bf16(S[i][2 * n + 1], kt, wb[half][n][2], wb[half][n][3]);
+                    }
+            }
+        }
+        publish();
+    }
+#pragma unroll
+    for (int i = 0; i < kOwnM; i++)
+#pragma unroll
+        for (int n = 0; n < kOwnN; n++)
+#pragma unroll
+            for (int r = 0; r < 2; r++) {
+                const int d = (m0 + i) * 16 + g8 + 8 * r, e = e0 + (n0 + n) * 8 + 2 * t4;
+                if (d < g.dim && e < g.vdim) *(float2*)(st + (size_t)d * g.vdim + e) = make_float2(S[i][n][2 * r], S[i][n][2 * r + 1]);
+            }
+}
+
+// ---- one token per sequence -----------------------------------------------------------------------------------------------------
+// One CTA per (head, token); a thread owns VEC neighbouring value columns and every `groups`-th key row, kept in registers (ROWS of
+// them; 0: re-read).  The ring entry written here is not one that any head reads in this step.
+constexpr int kStepThreads = 256;
+template <typename A, int VEC, int ROWS>
+__global__ void __launch_bounds__(kStepThreads) linear_step_kernel(const LinearArgs a) {
+    extern __shared__ float sm[];
+    pdl_launch_dependents();
+    pdl_wait();
+    const LinearShape& g = a.g;
+    const int h = blockIdx.x, t = blockIdx.y, rep = g.heads / g.groups, kg = h / rep, seq = a.tok_seq[t], pos = a.tok_pos[t], tid = threadIdx.x;
+    const int cols = g.vdim / VEC, groups = kStepThreads / cols, c = tid % cols, gr = tid / cols;
+    float *s_q = sm, *s_k = s_q + g.dim, *s_v = s_k + g.dim, *s_o = s_v + g.vdim;
+    float* st = a.state + ((size_t)seq * g.heads + h) * g.dim * g.vdim + c * VEC;
+    const bool live = pos > 0, mine = gr < groups;
+    float S[ROWS > 0 ? ROWS : 1][VEC];
+    auto load = [&](int d, float (&v)[VEC]) {
+#pragma unroll
+        for (int j = 0; j < VEC; j++) v[j] = 0.0f;
+        if (!live) return;
+        if constexpr (VEC == 4) { const float4 x = *(const float4*)(st + (size_t)d * g.vdim); v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; }
+        else v[0] = st[(size_t)d * g.vdim];
+    };
+    if (ROWS > 0 && mine) {  // the state's reads travel while the inputs are made
+#pragma unroll
+        for (int i = 0; i < ROWS; i++)
+            if (gr + i * groups < g.dim) load(gr + i * groups, S[i]);
+    }
+    const float2 bl = step_decay(a, (size_t)t, h);
+    const A* proj = (const A*)a.proj + (size_t)t * g.ld;
+    for (int i = tid; i < 2 * g.dim + g.vdim; i += kStepThreads) {
+        const int part = i < g.dim ? 0 : i < 2 * g.dim ? 1 : 2;  // q, k, v
+        const int at = part == 0 ? kg * g.dim + i : part == 1 ? kg * g.dim + i - g.dim : h * g.vdim + i - 2 * g.dim;
+        const A cur = proj[(part == 0 ? g.off_q : part == 1 ? g.off_k : g.off_v) + at];
+        float y = act_f<A>(cur);
+        if (g.kind == LinearKind::StateSpace) {
+            const int channel = (part == 0 ? g.off_q : part == 1 ? g.off_k : g.off_v) - g.off_v + at;
+            A* ring = (A*)a.ring + (size_t)seq * g.taps * g.channels + channel;
+            const float* w = a.conv + (size_t)channel * g.taps;
+            float acc = a.conv_b[channel];
+            for (int j = g.taps - 1; j > 0; j--)
+                if (pos - j >= 0) acc = fmaf(w[g.taps - 1 - j], act_f<A>(ring[(size_t)((pos - j) % g.taps) * g.channels]), acc);
+            y = act_f<A>(to_act<A>(silu_any(fmaf(w[g.taps - 1], y, acc))));  // the type that runs of tokens keep it in
+            if (part == 2 || h % rep == 0) ring[(size_t)(pos % g.taps) * g.channels] = cur;
+        }
+        sm[i] = y;
+    }
+    const float decay = expf(bl.y);
+    __syncthreads();
+    if (mine) {
+        float u[VEC], o[VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; j++) { u[j] = bl.x * s_v[c * VEC + j]; o[j] = 0.0f; }
+        auto turn = [&](int d, float (&v)[VEC]) {
+            const float k = s_k[d], q = s_q[d];
+#pragma unroll
+            for (int j = 0; j < VEC; j++) { v[j] = fmaf(k, u[j], v[j] * decay); o[j] = fmaf(v[j], q, o[j]); }
+            if constexpr (VEC == 4) *(float4*)(st + (size_t)d * g.vdim) = make_float4(v[0], v[1], v[2], v[3]);
+            else st[(size_t)d * g.vdim] = v[0];
+        };
+        if constexpr (ROWS > 0) {
+#pragma unroll
+            for (int i = 0; i < ROWS; i++)
+                if (gr + i * groups < g.dim) turn(gr + i * groups, S[i]);
+        } else {
+            for (int d = gr; d < g.dim; d += groups) { load(d, S[0]); turn(d, S[0]); }
+        }
+#pragma unroll
+        for (int j = 0; j < VEC; j++) s_o[gr * g.vdim + c * VEC + j] = o[j];
+    }
+    __syncthreads();
+    const float skip = a.skip ? a.skip[h] : 0.0f;
+    for (int e = tid; e < g.vdim; e += kStepThreads) {
+        float o = skip * s_v[e];
+        for (int i = 0; i < groups; i++) o += s_o[i * g.vdim + e];
+        a.o[((size_t)t * g.heads + h) * g.vdim + e] = o;
+    }
+}
+
+// One CTA per (token, part of the norm).
+template <typename A>
+__global__ void __launch_bounds__(256) linear_output_kernel(const LinearArgs a) {
+    __shared__ float sh[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const LinearShape& g = a.g;
+    const int inner = g.heads * g.vdim, n = inner / g.norm_parts, e0 = blockIdx.y * n;
+    const size_t t = blockIdx.x;
+    const bool gate_first = g.kind == LinearKind::StateSpace;
+    const float* o = a.o + t * inner + e0;
+    const A* gate = (const A*)a.proj + t * g.ld + g.off_g + e0;
+    auto value = [&](int e) { return gate_first ? o[e] * silu_any(act_f<A>(gate[e])) : o[e]; };
+    constexpr int kHeld = 8;  // elements of a thread that stay in registers between the passes
+    float v[kHeld], ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kHeld; i++) {
+        const int e = threadIdx.x + i * blockDim.x;
+        v[i] = e < n ? value(e) : 0.0f;
+        ss = fmaf(v[i], v[i], ss);
+    }
+    for (int e = threadIdx.x + kHeld * blockDim.x; e < n; e += blockDim.x) { const float x = value(e); ss = fmaf(x, x, ss); }
+    const float r = a.out_scale / sqrtf(block_sum_once(ss, sh) / (float)n + g.eps);
+    A* dst = (A*)a.out + t * a.ldo + e0;
+    auto put = [&](int e, float x) {
+        x *= r * a.norm_w[e0 + e];
+        dst[e] = to_act<A>(gate_first ? x : x * sigmoid_f(act_f<A>(gate[e])));
+    };
+#pragma unroll
+    for (int i = 0; i < kHeld; i++) {
+        const int e = threadIdx.x + i * blockDim.x;
+        if (e < n) put(e, v[i]);
+    }
+    for (int e = threadIdx.x + kHeld * blockDim.x; e < n; e += blockDim.x) put(e, value(e));
+}
+
+int padded_dim(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
+
+template <typename A>
+int32_t conv_dispatch(const LinearArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)((a.T + kConvTok - 1) / kConvTok), (unsigned)((a.g.channels + 255) / 256));
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(launch_pdl(kern, grid, dim3(128), 0, s, a));
+        return LC_OK;
+    };
+    switch (a.g.taps) {
+        case 2: return go(linear_conv_kernel<A, 2>);
+        case 3: return go(linear_conv_kernel<A, 3>);
+        case 4: return go(linear_conv_kernel<A, 4>);
+        default: return go(linear_conv_kernel<A, 0>);
+    }
+}
+
+template <typename A>
+int32_t scan_dispatch(const LinearArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)a.n_runs, (unsigned)a.g.heads, (unsigned)((a.g.vdim + 31) / 32));
+    const int dp = padded_dim(a.g.dim);
+    const size_t smem = (size_t)kScanTok * (2 * dp + 32 + 2) * sizeof(float);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+        LC_CUDA(launch_pdl(kern, grid, dim3(128), smem, s, a));
+        return LC_OK;
+    };
+    switch (dp) {
+        case 32: return go(linear_scan_kernel<A, 8>);
+        case 64: return go(linear_scan_kernel<A, 16>);
+        case 128: return go(linear_scan_kernel<A, 32>);
+        default: return go(linear_scan_kernel<A, 64>);
+    }
+}
+
+int32_t chunk_dispatch(const LinearArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)a.n_chunk_runs, (unsigned)a.g.heads, (unsigned)((a.g.vdim + kCols - 1) / kCols));
+    const int dp = padded_dim(a.g.dim);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, chunk_smem(dp)));
+        LC_CUDA(launch_pdl(kern, grid, dim3(128), chunk_smem(dp), s, a));
+        return LC_OK;
+    };
+    switch (dp) {
+        case 32: return go(linear_chunk_kernel<32>);
+        case 64: return go(linear_chunk_kernel<64>);
+        case 128: return go(linear_chunk_kernel<128>);
+        default: return go(linear_chunk_kernel<256>);
+    }
+}
+
+template <typename A>
+int32_t step_dispatch(const LinearArgs& a, cudaStream_t s) {
+    const int vec = a.g.vdim % 4 == 0 ? 4 : 1, cols = a.g.vdim / vec;
+    LC_CHECK(cols <= kStepThreads, LC_ERR_UNSUPPORTED, "linear recurrence: %d value dimensions per head", a.g.vdim);
+    const int groups = kStepThreads / cols, rows = (a.g.dim + groups - 1) / groups;
+    const size_t smem = (size_t)(2 * a.g.dim + a.g.vdim + groups * a.g.vdim) * sizeof(float);
+    const dim3 grid((unsigned)a.g.heads, (unsigned)a.T);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(ensure_smem_limit((const void*)kern, smem));
+        LC_CUDA(launch_pdl(kern, grid, dim3(kStepThreads), smem, s, a));
+        return LC_OK;
+    };
+    if (vec == 4) return rows <= 4 ? go(linear_step_kernel<A, 4, 4>) : rows <= 8 ? go(linear_step_kernel<A, 4, 8>) : rows <= 16 ? go(linear_step_kernel<A, 4, 16>) : go(linear_step_kernel<A, 4, 0>);
+    return rows <= 16 ? go(linear_step_kernel<A, 1, 16>) : go(linear_step_kernel<A, 1, 0>);
+}
+
+}  // namespace
+
+bool linear_chunks_apply(const LinearShape& g, bool f32) { return !f32 && g.dim % 8 == 0 && g.vdim % 8 == 0 && g.dim <= 256; }
+
+int32_t launch_linear_runs(const LinearArgs& a, int* launches, cudaStream_t s) {
+    LC_CHECK(a.g.dim <= 256, LC_ERR_UNSUPPORTED, "linear recurrence: %d state dimensions per head (at most 256)", a.g.dim);
+    const bool conv = a.g.kind == LinearKind::StateSpace;
+    if (conv) { LC_TRY(a.f32 ? conv_dispatch<float>(a, s) : conv_dispatch<bf16>(a, s)); ++*launches; }
+    if (a.n_runs) { LC_TRY(a.f32 ? scan_dispatch<float>(a, s) : scan_dispatch<bf16>(a, s)); ++*launches; }
+    if (a.n_chunk_runs) { LC_TRY(chunk_dispatch(a, s)); ++*launches; }
+    if (!conv) return LC_OK;
+    const dim3 grid((unsigned)a.n_all_runs, (unsigned)((a.g.channels + 255) / 256));
+    if (a.f32) LC_CUDA(launch_pdl(linear_keep_kernel<float>, grid, dim3(256), 0, s, a));
+    else LC_CUDA(launch_pdl(linear_keep_kernel<bf16>, grid, dim3(256), 0, s, a));
+    ++*launches;
+    return LC_OK;
+}
+int32_t launch_linear_step(const LinearArgs& a, cudaStream_t s) { return a.f32 ? step_dispatch<float>(a, s) : step_dispatch<bf16>(a, s); }
+int32_t launch_linear_output(const LinearArgs& a, cudaStream_t s) {
+    const int n = a.g.heads * a.g.vdim / a.g.norm_parts;
+    const dim3 grid((unsigned)a.T, (unsigned)a.g.norm_parts), block((unsigned)std::min(256, (n + 31) / 32 * 32));
+    if (a.f32) LC_CUDA(launch_pdl(linear_output_kernel<float>, grid, block, 0, s, a));
+    else LC_CUDA(launch_pdl(linear_output_kernel<bf16>, grid, block, 0, s, a));
+    return LC_OK;
+}
+
+}  // namespace lc

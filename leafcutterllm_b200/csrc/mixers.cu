@@ -100,10 +100,11 @@ __device__ __forceinline__ float sq4(float4 v, float ss) { return fmaf(v.x, v.x,
 __device__ __forceinline__ void add4(float4& y, float w, float4 v) { y.x = fmaf(w, v.x, y.x); y.y = fmaf(w, v.y, y.y); y.z = fmaf(w, v.z, y.z); y.w = fmaf(w, v.w, y.w); }
 
 // VEC = 4: rows of a multiple of four elements; a row of up to 16 elements per thread stays in registers between its passes.
-template <typename A, int VEC, bool MOE>
+template <typename A, int VEC, bool MOE, bool PAIR>
 __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
     constexpr int kHeld = 4;
-    __shared__ float sh[32], sh2[32];
+    constexpr bool kMade = MOE || PAIR;  // the output is made here, not read
+    __shared__ float sh[32], sh2[32], sh_p[2][32];
     __shared__ long long s_row[kMaxChoices];
     __shared__ float s_w[kMaxChoices], s_gate;
     pdl_launch_dependents();
@@ -128,10 +129,30 @@ __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
         for (int j = 0; j < a.moe.top; j++) own += s_row[j] < 0 ? s_w[j] : 0.0f;
         gate = s_gate;
     }
+    const float* y2 = PAIR ? a.pair.y2 + t * width : nullptr;
+    float f0 = 0.0f, f1 = 0.0f;  // half the reciprocal roots of the pair's mean squares
+    if constexpr (PAIR) {
+        float s0 = 0.0f, s1 = 0.0f;
+        if constexpr (VEC == 4)
+            for (int c = threadIdx.x * 4; c < width; c += blockDim.x * 4) { s0 = sq4(*(const float4*)(yr + c), s0); s1 = sq4(*(const float4*)(y2 + c), s1); }
+        else
+            for (int c = threadIdx.x; c < width; c += blockDim.x) { s0 = fmaf(yr[c], yr[c], s0); s1 = fmaf(y2[c], y2[c], s1); }
+        s0 = warp_sum(s0); s1 = warp_sum(s1);
+        if ((threadIdx.x & 31) == 0) { sh_p[0][threadIdx.x >> 5] = s0; sh_p[1][threadIdx.x >> 5] = s1; }
+        __syncthreads();
+        s0 = s1 = 0.0f;
+        for (unsigned w = 0; w < blockDim.x / 32; w++) { s0 += sh_p[0][w]; s1 += sh_p[1][w]; }
+        f0 = 0.5f / sqrtf(s0 / (float)width + a.eps);
+        f1 = 0.5f / sqrtf(s1 / (float)width + a.eps);
+    }
     float ss = 0.0f;
     if constexpr (VEC == 4) {
         float4 yv[kHeld], xv[kHeld];
         auto out_at = [&](int c) {
+            if constexpr (PAIR) {
+                const float4 p = *(const float4*)(yr + c), q = *(const float4*)(y2 + c), u = *(const float4*)(a.pair.w0 + c), v = *(const float4*)(a.pair.w1 + c);
+                return make_float4(p.x * f0 * u.x + q.x * f1 * v.x, p.y * f0 * u.y + q.y * f1 * v.y, p.z * f0 * u.z + q.z * f1 * v.z, p.w * f0 * u.w + q.w * f1 * v.w);
+            }
             if constexpr (!MOE) return *(const float4*)(yr + c);
             float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
             if (a.moe.gate) add4(y, gate, *(const float4*)(yr + c));
@@ -152,10 +173,10 @@ __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
         }
         for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < width; c += blockDim.x * 4) {
             const float4 v = out_at(c);
-            if (MOE) *(float4*)(yr + c) = v;
+            if (kMade) *(float4*)(yr + c) = v;
             ss = sq4(v, ss);
         }
-        if (MOE && !a.x) return;
+        if (kMade && !a.x) return;
         ss = block_sum_once(ss, sh);
         const float r = 1.0f / sqrtf(ss / (float)width + a.eps);
         float s2 = 0.0f;
@@ -194,10 +215,13 @@ __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
                     if (s_row[j] >= 0) v = fmaf(s_w[j], act_f<A>(((const A*)a.moe.rows)[s_row[j] + c]), v);
                 if (own != 0.0f) v = fmaf(own, act_f<A>(hr[c]), v);
                 yr[c] = v;
+            } else if constexpr (PAIR) {
+                v = yr[c] * f0 * a.pair.w0[c] + y2[c] * f1 * a.pair.w1[c];
+                yr[c] = v;
             } else v = yr[c];
             ss = fmaf(v, v, ss);
         }
-        if (MOE && !a.x) return;
+        if (kMade && !a.x) return;
         ss = block_sum_once(ss, sh);
         const float r = 1.0f / sqrtf(ss / (float)width + a.eps);
         float s2 = 0.0f;
@@ -732,19 +756,21 @@ int32_t launch_act_rows(const float* x, int width, int T, void* act, int ld_act,
 }
 int32_t launch_residual(const ResidualArgs& a, cudaStream_t s) {
     const dim3 grid((unsigned)a.T), block((unsigned)norm_threads(a.width));
-    const bool moe = a.moe.rows != nullptr;
-    const bool vec = a.width % 4 == 0 && (uintptr_t)a.w % 16 == 0 && (uintptr_t)a.w_next % 16 == 0 && (a.moe.ld_rows | a.moe.ld_h | a.ld_act) % 4 == 0;
+    const bool moe = a.moe.rows != nullptr, pair = a.pair.y2 != nullptr;
+    const bool vec = a.width % 4 == 0 && ((uintptr_t)a.pair.w0 | (uintptr_t)a.pair.w1) % 16 == 0 && (uintptr_t)a.w % 16 == 0 && (uintptr_t)a.w_next % 16 == 0 && (a.moe.ld_rows | a.moe.ld_h | a.ld_act) % 4 == 0;
     LC_CHECK(a.moe.top <= kMaxChoices && (!a.w_next || a.act), LC_ERR_INVALID, "residual sum: bad argument");
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(launch_pdl(kern, grid, block, 0, s, a));
         return LC_OK;
     };
     if (a.f32) {
-        if (moe) return vec ? go(residual_kernel<float, 4, true>) : go(residual_kernel<float, 1, true>);
-        return vec ? go(residual_kernel<float, 4, false>) : go(residual_kernel<float, 1, false>);
+        if (moe) return vec ? go(residual_kernel<float, 4, true, false>) : go(residual_kernel<float, 1, true, false>);
+        if (pair) return vec ? go(residual_kernel<float, 4, false, true>) : go(residual_kernel<float, 1, false, true>);
+        return vec ? go(residual_kernel<float, 4, false, false>) : go(residual_kernel<float, 1, false, false>);
     }
-    if (moe) return vec ? go(residual_kernel<bf16, 4, true>) : go(residual_kernel<bf16, 1, true>);
-    return vec ? go(residual_kernel<bf16, 4, false>) : go(residual_kernel<bf16, 1, false>);
+    if (moe) return vec ? go(residual_kernel<bf16, 4, true, false>) : go(residual_kernel<bf16, 1, true, false>);
+    if (pair) return vec ? go(residual_kernel<bf16, 4, false, true>) : go(residual_kernel<bf16, 1, false, true>);
+    return vec ? go(residual_kernel<bf16, 4, false, false>) : go(residual_kernel<bf16, 1, false, false>);
 }
 int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, float eps, int width, int n, void* out, int ldo, bool f32, cudaStream_t s) {
     const dim3 grid((unsigned)n), block((unsigned)norm_threads(width));
