@@ -185,15 +185,18 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
         return even ? *(const float2*)(row + c) : make_float2(row[c], c + 1 < n ? row[c + 1] : 0.0f);
     };
     const int t0 = blockIdx.x * stretch, t1 = min(a.T, t0 + stretch);
-    float2 w[NP][kTaps], win[NP][kWin], gain[NP];  // win[.][j]: the input j + 1 tokens back
+    float w[NP][2][kTaps], win[NP][2][kWin];  // win[.][.][j]: the input j + 1 tokens back
+    float2 gain[NP];
     const float* gw = is_q ? a.q_norm : a.k_norm;
 #pragma unroll
     for (int p = 0; p < NP; p++) {
         const int c = 2 * (lane + 32 * p);
         if constexpr (TAPS > 0)
 #pragma unroll
-            for (int j = 0; j < TAPS; j++)
-                w[p][j] = make_float2(c < n ? a.conv[(size_t)(ch0 + c) * TAPS + j] : 0.0f, c + 1 < n ? a.conv[(size_t)(ch0 + c + 1) * TAPS + j] : 0.0f);
+            for (int j = 0; j < TAPS; j++) {
+                w[p][0][j] = c < n ? a.conv[(size_t)(ch0 + c) * TAPS + j] : 0.0f;
+                w[p][1][j] = c + 1 < n ? a.conv[(size_t)(ch0 + c + 1) * TAPS + j] : 0.0f;
+            }
         gain[p] = g.norm == QkNorm::PerHead && !is_v ? make_float2(c < n ? gw[c] : 0.0f, c + 1 < n ? gw[c + 1] : 0.0f) : make_float2(1.0f, 1.0f);
     }
     int prev_seq = -1, prev_pos = -1;
@@ -216,16 +219,20 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
             const float2 u = pair_at(row, c);
             x[p] = u;
             if constexpr (TAPS > 0) {
-                if (fresh)
+                if (fresh) {
 #pragma unroll
-                    for (int j = 1; j < TAPS; j++) win[p][j - 1] = back(j, c);
+                    for (int j = 1; j < TAPS; j++) {
+                        const float2 v = back(j, c);
+                        win[p][0][j - 1] = v.x; win[p][1][j - 1] = v.y;
+                    }
+                }
                 float2 y = make_float2(0.0f, 0.0f);
 #pragma unroll
-                for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[p][TAPS - 1 - j].x, win[p][j - 1].x, y.x); y.y = fmaf(w[p][TAPS - 1 - j].y, win[p][j - 1].y, y.y); }
-                x[p] = make_float2(fmaf(w[p][TAPS - 1].x, u.x, y.x), fmaf(w[p][TAPS - 1].y, u.y, y.y));
+                for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[p][0][TAPS - 1 - j], win[p][0][j - 1], y.x); y.y = fmaf(w[p][1][TAPS - 1 - j], win[p][1][j - 1], y.y); }
+                x[p] = make_float2(fmaf(w[p][0][TAPS - 1], u.x, y.x), fmaf(w[p][1][TAPS - 1], u.y, y.y));
 #pragma unroll
-                for (int j = TAPS - 2; j > 0; j--) win[p][j] = win[p][j - 1];
-                win[p][0] = u;
+                for (int j = TAPS - 2; j > 0; j--) { win[p][0][j] = win[p][0][j - 1]; win[p][1][j] = win[p][1][j - 1]; }
+                win[p][0][0] = u.x; win[p][1][0] = u.y;
             } else if constexpr (TAPS < 0) {
                 float2 y = make_float2(0.0f, 0.0f);
                 if (c < n)

@@ -62,10 +62,15 @@ __global__ void __launch_bounds__(128) linear_conv_kernel(const LinearArgs a) {
     const A* ring = (const A*)a.ring + c;
     const float2 bias = make_float2(a.conv_b[c], both ? a.conv_b[c + 1] : 0.0f);
     auto weight = [&](int j) { return make_float2(a.conv[(size_t)c * taps + j], both ? a.conv[(size_t)(c + 1) * taps + j] : 0.0f); };
-    float2 w[kT], win[kT];
-    if constexpr (TAPS > 0)
+    float w[2][kT], win[2][kT];  // win[.][j]: the input j + 1 tokens back
+    if constexpr (TAPS > 0) {
 #pragma unroll
-        for (int j = 0; j < TAPS; j++) w[j] = weight(j);
+        for (int j = 0; j < TAPS; j++) {
+            const float2 v = weight(j);
+            w[0][j] = v.x; w[1][j] = v.y;
+            win[0][j] = win[1][j] = 0.0f;
+        }
+    }
     const int t0 = blockIdx.x * kConvTok, t1 = min(a.T, t0 + kConvTok);
     int prev_seq = -1, prev_pos = -1;
     for (int t = t0; t < t1; t++) {
@@ -80,15 +85,19 @@ __global__ void __launch_bounds__(128) linear_conv_kernel(const LinearArgs a) {
         const float2 u = two<A>(in + (size_t)t * g.ld);
         float2 y = bias;
         if constexpr (TAPS > 0) {
-            if (seq != prev_seq || pos != prev_pos + 1)
+            if (seq != prev_seq || pos != prev_pos + 1) {
 #pragma unroll
-                for (int j = 1; j < TAPS; j++) win[j - 1] = back(j);
+                for (int j = 1; j < TAPS; j++) {
+                    const float2 v = back(j);
+                    win[0][j - 1] = v.x; win[1][j - 1] = v.y;
+                }
+            }
 #pragma unroll
-            for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[TAPS - 1 - j].x, win[j - 1].x, y.x); y.y = fmaf(w[TAPS - 1 - j].y, win[j - 1].y, y.y); }
-            y.x = fmaf(w[TAPS - 1].x, u.x, y.x); y.y = fmaf(w[TAPS - 1].y, u.y, y.y);
+            for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[0][TAPS - 1 - j], win[0][j - 1], y.x); y.y = fmaf(w[1][TAPS - 1 - j], win[1][j - 1], y.y); }
+            y.x = fmaf(w[0][TAPS - 1], u.x, y.x); y.y = fmaf(w[1][TAPS - 1], u.y, y.y);
 #pragma unroll
-            for (int j = TAPS - 1; j > 0; j--) win[j] = win[j - 1];
-            win[0] = u;
+            for (int j = TAPS - 1; j > 0; j--) { win[0][j] = win[0][j - 1]; win[1][j] = win[1][j - 1]; }
+            win[0][0] = u.x; win[1][0] = u.y;
             prev_seq = seq; prev_pos = pos;
         } else {
             for (int j = taps - 1; j >= 0; j--) {
