@@ -208,7 +208,8 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
             if (pos - j < 0) return make_float2(0.0f, 0.0f);
             const int tt = t - j;
             if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) return pair_at(a.proj + (size_t)tt * a.ld_proj + col0, c);
-            return pair_at(a.ring + ((size_t)seq * taps + (pos - j) % taps) * channels + ch0, c);
+            const float* r = a.ring + ((size_t)seq * taps + (pos - j) % taps) * channels + ch0 + c;  // rows of any length: not aligned for pairs
+            return make_float2(c < n ? r[0] : 0.0f, c + 1 < n ? r[1] : 0.0f);
         };
         float2 x[NP];
         const bool fresh = seq != prev_seq || pos != prev_pos + 1;

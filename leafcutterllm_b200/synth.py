@@ -120,14 +120,47 @@ class LayeredSpec:
             return name, TYPE_BF16, (cols, rows), "normal"
         def vec(name, n, kind="ones"):
             return name, TYPE_BF16, (n,), kind
+        munisun = c["architecture"] == "Munisun"
+        gain = "zeros" if munisun else "ones"  # Munisun's layer norms are stored around zero
         yield mat("embed", c["vocab"], W)
+        if munisun:
+            yield mat("side.embed", c["vocab"], len(c["layers"]) * c["token_side"]["dim"])
         for i, ly in enumerate(c["layers"]):
             m, p = ly["mixer"], f"l{i}.mix."
-            H, D, E = m["heads"], m["dim"], m["vdim"]
-            both = ("", "b") if c["architecture"] == "Tenetar" else ("",)  # norms on inputs and outputs, or on outputs only
+            H, D, E = (0, 0, 0) if munisun else (m["heads"], m["dim"], m["vdim"])
+            both = ("",) if c["architecture"] == "Varasun" else ("", "b")  # norms on outputs only, or on inputs and outputs
             for end in both:
-                yield vec(f"l{i}.norm1{end}", W)
-            if ly["type"] == "attention":
+                yield vec(f"l{i}.norm1{end}", W, gain)
+            if munisun:
+                a, r, left, right = m["left"], m["right"], p + "left.", p + "right."
+                nq, nk, nv, inner = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], a["kv_heads"] * a["vdim"], r["heads"] * r["vdim"]
+                for t, n in (("q", nq), ("k", nk), ("v", nv)):
+                    yield mat(left + t, n, W)
+                    if "conv" in a:
+                        yield mat(left + t + ".conv", n, a["conv"])
+                yield mat(left + "o", W, a["heads"] * a["vdim"])
+                if ly["type"] == "parallel":
+                    yield vec(left + "q.norm", a["dim"])
+                    yield vec(left + "k.norm", a["dim"])
+                    yield mat(left + "g", a["heads"] * a["vdim"], W)
+                    channels = inner + 2 * r["groups"] * r["state"]
+                    yield mat(right + "in", inner + channels + r["heads"], W)
+                    yield mat(right + "conv", channels, r["conv"])
+                    yield vec(right + "conv.b", channels, "normal")
+                    for t in ("dt_bias", "A_log", "D"):
+                        yield vec(right + t, r["heads"], "normal")
+                else:
+                    for t, n in (("q", r["heads"] * r["dim"]), ("k", r["heads"] * r["dim"]), ("v", inner), ("g", inner)):
+                        yield mat(right + t, n, W)
+                    yield vec(left + "out", W)
+                    yield vec(right + "out", W)
+                yield vec(right + "norm", inner)
+                yield mat(right + "o", W, inner)
+                n = c["token_side"]["dim"]
+                yield mat(f"l{i}.side.gate", n, W)
+                yield mat(f"l{i}.side.proj", W, n)
+                yield vec(f"l{i}.side.norm", W)
+            elif ly["type"] == "attention":
                 G = m["kv_heads"]
                 yield mat(p + "q", H * D, W)
                 yield vec(p + "q.norm", H * D)
@@ -165,25 +198,29 @@ class LayeredSpec:
             if mlp is None:
                 continue
             for end in both:
-                yield vec(f"l{i}.norm2{end}", W)
+                yield vec(f"l{i}.norm2{end}", W, gain)
             if mlp["kind"] == "moe":
-                r, F, SF = mlp["router"], mlp["expert"]["ff"], mlp["shared"]["ff"]
-                n = r["experts"] + r["identity"]
+                r, F, SF = mlp["router"], mlp["expert"]["ff"], mlp.get("shared", {}).get("ff", 0)
+                n = r["experts"] + r.get("identity", 0)
                 yield mat(p + "router", n, W)
                 yield vec(p + "correction", n, "zeros")  # random routers are balanced as they are
                 for e in range(r["experts"]):
+                    if munisun:
+                        yield mat(f"{p}e{e}.gate", F, W)
                     yield mat(f"{p}e{e}.up", F, W)
                     yield mat(f"{p}e{e}.down", W, F)
+                if not SF:
+                    continue
                 yield mat(p + "shared.up", SF, W)
                 yield mat(p + "shared.down", W, SF)
                 yield mat(p + "shared.sg", 1, W)
                 continue
             F = mlp["ff"]
-            if c["architecture"] == "Tenetar":
+            if c["architecture"] != "Varasun":
                 yield mat(p + "gate", F, W)
             yield mat(p + "up", F, W)
             yield mat(p + "down", W, F)
-        yield vec("final.norm", W)
+        yield vec("final.norm", W, gain)
         yield mat("head", c["vocab"], W)
 
 
@@ -216,6 +253,25 @@ def tenetar_spec(name: str, width: int, pattern: str, ff: int, vocab: int, heads
                "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": groups, "keep": keep}}}
         layers.append({"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": ff} if ch == "d" else moe})
     return LayeredSpec(name, {"architecture": "Tenetar", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5}, "layers": layers})
+
+
+def munisun_spec(name: str, width: int, pattern: str, ff: int, vocab: int, heads: int, kv_heads: int, experts: int, top: int, groups: int, keep: int, expert_ff: int,
+                 head_dim: int = 128, space_heads: int = 0, space_dim: int = 64, space_state: int = 128, space_groups: int = 8, side: int = 256) -> LayeredSpec:
+    """pattern: two letters per layer: s = attention beside a state space, l = attention beside lightning attention; then d = dense
+    feed-forward, m = mixture, n = none."""
+    layers = []
+    space_heads = space_heads or 2 * width // space_dim
+    for kind, mlp in zip(pattern[::2], pattern[1::2]):
+        left = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "rot": {"dims": head_dim, "base": 500000.0}}
+        if kind == "s":
+            left["rot"]["scaling"] = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}
+            mixer = {"left": dict(left, softcap=50.0), "left_scale": 1.0, "right_scale": 1.0,
+                     "right": {"heads": space_heads, "vdim": space_dim, "state": space_state, "groups": space_groups, "conv": 4, "norm_groups": space_groups}}
+        else:
+            mixer = {"left": dict(left, conv=4), "right": {"heads": heads, "dim": head_dim, "vdim": head_dim, "decay": [1.0 - 2.0 ** (-3.0 - 8.0 * h / heads) for h in range(heads)]}}
+        moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
+        layers.append({"type": "parallel" if kind == "s" else "parallel_2", "mixer": mixer, "mlp": {"d": {"kind": "dense", "ff": ff}, "m": moe, "n": None}[mlp]})
+    return LayeredSpec(name, {"architecture": "Munisun", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5}, "token_side": {"dim": side}, "layers": layers})
 
 
 def build_layered_engine(spec: LayeredSpec, seed: int = WEIGHT_SEED, **engine_kwargs):

@@ -113,6 +113,128 @@ def tenetar_mixed():
                            attention(window=1000, keep_first=0, kv_from=0), with_ff(attention(window=9, keep_first=2, kv_from=0), 17)])
 
 
+def conv_attention(heads=6, kv_heads=3, dim=20, vdim=12, rot_dims=8, base=10000.0, scaling=None, scale=0.4, softcap=None, conv=3):
+    """scaling: (factor, low, high, original).  conv None: the kind with norms per head ahead of the rotation and a gate."""
+    rot = {"dims": rot_dims, "base": base}
+    if scaling:
+        rot["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "rot": rot}
+    if softcap is not None:
+        m["softcap"] = softcap
+    return m if conv is None else dict(m, conv=conv)
+
+
+def gated_attention(heads=6, kv_heads=2, dim=28, vdim=20, rot_dims=12, base=500.0, scaling=(4.0, 1.0, 3.0, 40), scale=0.25, softcap=5.0):
+    return conv_attention(heads, kv_heads, dim, vdim, rot_dims, base, scaling, scale, softcap, None)
+
+
+def state_space(heads=6, groups=3, state=20, vdim=12, conv=4, norm_groups=2):
+    return {"heads": heads, "groups": groups, "state": state, "vdim": vdim, "conv": conv, "norm_groups": norm_groups}
+
+
+def lightning(decay=(0.3, 0.9, 0.99, 1.0, 0.0), dim=12, vdim=20):
+    return {"heads": len(decay), "dim": dim, "vdim": vdim, "decay": list(decay)}
+
+
+def scaled_pair(left=None, right=None, left_scale=0.7, right_scale=1.2):
+    return {"type": "parallel", "mixer": {"left": left or gated_attention(), "right": right or state_space(), "left_scale": left_scale, "right_scale": right_scale}, "mlp": None}
+
+
+def normed_pair(left=None, right=None):
+    return {"type": "parallel_2", "mixer": {"left": left or conv_attention(), "right": right or lightning()}, "mlp": None}
+
+
+def with_gated_experts(layer, experts=12, top=3, groups=3, keep=2, ff=24):
+    return dict(layer, mlp={"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}})
+
+
+def munisun_config(layers, width=104, vocab=131, eps=1e-5, embed_scale=1.7, side=11):
+    return {"architecture": "Munisun", "width": width, "vocab": vocab, "norm": {"eps": eps}, "embedding": {"scale": embed_scale}, "token_side": {"dim": side}, "layers": layers}
+
+
+def munisun_weights(cfg, seed=0, fixed_choice=False, correction=0.1):
+    """Random weights, already rounded to bf16.  fixed_choice: as for tenetar_weights (no two sums of two corrections are close)."""
+    rng = np.random.default_rng(seed)
+    W, side = cfg["width"], cfg["token_side"]["dim"]
+    w = {}
+
+    def mat(name, n, k, gain=1.0):
+        w[name] = rng.normal(0, gain / np.sqrt(k), (n, k))
+
+    def gain(name, n, about=1.0):
+        w[name] = rng.normal(about, 0.2, n)
+
+    w["embed"] = rng.normal(0, 0.4, (cfg["vocab"], W))
+    w["side.embed"] = rng.normal(0, 1.0, (cfg["vocab"], len(cfg["layers"]) * side))
+    for i, ly in enumerate(cfg["layers"]):
+        l, p, q = "l%d." % i, "l%d.mix.left." % i, "l%d.mix.right." % i
+        for n in ("norm1", "norm1b"):
+            gain(l + n, W, 0.0)
+        m = ly["mixer"]["left"]
+        rows = {"q": m["heads"] * m["dim"], "k": m["kv_heads"] * m["dim"], "v": m["kv_heads"] * m["vdim"]}
+        for n, r in rows.items():
+            mat(p + n, r, W)
+            if "conv" in m:
+                w[p + n + ".conv"] = rng.normal(0, 0.6, (r, m["conv"]))
+        mat(p + "o", W, m["heads"] * m["vdim"])
+        if ly["type"] == "parallel":
+            gain(p + "q.norm", m["dim"])
+            gain(p + "k.norm", m["dim"])
+            mat(p + "g", m["heads"] * m["vdim"], W)
+            m = ly["mixer"]["right"]
+            inner, GN = m["heads"] * m["vdim"], m["groups"] * m["state"]
+            mat(q + "in", 2 * inner + 2 * GN + m["heads"], W)
+            w[q + "conv"] = rng.normal(0, 0.6, (inner + 2 * GN, m["conv"]))
+            w[q + "conv.b"] = rng.normal(0, 0.3, inner + 2 * GN)
+            w[q + "dt_bias"] = rng.uniform(-4, 1, m["heads"])
+            w[q + "A_log"] = rng.uniform(-3, 1.5, m["heads"])
+            w[q + "D"] = rng.normal(0, 1, m["heads"])
+        else:
+            m = ly["mixer"]["right"]
+            inner = m["heads"] * m["vdim"]
+            mat(q + "q", m["heads"] * m["dim"], W)
+            mat(q + "k", m["heads"] * m["dim"], W)
+            mat(q + "v", inner, W)
+            mat(q + "g", inner, W)
+            gain(p + "out", W)
+            gain(q + "out", W)
+        gain(q + "norm", inner)
+        mat(q + "o", W, inner)
+        mlp, p = ly["mlp"], l + "mlp."
+        if mlp is not None:
+            for n in ("norm2", "norm2b"):
+                gain(l + n, W, 0.0)
+            if mlp["kind"] == "dense":
+                mat(p + "gate", mlp["ff"], W)
+                mat(p + "up", mlp["ff"], W)
+                mat(p + "down", W, mlp["ff"])
+            else:
+                r, F = mlp["router"], mlp["expert"]["ff"]
+                n = r["experts"]
+                mat(p + "router", n, W, 1.5)
+                w[p + "correction"] = 3.0 * 2.0 ** rng.permutation(n) - 100.0 if fixed_choice else rng.normal(-correction, correction, n)
+                for e in range(n):
+                    mat(p + "e%d.gate" % e, F, W)
+                    mat(p + "e%d.up" % e, F, W)
+                    mat(p + "e%d.down" % e, W, F)
+        mat(l + "side.gate", side, W)
+        mat(l + "side.proj", W, side)
+        gain(l + "side.norm", W)
+    gain("final.norm", W, 0.0)
+    mat("head", cfg["vocab"], W, 2.0)
+    return {n: bf16_round(a) for n, a in w.items()}
+
+
+def munisun_mixed():
+    """Both kinds of layers in turn, every kind of feed-forward and none, sizes that differ from each other."""
+    return munisun_config([with_ff(normed_pair(), 40), with_gated_experts(scaled_pair()),
+                           with_gated_experts(normed_pair(conv_attention(heads=4, kv_heads=4, dim=16, vdim=24, rot_dims=16, conv=2), lightning((0.95, 0.5), dim=40, vdim=8)),
+                                              experts=10, top=4, groups=5, keep=3, ff=31),
+                           scaled_pair(gated_attention(heads=4, kv_heads=1, dim=16, vdim=24, rot_dims=16, scaling=None, softcap=None),
+                                       state_space(heads=2, groups=1, state=24, vdim=40, conv=3, norm_groups=5)),
+                           with_ff(scaled_pair(right=state_space(heads=4, groups=4, state=16, vdim=8, conv=2, norm_groups=1)), 17)])
+
+
 def weights(cfg, seed=0, decay_rank=5, gate_rank=7, spread=1.0):
     """Random weights, already rounded to bf16.  Products keep about unit size; decays range from slow to fast."""
     rng = np.random.default_rng(seed)
@@ -197,7 +319,7 @@ def rel_rms(got, want):
     return float(d.max() / np.sqrt(np.mean(want ** 2)))
 
 
-# Bounds on the error of the worst row and of all rows together: f32 rounding, and the rounding of bf16 activations.
+# Bounds on the error of the worst row and, from eight rows on, of all rows together: f32 rounding, and the rounding of bf16 activations.
 WORST_ROW = {"float32": 3e-5, "bfloat16": 6e-2}
 ALL_ROWS = {"float32": 1e-5, "bfloat16": 2e-2}
 
@@ -206,4 +328,9 @@ def check(got, want, dtype, slack=1):
     got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
     worst = rel_rms(got, want)
     total = float(np.sqrt(np.mean((got - want) ** 2) / np.mean(want ** 2)))
-    assert worst < slack * WORST_ROW[dtype] and total < slack * ALL_ROWS[dtype], (worst, total)
+    assert worst < slack * WORST_ROW[dtype] and (total < slack * ALL_ROWS[dtype] or got.size < 8 * got.shape[-1]), (worst, total)
+
+
+def rounding(cfg, dtype):
+    """Slack for Munisun in bf16: branches are brought to unit size before they meet, which enlarges the rounding of small outputs."""
+    return 3 if cfg["architecture"] == "Munisun" and dtype == "bfloat16" else 1

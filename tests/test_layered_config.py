@@ -117,6 +117,90 @@ def test_choice_of_experts_by_definition():
     assert sorted(e for e, _ in P.choose_experts(z, low, 3, 2, 4)) == [2, 3, 4, 5]
 
 
+@pytest.mark.parametrize("cuts", [[1] * 60, [2, 5, 1, 9, 6, 37], [58, 2]])
+def test_plain_munisun_in_portions_equals_the_whole(cuts):
+    cfg = U.munisun_mixed()
+    m = P.plain_model(cfg, U.munisun_weights(cfg))
+    toks = U.tokens(60, cfg["vocab"])
+    whole = m.forward(toks, m.new_state())
+    st, parts, at = m.new_state(), [], 0
+    for c in cuts:
+        parts.append(m.forward(toks[at : at + c], st))
+        at += c
+    assert np.abs(np.concatenate(parts) - whole).max() < 1e-9
+
+
+def test_frequencies_by_wavelength():
+    """Pairs of short wavelength stay, those of long wavelength are stretched by the factor, and the blend is continuous between."""
+    rot = {"dims": 64, "base": 10000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 512}}
+    f, g = 10000.0 ** (-np.arange(32) / 32.0), P.wavelength_frequencies(rot)
+    turns = 512 * f / (2 * np.pi)
+    assert np.allclose(g[turns > 4], f[turns > 4]) and np.allclose(g[turns < 1], f[turns < 1] / 8)
+    mid = (turns >= 1) & (turns <= 4)
+    assert mid.any() and (turns > 4).any() and (turns < 1).any()
+    assert (g[mid] <= f[mid]).all() and (g[mid] >= f[mid] / 8).all() and (np.diff(g) < 0).all()
+
+
+def test_decayed_sums_by_definition():
+    """Token t reads every earlier one with the product of the decays behind it."""
+    rng = np.random.default_rng(8)
+    q, k, v, d = rng.normal(size=(9, 4)), rng.normal(size=(9, 4)), rng.normal(size=(9, 3)), rng.uniform(0.2, 1.0, 9)
+    got = P.decayed_sums(q, k, v, d, np.zeros((4, 3)))
+    for t in range(9):
+        want = sum((q[t] @ k[s]) * np.prod(d[s + 1 : t + 1]) * v[s] for s in range(t + 1))
+        assert np.allclose(got[t], want)
+
+
+def test_choice_by_sigmoid_by_definition():
+    z = np.array([3.0, -4.0, 1.0, 0.9, 0.5, -1.0])
+    s = P.sigmoid(z)
+    zero = np.zeros(6)
+    assert [e for e, _ in P.choose_by_sigmoid(z, zero, 1, 1, 3)] == [0, 2, 3]
+    assert [e for e, _ in P.choose_by_sigmoid(z, zero, 3, 1, 2)] == [2, 3]  # the sum of two ranks the groups, not the largest
+    picks = P.choose_by_sigmoid(z, np.array([-2.0, 0, 0, 0, 0, 0]), 1, 1, 2)  # the correction moves the choice, not the weight
+    assert [e for e, _ in picks] == [2, 3] and np.allclose([v for _, v in picks], s[[2, 3]])
+    low = np.array([-9.0, -9.0, -1, -1, -5.0, -5.0])  # a dropped group loses to negative scores of a kept one
+    assert sorted(e for e, _ in P.choose_by_sigmoid(z, low, 3, 2, 4)) == [2, 3, 4, 5]
+
+
+def test_norm_in_parts_and_bounded_scores_by_definition():
+    x = np.arange(1.0, 13.0).reshape(2, 6)
+    y = P.norm_in_parts(x, 3, 0.5)
+    assert np.isclose(y[1, 3], x[1, 3] / np.sqrt((x[1, 2] ** 2 + x[1, 3] ** 2) / 2 + 0.5))
+    q, k, v = np.ones((1, 1, 1)), np.array([[[9.0]], [[-9.0]]]), np.array([[[1.0]], [[0.0]]])
+    p = P.capped_attention(q, k, v, 1.0, 1, 2.0)[0, 0, 0]
+    assert np.isclose(p, 1 / (1 + np.exp(-2 * 2 * np.tanh(4.5))))
+
+
+def broken_munisun(change):
+    cfg = copy.deepcopy(U.munisun_mixed())
+    change(cfg)
+    return cfg
+
+
+@pytest.mark.parametrize("change,text", [
+    (lambda c: c.pop("token_side"), "token_side"),
+    (lambda c: c["embedding"].pop("scale"), "scale"),
+    (lambda c: c["layers"][0].update(type="attention"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mixer"].pop("right"), "right"),
+    (lambda c: c["layers"][0]["mixer"]["left"].pop("conv"), "conv"),
+    (lambda c: c["layers"][0]["mixer"]["left"].update(kv_from=0), "kv_from"),
+    (lambda c: c["layers"][0]["mixer"]["right"].update(decay=[0.5]), "decay"),
+    (lambda c: c["layers"][0]["mixer"]["right"]["decay"].__setitem__(0, 1.5), "decay"),
+    (lambda c: c["layers"][1]["mixer"].pop("left_scale"), "left_scale"),
+    (lambda c: c["layers"][1]["mixer"]["left"].update(softcap=0), "softcap"),
+    (lambda c: c["layers"][1]["mixer"]["left"]["rot"]["scaling"].pop("high"), "high"),
+    (lambda c: c["layers"][1]["mixer"]["right"].update(groups=4), "key heads"),
+    (lambda c: c["layers"][1]["mixer"]["right"].update(norm_groups=7), "norm_groups"),
+    (lambda c: c["layers"][1]["mlp"].update(shared={"ff": 8}), "shared"),
+    (lambda c: c["layers"][1]["mlp"]["router"].update(top=9), "top"),
+])
+def test_munisun_config_errors_are_named(lc, change, text):
+    with pytest.raises(lc.LeafcutterError) as e:
+        lc.Engine.from_config(broken_munisun(change))
+    assert text in str(e.value)
+
+
 def broken_tenetar(change):
     cfg = copy.deepcopy(U.tenetar_mixed())
     change(cfg)

@@ -18,11 +18,14 @@ def mixed_config():
                      U.with_ff(U.latent(heads=2, dim=16, rot_dim=8, vdim=24, kv_rank=48, q_rank=20, scaling=None), 56)])
 
 
-@pytest.fixture(scope="module", params=["varasun", "tenetar"])
+@pytest.fixture(scope="module", params=["varasun", "tenetar", "munisun"])
 def model(request):
     if request.param == "varasun":
         cfg = mixed_config()
         w = U.weights(cfg, 11)
+    elif request.param == "munisun":
+        cfg = U.munisun_mixed()
+        w = U.munisun_weights(cfg, 13, fixed_choice=True)
     else:
         cfg = U.tenetar_mixed()
         w = U.tenetar_weights(cfg, 12, fixed_choice=True)
@@ -55,7 +58,7 @@ def test_prompts_in_portions(gpu, model, sizes, dtype):
     toks = U.tokens(n, cfg["vocab"], n)
     eng = U.engine(gpu, cfg, w, dtype, max_seq_len=320)
     want = m.forward(toks, m.new_state())
-    U.check(run_cut(eng, 0, toks, portions(n, sizes)), want, dtype)
+    U.check(run_cut(eng, 0, toks, portions(n, sizes)), want, dtype, U.rounding(cfg, dtype))
     eng.close()
 
 
@@ -67,17 +70,22 @@ def test_first_tokens(gpu, model, dtype):
         for cuts in ([n], [1] * n):
             eng.kv_clear()
             toks = U.tokens(n, cfg["vocab"], 70 + n)
-            U.check(run_cut(eng, 0, toks, cuts), m.forward(toks, m.new_state()), dtype)
+            U.check(run_cut(eng, 0, toks, cuts), m.forward(toks, m.new_state()), dtype, U.rounding(cfg, dtype))
     eng.close()
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("design", ["varasun", "tenetar"])
+@pytest.mark.parametrize("design", ["varasun", "tenetar", "munisun"])
 def test_a_call_longer_than_one_pass(gpu, design, dtype):
     """More tokens in one call than a pass takes (2048): the second pass continues from the first one's cache and state."""
     if design == "varasun":
         cfg = U.config([U.delta(heads=1, kv_heads=1, dim=16, vdim=16, conv=4), U.latent(heads=2, dim=8, rot_dim=8, vdim=8, kv_rank=24, q_rank=16)], width=32, vocab=40)
         w = U.weights(cfg, 3)
+    elif design == "munisun":
+        cfg = U.munisun_config([U.with_gated_experts(U.scaled_pair(U.gated_attention(heads=2, kv_heads=1, dim=8, vdim=8, rot_dims=4), U.state_space(heads=2, groups=1, state=16, vdim=8)),
+                                                     experts=6, top=2, groups=3, keep=2),
+                                U.normed_pair(U.conv_attention(heads=2, kv_heads=1, dim=8, vdim=8), U.lightning((0.9, 0.999), dim=8, vdim=8))], width=32, vocab=40)
+        w = U.munisun_weights(cfg, 3, fixed_choice=True)
     else:
         cfg = U.tenetar_config([U.with_experts(U.attention(heads=2, kv_heads=1, dim=8, vdim=8, window=700, keep_first=70), experts=5, identity=1, top=2, groups=2, keep=1),
                                 U.attention(heads=2, kv_heads=1, dim=8, vdim=8, window=3000, keep_first=0, kv_from=0)], width=32, vocab=40)
@@ -87,7 +95,7 @@ def test_a_call_longer_than_one_pass(gpu, design, dtype):
     eng = U.engine(gpu, cfg, w, dtype, max_seq_len=2304, max_seqs=2)
     got, _ = eng.step([0, 1], [a, b], [[0, 1499], [546, 547, 548, 549, 702]])
     want = np.concatenate([m.forward(a, m.new_state())[[0, 1499]], m.forward(b, m.new_state())[[546, 547, 548, 549, 702]]])
-    U.check(got, want, dtype)
+    U.check(got, want, dtype, U.rounding(cfg, dtype))
     eng.close()
 
 
@@ -107,7 +115,7 @@ def test_unequal_batches_equal_each_alone(gpu, model, dtype):
         places = [list(range(0, n, 2)) if s != 1 else [] for s, n in step]
         got, nxt = eng.step(ids, parts, places)
         exp = np.concatenate([want[s][[at[s] + p for p in pl]] for (s, n), pl in zip(step, places)])
-        U.check(got, exp, dtype)
+        U.check(got, exp, dtype, U.rounding(cfg, dtype))
         assert (nxt == got.argmax(axis=1)).all()
         for s, n in step:
             at[s] += n
@@ -129,15 +137,16 @@ def test_pages_and_slots_are_used_again(gpu, model, dtype):
         n = int(rng.integers(1, 64))
         toks = U.tokens(n, cfg["vocab"], 200 + i)
         cuts = portions(n, [int(rng.integers(1, 33)), 1, 2])
-        U.check(run_cut(eng, s, toks, cuts), m.forward(toks, m.new_state()), dtype)
+        U.check(run_cut(eng, s, toks, cuts), m.forward(toks, m.new_state()), dtype, U.rounding(cfg, dtype))
     eng.close()
 
 
 @pytest.mark.parametrize("sizes", [[260], [1], [2, 70], [33, 1, 1, 2]])
-def test_choices_that_follow_the_token(gpu, sizes):
+@pytest.mark.parametrize("design", ["tenetar", "munisun"])
+def test_choices_that_follow_the_token(gpu, design, sizes):
     """Every token its own experts (in 32-bit, where rounding does not move a choice): portions, then other sequences beside it."""
-    cfg = U.tenetar_mixed()
-    w = U.tenetar_weights(cfg, 21)
+    cfg = U.tenetar_mixed() if design == "tenetar" else U.munisun_mixed()
+    w = U.tenetar_weights(cfg, 21) if design == "tenetar" else U.munisun_weights(cfg, 21)
     m = P.plain_model(cfg, w)
     toks = U.tokens(260, cfg["vocab"], 9)
     want = m.forward(toks, m.new_state())
@@ -251,12 +260,17 @@ def test_long_decoding_and_greedy_generation(gpu, model):
 
 
 @pytest.mark.parametrize("n_seqs", [1, 5, 20, 70])
-@pytest.mark.parametrize("design", ["varasun", "tenetar"])
+@pytest.mark.parametrize("design", ["varasun", "tenetar", "munisun"])
 def test_decode_batches_of_every_product_form(gpu, design, n_seqs):
     """Decode steps whose token count selects different tiles, at contexts on both sides of page and key-tile edges."""
     if design == "varasun":
         cfg = U.config([U.with_ff(U.delta(heads=2, kv_heads=1, dim=64, vdim=64), 136), U.latent(heads=20, dim=32, rot_dim=16, vdim=32, kv_rank=96, q_rank=64)], width=128)
         w = U.weights(cfg, 4)
+    elif design == "munisun":
+        cfg = U.munisun_config([U.with_ff(U.scaled_pair(U.gated_attention(heads=20, kv_heads=2, dim=32, vdim=32), U.state_space(heads=4, groups=2, state=64, vdim=64)), 136),
+                                U.with_gated_experts(U.normed_pair(U.conv_attention(heads=20, kv_heads=2, dim=32, vdim=32), U.lightning((0.9, 0.999, 0.5), dim=64, vdim=32)),
+                                                     experts=8, top=3, groups=4, keep=3, ff=130)], width=128, side=40)
+        w = U.munisun_weights(cfg, 4, fixed_choice=True)
     else:
         cfg = U.tenetar_config([U.with_ff(U.attention(heads=20, kv_heads=2, dim=32, vdim=32, window=64, keep_first=16), 136),
                                 U.with_experts(U.attention(heads=20, kv_heads=2, dim=32, vdim=32, window=150, keep_first=0, kv_from=0), experts=6, identity=2, top=3, groups=4,
@@ -270,7 +284,7 @@ def test_decode_batches_of_every_product_form(gpu, design, n_seqs):
     for j in range(3):
         got, _ = eng.step(list(range(n_seqs)), [[t[n + j]] for t, n in zip(toks, lens)], [[0]] * n_seqs)
         want = np.array([m.forward(t[: n + j + 1], m.new_state())[-1] for t, n in zip(toks[:10], lens)])
-        U.check(got[:10], want, "bfloat16")
+        U.check(got[:10], want, "bfloat16", U.rounding(cfg, "bfloat16"))
     eng.close()
 
 
@@ -282,7 +296,7 @@ def test_checkpoint_directory_and_trace_runner(gpu, model, tmp_path, monkeypatch
     eng = Engine.load_dir(str(tmp_path), max_seq_len=64, dtype=dtype)
     toks = U.tokens(33, cfg["vocab"], 5)
     want = m.forward(toks, m.new_state())
-    U.check(eng.forward(toks)[None], want[-1:], dtype)
+    U.check(eng.forward(toks)[None], want[-1:], dtype, U.rounding(cfg, dtype))
     eng.close()
     from leafcutterllm_b200.__main__ import main
     st, picks = m.new_state(), []
@@ -301,22 +315,22 @@ def test_checkpoint_directory_and_trace_runner(gpu, model, tmp_path, monkeypatch
     assert trace.main(["--model", str(tmp_path), "--dtype", dtype, "--out", str(out), "--max-tokens", "192"]) == 0
     assert capsys.readouterr().out.split() == ["done", "0", "done", "1", "done", "2"]
     got = np.fromfile(out / "0.f32", "<f4").reshape(2, -1)
-    U.check(got, want[[19, 3]], dtype)
+    U.check(got, want[[19, 3]], dtype, U.rounding(cfg, dtype))
     assert not (out / "1.f32").exists()
     got = np.fromfile(out / "2.f32", "<f4").reshape(2, -1)
-    U.check(got, want[[32, 20]], dtype)
+    U.check(got, want[[32, 20]], dtype, U.rounding(cfg, dtype))
 
 
 def test_incomplete_models_are_named(gpu, model):
     cfg, w, _ = model
-    tenetar = cfg["architecture"] == "Tenetar"
-    dropped = ("l1.mlp.e3.down", "l2.mlp.correction", "l0.norm1b", "l3.mix.q.norm") if tenetar else ("l1.mix.uk", "l0.mix.a1")
+    dropped = {"Tenetar": ("l1.mlp.e3.down", "l2.mlp.correction", "l0.norm1b", "l3.mix.q.norm"), "Varasun": ("l1.mix.uk", "l0.mix.a1"),
+               "Munisun": ("l0.mix.left.k.conv", "l1.mix.right.conv.b", "l1.mix.left.g", "l2.mlp.e9.gate", "l3.side.norm", "side.embed", "l0.mix.right.out")}[cfg["architecture"]]
     for drop, status in [(n, -6) for n in dropped + ("final.norm",)]:
         with pytest.raises(gpu.LeafcutterError) as e:
             U.engine(gpu, cfg, {n: a for n, a in w.items() if n != drop})
         assert e.value.status == status and drop in str(e.value)
     wrong = dict(w)
-    name = "l2.mlp.e1.up" if tenetar else "l1.mix.uv"
+    name = {"Tenetar": "l2.mlp.e1.up", "Varasun": "l1.mix.uv", "Munisun": "l1.mix.right.in"}[cfg["architecture"]]
     wrong[name] = w[name][:-1]
     with pytest.raises(gpu.LeafcutterError) as e:
         U.engine(gpu, cfg, wrong)
