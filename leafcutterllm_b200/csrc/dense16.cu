@@ -58,24 +58,24 @@ struct DenseParams {
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // The epilogue is a template parameter of the kernels; kEpiAny stands for the rarer elementwise ones, told apart at run time.
 constexpr int kEpiAny = -1;
-constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS || epi == DENSE_GELU_TABLE ? kEpiAny : epi; }
+constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS ? kEpiAny : epi; }
 constexpr bool epi_splits(int epi) { return epi == DENSE_SPLIT_RELU2 || epi == DENSE_SPLIT_SILU; }
 __device__ __forceinline__ float silu_of(float g) { return g / (1.0f + expf(-g)); }
-__device__ __forceinline__ float gelu_of(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+// z (1 + tanh u) / 2 = z / (1 + e^(-2u)), u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_of(float z) { return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))); }
 // ea, eb: the row's constants; `second`: behind the split of DENSE_SPLIT_*
 template <int EPI>
 __device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool second, float ea, float eb, float y, int row, int t) {
     const float r = fmaxf(y, 0.0f);
     if constexpr (EPI == DENSE_RELU2) return r * r;
     else if constexpr (EPI == DENSE_SPLIT_RELU2) return second ? r * r : y;
-    else if constexpr (EPI == DENSE_SPLIT_SILU) return second && row < p.silu_end ? silu_of(y) : y;
+    else if constexpr (EPI == DENSE_GELU_TABLE) {
+        if (t >= p.T || row >= p.n) return 0.0f;
+        const int64_t id = p.ids[t];
+        return id >= 0 && id < p.table_rows ? gelu_of(y) * __bfloat162float(p.table[(size_t)id * p.table_ld + row]) : 0.0f;
+    } else if constexpr (EPI == DENSE_SPLIT_SILU) return second && row < p.silu_end ? silu_of(y) : y;
     else if constexpr (EPI == kEpiAny) {
         if (p.epi == DENSE_LOG_DECAY) return -ea * softplus_f(y + eb);
-        if (p.epi == DENSE_GELU_TABLE) {
-            if (t >= p.T || row >= p.n) return 0.0f;
-            const int64_t id = p.ids[t];
-            return id >= 0 && id < p.table_rows ? gelu_of(y) * __bfloat162float(p.table[(size_t)id * p.table_ld + row]) : 0.0f;
-        }
         const float v = y * p.scale;
         return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v;
     } else return y;
@@ -589,6 +589,7 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
             case DENSE_GATED_SILU: return go(dense_f32_kernel<DENSE_GATED_SILU>);
             case DENSE_SPLIT_RELU2: return go(dense_f32_kernel<DENSE_SPLIT_RELU2>);
             case DENSE_SPLIT_SILU: return go(dense_f32_kernel<DENSE_SPLIT_SILU>);
+            case DENSE_GELU_TABLE: return go(dense_f32_kernel<DENSE_GELU_TABLE>);
             default: return go(dense_f32_kernel<kEpiAny>);
         }
     }
@@ -624,6 +625,7 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
         case DENSE_GATED_SILU: return launch_tiles<false, DENSE_GATED_SILU>(NT, a, *tx, p, s);
         case DENSE_SPLIT_RELU2: return launch_tiles<false, DENSE_SPLIT_RELU2>(NT, a, *tx, p, s);
         case DENSE_SPLIT_SILU: return launch_tiles<false, DENSE_SPLIT_SILU>(NT, a, *tx, p, s);
+        case DENSE_GELU_TABLE: return launch_tiles<false, DENSE_GELU_TABLE>(NT, a, *tx, p, s);
         default: return launch_tiles<false, kEpiAny>(NT, a, *tx, p, s);
     }
 }

@@ -200,110 +200,125 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
         gain[p] = g.norm == QkNorm::PerHead && !is_v ? make_float2(c < n ? gw[c] : 0.0f, c + 1 < n ? gw[c + 1] : 0.0f) : make_float2(1.0f, 1.0f);
     }
     int prev_seq = -1, prev_pos = -1;
-    for (int t = t0; t < t1; t++) {
-        const int seq = a.tok_seq[t], pos = a.tok_pos[t];
-        const float* row = a.proj + (size_t)t * a.ld_proj + col0;
-        // the inputs j tokens back: from the call's rows as far as they belong to this run, from the ring before that, zero before the start
-        auto back = [&](int j, int c) {
-            if (pos - j < 0) return make_float2(0.0f, 0.0f);
-            const int tt = t - j;
-            if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) return pair_at(a.proj + (size_t)tt * a.ld_proj + col0, c);
-            const float* r = a.ring + ((size_t)seq * taps + (pos - j) % taps) * channels + ch0 + c;  // rows of any length: not aligned for pairs
-            return make_float2(c < n ? r[0] : 0.0f, c + 1 < n ? r[1] : 0.0f);
-        };
-        float2 x[NP];
-        const bool fresh = seq != prev_seq || pos != prev_pos + 1;
-        float ss = 0.0f;
+    constexpr int kAhead = NP == 1 || (NP == 2 && TAPS == 0) ? 4 : 2;  // tokens whose rows are fetched together
+    float2 ahead[kAhead][NP];
+    int seq_a[kAhead], pos_a[kAhead];
+    for (int tb = t0; tb < t1; tb += kAhead) {
 #pragma unroll
-        for (int p = 0; p < NP; p++) {
-            const int c = 2 * (lane + 32 * p);
-            const float2 u = pair_at(row, c);
-            x[p] = u;
-            if constexpr (TAPS > 0) {
-                if (fresh) {
+        for (int v = 0; v < kAhead; v++) {
+            const int t = min(tb + v, t1 - 1);
+            seq_a[v] = a.tok_seq[t]; pos_a[v] = a.tok_pos[t];
+            const float* row = a.proj + (size_t)t * a.ld_proj + col0;
 #pragma unroll
-                    for (int j = 1; j < TAPS; j++) {
-                        const float2 v = back(j, c);
-                        win[p][0][j - 1] = v.x; win[p][1][j - 1] = v.y;
+            for (int p = 0; p < NP; p++) ahead[v][p] = pair_at(row, 2 * (lane + 32 * p));
+        }
+#pragma unroll
+        for (int v = 0; v < kAhead; v++) {
+            const int t = tb + v;
+            if (t >= t1) break;
+            const int seq = seq_a[v], pos = pos_a[v];
+            // the inputs j tokens back: from the call's rows as far as they belong to this run, from the ring before that, zero before the start
+            auto back = [&](int j, int c) {
+                if (pos - j < 0) return make_float2(0.0f, 0.0f);
+                const int tt = t - j;
+                if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) return pair_at(a.proj + (size_t)tt * a.ld_proj + col0, c);
+                const float* r = a.ring + ((size_t)seq * taps + (pos - j) % taps) * channels + ch0 + c;  // rows of any length: not aligned for pairs
+                return make_float2(c < n ? r[0] : 0.0f, c + 1 < n ? r[1] : 0.0f);
+            };
+            float2 x[NP];
+            const bool fresh = seq != prev_seq || pos != prev_pos + 1;
+            float ss = 0.0f;
+#pragma unroll
+            for (int p = 0; p < NP; p++) {
+                const int c = 2 * (lane + 32 * p);
+                const float2 u = ahead[v][p];
+                x[p] = u;
+                if constexpr (TAPS > 0) {
+                    if (fresh) {
+#pragma unroll
+                        for (int j = 1; j < TAPS; j++) {
+                            const float2 v = back(j, c);
+                            win[p][0][j - 1] = v.x; win[p][1][j - 1] = v.y;
+                        }
                     }
+                    float2 y = make_float2(0.0f, 0.0f);
+#pragma unroll
+                    for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[p][0][TAPS - 1 - j], win[p][0][j - 1], y.x); y.y = fmaf(w[p][1][TAPS - 1 - j], win[p][1][j - 1], y.y); }
+                    x[p] = make_float2(fmaf(w[p][0][TAPS - 1], u.x, y.x), fmaf(w[p][1][TAPS - 1], u.y, y.y));
+#pragma unroll
+                    for (int j = TAPS - 2; j > 0; j--) { win[p][0][j] = win[p][0][j - 1]; win[p][1][j] = win[p][1][j - 1]; }
+                    win[p][0][0] = u.x; win[p][1][0] = u.y;
+                } else if constexpr (TAPS < 0) {
+                    float2 y = make_float2(0.0f, 0.0f);
+                    if (c < n)
+                        for (int j = taps - 1; j >= 0; j--) {
+                            const float2 v = j == 0 ? u : back(j, c);
+                            const float* cw = a.conv + (size_t)(ch0 + c) * taps + taps - 1 - j;
+                            y.x = fmaf(cw[0], v.x, y.x);
+                            if (c + 1 < n) y.y = fmaf(cw[taps], v.y, y.y);
+                        }
+                    x[p] = y;
                 }
-                float2 y = make_float2(0.0f, 0.0f);
+                if (TAPS != 0 && a.one_each && c < n) {
+                    float* r = a.ring + ((size_t)seq * taps + pos % taps) * channels + ch0 + c;
+                    r[0] = u.x;
+                    if (c + 1 < n) r[1] = u.y;
+                }
+                ss = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, ss));
+            }
+            prev_seq = seq; prev_pos = pos;
+            if (!is_v) {
+                if (g.norm == QkNorm::PerHead) {
+                    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
 #pragma unroll
-                for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[p][0][TAPS - 1 - j], win[p][0][j - 1], y.x); y.y = fmaf(w[p][1][TAPS - 1 - j], win[p][1][j - 1], y.y); }
-                x[p] = make_float2(fmaf(w[p][0][TAPS - 1], u.x, y.x), fmaf(w[p][1][TAPS - 1], u.y, y.y));
+                    for (int p = 0; p < NP; p++) { x[p].x *= r * gain[p].x; x[p].y *= r * gain[p].y; }
+                }
+                const float2* tab = a.rot + (size_t)pos * half;
+                if (g.pairs == AttnPairs::Neighbours) {
 #pragma unroll
-                for (int j = TAPS - 2; j > 0; j--) { win[p][0][j] = win[p][0][j - 1]; win[p][1][j] = win[p][1][j - 1]; }
-                win[p][0][0] = u.x; win[p][1][0] = u.y;
-            } else if constexpr (TAPS < 0) {
-                float2 y = make_float2(0.0f, 0.0f);
-                if (c < n)
-                    for (int j = taps - 1; j >= 0; j--) {
-                        const float2 v = j == 0 ? u : back(j, c);
-                        const float* cw = a.conv + (size_t)(ch0 + c) * taps + taps - 1 - j;
-                        y.x = fmaf(cw[0], v.x, y.x);
-                        if (c + 1 < n) y.y = fmaf(cw[taps], v.y, y.y);
+                    for (int p = 0; p < NP; p++) {
+                        const int i = lane + 32 * p;
+                        if (i < half) { const float2 cs = tab[i], u = x[p]; x[p] = make_float2(u.x * cs.x - u.y * cs.y, u.y * cs.x + u.x * cs.y); }
                     }
-                x[p] = y;
-            }
-            if (TAPS != 0 && a.one_each && c < n) {
-                float* r = a.ring + ((size_t)seq * taps + pos % taps) * channels + ch0 + c;
-                r[0] = u.x;
-                if (c + 1 < n) r[1] = u.y;
-            }
-            ss = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, ss));
-        }
-        prev_seq = seq; prev_pos = pos;
-        if (!is_v) {
-            if (g.norm == QkNorm::PerHead) {
-                const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
+                } else if (half > 0) {
+                    __syncwarp();
 #pragma unroll
-                for (int p = 0; p < NP; p++) { x[p].x *= r * gain[p].x; x[p].y *= r * gain[p].y; }
-            }
-            const float2* tab = a.rot + (size_t)pos * half;
-            if (g.pairs == AttnPairs::Neighbours) {
+                    for (int p = 0; p < NP; p++) *(float2*)(s_x[warp] + 2 * (lane + 32 * p)) = x[p];
+                    __syncwarp();
+                    auto turned = [&](int c, float v) {
+                        if (c >= 2 * half) return v;
+                        const float2 cs = tab[c < half ? c : c - half];
+                        return c < half ? v * cs.x - s_x[warp][c + half] * cs.y : v * cs.x + s_x[warp][c - half] * cs.y;
+                    };
 #pragma unroll
-                for (int p = 0; p < NP; p++) {
-                    const int i = lane + 32 * p;
-                    if (i < half) { const float2 cs = tab[i], u = x[p]; x[p] = make_float2(u.x * cs.x - u.y * cs.y, u.y * cs.x + u.x * cs.y); }
+                    for (int p = 0; p < NP; p++) { const int c = 2 * (lane + 32 * p); x[p] = make_float2(turned(c, x[p].x), turned(c + 1, x[p].y)); }
                 }
-            } else if (half > 0) {
-                __syncwarp();
+                if (g.norm == QkNorm::PerHeadAfter) {
+                    ss = 0.0f;
 #pragma unroll
-                for (int p = 0; p < NP; p++) *(float2*)(s_x[warp] + 2 * (lane + 32 * p)) = x[p];
-                __syncwarp();
-                auto turned = [&](int c, float v) {
-                    if (c >= 2 * half) return v;
-                    const float2 cs = tab[c < half ? c : c - half];
-                    return c < half ? v * cs.x - s_x[warp][c + half] * cs.y : v * cs.x + s_x[warp][c - half] * cs.y;
-                };
+                    for (int p = 0; p < NP; p++) ss = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, ss));
+                    const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
 #pragma unroll
-                for (int p = 0; p < NP; p++) { const int c = 2 * (lane + 32 * p); x[p] = make_float2(turned(c, x[p].x), turned(c + 1, x[p].y)); }
+                    for (int p = 0; p < NP; p++) { x[p].x *= r; x[p].y *= r; }
+                }
             }
-            if (g.norm == QkNorm::PerHeadAfter) {
-                ss = 0.0f;
-#pragma unroll
-                for (int p = 0; p < NP; p++) ss = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, ss));
-                const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
-#pragma unroll
-                for (int p = 0; p < NP; p++) { x[p].x *= r; x[p].y *= r; }
+            A* dst;
+            int swz = 0;
+            if (is_q) dst = (A*)a.q + ((size_t)t * g.heads + h) * g.dp;
+            else {
+                const int page = a.page_table[(size_t)seq * a.pages_per_seq + pos / a.page_tokens];
+                const size_t at = ((size_t)page * g.kv_heads + h) * a.page_tokens + pos % a.page_tokens;
+                dst = is_v ? (A*)a.v_cache + at * g.v_pitch : (A*)a.k_cache + at * g.k_pitch;
+                swz = is_v ? g.v_swz : g.k_swz;
             }
-        }
-        A* dst;
-        int swz = 0;
-        if (is_q) dst = (A*)a.q + ((size_t)t * g.heads + h) * g.dp;
-        else {
-            const int page = a.page_table[(size_t)seq * a.pages_per_seq + pos / a.page_tokens];
-            const size_t at = ((size_t)page * g.kv_heads + h) * a.page_tokens + pos % a.page_tokens;
-            dst = is_v ? (A*)a.v_cache + at * g.v_pitch : (A*)a.k_cache + at * g.k_pitch;
-            swz = is_v ? g.v_swz : g.k_swz;
-        }
 #pragma unroll
-        for (int p = 0; p < NP; p++) {
-            const int c = 2 * (lane + 32 * p);
-            if (c >= n) continue;
-            A* d = dst + cell_of(c, pos, swz);
-            if (c + 1 < n) put2<A>(d, x[p]);
-            else d[0] = to_act<A>(x[p].x);
+            for (int p = 0; p < NP; p++) {
+                const int c = 2 * (lane + 32 * p);
+                if (c >= n) continue;
+                A* d = dst + cell_of(c, pos, swz);
+                if (c + 1 < n) put2<A>(d, x[p]);
+                else d[0] = to_act<A>(x[p].x);
+            }
         }
     }
 }
@@ -750,7 +765,7 @@ int pitch_of(int n8, bool f32, int* swz) {
 bool tensor_form(const AttnShape& g, bool f32) { return !f32 && g.ep <= 256 && tokens_smem(g) <= kMaxSmem - 4096 && tiles_smem(g) <= kMaxSmem - 1024; }
 template <typename A, int TAPS>
 int32_t head_prep_pairs(const AttnArgs& a, cudaStream_t s) {
-    const int pairs = (std::max(a.g.dim, a.g.vdim) + 63) / 64, stretch = a.T < 256 ? 1 : 8;
+    const int pairs = (std::max(a.g.dim, a.g.vdim) + 63) / 64, stretch = a.T < 256 ? 1 : 16;
     const dim3 grid((unsigned)((a.T + stretch - 1) / stretch), (unsigned)((a.g.heads + 2 * a.g.kv_heads + 7) / 8));
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(launch_pdl(kern, grid, dim3(256), 0, s, a, stretch));

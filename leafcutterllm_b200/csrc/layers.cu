@@ -371,10 +371,19 @@ int32_t bind_pair(lc_model* m, StackLayer& L, const std::string& p) {
     L.mixed_ld = L.mixed_off + round8(inner);
     const PackMap heads{sa.vdim, a.ep, 0, 0};
     if (L.s.combine == Combine::Normed) {
-        LC_TRY(plain_weight(m, pl + "o", W, sa.heads * sa.vdim, &L.out, heads, L.mixed_off));
-        LC_TRY(plain_weight(m, pr + "o", W, inner, &L.out2));
         LC_TRY(model_gain_f32(m, pl + "out", W, &L.out_norm[0]));
-        return model_gain_f32(m, pr + "out", W, &L.out_norm[1]);
+        LC_TRY(model_gain_f32(m, pr + "out", W, &L.out_norm[1]));
+        if (2 * L.mixed_off == L.mixed_ld) {  // rows of equal length: one batch of two
+            LC_TRY(talloc(st, &d, (size_t)W * L.mixed_ld * 2));
+            DevTensor* t = nullptr;
+            LC_TRY(matrix(m, pl + "o", W, sa.heads * sa.vdim, &t));
+            LC_TRY(launch_pack((const bf16*)t->view, W, sa.heads * sa.vdim, (bf16*)d, L.mixed_off, PackMap(), heads, false, m->stream));
+            LC_TRY(matrix(m, pr + "o", W, inner, &t));
+            LC_TRY(launch_pack((const bf16*)t->view, W, inner, (bf16*)d + (size_t)W * L.mixed_off, L.mixed_off, PackMap(), PackMap(), false, m->stream));
+            return dense_weight_init(&L.out, (const bf16*)d, W, L.mixed_off, L.mixed_off, 2, (size_t)W * L.mixed_off);
+        }
+        LC_TRY(plain_weight(m, pl + "o", W, sa.heads * sa.vdim, &L.out, heads, L.mixed_off));
+        return plain_weight(m, pr + "o", W, inner, &L.out2);
     }
     LC_TRY(talloc(st, &d, (size_t)W * L.mixed_ld * 2));
     DevTensor* t = nullptr;
@@ -560,8 +569,7 @@ int32_t recur(lc_model* m, const MixerUnit& L, LinearArgs a, int T, bool decode_
     a.ring = L.ring; a.in = st.lin; a.state = L.state; a.tok_seq = m->d_tok_seq; a.tok_pos = m->d_tok_pos; a.T = T; a.o = st.o; a.norm_w = L.o_norm; a.f32 = st.f32;
     int launches = 1;
     if (decode_step) {
-        LC_TRY(launch_linear_step(a, m->stream));
-        launches++;
+        LC_TRY(launch_linear_step(a, &launches, m->stream));
     } else {
         a.runs = st.d_short_runs; a.n_runs = st.n_short_runs; a.chunk_runs = st.d_chunk_runs; a.n_chunk_runs = st.n_chunk_runs; a.all_runs = st.d_runs; a.n_all_runs = st.n_runs;
         LC_TRY(launch_linear_runs(a, &launches, m->stream));
@@ -586,6 +594,11 @@ int32_t pair_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bo
     LinearArgs b;
     b.out = (void*)at(st, st.mixed, (size_t)L.mixed_off); b.ldo = L.mixed_ld; b.out_scale = normed ? 1.0f : L.s.mix_scale[1];
     LC_TRY(recur(m, L.mix[1], b, T, decode_step));
+    if (normed && L.out.batch == 2) {
+        DenseArgs o;
+        o.x_batch = (size_t)L.mixed_off; o.out_batch = (size_t)m->t_cap * st.spec.width;
+        return product(m, L.out, st.mixed, L.mixed_ld, T, st.y, st.spec.width, true, DENSE_STORE, o);
+    }
     LC_TRY(product(m, L.out, st.mixed, L.mixed_ld, T, st.y, st.spec.width, true));
     return normed ? product(m, L.out2, b.out, L.mixed_ld, T, st.y2, st.spec.width, true) : LC_OK;
 }
@@ -826,10 +839,11 @@ int32_t stack_alloc(lc_model* m) {
     LC_TRY(zalloc(st, &st.cq, T * cq * e)); LC_TRY(zalloc(st, &st.q, T * q * e));
     LC_TRY(zalloc(st, &st.q_abs, T * qa * e)); LC_TRY(zalloc(st, &st.o_lat, T * qa * e));
     LC_TRY(zalloc(st, &st.ffn, T * ffn * e)); LC_TRY(zalloc(st, &st.last, (size_t)m->head_rows * st.width_p * e));
-    if (pairs) LC_TRY(zalloc(st, (void**)&st.y2, T * st.spec.width * 4));
     if (lin) LC_TRY(zalloc(st, &st.lin, T * lin * e));
     if (st.spec.side_dim) LC_TRY(zalloc(st, &st.side, T * round8(st.spec.side_dim) * e));
-    LC_TRY(zalloc(st, (void**)&st.y, T * st.spec.width * 4)); LC_TRY(zalloc(st, (void**)&st.log_decay, T * ld * 4));
+    LC_TRY(zalloc(st, (void**)&st.y, (pairs ? 2 : 1) * T * st.spec.width * 4));
+    if (pairs) st.y2 = st.y + T * st.spec.width;
+    LC_TRY(zalloc(st, (void**)&st.log_decay, T * ld * 4));
     LC_TRY(zalloc(st, (void**)&st.qk, T * qk * 4)); LC_TRY(zalloc(st, (void**)&st.v, T * v * 4)); LC_TRY(zalloc(st, (void**)&st.o, T * v * 4));
     LC_TRY(zalloc(st, (void**)&st.d_runs, T * sizeof(SeqRun)));
     LC_TRY(zalloc(st, (void**)&st.d_short_runs, T * sizeof(SeqRun))); LC_TRY(zalloc(st, (void**)&st.d_chunks, T * sizeof(DeltaChunk)));

@@ -316,7 +316,7 @@ struct LinearArgs {
 };
 bool linear_chunks_apply(const LinearShape& g, bool f32);
 int32_t launch_linear_runs(const LinearArgs& a, int* launches, cudaStream_t s);  // convolutions, the recurrence over all runs, the kept inputs
-int32_t launch_linear_step(const LinearArgs& a, cudaStream_t s);                 // the same for one token per sequence
+int32_t launch_linear_step(const LinearArgs& a, int* launches, cudaStream_t s);  // the same for one token per sequence
 int32_t launch_linear_output(const LinearArgs& a, cudaStream_t s);               // gate and norm
 
 // ---- expert_choice.cu: routing ---------------------------------------------------------------------------------------------

@@ -8,13 +8,14 @@
 //                           o_t = e^(G_t) S0^T q_t + sum_(s <= t) (q_t . k_s) e^(G_t - G_s) b_s v_s,
 //                           S = e^(G_end) S0 + sum_s k_s (e^(G_end - G_s) b_s v_s)^T;
 //                         q, k and v enter as they are, the f32 factors (weights, scaled values, S0) as two bf16 halves
-//   linear_step_kernel    one token per sequence: convolution, recurrence
+//   linear_step_kernel    one token per sequence: convolution, recurrence; many items: linear_ring_kernel behind linear_conv_kernel
 //   linear_output_kernel  gate and norm: Constant rms_norm(o) w sigmoid(gate) over all heads, StateSpace rms_norm(o silu(gate)) w in parts
 #include <algorithm>
 #include <cmath>
 #include "lc_mixers.h"
 #include "lc_mma.cuh"
 #include "lc_tma.cuh"
+#include "lc_umma.cuh"
 
 namespace lc {
 
@@ -44,12 +45,12 @@ template <typename A> __device__ __forceinline__ void put_two(A* p, float2 v);
 template <> __device__ __forceinline__ void put_two<float>(float* p, float2 v) { *(float2*)p = v; }
 template <> __device__ __forceinline__ void put_two<bf16>(bf16* p, float2 v) { *(uint32_t*)p = pack2(v.x, v.y); }
 
-// A thread walks kConvTok tokens of two neighbouring channels and keeps their last inputs in registers (TAPS of them; 0: any
+// A thread walks `stretch` tokens of two neighbouring channels and keeps their last inputs in registers (TAPS of them; 0: any
 // number, re-read).  Inputs of earlier positions come from the call's rows as far as they belong to the same run, from the ring
-// before that, and are zero before the sequence's start.
-constexpr int kConvTok = 16;
+// before that, and are zero before the sequence's start.  one_each: every token is the only one of its sequence; its inputs enter the
+// ring here (an entry that no convolution of this call reads).
 template <typename A, int TAPS>
-__global__ void __launch_bounds__(128) linear_conv_kernel(const LinearArgs a) {
+__global__ void __launch_bounds__(128) linear_conv_kernel(const LinearArgs a, int stretch, int one_each) {
     pdl_launch_dependents();
     pdl_wait();
     const LinearShape& g = a.g;
@@ -71,41 +72,60 @@ __global__ void __launch_bounds__(128) linear_conv_kernel(const LinearArgs a) {
             win[0][j] = win[1][j] = 0.0f;
         }
     }
-    const int t0 = blockIdx.x * kConvTok, t1 = min(a.T, t0 + kConvTok);
+    const int t0 = blockIdx.x * stretch, t1 = min(a.T, t0 + stretch);
     int prev_seq = -1, prev_pos = -1;
-    for (int t = t0; t < t1; t++) {
-        const int seq = a.tok_seq[t], pos = a.tok_pos[t];
-        auto back = [&](int j) {
-            if (pos - j < 0) return make_float2(0.0f, 0.0f);
-            const int tt = t - j;
-            if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) return two<A>(in + (size_t)tt * g.ld);
-            const A* r = ring + ((size_t)seq * taps + (pos - j) % taps) * g.channels;
-            return make_float2(act_f<A>(r[0]), both ? act_f<A>(r[1]) : 0.0f);
-        };
-        const float2 u = two<A>(in + (size_t)t * g.ld);
-        float2 y = bias;
-        if constexpr (TAPS > 0) {
-            if (seq != prev_seq || pos != prev_pos + 1) {
+    constexpr int kAhead = 4;  // tokens whose inputs are fetched together
+    for (int tb = t0; tb < t1; tb += kAhead) {
+        float2 ahead[kAhead];
+        int seq_a[kAhead], pos_a[kAhead];
 #pragma unroll
-                for (int j = 1; j < TAPS; j++) {
-                    const float2 v = back(j);
-                    win[0][j - 1] = v.x; win[1][j - 1] = v.y;
+        for (int v = 0; v < kAhead; v++) {
+            const int t = min(tb + v, t1 - 1);
+            seq_a[v] = a.tok_seq[t]; pos_a[v] = a.tok_pos[t];
+            ahead[v] = two<A>(in + (size_t)t * g.ld);
+        }
+#pragma unroll
+        for (int v = 0; v < kAhead; v++) {
+            const int t = tb + v;
+            if (t >= t1) break;
+            const int seq = seq_a[v], pos = pos_a[v];
+            auto back = [&](int j) {
+                if (pos - j < 0) return make_float2(0.0f, 0.0f);
+                const int tt = t - j;
+                if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) return two<A>(in + (size_t)tt * g.ld);
+                const A* r = ring + ((size_t)seq * taps + (pos - j) % taps) * g.channels;
+                return make_float2(act_f<A>(r[0]), both ? act_f<A>(r[1]) : 0.0f);
+            };
+            const float2 u = ahead[v];
+            float2 y = bias;
+            if constexpr (TAPS > 0) {
+                if (seq != prev_seq || pos != prev_pos + 1) {
+#pragma unroll
+                    for (int j = 1; j < TAPS; j++) {
+                        const float2 v = back(j);
+                        win[0][j - 1] = v.x; win[1][j - 1] = v.y;
+                    }
+                }
+#pragma unroll
+                for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[0][TAPS - 1 - j], win[0][j - 1], y.x); y.y = fmaf(w[1][TAPS - 1 - j], win[1][j - 1], y.y); }
+                y.x = fmaf(w[0][TAPS - 1], u.x, y.x); y.y = fmaf(w[1][TAPS - 1], u.y, y.y);
+#pragma unroll
+                for (int j = TAPS - 1; j > 0; j--) { win[0][j] = win[0][j - 1]; win[1][j] = win[1][j - 1]; }
+                win[0][0] = u.x; win[1][0] = u.y;
+                prev_seq = seq; prev_pos = pos;
+            } else {
+                for (int j = taps - 1; j >= 0; j--) {
+                    const float2 v = j == 0 ? u : back(j), cw = weight(taps - 1 - j);
+                    y.x = fmaf(cw.x, v.x, y.x); y.y = fmaf(cw.y, v.y, y.y);
                 }
             }
-#pragma unroll
-            for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[0][TAPS - 1 - j], win[0][j - 1], y.x); y.y = fmaf(w[1][TAPS - 1 - j], win[1][j - 1], y.y); }
-            y.x = fmaf(w[0][TAPS - 1], u.x, y.x); y.y = fmaf(w[1][TAPS - 1], u.y, y.y);
-#pragma unroll
-            for (int j = TAPS - 1; j > 0; j--) { win[0][j] = win[0][j - 1]; win[1][j] = win[1][j - 1]; }
-            win[0][0] = u.x; win[1][0] = u.y;
-            prev_seq = seq; prev_pos = pos;
-        } else {
-            for (int j = taps - 1; j >= 0; j--) {
-                const float2 v = j == 0 ? u : back(j), cw = weight(taps - 1 - j);
-                y.x = fmaf(cw.x, v.x, y.x); y.y = fmaf(cw.y, v.y, y.y);
+            put_two<A>((A*)a.in + (size_t)t * g.ld_in + c, make_float2(silu_any(y.x), silu_any(y.y)));
+            if (one_each) {
+                A* r = (A*)a.ring + ((size_t)seq * taps + pos % taps) * g.channels + c;
+                r[0] = to_act<A>(u.x);
+                if (both) r[1] = to_act<A>(u.y);
             }
         }
-        put_two<A>((A*)a.in + (size_t)t * g.ld_in + c, make_float2(silu_any(y.x), silu_any(y.y)));
     }
 }
 
@@ -191,20 +211,21 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(const LinearArgs a) {
 }
 
 // ---- long runs --------------------------------------------------------------------------------------------------------------
-// A CTA of four warps walks the chunks of one run for 32 value columns of one head.  Per chunk a warp owns 16 tokens of the
-// read-outs and a quarter of S's key rows (DP: `dim` padded; few rows: a quarter of the (16 x 8) tiles), which stays in registers
-// as the accumulators of its update; its halves are published for the next chunk's read-outs.
+// A CTA of eight warps walks the chunks of one run for 32 value columns of one head.  Per chunk a warp owns 16 tokens and 16 columns
+// of the read-outs, and an eighth of S (DP: `dim` padded; 32 key rows: a quarter, in four warps), which stays in registers as the
+// accumulators of its update; its halves are published for the next chunk's read-outs.
 constexpr int kC = kDeltaChunk, kCols = 32, kVP = kCols + 8;
 __host__ __device__ constexpr size_t chunk_smem(int dp) {
-    return (size_t)(2 * 2 * kC * (dp + 8) + 2 * kC * kVP + 2 * dp * kVP + 2 * kC * kVP) * 2 + 3 * kC * sizeof(float);
+    return (size_t)(2 * 2 * kC * (dp + 8) + 2 * kC * kVP + 2 * dp * kVP + 2 * kC * kVP) * 2 + 6 * kC * sizeof(float);
 }
+constexpr int kChunkThreads = 256;
 template <int DP>
-__global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
-    constexpr int QP = DP + 8, kMT = DP / 16, kOwnM = kMT >= 4 ? kMT / 4 : 1, kOwnN = kMT >= 4 ? 4 : 2;
+__global__ void __launch_bounds__(kChunkThreads, DP <= 128 ? 2 : 1) linear_chunk_kernel(const LinearArgs a) {
+    constexpr int QP = DP + 8, kMT = DP / 16, kOwnM = kMT >= 8 ? kMT / 8 : 1, kOwnN = kMT >= 8 ? 4 : 2;
     static_assert(kMT >= 2, "at least two tiles of key rows");
     extern __shared__ __align__(16) unsigned char smem[];
     bf16 *s_q = (bf16*)smem, *s_k = s_q + 2 * kC * QP, *s_v = s_k + 2 * kC * QP, *s_S = s_v + 2 * kC * kVP, *s_w = s_S + 2 * DP * kVP;
-    float *s_gh = (float*)(s_w + 2 * kC * kVP), *s_gl = s_gh + kC, *s_b = s_gl + kC;  // G in log2 units as a sum of two floats
+    float* s_sums = (float*)(s_w + 2 * kC * kVP);  // of this chunk and the next: G in log2 units as a sum of two floats, the steps
     pdl_launch_dependents();
     pdl_wait();
     const LinearShape& g = a.g;
@@ -214,12 +235,14 @@ __global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
     const Rows<bf16> src = rows_of<bf16>(a);
     const float skip = a.skip ? a.skip[h] : 0.0f;
     float* st = a.state + ((size_t)cr.run.seq * g.heads + h) * g.dim * g.vdim;
-    const int m0 = kMT >= 4 ? warp * kOwnM : warp & 1, n0 = kMT >= 4 ? 0 : (warp >> 1) * 2;
+    const int rb = warp & 3, ch = (warp >> 2) * 16;  // this warp's tokens (16 rb ..) and columns of the read-outs
+    const bool owner = kMT >= 4 || warp < 4;
+    const int m0 = kMT >= 8 ? warp * kOwnM : kMT == 4 ? warp & 3 : warp & 1, n0 = kMT >= 8 ? 0 : kMT == 4 ? (warp >> 2) * 2 : (warp >> 1 & 1) * 2;
     const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), v_sm = smem_u32(s_v), S_sm = smem_u32(s_S), w_sm = smem_u32(s_w);
     auto load = [&](int c) {
         const int buf = c & 1, left = cr.run.n - c * kC;
         const bf16* row = src.p + (size_t)(cr.run.tok0 + c * kC) * src.ld;
-        for (int i = tid; i < kC * (DP / 8); i += 128) {
+        for (int i = tid; i < kC * (DP / 8); i += kChunkThreads) {
             const int t = i / (DP / 8), d = (i - t * (DP / 8)) * 8;
             const bool in = t < left && d < g.dim;
             const bf16* p = row + (in ? (size_t)t * src.ld + kg * g.dim + d : 0);
@@ -227,7 +250,7 @@ __global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
             cp16(q_sm + at, p + (in ? src.q : 0), in ? 16 : 0);
             cp16(k_sm + at, p + (in ? src.k : 0), in ? 16 : 0);
         }
-        for (int i = tid; i < kC * (kCols / 8); i += 128) {
+        for (int i = tid; i < kC * (kCols / 8); i += kChunkThreads) {
             const int t = i / (kCols / 8), e = (i & (kCols / 8 - 1)) * 8;
             const bool in = t < left && e0 + e < g.vdim;
             cp16(v_sm + (uint32_t)((buf * kC + t) * kVP + e) * 2, row + (in ? (size_t)t * src.ld + src.v + h * g.vdim + e0 + e : 0), in ? 16 : 0);
@@ -243,8 +266,28 @@ __global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
                 bl[j] = t < cr.run.n ? step_decay(a, (size_t)(cr.run.tok0 + t), h) : make_float2(0.0f, 0.0f);
             }
     };
+    auto sums = [&](int c) {
+        if (warp != 0) return;
+        float* g2 = s_sums + (c & 1) * 3 * kC;
+        const double l0 = (double)bl[0].y * 1.4426950408889634, l1 = (double)bl[1].y * 1.4426950408889634;
+        double sum = l0 + l1;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double up = __shfl_up_sync(0xffffffffu, sum, o);
+            if (lane >= o) sum += up;
+        }
+        const double at[2] = {sum - l1, sum};
+#pragma unroll
+        for (int j = 0; j < 2; j++) {
+            const float hi = (float)at[j];
+            g2[2 * lane + j] = hi;
+            g2[kC + 2 * lane + j] = (float)(at[j] - (double)hi);
+            g2[2 * kC + 2 * lane + j] = bl[j].x;
+        }
+    };
     load(0);
     fetch(0);
+    sums(0);
     float S[kOwnM][kOwnN][4];
 #pragma unroll
     for (int i = 0; i < kOwnM; i++)
@@ -254,10 +297,11 @@ __global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
             for (int r = 0; r < 2; r++) {
                 const int d = (m0 + i) * 16 + g8 + 8 * r, e = e0 + (n0 + n) * 8 + 2 * t4;
                 float2 v = make_float2(0.0f, 0.0f);
-                if (cr.run.pos0 > 0 && d < g.dim && e < g.vdim) v = *(const float2*)(st + (size_t)d * g.vdim + e);
+                if (owner && cr.run.pos0 > 0 && d < g.dim && e < g.vdim) v = *(const float2*)(st + (size_t)d * g.vdim + e);
                 S[i][n][2 * r] = v.x; S[i][n][2 * r + 1] = v.y;
             }
     auto publish = [&]() {
+        if (!owner) return;
 #pragma unroll
         for (int i = 0; i < kOwnM; i++)
 #pragma unroll
@@ -275,28 +319,12 @@ __global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
     const int krow = (lane & 7) + ((lane >> 4) << 3), kcol = ((lane >> 3) & 1) * 8, vrow = lane & 15, vcol = (lane >> 4) * 8;
     for (int c = 0; c < cr.n_chunks; c++) {
         const int buf = c & 1;
-        if (warp == 0) {
-            const double l0 = (double)bl[0].y * 1.4426950408889634, l1 = (double)bl[1].y * 1.4426950408889634;
-            double sum = l0 + l1;
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const double up = __shfl_up_sync(0xffffffffu, sum, o);
-                if (lane >= o) sum += up;
-            }
-            const double at[2] = {sum - l1, sum};
-#pragma unroll
-            for (int j = 0; j < 2; j++) {
-                const float hi = (float)at[j];
-                s_gh[2 * lane + j] = hi;
-                s_gl[2 * lane + j] = (float)(at[j] - (double)hi);
-                s_b[2 * lane + j] = bl[j].x;
-            }
-        }
+        const float *s_gh = s_sums + buf * 3 * kC, *s_gl = s_gh + kC, *s_b = s_gl + kC;
         cp_wait<0>();
         __syncthreads();  // the chunk's rows, G and S are there; nobody reads the other buffers any more
         if (c + 1 < cr.n_chunks) { load(c + 1); fetch(c + 1); }
         const float eh = s_gh[kC - 1], el = s_gl[kC - 1], keep = exp2f(eh + el);
-        for (int i = tid; i < kC * (kCols / 2); i += 128) {  // values on their way into S
+        for (int i = tid; i < kC * (kCols / 2); i += kChunkThreads) {  // values on their way into S
             const int t = i / (kCols / 2), e = (i & (kCols / 2 - 1)) * 2;
             const float f = s_b[t] * exp2f((eh - s_gh[t]) + (el - s_gl[t]));
             const float2 v = two<bf16>(s_v + (buf * kC + t) * kVP + e);
@@ -305,38 +333,36 @@ __global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
             *(uint32_t*)(s_w + t * kVP + e) = hi;
             *(uint32_t*)(s_w + (kC + t) * kVP + e) = lo;
         }
-        float p[8][4], o[4][4], oi[4][4];
+        float p[8][4], o[2][4], oi[2][4];
 #pragma unroll
         for (int n = 0; n < 8; n++) p[n][0] = p[n][1] = p[n][2] = p[n][3] = 0.0f;
 #pragma unroll
-        for (int n = 0; n < 4; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = oi[n][0] = oi[n][1] = oi[n][2] = oi[n][3] = 0.0f;
+        for (int n = 0; n < 2; n++) o[n][0] = o[n][1] = o[n][2] = o[n][3] = oi[n][0] = oi[n][1] = oi[n][2] = oi[n][3] = 0.0f;
 #pragma unroll 2
         for (int kk = 0; kk < DP / 16; kk++) {
             uint32_t q4[4];
-            ldsm4(q_sm + (uint32_t)((buf * kC + 16 * warp + vrow) * QP + 16 * kk + vcol) * 2, q4);
+            ldsm4(q_sm + (uint32_t)((buf * kC + 16 * rb + vrow) * QP + 16 * kk + vcol) * 2, q4);
 #pragma unroll
             for (int n = 0; n < 4; n++) {
-                if (n > warp) break;
+                if (n > rb) break;
                 uint32_t kb[4];
                 ldsm4(k_sm + (uint32_t)((buf * kC + 16 * n + krow) * QP + 16 * kk + kcol) * 2, kb);
                 mma_bf16(p[2 * n], q4, kb[0], kb[1]);
                 mma_bf16(p[2 * n + 1], q4, kb[2], kb[3]);
             }
 #pragma unroll
-            for (int n = 0; n < 2; n++)
-#pragma unroll
-                for (int half = 0; half < 2; half++) {
-                    uint32_t sb[4];
-                    ldsm4t(S_sm + (uint32_t)((half * DP + 16 * kk + vrow) * kVP + 16 * n + vcol) * 2, sb);
-                    mma_bf16(oi[2 * n], q4, sb[0], sb[1]);
-                    mma_bf16(oi[2 * n + 1], q4, sb[2], sb[3]);
-                }
+            for (int half = 0; half < 2; half++) {
+                uint32_t sb[4];
+                ldsm4t(S_sm + (uint32_t)((half * DP + 16 * kk + vrow) * kVP + ch + vcol) * 2, sb);
+                mma_bf16(oi[0], q4, sb[0], sb[1]);
+                mma_bf16(oi[1], q4, sb[2], sb[3]);
+            }
         }
-        const int tr[2] = {16 * warp + g8, 16 * warp + g8 + 8};
+        const int tr[2] = {16 * rb + g8, 16 * rb + g8 + 8};
         const float gh[2] = {s_gh[tr[0]], s_gh[tr[1]]}, gl[2] = {s_gl[tr[0]], s_gl[tr[1]]};
 #pragma unroll
         for (int ks = 0; ks < 4; ks++) {
-            if (ks > warp) break;
+            if (ks > rb) break;
             uint32_t ph[4], pl[4];
 #pragma unroll
             for (int hs = 0; hs < 2; hs++) {
@@ -350,30 +376,29 @@ __global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
                 split2(f[0], f[1], ph[2 * hs], pl[2 * hs]);
                 split2(f[2], f[3], ph[2 * hs + 1], pl[2 * hs + 1]);
             }
-#pragma unroll
-            for (int n = 0; n < 2; n++) {
-                uint32_t b[4];
-                ldsm4t(v_sm + (uint32_t)((buf * kC + 16 * ks + vrow) * kVP + 16 * n + vcol) * 2, b);
-                mma_bf16(o[2 * n], ph, b[0], b[1]);
-                mma_bf16(o[2 * n + 1], ph, b[2], b[3]);
-                mma_bf16(o[2 * n], pl, b[0], b[1]);
-                mma_bf16(o[2 * n + 1], pl, b[2], b[3]);
-            }
+            uint32_t b[4];
+            ldsm4t(v_sm + (uint32_t)((buf * kC + 16 * ks + vrow) * kVP + ch + vcol) * 2, b);
+            mma_bf16(o[0], ph, b[0], b[1]);
+            mma_bf16(o[1], ph, b[2], b[3]);
+            mma_bf16(o[0], pl, b[0], b[1]);
+            mma_bf16(o[1], pl, b[2], b[3]);
         }
 #pragma unroll
         for (int r = 0; r < 2; r++) {
             const int t = c * kC + tr[r];
             if (t >= cr.run.n) continue;
             const float f = exp2f(gh[r] + gl[r]);
-            float* dst = a.o + (size_t)(cr.run.tok0 + t) * g.heads * g.vdim + h * g.vdim + e0 + 2 * t4;
+            float* dst = a.o + (size_t)(cr.run.tok0 + t) * g.heads * g.vdim + h * g.vdim + e0 + ch + 2 * t4;
 #pragma unroll
-            for (int n = 0; n < 4; n++) {
-                if (e0 + 8 * n >= g.vdim) break;
-                const float2 v = two<bf16>(s_v + (buf * kC + tr[r]) * kVP + 8 * n + 2 * t4);
+            for (int n = 0; n < 2; n++) {
+                if (e0 + ch + 8 * n >= g.vdim) break;
+                const float2 v = two<bf16>(s_v + (buf * kC + tr[r]) * kVP + ch + 8 * n + 2 * t4);
                 *(float2*)(dst + 8 * n) = make_float2(fmaf(f, oi[n][2 * r], o[n][2 * r]) + skip * v.x, fmaf(f, oi[n][2 * r + 1], o[n][2 * r + 1]) + skip * v.y);
             }
         }
+        if (c + 1 < cr.n_chunks) sums(c + 1);
         __syncthreads();  // the scaled values are there, S has been read
+        if (!owner) continue;
 #pragma unroll
         for (int i = 0; i < kOwnM; i++)
 #pragma unroll
@@ -407,7 +432,7 @@ __global__ void __launch_bounds__(128) linear_chunk_kernel(const LinearArgs a) {
 #pragma unroll
             for (int r = 0; r < 2; r++) {
                 const int d = (m0 + i) * 16 + g8 + 8 * r, e = e0 + (n0 + n) * 8 + 2 * t4;
-                if (d < g.dim && e < g.vdim) *(float2*)(st + (size_t)d * g.vdim + e) = make_float2(S[i][n][2 * r], S[i][n][2 * r + 1]);
+                if (owner && d < g.dim && e < g.vdim) *(float2*)(st + (size_t)d * g.vdim + e) = make_float2(S[i][n][2 * r], S[i][n][2 * r + 1]);
             }
 }
 
@@ -490,7 +515,195 @@ __global__ void __launch_bounds__(kStepThreads) linear_step_kernel(const LinearA
     }
 }
 
-// One CTA per (token, part of the norm).
+// The same for many (head, token) items: one CTA per SM walks them with the states in a ring of bulk copies, so that reads, sums and
+// writes of neighbouring items overlap.  The ninth warp's lane 0 issues the copies: a state and the item's rows of q, k and v in (behind
+// the convolutions), the new state out.  A stage is filled again once its store has been read.
+constexpr int kRingThreads = kStepThreads + 32;
+struct RingShape { int stages, state_bytes, stage_bytes; };  // a stage: state | q | k | v
+template <typename A>
+__global__ void __launch_bounds__(kRingThreads, 1) linear_ring_kernel(const LinearArgs a, const RingShape rs, int* error_flag) {
+    extern __shared__ __align__(128) unsigned char ring_smem[];
+    __shared__ uint64_t s_full[8], s_done[8];
+    pdl_launch_dependents();
+    const LinearShape& g = a.g;
+    const int tid = threadIdx.x, items = g.heads * a.T, rep = g.heads / g.groups, mine = items > (int)blockIdx.x ? (items - (int)blockIdx.x - 1) / (int)gridDim.x + 1 : 0;
+    float* s_o = (float*)(ring_smem + (size_t)rs.stages * rs.stage_bytes);  // [2][groups][vdim]
+    if (tid == 0) {
+        for (int i = 0; i < rs.stages; i++) { mbar_init(&s_full[i], 1); mbar_init(&s_done[i], kStepThreads); }
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    }
+    __syncthreads();
+    pdl_wait();
+    auto head_of = [&](int j) { return (int)((blockIdx.x + j * gridDim.x) % g.heads); };
+    auto token_of = [&](int j) { return (int)((blockIdx.x + j * gridDim.x) / g.heads); };
+    const size_t state_elems = (size_t)g.dim * g.vdim;
+    if (tid >= kStepThreads) {
+        const int lane = tid & 31;
+        const Rows<A> src = rows_of<A>(a);
+        int seqs = 0, seqs0 = -32;  // of items seqs0 .. seqs0 + 31, a lane each
+        auto seq_of = [&](int j) {
+            if (j >= seqs0 + 32) { seqs0 = j; seqs = j + lane < mine ? a.tok_seq[token_of(j + lane)] : 0; }
+            return __shfl_sync(0xffffffffu, seqs, j - seqs0);
+        };
+        auto load = [&](int j, int seq) {
+            if (lane != 0) return;
+            const int h = head_of(j), t = token_of(j), kg = h / rep, st = j % rs.stages;
+            unsigned char* dst = ring_smem + (size_t)st * rs.stage_bytes;
+            const A* row = src.p + (size_t)t * src.ld;
+            const uint32_t nd = (uint32_t)(g.dim * sizeof(A)), nv = (uint32_t)(g.vdim * sizeof(A));
+            mbar_expect_tx(&s_full[st], (uint32_t)rs.state_bytes + 2 * nd + nv);
+            bulk_load(dst, a.state + ((size_t)seq * g.heads + h) * state_elems, (uint32_t)rs.state_bytes, &s_full[st]);
+            bulk_load(dst + rs.state_bytes, row + src.q + kg * g.dim, nd, &s_full[st]);
+            bulk_load(dst + rs.state_bytes + nd, row + src.k + kg * g.dim, nd, &s_full[st]);
+            bulk_load(dst + rs.state_bytes + 2 * nd, row + src.v + h * g.vdim, nv, &s_full[st]);
+        };
+        // seqs of an item are needed twice, at its load and at its store: the ring of the last loads' slots
+        int slot[8];
+#pragma unroll
+        for (int i = 0; i < 8; i++) slot[i] = 0;
+        int loaded = 0, stored = 0;
+        auto load_next = [&]() {
+            const int seq = seq_of(loaded);
+#pragma unroll
+            for (int i = 0; i < 8; i++)
+                if (i == loaded % rs.stages) slot[i] = seq;
+            load(loaded, seq);
+            loaded++;
+        };
+        while (loaded < min(mine, rs.stages)) load_next();
+        bool ok = true;
+        for (; stored < mine; stored++) {
+            const int st = stored % rs.stages;
+            if (!mbar_wait(&s_done[st], (uint32_t)(stored / rs.stages) & 1)) { ok = false; break; }
+            int seq = 0;
+#pragma unroll
+            for (int i = 0; i < 8; i++)
+                if (i == st) seq = slot[i];
+            if (lane == 0) {
+                bulk_store(a.state + ((size_t)seq * g.heads + head_of(stored)) * state_elems, ring_smem + (size_t)st * rs.stage_bytes, (uint32_t)rs.state_bytes);
+                bulk_commit();
+            }
+            if (stored > 0 && loaded < mine) {  // the stage before this one has been written out
+                if (lane == 0) bulk_wait_read<1>();
+                __syncwarp();
+                load_next();
+            }
+        }
+        if (lane == 0) {
+            if (!ok) {
+                atomicExch(error_flag, 17);
+                for (int j = stored; j < loaded; j++) mbar_wait(&s_full[j % rs.stages], (uint32_t)(j / rs.stages) & 1);
+            }
+            bulk_wait<0>();
+        }
+        return;
+    }
+    const int cols = g.vdim / 4, groups = kStepThreads / cols, c = tid % cols, gr = tid / cols;
+    // what an item's factors are made of, fetched one item ahead
+    auto fetch = [&](int j, float2& bl, int& pos) {
+        if (j >= mine) return;
+        bl = step_decay(a, (size_t)token_of(j), head_of(j));
+        pos = a.tok_pos[token_of(j)];
+    };
+    float2 bl = make_float2(0.0f, 0.0f);
+    int pos = 0;
+    fetch(0, bl, pos);
+    bool ok = true;
+    for (int j = 0; j < mine; j++) {
+        const int st = j % rs.stages, h = head_of(j), t = token_of(j);
+        float2 bl_next = bl;
+        int pos_next = pos;
+        fetch(j + 1, bl_next, pos_next);
+        const float decay = pos > 0 ? expf(bl.y) : 0.0f;
+        if (ok && !mbar_wait(&s_full[st], (uint32_t)(j / rs.stages) & 1)) { ok = false; atomicExch(error_flag, 17); }  // every thread goes on to the barriers
+        float* S = (float*)(ring_smem + (size_t)st * rs.stage_bytes);
+        const A *q = (const A*)(S + state_elems), *k = q + g.dim, *v = k + g.dim;
+        float* so = s_o + (j & 1) * groups * g.vdim;
+        if (gr < groups) {
+            float4 u = make_float4(bl.x * act_f<A>(v[4 * c]), bl.x * act_f<A>(v[4 * c + 1]), bl.x * act_f<A>(v[4 * c + 2]), bl.x * act_f<A>(v[4 * c + 3]));
+            float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+            for (int d = gr; d < g.dim; d += groups) {
+                float4* at = (float4*)(S + (size_t)d * g.vdim) + c;
+                float4 x = *at;
+                if (pos == 0) x = make_float4(0.f, 0.f, 0.f, 0.f);
+                const float kk = act_f<A>(k[d]), qq = act_f<A>(q[d]);
+                x.x = fmaf(kk, u.x, x.x * decay); x.y = fmaf(kk, u.y, x.y * decay); x.z = fmaf(kk, u.z, x.z * decay); x.w = fmaf(kk, u.w, x.w * decay);
+                o.x = fmaf(x.x, qq, o.x); o.y = fmaf(x.y, qq, o.y); o.z = fmaf(x.z, qq, o.z); o.w = fmaf(x.w, qq, o.w);
+                *at = x;
+            }
+            *((float4*)(so + gr * g.vdim) + c) = o;
+        }
+        const float skip = a.skip ? a.skip[h] : 0.0f;
+        float own = 0.0f;
+        if (tid < g.vdim) own = skip * act_f<A>(v[tid]);
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+        mbar_arrive(&s_done[st]);
+        asm volatile("bar.sync 1, %0;" ::"n"(kStepThreads) : "memory");
+        if (tid < g.vdim) {
+            for (int i = 0; i < groups; i++) own += so[i * g.vdim + tid];
+            a.o[((size_t)t * g.heads + h) * g.vdim + tid] = own;
+        }
+        bl = bl_next; pos = pos_next;
+    }
+}
+
+// One CTA per (token, part of the norm); VEC = 4: rows and parts are multiples of four.
+template <typename A> __device__ __forceinline__ float4 four(const A* p);
+template <> __device__ __forceinline__ float4 four<float>(const float* p) { return *(const float4*)p; }
+template <> __device__ __forceinline__ float4 four<bf16>(const bf16* p) {
+    const uint2 v = *(const uint2*)p;
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
+}
+template <typename A> __device__ __forceinline__ void put_four(A* p, float4 v);
+template <> __device__ __forceinline__ void put_four<float>(float* p, float4 v) { *(float4*)p = v; }
+template <> __device__ __forceinline__ void put_four<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
+
+template <typename A>
+__global__ void __launch_bounds__(512) linear_output4_kernel(const LinearArgs a) {
+    __shared__ float sh[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const LinearShape& g = a.g;
+    const int inner = g.heads * g.vdim, n = inner / g.norm_parts, e0 = blockIdx.y * n;
+    const size_t t = blockIdx.x;
+    const bool gate_first = g.kind == LinearKind::StateSpace;
+    const float *o = a.o + t * inner + e0, *w = a.norm_w + e0;
+    const A* gate = (const A*)a.proj + t * g.ld + g.off_g + e0;
+    A* dst = (A*)a.out + t * a.ldo + e0;
+    constexpr int kHeld = 2;  // vectors of a thread that stay in registers between the passes
+    auto value = [&](int e, float4& z) {
+        float4 v = *(const float4*)(o + e);
+        z = four<A>(gate + e);
+        if (gate_first) { v.x *= silu_any(z.x); v.y *= silu_any(z.y); v.z *= silu_any(z.z); v.w *= silu_any(z.w); }
+        return v;
+    };
+    float4 v[kHeld], z[kHeld];
+    float ss = 0.0f;
+    auto square = [&](float4 x) { ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, fmaf(x.w, x.w, ss)))); };
+#pragma unroll
+    for (int i = 0; i < kHeld; i++) {
+        const int e = (threadIdx.x + i * blockDim.x) * 4;
+        if (e < n) v[i] = value(e, z[i]);
+        else v[i] = z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        square(v[i]);
+    }
+    for (int e = (threadIdx.x + kHeld * blockDim.x) * 4; e < n; e += blockDim.x * 4) { float4 y; square(value(e, y)); }
+    const float r = a.out_scale / sqrtf(block_sum_once(ss, sh) / (float)n + g.eps);
+    auto put = [&](int e, float4 x, float4 y) {
+        const float4 b = *(const float4*)(w + e);
+        x.x *= r * b.x; x.y *= r * b.y; x.z *= r * b.z; x.w *= r * b.w;
+        if (!gate_first) { x.x *= sigmoid_f(y.x); x.y *= sigmoid_f(y.y); x.z *= sigmoid_f(y.z); x.w *= sigmoid_f(y.w); }
+        put_four<A>(dst + e, x);
+    };
+#pragma unroll
+    for (int i = 0; i < kHeld; i++) {
+        const int e = (threadIdx.x + i * blockDim.x) * 4;
+        if (e < n) put(e, v[i], z[i]);
+    }
+    for (int e = (threadIdx.x + kHeld * blockDim.x) * 4; e < n; e += blockDim.x * 4) { float4 y; const float4 x = value(e, y); put(e, x, y); }
+}
 template <typename A>
 __global__ void __launch_bounds__(256) linear_output_kernel(const LinearArgs a) {
     __shared__ float sh[32];
@@ -529,10 +742,11 @@ __global__ void __launch_bounds__(256) linear_output_kernel(const LinearArgs a) 
 int padded_dim(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
 
 template <typename A>
-int32_t conv_dispatch(const LinearArgs& a, cudaStream_t s) {
-    const dim3 grid((unsigned)((a.T + kConvTok - 1) / kConvTok), (unsigned)((a.g.channels + 255) / 256));
+int32_t conv_dispatch(const LinearArgs& a, bool one_each, cudaStream_t s) {
+    const int stretch = a.T < 256 ? 1 : 16;
+    const dim3 grid((unsigned)((a.T + stretch - 1) / stretch), (unsigned)((a.g.channels + 255) / 256));
     auto go = [&](auto kern) -> int32_t {
-        LC_CUDA(launch_pdl(kern, grid, dim3(128), 0, s, a));
+        LC_CUDA(launch_pdl(kern, grid, dim3(128), 0, s, a, stretch, one_each ? 1 : 0));
         return LC_OK;
     };
     switch (a.g.taps) {
@@ -566,7 +780,7 @@ int32_t chunk_dispatch(const LinearArgs& a, cudaStream_t s) {
     const int dp = padded_dim(a.g.dim);
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(ensure_smem_limit((const void*)kern, chunk_smem(dp)));
-        LC_CUDA(launch_pdl(kern, grid, dim3(128), chunk_smem(dp), s, a));
+        LC_CUDA(launch_pdl(kern, grid, dim3(kChunkThreads), chunk_smem(dp), s, a));
         return LC_OK;
     };
     switch (dp) {
@@ -593,6 +807,28 @@ int32_t step_dispatch(const LinearArgs& a, cudaStream_t s) {
     return rows <= 16 ? go(linear_step_kernel<A, 1, 16>) : go(linear_step_kernel<A, 1, 0>);
 }
 
+// How the ring of states fits; stages 0: it does not, or there are too few items for it.
+RingShape ring_shape(const LinearArgs& a) {
+    const LinearShape& g = a.g;
+    const int elt = a.f32 ? 4 : 2, groups = g.vdim >= 4 ? kStepThreads / (g.vdim / 4) : 0;
+    RingShape r{0, g.dim * g.vdim * 4, 0};
+    if (g.dim % 8 || g.vdim % 8 || g.vdim > kStepThreads || g.heads * a.T < 2 * sm_count()) return r;
+    r.stage_bytes = (r.state_bytes + (2 * g.dim + g.vdim) * elt + 127) / 128 * 128;
+    const int room = (int)kMaxSmem - 1024 - 2 * groups * g.vdim * 4, stages = room / r.stage_bytes;
+    r.stages = stages < 3 ? 0 : std::min(stages, 6);
+    return r;
+}
+template <typename A>
+int32_t ring_dispatch(const LinearArgs& a, int* launches, cudaStream_t s) {
+    if (a.g.kind == LinearKind::StateSpace) { LC_TRY(conv_dispatch<A>(a, true, s)); ++*launches; }
+    const RingShape r = ring_shape(a);
+    const size_t smem = (size_t)r.stages * r.stage_bytes + (size_t)2 * (kStepThreads / (a.g.vdim / 4)) * a.g.vdim * 4;
+    LC_CUDA(ensure_smem_limit((const void*)linear_ring_kernel<A>, smem));
+    LC_CUDA(launch_pdl(linear_ring_kernel<A>, dim3((unsigned)std::min(a.g.heads * a.T, sm_count())), dim3(kRingThreads), smem, s, a, r, gemv_error_flag_dev()));
+    ++*launches;
+    return LC_OK;
+}
+
 }  // namespace
 
 bool linear_chunks_apply(const LinearShape& g, bool f32) { return !f32 && g.dim % 8 == 0 && g.vdim % 8 == 0 && g.dim <= 256; }
@@ -600,7 +836,7 @@ bool linear_chunks_apply(const LinearShape& g, bool f32) { return !f32 && g.dim 
 int32_t launch_linear_runs(const LinearArgs& a, int* launches, cudaStream_t s) {
     LC_CHECK(a.g.dim <= 256, LC_ERR_UNSUPPORTED, "linear recurrence: %d state dimensions per head (at most 256)", a.g.dim);
     const bool conv = a.g.kind == LinearKind::StateSpace;
-    if (conv) { LC_TRY(a.f32 ? conv_dispatch<float>(a, s) : conv_dispatch<bf16>(a, s)); ++*launches; }
+    if (conv) { LC_TRY(a.f32 ? conv_dispatch<float>(a, false, s) : conv_dispatch<bf16>(a, false, s)); ++*launches; }
     if (a.n_runs) { LC_TRY(a.f32 ? scan_dispatch<float>(a, s) : scan_dispatch<bf16>(a, s)); ++*launches; }
     if (a.n_chunk_runs) { LC_TRY(chunk_dispatch(a, s)); ++*launches; }
     if (!conv) return LC_OK;
@@ -610,9 +846,19 @@ int32_t launch_linear_runs(const LinearArgs& a, int* launches, cudaStream_t s) {
     ++*launches;
     return LC_OK;
 }
-int32_t launch_linear_step(const LinearArgs& a, cudaStream_t s) { return a.f32 ? step_dispatch<float>(a, s) : step_dispatch<bf16>(a, s); }
+int32_t launch_linear_step(const LinearArgs& a, int* launches, cudaStream_t s) {
+    if (ring_shape(a).stages) return a.f32 ? ring_dispatch<float>(a, launches, s) : ring_dispatch<bf16>(a, launches, s);
+    ++*launches;
+    return a.f32 ? step_dispatch<float>(a, s) : step_dispatch<bf16>(a, s);
+}
 int32_t launch_linear_output(const LinearArgs& a, cudaStream_t s) {
     const int n = a.g.heads * a.g.vdim / a.g.norm_parts;
+    if (n % 4 == 0 && a.ldo % 4 == 0 && a.g.off_g % 4 == 0 && (uintptr_t)a.norm_w % 16 == 0) {
+        const dim3 grid((unsigned)a.T, (unsigned)a.g.norm_parts), block((unsigned)std::max(32, std::min(512, (n / 8 + 31) / 32 * 32)));
+        if (a.f32) LC_CUDA(launch_pdl(linear_output4_kernel<float>, grid, block, 0, s, a));
+        else LC_CUDA(launch_pdl(linear_output4_kernel<bf16>, grid, block, 0, s, a));
+        return LC_OK;
+    }
     const dim3 grid((unsigned)a.T, (unsigned)a.g.norm_parts), block((unsigned)std::min(256, (n + 31) / 32 * 32));
     if (a.f32) LC_CUDA(launch_pdl(linear_output_kernel<float>, grid, block, 0, s, a));
     else LC_CUDA(launch_pdl(linear_output_kernel<bf16>, grid, block, 0, s, a));

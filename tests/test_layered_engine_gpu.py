@@ -335,3 +335,32 @@ def test_incomplete_models_are_named(gpu, model):
     with pytest.raises(gpu.LeafcutterError) as e:
         U.engine(gpu, cfg, wrong)
     assert e.value.status == -1 and name in str(e.value)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("shape", [dict(heads=8, groups=2, state=16, vdim=8, conv=4), dict(heads=16, groups=16, state=64, vdim=64, conv=2), dict(heads=12, groups=4, state=40, vdim=24, conv=3)])
+def test_states_of_many_sequences_step_by_step(gpu, shape, dtype):
+    """Decode steps of so many states that they pass through a ring of copies; new sequences among them, slots in no order."""
+    heads, dim, vdim = shape["heads"], shape["state"], shape["vdim"]
+    small = U.conv_attention(heads=1, kv_heads=1, dim=8, vdim=8, rot_dims=2)
+    cfg = U.munisun_config([U.scaled_pair(U.gated_attention(heads=1, kv_heads=1, dim=8, vdim=8, rot_dims=2), U.state_space(norm_groups=2, **shape)),
+                            U.normed_pair(small, U.lightning(tuple(1.0 - 0.9 ** h for h in range(heads)), dim=dim, vdim=vdim))], width=48, vocab=50)
+    w = U.munisun_weights(cfg, 5)
+    m = P.plain_model(cfg, w)
+    n_seqs = 75
+    eng = U.engine(gpu, cfg, w, dtype, max_seq_len=64, max_seqs=n_seqs)
+    slots = np.random.default_rng(1).permutation(n_seqs).tolist()
+    lens = [(0, 1, 2, 5, 33, 40)[i % 6] for i in range(n_seqs)]
+    toks = [U.tokens(n + 6, 50, 900 + i) for i, n in enumerate(lens)]
+    started = [i for i in range(n_seqs) if lens[i]]
+    eng.step([slots[i] for i in started], [toks[i][: lens[i]] for i in started], [[] for _ in started])
+    looked = [0, 1, 2, 3, 4, 5, 36, 70, 73, 74]
+    states = {i: m.new_state() for i in looked}
+    for i in looked:
+        if lens[i]:
+            m.forward(toks[i][: lens[i]], states[i])
+    for j in range(6):
+        got, _ = eng.step(slots, [[t[n + j]] for t, n in zip(toks, lens)], [[0]] * n_seqs)
+        want = np.array([m.forward([toks[i][lens[i] + j]], states[i])[0] for i in looked])
+        U.check(got[looked], want, dtype, U.rounding(cfg, dtype))
+    eng.close()
