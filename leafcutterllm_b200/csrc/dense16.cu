@@ -63,17 +63,21 @@ constexpr bool epi_splits(int epi) { return epi == DENSE_SPLIT_RELU2 || epi == D
 __device__ __forceinline__ float silu_of(float g) { return g / (1.0f + expf(-g)); }
 // z (1 + tanh u) / 2 = z / (1 + e^(-2u)), u = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_of(float z) { return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))); }
+// Element `row` of token t's row in the table, 0 for ids outside it.  The loads do not depend on a branch, so those of many tokens
+// travel together; rows and tokens outside the product read a valid place.
+__device__ __forceinline__ float table_factor(const DenseParams& p, int row, int t) {
+    const int64_t id = p.ids[min(t, p.T - 1)];
+    const bool ok = id >= 0 && id < p.table_rows;
+    const float f = __bfloat162float(__ldg(p.table + (size_t)(ok ? id : 0) * p.table_ld + min(row, p.n - 1)));
+    return ok ? f : 0.0f;
+}
 // ea, eb: the row's constants; `second`: behind the split of DENSE_SPLIT_*
 template <int EPI>
-__device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool second, float ea, float eb, float y, int row, int t) {
+__device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool second, float ea, float eb, float y, int row) {
     const float r = fmaxf(y, 0.0f);
     if constexpr (EPI == DENSE_RELU2) return r * r;
     else if constexpr (EPI == DENSE_SPLIT_RELU2) return second ? r * r : y;
-    else if constexpr (EPI == DENSE_GELU_TABLE) {
-        if (t >= p.T || row >= p.n) return 0.0f;
-        const int64_t id = p.ids[t];
-        return id >= 0 && id < p.table_rows ? gelu_of(y) * __bfloat162float(p.table[(size_t)id * p.table_ld + row]) : 0.0f;
-    } else if constexpr (EPI == DENSE_SPLIT_SILU) return second && row < p.silu_end ? silu_of(y) : y;
+    else if constexpr (EPI == DENSE_SPLIT_SILU) return second && row < p.silu_end ? silu_of(y) : y;
     else if constexpr (EPI == kEpiAny) {
         if (p.epi == DENSE_LOG_DECAY) return -ea * softplus_f(y + eb);
         const float v = y * p.scale;
@@ -102,6 +106,15 @@ __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int r
         }
         return;
     }
+    if constexpr (EPI == DENSE_GELU_TABLE) {  // all factors ahead of the first store
+        float u[16];
+#pragma unroll
+        for (int j = 0; j < 16; j++) u[j] = table_factor(p, row, t0 + j);
+#pragma unroll
+        for (int j = 0; j < 16; j++) u[j] *= gelu_of(v[j]);
+        dense_store16<DENSE_STORE>(p, b, row, t0, m, u, ea, eb);
+        return;
+    }
     // a warp's 32 rows lie on one side of a split
     const bool second = epi_splits(EPI) && row >= p.split;
     const int ldo = second ? p.ldo2 : p.ldo, r = second ? row - p.split : row;
@@ -112,13 +125,13 @@ __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int r
         float* o = (float*)out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * ldo] = dense_epilogue<EPI>(p, second, ea, eb, v[j], row, t0 + j);
+            if (j < m) o[(size_t)j * ldo] = dense_epilogue<EPI>(p, second, ea, eb, v[j], row);
     } else if ((p.n & 1) == 0 && (ldo & 1) == 0) {  // row pairs stay inside the matrix and 4-byte aligned
         const bool odd = row & 1;
         __nv_bfloat16* o = (__nv_bfloat16*)out + at - (odd ? 1 : 0);
 #pragma unroll
         for (int j = 0; j < 16; j += 2) {
-            const float x = dense_epilogue<EPI>(p, second, ea, eb, v[j], row, t0 + j), y = dense_epilogue<EPI>(p, second, ea, eb, v[j + 1], row, t0 + j + 1);
+            const float x = dense_epilogue<EPI>(p, second, ea, eb, v[j], row), y = dense_epilogue<EPI>(p, second, ea, eb, v[j + 1], row);
             const float other = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
             const __nv_bfloat162 pr = odd ? __floats2bfloat162_rn(other, y) : __floats2bfloat162_rn(x, other);
             const int jj = j + (odd ? 1 : 0);
@@ -129,7 +142,7 @@ __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int r
         __nv_bfloat16* o = (__nv_bfloat16*)out + at;
 #pragma unroll
         for (int j = 0; j < 16; j++)
-            if (j < m) o[(size_t)j * ldo] = __float2bfloat16_rn(dense_epilogue<EPI>(p, second, ea, eb, v[j], row, t0 + j));
+            if (j < m) o[(size_t)j * ldo] = __float2bfloat16_rn(dense_epilogue<EPI>(p, second, ea, eb, v[j], row));
     }
 }
 
@@ -445,10 +458,14 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
                 continue;
             }
             if (t >= T || row >= p.n) continue;
+            if constexpr (EPI == DENSE_GELU_TABLE) {
+                ((float*)p.out)[(size_t)t * p.ldo + row] = gelu_of(acc[i][j]) * table_factor(p, row, t);
+                continue;
+            }
             float ea, eb;
             dense_row_constants(p, row, ea, eb);
-            if (epi_splits(EPI) && row >= p.split) ((float*)p.out2)[(size_t)t * p.ldo2 + row - p.split] = dense_epilogue<EPI>(p, true, ea, eb, acc[i][j], row, t);
-            else ((float*)p.out)[(p.off ? 0 : (size_t)b * p.out_batch) + (size_t)(row0 + t) * p.ldo + row] = dense_epilogue<EPI>(p, false, ea, eb, acc[i][j], row, t);
+            if (epi_splits(EPI) && row >= p.split) ((float*)p.out2)[(size_t)t * p.ldo2 + row - p.split] = dense_epilogue<EPI>(p, true, ea, eb, acc[i][j], row);
+            else ((float*)p.out)[(p.off ? 0 : (size_t)b * p.out_batch) + (size_t)(row0 + t) * p.ldo + row] = dense_epilogue<EPI>(p, false, ea, eb, acc[i][j], row);
         }
     }
 }

@@ -166,7 +166,7 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a) {
 // elements, lane + 32 p, and keeps its channels' last inputs while it walks the stretch (TAPS of them; 0: no convolution; -1: any
 // number, re-read).
 template <typename A, int TAPS, int NP>
-__global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, int stretch) {
+__global__ void __launch_bounds__(256, NP <= 2 ? (TAPS == 0 ? 4 : 3) : 1) attn_head_prep_kernel(const AttnArgs a, int stretch) {
     constexpr int kWin = TAPS > 1 ? TAPS - 1 : 1, kTaps = TAPS > 0 ? TAPS : 1;
     __shared__ float s_x[8][64 * NP];
     pdl_launch_dependents();
@@ -200,7 +200,8 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
         gain[p] = g.norm == QkNorm::PerHead && !is_v ? make_float2(c < n ? gw[c] : 0.0f, c + 1 < n ? gw[c + 1] : 0.0f) : make_float2(1.0f, 1.0f);
     }
     int prev_seq = -1, prev_pos = -1;
-    constexpr int kAhead = NP == 1 || (NP == 2 && TAPS == 0) ? 4 : 2;  // tokens whose rows are fetched together
+    constexpr int kAhead = NP <= 2 ? 4 : 2;  // tokens whose rows are fetched together
+    const bool near = g.pairs == AttnPairs::Neighbours && !is_v;
     float2 ahead[kAhead][NP];
     int seq_a[kAhead], pos_a[kAhead];
     for (int tb = t0; tb < t1; tb += kAhead) {
@@ -210,7 +211,10 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
             seq_a[v] = a.tok_seq[t]; pos_a[v] = a.tok_pos[t];
             const float* row = a.proj + (size_t)t * a.ld_proj + col0;
 #pragma unroll
-            for (int p = 0; p < NP; p++) ahead[v][p] = pair_at(row, 2 * (lane + 32 * p));
+            for (int p = 0; p < NP; p++) {
+                const int i = lane + 32 * p;
+                ahead[v][p] = pair_at(row, 2 * i);
+            }
         }
 #pragma unroll
         for (int v = 0; v < kAhead; v++) {
@@ -234,11 +238,14 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
                 const float2 u = ahead[v][p];
                 x[p] = u;
                 if constexpr (TAPS > 0) {
-                    if (fresh) {
+                    if (fresh) {  // all of them on their way at once
 #pragma unroll
                         for (int j = 1; j < TAPS; j++) {
-                            const float2 v = back(j, c);
-                            win[p][0][j - 1] = v.x; win[p][1][j - 1] = v.y;
+                            const int tt = max(t - j, 0);
+                            const bool here = t - j >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j, some = pos - j >= 0;
+                            const float* r = here ? a.proj + (size_t)tt * a.ld_proj + col0 : a.ring + ((size_t)seq * TAPS + (some ? (pos - j) % TAPS : 0)) * channels + ch0;
+                            win[p][0][j - 1] = some && c < n ? r[c] : 0.0f;
+                            win[p][1][j - 1] = some && c + 1 < n ? r[c + 1] : 0.0f;
                         }
                     }
                     float2 y = make_float2(0.0f, 0.0f);
@@ -273,20 +280,20 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
 #pragma unroll
                     for (int p = 0; p < NP; p++) { x[p].x *= r * gain[p].x; x[p].y *= r * gain[p].y; }
                 }
-                const float2* tab = a.rot + (size_t)pos * half;
-                if (g.pairs == AttnPairs::Neighbours) {
+                if (near) {
 #pragma unroll
                     for (int p = 0; p < NP; p++) {
                         const int i = lane + 32 * p;
-                        if (i < half) { const float2 cs = tab[i], u = x[p]; x[p] = make_float2(u.x * cs.x - u.y * cs.y, u.y * cs.x + u.x * cs.y); }
+                        if (i < half) { const float2 cs = __ldg(a.rot + (size_t)pos * half + i), u = x[p]; x[p] = make_float2(u.x * cs.x - u.y * cs.y, u.y * cs.x + u.x * cs.y); }
                     }
                 } else if (half > 0) {
+                    const float2* tab = a.rot + (size_t)pos * half;
                     __syncwarp();
 #pragma unroll
                     for (int p = 0; p < NP; p++) *(float2*)(s_x[warp] + 2 * (lane + 32 * p)) = x[p];
                     __syncwarp();
-                    auto turned = [&](int c, float v) {
-                        if (c >= 2 * half) return v;
+                    auto turned = [&](int c, float z) {
+                        if (c >= 2 * half) return z;
                         const float2 cs = tab[c < half ? c : c - half];
                         return c < half ? v * cs.x - s_x[warp][c + half] * cs.y : v * cs.x + s_x[warp][c - half] * cs.y;
                     };
@@ -306,7 +313,7 @@ __global__ void __launch_bounds__(256) attn_head_prep_kernel(const AttnArgs a, i
             int swz = 0;
             if (is_q) dst = (A*)a.q + ((size_t)t * g.heads + h) * g.dp;
             else {
-                const int page = a.page_table[(size_t)seq * a.pages_per_seq + pos / a.page_tokens];
+                const int page = __ldg(a.page_table + (size_t)seq * a.pages_per_seq + pos / a.page_tokens);
                 const size_t at = ((size_t)page * g.kv_heads + h) * a.page_tokens + pos % a.page_tokens;
                 dst = is_v ? (A*)a.v_cache + at * g.v_pitch : (A*)a.k_cache + at * g.k_pitch;
                 swz = is_v ? g.v_swz : g.k_swz;
@@ -765,7 +772,7 @@ int pitch_of(int n8, bool f32, int* swz) {
 bool tensor_form(const AttnShape& g, bool f32) { return !f32 && g.ep <= 256 && tokens_smem(g) <= kMaxSmem - 4096 && tiles_smem(g) <= kMaxSmem - 1024; }
 template <typename A, int TAPS>
 int32_t head_prep_pairs(const AttnArgs& a, cudaStream_t s) {
-    const int pairs = (std::max(a.g.dim, a.g.vdim) + 63) / 64, stretch = a.T < 256 ? 1 : 16;
+    const int pairs = (std::max(a.g.dim, a.g.vdim) + 63) / 64, stretch = a.T < 256 ? 1 : TAPS == 0 ? 4 : 16;
     const dim3 grid((unsigned)((a.T + stretch - 1) / stretch), (unsigned)((a.g.heads + 2 * a.g.kv_heads + 7) / 8));
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(launch_pdl(kern, grid, dim3(256), 0, s, a, stretch));

@@ -21,7 +21,12 @@ namespace lc {
 
 namespace {
 
-__device__ __forceinline__ float silu_any(float v) { return v / (1.0f + expf(-v)); }
+// of activations: with the quick exponential and division where the result is rounded to bf16
+template <typename A> __device__ __forceinline__ float sigmoid_of(float v) {
+    if constexpr (sizeof(A) == 2) return __fdividef(1.0f, 1.0f + __expf(-v));
+    else return 1.0f / (1.0f + expf(-v));
+}
+template <typename A> __device__ __forceinline__ float silu_any(float v) { return v * sigmoid_of<A>(v); }
 __device__ __forceinline__ float softplus_of(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // (b, l) of head h at token t
 __device__ __forceinline__ float2 step_decay(const LinearArgs& a, size_t t, int h) {
@@ -119,7 +124,7 @@ __global__ void __launch_bounds__(128) linear_conv_kernel(const LinearArgs a, in
                     y.x = fmaf(cw.x, v.x, y.x); y.y = fmaf(cw.y, v.y, y.y);
                 }
             }
-            put_two<A>((A*)a.in + (size_t)t * g.ld_in + c, make_float2(silu_any(y.x), silu_any(y.y)));
+            put_two<A>((A*)a.in + (size_t)t * g.ld_in + c, make_float2(silu_any<A>(y.x), silu_any<A>(y.y)));
             if (one_each) {
                 A* r = (A*)a.ring + ((size_t)seq * taps + pos % taps) * g.channels + c;
                 r[0] = to_act<A>(u.x);
@@ -235,7 +240,8 @@ __global__ void __launch_bounds__(kChunkThreads, DP <= 128 ? 2 : 1) linear_chunk
     const Rows<bf16> src = rows_of<bf16>(a);
     const float skip = a.skip ? a.skip[h] : 0.0f;
     float* st = a.state + ((size_t)cr.run.seq * g.heads + h) * g.dim * g.vdim;
-    const int rb = warp & 3, ch = (warp >> 2) * 16;  // this warp's tokens (16 rb ..) and columns of the read-outs
+    // this warp's tokens (16 rb ..) and columns of the read-outs; the two warps of a scheduler (warp & 3) share the triangle evenly
+    const int rb = warp < 4 ? warp : 7 - warp, ch = (warp >> 2) * 16;
     const bool owner = kMT >= 4 || warp < 4;
     const int m0 = kMT >= 8 ? warp * kOwnM : kMT == 4 ? warp & 3 : warp & 1, n0 = kMT >= 8 ? 0 : kMT == 4 ? (warp >> 2) * 2 : (warp >> 1 & 1) * 2;
     const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), v_sm = smem_u32(s_v), S_sm = smem_u32(s_S), w_sm = smem_u32(s_w);
@@ -478,7 +484,7 @@ __global__ void __launch_bounds__(kStepThreads) linear_step_kernel(const LinearA
             float acc = a.conv_b[channel];
             for (int j = g.taps - 1; j > 0; j--)
                 if (pos - j >= 0) acc = fmaf(w[g.taps - 1 - j], act_f<A>(ring[(size_t)((pos - j) % g.taps) * g.channels]), acc);
-            y = act_f<A>(to_act<A>(silu_any(fmaf(w[g.taps - 1], y, acc))));  // the type that runs of tokens keep it in
+            y = act_f<A>(to_act<A>(silu_any<A>(fmaf(w[g.taps - 1], y, acc))));  // the type that runs of tokens keep it in
             if (part == 2 || h % rep == 0) ring[(size_t)(pos % g.taps) * g.channels] = cur;
         }
         sm[i] = y;
@@ -676,7 +682,7 @@ __global__ void __launch_bounds__(512) linear_output4_kernel(const LinearArgs a)
     auto value = [&](int e, float4& z) {
         float4 v = *(const float4*)(o + e);
         z = four<A>(gate + e);
-        if (gate_first) { v.x *= silu_any(z.x); v.y *= silu_any(z.y); v.z *= silu_any(z.z); v.w *= silu_any(z.w); }
+        if (gate_first) { v.x *= silu_any<A>(z.x); v.y *= silu_any<A>(z.y); v.z *= silu_any<A>(z.z); v.w *= silu_any<A>(z.w); }
         return v;
     };
     float4 v[kHeld], z[kHeld];
@@ -694,7 +700,7 @@ __global__ void __launch_bounds__(512) linear_output4_kernel(const LinearArgs a)
     auto put = [&](int e, float4 x, float4 y) {
         const float4 b = *(const float4*)(w + e);
         x.x *= r * b.x; x.y *= r * b.y; x.z *= r * b.z; x.w *= r * b.w;
-        if (!gate_first) { x.x *= sigmoid_f(y.x); x.y *= sigmoid_f(y.y); x.z *= sigmoid_f(y.z); x.w *= sigmoid_f(y.w); }
+        if (!gate_first) { x.x *= sigmoid_of<A>(y.x); x.y *= sigmoid_of<A>(y.y); x.z *= sigmoid_of<A>(y.z); x.w *= sigmoid_of<A>(y.w); }
         put_four<A>(dst + e, x);
     };
 #pragma unroll
@@ -715,7 +721,7 @@ __global__ void __launch_bounds__(256) linear_output_kernel(const LinearArgs a) 
     const bool gate_first = g.kind == LinearKind::StateSpace;
     const float* o = a.o + t * inner + e0;
     const A* gate = (const A*)a.proj + t * g.ld + g.off_g + e0;
-    auto value = [&](int e) { return gate_first ? o[e] * silu_any(act_f<A>(gate[e])) : o[e]; };
+    auto value = [&](int e) { return gate_first ? o[e] * silu_any<A>(act_f<A>(gate[e])) : o[e]; };
     constexpr int kHeld = 8;  // elements of a thread that stay in registers between the passes
     float v[kHeld], ss = 0.0f;
 #pragma unroll
@@ -729,7 +735,7 @@ __global__ void __launch_bounds__(256) linear_output_kernel(const LinearArgs a) 
     A* dst = (A*)a.out + t * a.ldo + e0;
     auto put = [&](int e, float x) {
         x *= r * a.norm_w[e0 + e];
-        dst[e] = to_act<A>(gate_first ? x : x * sigmoid_f(act_f<A>(gate[e])));
+        dst[e] = to_act<A>(gate_first ? x : x * sigmoid_of<A>(act_f<A>(gate[e])));
     };
 #pragma unroll
     for (int i = 0; i < kHeld; i++) {
