@@ -315,6 +315,13 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
             const int row = r.m * kM + row_in, t0 = r.t0, ob = GROUPED ? 0 : r.b;
             float ea, eb;
             dense_row_constants(p, row, ea, eb);
+            if constexpr (EPI == DENSE_GELU_TABLE) {  // the warp's part of its tokens' rows, a lane each, while the products run
+                const int t = t0 + c_lo + lane;
+                if (lane < kHalf && t < p.T && row - lane < p.n) {
+                    const int64_t id = p.ids[t];
+                    if (id >= 0 && id < p.table_rows) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.table + (size_t)id * p.table_ld + row - lane));
+                }
+            }
             if (!mbar_wait(&acc_full[set], (uint32_t)(tile / 2) & 1)) { *stop = 1; if (lane == 0) atomicExch(p.error_flag, 13); break; }
             tc_fence_after();
             const uint32_t base = tmem + (uint32_t)set * kCols + ((uint32_t)(quarter * 32) << 16);

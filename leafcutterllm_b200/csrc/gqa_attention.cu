@@ -77,9 +77,6 @@ __device__ __forceinline__ void request_rows(const AttnArgs& a, const int32_t* p
 template <typename A> __device__ __forceinline__ void put4(A* p, float4 v);
 template <> __device__ __forceinline__ void put4<float>(float* p, float4 v) { *(float4*)p = v; }
 template <> __device__ __forceinline__ void put4<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
-template <typename A> __device__ __forceinline__ void put2(A* p, float2 v);
-template <> __device__ __forceinline__ void put2<float>(float* p, float2 v) { *(float2*)p = v; }
-template <> __device__ __forceinline__ void put2<bf16>(bf16* p, float2 v) { *(uint32_t*)p = pack2(v.x, v.y); }
 
 // One CTA per token and share of its elements; VEC = 4: dim, vdim and the rotated half are multiples of four.
 template <typename A, int VEC>
@@ -162,13 +159,14 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a) {
     }
 }
 
-// Norms per head: one warp per (stretch of tokens, head): the heads of q, then of k, then of v.  A lane owns pairs of neighbouring
-// elements, lane + 32 p, and keeps its channels' last inputs while it walks the stretch (TAPS of them; 0: no convolution; -1: any
-// number, re-read).
-template <typename A, int TAPS, int NP>
-__global__ void __launch_bounds__(256, NP <= 2 ? (TAPS == 0 ? 4 : 3) : 1) attn_head_prep_kernel(const AttnArgs a, int stretch) {
+// Norms per head: one warp per (stretch of tokens, head): the heads of q, then of k, then of v.  A lane owns four neighbouring
+// elements, from 4 (lane + 32 p) on, and keeps its channels' last inputs while it walks the stretch (TAPS of them; 0: no
+// convolution; -1: any number, re-read).  AHEAD: tokens whose rows, angles and pages are fetched together; behind the last one it
+// is taken again, with the same result.
+template <typename A, int TAPS, int NQ, int AHEAD>
+__global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head_prep_kernel(const AttnArgs a, int stretch) {
     constexpr int kWin = TAPS > 1 ? TAPS - 1 : 1, kTaps = TAPS > 0 ? TAPS : 1;
-    __shared__ float s_x[8][64 * NP];
+    __shared__ float s_x[8][128 * NQ];
     pdl_launch_dependents();
     pdl_wait();
     const AttnShape& g = a.g;
@@ -179,152 +177,182 @@ __global__ void __launch_bounds__(256, NP <= 2 ? (TAPS == 0 ? 4 : 3) : 1) attn_h
     const int nq = g.heads * g.dim, nk = g.kv_heads * g.dim, channels = nq + nk + g.kv_heads * g.vdim;
     const int ch0 = (is_q ? 0 : is_v ? nq + nk : nq) + h * n, col0 = (is_q ? 0 : is_v ? a.off_v : a.off_k) + h * n;
     const int taps = TAPS > 0 ? TAPS : g.taps;
-    const bool even = (n & 1) == 0;  // then pairs are 8-byte aligned
-    auto pair_at = [&](const float* row, int c) {
-        if (c >= n) return make_float2(0.0f, 0.0f);
-        return even ? *(const float2*)(row + c) : make_float2(row[c], c + 1 < n ? row[c + 1] : 0.0f);
+    const bool vec = (n & 3) == 0;  // then a lane's elements exist together and lie 16-byte aligned in the projected rows
+    const bool near = g.pairs == AttnPairs::Neighbours && !is_v, near4 = near && (half & 1) == 0;
+    auto four_at = [&](const float* row, int c, float (&x)[4]) {
+        if (vec) {
+            const float4 u = c < n ? *(const float4*)(row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            x[0] = u.x; x[1] = u.y; x[2] = u.z; x[3] = u.w;
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; e++) x[e] = c + e < n ? row[c + e] : 0.0f;
+        }
+    };
+    auto angles_at = [&](int pos, int c, float2 (&cs)[2]) {  // of the pairs (c, c + 1) and (c + 2, c + 3)
+        cs[0] = cs[1] = make_float2(1.0f, 0.0f);
+        const float2* tab = a.rot + (size_t)pos * half + c / 2;
+        if (near4) {
+            if (c < 2 * half) { const float4 u = __ldg((const float4*)tab); cs[0] = make_float2(u.x, u.y); cs[1] = make_float2(u.z, u.w); }
+        } else if (near) {
+            if (c < 2 * half) cs[0] = __ldg(tab);
+            if (c + 2 < 2 * half) cs[1] = __ldg(tab + 1);
+        }
     };
     const int t0 = blockIdx.x * stretch, t1 = min(a.T, t0 + stretch);
-    float w[NP][2][kTaps], win[NP][2][kWin];  // win[.][.][j]: the input j + 1 tokens back
-    float2 gain[NP];
+    float w[NQ][4][kTaps], win[NQ][4][kWin], gain[NQ][4];  // win[.][.][j]: the input j + 1 tokens back
     const float* gw = is_q ? a.q_norm : a.k_norm;
 #pragma unroll
-    for (int p = 0; p < NP; p++) {
-        const int c = 2 * (lane + 32 * p);
-        if constexpr (TAPS > 0)
+    for (int p = 0; p < NQ; p++)
 #pragma unroll
-            for (int j = 0; j < TAPS; j++) {
-                w[p][0][j] = c < n ? a.conv[(size_t)(ch0 + c) * TAPS + j] : 0.0f;
-                w[p][1][j] = c + 1 < n ? a.conv[(size_t)(ch0 + c + 1) * TAPS + j] : 0.0f;
-            }
-        gain[p] = g.norm == QkNorm::PerHead && !is_v ? make_float2(c < n ? gw[c] : 0.0f, c + 1 < n ? gw[c + 1] : 0.0f) : make_float2(1.0f, 1.0f);
-    }
+        for (int e = 0; e < 4; e++) {
+            const int c = 4 * (lane + 32 * p) + e;
+            if constexpr (TAPS > 0)
+#pragma unroll
+                for (int j = 0; j < TAPS; j++) w[p][e][j] = c < n ? a.conv[(size_t)(ch0 + c) * TAPS + j] : 0.0f;
+            gain[p][e] = g.norm != QkNorm::PerHead || is_v ? 1.0f : c < n ? gw[c] : 0.0f;
+        }
     int prev_seq = -1, prev_pos = -1;
-    constexpr int kAhead = NP <= 2 ? 4 : 2;  // tokens whose rows are fetched together
-    const bool near = g.pairs == AttnPairs::Neighbours && !is_v;
-    float2 ahead[kAhead][NP];
-    int seq_a[kAhead], pos_a[kAhead];
-    for (int tb = t0; tb < t1; tb += kAhead) {
+    float ahead[AHEAD][NQ][4];
+    float2 turn[AHEAD][NQ][2];
+    int seq_a[AHEAD], pos_a[AHEAD], page_a[AHEAD];
+    for (int tb = t0; tb < t1; tb += AHEAD) {
 #pragma unroll
-        for (int v = 0; v < kAhead; v++) {
+        for (int v = 0; v < AHEAD; v++) {
             const int t = min(tb + v, t1 - 1);
             seq_a[v] = a.tok_seq[t]; pos_a[v] = a.tok_pos[t];
             const float* row = a.proj + (size_t)t * a.ld_proj + col0;
 #pragma unroll
-            for (int p = 0; p < NP; p++) {
-                const int i = lane + 32 * p;
-                ahead[v][p] = pair_at(row, 2 * i);
+            for (int p = 0; p < NQ; p++) {
+                four_at(row, 4 * (lane + 32 * p), ahead[v][p]);
+                angles_at(pos_a[v], 4 * (lane + 32 * p), turn[v][p]);
             }
+            page_a[v] = is_q ? 0 : __ldg(a.page_table + (size_t)seq_a[v] * a.pages_per_seq + pos_a[v] / a.page_tokens);
         }
 #pragma unroll
-        for (int v = 0; v < kAhead; v++) {
-            const int t = tb + v;
-            if (t >= t1) break;
-            const int seq = seq_a[v], pos = pos_a[v];
-            // the inputs j tokens back: from the call's rows as far as they belong to this run, from the ring before that, zero before the start
-            auto back = [&](int j, int c) {
-                if (pos - j < 0) return make_float2(0.0f, 0.0f);
-                const int tt = t - j;
-                if (tt >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j) return pair_at(a.proj + (size_t)tt * a.ld_proj + col0, c);
-                const float* r = a.ring + ((size_t)seq * taps + (pos - j) % taps) * channels + ch0 + c;  // rows of any length: not aligned for pairs
-                return make_float2(c < n ? r[0] : 0.0f, c + 1 < n ? r[1] : 0.0f);
+        for (int v = 0; v < AHEAD; v++) {
+            const int t = min(tb + v, t1 - 1), seq = seq_a[v], pos = pos_a[v];
+            // where the inputs j tokens back are: the call's rows as far as they belong to this run, the ring before that (zero before the start)
+            auto back_row = [&](int j) {
+                const int tt = max(t - j, 0);
+                const bool here = t - j >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j;
+                return here ? a.proj + (size_t)tt * a.ld_proj + col0 : a.ring + ((size_t)seq * taps + (pos >= j ? (pos - j) % taps : 0)) * channels + ch0;
             };
-            float2 x[NP];
-            const bool fresh = seq != prev_seq || pos != prev_pos + 1;
+            float x[NQ][4];
+            if constexpr (TAPS > 0)
+                if (seq != prev_seq || pos != prev_pos + 1) {
+#pragma unroll
+                    for (int j = 1; j < TAPS; j++) {
+                        const float* r = back_row(j);
+#pragma unroll
+                        for (int p = 0; p < NQ; p++)
+#pragma unroll
+                            for (int e = 0; e < 4; e++) {
+                                const int c = 4 * (lane + 32 * p) + e;
+                                win[p][e][j - 1] = pos >= j && c < n ? r[c] : 0.0f;
+                            }
+                    }
+                }
             float ss = 0.0f;
 #pragma unroll
-            for (int p = 0; p < NP; p++) {
-                const int c = 2 * (lane + 32 * p);
-                const float2 u = ahead[v][p];
-                x[p] = u;
-                if constexpr (TAPS > 0) {
-                    if (fresh) {  // all of them on their way at once
+            for (int p = 0; p < NQ; p++)
 #pragma unroll
-                        for (int j = 1; j < TAPS; j++) {
-                            const int tt = max(t - j, 0);
-                            const bool here = t - j >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j, some = pos - j >= 0;
-                            const float* r = here ? a.proj + (size_t)tt * a.ld_proj + col0 : a.ring + ((size_t)seq * TAPS + (some ? (pos - j) % TAPS : 0)) * channels + ch0;
-                            win[p][0][j - 1] = some && c < n ? r[c] : 0.0f;
-                            win[p][1][j - 1] = some && c + 1 < n ? r[c + 1] : 0.0f;
-                        }
+                for (int e = 0; e < 4; e++) {
+                    const float u = ahead[v][p][e];
+                    float y = u;
+                    if constexpr (TAPS > 0) {
+                        y = 0.0f;
+#pragma unroll
+                        for (int j = TAPS - 1; j > 0; j--) y = fmaf(w[p][e][TAPS - 1 - j], win[p][e][j - 1], y);
+                        y = fmaf(w[p][e][TAPS - 1], u, y);
+#pragma unroll
+                        for (int j = TAPS - 2; j > 0; j--) win[p][e][j] = win[p][e][j - 1];
+                        win[p][e][0] = u;
+                    } else if constexpr (TAPS < 0) {
+                        y = 0.0f;
+                        const int c = 4 * (lane + 32 * p) + e;
+                        if (c < n)
+                            for (int j = taps - 1; j >= 0; j--) {
+                                const float z = j == 0 ? u : pos >= j ? back_row(j)[c] : 0.0f;
+                                y = fmaf(a.conv[(size_t)(ch0 + c) * taps + taps - 1 - j], z, y);
+                            }
                     }
-                    float2 y = make_float2(0.0f, 0.0f);
-#pragma unroll
-                    for (int j = TAPS - 1; j > 0; j--) { y.x = fmaf(w[p][0][TAPS - 1 - j], win[p][0][j - 1], y.x); y.y = fmaf(w[p][1][TAPS - 1 - j], win[p][1][j - 1], y.y); }
-                    x[p] = make_float2(fmaf(w[p][0][TAPS - 1], u.x, y.x), fmaf(w[p][1][TAPS - 1], u.y, y.y));
-#pragma unroll
-                    for (int j = TAPS - 2; j > 0; j--) { win[p][0][j] = win[p][0][j - 1]; win[p][1][j] = win[p][1][j - 1]; }
-                    win[p][0][0] = u.x; win[p][1][0] = u.y;
-                } else if constexpr (TAPS < 0) {
-                    float2 y = make_float2(0.0f, 0.0f);
-                    if (c < n)
-                        for (int j = taps - 1; j >= 0; j--) {
-                            const float2 v = j == 0 ? u : back(j, c);
-                            const float* cw = a.conv + (size_t)(ch0 + c) * taps + taps - 1 - j;
-                            y.x = fmaf(cw[0], v.x, y.x);
-                            if (c + 1 < n) y.y = fmaf(cw[taps], v.y, y.y);
-                        }
-                    x[p] = y;
+                    x[p][e] = y;
+                    ss = fmaf(y, y, ss);
                 }
-                if (TAPS != 0 && a.one_each && c < n) {
-                    float* r = a.ring + ((size_t)seq * taps + pos % taps) * channels + ch0 + c;
-                    r[0] = u.x;
-                    if (c + 1 < n) r[1] = u.y;
-                }
-                ss = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, ss));
-            }
+            if (TAPS != 0 && a.one_each)
+#pragma unroll
+                for (int p = 0; p < NQ; p++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const int c = 4 * (lane + 32 * p) + e;
+                        if (c < n) a.ring[((size_t)seq * taps + pos % taps) * channels + ch0 + c] = ahead[v][p][e];
+                    }
             prev_seq = seq; prev_pos = pos;
             if (!is_v) {
                 if (g.norm == QkNorm::PerHead) {
                     const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
 #pragma unroll
-                    for (int p = 0; p < NP; p++) { x[p].x *= r * gain[p].x; x[p].y *= r * gain[p].y; }
+                    for (int p = 0; p < NQ; p++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++) x[p][e] *= r * gain[p][e];
                 }
                 if (near) {
 #pragma unroll
-                    for (int p = 0; p < NP; p++) {
-                        const int i = lane + 32 * p;
-                        if (i < half) { const float2 cs = __ldg(a.rot + (size_t)pos * half + i), u = x[p]; x[p] = make_float2(u.x * cs.x - u.y * cs.y, u.y * cs.x + u.x * cs.y); }
-                    }
+                    for (int p = 0; p < NQ; p++)
+#pragma unroll
+                        for (int e = 0; e < 4; e += 2) {
+                            const float2 cs = turn[v][p][e / 2];
+                            const float y = x[p][e], z = x[p][e + 1];
+                            x[p][e] = y * cs.x - z * cs.y;
+                            x[p][e + 1] = z * cs.x + y * cs.y;
+                        }
                 } else if (half > 0) {
                     const float2* tab = a.rot + (size_t)pos * half;
                     __syncwarp();
 #pragma unroll
-                    for (int p = 0; p < NP; p++) *(float2*)(s_x[warp] + 2 * (lane + 32 * p)) = x[p];
+                    for (int p = 0; p < NQ; p++) *(float4*)(s_x[warp] + 4 * (lane + 32 * p)) = make_float4(x[p][0], x[p][1], x[p][2], x[p][3]);
                     __syncwarp();
-                    auto turned = [&](int c, float z) {
-                        if (c >= 2 * half) return z;
-                        const float2 cs = tab[c < half ? c : c - half];
-                        return c < half ? v * cs.x - s_x[warp][c + half] * cs.y : v * cs.x + s_x[warp][c - half] * cs.y;
-                    };
 #pragma unroll
-                    for (int p = 0; p < NP; p++) { const int c = 2 * (lane + 32 * p); x[p] = make_float2(turned(c, x[p].x), turned(c + 1, x[p].y)); }
+                    for (int p = 0; p < NQ; p++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const int c = 4 * (lane + 32 * p) + e;
+                            if (c >= 2 * half) continue;
+                            const float2 cs = tab[c < half ? c : c - half];
+                            x[p][e] = c < half ? x[p][e] * cs.x - s_x[warp][c + half] * cs.y : x[p][e] * cs.x + s_x[warp][c - half] * cs.y;
+                        }
                 }
                 if (g.norm == QkNorm::PerHeadAfter) {
                     ss = 0.0f;
 #pragma unroll
-                    for (int p = 0; p < NP; p++) ss = fmaf(x[p].x, x[p].x, fmaf(x[p].y, x[p].y, ss));
+                    for (int p = 0; p < NQ; p++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++) ss = fmaf(x[p][e], x[p][e], ss);
                     const float r = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
 #pragma unroll
-                    for (int p = 0; p < NP; p++) { x[p].x *= r; x[p].y *= r; }
+                    for (int p = 0; p < NQ; p++)
+#pragma unroll
+                        for (int e = 0; e < 4; e++) x[p][e] *= r;
                 }
             }
             A* dst;
             int swz = 0;
             if (is_q) dst = (A*)a.q + ((size_t)t * g.heads + h) * g.dp;
             else {
-                const int page = __ldg(a.page_table + (size_t)seq * a.pages_per_seq + pos / a.page_tokens);
-                const size_t at = ((size_t)page * g.kv_heads + h) * a.page_tokens + pos % a.page_tokens;
+                const size_t at = ((size_t)page_a[v] * g.kv_heads + h) * a.page_tokens + pos % a.page_tokens;
                 dst = is_v ? (A*)a.v_cache + at * g.v_pitch : (A*)a.k_cache + at * g.k_pitch;
                 swz = is_v ? g.v_swz : g.k_swz;
             }
 #pragma unroll
-            for (int p = 0; p < NP; p++) {
-                const int c = 2 * (lane + 32 * p);
+            for (int p = 0; p < NQ; p++) {
+                const int c = 4 * (lane + 32 * p);
                 if (c >= n) continue;
                 A* d = dst + cell_of(c, pos, swz);
-                if (c + 1 < n) put2<A>(d, x[p]);
-                else d[0] = to_act<A>(x[p].x);
+                if (vec) put4<A>(d, make_float4(x[p][0], x[p][1], x[p][2], x[p][3]));
+                else
+#pragma unroll
+                    for (int e = 0; e < 4; e++)
+                        if (c + e < n) d[e] = to_act<A>(x[p][e]);
             }
         }
     }
@@ -771,26 +799,29 @@ int pitch_of(int n8, bool f32, int* swz) {
 }
 bool tensor_form(const AttnShape& g, bool f32) { return !f32 && g.ep <= 256 && tokens_smem(g) <= kMaxSmem - 4096 && tiles_smem(g) <= kMaxSmem - 1024; }
 template <typename A, int TAPS>
-int32_t head_prep_pairs(const AttnArgs& a, cudaStream_t s) {
-    const int pairs = (std::max(a.g.dim, a.g.vdim) + 63) / 64, stretch = a.T < 256 ? 1 : TAPS == 0 ? 4 : 16;
-    const dim3 grid((unsigned)((a.T + stretch - 1) / stretch), (unsigned)((a.g.heads + 2 * a.g.kv_heads + 7) / 8));
-    auto go = [&](auto kern) -> int32_t {
+int32_t head_prep_taps(const AttnArgs& a, cudaStream_t s) {
+    const int widest = std::max(a.g.dim, a.g.vdim);
+    auto go = [&](auto kern, int stretch) -> int32_t {
+        const dim3 grid((unsigned)((a.T + stretch - 1) / stretch), (unsigned)((a.g.heads + 2 * a.g.kv_heads + 7) / 8));
         LC_CUDA(launch_pdl(kern, grid, dim3(256), 0, s, a, stretch));
         return LC_OK;
     };
-    LC_CHECK(pairs <= 8, LC_ERR_UNSUPPORTED, "attention: heads of %d and %d dimensions (at most 512)", a.g.dim, a.g.vdim);
-    return pairs == 1 ? go(attn_head_prep_kernel<A, TAPS, 1>) : pairs == 2 ? go(attn_head_prep_kernel<A, TAPS, 2>) : pairs <= 4 ? go(attn_head_prep_kernel<A, TAPS, 4>)
-                                                                                                                            : go(attn_head_prep_kernel<A, TAPS, 8>);
+    LC_CHECK(widest <= 512, LC_ERR_UNSUPPORTED, "attention: heads of %d and %d dimensions (at most 512)", a.g.dim, a.g.vdim);
+    if constexpr (sizeof(A) == 2 && TAPS >= 0)
+        if (a.T >= 256 && widest <= 128) return go(attn_head_prep_kernel<A, TAPS, 1, 2>, TAPS ? 16 : 4);
+    const int stretch = a.T < 256 ? 1 : 8;
+    return widest <= 128 ? go(attn_head_prep_kernel<A, TAPS, 1, 1>, stretch) : widest <= 256 ? go(attn_head_prep_kernel<A, TAPS, 2, 1>, stretch)
+                                                                                             : go(attn_head_prep_kernel<A, TAPS, 4, 1>, stretch);
 }
 template <typename A>
 int32_t head_prep(const AttnArgs& a, cudaStream_t s) {
     LC_CHECK(a.off_k >= 0, LC_ERR_UNSUPPORTED, "attention: norms per head over another layer's cache");
     switch (a.g.taps) {
-        case 0: return head_prep_pairs<A, 0>(a, s);
-        case 2: return head_prep_pairs<A, 2>(a, s);
-        case 3: return head_prep_pairs<A, 3>(a, s);
-        case 4: return head_prep_pairs<A, 4>(a, s);
-        default: return head_prep_pairs<A, -1>(a, s);
+        case 0: return head_prep_taps<A, 0>(a, s);
+        case 2: return head_prep_taps<A, 2>(a, s);
+        case 3: return head_prep_taps<A, 3>(a, s);
+        case 4: return head_prep_taps<A, 4>(a, s);
+        default: return head_prep_taps<A, -1>(a, s);
     }
 }
 int cells(const AttnShape& g) { return g.kv_heads * ((g.heads / g.kv_heads + 15) / 16); }

@@ -49,6 +49,15 @@ template <> __device__ __forceinline__ float2 two<bf16>(const bf16* p) { return 
 template <typename A> __device__ __forceinline__ void put_two(A* p, float2 v);
 template <> __device__ __forceinline__ void put_two<float>(float* p, float2 v) { *(float2*)p = v; }
 template <> __device__ __forceinline__ void put_two<bf16>(bf16* p, float2 v) { *(uint32_t*)p = pack2(v.x, v.y); }
+template <typename A> __device__ __forceinline__ float4 four(const A* p);
+template <> __device__ __forceinline__ float4 four<float>(const float* p) { return *(const float4*)p; }
+template <> __device__ __forceinline__ float4 four<bf16>(const bf16* p) {
+    const uint2 v = *(const uint2*)p;
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
+}
+template <typename A> __device__ __forceinline__ void put_four(A* p, float4 v);
+template <> __device__ __forceinline__ void put_four<float>(float* p, float4 v) { *(float4*)p = v; }
+template <> __device__ __forceinline__ void put_four<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
 
 // A thread walks `stretch` tokens of two neighbouring channels and keeps their last inputs in registers (TAPS of them; 0: any
 // number, re-read).  Inputs of earlier positions come from the call's rows as far as they belong to the same run, from the ring
@@ -106,9 +115,12 @@ __global__ void __launch_bounds__(128) linear_conv_kernel(const LinearArgs a, in
             if constexpr (TAPS > 0) {
                 if (seq != prev_seq || pos != prev_pos + 1) {
 #pragma unroll
-                    for (int j = 1; j < TAPS; j++) {
-                        const float2 v = back(j);
-                        win[0][j - 1] = v.x; win[1][j - 1] = v.y;
+                    for (int j = 1; j < TAPS; j++) {  // all of them on their way at once
+                        const int tt = max(t - j, 0);
+                        const bool here = t - j >= 0 && a.tok_seq[tt] == seq && a.tok_pos[tt] == pos - j;
+                        const A* r = here ? in + (size_t)tt * g.ld : ring + ((size_t)seq * TAPS + (pos >= j ? (pos - j) % TAPS : 0)) * g.channels;
+                        win[0][j - 1] = pos >= j ? act_f<A>(r[0]) : 0.0f;
+                        win[1][j - 1] = pos >= j && both ? act_f<A>(r[1]) : 0.0f;
                     }
                 }
 #pragma unroll
@@ -655,17 +667,7 @@ __global__ void __launch_bounds__(kRingThreads, 1) linear_ring_kernel(const Line
     }
 }
 
-// One CTA per (token, part of the norm); VEC = 4: rows and parts are multiples of four.
-template <typename A> __device__ __forceinline__ float4 four(const A* p);
-template <> __device__ __forceinline__ float4 four<float>(const float* p) { return *(const float4*)p; }
-template <> __device__ __forceinline__ float4 four<bf16>(const bf16* p) {
-    const uint2 v = *(const uint2*)p;
-    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
-}
-template <typename A> __device__ __forceinline__ void put_four(A* p, float4 v);
-template <> __device__ __forceinline__ void put_four<float>(float* p, float4 v) { *(float4*)p = v; }
-template <> __device__ __forceinline__ void put_four<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
-
+// One CTA per (token, part of the norm); linear_output4_kernel: rows and parts are multiples of four.
 template <typename A>
 __global__ void __launch_bounds__(512) linear_output4_kernel(const LinearArgs a) {
     __shared__ float sh[32];
