@@ -184,7 +184,7 @@ int32_t parse_lightning(const Fields& m, MixerSpec* out) {
     LC_CHECK((int)d->arr.size() == out->heads, LC_ERR_INVALID, "config: %s: %zu values of 'decay' for %d heads", m.where.c_str(), d->arr.size(), out->heads);
     for (const JValue& v : d->arr) {
         LC_CHECK(v.kind == JValue::NUM && v.num >= 0.0 && v.num <= 1.0, LC_ERR_INVALID, "config: %s: 'decay' is not in 0 .. 1", m.where.c_str());
-        out->log_decay.push_back((float)std::fmax(std::log(v.num), -1e4));  // far below where exp ends, and still a number
+        out->decay.push_back(v.num);
     }
     return LC_OK;
 }

@@ -441,6 +441,7 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
             xs[c][r] = (t0 + r < T && kk < k) ? x[(size_t)x_row[r] * ldx + kk] : 0.0f;
         }
         __syncthreads();
+        float part[4][4] = {};  // sums of a tile of k join the others as one: the rounding grows with the tiles, not with k
 #pragma unroll
         for (int c = 0; c < KT; c++) {
             float a[4], q[4];
@@ -449,8 +450,12 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
 #pragma unroll
             for (int i = 0; i < 4; i++)
 #pragma unroll
-                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(q[i], a[j], acc[i][j]);
+                for (int j = 0; j < 4; j++) part[i][j] = fmaf(q[i], a[j], part[i][j]);
         }
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) acc[i][j] += part[i][j];
         __syncthreads();
     }
 #pragma unroll

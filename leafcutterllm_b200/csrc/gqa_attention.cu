@@ -410,12 +410,12 @@ __global__ void __launch_bounds__(kPlainThreads) attn_plain_kernel(const AttnArg
         m = mt;
         const int nk = min(kPlainThreads, n - k0);
         for (int c = threadIdx.x; c < g.vdim; c += kPlainThreads) {
-            float o = s_o[c] * corr;
+            float o = 0.0f;
             for (int j = 0; j < nk; j++) {
                 const int at = k0 + j, key = at < sn.keep ? at : sn.lo + at - sn.keep;
                 o = fmaf(s_p[j], act_f<A>(((const A*)a.v_cache)[s_row[j] * g.v_pitch + cell_of(c, key, g.v_swz)]), o);
             }
-            s_o[c] = o;
+            s_o[c] = fmaf(s_o[c], corr, o);
         }
         __syncthreads();
     }

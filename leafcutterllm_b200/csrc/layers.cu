@@ -360,11 +360,18 @@ int32_t bind_pair(lc_model* m, StackLayer& L, const std::string& p) {
         LC_TRY(model_gain_f32(m, pr + "D", sb.heads, &b.skip));
         LC_TRY(changed_gain(m, pr + "A_log", sb.heads, [](float v) { return std::exp(v); }, &b.a_exp));
     } else {
+        std::vector<float> table((size_t)sb.heads * 3);  // factors, then their logarithms
+        for (int h = 0; h < sb.heads; h++) {
+            table[2 * h] = (float)sb.decay[h];
+            table[2 * h + 1] = (float)(sb.decay[h] - (double)table[2 * h]);
+            table[2 * sb.heads + h] = (float)std::fmax(std::log(sb.decay[h]), -1e4);  // far below where exp ends, and still a number
+        }
         void* dec = nullptr;
-        LC_TRY(zalloc(st, &dec, (size_t)sb.heads * 4));
-        LC_CUDA(cudaMemcpyAsync(dec, sb.log_decay.data(), (size_t)sb.heads * 4, cudaMemcpyHostToDevice, m->stream));
+        LC_TRY(zalloc(st, &dec, table.size() * 4));
+        LC_CUDA(cudaMemcpyAsync(dec, table.data(), table.size() * 4, cudaMemcpyHostToDevice, m->stream));
         LC_CUDA(cudaStreamSynchronize(m->stream));
-        b.log_decay = (const float*)dec;
+        b.decay = (const float2*)dec;
+        b.log_decay = (const float*)dec + 2 * sb.heads;
     }
     // outputs
     L.mixed_off = sa.heads * a.ep;
@@ -565,7 +572,7 @@ int32_t attention_block(lc_model* m, MixerUnit& L, const void* x, int ldx, int T
 
 int32_t recur(lc_model* m, const MixerUnit& L, LinearArgs a, int T, bool decode_step) {
     LayerStack& st = *m->stack;
-    a.g = L.ng; a.proj = st.proj; a.dt = st.projf; a.conv = L.conv; a.conv_b = L.conv_b; a.dt_bias = L.dt_bias; a.a_exp = L.a_exp; a.skip = L.skip; a.log_decay = L.log_decay;
+    a.g = L.ng; a.proj = st.proj; a.dt = st.projf; a.conv = L.conv; a.conv_b = L.conv_b; a.dt_bias = L.dt_bias; a.a_exp = L.a_exp; a.skip = L.skip; a.log_decay = L.log_decay; a.decay = L.decay;
     a.ring = L.ring; a.in = st.lin; a.state = L.state; a.tok_seq = m->d_tok_seq; a.tok_pos = m->d_tok_pos; a.T = T; a.o = st.o; a.norm_w = L.o_norm; a.f32 = st.f32;
     int launches = 1;
     if (decode_step) {

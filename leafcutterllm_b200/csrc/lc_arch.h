@@ -74,7 +74,7 @@ struct MixerSpec {
     // LinearState
     LinearKind linear = LinearKind::Constant;
     int norm_parts = 1;
-    std::vector<float> log_decay;                 // Constant: per head
+    std::vector<double> decay;                    // Constant: per head
 };
 
 // Two mixers over one input.  Scaled: scale[0] left + scale[1] right.  Normed: half the sum of the two, each through an RMS norm.

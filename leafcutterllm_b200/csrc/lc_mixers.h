@@ -296,6 +296,7 @@ struct LinearArgs {
     const float* dt = nullptr;         // [T][ld_dt] 32-bit part of the projection
     const float *conv = nullptr, *conv_b = nullptr, *dt_bias = nullptr, *a_exp = nullptr, *skip = nullptr;  // StateSpace; a_exp = e^A_log
     const float* log_decay = nullptr;  // Constant: [heads]
+    const float2* decay = nullptr;     // Constant: [heads] the factors as sums of two floats: one float's rounding would add up over thousands of tokens
     void* ring = nullptr;              // [slot][taps][channels] activations
     void* in = nullptr;                // StateSpace: [T][ld_in] v | k | q behind convolution and silu
     float* state = nullptr;            // [slot][heads][dim][vdim]
@@ -363,6 +364,7 @@ struct MixerUnit {
     // LinearState
     LinearShape ng{};
     const float *conv_b = nullptr, *skip = nullptr, *log_decay = nullptr;
+    const float2* decay = nullptr;
 };
 struct StackLayer {
     LayerSpec s;

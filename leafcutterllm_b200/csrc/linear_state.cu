@@ -34,6 +34,9 @@ __device__ __forceinline__ float2 step_decay(const LinearArgs& a, size_t t, int 
     const float b = softplus_of(a.dt[t * a.g.ld_dt + a.g.off_dt + h] + a.dt_bias[h]);
     return make_float2(b, -a.a_exp[h] * b);
 }
+// e^l as a sum of two floats
+__device__ __forceinline__ float2 decay_of(const LinearArgs& a, int h, float l) { return a.g.kind == LinearKind::Constant ? a.decay[h] : make_float2(expf(l), 0.0f); }
+__device__ __forceinline__ float decayed(float s, float2 d) { return fmaf(s, d.x, s * d.y); }
 // Rows of v | k | q that the recurrence reads.
 template <typename A> struct Rows { const A* p; int ld, v, k, q; };
 template <typename A>
@@ -166,7 +169,8 @@ template <typename A, int DPL>
 __global__ void __launch_bounds__(128) linear_scan_kernel(const LinearArgs a) {
     constexpr int DP = DPL * 4;
     extern __shared__ __align__(16) float sm[];
-    float *s_q = sm, *s_k = s_q + kScanTok * DP, *s_v = s_k + kScanTok * DP, *s_b = s_v + kScanTok * 32, *s_g = s_b + kScanTok;
+    float *s_q = sm, *s_k = s_q + kScanTok * DP, *s_v = s_k + kScanTok * DP, *s_b = s_v + kScanTok * 32;
+    float2* s_g = (float2*)(s_b + kScanTok);
     pdl_launch_dependents();
     pdl_wait();
     const LinearShape& g = a.g;
@@ -198,12 +202,13 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(const LinearArgs a) {
         if (threadIdx.x < m) {
             const float2 bl = step_decay(a, (size_t)(run.tok0 + c0 + threadIdx.x), h);
             s_b[threadIdx.x] = bl.x;
-            s_g[threadIdx.x] = expf(bl.y);
+            s_g[threadIdx.x] = decay_of(a, h, bl.y);
         }
         __syncthreads();
         for (int t = 0; t < m; t++) {
             const float4 *q4 = (const float4*)(s_q + t * DP), *k4 = (const float4*)(s_k + t * DP);
-            const float v = s_v[t * 32 + col], u = s_b[t] * v, decay = s_g[t];
+            const float v = s_v[t * 32 + col], u = s_b[t] * v;
+            const float2 decay = s_g[t];
             float o = 0.0f;
 #pragma unroll
             for (int i = 0; i < DPL / 4; i++) {
@@ -211,7 +216,7 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(const LinearArgs a) {
                 const float kk[4] = {kv.x, kv.y, kv.z, kv.w}, qq[4] = {qv.x, qv.y, qv.z, qv.w};
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
-                    S[4 * i + j] = fmaf(kk[j], u, S[4 * i + j] * decay);
+                    S[4 * i + j] = fmaf(kk[j], u, decayed(S[4 * i + j], decay));
                     o = fmaf(S[4 * i + j], qq[j], o);
                 }
             }
@@ -501,7 +506,7 @@ __global__ void __launch_bounds__(kStepThreads) linear_step_kernel(const LinearA
         }
         sm[i] = y;
     }
-    const float decay = expf(bl.y);
+    const float2 decay = decay_of(a, h, bl.y);
     __syncthreads();
     if (mine) {
         float u[VEC], o[VEC];
@@ -510,7 +515,7 @@ __global__ void __launch_bounds__(kStepThreads) linear_step_kernel(const LinearA
         auto turn = [&](int d, float (&v)[VEC]) {
             const float k = s_k[d], q = s_q[d];
 #pragma unroll
-            for (int j = 0; j < VEC; j++) { v[j] = fmaf(k, u[j], v[j] * decay); o[j] = fmaf(v[j], q, o[j]); }
+            for (int j = 0; j < VEC; j++) { v[j] = fmaf(k, u[j], decayed(v[j], decay)); o[j] = fmaf(v[j], q, o[j]); }
             if constexpr (VEC == 4) *(float4*)(st + (size_t)d * g.vdim) = make_float4(v[0], v[1], v[2], v[3]);
             else st[(size_t)d * g.vdim] = v[0];
         };
@@ -633,7 +638,7 @@ __global__ void __launch_bounds__(kRingThreads, 1) linear_ring_kernel(const Line
         float2 bl_next = bl;
         int pos_next = pos;
         fetch(j + 1, bl_next, pos_next);
-        const float decay = pos > 0 ? expf(bl.y) : 0.0f;
+        const float2 decay = pos > 0 ? decay_of(a, h, bl.y) : make_float2(0.0f, 0.0f);
         if (ok && !mbar_wait(&s_full[st], (uint32_t)(j / rs.stages) & 1)) { ok = false; atomicExch(error_flag, 17); }  // every thread goes on to the barriers
         float* S = (float*)(ring_smem + (size_t)st * rs.stage_bytes);
         const A *q = (const A*)(S + state_elems), *k = q + g.dim, *v = k + g.dim;
@@ -647,7 +652,8 @@ __global__ void __launch_bounds__(kRingThreads, 1) linear_ring_kernel(const Line
                 float4 x = *at;
                 if (pos == 0) x = make_float4(0.f, 0.f, 0.f, 0.f);
                 const float kk = act_f<A>(k[d]), qq = act_f<A>(q[d]);
-                x.x = fmaf(kk, u.x, x.x * decay); x.y = fmaf(kk, u.y, x.y * decay); x.z = fmaf(kk, u.z, x.z * decay); x.w = fmaf(kk, u.w, x.w * decay);
+                x.x = fmaf(kk, u.x, decayed(x.x, decay)); x.y = fmaf(kk, u.y, decayed(x.y, decay));
+                x.z = fmaf(kk, u.z, decayed(x.z, decay)); x.w = fmaf(kk, u.w, decayed(x.w, decay));
                 o.x = fmaf(x.x, qq, o.x); o.y = fmaf(x.y, qq, o.y); o.z = fmaf(x.z, qq, o.z); o.w = fmaf(x.w, qq, o.w);
                 *at = x;
             }
@@ -769,7 +775,7 @@ template <typename A>
 int32_t scan_dispatch(const LinearArgs& a, cudaStream_t s) {
     const dim3 grid((unsigned)a.n_runs, (unsigned)a.g.heads, (unsigned)((a.g.vdim + 31) / 32));
     const int dp = padded_dim(a.g.dim);
-    const size_t smem = (size_t)kScanTok * (2 * dp + 32 + 2) * sizeof(float);
+    const size_t smem = (size_t)kScanTok * (2 * dp + 32 + 3) * sizeof(float);
     auto go = [&](auto kern) -> int32_t {
         LC_CUDA(ensure_smem_limit((const void*)kern, smem));
         LC_CUDA(launch_pdl(kern, grid, dim3(128), smem, s, a));
