@@ -303,6 +303,8 @@ int32_t bind_pair(lc_model* m, StackLayer& L, const std::string& p) {
     const std::string pl = p + "left.", pr = p + "right.";
     const int W = st.spec.width, nq = sa.heads * sa.dim, nk = sa.kv_heads * sa.dim, nv = sa.kv_heads * sa.vdim, inner = sb.heads * sb.vdim;
     const bool space = sb.linear == LinearKind::StateSpace;
+    LC_CHECK(sb.dim <= 256 && std::max(sa.dim, sa.vdim) <= 512, LC_ERR_UNSUPPORTED, "%s: %d state dimensions (at most 256), heads of %d and %d dimensions (at most 512)", p.c_str(),
+             sb.dim, sa.dim, sa.vdim);
     attention_shape(st, a);
     LinearShape& g = b.ng;
     g.kind = sb.linear; g.heads = sb.heads; g.groups = sb.kv_heads; g.dim = sb.dim; g.vdim = sb.vdim; g.taps = sb.conv_taps; g.norm_parts = sb.norm_parts; g.eps = st.spec.eps;

@@ -100,6 +100,7 @@ __device__ __forceinline__ float sq4(float4 v, float ss) { return fmaf(v.x, v.x,
 __device__ __forceinline__ void add4(float4& y, float w, float4 v) { y.x = fmaf(w, v.x, y.x); y.y = fmaf(w, v.y, y.y); y.z = fmaf(w, v.z, y.z); y.w = fmaf(w, v.w, y.w); }
 
 // VEC = 4: rows of a multiple of four elements; a row of up to 16 elements per thread stays in registers between its passes.
+// MOE, PAIR: the output is first made from a mixture's parts (MoeSum) or from two mixers' outputs (PairSum).
 template <typename A, int VEC, bool MOE, bool PAIR>
 __global__ void __launch_bounds__(512) residual_kernel(const ResidualArgs a) {
     constexpr int kHeld = 4;
