@@ -471,5 +471,149 @@ class PlainMunisun:
         return linear(self.norm("final.norm", x), w["head"])
 
 
+# ---- delta rule with separate removal, attention with biases and a gate per head, token pairs, averages over depth ---------------
+def general_delta_rule(r, k, v, w, a, state, unit_eps=1e-6):
+    """One head: the state loses its part along the unit key (each key channel at its own rate a) and fades by w, both seen from the
+    state before the token; then the token is added and the result read with r.  r, k, v, w, a: [T, n]; state: [n, n], changed in place."""
+    out = np.zeros_like(v)
+    for t in range(len(v)):
+        u = unit(k[t], unit_eps)
+        held = u @ state
+        state *= w[t][:, None]
+        state -= np.outer(a[t] * u, held)
+        state += np.outer(k[t], v[t])
+        out[t] = r[t] @ state
+    return out
+
+
+def query_temperature(pos, temp):
+    """Factor on the queries at positions `pos`."""
+    return 1.0 + temp["coef"] * np.log(np.floor((np.asarray(pos) + 1) / temp["every"]) + 1.0)
+
+
+def masked_attention(q, k, v, scale, cap, seen):
+    """Softmax over the keys in `seen` [T, S]; H query heads over G key/value heads; scores bounded unless cap is None."""
+    H, G = q.shape[1], k.shape[1]
+    out = np.zeros(q.shape[:2] + (v.shape[2],))
+    for h in range(H):
+        s = q[:, h] @ k[:, h // (H // G)].T * scale
+        if cap is not None:
+            s = cap * np.tanh(s / cap)
+        s = np.where(seen, s, -np.inf)
+        e = np.exp(s - s.max(axis=1, keepdims=True))
+        out[:, h] = e / e.sum(axis=1, keepdims=True) @ v[:, h // (H // G)]
+    return out
+
+
+def rotate_half_pairs(x, pos, rot):
+    """Dimension i of the first rot.dims is paired with i + dims / 2; frequencies and magnitude of the config's scaling."""
+    f, mag = yarn_frequencies(rot)
+    half = rot["dims"] // 2
+    a = np.asarray(pos, np.float64)[:, None, None] * f
+    cos, sin = np.cos(a) * mag, np.sin(a) * mag
+    u, v = x[..., :half], x[..., half : 2 * half]
+    return np.concatenate([u * cos - v * sin, v * cos + u * sin, x[..., 2 * half :]], axis=-1)
+
+
+def pair_rows(tokens, before, bigram):
+    """Row of the pair table for every token; `before`: the token ahead of the first one, None at the start of a sequence."""
+    rows, prev = [], before
+    for t in tokens:
+        rows.append(bigram["buckets"] if prev is None else (int(prev) * bigram["mul_prev"] + int(t) * bigram["mul_cur"]) % bigram["buckets"])
+        prev = t
+    return rows
+
+
+def gated_gelu(x, gate, up, down):
+    return linear(gelu_tanh(linear(x, gate)) * linear(x, up), down)
+
+
+class PlainNepudra:
+    """Norms (one number each) on the sublayers' inputs; behind every layer a weighted sum of the embedding and all layers' results."""
+
+    def __init__(self, config, w):
+        self.c = config
+        self.w = {n: np.asarray(a, np.float64) for n, a in w.items()}
+        self.eps = config["norm"]["eps"]
+
+    def new_state(self):
+        return {"pos": 0, "last": None, "layers": [dict() for _ in self.c["layers"]]}
+
+    def norm(self, name, x):
+        return rms_norm(x, self.eps) * self.w[name].reshape(())
+
+    def general_delta(self, i, x, st):
+        m, p, w, T = self.c["layers"][i]["mixer"], "l%d.mix." % i, self.w, len(x)
+        H, D = m["heads"], m["dim"]
+        heads = lambda z: z.reshape(T, H, D)
+        r, k, v = (heads(linear(x, w[p + n])) for n in "rkv")
+        decay = heads(np.exp(-np.exp(-0.5) * sigmoid(linear(np.tanh(linear(x, w[p + "w1"])), w[p + "w2"]) + w[p + "w0"])))
+        a = heads(sigmoid(linear(x, w[p + "a"]) + w[p + "a.b"]))
+        if not st:
+            st["S"] = np.zeros((H, D, D))
+        o = np.stack([general_delta_rule(r[:, h], k[:, h], v[:, h], decay[:, h], a[:, h], st["S"][h]) for h in range(H)], axis=1)
+        o = rms_norm(o, self.eps).reshape(T, H * D) * w[p + "norm"]
+        return linear(o * sigmoid(linear(x, w[p + "g"])), w[p + "o"])
+
+    def attention(self, i, x, layers, first):
+        """Both kinds: `layers` holds all layers' states."""
+        ly = self.c["layers"][i]
+        m, p, w, T = ly["mixer"], "l%d.mix." % i, self.w, len(x)
+        H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        pos = first + np.arange(T)
+        second = ly["type"] == "attention_2"
+
+        def placed(z, n):
+            if second:
+                z = rms_norm(z, self.eps, w[p + n + ".norm"])
+            return rotate_half_pairs(z, pos, m["rot"]) if "rot" in m else z
+
+        q = placed((linear(x, w[p + "q"]) + w[p + "q.b"]).reshape(T, H, D), "q")
+        if "q_temp" in m:
+            q = q * query_temperature(pos, m["q_temp"])[:, None, None]
+        src = m.get("kv_from")
+        st = layers[i if src is None else src]
+        if src is None:
+            k = placed((linear(x, w[p + "k"]) + w[p + "k.b"]).reshape(T, G, D), "k")
+            v = (linear(x, w[p + "v"]) + w[p + "v.b"]).reshape(T, G, E)
+            st["k"] = np.concatenate([st["k"], k]) if "k" in st else k
+            st["v"] = np.concatenate([st["v"], v]) if "v" in st else v
+        size = m["mask"]["size"] if "mask" in m else first + T
+        o = masked_attention(q, st["k"], st["v"], m["scale"], m.get("softcap"), visible(pos, len(st["k"]), size, 0))
+        o = o * sigmoid(linear(x, w[p + "g"]))[:, :, None]
+        y = linear(o.reshape(T, H * E), w[p + "o"])
+        return y if second else y + w[p + "o.b"]
+
+    def mix(self, i, x, layers, first):
+        if self.c["layers"][i]["type"] == "general_delta":
+            return self.general_delta(i, x, layers[i])
+        return self.attention(i, x, layers, first)
+
+    def feed_forward(self, i, x):
+        p, w = "l%d.mlp." % i, self.w
+        return gated_gelu(x, w[p + "gate"], w[p + "up"], w[p + "down"])
+
+    def embed(self, tokens, state):
+        x = self.w["embed"][np.asarray(tokens)] + self.w["bigram"][pair_rows(tokens, state["last"], self.c["embedding"]["bigram"])]
+        state["last"] = tokens[-1]
+        return x
+
+    def forward(self, tokens, state, trace=None):
+        first = state["pos"]
+        x = self.embed(tokens, state)
+        depth = [x]
+        for i, ly in enumerate(self.c["layers"]):
+            l = "l%d." % i
+            x = x + self.mix(i, self.norm(l + "norm1", x), state["layers"], first)
+            if ly["mlp"] is not None:
+                x = x + self.feed_forward(i, self.norm(l + "norm2", x))
+            depth.append(x)
+            x = sum(c * y for c, y in zip(self.w[l + "dwa"], depth))
+            if trace is not None:
+                trace.append(x.copy())
+        state["pos"] = first + len(tokens)
+        return linear(self.norm("final.norm", x), self.w["head"])
+
+
 def plain_model(config, w):
-    return {"Varasun": PlainModel, "Tenetar": PlainTenetar, "Munisun": PlainMunisun}[config["architecture"]](config, w)
+    return {"Varasun": PlainModel, "Tenetar": PlainTenetar, "Munisun": PlainMunisun, "Nepudra": PlainNepudra}[config["architecture"]](config, w)
