@@ -11,7 +11,7 @@
 namespace lc {
 
 const char* mixer_name(MixerKind k) {
-    return k == MixerKind::ChannelDelta ? "channel_delta" : k == MixerKind::LatentAttention ? "latent_attention" : k == MixerKind::Attention ? "attention" : "linear_state";
+    return k == MixerKind::ChannelDelta ? "channel_delta" : k == MixerKind::LatentAttention ? "latent_attention" : k == MixerKind::Attention ? "attention" : k == MixerKind::GeneralDelta ? "general_delta" : "linear_state";
 }
 
 void rotary_frequencies(const RotarySpec& r, std::vector<double>* freq, double* magnitude) {
@@ -212,9 +212,44 @@ int32_t parse_parallel(const Fields& m, const std::string& type, int index, Laye
     return parse_lightning(right, &out->mix[1]);
 }
 
-// What the designs do not share: the types of layers, the kind of feed-forward that "dense" means, how routers work.
+// One mixer per layer, by its parser.
+template <int32_t (*PARSE)(const Fields&, MixerSpec*)>
+int32_t single(const Fields& m, const std::string&, int, LayerSpec* out) { return PARSE(m, &out->mix[0]); }
+
+int32_t parse_sunk_attention(const Fields& m, const std::string&, int index, LayerSpec* out) { return parse_attention(m, index, RotaryScaling::Yarn, &out->mix[0]); }
+
+// Attention with biases and a gate per head; the first kind bounds its scores and warms its queries, the second has norms per head.
+int32_t parse_head_gated(const Fields& m, const std::string& type, int index, LayerSpec* out) {
+    MixerSpec& a = out->mix[0];
+    LC_TRY(parse_attention(m, index, RotaryScaling::Yarn, &a));
+    const bool second = type == "attention_2";
+    a.qk_norm = second ? QkNorm::PerHead : QkNorm::None;
+    a.head_gate = a.qkv_bias = true;
+    a.out_bias = !second;
+    if (m.has("q_temp")) {
+        Fields t;
+        LC_TRY(m.child("q_temp", &t));
+        LC_TRY(t.real("coef", &a.q_temp.coef));
+        LC_TRY(t.real("every", &a.q_temp.every));
+        LC_CHECK(a.q_temp.every > 0.0, LC_ERR_INVALID, "config: %s: 'every' = %g", t.where.c_str(), a.q_temp.every);
+    }
+    return LC_OK;
+}
+
+int32_t parse_general_delta(const Fields& m, MixerSpec* out) {
+    out->kind = MixerKind::GeneralDelta;
+    LC_TRY(m.integer("heads", &out->heads, 1));
+    LC_TRY(m.integer("dim", &out->dim, 1));
+    out->kv_heads = out->heads;
+    out->vdim = out->dim;
+    out->decay_scale = std::exp(-0.5);
+    return LC_OK;
+}
+
+// What the designs do not share: the types of layers and what they hold, the kind of feed-forward that "dense" means, how routers work.
+struct LayerType { const char* name; int32_t (*parse)(const Fields& mixer, const std::string& type, int index, LayerSpec* out); };
 struct Rules {
-    std::initializer_list<const char*> types;
+    std::initializer_list<LayerType> types;
     FfnKind dense;
     bool mixtures = false;
     MoeSpec moe;
@@ -253,13 +288,11 @@ int32_t parse_layer(const JValue& v, int index, const Rules& rules, LayerSpec* o
     const JValue *type = f.need("type", JValue::STR), *mixer = f.need("mixer", JValue::OBJ);
     if (!type || !mixer) return LC_ERR_INVALID;
     const Fields m{mixer, f.where + ".mixer"};
-    bool known = false;
-    for (const char* t : rules.types) known = known || type->str == t;
+    const LayerType* known = nullptr;
+    for (const LayerType& t : rules.types)
+        if (type->str == t.name) known = &t;
     LC_CHECK(known, LC_ERR_UNSUPPORTED, "config: %s: unknown mixer type '%s'", f.where.c_str(), type->str.c_str());
-    if (type->str == mixer_name(MixerKind::ChannelDelta)) LC_TRY(parse_delta(m, &out->mix[0]));
-    else if (type->str == mixer_name(MixerKind::LatentAttention)) LC_TRY(parse_latent(m, &out->mix[0]));
-    else if (type->str == mixer_name(MixerKind::Attention)) LC_TRY(parse_attention(m, index, RotaryScaling::Yarn, &out->mix[0]));
-    else LC_TRY(parse_parallel(m, type->str, index, out));
+    LC_TRY(known->parse(m, type->str, index, out));
     if (f.has("mlp")) {
         Fields p;
         LC_TRY(f.child("mlp", &p));
@@ -308,7 +341,7 @@ int32_t parse_varasun(const JValue& cfg, ArchSpec* out) {
     Fields f{&cfg, "the model"};
     LC_TRY(f.real("logit_scale", &out->logit_scale));
     LC_TRY(f.real("logit_softcap", &out->logit_softcap));
-    return parse_stack(f, Rules{{"channel_delta", "latent_attention"}, FfnKind::Relu2}, out);
+    return parse_stack(f, Rules{{{"channel_delta", single<parse_delta>}, {"latent_attention", single<parse_latent>}}, FfnKind::Relu2}, out);
 }
 
 // Tenetar: windowed attention layers, some of which read an earlier layer's keys and values, with gated or mixture
@@ -318,7 +351,7 @@ int32_t parse_tenetar(const JValue& cfg, ArchSpec* out) {
     LC_TRY(f.child("embedding", &e));
     LC_TRY(e.real("scale", &out->embed_scale));
     out->norm_inputs = true;
-    return parse_stack(f, Rules{{"attention"}, FfnKind::GatedSilu, true}, out);
+    return parse_stack(f, Rules{{{"attention", parse_sunk_attention}}, FfnKind::GatedSilu, true}, out);
 }
 
 // Munisun: attention and a linear recurrence side by side in every layer, gated or mixture feed-forwards, norms (stored around
@@ -330,15 +363,33 @@ int32_t parse_munisun(const JValue& cfg, ArchSpec* out) {
     LC_TRY(f.child("token_side", &side));
     LC_TRY(side.integer("dim", &out->side_dim, 1));
     out->norm_inputs = out->norm_one_plus = true;
-    Rules r{{"parallel", "parallel_2"}, FfnKind::GatedSilu, true};
+    Rules r{{{"parallel", parse_parallel}, {"parallel_2", parse_parallel}}, FfnKind::GatedSilu, true};
     r.moe.score = RouterScore::Sigmoid;
     r.moe.group_top = 2;
     r.moe.gated = true;
     return parse_stack(f, r, out);
 }
 
+// Nepudra: attention of two kinds and a delta rule with separate removal, norms on the sublayers' inputs, an embedding per pair of
+// tokens, averages over depth.
+int32_t parse_nepudra(const JValue& cfg, ArchSpec* out) {
+    Fields f{&cfg, "the model"}, e, b;
+    LC_TRY(f.child("embedding", &e));
+    LC_TRY(e.child("bigram", &b));
+    int buckets = 0;
+    double mul[2];
+    LC_TRY(b.integer("buckets", &buckets, 1));
+    LC_TRY(b.real("mul_prev", &mul[0]));
+    LC_TRY(b.real("mul_cur", &mul[1]));
+    for (double v : mul) LC_CHECK(v == std::floor(v) && v >= 0.0 && v < 9007199254740992.0, LC_ERR_INVALID, "config: %s: a factor of %g", b.where.c_str(), v);
+    out->bigram = BigramSpec{buckets, (int64_t)mul[0] % buckets, (int64_t)mul[1] % buckets};
+    out->norm_inputs = out->norm_scalar = out->depth_average = true;
+    out->norm_outputs = false;
+    return parse_stack(f, Rules{{{"attention", parse_head_gated}, {"attention_2", parse_head_gated}, {"general_delta", single<parse_general_delta>}}, FfnKind::GatedGelu}, out);
+}
+
 struct ArchEntry { const char* name; int32_t (*parse)(const JValue&, ArchSpec*); };
-const ArchEntry kRegistry[] = {{"Varasun", parse_varasun}, {"Tenetar", parse_tenetar}, {"Munisun", parse_munisun}};
+const ArchEntry kRegistry[] = {{"Varasun", parse_varasun}, {"Tenetar", parse_tenetar}, {"Munisun", parse_munisun}, {"Nepudra", parse_nepudra}};
 
 uint32_t safetensors_type(const std::string& dtype) {
     if (dtype == "BF16") return LC_TYPE_BF16;

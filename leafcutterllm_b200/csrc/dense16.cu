@@ -45,7 +45,7 @@ struct DenseParams {
     int out_f32, epi, e_div;
     float scale, cap;
     void* out2;
-    int ldo2, split, silu_end;
+    int ldo2, split, act_end;
     const __nv_bfloat16* table;
     const int64_t* ids;
     int table_ld, table_rows;
@@ -58,11 +58,13 @@ struct DenseParams {
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // The epilogue is a template parameter of the kernels; kEpiAny stands for the rarer elementwise ones, told apart at run time.
 constexpr int kEpiAny = -1;
-constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS ? kEpiAny : epi; }
-constexpr bool epi_splits(int epi) { return epi == DENSE_SPLIT_RELU2 || epi == DENSE_SPLIT_SILU; }
+constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS || epi == DENSE_SIGMOID_DECAY ? kEpiAny : epi; }
+constexpr bool epi_splits(int epi) { return epi == DENSE_SPLIT_RELU2 || epi == DENSE_SPLIT_SILU || epi == DENSE_SPLIT_TANH; }
+constexpr bool epi_gated(int epi) { return epi == DENSE_GATED_SILU || epi == DENSE_GATED_GELU; }
 __device__ __forceinline__ float silu_of(float g) { return g / (1.0f + expf(-g)); }
 // z (1 + tanh u) / 2 = z / (1 + e^(-2u)), u = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_of(float z) { return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))); }
+template <int EPI> __device__ __forceinline__ float gate_of(float g) { return EPI == DENSE_GATED_GELU ? gelu_of(g) : silu_of(g); }
 // Element `row` of token t's row in the table, 0 for ids outside it.  The loads do not depend on a branch, so those of many tokens
 // travel together; rows and tokens outside the product read a valid place.
 __device__ __forceinline__ float table_factor(const DenseParams& p, int row, int t) {
@@ -77,9 +79,12 @@ __device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool secon
     const float r = fmaxf(y, 0.0f);
     if constexpr (EPI == DENSE_RELU2) return r * r;
     else if constexpr (EPI == DENSE_SPLIT_RELU2) return second ? r * r : y;
-    else if constexpr (EPI == DENSE_SPLIT_SILU) return second && row < p.silu_end ? silu_of(y) : y;
+    else if constexpr (EPI == DENSE_SPLIT_SILU) return second && row < p.act_end ? silu_of(y) : y;
+    else if constexpr (EPI == DENSE_SPLIT_TANH) return second && row < p.act_end ? tanhf(y) : y;
+    else if constexpr (EPI == DENSE_BIAS) return y + eb;
     else if constexpr (EPI == kEpiAny) {
         if (p.epi == DENSE_LOG_DECAY) return -ea * softplus_f(y + eb);
+        if (p.epi == DENSE_SIGMOID_DECAY) return -p.scale / (1.0f + expf(-(y + eb)));
         const float v = y * p.scale;
         return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v;
     } else return y;
@@ -87,18 +92,19 @@ __device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool secon
 __device__ __forceinline__ void dense_row_constants(const DenseParams& p, int row, float& ea, float& eb) {
     ea = eb = 0.0f;
     if (p.epi == DENSE_LOG_DECAY && row < p.n) { ea = p.e0[row / p.e_div]; eb = p.e1[row]; }
+    if ((p.epi == DENSE_BIAS || p.epi == DENSE_SIGMOID_DECAY) && row < p.n) eb = p.e1[row];
 }
 // 16 accumulators of weight row `row`, tokens t0 .. t0 + m - 1 (m may exceed 16), for a whole warp (lane = row).  bf16: lane
 // pairs swap halves, so a lane stores two rows of every other token.
 template <int EPI>
 __device__ __forceinline__ void dense_store16(const DenseParams& p, int b, int row, int t0, int m, const float (&v)[16], float ea, float eb) {
-    if constexpr (EPI == DENSE_GATED_SILU) {  // even lanes hold gates, odd ones the matching values; each makes every other token's output
+    if constexpr (epi_gated(EPI)) {  // even lanes hold gates, odd ones the matching values; each makes every other token's output
         const bool odd = row & 1;
         const size_t at = (size_t)b * p.out_batch + (size_t)t0 * p.ldo + (row >> 1);
 #pragma unroll
         for (int j = 0; j < 16; j += 2) {
             const float other = __shfl_xor_sync(0xffffffffu, odd ? v[j] : v[j + 1], 1);
-            const float y = odd ? silu_of(other) * v[j + 1] : silu_of(v[j]) * other;
+            const float y = odd ? gate_of<EPI>(other) * v[j + 1] : gate_of<EPI>(v[j]) * other;
             const int jj = j + (odd ? 1 : 0);
             if (jj >= m || row >= p.n) continue;
             if (p.out_f32) ((float*)p.out)[at + (size_t)jj * p.ldo] = y;
@@ -464,9 +470,9 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(const __nv_bfloat16* __r
 #pragma unroll
         for (int j = 0; j < 4; j++) {
             const int row = r0 + tr + 16 * j;
-            if constexpr (EPI == DENSE_GATED_SILU) {
+            if constexpr (epi_gated(EPI)) {
                 const float up = __shfl_xor_sync(0xffffffffu, acc[i][j], 1);
-                if (t < T && row < p.n && (row & 1) == 0) ((float*)p.out)[(size_t)(row0 + t) * p.ldo + (row >> 1)] = silu_of(acc[i][j]) * up;
+                if (t < T && row < p.n && (row & 1) == 0) ((float*)p.out)[(size_t)(row0 + t) * p.ldo + (row >> 1)] = gate_of<EPI>(acc[i][j]) * up;
                 continue;
             }
             if (t >= T || row >= p.n) continue;
@@ -601,10 +607,10 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
     p.n = w.n; p.T = a.T; p.ldo = a.ldo; p.batch = w.batch;
     p.out_f32 = a.out_f32 || a.f32; p.epi = a.epi; p.e_div = a.e_div; p.scale = a.scale; p.cap = a.cap;
     p.error_flag = gemv_error_flag_dev();
-    p.out2 = a.out2; p.ldo2 = a.ldo2; p.split = a.split; p.silu_end = a.silu_end;
+    p.out2 = a.out2; p.ldo2 = a.ldo2; p.split = a.split; p.act_end = a.act_end;
     p.table = a.table; p.table_ld = a.table_ld; p.table_rows = a.table_rows; p.ids = a.ids;
     if (a.plan) { p.tiles = a.plan->tiles; p.n_tiles = a.plan->n_tiles; p.off = a.plan->off; p.lists = a.gather ? a.plan->lists : nullptr; p.list_stride = a.plan->list_stride; }
-    LC_CHECK((a.epi != DENSE_GATED_SILU || w.n % 2 == 0) && (!epi_splits(a.epi) || (a.split % 32 == 0 && w.batch == 1)), LC_ERR_INVALID, "dense product: epilogue layout");
+    LC_CHECK((!epi_gated(a.epi) || w.n % 2 == 0) && (!epi_splits(a.epi) || (a.split % 32 == 0 && w.batch == 1)), LC_ERR_INVALID, "dense product: epilogue layout");
     LC_CHECK(a.f32 ? w.data != nullptr : w.tiles != nullptr, LC_ERR_STATE, "dense product: the weight is not in the form this product reads");
     if (a.f32) {
         const dim3 grid((unsigned)((w.n + 63) / 64), (unsigned)((a.T + 63) / 64), (unsigned)w.batch);
@@ -619,6 +625,9 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
             case DENSE_SPLIT_RELU2: return go(dense_f32_kernel<DENSE_SPLIT_RELU2>);
             case DENSE_SPLIT_SILU: return go(dense_f32_kernel<DENSE_SPLIT_SILU>);
             case DENSE_GELU_TABLE: return go(dense_f32_kernel<DENSE_GELU_TABLE>);
+            case DENSE_GATED_GELU: return go(dense_f32_kernel<DENSE_GATED_GELU>);
+            case DENSE_BIAS: return go(dense_f32_kernel<DENSE_BIAS>);
+            case DENSE_SPLIT_TANH: return go(dense_f32_kernel<DENSE_SPLIT_TANH>);
             default: return go(dense_f32_kernel<kEpiAny>);
         }
     }
@@ -655,6 +664,9 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
         case DENSE_SPLIT_RELU2: return launch_tiles<false, DENSE_SPLIT_RELU2>(NT, a, *tx, p, s);
         case DENSE_SPLIT_SILU: return launch_tiles<false, DENSE_SPLIT_SILU>(NT, a, *tx, p, s);
         case DENSE_GELU_TABLE: return launch_tiles<false, DENSE_GELU_TABLE>(NT, a, *tx, p, s);
+        case DENSE_GATED_GELU: return launch_tiles<false, DENSE_GATED_GELU>(NT, a, *tx, p, s);
+        case DENSE_BIAS: return launch_tiles<false, DENSE_BIAS>(NT, a, *tx, p, s);
+        case DENSE_SPLIT_TANH: return launch_tiles<false, DENSE_SPLIT_TANH>(NT, a, *tx, p, s);
         default: return launch_tiles<false, kEpiAny>(NT, a, *tx, p, s);
     }
 }

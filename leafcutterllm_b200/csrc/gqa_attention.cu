@@ -1,7 +1,8 @@
 // Attention of query heads over shared key/value heads in a paged cache, under a window with kept first tokens (MaskSpec) and
 // with a sink: exp(sink[head]) joins the softmax denominator, without key or value.  Scores may be bounded by a tanh, outputs gated.
 //   attn_prep_kernel    RMS norm over all of a token's q and over all of its k, rotation of halves, cache append
-//   attn_head_prep_kernel  the same for norms per head: short convolutions, norm ahead of the rotation or behind it, either pairing
+//   attn_head_prep_kernel  the same for norms per head or none: short convolutions, norm ahead of the rotation or behind it, either
+//                       pairing, a factor per position on the queries
 //   attn_plain_kernel   any shape, f32 arithmetic throughout; models in true 32-bit
 //   attn_tokens_kernel  few tokens per sequence (decode): the query heads of one kv head of one token are the rows of the
 //                       products; every warp walks key tiles of its own
@@ -49,6 +50,8 @@ __device__ __forceinline__ Tiles tiles_of(const Seen& s, int last, int size) {
 // A score in log2 units, bounded: k.x * tanh(dot * scale / cap) with k = (cap, 2 scale / cap) times log2 e.
 __device__ __forceinline__ float2 cap_constants(const AttnShape& g) { return make_float2(g.cap * kLog2e, g.cap > 0.0f ? 2.0f * g.scale / g.cap * kLog2e : 0.0f); }
 __device__ __forceinline__ float capped(float dot, float2 k) { return k.x - k.x * __fdividef(2.0f, 1.0f + exp2f(dot * k.y)); }
+// The factor on all of head h of token t's output.
+__device__ __forceinline__ float head_factor(const AttnArgs& a, size_t t, int h) { return a.head_gate ? sigmoid_f(a.head_gate[t * a.ld_proj + h]) : 1.0f; }
 // The factor on element c of head h of token t's output.
 template <typename A>
 __device__ __forceinline__ float out_factor(const AttnArgs& a, size_t t, int h, int c) {
@@ -171,7 +174,7 @@ __global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head
     pdl_wait();
     const AttnShape& g = a.g;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.y * 8 + warp;
-    if (unit >= g.heads + 2 * g.kv_heads) return;
+    if (unit >= g.heads + (a.off_k >= 0 ? 2 * g.kv_heads : 0)) return;
     const bool is_q = unit < g.heads, is_v = unit >= g.heads + g.kv_heads;
     const int h = is_q ? unit : is_v ? unit - g.heads - g.kv_heads : unit - g.heads, n = is_v ? g.vdim : g.dim, half = g.rot_dims / 2;
     const int nq = g.heads * g.dim, nk = g.kv_heads * g.dim, channels = nq + nk + g.kv_heads * g.vdim;
@@ -335,6 +338,13 @@ __global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head
                         for (int e = 0; e < 4; e++) x[p][e] *= r;
                 }
             }
+            if (is_q && a.q_factor) {
+                const float f = __ldg(a.q_factor + pos);
+#pragma unroll
+                for (int p = 0; p < NQ; p++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) x[p][e] *= f;
+            }
             A* dst;
             int swz = 0;
             if (is_q) dst = (A*)a.q + ((size_t)t * g.heads + h) * g.dp;
@@ -420,7 +430,8 @@ __global__ void __launch_bounds__(kPlainThreads) attn_plain_kernel(const AttnArg
         __syncthreads();
     }
     A* out = (A*)a.out + (size_t)t * a.ldo + (size_t)h * g.ep;
-    for (int c = threadIdx.x; c < g.ep; c += kPlainThreads) out[c] = to_act<A>(c < g.vdim ? s_o[c] / l * out_factor<A>(a, t, h, c) : 0.0f);
+    const float hf = head_factor(a, t, h);
+    for (int c = threadIdx.x; c < g.ep; c += kPlainThreads) out[c] = to_act<A>(c < g.vdim ? s_o[c] / l * hf * out_factor<A>(a, t, h, c) : 0.0f);
 }
 
 // ---- few tokens per sequence ------------------------------------------------------------------------------------------------
@@ -577,7 +588,8 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
             f[w] = m == -INFINITY ? 0.0f : exp2f(s_ml[w][tid][0] - m);
             l += f[w] * s_ml[w][tid][1];
         }
-        for (int w = 0; w < kDecWarps; w++) s_scale[w][tid] = pieces == 1 ? f[w] / l : f[w];
+        const float last = pieces == 1 ? head_factor(a, t, h0 + tid) / l : 1.0f;
+        for (int w = 0; w < kDecWarps; w++) s_scale[w][tid] = f[w] * last;
         if (pieces > 1) {
             float* ml = pt_out.ml + ((((size_t)t * gridDim.y + blockIdx.y) * pieces + blockIdx.z) * 16 + tid) * 2;
             ml[0] = m; ml[1] = l;
@@ -612,7 +624,7 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
         const float* ml = pt_out.ml + ((cell * pieces + min(lane, pieces - 1)) * 16 + row) * 2;
         const float pm = lane < pieces ? __ldcg(ml) : -INFINITY, pl = lane < pieces ? __ldcg(ml + 1) : 0.0f, sk = sink_of(row), m = fmaxf(warp_max(pm), sk);
         const float f = pm == -INFINITY ? 0.0f : exp2f(pm - m), l = warp_sum(f * pl) + (a.sink ? exp2f(sk - m) : 0.0f);
-        if (lane < pieces) s_scale[lane][row] = f / l;
+        if (lane < pieces) s_scale[lane][row] = f / l * head_factor(a, t, h0 + row);
     }
     __syncthreads();
     for (int i = tid; i < nh * vec; i += 32 * kDecWarps) {
@@ -766,7 +778,7 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
         l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
         l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
         if (row >= tl.n) continue;
-        const float m = fmaxf(m_run[r], sink), f = exp2f(m_run[r] - m), inv = f / (l_run[r] * f + (a.sink ? exp2f(sink - m) : 0.0f));
+        const float m = fmaxf(m_run[r], sink), f = exp2f(m_run[r] - m), inv = f / (l_run[r] * f + (a.sink ? exp2f(sink - m) : 0.0f)) * head_factor(a, tl.tok0 + row, h);
         bf16* dst = (bf16*)a.out + (size_t)(tl.tok0 + row) * a.ldo + (size_t)h * g.ep + 2 * t4;
 #pragma unroll
         for (int n = 0; n < NV; n++) {
@@ -802,7 +814,7 @@ template <typename A, int TAPS>
 int32_t head_prep_taps(const AttnArgs& a, cudaStream_t s) {
     const int widest = std::max(a.g.dim, a.g.vdim);
     auto go = [&](auto kern, int stretch) -> int32_t {
-        const dim3 grid((unsigned)((a.T + stretch - 1) / stretch), (unsigned)((a.g.heads + 2 * a.g.kv_heads + 7) / 8));
+        const dim3 grid((unsigned)((a.T + stretch - 1) / stretch), (unsigned)((a.g.heads + (a.off_k >= 0 ? 2 * a.g.kv_heads : 0) + 7) / 8));
         LC_CUDA(launch_pdl(kern, grid, dim3(256), 0, s, a, stretch));
         return LC_OK;
     };
@@ -815,7 +827,7 @@ int32_t head_prep_taps(const AttnArgs& a, cudaStream_t s) {
 }
 template <typename A>
 int32_t head_prep(const AttnArgs& a, cudaStream_t s) {
-    LC_CHECK(a.off_k >= 0, LC_ERR_UNSUPPORTED, "attention: norms per head over another layer's cache");
+    LC_CHECK(a.off_k >= 0 || a.g.taps == 0, LC_ERR_UNSUPPORTED, "attention: convolutions over another layer's cache");
     switch (a.g.taps) {
         case 0: return head_prep_taps<A, 0>(a, s);
         case 2: return head_prep_taps<A, 2>(a, s);
@@ -842,7 +854,7 @@ int32_t launch_attn_keep(const AttnArgs& a, const SeqRun* runs, int n_runs, cuda
 int32_t launch_attn_prep(const AttnArgs& a, cudaStream_t s) {
     const AttnShape& g = a.g;
     if (g.norm != QkNorm::AllHeads) return a.f32 ? head_prep<float>(a, s) : head_prep<bf16>(a, s);
-    LC_CHECK(g.pairs == AttnPairs::Halves && g.taps == 0, LC_ERR_UNSUPPORTED, "attention: norms over all heads with neighbouring pairs or convolutions");
+    LC_CHECK(g.pairs == AttnPairs::Halves && g.taps == 0 && !a.q_factor, LC_ERR_UNSUPPORTED, "attention: norms over all heads with neighbouring pairs, convolutions or factors on queries");
     const bool vec = g.dim % 4 == 0 && g.vdim % 4 == 0 && g.rot_dims % 8 == 0;
     // few tokens: several CTAs each, all of which sum the whole rows
     const dim3 grid((unsigned)a.T, (unsigned)(a.T < 32 ? std::max(1, std::min(8, (g.heads + g.kv_heads) * g.dim / 1024)) : 1));

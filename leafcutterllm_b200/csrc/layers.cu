@@ -4,17 +4,21 @@
 //                    vectors -> recurrence -> per-head norm and gate -> out
 //   LatentAttention  in = dq | dkv (one product)  ->  latent norms, key rotation, cache append  ->  uq -> (per head) uk^T
 //                    -> attention over the latents -> (per head) uv -> out
-//   Attention        in = q | k | v (one product)  ->  norms over all heads, rotation, cache append  ->  attention -> out
+//   Attention        in = q | k | v | gates per head (one product, biases in its epilogue)  ->  norms over all heads or per head,
+//                    rotation, factors on queries, cache append  ->  attention (gated) -> out
+//   GeneralDelta     in = r | k | v | a (32-bit) | w1 (through tanh) | g (one product)  ->  w2 (log decay in its epilogue)  ->
+//                    recurrence -> per-head norm and gate -> out
 //   Attention and    in = both mixers' projections (one product, silu where a mixer wants it)  ->  convolutions, norms, rotation, cache
 //   LinearState      append -> attention (gated) | convolutions -> recurrence -> norm and gate  ->  out: one product over both outputs side
 //   side by side     by side, or one each where they are normed before they meet
 //   Relu2            up (squared relu in its epilogue) -> down
-//   GatedSilu        gate and up rows in turn (one product, silu(gate) * up in its epilogue) -> down
+//   GatedSilu, GatedGelu  gate and up rows in turn (one product, act(gate) * up in its epilogue) -> down
 //   Moe              router | shared gate | shared up (one product) -> choice, token lists -> experts' up, experts' down
 //                    (grouped products), shared down
 //   token input      gate (gelu times the token's row of a table in its epilogue) -> proj
-// each followed by x += rms_norm(y) w (for Moe on the weighted sum of the experts' rows), which also writes the activations the
-// next product reads: the sum, or its norm where the design has norms on inputs and no token input follows.
+// each followed by x += rms_norm(y) w (for Moe on the weighted sum of the experts' rows) or, without norms on outputs, x += y, which
+// also takes the sum over depth at a layer's end and writes the activations the next product reads: the sum, or its norm where the
+// design has norms on inputs and no token input follows.
 #include <cmath>
 #include <cstring>
 #include "lc_model.h"
@@ -33,6 +37,15 @@ int32_t zalloc(LayerStack& st, void** p, size_t bytes) {
     st.owned.push_back(q);
     LC_CUDA(cudaMemsetAsync(q, 0, std::max<size_t>(bytes, 16), stream()));
     *p = q;
+    return LC_OK;
+}
+
+int32_t upload(LayerStack& st, const std::vector<float>& h, const float** out, cudaStream_t s) {
+    void* d = nullptr;
+    LC_TRY(zalloc(st, &d, h.size() * 4));
+    LC_CUDA(cudaMemcpyAsync(d, h.data(), h.size() * 4, cudaMemcpyHostToDevice, s));
+    LC_CUDA(cudaStreamSynchronize(s));
+    *out = (const float*)d;
     return LC_OK;
 }
 
@@ -134,17 +147,21 @@ int32_t changed_gain(lc_model* m, const std::string& name, int n, F f, const flo
     LC_CUDA(cudaMemcpyAsync(h.data(), g, h.size() * 4, cudaMemcpyDeviceToHost, m->stream));
     LC_CUDA(cudaStreamSynchronize(m->stream));
     for (float& v : h) v = f(v);
-    void* d = nullptr;
-    LC_TRY(zalloc(*m->stack, &d, h.size() * 4));
-    LC_CUDA(cudaMemcpyAsync(d, h.data(), h.size() * 4, cudaMemcpyHostToDevice, m->stream));
-    LC_CUDA(cudaStreamSynchronize(m->stream));
-    *out = (const float*)d;
-    return LC_OK;
+    return upload(*m->stack, h, out, m->stream);
 }
 
 // The weight of one of the model's norms.
 int32_t norm_gain(lc_model* m, const std::string& name, const float** out) {
-    const ArchSpec& sp = m->stack->spec;
+    LayerStack& st = *m->stack;
+    const ArchSpec& sp = st.spec;
+    if (sp.norm_scalar) {  // one number, for every element
+        const float* g = nullptr;
+        float v = 0.0f;
+        LC_TRY(model_gain_f32(m, name, 1, &g));
+        LC_CUDA(cudaMemcpyAsync(&v, g, 4, cudaMemcpyDeviceToHost, m->stream));
+        LC_CUDA(cudaStreamSynchronize(m->stream));
+        return upload(st, std::vector<float>((size_t)sp.width, v), out, m->stream);
+    }
     return sp.norm_one_plus ? changed_gain(m, name, sp.width, [](float v) { return 1.0f + v; }, out) : model_gain_f32(m, name, sp.width, out);
 }
 
@@ -277,22 +294,81 @@ void attention_shape(const LayerStack& st, MixerUnit& L) {
     L.ep = g.ep;
 }
 
+// The factors on queries of every position.
+int32_t q_factor_table(lc_model* m, const QueryTemperature& t, const float** out) {
+    LayerStack& st = *m->stack;
+    for (auto& f : st.q_factors)
+        if (f.first == t) { *out = f.second; return LC_OK; }
+    std::vector<float> h((size_t)m->cfg.max_seq_len);
+    for (size_t p = 0; p < h.size(); p++) h[p] = (float)(1.0 + t.coef * std::log(std::floor((double)(p + 1) / t.every) + 1.0));
+    LC_TRY(upload(st, h, out, m->stream));
+    st.q_factors.push_back({t, *out});
+    return LC_OK;
+}
+
 int32_t bind_attention(lc_model* m, MixerUnit& L, const std::string& p) {
+    LayerStack& st = *m->stack;
     const MixerSpec& s = L.s;
-    const int W = m->stack->spec.width, nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
-    attention_shape(*m->stack, L);
-    std::vector<int> offs;
-    if (s.kv_from < 0) {
-        LC_TRY(fused_weight(m, {p + "q", p + "k", p + "v"}, {nq, nk, nv}, W, &L.in, &offs));
-        L.off_k = offs[1]; L.off_v = offs[2];
-        LC_TRY(model_gain_f32(m, p + "k.norm", nk, &L.k_norm));
-    } else {
-        LC_TRY(plain_weight(m, p + "q", nq, W, &L.in));
+    const bool own = s.kv_from < 0;
+    const int W = st.spec.width, nq = s.heads * s.dim, nk = s.kv_heads * s.dim, nv = s.kv_heads * s.vdim;
+    LC_CHECK(s.qk_norm == QkNorm::AllHeads || std::max(s.dim, s.vdim) <= 512, LC_ERR_UNSUPPORTED, "%s: heads of %d and %d dimensions (at most 512)", p.c_str(), s.dim, s.vdim);
+    attention_shape(st, L);
+    std::vector<std::string> names = {p + "q"};
+    std::vector<int> rows = {nq}, offs;
+    if (own) { names.insert(names.end(), {p + "k", p + "v"}); rows.insert(rows.end(), {nk, nv}); }
+    const size_t biased = names.size();
+    if (s.head_gate) { names.push_back(p + "g"); rows.push_back(s.heads); }
+    if (names.size() == 1) { LC_TRY(plain_weight(m, p + "q", nq, W, &L.in)); offs = {0}; }
+    else LC_TRY(fused_weight(m, names, rows, W, &L.in, &offs));
+    if (own) { L.off_k = offs[1]; L.off_v = offs[2]; }
+    if (s.head_gate) L.off_hg = offs[biased];
+    if (s.qkv_bias) {
+        void* d = nullptr;
+        LC_TRY(zalloc(st, &d, (size_t)L.in.n * 4));
+        L.in_bias = (const float*)d;
+        for (size_t i = 0; i < biased; i++) {
+            const float* b = nullptr;
+            LC_TRY(model_gain_f32(m, names[i] + ".b", rows[i], &b));
+            LC_CUDA(cudaMemcpyAsync((float*)d + offs[i], b, (size_t)rows[i] * 4, cudaMemcpyDeviceToDevice, m->stream));
+        }
     }
-    LC_TRY(model_gain_f32(m, p + "q.norm", nq, &L.q_norm));
+    if (s.out_bias) LC_TRY(model_gain_f32(m, p + "o.b", W, &L.out_bias));
+    if (s.q_temp.coef != 0.0) LC_TRY(q_factor_table(m, s.q_temp, &L.q_factor));
+    if (s.qk_norm == QkNorm::AllHeads || s.qk_norm == QkNorm::PerHead) {
+        const bool all = s.qk_norm == QkNorm::AllHeads;
+        LC_TRY(model_gain_f32(m, p + "q.norm", all ? nq : s.dim, &L.q_norm));
+        if (own) LC_TRY(model_gain_f32(m, p + "k.norm", all ? nk : s.dim, &L.k_norm));
+    }
     if (m->tensors.count(p + "sink")) LC_TRY(model_gain_f32(m, p + "sink", s.heads, &L.sink));
     LC_TRY(plain_weight(m, p + "o", W, s.heads * s.vdim, &L.out, PackMap{s.vdim, L.ep, 0, 0}, s.heads * L.ep));
     return s.rot.dims ? rot_table(m, s.rot, &L.rot) : LC_OK;
+}
+
+int32_t bind_general_delta(lc_model* m, MixerUnit& L, const std::string& p) {
+    LayerStack& st = *m->stack;
+    const MixerSpec& s = L.s;
+    const int W = st.spec.width, n = s.heads * s.dim, n8 = round8(n), rank = rows_of(m, p + "w1"), ld = round8(W);
+    LC_CHECK(rank > 0, LC_ERR_MISSING, "missing tensor %sw1", p.c_str());
+    LC_CHECK(s.dim <= 256, LC_ERR_UNSUPPORTED, "%s: %d dimensions per head (at most 256)", p.c_str(), s.dim);
+    L.in_split = (4 * n8 + 31) / 32 * 32;
+    L.act_end = L.in_split + round8(rank);
+    const struct { const char* name; int rows, at; } parts[] = {{"r", n, 0}, {"k", n, n8}, {"v", n, 2 * n8}, {"a", n, 3 * n8}, {"w1", rank, L.in_split}, {"g", n, L.act_end}};
+    const int total = L.act_end + n8;
+    void* d = nullptr;
+    LC_TRY(talloc(st, &d, (size_t)total * ld * 2));
+    for (const auto& q : parts) {
+        DevTensor* t = nullptr;
+        LC_TRY(matrix(m, p + q.name, q.rows, W, &t));
+        LC_TRY(launch_pack((const bf16*)t->view, q.rows, W, (bf16*)d + (size_t)q.at * ld, ld, PackMap(), PackMap(), false, m->stream));
+    }
+    LC_TRY(dense_weight_init(&L.in, (const bf16*)d, total, W, ld));
+    L.off_g = L.act_end - L.in_split;
+    L.gg = GeneralShape{s.heads, s.dim, L.in_split, n8, 2 * n8, 3 * n8, s.unit_eps, st.spec.eps};
+    LC_TRY(plain_weight(m, p + "w2", n, rank, &L.a2));
+    LC_TRY(model_gain_f32(m, p + "w0", n, &L.dt_bias));
+    LC_TRY(model_gain_f32(m, p + "a.b", n, &L.a_bias));
+    LC_TRY(model_gain_f32(m, p + "norm", n, &L.o_norm));
+    return plain_weight(m, p + "o", W, n, &L.out);
 }
 
 // Attention and a linear recurrence side by side.
@@ -325,8 +401,8 @@ int32_t bind_pair(lc_model* m, StackLayer& L, const std::string& p) {
     }
     auto rows_of_parts = [](const std::vector<Part>& ps) { int n = 0; for (const Part& q : ps) n += round8(q.rows); return n; };
     L.in_split = (rows_of_parts(wide) + 31) / 32 * 32;
-    L.silu_end = L.in_split + rows_of_parts(silu);
-    const int total = L.silu_end + rows_of_parts(plain), ld = round8(W);
+    L.act_end = L.in_split + rows_of_parts(silu);
+    const int total = L.act_end + rows_of_parts(plain), ld = round8(W);
     void* d = nullptr;
     LC_TRY(talloc(st, &d, (size_t)total * ld * 2));
     auto place = [&](const std::vector<Part>& ps, int at, int base) -> int32_t {
@@ -341,7 +417,7 @@ int32_t bind_pair(lc_model* m, StackLayer& L, const std::string& p) {
     };
     LC_TRY(place(wide, 0, 0));
     LC_TRY(place(silu, L.in_split, L.in_split));
-    LC_TRY(place(plain, L.silu_end, L.in_split));
+    LC_TRY(place(plain, L.act_end, L.in_split));
     LC_TRY(dense_weight_init(&L.in, (const bf16*)d, total, W, ld));
     g.ld = total - L.in_split;
     g.ld_dt = L.in_split;
@@ -426,7 +502,7 @@ int32_t bind_ffn(lc_model* m, StackLayer& L, const std::string& p) {
         LC_TRY(plain_weight(m, p + "up", s.ff, W, &L.up));
         return plain_weight(m, p + "down", W, s.ff, &L.down);
     }
-    if (s.ffn == FfnKind::GatedSilu) {
+    if (s.ffn == FfnKind::GatedSilu || s.ffn == FfnKind::GatedGelu) {
         void* d = nullptr;
         LC_TRY(talloc(st, &d, (size_t)2 * s.ff * ld * 2));
         const char* part[2] = {"gate", "up"};
@@ -492,8 +568,39 @@ int32_t delta_block(lc_model* m, MixerUnit& L, const void* x, int ldx, int T, bo
         d.chunks = st.d_chunks; d.n_chunks = st.n_chunks; d.chunk_runs = st.d_chunk_runs; d.n_chunk_runs = st.n_chunk_runs;
         if (d.n_runs) LC_TRY(launch_delta_scan(d, m->stream));
         if (d.n_chunk_runs) LC_TRY(launch_delta_chunks(d, (float*)st.chunk_scratch.p, m->stream));
-        LC_TRY(launch_delta_output(d, m->stream));
+        HeadNormArgs o;
+        o.o = st.o; o.heads = s.heads; o.n = s.vdim; o.T = T; o.eps = st.spec.eps; o.w = L.o_norm; o.gate = st.gate; o.ld_gate = nv; o.out = st.mixed; o.ldo = d.ldo; o.f32 = st.f32;
+        LC_TRY(launch_head_norm(o, m->stream));
         m->launches_in_call += 2 + (d.n_runs ? 1 : 0) + (d.n_chunk_runs ? 2 : 0);
+    }
+    return product(m, L.out, st.mixed, d.ldo, T, st.y, st.spec.width, true);
+}
+
+int32_t general_delta_block(lc_model* m, MixerUnit& L, const void* x, int ldx, int T, bool decode_step) {
+    LayerStack& st = *m->stack;
+    const MixerSpec& s = L.s;
+    const int n = s.heads * s.dim, ld_act = L.in.n - L.in_split;
+    DenseArgs in, e;
+    in.split = L.in_split; in.act_end = L.act_end; in.out2 = st.proj; in.ldo2 = ld_act;
+    LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in_split, true, DENSE_SPLIT_TANH, in));
+    e.e1 = L.dt_bias; e.scale = (float)s.decay_scale;
+    LC_TRY(product(m, L.a2, st.proj, ld_act, T, st.log_decay, n, true, DENSE_SIGMOID_DECAY, e));
+    GeneralArgs d;
+    d.g = L.gg; d.proj = st.projf; d.a_bias = L.a_bias; d.log_decay = st.log_decay; d.state = L.state; d.tok_seq = m->d_tok_seq; d.tok_pos = m->d_tok_pos; d.T = T; d.o = st.o;
+    d.norm_w = L.o_norm; d.gate = at(st, st.proj, (size_t)L.off_g); d.ld_gate = ld_act; d.out = st.mixed; d.ldo = round8(n); d.f32 = st.f32;
+    if (decode_step) {
+        LC_TRY(launch_general_step(d, m->stream));
+        m->launches_in_call += 1;
+    } else {
+        d.runs = st.d_short_runs; d.n_runs = st.n_short_runs;
+        d.chunks = st.d_chunks; d.n_chunks = st.n_chunks; d.chunk_runs = st.d_chunk_runs; d.n_chunk_runs = st.n_chunk_runs;
+        if (d.n_runs) LC_TRY(launch_general_scan(d, m->stream));
+        if (d.n_chunk_runs) LC_TRY(launch_general_chunks(d, (float*)st.chunk_scratch.p, m->stream));
+        HeadNormArgs o;
+        o.o = st.o; o.heads = s.heads; o.n = s.dim; o.T = T; o.eps = st.spec.eps; o.w = L.o_norm; o.w_stride = s.dim; o.gate = d.gate; o.ld_gate = ld_act; o.out = st.mixed;
+        o.ldo = d.ldo; o.f32 = st.f32;
+        LC_TRY(launch_head_norm(o, m->stream));
+        m->launches_in_call += 1 + (d.n_runs ? 1 : 0) + (d.n_chunk_runs ? 2 : 0);
     }
     return product(m, L.out, st.mixed, d.ldo, T, st.y, st.spec.width, true);
 }
@@ -544,6 +651,7 @@ int32_t attend(lc_model* m, const MixerUnit& L, const MixerUnit& src, AttnArgs a
     a.conv = L.conv; a.ring = (float*)L.ring; a.one_each = decode_step;
     a.q = st.q; a.k_cache = src.k_cache; a.v_cache = src.v_cache; a.page_tokens = m->page_tokens; a.page_table = m->d_page_table; a.tok_seq = m->d_tok_seq;
     a.tok_pos = m->d_tok_pos; a.pages_per_seq = m->pages_per_seq; a.T = T; a.sink = L.sink; a.f32 = st.f32;
+    a.q_factor = L.q_factor; a.head_gate = L.off_hg >= 0 ? st.projf + L.off_hg : nullptr;
     LC_TRY(launch_attn_prep(a, m->stream));
     m->launches_in_call += 1;
     if (L.ag.taps > 0 && !decode_step) {
@@ -565,11 +673,13 @@ int32_t attend(lc_model* m, const MixerUnit& L, const MixerUnit& src, AttnArgs a
 
 int32_t attention_block(lc_model* m, MixerUnit& L, const void* x, int ldx, int T, bool decode_step) {
     LayerStack& st = *m->stack;
-    LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in.n, true));
+    DenseArgs in, out;
+    in.e1 = L.in_bias; out.e1 = L.out_bias;
+    LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in.n, true, L.in_bias ? DENSE_BIAS : DENSE_STORE, in));
     AttnArgs a;
     a.ld_proj = L.in.n; a.out = st.mixed; a.ldo = L.ag.heads * L.ep;
     LC_TRY(attend(m, L, L.s.kv_from < 0 ? L : st.layers[(size_t)L.s.kv_from].mix[0], a, T, decode_step));
-    return product(m, L.out, st.mixed, a.ldo, T, st.y, st.spec.width, true);
+    return product(m, L.out, st.mixed, a.ldo, T, st.y, st.spec.width, true, L.out_bias ? DENSE_BIAS : DENSE_STORE, out);
 }
 
 int32_t recur(lc_model* m, const MixerUnit& L, LinearArgs a, int T, bool decode_step) {
@@ -593,7 +703,7 @@ int32_t pair_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, bo
     LayerStack& st = *m->stack;
     DenseArgs in;
     const int ld_act = L.in.n - L.in_split;
-    in.split = L.in_split; in.silu_end = L.silu_end; in.out2 = st.proj; in.ldo2 = ld_act;
+    in.split = L.in_split; in.act_end = L.act_end; in.out2 = st.proj; in.ldo2 = ld_act;
     LC_TRY(product(m, L.in, x, ldx, T, st.projf, L.in_split, true, DENSE_SPLIT_SILU, in));
     const bool normed = L.s.combine == Combine::Normed;
     AttnArgs a;
@@ -677,7 +787,7 @@ int32_t ffn_block(lc_model* m, StackLayer& L, const void* x, int ldx, int T, boo
     LayerStack& st = *m->stack;
     if (L.s.ffn == FfnKind::Moe) return moe_block(m, L, x, ldx, T, decode_step);
     const int ldf = round8(L.s.ff);
-    LC_TRY(product(m, L.up, x, ldx, T, st.ffn, ldf, false, L.s.ffn == FfnKind::GatedSilu ? DENSE_GATED_SILU : DENSE_RELU2));
+    LC_TRY(product(m, L.up, x, ldx, T, st.ffn, ldf, false, L.s.ffn == FfnKind::GatedSilu ? DENSE_GATED_SILU : L.s.ffn == FfnKind::GatedGelu ? DENSE_GATED_GELU : DENSE_RELU2));
     return product(m, L.down, st.ffn, ldf, T, st.y, st.spec.width, true);
 }
 
@@ -704,9 +814,11 @@ int32_t stack_bind(lc_model* m) {
         if (L.s.combine != Combine::Single) LC_TRY(bind_pair(m, L, p + "mix."));
         else if (u.s.kind == MixerKind::ChannelDelta) LC_TRY(bind_delta(m, u, p + "mix."));
         else if (u.s.kind == MixerKind::LatentAttention) LC_TRY(bind_latent(m, u, p + "mix."));
+        else if (u.s.kind == MixerKind::GeneralDelta) LC_TRY(bind_general_delta(m, u, p + "mix."));
         else LC_TRY(bind_attention(m, u, p + "mix."));
         auto norms = [&](const std::string& name, const float** in, const float** out) -> int32_t {
             if (sp.norm_inputs) LC_TRY(norm_gain(m, name, in));
+            if (!sp.norm_outputs) return LC_OK;
             return norm_gain(m, sp.norm_inputs ? name + "b" : name, out);
         };
         LC_TRY(norms(p + "norm1", &L.norm1_in, &L.norm1_out));
@@ -714,6 +826,7 @@ int32_t stack_bind(lc_model* m) {
             LC_TRY(bind_ffn(m, L, p + "mlp."));
             LC_TRY(norms(p + "norm2", &L.norm2_in, &L.norm2_out));
         }
+        if (sp.depth_average) LC_TRY(model_gain_f32(m, p + "dwa", (int)i + 2, &L.dwa));
         if (sp.side_dim) {
             LC_TRY(plain_weight(m, p + "side.gate", sp.side_dim, sp.width, &L.side_gate));
             LC_TRY(plain_weight(m, p + "side.proj", sp.width, sp.side_dim, &L.side_proj));
@@ -729,6 +842,10 @@ int32_t stack_bind(lc_model* m) {
     if (sp.side_dim) {
         LC_TRY(matrix(m, "side.embed", sp.vocab, (int)sp.layers.size() * sp.side_dim, &e));
         st.side_embed = (const bf16*)e->view;
+    }
+    if (sp.bigram.buckets) {
+        LC_TRY(matrix(m, "bigram", (int)sp.bigram.buckets + 1, sp.width, &e));
+        st.bigram = (const bf16*)e->view;
     }
     st.packed.clear();  // the tables are read as they are
     LC_TRY(norm_gain(m, "final.norm", &st.final_norm));
@@ -760,6 +877,17 @@ int32_t stack_alloc(lc_model* m) {
             st.delta_chunks = st.delta_chunks && delta_chunks_apply(L.dg, st.f32);
             st.chunk_bytes = std::max(st.chunk_bytes, delta_chunk_bytes(L.dg));
             st.state_bytes_per_seq += S * 4 + ring * e;
+        } else if (s.kind == MixerKind::GeneralDelta) {
+            const size_t n = (size_t)s.heads * s.dim, S = n * s.dim;
+            proj = std::max(proj, (size_t)(L.in.n - L.in_split));
+            projf = std::max(projf, (size_t)L.in_split);
+            mixed = std::max(mixed, (size_t)round8((int)n));
+            ld = std::max(ld, n);
+            v = std::max(v, n);
+            LC_TRY(zalloc(st, (void**)&L.state, (size_t)m->max_seqs * S * 4));
+            st.delta_chunks = st.delta_chunks && general_chunks_apply(L.gg, s.decay_scale, st.f32);
+            st.chunk_bytes = std::max(st.chunk_bytes, general_chunk_bytes(L.gg));
+            st.state_bytes_per_seq += S * 4;
         } else if (s.kind == MixerKind::Attention) {
             const AttnShape& g = L.ag;
             projf = std::max(projf, (size_t)L.in.n);
@@ -849,6 +977,8 @@ int32_t stack_alloc(lc_model* m) {
     LC_TRY(zalloc(st, &st.q_abs, T * qa * e)); LC_TRY(zalloc(st, &st.o_lat, T * qa * e));
     LC_TRY(zalloc(st, &st.ffn, T * ffn * e)); LC_TRY(zalloc(st, &st.last, (size_t)m->head_rows * st.width_p * e));
     if (lin) LC_TRY(zalloc(st, &st.lin, T * lin * e));
+    if (st.bigram) LC_TRY(zalloc(st, (void**)&st.last_token, (size_t)m->max_seqs * 4));
+    if (st.spec.depth_average) LC_TRY(zalloc(st, (void**)&st.depth, (st.layers.size() + 1) * T * st.spec.width * 4));
     if (st.spec.side_dim) LC_TRY(zalloc(st, &st.side, T * round8(st.spec.side_dim) * e));
     LC_TRY(zalloc(st, (void**)&st.y, (pairs ? 2 : 1) * T * st.spec.width * 4));
     if (pairs) st.y2 = st.y + T * st.spec.width;
@@ -873,7 +1003,7 @@ void stack_free(lc_model* m) {
 // Cache and state a one-token step at position `ctx` reads and writes.
 uint64_t stack_step_bytes(const lc_model* m, int ctx) {
     const LayerStack& st = *m->stack;
-    uint64_t b = 2 * st.state_bytes_per_seq + (uint64_t)st.layers.size() * st.spec.side_dim * 2;
+    uint64_t b = 2 * st.state_bytes_per_seq + (uint64_t)st.layers.size() * st.spec.side_dim * 2 + (st.bigram ? (uint64_t)st.spec.width * 2 : 0);
     for (const StackLayer& layer : st.layers) {
         const MixerUnit& L = layer.mix[0];
         if (L.s.kind == MixerKind::LatentAttention) b += (uint64_t)(ctx + 1) * (L.lg.cp + L.lg.rp) * elt(st);
@@ -886,7 +1016,7 @@ uint64_t stack_step_bytes(const lc_model* m, int ctx) {
 
 uint64_t stack_table_bytes(const lc_model* m) {
     const ArchSpec& sp = m->stack->spec;
-    return (uint64_t)sp.vocab * sp.layers.size() * sp.side_dim * 2;
+    return (uint64_t)sp.vocab * sp.layers.size() * sp.side_dim * 2 + (sp.bigram.buckets ? (uint64_t)(sp.bigram.buckets + 1) * sp.width * 2 : 0);
 }
 
 // What a call's tokens mean to the layers: runs of consecutive positions, those of at least kTileRun tokens also as tiles
@@ -962,6 +1092,7 @@ int32_t stack_mixer(lc_model* m, int l, const void* x, int ldx, int T, bool deco
     switch (L.mix[0].s.kind) {
         case MixerKind::ChannelDelta: return delta_block(m, L.mix[0], x, ldx, T, decode_step);
         case MixerKind::LatentAttention: return latent_block(m, L.mix[0], x, ldx, T, decode_step);
+        case MixerKind::GeneralDelta: return general_delta_block(m, L.mix[0], x, ldx, T, decode_step);
         default: return attention_block(m, L.mix[0], x, ldx, T, decode_step);
     }
 }
@@ -971,9 +1102,17 @@ int32_t stack_run_layers(lc_model* m, int T, bool decode_step) {
     const int W = st.spec.width;
     int ldx = 0;
     const void* x = layer_input(m, &ldx);
-    LC_TRY(launch_embed_rows(st.embed, st.spec.vocab, W, m->d_tokens, T, st.spec.embed_scale, st.layers[0].norm1_in, st.spec.eps, m->d_hidden, st.xa, st.width_p, st.f32,
-                             m->stream));
+    EmbedArgs e;
+    e.table = st.embed; e.rows = st.spec.vocab; e.width = W; e.T = T; e.ids = m->d_tokens; e.scale = st.spec.embed_scale; e.eps = st.spec.eps; e.w = st.layers[0].norm1_in;
+    e.x = m->d_hidden; e.copy = st.depth; e.act = st.xa; e.ld_act = st.width_p; e.f32 = st.f32;
+    e.pair.table = st.bigram; e.pair.rows = st.spec.bigram; e.pair.tok_seq = m->d_tok_seq; e.pair.tok_pos = m->d_tok_pos; e.pair.last = st.last_token; e.pair.one_each = decode_step;
+    LC_TRY(launch_embed_rows(e, m->stream));
     m->launches_in_call += 1;
+    if (st.bigram && !decode_step) {
+        LC_TRY(launch_keep_tokens(st.d_runs, st.n_runs, m->d_tokens, st.last_token, m->stream));
+        m->launches_in_call += 1;
+    }
+    const size_t plane = (size_t)m->t_cap * W;
     ResidualArgs r;
     r.y = st.y; r.eps = st.spec.eps; r.width = W; r.T = T; r.x = m->d_hidden; r.ld_act = st.width_p; r.f32 = st.f32;
     for (size_t l = 0; l < st.layers.size(); l++) {
@@ -981,7 +1120,9 @@ int32_t stack_run_layers(lc_model* m, int T, bool decode_step) {
         const bool ffn = L.s.ffn != FfnKind::None, last = l + 1 == st.layers.size(), side = st.spec.side_dim > 0;
         const float* after = last ? nullptr : st.layers[l + 1].norm1_in;  // the norm ahead of the next layer; the last sum is read in f32
         // plain_next: the sum itself is read next, not its norm
-        auto sum = [&](const float* w, const float* next, bool moe, bool pair, bool plain_next) -> int32_t {
+        auto sum = [&](const float* w, const float* next, bool moe, bool pair, bool plain_next, bool end) -> int32_t {
+            r.depth = DepthSum();
+            if (end && st.depth) { r.depth.past = st.depth; r.depth.keep = st.depth + (l + 1) * plane; r.depth.stride = plane; r.depth.c = L.dwa; r.depth.n = (int)l + 1; }
             r.w = w; r.w_next = plain_next ? nullptr : next; r.act = st.spec.norm_inputs && !plain_next && !next ? nullptr : st.xa;
             r.moe = moe ? moe_sum(st, L, x, ldx) : MoeSum();
             r.pair = pair ? pair_sum(st, L) : PairSum();
@@ -989,14 +1130,14 @@ int32_t stack_run_layers(lc_model* m, int T, bool decode_step) {
             return launch_residual(r, m->stream);
         };
         LC_TRY(stack_mixer(m, (int)l, x, ldx, T, decode_step));
-        LC_TRY(sum(L.norm1_out, ffn ? L.norm2_in : after, false, L.s.combine == Combine::Normed, side && !ffn));
+        LC_TRY(sum(L.norm1_out, ffn ? L.norm2_in : after, false, L.s.combine == Combine::Normed, side && !ffn, !side && !ffn));
         if (ffn) {
             LC_TRY(ffn_block(m, L, x, ldx, T, decode_step));
-            LC_TRY(sum(L.norm2_out, after, L.s.ffn == FfnKind::Moe, false, side));
+            LC_TRY(sum(L.norm2_out, after, L.s.ffn == FfnKind::Moe, false, side, !side));
         }
         if (!side) continue;
         LC_TRY(side_block(m, (int)l, T));
-        LC_TRY(sum(L.side_norm, after, false, false, false));
+        LC_TRY(sum(L.side_norm, after, false, false, false, true));
     }
     return LC_OK;
 }

@@ -7,9 +7,9 @@
 
 namespace lc {
 
-enum class MixerKind { ChannelDelta, LatentAttention, Attention, LinearState };
-// Relu2: down(relu(up x)^2).  GatedSilu: down(silu(gate x) * (up x)).  Moe: a mixture of such (MoeSpec).
-enum class FfnKind { None, Relu2, GatedSilu, Moe };
+enum class MixerKind { ChannelDelta, LatentAttention, Attention, LinearState, GeneralDelta };
+// Relu2: down(relu(up x)^2).  GatedSilu, GatedGelu: down(act(gate x) * (up x)), gelu in its tanh form.  Moe: a mixture of such (MoeSpec).
+enum class FfnKind { None, Relu2, GatedSilu, GatedGelu, Moe };
 const char* mixer_name(MixerKind k);
 
 // Rotary embedding, optionally with scaled frequencies: YaRN's interpolation over pairs, or by wavelength (pairs that turn more
@@ -46,8 +46,13 @@ struct MoeSpec {
 };
 
 // Norms of attention's queries and keys: over all heads together ahead of the rotation (weights of all heads), per head ahead of it
-// (one weight of `dim`), per head behind it (no weight).
-enum class QkNorm { AllHeads, PerHead, PerHeadAfter };
+// (one weight of `dim`), per head behind it (no weight), none.
+enum class QkNorm { AllHeads, PerHead, PerHeadAfter, None };
+// Factor 1 + coef ln(floor((position + 1) / every) + 1) on attention's queries (coef 0: none).
+struct QueryTemperature {
+    double coef = 0.0, every = 1.0;
+    bool operator==(const QueryTemperature& o) const { return coef == o.coef && every == o.every; }
+};
 // The two dimensions of a rotation pair: i and i + dims / 2, or 2i and 2i + 1.
 enum class AttnPairs { Halves, Neighbours };
 // LinearState: S = decay S + step k v^T, read with q, per head.  Constant: decays from the config, q, k and v through silu, the heads
@@ -71,6 +76,12 @@ struct MixerSpec {
     AttnPairs pairs = AttnPairs::Halves;
     float softcap = 0.0f;                         // scores through cap * tanh(. / cap); 0: none
     bool out_gate = false;                        // a sigmoid gate per output element
+    bool head_gate = false;                       // a sigmoid gate per head
+    bool qkv_bias = false, out_bias = false;
+    QueryTemperature q_temp;
+    // GeneralDelta: S = diag(w) S - (a u) (u^T S) + k v^T over the old S, u the unit key; w = exp(-decay_scale * sigmoid(.)) and a =
+    // sigmoid(.) per key channel
+    double decay_scale = 0.0;
     // LinearState
     LinearKind linear = LinearKind::Constant;
     int norm_parts = 1;
@@ -89,16 +100,25 @@ struct LayerSpec {
     MoeSpec moe;
 };
 
+// A second embedding by (previous token, token): row (previous * mul_prev + token * mul_cur) mod buckets, for a sequence's first
+// token row `buckets` (0 buckets: none).  The factors are kept modulo buckets.
+struct BigramSpec { int64_t buckets = 0, mul_prev = 0, mul_cur = 0; };
+
 // A stack of layers with norms on the sublayers' outputs, x += norm1(mixer(x)), x += norm2(ffn(x)); norm_inputs: on their
-// inputs too, x += norm1b(mixer(norm1(x))), x += norm2b(ffn(norm2(x))).  side_dim: every layer ends with
-// x += norm(proj(gelu(gate x) * e)), e the layer's part of the token's row in a table of [vocab, layers * side_dim].
+// inputs too, x += norm1b(mixer(norm1(x))), x += norm2b(ffn(norm2(x))), or (norm_outputs false) there alone, x += mixer(norm1(x)),
+// x += ffn(norm2(x)).  side_dim: every layer ends with x += norm(proj(gelu(gate x) * e)), e the layer's part of the token's row in
+// a table of [vocab, layers * side_dim].  depth_average: what leaves layer i is sum_j dwa[j] X_j over the embedding X_0 and the
+// results X_1 .. X_(i + 1) of the layers so far, before their averaging.
 struct ArchSpec {
     std::string name;
     std::vector<LayerSpec> layers;
     int width = 0, vocab = 0;
     float eps = 1e-6f;
-    bool norm_inputs = false;
+    bool norm_inputs = false, norm_outputs = true;
     bool norm_one_plus = false;  // norm weights stored around zero: 1 + w
+    bool norm_scalar = false;    // one number for all elements
+    bool depth_average = false;
+    BigramSpec bigram;
     int side_dim = 0;
     float embed_scale = 1.0f;
     float logit_scale = 1.0f, logit_softcap = 0.0f;  // softcap 0: none

@@ -32,8 +32,12 @@ enum DenseEpilogue {
     DENSE_LOGITS = 3,     // y * scale, then cap * tanh(. / cap) when cap > 0
     DENSE_GATED_SILU = 4, // rows in pairs (2i: gate, 2i + 1: up): out row i = silu(gate) * up
     DENSE_SPLIT_RELU2 = 5, // rows below `split` as they are, in 32-bit, to `out`; the others squared relu, in the activations' type, to out2
-    DENSE_SPLIT_SILU = 6,  // the same with silu up to row `silu_end`, and the rest as they are
-    DENSE_GELU_TABLE = 7   // gelu (tanh form) times element `row` of the token's row in a table (0 for ids outside it)
+    DENSE_SPLIT_SILU = 6,  // the same with silu up to row `act_end`, and the rest as they are
+    DENSE_GELU_TABLE = 7,  // gelu (tanh form) times element `row` of the token's row in a table (0 for ids outside it)
+    DENSE_GATED_GELU = 8,  // as DENSE_GATED_SILU with gelu (tanh form)
+    DENSE_BIAS = 9,        // y + e1[row]
+    DENSE_SPLIT_TANH = 10, // as DENSE_SPLIT_SILU with tanh
+    DENSE_SIGMOID_DECAY = 11  // -scale * sigmoid(y + e1[row])
 };
 // A product of one of several matrices per token (experts): the tokens come as tiles of rows that share a matrix.
 struct ExpertTile { int32_t expert, first, rows, row0; };  // rows first .. first + rows - 1 of the expert's list; row0: the first one's row in expert order
@@ -63,7 +67,7 @@ struct DenseArgs {
     float scale = 1.0f, cap = 0.0f;
     void* out2 = nullptr;         // DENSE_SPLIT_*
     int ldo2 = 0, split = 0;      // split: a multiple of 32
-    int silu_end = 0;             // DENSE_SPLIT_SILU
+    int act_end = 0;              // DENSE_SPLIT_SILU, DENSE_SPLIT_TANH
     const __nv_bfloat16* table = nullptr;  // DENSE_GELU_TABLE: rows table_ld apart
     int table_ld = 0, table_rows = 0;
     const int64_t* ids = nullptr;
@@ -94,10 +98,28 @@ struct SeqRun { int32_t tok0, n, seq, pos0; };
 struct PackMap { int len = 0, stride = 0, split = 0, shift = 0; };
 int32_t launch_pack(const __nv_bfloat16* src, int rows, int cols, __nv_bfloat16* dst, int ld, PackMap row, PackMap col, bool transpose, cudaStream_t s);
 
-// x[t] = embed[ids[t]] * scale in f32; act != null: the same as activations, through rms_norm(.) * w when w is given.  ids
-// outside the table give zero rows
-int32_t launch_embed_rows(const __nv_bfloat16* table, int rows, int width, const int64_t* ids, int T, float scale, const float* w, float eps, float* x, void* act, int ld_act,
-                          bool f32, cudaStream_t s);
+// x[t] = embed[ids[t]] * scale in f32 (+ the row of the token pair); act != null: the same as activations, through rms_norm(.) * w
+// when w is given.  ids outside the table give zero rows
+struct PairEmbed {
+    const __nv_bfloat16* table = nullptr;  // [buckets + 1][width]; null: none
+    BigramSpec rows;
+    const int32_t *tok_seq = nullptr, *tok_pos = nullptr;
+    int32_t* last = nullptr;               // [slot] the sequence's last token of earlier calls
+    bool one_each = false;                 // every token is the only one of its sequence: `last` is brought up to date too
+};
+struct EmbedArgs {
+    const __nv_bfloat16* table = nullptr;
+    int rows = 0, width = 0, T = 0;
+    const int64_t* ids = nullptr;
+    float scale = 1.0f, eps = 1e-6f;
+    const float* w = nullptr;
+    float *x = nullptr, *copy = nullptr;   // copy: a second one, or null
+    void* act = nullptr;
+    int ld_act = 0;
+    bool f32 = false;
+    PairEmbed pair;
+};
+int32_t launch_embed_rows(const EmbedArgs& a, cudaStream_t s);
 // act[t] = bf16(x[t])
 int32_t launch_act_rows(const float* x, int width, int T, void* act, int ld_act, cudaStream_t s);
 // The output of a mixture of experts at one token: gate * y + sum over the choices of weight * (expert's row, or the input for
@@ -117,8 +139,15 @@ struct MoeSum {
 struct PairSum {
     const float *y2 = nullptr, *w0 = nullptr, *w1 = nullptr;  // y2 null: no pair
 };
-// x[t] += rms_norm(y[t]) * w; act != null: the sum as activations, through rms_norm(.) * w_next when that is given.  With a
-// mixture or a pair y is first replaced by its output (x null: nothing more happens).
+// What leaves a layer: sum_j c[j] X_j over n rows of earlier results (planes `stride` apart) and, with c[n], this one, kept in `keep`.
+struct DepthSum {
+    const float *past = nullptr, *c = nullptr;
+    float* keep = nullptr;                                    // null: no sum over depth
+    size_t stride = 0;
+    int n = 0;
+};
+// x[t] += rms_norm(y[t]) * w, or += y[t] without w; act != null: the sum as activations, through rms_norm(.) * w_next when that is
+// given.  With a mixture or a pair y is first replaced by its output (x null: nothing more happens).
 struct ResidualArgs {
     float* y = nullptr;
     const float *w = nullptr, *w_next = nullptr;
@@ -130,10 +159,28 @@ struct ResidualArgs {
     bool f32 = false;
     MoeSum moe;
     PairSum pair;
+    DepthSum depth;                    // only without w
 };
 int32_t launch_residual(const ResidualArgs& a, cudaStream_t s);
 // out[i] = rms_norm(x[idx ? idx[i] : i]) * w as activations
 int32_t launch_norm_rows(const float* x, const int32_t* idx, const float* w, float eps, int width, int n, void* out, int ldo, bool f32, cudaStream_t s);
+// last[slot] = the last token of every run, behind the embedding
+int32_t launch_keep_tokens(const SeqRun* runs, int n_runs, const int64_t* ids, int32_t* last, cudaStream_t s);
+
+// Per head: o / rms(o) * w * sigmoid(gate), as activations.
+struct HeadNormArgs {
+    const float* o = nullptr;          // [T][heads * n]
+    int heads = 0, n = 0, T = 0;
+    float eps = 1e-6f;
+    const float* w = nullptr;          // heads w_stride apart (0: shared)
+    int w_stride = 0;
+    const void* gate = nullptr;        // [T][ld_gate] activations, before the sigmoid
+    int ld_gate = 0;
+    void* out = nullptr;               // [T][ldo] activations
+    int ldo = 0;
+    bool f32 = false;
+};
+int32_t launch_head_norm(const HeadNormArgs& a, cudaStream_t s);
 
 // Gated delta rule with one decay per key channel.  `proj` rows hold q | k | v | ... | beta logits as projected; the inputs of
 // the short convolutions of the last `taps` positions live in `ring` [slot][taps][channels], entry position % taps.
@@ -166,8 +213,7 @@ struct DeltaArgs {
 };
 int32_t launch_delta_prep(const DeltaArgs& a, cudaStream_t s);   // convolutions, silu, unit vectors
 int32_t launch_delta_scan(const DeltaArgs& a, cudaStream_t s);   // the recurrence over every run; leaves state and ring for the next call
-int32_t launch_delta_output(const DeltaArgs& a, cudaStream_t s); // per-head norm, gate
-int32_t launch_delta_step(const DeltaArgs& a, cudaStream_t s);   // the three for one new token per sequence (rows of tok_seq / tok_pos)
+int32_t launch_delta_step(const DeltaArgs& a, cudaStream_t s);   // the two with norm and gate for one new token per sequence (rows of tok_seq / tok_pos)
 
 // delta_chunk.cu: the recurrence over `chunk_runs`, in chunks; scratch of delta_chunk_bytes per chunk
 bool delta_chunks_apply(const DeltaShape& g, bool f32);
@@ -265,6 +311,8 @@ struct AttnArgs {
     const float* sink = nullptr;       // [heads] or null
     const void* gate = nullptr;        // [T][ld_gate] activations, heads vdim apart: sigmoid(gate) on the output; null: none
     int ld_gate = 0;
+    const float* head_gate = nullptr;  // [T][ld_proj] one number per head: sigmoid(.) on the head's output; null: none
+    const float* q_factor = nullptr;   // [position] on the queries; null: none
     float out_scale = 1.0f;
     void* out = nullptr;               // [T][ldo], heads ep apart
     int ldo = 0;
@@ -320,6 +368,41 @@ int32_t launch_linear_runs(const LinearArgs& a, int* launches, cudaStream_t s); 
 int32_t launch_linear_step(const LinearArgs& a, int* launches, cudaStream_t s);  // the same for one token per sequence
 int32_t launch_linear_output(const LinearArgs& a, cudaStream_t s);               // gate and norm
 
+// ---- general_delta.cu: S_t = diag(w) S_(t-1) - (a u) (u^T S_(t-1)) + k v^T, o_t = S_t^T r, per head, S in f32; u = k / sqrt(|k|^2 + unit_eps),
+// a = sigmoid(. + a_bias), all of r, k, v, a and the state dim wide -----------------------------------------------------------------------
+struct GeneralShape {
+    int heads, dim;
+    int ld, off_k, off_v, off_a;       // columns of the projected rows (r at 0)
+    float unit_eps, eps;
+};
+constexpr int kGeneralChunk = 32;      // tokens per step of the chunked form
+struct GeneralArgs {
+    GeneralShape g;
+    const float* proj = nullptr;       // [T][ld] r | k | v | a
+    const float* a_bias = nullptr;     // [heads * dim]
+    const float* log_decay = nullptr;  // [T][heads * dim], ln w
+    float* state = nullptr;            // [slot][heads][dim][dim]
+    const int32_t *tok_seq = nullptr, *tok_pos = nullptr;
+    int T = 0;
+    float* o = nullptr;                // [T][heads * dim]
+    const SeqRun* runs = nullptr;      // walked token by token
+    int n_runs = 0;
+    const DeltaChunk* chunks = nullptr;         // longer runs
+    const DeltaChunkRun* chunk_runs = nullptr;
+    int n_chunks = 0, n_chunk_runs = 0;
+    const float* norm_w = nullptr;     // the step alone: norm, gate and output as in HeadNormArgs
+    const void* gate = nullptr;
+    int ld_gate = 0;
+    void* out = nullptr;
+    int ldo = 0;
+    bool f32 = false;
+};
+bool general_chunks_apply(const GeneralShape& g, double decay_scale, bool f32);
+size_t general_chunk_bytes(const GeneralShape& g);               // scratch per chunk of kDeltaChunk tokens
+int32_t launch_general_scan(const GeneralArgs& a, cudaStream_t s);
+int32_t launch_general_chunks(const GeneralArgs& a, float* scratch, cudaStream_t s);
+int32_t launch_general_step(const GeneralArgs& a, cudaStream_t s);  // one token per sequence, with norm and gate
+
 // ---- expert_choice.cu: routing ---------------------------------------------------------------------------------------------
 struct ChoiceArgs {
     MoeSpec m;
@@ -344,7 +427,7 @@ struct MixerUnit {
     // ChannelDelta: `in` = q | k | v | a1 | g1 | b
     DenseWeight a2, g2;
     DeltaShape dg{};
-    int off_a = 0, off_g = 0;
+    int off_a = 0, off_g = 0;       // off_g also: the output gate of GeneralDelta and Attention, in the activations' part
     const float *conv = nullptr, *a_exp = nullptr, *dt_bias = nullptr, *o_norm = nullptr;
     float* state = nullptr;
     void* ring = nullptr;
@@ -358,9 +441,15 @@ struct MixerUnit {
     void* cache = nullptr;
     // Attention: `in` = q | k | v (q alone when another layer's cache is read)
     AttnShape ag{};
-    int off_k = -1, off_v = 0;      // off_g: the output gate, in the activations' part
+    int off_k = -1, off_v = 0;
     const float *k_norm = nullptr, *sink = nullptr;
     void *k_cache = nullptr, *v_cache = nullptr;
+    const float *in_bias = nullptr, *out_bias = nullptr, *q_factor = nullptr;
+    int off_hg = -1;                // the gates per head
+    // GeneralDelta: `in` = r | k | v | a (32-bit, below in_split) | w1 | g; a2 = w2, dt_bias = its bias
+    GeneralShape gg{};
+    int in_split = 0, act_end = 0;
+    const float* a_bias = nullptr;
     // LinearState
     LinearShape ng{};
     const float *conv_b = nullptr, *skip = nullptr, *log_decay = nullptr;
@@ -370,10 +459,10 @@ struct StackLayer {
     LayerSpec s;
     MixerUnit mix[2];
     // two mixers side by side: what both read projected by one product, 32-bit rows below in_split, activations behind it (silu up
-    // to row silu_end); their outputs lie side by side in rows of mixed_ld, the second one's from mixed_off on, and leave through
+    // to row act_end); their outputs lie side by side in rows of mixed_ld, the second one's from mixed_off on, and leave through
     // `out` together (Scaled) or through one matrix each (Normed)
     DenseWeight in, out, out2;
-    int in_split = 0, silu_end = 0, mixed_off = 0, mixed_ld = 0;
+    int in_split = 0, act_end = 0, mixed_off = 0, mixed_ld = 0;
     const float* out_norm[2] = {nullptr, nullptr};
     // norms of the sublayers' inputs (null: none) and outputs
     const float *norm1_in = nullptr, *norm1_out = nullptr, *norm2_in = nullptr, *norm2_out = nullptr;
@@ -383,6 +472,7 @@ struct StackLayer {
     int off_gate = 0, route_split = 0;
     const float* correction = nullptr;
     uint64_t expert_bytes = 0;         // one expert's matrices
+    const float* dwa = nullptr;        // weights of the sum over depth
     // token input
     DenseWeight side_gate, side_proj;
     const float* side_norm = nullptr;
@@ -393,13 +483,16 @@ struct LayerStack {
     std::vector<StackLayer> layers;
     DenseWeight head;
     const __nv_bfloat16* embed = nullptr;
-    const __nv_bfloat16* side_embed = nullptr;
+    const __nv_bfloat16 *side_embed = nullptr, *bigram = nullptr;
+    int32_t* last_token = nullptr;     // [slot], for the pair embedding
+    float* depth = nullptr;            // [layers + 1][t_cap][width]: the call's embedding and layers' results
     const float* final_norm = nullptr;
     DenseWorkspace ws;
     std::vector<void*> owned;
     std::vector<void*> temps;          // plain copies of weights, dropped once their blocks exist
     std::vector<std::string> packed;   // checkpoint tensors whose bytes live on in blocks only
     std::vector<std::pair<RotarySpec, const float2*>> rot_tables;
+    std::vector<std::pair<QueryTemperature, const float*>> q_factors;
     uint64_t cache_bytes_per_token = 0, state_bytes_per_seq = 0;
     // step buffers for t_cap tokens
     int width_p = 0;

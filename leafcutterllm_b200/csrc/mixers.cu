@@ -55,30 +55,53 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const __nv_bfloat16* __
     }
 }
 
-// The same with a factor on the row and, w != null, the row's norm as activations.
-template <typename A>
-__global__ void __launch_bounds__(256) embed_norm_kernel(const bf16* __restrict__ table, int rows, int width, const int64_t* __restrict__ ids, float scale,
-                                                         const float* __restrict__ w, float eps, float* __restrict__ x, A* __restrict__ act, int ld_act) {
+// The same with a factor on the row, the token pair's row (PAIR) and, w != null, the sum's norm as activations.
+template <typename A, bool PAIR>
+__global__ void __launch_bounds__(256) embed_norm_kernel(const EmbedArgs a) {
     __shared__ float sh[32];
     pdl_launch_dependents();
     pdl_wait();
     const size_t t = blockIdx.x;
-    const int64_t id = ids[t];
-    const bool ok = id >= 0 && id < rows;
-    const bf16* src = table + (size_t)(ok ? id : 0) * width;
+    const int width = a.width;
+    const int64_t id = a.ids[t];
+    const bool ok = id >= 0 && id < a.rows;
+    const bf16 *src = a.table + (size_t)(ok ? id : 0) * width, *two = nullptr;
+    if constexpr (PAIR) {
+        const PairEmbed& p = a.pair;
+        const int seq = p.tok_seq[t], pos = p.tok_pos[t];
+        int64_t row = p.rows.buckets;
+        if (pos > 0) {
+            const bool here = t > 0 && p.tok_seq[t - 1] == seq && p.tok_pos[t - 1] == pos - 1;
+            const int64_t prev = here ? a.ids[t - 1] : (int64_t)p.last[seq];
+            row = (prev % p.rows.buckets * p.rows.mul_prev + id % p.rows.buckets * p.rows.mul_cur) % p.rows.buckets;
+            if (row < 0) row += p.rows.buckets;
+        }
+        two = p.table + (size_t)row * width;
+        if (p.one_each) {
+            __syncthreads();  // every thread has read the token before
+            if (threadIdx.x == 0) p.last[seq] = (int32_t)id;
+        }
+    }
+    auto at = [&](int c) { return ok ? fmaf(__bfloat162float(src[c]), a.scale, PAIR ? __bfloat162float(two[c]) : 0.0f) : 0.0f; };
     float ss = 0.0f;
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
-        const float v = ok ? __bfloat162float(src[c]) * scale : 0.0f;
-        x[t * width + c] = v;
+        const float v = at(c);
+        a.x[t * width + c] = v;
+        if (a.copy) a.copy[t * width + c] = v;
         ss = fmaf(v, v, ss);
     }
-    if (!act) return;
+    if (!a.act) return;
     float r = 1.0f;
-    if (w) r = 1.0f / sqrtf(block_sum_once(ss, sh) / (float)width + eps);
-    for (int c = threadIdx.x; c < width; c += blockDim.x) {
-        const float v = (ok ? __bfloat162float(src[c]) * scale : 0.0f) * r;
-        act[t * ld_act + c] = to_act<A>(w ? v * w[c] : v);
-    }
+    if (a.w) r = 1.0f / sqrtf(block_sum_once(ss, sh) / (float)width + a.eps);
+    A* act = (A*)a.act + t * a.ld_act;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) act[c] = to_act<A>(a.w ? at(c) * r * a.w[c] : at(c));
+}
+
+__global__ void keep_tokens_kernel(const SeqRun* __restrict__ runs, int n, const int64_t* __restrict__ ids, int32_t* __restrict__ last) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) last[runs[i].seq] = (int32_t)ids[runs[i].tok0 + runs[i].n - 1];
 }
 
 __global__ void __launch_bounds__(256) act_rows_kernel(const float* __restrict__ x, int width, __nv_bfloat16* __restrict__ act, int ld_act) {
@@ -98,6 +121,88 @@ template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { 
 template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
 __device__ __forceinline__ float sq4(float4 v, float ss) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss)))); }
 __device__ __forceinline__ void add4(float4& y, float w, float4 v) { y.x = fmaf(w, v.x, y.x); y.y = fmaf(w, v.y, y.y); y.z = fmaf(w, v.z, y.z); y.w = fmaf(w, v.w, y.w); }
+
+// x += y, the sum over depth (DEPTH), the next sublayer's norm.  VEC as below.
+template <typename A, int VEC, bool DEPTH>
+__global__ void __launch_bounds__(512) plain_residual_kernel(const ResidualArgs a) {
+    constexpr int kHeld = VEC == 4 ? 4 : 8;
+    __shared__ float sh[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t row = (size_t)blockIdx.x * a.width;
+    const int width = a.width, step = blockDim.x * VEC;
+    const float* yr = a.y + row;
+    float* xr = a.x + row;
+    A* ar = a.act ? (A*)a.act + (size_t)blockIdx.x * a.ld_act : nullptr;
+    struct Part { float v[VEC]; };
+    auto get = [&](const float* p) {
+        Part r;
+        if constexpr (VEC == 4) { const float4 f = *(const float4*)p; r.v[0] = f.x; r.v[1] = f.y; r.v[2] = f.z; r.v[3] = f.w; }
+        else r.v[0] = *p;
+        return r;
+    };
+    auto put = [&](float* p, const Part& r) {
+        if constexpr (VEC == 4) *(float4*)p = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
+        else *p = r.v[0];
+    };
+    auto sum = [&](int c) {
+        Part s = get(xr + c);
+        const Part y = get(yr + c);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) s.v[e] += y.v[e];
+        if constexpr (DEPTH) {
+            const DepthSum& d = a.depth;
+            put(d.keep + row + c, s);
+            const float own = __ldg(d.c + d.n);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) s.v[e] *= own;
+#pragma unroll 8
+            for (int j = 0; j < d.n; j++) {
+                const Part z = get(d.past + j * d.stride + row + c);
+                const float f = __ldg(d.c + j);
+#pragma unroll
+                for (int e = 0; e < VEC; e++) s.v[e] = fmaf(f, z.v[e], s.v[e]);
+            }
+        }
+        put(xr + c, s);
+        return s;
+    };
+    Part held[kHeld];
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < kHeld; i++) {
+        const int c = threadIdx.x * VEC + i * step;
+        if (c < width) {
+            held[i] = sum(c);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) ss = fmaf(held[i].v[e], held[i].v[e], ss);
+        }
+    }
+    for (int c = threadIdx.x * VEC + kHeld * step; c < width; c += step) {
+        const Part s = sum(c);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) ss = fmaf(s.v[e], s.v[e], ss);
+    }
+    if (!ar) return;
+    const float* wn = a.w_next;
+    const float r = wn ? 1.0f / sqrtf(block_sum_once(ss, sh) / (float)width + a.eps) : 1.0f;
+    auto next = [&](int c, const Part& s) {
+        Part n = s;
+        if (wn) {
+            const Part g = get(wn + c);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) n.v[e] = s.v[e] * r * g.v[e];
+        }
+        if constexpr (VEC == 4) store4<A>(ar + c, make_float4(n.v[0], n.v[1], n.v[2], n.v[3]));
+        else ar[c] = to_act<A>(n.v[0]);
+    };
+#pragma unroll
+    for (int i = 0; i < kHeld; i++) {
+        const int c = threadIdx.x * VEC + i * step;
+        if (c < width) next(c, held[i]);
+    }
+    for (int c = threadIdx.x * VEC + kHeld * step; c < width; c += step) next(c, get(xr + c));
+}
 
 // VEC = 4: rows of a multiple of four elements; a row of up to 16 elements per thread stays in registers between its passes.
 // MOE, PAIR: the output is first made from a mixture's parts (MoeSum) or from two mixers' outputs (PairSum).
@@ -457,22 +562,21 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaArgs a) {
     if (blockIdx.z == 0) delta_keep_inputs<A>(a, run, h, threadIdx.x, 128);
 }
 
-// One warp per (token, head): o / rms(o) * norm * sigmoid(gate)
+// One warp per (token, head)
 template <typename A>
-__global__ void __launch_bounds__(256) delta_output_kernel(const DeltaArgs a) {
+__global__ void __launch_bounds__(256) head_norm_kernel(const HeadNormArgs a) {
     pdl_launch_dependents();
     pdl_wait();
-    const DeltaShape& g = a.g;
     const int t = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (h >= g.heads) return;
-    const float* o = a.o + ((size_t)t * g.heads + h) * g.vdim;
-    const A* gate = (const A*)a.gate + ((size_t)t * g.heads + h) * g.vdim;
+    if (h >= a.heads) return;
+    const float *o = a.o + ((size_t)t * a.heads + h) * a.n, *w = a.w + (size_t)h * a.w_stride;
+    const A* gate = (const A*)a.gate + (size_t)t * a.ld_gate + (size_t)h * a.n;
     float ss = 0.0f;
-    for (int i = lane; i < g.vdim; i += 32) ss = fmaf(o[i], o[i], ss);
+    for (int i = lane; i < a.n; i += 32) ss = fmaf(o[i], o[i], ss);
     ss = warp_sum(ss);
-    const float r = 1.0f / sqrtf(ss / (float)g.vdim + g.eps);
-    A* dst = (A*)a.out + (size_t)t * a.ldo + h * g.vdim;
-    for (int i = lane; i < g.vdim; i += 32) dst[i] = to_act<A>(o[i] * r * a.norm_w[i] * sigmoid_f(act_f<A>(gate[i])));
+    const float r = 1.0f / sqrtf(ss / (float)a.n + a.eps);
+    A* dst = (A*)a.out + (size_t)t * a.ldo + h * a.n;
+    for (int i = lane; i < a.n; i += 32) dst[i] = to_act<A>(o[i] * r * w[i] * sigmoid_f(act_f<A>(gate[i])));
 }
 
 // One new token of every sequence: convolutions, unit vectors, recurrence, norm and gate of one head of one token per CTA.
@@ -743,12 +847,21 @@ int32_t launch_pack(const __nv_bfloat16* src, int rows, int cols, __nv_bfloat16*
     LC_CUDA(cudaGetLastError());
     return LC_OK;
 }
-int32_t launch_embed_rows(const __nv_bfloat16* table, int rows, int width, const int64_t* ids, int T, float scale, const float* w, float eps, float* x, void* act, int ld_act,
-                          bool f32, cudaStream_t s) {
-    const dim3 grid((unsigned)T), block(256);
-    if (scale == 1.0f && !w && !(f32 && act)) LC_CUDA(launch_pdl(embed_rows_kernel, grid, block, 0, s, table, rows, width, ids, x, (bf16*)act, ld_act));
-    else if (f32) LC_CUDA(launch_pdl(embed_norm_kernel<float>, grid, block, 0, s, table, rows, width, ids, scale, w, eps, x, (float*)act, ld_act));
-    else LC_CUDA(launch_pdl(embed_norm_kernel<bf16>, grid, block, 0, s, table, rows, width, ids, scale, w, eps, x, (bf16*)act, ld_act));
+int32_t launch_embed_rows(const EmbedArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)a.T), block(256);
+    auto go = [&](auto kern) -> int32_t {
+        LC_CUDA(launch_pdl(kern, grid, block, 0, s, a));
+        return LC_OK;
+    };
+    if (a.pair.table) return a.f32 ? go(embed_norm_kernel<float, true>) : go(embed_norm_kernel<bf16, true>);
+    if (a.scale == 1.0f && !a.w && !a.copy && !(a.f32 && a.act)) {
+        LC_CUDA(launch_pdl(embed_rows_kernel, grid, block, 0, s, a.table, a.rows, a.width, a.ids, a.x, (bf16*)a.act, a.ld_act));
+        return LC_OK;
+    }
+    return a.f32 ? go(embed_norm_kernel<float, false>) : go(embed_norm_kernel<bf16, false>);
+}
+int32_t launch_keep_tokens(const SeqRun* runs, int n_runs, const int64_t* ids, int32_t* last, cudaStream_t s) {
+    LC_CUDA(launch_pdl(keep_tokens_kernel, dim3((unsigned)((n_runs + 127) / 128)), dim3(128), 0, s, runs, n_runs, ids, last));
     return LC_OK;
 }
 int32_t launch_act_rows(const float* x, int width, int T, void* act, int ld_act, cudaStream_t s) {
@@ -764,6 +877,15 @@ int32_t launch_residual(const ResidualArgs& a, cudaStream_t s) {
         LC_CUDA(launch_pdl(kern, grid, block, 0, s, a));
         return LC_OK;
     };
+    if (!a.w) {
+        LC_CHECK(!moe && !pair, LC_ERR_UNSUPPORTED, "residual sum: a mixture or a pair without an output norm");
+        const bool deep = a.depth.keep != nullptr;
+        if (a.f32) return deep ? (vec ? go(plain_residual_kernel<float, 4, true>) : go(plain_residual_kernel<float, 1, true>))
+                               : (vec ? go(plain_residual_kernel<float, 4, false>) : go(plain_residual_kernel<float, 1, false>));
+        return deep ? (vec ? go(plain_residual_kernel<bf16, 4, true>) : go(plain_residual_kernel<bf16, 1, true>))
+                    : (vec ? go(plain_residual_kernel<bf16, 4, false>) : go(plain_residual_kernel<bf16, 1, false>));
+    }
+    LC_CHECK(!a.depth.keep, LC_ERR_UNSUPPORTED, "residual sum: a sum over depth behind an output norm");
     if (a.f32) {
         if (moe) return vec ? go(residual_kernel<float, 4, true, false>) : go(residual_kernel<float, 1, true, false>);
         if (pair) return vec ? go(residual_kernel<float, 4, false, true>) : go(residual_kernel<float, 1, false, true>);
@@ -785,10 +907,10 @@ int32_t launch_delta_prep(const DeltaArgs& a, cudaStream_t s) {
 }
 int32_t launch_delta_scan(const DeltaArgs& a, cudaStream_t s) { return a.f32 ? scan_dispatch<float>(a, s) : scan_dispatch<__nv_bfloat16>(a, s); }
 int32_t launch_delta_step(const DeltaArgs& a, cudaStream_t s) { return a.f32 ? step_dispatch<float>(a, s) : step_dispatch<__nv_bfloat16>(a, s); }
-int32_t launch_delta_output(const DeltaArgs& a, cudaStream_t s) {
-    const dim3 grid((unsigned)a.T, (unsigned)((a.g.heads + 7) / 8));
-    if (a.f32) LC_CUDA(launch_pdl(delta_output_kernel<float>, grid, dim3(256), 0, s, a));
-    else LC_CUDA(launch_pdl(delta_output_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, a));
+int32_t launch_head_norm(const HeadNormArgs& a, cudaStream_t s) {
+    const dim3 grid((unsigned)a.T, (unsigned)((a.heads + 7) / 8));
+    if (a.f32) LC_CUDA(launch_pdl(head_norm_kernel<float>, grid, dim3(256), 0, s, a));
+    else LC_CUDA(launch_pdl(head_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, a));
     return LC_OK;
 }
 int32_t launch_latent_prep(const LatentArgs& a, cudaStream_t s) {
