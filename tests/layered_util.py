@@ -235,6 +235,92 @@ def munisun_mixed():
                            with_ff(scaled_pair(right=state_space(heads=4, groups=4, state=16, vdim=8, conv=2, norm_groups=1)), 17)])
 
 
+def warm_attention(heads=6, kv_heads=2, dim=20, vdim=12, scale=0.3, softcap=9.0, temp=(0.7, 11), kv_from=None):
+    """Unrotated attention; temp: (coef, every) of the factor on queries."""
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
+    if softcap is not None:
+        m["softcap"] = softcap
+    if temp:
+        m["q_temp"] = dict(zip(("coef", "every"), temp))
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": None}
+
+
+def normed_attention(heads=4, kv_heads=4, dim=28, vdim=20, rot_dims=12, base=700.0, scaling=(3.0, 64, 8.0, 1.0), scale=0.25, window=37):
+    rot = {"dims": rot_dims, "base": base}
+    if scaling:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return {"type": "attention_2", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "rot": rot, "mask": {"size": window}}, "mlp": None}
+
+
+def general_delta(heads=3, dim=20):
+    return {"type": "general_delta", "mixer": {"heads": heads, "dim": dim}, "mlp": None}
+
+
+def nepudra_config(layers, width=104, vocab=131, eps=1e-5, bigram=(77, 31, 1009)):
+    """bigram: (buckets, mul_prev, mul_cur)."""
+    return {"architecture": "Nepudra", "width": width, "vocab": vocab, "norm": {"eps": eps},
+            "embedding": {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))}, "layers": layers}
+
+
+def nepudra_weights(cfg, seed=0, rank=6, depth=0.3):
+    """Random weights, already rounded to bf16.  depth: how much earlier results weigh in the sums behind the layers."""
+    rng = np.random.default_rng(seed)
+    W = cfg["width"]
+    w = {}
+
+    def mat(name, n, k, gain=1.0):
+        w[name] = rng.normal(0, gain / np.sqrt(k), (n, k))
+
+    def gain(name, n=()):
+        w[name] = rng.normal(1, 0.2, n)
+
+    w["embed"] = rng.normal(0, 0.8, (cfg["vocab"], W))
+    w["bigram"] = rng.normal(0, 0.8, (cfg["embedding"]["bigram"]["buckets"] + 1, W))
+    for i, ly in enumerate(cfg["layers"]):
+        m, l, p = ly["mixer"], "l%d." % i, "l%d.mix." % i
+        H, D = m["heads"], m["dim"]
+        gain(l + "norm1")
+        if ly["type"] == "general_delta":
+            for n in "rkvga":
+                mat(p + n, H * D, W)
+            w[p + "a.b"] = rng.normal(0, 1.0, H * D)
+            mat(p + "w1", rank, W)
+            mat(p + "w2", H * D, rank, 2.0)
+            w[p + "w0"] = rng.normal(-1, 2.0, H * D)
+            gain(p + "norm", H * D)
+            mat(p + "o", W, H * D)
+        else:
+            G, E, second = m["kv_heads"], m["vdim"], ly["type"] == "attention_2"
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * E)):
+                if n == "q" or m.get("kv_from") is None:
+                    mat(p + n, rows, W)
+                    w[p + n + ".b"] = rng.normal(0, 0.5, rows)
+                    if second and n != "v":
+                        gain(p + n + ".norm", D)
+            mat(p + "g", H, W)
+            mat(p + "o", W, H * E)
+            if not second:
+                w[p + "o.b"] = rng.normal(0, 0.5, W)
+        if ly["mlp"] is not None:
+            gain(l + "norm2")
+            mat(l + "mlp.gate", ly["mlp"]["ff"], W)
+            mat(l + "mlp.up", ly["mlp"]["ff"], W)
+            mat(l + "mlp.down", W, ly["mlp"]["ff"])
+        w[l + "dwa"] = np.append(rng.normal(0, depth, i + 1), 1.0)
+    gain("final.norm")
+    mat("head", cfg["vocab"], W, 2.0)
+    return {n: bf16_round(a).reshape(np.shape(a)) for n, a in w.items()}
+
+
+def nepudra_mixed():
+    """Every kind of layer more than once, with and without feed-forward, a cache read by two other layers, sizes that differ."""
+    return nepudra_config([general_delta(), with_ff(warm_attention(), 40), normed_attention(), with_ff(general_delta(heads=2, dim=36), 17),
+                           warm_attention(kv_from=1, temp=(0.4, 64), softcap=30.0, scale=0.5), with_ff(normed_attention(heads=8, kv_heads=2, dim=16, vdim=24, rot_dims=16, window=16, scaling=None), 24),
+                           with_ff(warm_attention(heads=2, kv_from=1, temp=None, softcap=None), 31)])
+
+
 def weights(cfg, seed=0, decay_rank=5, gate_rank=7, spread=1.0):
     """Random weights, already rounded to bf16.  Products keep about unit size; decays range from slow to fast."""
     rng = np.random.default_rng(seed)
@@ -302,7 +388,7 @@ def engine(lc, cfg, w, dtype="float32", **kw):
     from leafcutterllm_b200 import Engine
     eng = Engine.from_config(cfg, dtype=dtype, **kw)
     for n, a in w.items():
-        eng.set_tensor(n, lc.TYPE_BF16, tuple(reversed(a.shape)), bf16_bytes(a))
+        eng.set_tensor(n, lc.TYPE_BF16, tuple(reversed(a.shape)) or (1,), bf16_bytes(a))
     eng.finalize()
     return eng
 

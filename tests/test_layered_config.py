@@ -172,6 +172,81 @@ def test_norm_in_parts_and_bounded_scores_by_definition():
     assert np.isclose(p, 1 / (1 + np.exp(-2 * 2 * np.tanh(4.5))))
 
 
+@pytest.mark.parametrize("cuts", [[1] * 60, [2, 5, 1, 9, 6, 37], [58, 2]])
+def test_plain_nepudra_in_portions_equals_the_whole(cuts):
+    cfg = U.nepudra_mixed()
+    m = P.plain_model(cfg, U.nepudra_weights(cfg))
+    toks = U.tokens(60, cfg["vocab"])
+    whole = m.forward(toks, m.new_state())
+    st, parts, at = m.new_state(), [], 0
+    for c in cuts:
+        parts.append(m.forward(toks[at : at + c], st))
+        at += c
+    assert np.abs(np.concatenate(parts) - whole).max() < 1e-9
+
+
+def test_general_delta_rule_by_definition():
+    """Without removal it is a decayed sum; with full removal and no decay a repeated unit key replaces what it wrote before."""
+    rng = np.random.default_rng(9)
+    r, k, v = rng.normal(size=(7, 5)), rng.normal(size=(7, 5)), rng.normal(size=(7, 5))
+    w = rng.uniform(0.5, 1.0, (7, 5))
+    got = P.general_delta_rule(r, k, v, w, np.zeros((7, 5)), np.zeros((5, 5)))
+    for t in range(7):
+        want = sum((r[t] * np.prod(w[s + 1 : t + 1], axis=0)) @ k[s] * v[s] for s in range(t + 1))
+        assert np.allclose(got[t], want)
+    key = np.tile(P.unit(k[:1], 0.0), (7, 1))
+    assert np.allclose(P.general_delta_rule(key, key, v, np.ones((7, 5)), np.ones((7, 5)), np.zeros((5, 5)), 0.0), v)
+    # removal and decay both look at the state before the token
+    S, u = rng.normal(size=(5, 5)), P.unit(k[0])
+    want = np.diag(w[0]) @ S - np.outer(0.3 * u, u @ S) + np.outer(k[0], v[0])
+    assert np.allclose(P.general_delta_rule(r[:1], k[:1], v[:1], w[:1], np.full((1, 5), 0.3), S.copy())[0], want.T @ r[0])
+
+
+def test_query_temperature_and_token_pairs_by_definition():
+    f = P.query_temperature(np.arange(9), {"coef": 0.5, "every": 4})
+    assert np.allclose(f, [1, 1, 1] + [1 + 0.5 * np.log(2)] * 4 + [1 + 0.5 * np.log(3)] * 2)
+    rows = {"buckets": 10, "mul_prev": 3, "mul_cur": 7}
+    assert P.pair_rows([4, 5, 0], None, rows) == [10, (12 + 35) % 10, 5] and P.pair_rows([4], 5, rows) == [(15 + 28) % 10]
+
+
+def test_rotation_of_half_pairs_takes_the_scaled_frequencies():
+    rot = {"dims": 8, "base": 50.0, "scaling": {"factor": 4.0, "original": 32, "fast": 4.0, "slow": 1.0}}
+    f, mag = P.yarn_frequencies(rot)
+    x = np.random.default_rng(1).normal(size=(1, 1, 11))
+    y = P.rotate_half_pairs(x, [5], rot)[0, 0]
+    assert np.allclose(y[8:], x[0, 0, 8:]) and np.isclose(y[1], mag * (x[0, 0, 1] * np.cos(5 * f[1]) - x[0, 0, 5] * np.sin(5 * f[1])))
+    plain = {"dims": 8, "base": 50.0}
+    assert np.allclose(P.rotate_half_pairs(x, [5], plain), P.rotate_halves(x, [5], 8, 50.0))
+
+
+def broken_nepudra(change):
+    cfg = copy.deepcopy(U.nepudra_mixed())
+    change(cfg)
+    return cfg
+
+
+@pytest.mark.parametrize("change,text", [
+    (lambda c: c["embedding"].pop("bigram"), "bigram"),
+    (lambda c: c["embedding"]["bigram"].update(buckets=0), "buckets"),
+    (lambda c: c["embedding"]["bigram"].update(mul_cur=1.5), "factor"),
+    (lambda c: c["layers"][0].update(type="channel_delta"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mixer"].pop("dim"), "dim"),
+    (lambda c: c["layers"][1]["mixer"]["q_temp"].update(every=0), "every"),
+    (lambda c: c["layers"][1]["mixer"].update(softcap=-1), "softcap"),
+    (lambda c: c["layers"][1]["mixer"].pop("vdim"), "vdim"),
+    (lambda c: c["layers"][2]["mixer"]["rot"].update(dims=30), "rotated"),
+    (lambda c: c["layers"][2]["mixer"]["mask"].update(size=0), "size"),
+    (lambda c: c["layers"][4]["mixer"].update(kv_from=0), "cannot read"),
+    (lambda c: c["layers"][4]["mixer"].update(kv_from=4), "earlier"),
+    (lambda c: c["layers"][6]["mixer"].update(kv_from=4), "cannot read"),
+    (lambda c: c["layers"][6]["mlp"].update(kind="moe"), "unknown kind"),
+])
+def test_nepudra_config_errors_are_named(lc, change, text):
+    with pytest.raises(lc.LeafcutterError) as e:
+        lc.Engine.from_config(broken_nepudra(change))
+    assert text in str(e.value)
+
+
 def broken_munisun(change):
     cfg = copy.deepcopy(U.munisun_mixed())
     change(cfg)

@@ -18,7 +18,7 @@ def mixed_config():
                      U.with_ff(U.latent(heads=2, dim=16, rot_dim=8, vdim=24, kv_rank=48, q_rank=20, scaling=None), 56)])
 
 
-@pytest.fixture(scope="module", params=["varasun", "tenetar", "munisun"])
+@pytest.fixture(scope="module", params=["varasun", "tenetar", "munisun", "nepudra"])
 def model(request):
     if request.param == "varasun":
         cfg = mixed_config()
@@ -26,6 +26,9 @@ def model(request):
     elif request.param == "munisun":
         cfg = U.munisun_mixed()
         w = U.munisun_weights(cfg, 13, fixed_choice=True)
+    elif request.param == "nepudra":
+        cfg = U.nepudra_mixed()
+        w = U.nepudra_weights(cfg, 14)
     else:
         cfg = U.tenetar_mixed()
         w = U.tenetar_weights(cfg, 12, fixed_choice=True)
@@ -75,7 +78,7 @@ def test_first_tokens(gpu, model, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("design", ["varasun", "tenetar", "munisun"])
+@pytest.mark.parametrize("design", ["varasun", "tenetar", "munisun", "nepudra"])
 def test_a_call_longer_than_one_pass(gpu, design, dtype):
     """More tokens in one call than a pass takes (2048): the second pass continues from the first one's cache and state."""
     if design == "varasun":
@@ -86,6 +89,10 @@ def test_a_call_longer_than_one_pass(gpu, design, dtype):
                                                      experts=6, top=2, groups=3, keep=2),
                                 U.normed_pair(U.conv_attention(heads=2, kv_heads=1, dim=8, vdim=8), U.lightning((0.9, 0.999), dim=8, vdim=8))], width=32, vocab=40)
         w = U.munisun_weights(cfg, 3, fixed_choice=True)
+    elif design == "nepudra":
+        cfg = U.nepudra_config([U.general_delta(heads=2, dim=16), U.warm_attention(heads=2, kv_heads=1, dim=8, vdim=8, temp=(0.3, 500)),
+                                U.normed_attention(heads=2, kv_heads=1, dim=8, vdim=8, rot_dims=4, window=700)], width=32, vocab=40)
+        w = U.nepudra_weights(cfg, 3)
     else:
         cfg = U.tenetar_config([U.with_experts(U.attention(heads=2, kv_heads=1, dim=8, vdim=8, window=700, keep_first=70), experts=5, identity=1, top=2, groups=2, keep=1),
                                 U.attention(heads=2, kv_heads=1, dim=8, vdim=8, window=3000, keep_first=0, kv_from=0)], width=32, vocab=40)
@@ -260,7 +267,7 @@ def test_long_decoding_and_greedy_generation(gpu, model):
 
 
 @pytest.mark.parametrize("n_seqs", [1, 5, 20, 70])
-@pytest.mark.parametrize("design", ["varasun", "tenetar", "munisun"])
+@pytest.mark.parametrize("design", ["varasun", "tenetar", "munisun", "nepudra"])
 def test_decode_batches_of_every_product_form(gpu, design, n_seqs):
     """Decode steps whose token count selects different tiles, at contexts on both sides of page and key-tile edges."""
     if design == "varasun":
@@ -271,6 +278,11 @@ def test_decode_batches_of_every_product_form(gpu, design, n_seqs):
                                 U.with_gated_experts(U.normed_pair(U.conv_attention(heads=20, kv_heads=2, dim=32, vdim=32), U.lightning((0.9, 0.999, 0.5), dim=64, vdim=32)),
                                                      experts=8, top=3, groups=4, keep=3, ff=130)], width=128, side=40)
         w = U.munisun_weights(cfg, 4, fixed_choice=True)
+    elif design == "nepudra":
+        cfg = U.nepudra_config([U.with_ff(U.warm_attention(heads=20, kv_heads=2, dim=32, vdim=32, temp=(0.5, 20)), 136), U.general_delta(heads=4, dim=64),
+                                U.with_ff(U.warm_attention(heads=20, kv_heads=2, dim=32, vdim=32, kv_from=0), 72),
+                                U.normed_attention(heads=12, kv_heads=3, dim=64, vdim=32, rot_dims=64, window=64)], width=128)
+        w = U.nepudra_weights(cfg, 4)
     else:
         cfg = U.tenetar_config([U.with_ff(U.attention(heads=20, kv_heads=2, dim=32, vdim=32, window=64, keep_first=16), 136),
                                 U.with_experts(U.attention(heads=20, kv_heads=2, dim=32, vdim=32, window=150, keep_first=0, kv_from=0), experts=6, identity=2, top=3, groups=4,
@@ -324,13 +336,14 @@ def test_checkpoint_directory_and_trace_runner(gpu, model, tmp_path, monkeypatch
 def test_incomplete_models_are_named(gpu, model):
     cfg, w, _ = model
     dropped = {"Tenetar": ("l1.mlp.e3.down", "l2.mlp.correction", "l0.norm1b", "l3.mix.q.norm"), "Varasun": ("l1.mix.uk", "l0.mix.a1"),
-               "Munisun": ("l0.mix.left.k.conv", "l1.mix.right.conv.b", "l1.mix.left.g", "l2.mlp.e9.gate", "l3.side.norm", "side.embed", "l0.mix.right.out")}[cfg["architecture"]]
+               "Munisun": ("l0.mix.left.k.conv", "l1.mix.right.conv.b", "l1.mix.left.g", "l2.mlp.e9.gate", "l3.side.norm", "side.embed", "l0.mix.right.out"),
+               "Nepudra": ("bigram", "l0.mix.w1", "l0.mix.a.b", "l1.mix.k.b", "l1.mix.g", "l1.mix.o.b", "l2.mix.k.norm", "l3.norm2", "l4.dwa", "l4.mix.q.b")}[cfg["architecture"]]
     for drop, status in [(n, -6) for n in dropped + ("final.norm",)]:
         with pytest.raises(gpu.LeafcutterError) as e:
             U.engine(gpu, cfg, {n: a for n, a in w.items() if n != drop})
         assert e.value.status == status and drop in str(e.value)
     wrong = dict(w)
-    name = {"Tenetar": "l2.mlp.e1.up", "Varasun": "l1.mix.uv", "Munisun": "l1.mix.right.in"}[cfg["architecture"]]
+    name = {"Tenetar": "l2.mlp.e1.up", "Varasun": "l1.mix.uv", "Munisun": "l1.mix.right.in", "Nepudra": "l3.mix.w2"}[cfg["architecture"]]
     wrong[name] = w[name][:-1]
     with pytest.raises(gpu.LeafcutterError) as e:
         U.engine(gpu, cfg, wrong)
