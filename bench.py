@@ -300,9 +300,10 @@ def moe_decode(lc, synth, local: int, n_seqs: int = 16, prompt_len: int = 1024, 
 
 
 def layered_leg(lc, synth, local: int, sizes=("1b", "7b"), prompt_len: int = PROMPT_LEN, steps: int = 32, batches=(1, 16, 64), llama: bool = True, pattern: str = "",
-                designs=("varasun",), tenetar_pattern: str = "", munisun_pattern: str = "") -> dict:
+                designs=("varasun",), tenetar_pattern: str = "", munisun_pattern: str = "", nepudra_pattern: str = "") -> dict:
     """Varasun-shaped models (gated delta rule and latent attention layers, bf16, random weights) and Tenetar-shaped ones (windowed
-    attention with shared caches, mixtures of experts) or Munisun-shaped ones (attention beside a linear recurrence, mixtures) beside Llama-shaped models of the same width, depth, heads and FFN width
+    attention with shared caches, mixtures of experts), Munisun-shaped ones (attention beside a linear recurrence, mixtures) or
+    Nepudra-shaped ones (a delta rule with separate removal, attention of two kinds, sums over depth) beside Llama-shaped models of the same width, depth, heads and FFN width
     (16-bit and Q4_K weights; with Tenetar also a Llama-shaped mixture of the same experts, Q4_K): prefill of one prompt and decode
     steps at several batch sizes, all contexts of prompt_len tokens.  The weights of a step exceed L2, so nothing is flushed
     between steps."""
@@ -313,6 +314,7 @@ def layered_leg(lc, synth, local: int, sizes=("1b", "7b"), prompt_len: int = PRO
     tenetar_pattern = tenetar_pattern or "dmmmmsss"
     pattern = pattern or "dddaddda"
     munisun_pattern = munisun_pattern or "ldsmlmsmlmsmlmsm"
+    nepudra_pattern = nepudra_pattern or "gngwgngs"
     out = {"prompt_len": prompt_len, "pattern": pattern, "peak_gbs": peak, "peak_source": which}
 
     def measure(build, vocab):
@@ -364,6 +366,9 @@ def layered_leg(lc, synth, local: int, sizes=("1b", "7b"), prompt_len: int = PRO
             ex = {k: v for k, v in experts[size].items() if k not in ("identity", "shared_ff")}
             us = synth.munisun_spec(size, sh["width"], munisun_pattern, sh["ff"], 32000, sh["heads"], **ex)
             out[size]["munisun"] = dict(measure(lambda b: synth.build_layered_engine(us, max_seq_len=cap, max_seqs=b, device=local), 32000), pattern=munisun_pattern)
+        if "nepudra" in designs:
+            ns = synth.nepudra_spec(size, sh["width"], nepudra_pattern, sh["ff"], 32000, sh["heads"], experts[size]["kv_heads"])
+            out[size]["nepudra"] = dict(measure(lambda b: synth.build_layered_engine(ns, max_seq_len=cap, max_seqs=b, device=local), 32000), pattern=nepudra_pattern)
         if llama:
             for tag, typ in (("llama_f16", lc.TYPE_F16), ("llama_q4k", lc.TYPE_Q4_K)):
                 ls = synth.ModelSpec(size + tag, len(pattern), sh["width"], sh["heads"], sh["heads"], sh["ff"], 32000, 10000.0, typ, typ, typ)
@@ -878,9 +883,10 @@ def main():
     ap.add_argument("--layered-sizes", default="1b,7b", help="--only layered: which sizes")
     ap.add_argument("--layered-batches", default="1,16,64", help="--only layered: sequences per decode step")
     ap.add_argument("--layered-pattern", default="", help="--only layered: one letter per layer (d = gated delta rule, a = latent attention)")
-    ap.add_argument("--layered-designs", default="varasun", help="--only layered: which designs (varasun,tenetar,munisun)")
+    ap.add_argument("--layered-designs", default="varasun", help="--only layered: which designs (varasun,tenetar,munisun,nepudra)")
     ap.add_argument("--tenetar-pattern", default="", help="--only layered: one letter per Tenetar layer (d = dense feed-forward, m = mixture, s = mixture on the last own cache)")
     ap.add_argument("--munisun-pattern", default="", help="--only layered: two letters per Munisun layer (s = beside a state space, l = beside lightning attention; then d = dense feed-forward, m = mixture, n = none)")
+    ap.add_argument("--nepudra-pattern", default="", help="--only layered: one letter per Nepudra layer (g = delta rule with separate removal, w = attention over everything, s = the same on the last w's cache, n = windowed attention)")
     ap.add_argument("--no-llama", action="store_true", help="--only layered: skip the Llama-shaped models")
     ap.add_argument("--tp", type=int, default=8, help="--only tp-ranks: ranks the model is cut over")
     ap.add_argument("--profile-range", action="store_true", help="bracket the timed decode loop with cudaProfilerStart/Stop")
@@ -925,7 +931,7 @@ def main():
         lc._capi.check(lc.load().lc_set_device(0))
         print(json.dumps(layered_leg(lc, synth, 0, sizes=tuple(args.layered_sizes.split(",")), prompt_len=args.prompt_len, steps=min(args.steps, 32),
                                      batches=tuple(int(v) for v in args.layered_batches.split(",")), llama=not args.no_llama, pattern=args.layered_pattern,
-                                     designs=tuple(args.layered_designs.split(",")), tenetar_pattern=args.tenetar_pattern, munisun_pattern=args.munisun_pattern)))
+                                     designs=tuple(args.layered_designs.split(",")), tenetar_pattern=args.tenetar_pattern, munisun_pattern=args.munisun_pattern, nepudra_pattern=args.nepudra_pattern)))
     elif args.only == "tcgen05-probe":
         import ctypes as C
         import leafcutterllm_b200 as lc

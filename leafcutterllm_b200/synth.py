@@ -120,18 +120,44 @@ class LayeredSpec:
             return name, TYPE_BF16, (cols, rows), "normal"
         def vec(name, n, kind="ones"):
             return name, TYPE_BF16, (n,), kind
-        munisun = c["architecture"] == "Munisun"
+        munisun, nepudra = c["architecture"] == "Munisun", c["architecture"] == "Nepudra"
         gain = "zeros" if munisun else "ones"  # Munisun's layer norms are stored around zero
         yield mat("embed", c["vocab"], W)
+        if nepudra:
+            yield mat("bigram", c["embedding"]["bigram"]["buckets"] + 1, W)
         if munisun:
             yield mat("side.embed", c["vocab"], len(c["layers"]) * c["token_side"]["dim"])
         for i, ly in enumerate(c["layers"]):
             m, p = ly["mixer"], f"l{i}.mix."
-            H, D, E = (0, 0, 0) if munisun else (m["heads"], m["dim"], m["vdim"])
-            both = ("",) if c["architecture"] == "Varasun" else ("", "b")  # norms on outputs only, or on inputs and outputs
+            H, D, E = (0, 0, 0) if munisun else (m["heads"], m["dim"], m.get("vdim", m["dim"]))
+            both = ("", "b") if c["architecture"] in ("Tenetar", "Munisun") else ("",)  # norms on inputs and outputs, or on one of them
+            wide = 1 if nepudra else W
             for end in both:
-                yield vec(f"l{i}.norm1{end}", W, gain)
-            if munisun:
+                yield vec(f"l{i}.norm1{end}", wide, gain)
+            if nepudra:
+                yield vec(f"l{i}.dwa", i + 2)
+            if ly["type"] == "general_delta":
+                for t in "rkvga":
+                    yield mat(p + t, H * D, W)
+                yield vec(p + "a.b", H * D, "normal")
+                yield mat(p + "w1", self.decay_rank, W)
+                yield mat(p + "w2", H * D, self.decay_rank)
+                yield vec(p + "w0", H * D, "normal")
+                yield vec(p + "norm", H * D)
+                yield mat(p + "o", W, H * D)
+            elif nepudra:
+                G, second = m["kv_heads"], ly["type"] == "attention_2"
+                for t, n in (("q", H * D), ("k", G * D), ("v", G * E)):
+                    if t == "q" or "kv_from" not in m:
+                        yield mat(p + t, n, W)
+                        yield vec(p + t + ".b", n, "normal")
+                        if second and t != "v":
+                            yield vec(p + t + ".norm", D)
+                yield mat(p + "g", H, W)
+                yield mat(p + "o", W, H * E)
+                if not second:
+                    yield vec(p + "o.b", W, "normal")
+            elif munisun:
                 a, r, left, right = m["left"], m["right"], p + "left.", p + "right."
                 nq, nk, nv, inner = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], a["kv_heads"] * a["vdim"], r["heads"] * r["vdim"]
                 for t, n in (("q", nq), ("k", nk), ("v", nv)):
@@ -198,7 +224,7 @@ class LayeredSpec:
             if mlp is None:
                 continue
             for end in both:
-                yield vec(f"l{i}.norm2{end}", W, gain)
+                yield vec(f"l{i}.norm2{end}", wide, gain)
             if mlp["kind"] == "moe":
                 r, F, SF = mlp["router"], mlp["expert"]["ff"], mlp.get("shared", {}).get("ff", 0)
                 n = r["experts"] + r.get("identity", 0)
@@ -220,7 +246,7 @@ class LayeredSpec:
                 yield mat(p + "gate", F, W)
             yield mat(p + "up", F, W)
             yield mat(p + "down", W, F)
-        yield vec("final.norm", W, gain)
+        yield vec("final.norm", 1 if nepudra else W, gain)
         yield mat("head", c["vocab"], W)
 
 
@@ -272,6 +298,28 @@ def munisun_spec(name: str, width: int, pattern: str, ff: int, vocab: int, heads
         moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
         layers.append({"type": "parallel" if kind == "s" else "parallel_2", "mixer": mixer, "mlp": {"d": {"kind": "dense", "ff": ff}, "m": moe, "n": None}[mlp]})
     return LayeredSpec(name, {"architecture": "Munisun", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5}, "token_side": {"dim": side}, "layers": layers})
+
+
+def nepudra_spec(name: str, width: int, pattern: str, ff: int, vocab: int, heads: int, kv_heads: int, head_dim: int = 128, state_dim: int = 64, rank: int = 64,
+                 window: int = 1024, buckets: int = 32003) -> LayeredSpec:
+    """pattern: one letter per layer: g = delta rule with separate removal, w = unrotated attention over everything, s = the same on the
+    last w's keys and values, n = windowed attention with norms per head; each with a gated feed-forward of `ff`."""
+    layers, own = [], 0
+    for i, ch in enumerate(pattern):
+        mixer = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5}
+        if ch == "g":
+            mixer = {"heads": width // state_dim, "dim": state_dim}
+        elif ch == "n":
+            mixer.update(mask={"size": window}, rot={"dims": head_dim, "base": 500000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+        else:
+            mixer.update(softcap=50.0, q_temp={"coef": 0.1, "every": 4096})
+            if ch == "s":
+                mixer["kv_from"] = own
+            else:
+                own = i
+        layers.append({"type": {"g": "general_delta", "n": "attention_2"}.get(ch, "attention"), "mixer": mixer, "mlp": {"kind": "dense", "ff": ff}})
+    config = {"architecture": "Nepudra", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "embedding": {"bigram": {"buckets": buckets, "mul_prev": 40503, "mul_cur": 1}}, "layers": layers}
+    return LayeredSpec(name, config, rank)
 
 
 def build_layered_engine(spec: LayeredSpec, seed: int = WEIGHT_SEED, **engine_kwargs):
