@@ -58,7 +58,7 @@ struct DenseParams {
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // The epilogue is a template parameter of the kernels; kEpiAny stands for the rarer elementwise ones, told apart at run time.
 constexpr int kEpiAny = -1;
-constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS || epi == DENSE_SIGMOID_DECAY ? kEpiAny : epi; }
+constexpr int epi_class(int epi) { return epi == DENSE_LOG_DECAY || epi == DENSE_LOGITS ? kEpiAny : epi; }
 constexpr bool epi_splits(int epi) { return epi == DENSE_SPLIT_RELU2 || epi == DENSE_SPLIT_SILU || epi == DENSE_SPLIT_TANH; }
 constexpr bool epi_gated(int epi) { return epi == DENSE_GATED_SILU || epi == DENSE_GATED_GELU; }
 __device__ __forceinline__ float silu_of(float g) { return g / (1.0f + expf(-g)); }
@@ -82,9 +82,9 @@ __device__ __forceinline__ float dense_epilogue(const DenseParams& p, bool secon
     else if constexpr (EPI == DENSE_SPLIT_SILU) return second && row < p.act_end ? silu_of(y) : y;
     else if constexpr (EPI == DENSE_SPLIT_TANH) return second && row < p.act_end ? tanhf(y) : y;
     else if constexpr (EPI == DENSE_BIAS) return y + eb;
+    else if constexpr (EPI == DENSE_SIGMOID_DECAY) return __fdividef(-p.scale, 1.0f + __expf(-(y + eb)));
     else if constexpr (EPI == kEpiAny) {
         if (p.epi == DENSE_LOG_DECAY) return -ea * softplus_f(y + eb);
-        if (p.epi == DENSE_SIGMOID_DECAY) return -p.scale / (1.0f + expf(-(y + eb)));
         const float v = y * p.scale;
         return p.cap > 0.0f ? p.cap * tanhf(v / p.cap) : v;
     } else return y;
@@ -628,6 +628,7 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
             case DENSE_GATED_GELU: return go(dense_f32_kernel<DENSE_GATED_GELU>);
             case DENSE_BIAS: return go(dense_f32_kernel<DENSE_BIAS>);
             case DENSE_SPLIT_TANH: return go(dense_f32_kernel<DENSE_SPLIT_TANH>);
+            case DENSE_SIGMOID_DECAY: return go(dense_f32_kernel<DENSE_SIGMOID_DECAY>);
             default: return go(dense_f32_kernel<kEpiAny>);
         }
     }
@@ -667,6 +668,7 @@ int32_t launch_dense(const DenseArgs& a, DenseWorkspace& ws, cudaStream_t s) {
         case DENSE_GATED_GELU: return launch_tiles<false, DENSE_GATED_GELU>(NT, a, *tx, p, s);
         case DENSE_BIAS: return launch_tiles<false, DENSE_BIAS>(NT, a, *tx, p, s);
         case DENSE_SPLIT_TANH: return launch_tiles<false, DENSE_SPLIT_TANH>(NT, a, *tx, p, s);
+        case DENSE_SIGMOID_DECAY: return launch_tiles<false, DENSE_SIGMOID_DECAY>(NT, a, *tx, p, s);
         default: return launch_tiles<false, kEpiAny>(NT, a, *tx, p, s);
     }
 }

@@ -4,16 +4,17 @@
 //   general_scan_kernel   runs of few tokens, and models in true 32-bit: token by token
 //   general_step_kernel   one token per sequence: recurrence, norm and gate of one head of one token per CTA; the state is read and
 //                         written once and stays in registers between
-//   general_chunk_kernel, general_carry_kernel   longer runs, kGeneralChunk tokens at a time:
+//   general_chunk_kernel, general_carry_kernel, general_read_kernel   longer runs, kGeneralChunk tokens at a time:
 // Inside a chunk let G_t be the sum of the log decays up to token t (per key channel) and S0 the state before the chunk.  Unrolled,
 //   z_t = (e^G_(t-1) u_t)^T S0 + sum_(s < t) (Auk_ts v_s - Aub_ts z_s),   Axy_ts = sum_d x_t e^(G_(t-1) - G_s) y_s,
 //   o_t = (e^G_t r_t)^T S0 + sum_(s <= t) (Brk_ts v_s - Brb_ts z_s),      Brx_ts = sum_d r_t e^(G_t - G_s) x_s.
 // Solving the triangular system for its two right-hand sides, Z = W S0 + Y with
 //   W = (I + Aub)^-1 (e^G_(t-1) u),   Y = (I + Aub)^-1 Auk V,
-// turns the chunk into one product per state and value column:
-//   [S; O] = [M; R] S0 + [C; P],   M = diag(e^G_end) - Bh^T W,  C = Kh^T V - Bh^T Y,  R = e^G r - Brb W,  P = Brk V - Brb Y,
+// makes the chunk linear in the state before it:
+//   S = M S0 + C,  O = R S0 + P,   M = diag(e^G_end) - Bh^T W,  C = Kh^T V - Bh^T Y,  R = e^G r - Brb W,  P = Brk V - Brb Y,
 // with Kh, Bh = e^(G_end - G_s) k_s, b_s.  general_chunk_kernel leaves M, R, C and P (all chunks of all heads at once),
-// general_carry_kernel walks the chunks (one CTA per run, head and 32 value columns).
+// general_carry_kernel walks the chunks' states (one CTA per run, head and 32 value columns), general_read_kernel makes the read-outs
+// (all at once again), their norm and gate.
 // The exponents are taken relative to the chunk's middle, G_t - G_m and G_m - G_s: with log decays of at most `decay_scale` per token
 // they stay below 16 decay_scale, so every factor is an ordinary number.
 #include <algorithm>
@@ -205,28 +206,43 @@ __global__ void __launch_bounds__(THREADS) general_step_kernel(const GeneralArgs
 }
 
 // ---- chunks -------------------------------------------------------------------------------------------------------------------
-constexpr int kT = kGeneralChunk, kPitch = kT + 4, kHalves = kDeltaChunk / kT, kThreads = 384, kWarps = kThreads / 32;
-// What general_chunk_kernel leaves of one (chunk, head), in floats: rows 0 .. dp - 1 belong to the state, dp .. dp + 31 to the tokens.
+constexpr int kT = kGeneralChunk, kPitch = kT + 4, kHalves = kDeltaChunk / kT;
+// What general_chunk_kernel leaves of one (chunk, head), in floats.
 struct ItemLayout {
     int dp;
-    __host__ __device__ int rows() const { return dp + kT; }
-    __host__ __device__ size_t co() const { return (size_t)dp * rows(); }           // M | R: [dp][rows] (transposed); C | P: [dp / 32][rows][32]
-    __host__ __device__ size_t size() const { return 2 * co(); }
+    __host__ __device__ size_t m() const { return 0; }                             // [dp][dp], transposed
+    __host__ __device__ size_t c() const { return (size_t)dp * dp; }               // [dp / 32][dp][32]; replaced by S0
+    __host__ __device__ size_t r() const { return (size_t)2 * dp * dp; }           // [dp][kT], transposed
+    __host__ __device__ size_t p() const { return r() + (size_t)dp * kT; }         // [kT][dp]
+    __host__ __device__ size_t size() const { return p() + (size_t)dp * kT; }
 };
 
 __device__ __forceinline__ void get4(float (&x)[4], const float* p) {
     const float4 f = *(const float4*)p;
     x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w;
 }
+// A warp's lanes over 4 x 4 tiles: LaneGrid<16> 2 rows of tiles by 16 columns, <8> 4 by 8.  Neighbouring lanes share a column and
+// every other lane a row, so that 16-byte loads of either operand reach the banks two lanes at a time.
+template <int COLS>
+struct LaneGrid {
+    static constexpr int kRows = 32 / COLS;
+    __device__ static __forceinline__ int row(int lane) { return (lane & 1) | (COLS == 8 ? (lane >> 4) << 1 : 0); }
+    __device__ static __forceinline__ int col(int lane) { return (lane >> 1) & (COLS - 1); }
+};
+constexpr int cols_per_warp(int dp) { return dp >= 64 ? 16 : 8; }
+constexpr int chunk_threads(int dp) { return dp <= 64 ? 192 : 384; }
+constexpr int chunk_ctas(int dp) { return dp <= 64 ? 3 : 1; }
 
 template <int DP>
-__global__ void __launch_bounds__(kThreads, DP <= 64 ? 2 : 1) general_chunk_kernel(const GeneralArgs a, float* __restrict__ scratch) {
-    constexpr int kQuads = (DP / 4 + kWarps - 1) / kWarps;  // fours of channels per warp
+__global__ void __launch_bounds__(chunk_threads(DP), chunk_ctas(DP)) general_chunk_kernel(const GeneralArgs a, float* __restrict__ scratch) {
+    constexpr int kThreads = chunk_threads(DP), kWarps = kThreads / 32, kQuads = (DP / 4 + kWarps - 1) / kWarps;  // fours of channels per warp
+    typedef LaneGrid<cols_per_warp(DP)> Lanes;
+    constexpr int kColBlocks = DP / 4 / cols_per_warp(DP);
     extern __shared__ __align__(16) float sm[];
-    // channel-major [DP][kPitch]: u e^(G_(t-1) - G_m), r e^(G_t - G_m), k e^(G_m - G_t), b e^(G_m - G_t)
-    float *s_u = sm, *s_r = s_u + DP * kPitch, *s_k = s_r + DP * kPitch, *s_b = s_k + DP * kPitch;
-    float *s_v = s_b + DP * kPitch, *s_x = s_v + kT * DP;                             // [kT][DP] v; [kT][2 DP] W | Y
-    float *s_auk = s_x + 2 * kT * DP, *s_aub = s_auk + kT * kPitch, *s_brk = s_aub + kT * kPitch, *s_brb = s_brk + kT * kPitch;
+    // channel-major [DP][kPitch]: u e^(G_(t-1) - G_m), r e^(G_t - G_m), k e^(G_m - G_t), b e^(G_m - G_t); the first two are read side by side
+    float *s_u = sm, *s_r = s_u + DP * kPitch + 8, *s_k = s_r + DP * kPitch, *s_b = s_k + DP * kPitch;
+    float *s_v = s_b + DP * kPitch, *s_y = s_v + kT * DP, *s_w = s_u;                 // [kT][DP] v, Y, W (in place of u)
+    float *s_auk = s_y + kT * DP, *s_aub = s_auk + kT * kPitch, *s_brk = s_aub + kT * kPitch, *s_brb = s_brk + kT * kPitch;
     float *s_cm = s_brb + kT * kPitch, *s_ce = s_cm + DP, *s_ge = s_ce + DP;          // e^G_m, e^(G_end - G_m), e^G_end
     float* s_len = s_ge + DP;                                                         // [kWarps][32]
     pdl_launch_dependents();
@@ -252,11 +268,11 @@ __global__ void __launch_bounds__(kThreads, DP <= 64 ? 2 : 1) general_chunk_kern
         const bool ok = lane < n;
         const size_t tok = tok0 + (ok ? lane : 0);
         const float *p = a.proj + tok * g.ld + h * dim, *l = a.log_decay + tok * g.heads * dim + h * dim, *ab = a.a_bias + h * dim;
-        float k[kQuads][4], ss = 0.0f;
+        float k[kQuads][4], ld[kQuads][4], ss = 0.0f;
 #pragma unroll
         for (int i = 0; i < kQuads; i++) {
             const int d = 4 * (warp + i * kWarps);
-            if (d < DP) four(p + g.off_k, d, ok, k[i]);
+            if (d < DP) { four(p + g.off_k, d, ok, k[i]); four(l, d, ok, ld[i]); }
             else k[i][0] = k[i][1] = k[i][2] = k[i][3] = 0.0f;
 #pragma unroll
             for (int j = 0; j < 4; j++) ss = fmaf(k[i][j], k[i][j], ss);
@@ -277,174 +293,209 @@ __global__ void __launch_bounds__(kThreads, DP <= 64 ? 2 : 1) general_chunk_kern
         for (int i = 0; i < kQuads; i++) {
             const int d0 = 4 * (warp + i * kWarps);
             if (d0 >= DP) break;
-            float r[4], ld[4], ra[4], bias[4];
+            float r[4], ra[4], bias[4], G[4];
             four(p, d0, ok, r);
-            four(l, d0, ok, ld);
             four(p + g.off_a, d0, ok, ra);
             four(ab, d0, true, bias);
 #pragma unroll
-            for (int j = 0; j < 4; j++) {
-                float G = ld[j] * kLog2e;
+            for (int j = 0; j < 4; j++) G[j] = ld[i][j] * kLog2e;
 #pragma unroll
-                for (int o = 1; o < 32; o *= 2) {
-                    const float y = __shfl_up_sync(0xffffffffu, G, o);
-                    if (lane >= o) G += y;
+            for (int o = 1; o < 32; o *= 2)
+#pragma unroll
+                for (int j = 0; j < 4; j++) {
+                    const float y = __shfl_up_sync(0xffffffffu, G[j], o);
+                    if (lane >= o) G[j] += y;
                 }
-                const float up = __shfl_up_sync(0xffffffffu, G, 1), gp = lane > 0 ? up : 0.0f, gm = __shfl_sync(0xffffffffu, G, kT / 2 - 1), ge = __shfl_sync(0xffffffffu, G, 31);
-                const float u = k[i][j] * rk, back = exp2f(gm - G);
+#pragma unroll
+            for (int j = 0; j < 4; j++) {
+                const float up = __shfl_up_sync(0xffffffffu, G[j], 1), gp = lane > 0 ? up : 0.0f, gm = __shfl_sync(0xffffffffu, G[j], kT / 2 - 1),
+                            ge = __shfl_sync(0xffffffffu, G[j], 31);
+                const float u = k[i][j] * rk, back = exp2f(gm - G[j]);
                 const int d = d0 + j, at = d * kPitch + lane;
                 s_u[at] = u * exp2f(gp - gm);
-                s_r[at] = r[j] * exp2f(G - gm);
+                s_r[at] = r[j] * exp2f(G[j] - gm);
                 s_k[at] = k[i][j] * back;
-                s_b[at] = sigmoid_f(ra[j] + bias[j]) * u * back;
+                s_b[at] = __fdividef(u, 1.0f + __expf(-(ra[j] + bias[j]))) * back;
                 if (lane == 0) { s_cm[d] = exp2f(gm); s_ce[d] = exp2f(ge - gm); s_ge[d] = exp2f(ge); }
             }
         }
     }
     __syncthreads();
-    // the four triangles, one 4 x 4 tile of two of them per thread and quarter of the channels
-    if (tid < 288) {
-        const int kq = tid & 3, pair = (tid >> 2) & 1;
-        int ti = 0, tj = tid >> 3;
+    // the four triangles, a 4 x 4 tile of two of them per thread and share of the channels
+    constexpr int kShares = kWarps >= 9 ? 4 : 2, kTiles = 16 / kShares;  // tiles per warp
+    if (warp * kTiles < 36) {
+        const int pair = lane & 1, share = lane / (2 * kTiles), tile = min(warp * kTiles + (lane >> 1) % kTiles, 35);
+        int ti = 0, tj = tile;
         while (tj > ti) { tj -= ti + 1; ti++; }
-        const float *x = (pair ? s_r : s_u) + 4 * ti, *yk = s_k + 4 * tj, *yb = s_b + 4 * tj;
+        const int d0 = 4 * (share & 1) + DP / 2 * (share >> 1);  // shares of neighbouring channel fours: other banks
+        const float *x = (pair ? s_r : s_u) + 4 * ti + d0 * kPitch, *yk = s_k + 4 * tj + d0 * kPitch, *yb = s_b + 4 * tj + d0 * kPitch;
         float ak[4][4] = {}, ab[4][4] = {};
 #pragma unroll 4
-        for (int d = kq; d < DP; d += 4) {
+        for (int i = 0; i < DP / kShares; i++) {
+            const int d = (i & 3) + (i >> 2) * 8;
             float xt[4], ks[4], bs[4];
             get4(xt, x + d * kPitch); get4(ks, yk + d * kPitch); get4(bs, yb + d * kPitch);
 #pragma unroll
-            for (int i = 0; i < 4; i++)
+            for (int p = 0; p < 4; p++)
 #pragma unroll
-                for (int j = 0; j < 4; j++) { ak[i][j] = fmaf(xt[i], ks[j], ak[i][j]); ab[i][j] = fmaf(xt[i], bs[j], ab[i][j]); }
+                for (int q = 0; q < 4; q++) { ak[p][q] = fmaf(xt[p], ks[q], ak[p][q]); ab[p][q] = fmaf(xt[p], bs[q], ab[p][q]); }
         }
-#pragma unroll
-        for (int i = 0; i < 4; i++)
-#pragma unroll
-            for (int j = 0; j < 4; j++) {
-                ak[i][j] += __shfl_xor_sync(0xffffffffu, ak[i][j], 1);
-                ak[i][j] += __shfl_xor_sync(0xffffffffu, ak[i][j], 2);
-                ab[i][j] += __shfl_xor_sync(0xffffffffu, ab[i][j], 1);
-                ab[i][j] += __shfl_xor_sync(0xffffffffu, ab[i][j], 2);
-                const int t = 4 * ti + i, s = 4 * tj + j;
-                if (s > t || (s == t && !pair)) ak[i][j] = ab[i][j] = 0.0f;
-            }
         float *mk = pair ? s_brk : s_auk, *mb = pair ? s_brb : s_aub;
 #pragma unroll
-        for (int i = 0; i < 4; i++)
-            if (kq == i) {
-                *(float4*)(mk + (4 * ti + i) * kPitch + 4 * tj) = make_float4(ak[i][0], ak[i][1], ak[i][2], ak[i][3]);
-                *(float4*)(mb + (4 * ti + i) * kPitch + 4 * tj) = make_float4(ab[i][0], ab[i][1], ab[i][2], ab[i][3]);
-            }
-    }
-    __syncthreads();
-    // forward substitution, one column of W or Y per thread
-    for (int col = tid; col < 2 * DP; col += kThreads) {
-        float x[kT];
-        if (col < DP) {
-            const float cm = s_cm[col];
+        for (int p = 0; p < 4; p++) {
 #pragma unroll
-            for (int t = 0; t < kT; t += 4) {
-                float q[4];
-                get4(q, s_u + col * kPitch + t);
+            for (int q = 0; q < 4; q++) {
 #pragma unroll
-                for (int j = 0; j < 4; j++) x[t + j] = q[j] * cm;
-            }
-        } else {
-            float v[kT];
-#pragma unroll
-            for (int t = 0; t < kT; t++) v[t] = s_v[t * DP + col - DP];
-#pragma unroll
-            for (int t = 0; t < kT; t++) {
-                float p[2] = {0.0f, 0.0f};
-#pragma unroll
-                for (int s = 0; s < t; s += 4) {
-                    float m[4];
-                    get4(m, s_auk + t * kPitch + s);
-#pragma unroll
-                    for (int j = 0; j < 4; j++)
-                        if (s + j < t) p[j & 1] = fmaf(m[j], v[s + j], p[j & 1]);
+                for (int o = 2 * kTiles; o < 32; o *= 2) {
+                    ak[p][q] += __shfl_xor_sync(0xffffffffu, ak[p][q], o);
+                    ab[p][q] += __shfl_xor_sync(0xffffffffu, ab[p][q], o);
                 }
-                x[t] = p[0] + p[1];
+                const int t = 4 * ti + p, s = 4 * tj + q;
+                if (s > t || (s == t && !pair)) ak[p][q] = ab[p][q] = 0.0f;
             }
-        }
-#pragma unroll
-        for (int t = 0; t < kT; t++) {
-            float p[2] = {0.0f, 0.0f};
-#pragma unroll
-            for (int s = 0; s < t; s += 4) {
-                float m[4];
-                get4(m, s_aub + t * kPitch + s);
-#pragma unroll
-                for (int j = 0; j < 4; j++)
-                    if (s + j < t) p[j & 1] = fmaf(m[j], x[s + j], p[j & 1]);
+            if ((p & (kShares - 1)) == share) {
+                *(float4*)(mk + (4 * ti + p) * kPitch + 4 * tj) = make_float4(ak[p][0], ak[p][1], ak[p][2], ak[p][3]);
+                *(float4*)(mb + (4 * ti + p) * kPitch + 4 * tj) = make_float4(ab[p][0], ab[p][1], ab[p][2], ab[p][3]);
             }
-            x[t] -= p[0] + p[1];
-            s_x[t * 2 * DP + col] = x[t];
         }
     }
     __syncthreads();
-    // M, R, C and P in tiles of 4 x 4
-    constexpr int kCols = DP / 4, kTasks = (DP + kT) / 4 * kCols;
-    for (int task = tid; task < kTasks; task += kThreads) {
-        const int e0 = task % kCols * 4, row0 = task / kCols * 4;
-        const bool token = row0 >= DP;
-        const int t0 = row0 - DP;
-        const float *lk = token ? s_brk + t0 * kPitch : s_k + row0 * kPitch, *lb = token ? s_brb + t0 * kPitch : s_b + row0 * kPitch;
-        const int end = token ? t0 + 4 : kT;
-        float m[4][4] = {}, c[4][4] = {};
-        for (int s = 0; s < end; s += 4) {
-            float xb[4][4], xk[4][4];
+    // Auk V, tiles of 4 x 4
+    for (int u = warp; u < kT / 4 / Lanes::kRows * kColBlocks; u += kWarps) {
+        const int t0 = 4 * (u / kColBlocks * Lanes::kRows + Lanes::row(lane)), e0 = 4 * (u % kColBlocks * cols_per_warp(DP) + Lanes::col(lane));
+        float y[4][4] = {};
+        for (int s = 0; s <= t0; s += 4) {
+            float m[4][4];
 #pragma unroll
-            for (int i = 0; i < 4; i++) { get4(xb[i], lb + i * kPitch + s); get4(xk[i], lk + i * kPitch + s); }
+            for (int i = 0; i < 4; i++) get4(m[i], s_auk + (t0 + i) * kPitch + s);
 #pragma unroll
             for (int j = 0; j < 4; j++) {
-                float w[4], y[4], v[4];
-                get4(w, s_x + (s + j) * 2 * DP + e0); get4(y, s_x + (s + j) * 2 * DP + DP + e0); get4(v, s_v + (s + j) * DP + e0);
+                float v[4];
+                get4(v, s_v + (s + j) * DP + e0);
 #pragma unroll
                 for (int i = 0; i < 4; i++)
 #pragma unroll
+                    for (int q = 0; q < 4; q++) y[i][q] = fmaf(m[i][j], v[q], y[i][q]);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; i++) *(float4*)(s_y + (t0 + i) * DP + e0) = make_float4(y[i][0], y[i][1], y[i][2], y[i][3]);
+    }
+    __syncthreads();
+    // forward substitution, one column of W or Y per thread
+    {
+        float x[kT];
+        if (tid < DP) {
+            const float cm = s_cm[tid];
+#pragma unroll
+            for (int t = 0; t < kT; t += 4) {
+                float q[4];
+                get4(q, s_u + tid * kPitch + t);
+#pragma unroll
+                for (int j = 0; j < 4; j++) x[t + j] = q[j] * cm;
+            }
+        } else if (tid < 2 * DP) {
+#pragma unroll
+            for (int t = 0; t < kT; t++) x[t] = s_y[t * DP + tid - DP];
+        }
+        __syncthreads();  // W takes the place of u
+        if (tid < 2 * DP) {
+            float* dst = tid < DP ? s_w + tid : s_y + tid - DP;
+            dst[0] = x[0];
+#pragma unroll
+            for (int t = 1; t < kT; t++) {
+                float p[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+                for (int s = 0; s < t; s += 4) {
+                    float m[4];
+                    get4(m, s_aub + t * kPitch + s);
+#pragma unroll
+                    for (int j = 0; j < 4; j++)
+                        if (s + j < t) p[j] = fmaf(m[j], x[s + j], p[j]);
+                }
+                x[t] -= (p[0] + p[1]) + (p[2] + p[3]);
+                dst[t * DP] = x[t];
+            }
+        }
+    }
+    __syncthreads();
+    // M and C (state rows), R and P (token rows): eight rows by four columns per thread
+    constexpr int kUnitRows = 8 * Lanes::kRows;
+    for (int u = warp; u < (DP + kT) / kUnitRows * kColBlocks; u += kWarps) {
+        const int base = u / kColBlocks * kUnitRows, e0 = 4 * (u % kColBlocks * cols_per_warp(DP) + Lanes::col(lane));
+        const bool token = base >= DP;
+        const int row0 = (token ? base - DP : base) + 4 * Lanes::row(lane), step = 4 * Lanes::kRows;  // rows row0 .. + 3 and row0 + step .. + 3
+        const float *lk = (token ? s_brk : s_k) + row0 * kPitch, *lb = (token ? s_brb : s_b) + row0 * kPitch;
+        const int end = token ? row0 + step + 4 : kT;
+        float m[8][4] = {}, c[8][4] = {};
+#pragma unroll 1
+        for (int s = 0; s < end; s += 2) {
+            float2 xb[8], xk[8];
+#pragma unroll
+            for (int i = 0; i < 8; i++) {
+                const int at = ((i >> 2) * step + (i & 3)) * kPitch + s;
+                // a token's upper rows end before the lower ones; what lies behind their end was not written
+                const bool live = !token || i >= 4 || s < row0 + 4;
+                xb[i] = live ? *(const float2*)(lb + at) : make_float2(0.0f, 0.0f);
+                xk[i] = live ? *(const float2*)(lk + at) : make_float2(0.0f, 0.0f);
+            }
+#pragma unroll
+            for (int j = 0; j < 2; j++) {
+                float w[4], y[4], v[4];
+                get4(w, s_w + (s + j) * DP + e0); get4(y, s_y + (s + j) * DP + e0); get4(v, s_v + (s + j) * DP + e0);
+#pragma unroll
+                for (int i = 0; i < 8; i++) {
+                    const float b = j ? -xb[i].y : -xb[i].x, k = j ? xk[i].y : xk[i].x;
+#pragma unroll
                     for (int q = 0; q < 4; q++) {
-                        m[i][q] = fmaf(-xb[i][j], w[q], m[i][q]);
-                        c[i][q] = fmaf(xk[i][j], v[q], c[i][q]);
-                        c[i][q] = fmaf(-xb[i][j], y[q], c[i][q]);
+                        m[i][q] = fmaf(b, w[q], m[i][q]);
+                        c[i][q] = fmaf(k, v[q], c[i][q]);
+                        c[i][q] = fmaf(b, y[q], c[i][q]);
                     }
+                }
             }
         }
-        if (token) {
 #pragma unroll
-            for (int q = 0; q < 4; q++) {
-                float r[4];
-                get4(r, s_r + (e0 + q) * kPitch + t0);
-                const float cm = s_cm[e0 + q];
+        for (int half = 0; half < 2; half++) {
+            const int row = row0 + half * step, i0 = 4 * half;
+            if (token) {
 #pragma unroll
-                for (int i = 0; i < 4; i++) m[i][q] = fmaf(r[i], cm, m[i][q]);
+                for (int q = 0; q < 4; q++) {
+                    float r[4];
+                    get4(r, s_r + (e0 + q) * kPitch + row);
+                    const float cm = s_cm[e0 + q];
+                    *(float4*)(out + L.r() + (size_t)(e0 + q) * kT + row) = make_float4(fmaf(r[0], cm, m[i0][q]), fmaf(r[1], cm, m[i0 + 1][q]), fmaf(r[2], cm, m[i0 + 2][q]), fmaf(r[3], cm, m[i0 + 3][q]));
+                }
+#pragma unroll
+                for (int i = 0; i < 4; i++) *(float4*)(out + L.p() + (size_t)(row + i) * DP + e0) = make_float4(c[i0 + i][0], c[i0 + i][1], c[i0 + i][2], c[i0 + i][3]);
+            } else {
+                float ce[4];
+                get4(ce, s_ce + row);
+#pragma unroll
+                for (int q = 0; q < 4; q++) {
+                    float x[4];
+#pragma unroll
+                    for (int i = 0; i < 4; i++) x[i] = fmaf(m[i0 + i][q], ce[i], e0 + q == row + i ? s_ge[row + i] : 0.0f);
+                    *(float4*)(out + L.m() + (size_t)(e0 + q) * DP + row) = make_float4(x[0], x[1], x[2], x[3]);
+                }
+                float* co = out + L.c() + (size_t)(e0 / 32) * DP * 32 + e0 % 32;
+#pragma unroll
+                for (int i = 0; i < 4; i++) *(float4*)(co + (size_t)(row + i) * 32) = make_float4(c[i0 + i][0] * ce[i], c[i0 + i][1] * ce[i], c[i0 + i][2] * ce[i], c[i0 + i][3] * ce[i]);
             }
-        } else {
-#pragma unroll
-            for (int i = 0; i < 4; i++) {
-                const float ce = s_ce[row0 + i];
-#pragma unroll
-                for (int q = 0; q < 4; q++) { m[i][q] = fmaf(m[i][q], ce, e0 + q == row0 + i ? s_ge[row0 + i] : 0.0f); c[i][q] *= ce; }
-            }
-        }
-        float* co = out + L.co() + (size_t)(e0 / 32) * L.rows() * 32 + e0 % 32;
-#pragma unroll
-        for (int i = 0; i < 4; i++) {
-            *(float4*)(out + (size_t)(e0 + i) * L.rows() + row0) = make_float4(m[0][i], m[1][i], m[2][i], m[3][i]);
-            *(float4*)(co + (size_t)(row0 + i) * 32) = make_float4(c[i][0], c[i][1], c[i][2], c[i][3]);
         }
     }
 }
 
-// A product of (dp + 32) x dp by dp x 32 per chunk, in 4 x 4 tiles; the operands of the chunk behind the next one travel meanwhile.
+// S = M S0 + C, one product of dp x dp by dp x 32 per chunk in 4 x 4 tiles, by two groups of warps that share its sum; the operands of
+// the next chunk travel meanwhile.  The state before every chunk takes the place of its C.
 template <int DP>
-__global__ void __launch_bounds__(2 * DP + 64) general_carry_kernel(const GeneralArgs a, const float* __restrict__ scratch, int* error_flag) {
-    constexpr int kRows = DP + kT, kMr = DP * kRows, kCo = kRows * 32;
+__global__ void __launch_bounds__(4 * DP) general_carry_kernel(const GeneralArgs a, float* __restrict__ scratch, int* error_flag) {
+    constexpr int kM = DP * DP, kC = DP * 32;
+    typedef LaneGrid<8> Lanes;
     extern __shared__ __align__(128) float sm[];
     __shared__ uint64_t full[2];
-    float *s_mr = sm, *s_co = s_mr + 2 * kMr, *s_S = s_co + 2 * kCo;
-    const int tid = threadIdx.x, rg = tid >> 3, eg = tid & 7;
+    float *s_m = sm, *s_c = s_m + 2 * kM, *s_S = s_c + 2 * kC, *s_part = s_S + kC;
+    const int tid = threadIdx.x, lane = tid & 31, group = tid / (2 * DP), warp = (tid >> 5) - group * (DP / 16), d0 = 16 * warp + 4 * Lanes::row(lane), e = 4 * Lanes::col(lane);
     if (tid == 0) {
         mbar_init(&full[0], 1);
         mbar_init(&full[1], 1);
@@ -456,81 +507,181 @@ __global__ void __launch_bounds__(2 * DP + 64) general_carry_kernel(const Genera
     pdl_wait();
     const GeneralShape& g = a.g;
     const DeltaChunkRun cr = a.chunk_runs[blockIdx.x];
-    const int h = blockIdx.y, e0 = blockIdx.z * 32, chunks = (cr.run.n + kT - 1) / kT;
+    const int h = blockIdx.y, e0 = blockIdx.z * 32 + e, chunks = (cr.run.n + kT - 1) / kT;
     const ItemLayout L{DP};
     float* st = a.state + ((size_t)cr.run.seq * g.heads + h) * g.dim * g.dim;
+    auto item = [&](int c) { return scratch + ((size_t)(cr.chunk0 * kHalves + c) * g.heads + h) * L.size(); };
     auto request = [&](int c) {  // one thread
-        const float* src = scratch + ((size_t)(cr.chunk0 * kHalves + c) * g.heads + h) * L.size();
-        mbar_expect_tx(&full[c & 1], (uint32_t)(kMr + kCo) * 4);
-        bulk_load(s_mr + (c & 1) * kMr, src, (uint32_t)kMr * 4, &full[c & 1]);
-        bulk_load(s_co + (c & 1) * kCo, src + L.co() + (size_t)blockIdx.z * kCo, (uint32_t)kCo * 4, &full[c & 1]);
+        const float* src = item(c);
+        mbar_expect_tx(&full[c & 1], (uint32_t)(kM + kC) * 4);
+        bulk_load(s_m + (c & 1) * kM, src + L.m(), (uint32_t)kM * 4, &full[c & 1]);
+        bulk_load(s_c + (c & 1) * kC, src + L.c() + (size_t)blockIdx.z * kC, (uint32_t)kC * 4, &full[c & 1]);
     };
     if (tid == 0) {
         request(0);
         if (chunks > 1) request(1);
     }
-    const bool owner = 4 * rg < DP;  // of state rows; the others make the tokens' read-outs
-    float S[4][4] = {};
+    float S[4][4] = {};  // of group 0: rows d0 .., columns e0 ..
     auto publish = [&]() {
 #pragma unroll
-        for (int i = 0; i < 4; i++) *(float4*)(s_S + (4 * rg + i) * 32 + 4 * eg) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+        for (int i = 0; i < 4; i++) *(float4*)(s_S + (d0 + i) * 32 + e) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
     };
-    if (owner) {
+    if (group == 0) {
         if (cr.run.pos0 > 0)
 #pragma unroll
             for (int i = 0; i < 4; i++)
 #pragma unroll
-                for (int j = 0; j < 4; j++) {
-                    const int d = 4 * rg + i, e = e0 + 4 * eg + j;
-                    if (d < g.dim && e < g.dim) S[i][j] = st[(size_t)d * g.dim + e];
-                }
+                for (int j = 0; j < 4; j++)
+                    if (d0 + i < g.dim && e0 + j < g.dim) S[i][j] = st[(size_t)(d0 + i) * g.dim + e0 + j];
         publish();
     }
     __syncthreads();
     for (int c = 0; c < chunks; c++) {
-        const float *mr = s_mr + (c & 1) * kMr + 4 * rg, *co = s_co + (c & 1) * kCo + 4 * rg * 32 + 4 * eg, *sp = s_S + 4 * eg;
+        const float *mp = s_m + (c & 1) * kM + d0 + group * (DP / 2) * DP, *sp = s_S + e + group * (DP / 2) * 32;
         if (!mbar_wait(&full[c & 1], (uint32_t)(c >> 1) & 1) && tid == 0) atomicExch(error_flag, 17);
+        float acc[4][4] = {};
+        if (group == 0) {
+            float* keep = item(c) + L.c() + (size_t)blockIdx.z * kC + e;
+            const float* add = s_c + (c & 1) * kC + e;
 #pragma unroll
-        for (int i = 0; i < 4; i++) get4(S[i], co + i * 32);
+            for (int i = 0; i < 4; i++) {
+                *(float4*)(keep + (d0 + i) * 32) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+                get4(acc[i], add + (d0 + i) * 32);
+            }
+        }
 #pragma unroll 8
-        for (int d = 0; d < DP; d++) {
+        for (int d = 0; d < DP / 2; d++) {
             float x[4], y[4];
-            get4(x, mr + d * kRows);
+            get4(x, mp + d * DP);
             get4(y, sp + d * 32);
 #pragma unroll
             for (int i = 0; i < 4; i++)
 #pragma unroll
-                for (int j = 0; j < 4; j++) S[i][j] = fmaf(x[i], y[j], S[i][j]);
+                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(x[i], y[j], acc[i][j]);
         }
+        if (group == 1)
+#pragma unroll
+            for (int i = 0; i < 4; i++) *(float4*)(s_part + (d0 + i) * 32 + e) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
         __syncthreads();
-        if (tid == 0 && c + 2 < chunks) request(c + 2);
-        if (owner) publish();
-        else {
-            const int t0 = c * kT + 4 * rg - DP;
+        if (tid == 2 * DP && c + 2 < chunks) request(c + 2);
+        if (group == 0) {
 #pragma unroll
             for (int i = 0; i < 4; i++) {
-                if (t0 + i >= cr.run.n) break;
-                float* o = a.o + (size_t)(cr.run.tok0 + t0 + i) * g.heads * g.dim + h * g.dim + e0 + 4 * eg;
+                float p[4];
+                get4(p, s_part + (d0 + i) * 32 + e);
 #pragma unroll
-                for (int j = 0; j < 4; j++)
-                    if (e0 + 4 * eg + j < g.dim) o[j] = S[i][j];
+                for (int j = 0; j < 4; j++) S[i][j] = acc[i][j] + p[j];
             }
+            publish();
         }
         __syncthreads();
     }
-    if (owner)
+    if (group == 0)
 #pragma unroll
         for (int i = 0; i < 4; i++)
 #pragma unroll
-            for (int j = 0; j < 4; j++) {
-                const int d = 4 * rg + i, e = e0 + 4 * eg + j;
-                if (d < g.dim && e < g.dim) st[(size_t)d * g.dim + e] = S[i][j];
-            }
+            for (int j = 0; j < 4; j++)
+                if (d0 + i < g.dim && e0 + j < g.dim) st[(size_t)(d0 + i) * g.dim + e0 + j] = S[i][j];
+}
+
+// O = R S0 + P of one (chunk, head), norm and gate.
+template <int DP>
+__global__ void __launch_bounds__(2 * DP) general_read_kernel(const GeneralArgs a, const float* __restrict__ scratch, int* error_flag) {
+    typedef LaneGrid<cols_per_warp(DP)> Lanes;
+    constexpr int kColBlocks = DP / 4 / cols_per_warp(DP);
+    extern __shared__ __align__(128) float sm[];
+    __shared__ uint64_t full;
+    __shared__ float s_ss[kColBlocks][kT];
+    float *s_S = sm, *s_R = sm + DP * DP;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cb = warp % kColBlocks;
+    const int t0 = 4 * (warp / kColBlocks * Lanes::kRows + Lanes::row(lane)), e0 = 4 * (cb * cols_per_warp(DP) + Lanes::col(lane));
+    if (tid == 0) {
+        mbar_init(&full, 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    }
+    pdl_launch_dependents();
+    __syncthreads();
+    pdl_wait();
+    const GeneralShape& g = a.g;
+    const DeltaChunk ck = a.chunks[blockIdx.x / kHalves];
+    const int sub = blockIdx.x % kHalves, n = min(kT, ck.n - sub * kT), h = blockIdx.y;
+    if (n <= 0) return;
+    const size_t tok0 = (size_t)ck.tok0 + sub * kT;
+    const ItemLayout L{DP};
+    const float* src = scratch + ((size_t)blockIdx.x * g.heads + h) * L.size();
+    if (tid == 0) {  // S0 and R lie one behind the other
+        mbar_expect_tx(&full, (uint32_t)(DP * DP + DP * kT) * 4);
+        bulk_load(s_S, src + L.c(), (uint32_t)(DP * DP + DP * kT) * 4, &full);
+    }
+    const bool vec = g.dim % 4 == 0;
+    float o[4][4], gate[4][4], w[4];
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        get4(o[i], src + L.p() + (size_t)(t0 + i) * DP + e0);
+        const bf16* gp = (const bf16*)a.gate + (tok0 + min(t0 + i, n - 1)) * a.ld_gate + (size_t)h * g.dim + e0;
+        if (vec) {
+            const uint2 u = e0 < g.dim ? *(const uint2*)gp : make_uint2(0u, 0u);
+            gate[i][0] = __uint_as_float(u.x << 16); gate[i][1] = __uint_as_float(u.x & 0xFFFF0000u);
+            gate[i][2] = __uint_as_float(u.y << 16); gate[i][3] = __uint_as_float(u.y & 0xFFFF0000u);
+        } else
+#pragma unroll
+            for (int j = 0; j < 4; j++) gate[i][j] = e0 + j < g.dim ? __bfloat162float(gp[j]) : 0.0f;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; j++) w[j] = e0 + j < g.dim ? a.norm_w[h * g.dim + e0 + j] : 0.0f;
+    if (!mbar_wait(&full, 0) && tid == 0) atomicExch(error_flag, 18);
+    const float *rp = s_R + t0, *sp = s_S + (e0 / 32) * DP * 32 + e0 % 32;
+#pragma unroll 8
+    for (int d = 0; d < DP; d++) {
+        float x[4], y[4];
+        get4(x, rp + d * kT);
+        get4(y, sp + d * 32);
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) o[i][j] = fmaf(x[i], y[j], o[i][j]);
+    }
+    float ss[4];
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        ss[i] = fmaf(o[i][0], o[i][0], fmaf(o[i][1], o[i][1], fmaf(o[i][2], o[i][2], o[i][3] * o[i][3])));
+#pragma unroll
+        for (int m = 2; m < 2 * cols_per_warp(DP); m *= 2) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], m);
+    }
+    if constexpr (kColBlocks > 1) {
+        if (Lanes::col(lane) == 0)
+#pragma unroll
+            for (int i = 0; i < 4; i++) s_ss[cb][t0 + i] = ss[i];
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            ss[i] = 0.0f;
+#pragma unroll
+            for (int b = 0; b < kColBlocks; b++) ss[i] += s_ss[b][t0 + i];
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        if (t0 + i >= n) break;
+        const float r = 1.0f / sqrtf(ss[i] / (float)g.dim + g.eps);
+        float y[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) y[j] = __fdividef(o[i][j] * r * w[j], 1.0f + __expf(-gate[i][j]));
+        bf16* dst = (bf16*)a.out + (tok0 + t0 + i) * a.ldo + (size_t)h * g.dim + e0;
+        if (vec) {
+            if (e0 < g.dim) *(uint2*)dst = make_uint2(pack2(y[0], y[1]), pack2(y[2], y[3]));
+        } else
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+                if (e0 + j < g.dim) dst[j] = __float2bfloat16_rn(y[j]);
+    }
 }
 
 int padded_dim(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : 128; }
-size_t chunk_smem(int dp) { return ((size_t)4 * dp * kPitch + 3 * kT * dp + 4 * kT * kPitch + 3 * dp + 32 * kWarps) * sizeof(float); }
-size_t carry_smem(int dp) { return ((size_t)2 * dp * (dp + kT) + 2 * (dp + kT) * 32 + dp * 32) * sizeof(float); }
+size_t chunk_smem(int dp) { return ((size_t)4 * dp * kPitch + 8 + 2 * kT * dp + 4 * kT * kPitch + 3 * dp + chunk_threads(dp)) * sizeof(float); }
+size_t carry_smem(int dp) { return ((size_t)2 * dp * dp + 4 * dp * 32) * sizeof(float); }
+size_t read_smem(int dp) { return ((size_t)dp * dp + dp * kT) * sizeof(float); }
 
 template <typename A>
 int32_t step_dispatch(const GeneralArgs& a, cudaStream_t s) {
@@ -571,19 +722,22 @@ int32_t launch_general_scan(const GeneralArgs& a, cudaStream_t s) {
     }
 }
 
+template <int DP>
+static int32_t run_chunks(const GeneralArgs& a, float* scratch, cudaStream_t s) {
+    const dim3 all((unsigned)(a.n_chunks * kHalves), (unsigned)a.g.heads), walk((unsigned)a.n_chunk_runs, (unsigned)a.g.heads, (unsigned)(DP / 32));
+    LC_CUDA(ensure_smem_limit((const void*)general_chunk_kernel<DP>, chunk_smem(DP)));
+    LC_CUDA(ensure_smem_limit((const void*)general_carry_kernel<DP>, carry_smem(DP)));
+    LC_CUDA(ensure_smem_limit((const void*)general_read_kernel<DP>, read_smem(DP)));
+    LC_CUDA(launch_pdl(general_chunk_kernel<DP>, all, dim3(chunk_threads(DP)), chunk_smem(DP), s, a, scratch));
+    LC_CUDA(launch_pdl(general_carry_kernel<DP>, walk, dim3(4 * DP), carry_smem(DP), s, a, scratch, gemv_error_flag_dev()));
+    LC_CUDA(launch_pdl(general_read_kernel<DP>, all, dim3(2 * DP), read_smem(DP), s, a, (const float*)scratch, gemv_error_flag_dev()));
+    return LC_OK;
+}
 int32_t launch_general_chunks(const GeneralArgs& a, float* scratch, cudaStream_t s) {
-    auto go = [&](auto chunk, auto carry, int dp) -> int32_t {
-        const dim3 g1((unsigned)(a.n_chunks * kHalves), (unsigned)a.g.heads), g2((unsigned)a.n_chunk_runs, (unsigned)a.g.heads, (unsigned)(dp / 32));
-        LC_CUDA(ensure_smem_limit((const void*)chunk, chunk_smem(dp)));
-        LC_CUDA(ensure_smem_limit((const void*)carry, carry_smem(dp)));
-        LC_CUDA(launch_pdl(chunk, g1, dim3(kThreads), chunk_smem(dp), s, a, scratch));
-        LC_CUDA(launch_pdl(carry, g2, dim3((unsigned)(2 * dp + 64)), carry_smem(dp), s, a, (const float*)scratch, gemv_error_flag_dev()));
-        return LC_OK;
-    };
     switch (padded_dim(a.g.dim)) {
-        case 32: return go(general_chunk_kernel<32>, general_carry_kernel<32>, 32);
-        case 64: return go(general_chunk_kernel<64>, general_carry_kernel<64>, 64);
-        default: return go(general_chunk_kernel<128>, general_carry_kernel<128>, 128);
+        case 32: return run_chunks<32>(a, scratch, s);
+        case 64: return run_chunks<64>(a, scratch, s);
+        default: return run_chunks<128>(a, scratch, s);
     }
 }
 

@@ -168,7 +168,7 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnArgs a) {
 // is taken again, with the same result.
 template <typename A, int TAPS, int NQ, int AHEAD>
 __global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head_prep_kernel(const AttnArgs a, int stretch) {
-    constexpr int kWin = TAPS > 1 ? TAPS - 1 : 1, kTaps = TAPS > 0 ? TAPS : 1;
+    constexpr int kWin = TAPS > 1 ? TAPS - 1 : 1, kTaps = TAPS > 0 ? TAPS : 1, kTurn = NQ == 1 && TAPS == 0 ? 4 : 2;
     __shared__ float s_x[8][128 * NQ];
     pdl_launch_dependents();
     pdl_wait();
@@ -182,6 +182,8 @@ __global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head
     const int taps = TAPS > 0 ? TAPS : g.taps;
     const bool vec = (n & 3) == 0;  // then a lane's elements exist together and lie 16-byte aligned in the projected rows
     const bool near = g.pairs == AttnPairs::Neighbours && !is_v, near4 = near && (half & 1) == 0;
+    // halves whose partners lie a whole number of lanes apart: exchanged between lanes, angles fetched ahead
+    const bool apart = kTurn == 4 && !is_v && half > 0 && !near && (half & 3) == 0;
     auto four_at = [&](const float* row, int c, float (&x)[4]) {
         if (vec) {
             const float4 u = c < n ? *(const float4*)(row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -191,8 +193,17 @@ __global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head
             for (int e = 0; e < 4; e++) x[e] = c + e < n ? row[c + e] : 0.0f;
         }
     };
-    auto angles_at = [&](int pos, int c, float2 (&cs)[2]) {  // of the pairs (c, c + 1) and (c + 2, c + 3)
-        cs[0] = cs[1] = make_float2(1.0f, 0.0f);
+    auto angles_at = [&](int pos, int c, float2 (&cs)[kTurn]) {  // of the pairs (c, c + 1) and (c + 2, c + 3), or of the four elements
+#pragma unroll
+        for (int i = 0; i < kTurn; i++) cs[i] = make_float2(1.0f, 0.0f);
+        if constexpr (kTurn == 4)
+            if (apart) {
+                if (c >= 2 * half) return;
+                const float4* p = (const float4*)(a.rot + (size_t)pos * half + (c < half ? c : c - half));
+                const float4 u = __ldg(p), z = __ldg(p + 1);
+                cs[0] = make_float2(u.x, u.y); cs[1] = make_float2(u.z, u.w); cs[2] = make_float2(z.x, z.y); cs[3] = make_float2(z.z, z.w);
+                return;
+            }
         const float2* tab = a.rot + (size_t)pos * half + c / 2;
         if (near4) {
             if (c < 2 * half) { const float4 u = __ldg((const float4*)tab); cs[0] = make_float2(u.x, u.y); cs[1] = make_float2(u.z, u.w); }
@@ -216,7 +227,7 @@ __global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head
         }
     int prev_seq = -1, prev_pos = -1;
     float ahead[AHEAD][NQ][4];
-    float2 turn[AHEAD][NQ][2];
+    float2 turn[AHEAD][NQ][kTurn];
     int seq_a[AHEAD], pos_a[AHEAD], page_a[AHEAD];
     for (int tb = t0; tb < t1; tb += AHEAD) {
 #pragma unroll
@@ -309,6 +320,14 @@ __global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head
                             x[p][e] = y * cs.x - z * cs.y;
                             x[p][e + 1] = z * cs.x + y * cs.y;
                         }
+                } else if (kTurn == 4 && apart) {
+                    const int c = 4 * lane, from = c < half ? lane + half / 4 : lane - half / 4;
+#pragma unroll
+                    for (int e = 0; e < 4; e++) {
+                        const float other = __shfl_sync(0xffffffffu, x[0][e], from & 31);
+                        const float2 cs = turn[v][0][kTurn == 4 ? e : 0];
+                        if (c < 2 * half) x[0][e] = x[0][e] * cs.x + (c < half ? -other : other) * cs.y;
+                    }
                 } else if (half > 0) {
                     const float2* tab = a.rot + (size_t)pos * half;
                     __syncwarp();

@@ -596,11 +596,14 @@ int32_t general_delta_block(lc_model* m, MixerUnit& L, const void* x, int ldx, i
         d.chunks = st.d_chunks; d.n_chunks = st.n_chunks; d.chunk_runs = st.d_chunk_runs; d.n_chunk_runs = st.n_chunk_runs;
         if (d.n_runs) LC_TRY(launch_general_scan(d, m->stream));
         if (d.n_chunk_runs) LC_TRY(launch_general_chunks(d, (float*)st.chunk_scratch.p, m->stream));
-        HeadNormArgs o;
-        o.o = st.o; o.heads = s.heads; o.n = s.dim; o.T = T; o.eps = st.spec.eps; o.w = L.o_norm; o.w_stride = s.dim; o.gate = d.gate; o.ld_gate = ld_act; o.out = st.mixed;
-        o.ldo = d.ldo; o.f32 = st.f32;
-        LC_TRY(launch_head_norm(o, m->stream));
-        m->launches_in_call += 1 + (d.n_runs ? 1 : 0) + (d.n_chunk_runs ? 2 : 0);
+        if (d.n_runs) {  // the chunks norm and gate their own tokens
+            HeadNormArgs o;
+            if (d.n_chunk_runs) { o.runs = d.runs; o.n_runs = d.n_runs; o.longest = st.longest_short; }
+            o.o = st.o; o.heads = s.heads; o.n = s.dim; o.T = T; o.eps = st.spec.eps; o.w = L.o_norm; o.w_stride = s.dim; o.gate = d.gate; o.ld_gate = ld_act; o.out = st.mixed;
+            o.ldo = d.ldo; o.f32 = st.f32;
+            LC_TRY(launch_head_norm(o, m->stream));
+        }
+        m->launches_in_call += (d.n_runs ? 2 : 0) + (d.n_chunk_runs ? 3 : 0);
     }
     return product(m, L.out, st.mixed, d.ldo, T, st.y, st.spec.width, true);
 }
@@ -1038,6 +1041,8 @@ int32_t stack_upload_runs(lc_model* m, const std::vector<int32_t>& seq, const st
         chunk_runs.push_back(DeltaChunkRun{r, (int32_t)chunks.size(), (r.n + kDeltaChunk - 1) / kDeltaChunk});
         for (int t = 0; t < r.n; t += kDeltaChunk) chunks.push_back(DeltaChunk{r.tok0 + t, std::min(kDeltaChunk, r.n - t)});
     }
+    st.longest_short = 0;
+    for (const SeqRun& r : shorts) st.longest_short = std::max(st.longest_short, r.n);
     st.n_short_runs = (int)shorts.size(); st.n_chunks = (int)chunks.size(); st.n_chunk_runs = (int)chunk_runs.size();
     if (!shorts.empty()) LC_CUDA(cudaMemcpyAsync(st.d_short_runs, shorts.data(), shorts.size() * sizeof(SeqRun), cudaMemcpyHostToDevice, m->stream));
     if (!chunks.empty()) {

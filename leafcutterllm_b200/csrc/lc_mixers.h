@@ -179,6 +179,8 @@ struct HeadNormArgs {
     void* out = nullptr;               // [T][ldo] activations
     int ldo = 0;
     bool f32 = false;
+    const SeqRun* runs = nullptr;      // only the tokens of these runs; longest: the most tokens of one
+    int n_runs = 0, longest = 0;
 };
 int32_t launch_head_norm(const HeadNormArgs& a, cudaStream_t s);
 
@@ -390,7 +392,7 @@ struct GeneralArgs {
     const DeltaChunk* chunks = nullptr;         // longer runs
     const DeltaChunkRun* chunk_runs = nullptr;
     int n_chunks = 0, n_chunk_runs = 0;
-    const float* norm_w = nullptr;     // the step alone: norm, gate and output as in HeadNormArgs
+    const float* norm_w = nullptr;     // step and chunks: norm, gate and output as in HeadNormArgs
     const void* gate = nullptr;
     int ld_gate = 0;
     void* out = nullptr;
@@ -400,7 +402,7 @@ struct GeneralArgs {
 bool general_chunks_apply(const GeneralShape& g, double decay_scale, bool f32);
 size_t general_chunk_bytes(const GeneralShape& g);               // scratch per chunk of kDeltaChunk tokens
 int32_t launch_general_scan(const GeneralArgs& a, cudaStream_t s);
-int32_t launch_general_chunks(const GeneralArgs& a, float* scratch, cudaStream_t s);
+int32_t launch_general_chunks(const GeneralArgs& a, float* scratch, cudaStream_t s);  // with norm and gate
 int32_t launch_general_step(const GeneralArgs& a, cudaStream_t s);  // one token per sequence, with norm and gate
 
 // ---- expert_choice.cu: routing ---------------------------------------------------------------------------------------------
@@ -506,7 +508,7 @@ struct LayerStack {
     SeqRun* d_short_runs = nullptr;
     DeltaChunk* d_chunks = nullptr;
     DeltaChunkRun* d_chunk_runs = nullptr;
-    int n_short_runs = 0, n_chunks = 0, n_chunk_runs = 0;
+    int n_short_runs = 0, n_chunks = 0, n_chunk_runs = 0, longest_short = 0;
     size_t chunk_bytes = 0;            // scratch per chunk, widest layer
     DevBuf chunk_scratch;
     // latent attention of the call: its first n_short tokens attend one by one, the others in tiles over projected contexts,

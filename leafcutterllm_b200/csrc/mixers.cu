@@ -30,6 +30,18 @@ __global__ void pack_kernel(const __nv_bfloat16* __restrict__ src, int rows, int
     }
 }
 
+template <typename A> __device__ __forceinline__ float4 load4(const A* p);
+template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *(const float4*)p; }
+template <> __device__ __forceinline__ float4 load4<bf16>(const bf16* p) {
+    const uint2 v = *(const uint2*)p;
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
+}
+template <typename A> __device__ __forceinline__ void store4(A* p, float4 v);
+template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { *(float4*)p = v; }
+template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
+__device__ __forceinline__ float sq4(float4 v, float ss) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss)))); }
+__device__ __forceinline__ void add4(float4& y, float w, float4 v) { y.x = fmaf(w, v.x, y.x); y.y = fmaf(w, v.y, y.y); y.z = fmaf(w, v.z, y.z); y.w = fmaf(w, v.w, y.w); }
+
 __global__ void __launch_bounds__(256) embed_rows_kernel(const __nv_bfloat16* __restrict__ table, int rows, int width, const int64_t* __restrict__ ids,
                                                          float* __restrict__ x, __nv_bfloat16* __restrict__ act, int ld_act) {
     pdl_launch_dependents();
@@ -56,8 +68,10 @@ __global__ void __launch_bounds__(256) embed_rows_kernel(const __nv_bfloat16* __
 }
 
 // The same with a factor on the row, the token pair's row (PAIR) and, w != null, the sum's norm as activations.
-template <typename A, bool PAIR>
-__global__ void __launch_bounds__(256) embed_norm_kernel(const EmbedArgs a) {
+// VEC = 8: rows of a multiple of eight elements.
+template <typename A, bool PAIR, int VEC>
+__global__ void __launch_bounds__(512) embed_norm_kernel(const EmbedArgs a) {
+    constexpr int kHeld = VEC == 8 ? 2 : 4;
     __shared__ float sh[32];
     pdl_launch_dependents();
     pdl_wait();
@@ -82,19 +96,58 @@ __global__ void __launch_bounds__(256) embed_norm_kernel(const EmbedArgs a) {
             if (threadIdx.x == 0) p.last[seq] = (int32_t)id;
         }
     }
-    auto at = [&](int c) { return ok ? fmaf(__bfloat162float(src[c]), a.scale, PAIR ? __bfloat162float(two[c]) : 0.0f) : 0.0f; };
+    struct Part { float v[VEC]; };
+    auto at = [&](int c) {
+        Part p;
+        if constexpr (VEC == 8) {
+            const uint4 s = *(const uint4*)(src + c), u = PAIR ? *(const uint4*)(two + c) : make_uint4(0u, 0u, 0u, 0u);
+            const uint32_t sw[4] = {s.x, s.y, s.z, s.w}, uw[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                p.v[2 * i] = fmaf(__uint_as_float(sw[i] << 16), a.scale, __uint_as_float(uw[i] << 16));
+                p.v[2 * i + 1] = fmaf(__uint_as_float(sw[i] & 0xFFFF0000u), a.scale, __uint_as_float(uw[i] & 0xFFFF0000u));
+            }
+        } else p.v[0] = fmaf(__bfloat162float(src[c]), a.scale, PAIR ? __bfloat162float(two[c]) : 0.0f);
+        if (!ok)
+#pragma unroll
+            for (int i = 0; i < VEC; i++) p.v[i] = 0.0f;
+        return p;
+    };
     float ss = 0.0f;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) {
-        const float v = at(c);
-        a.x[t * width + c] = v;
-        if (a.copy) a.copy[t * width + c] = v;
-        ss = fmaf(v, v, ss);
-    }
+    auto put = [&](int c, const Part& p) {
+        float* dst[2] = {a.x, a.copy};
+#pragma unroll
+        for (int d = 0; d < 2; d++) {
+            if (!dst[d]) continue;
+            float* o = dst[d] + t * width + c;
+            if constexpr (VEC == 8) { *(float4*)o = make_float4(p.v[0], p.v[1], p.v[2], p.v[3]); *(float4*)(o + 4) = make_float4(p.v[4], p.v[5], p.v[6], p.v[7]); }
+            else *o = p.v[0];
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; i++) ss = fmaf(p.v[i], p.v[i], ss);
+    };
+    const int step = blockDim.x * VEC, c0 = threadIdx.x * VEC;
+    Part held[kHeld];
+#pragma unroll
+    for (int i = 0; i < kHeld; i++)
+        if (c0 + i * step < width) held[i] = at(c0 + i * step);
+#pragma unroll
+    for (int i = 0; i < kHeld; i++)
+        if (c0 + i * step < width) put(c0 + i * step, held[i]);
+    for (int c = c0 + kHeld * step; c < width; c += step) put(c, at(c));
     if (!a.act) return;
-    float r = 1.0f;
-    if (a.w) r = 1.0f / sqrtf(block_sum_once(ss, sh) / (float)width + a.eps);
+    const float r = a.w ? 1.0f / sqrtf(block_sum_once(ss, sh) / (float)width + a.eps) : 1.0f;
     A* act = (A*)a.act + t * a.ld_act;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) act[c] = to_act<A>(a.w ? at(c) * r * a.w[c] : at(c));
+    auto next = [&](int c, Part p) {
+#pragma unroll
+        for (int i = 0; i < VEC; i++) p.v[i] = a.w ? p.v[i] * r * a.w[c + i] : p.v[i];
+        if constexpr (VEC == 8) { store4<A>(act + c, make_float4(p.v[0], p.v[1], p.v[2], p.v[3])); store4<A>(act + c + 4, make_float4(p.v[4], p.v[5], p.v[6], p.v[7])); }
+        else act[c] = to_act<A>(p.v[0]);
+    };
+#pragma unroll
+    for (int i = 0; i < kHeld; i++)
+        if (c0 + i * step < width) next(c0 + i * step, held[i]);
+    for (int c = c0 + kHeld * step; c < width; c += step) next(c, at(c));
 }
 
 __global__ void keep_tokens_kernel(const SeqRun* __restrict__ runs, int n, const int64_t* __restrict__ ids, int32_t* __restrict__ last) {
@@ -110,22 +163,10 @@ __global__ void __launch_bounds__(256) act_rows_kernel(const float* __restrict__
     for (int c = threadIdx.x; c < width; c += blockDim.x) act[(size_t)blockIdx.x * ld_act + c] = __float2bfloat16_rn(x[(size_t)blockIdx.x * width + c]);
 }
 
-template <typename A> __device__ __forceinline__ float4 load4(const A* p);
-template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *(const float4*)p; }
-template <> __device__ __forceinline__ float4 load4<bf16>(const bf16* p) {
-    const uint2 v = *(const uint2*)p;
-    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xFFFF0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xFFFF0000u));
-}
-template <typename A> __device__ __forceinline__ void store4(A* p, float4 v);
-template <> __device__ __forceinline__ void store4<float>(float* p, float4 v) { *(float4*)p = v; }
-template <> __device__ __forceinline__ void store4<bf16>(bf16* p, float4 v) { *(uint2*)p = make_uint2(pack2(v.x, v.y), pack2(v.z, v.w)); }
-__device__ __forceinline__ float sq4(float4 v, float ss) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss)))); }
-__device__ __forceinline__ void add4(float4& y, float w, float4 v) { y.x = fmaf(w, v.x, y.x); y.y = fmaf(w, v.y, y.y); y.z = fmaf(w, v.z, y.z); y.w = fmaf(w, v.w, y.w); }
-
 // x += y, the sum over depth (DEPTH), the next sublayer's norm.  VEC as below.
-template <typename A, int VEC, bool DEPTH>
-__global__ void __launch_bounds__(512) plain_residual_kernel(const ResidualArgs a) {
-    constexpr int kHeld = VEC == 4 ? 4 : 8;
+template <typename A, int VEC, bool DEPTH, int THREADS>
+__global__ void __launch_bounds__(THREADS) plain_residual_kernel(const ResidualArgs a) {
+    constexpr int kHeld = VEC == 4 ? 4 : 8, kAhead = 8;  // results of earlier layers that are fetched together
     __shared__ float sh[32];
     pdl_launch_dependents();
     pdl_wait();
@@ -152,17 +193,29 @@ __global__ void __launch_bounds__(512) plain_residual_kernel(const ResidualArgs 
         for (int e = 0; e < VEC; e++) s.v[e] += y.v[e];
         if constexpr (DEPTH) {
             const DepthSum& d = a.depth;
-            put(d.keep + row + c, s);
+            const Part result = s;
             const float own = __ldg(d.c + d.n);
 #pragma unroll
             for (int e = 0; e < VEC; e++) s.v[e] *= own;
-#pragma unroll 8
-            for (int j = 0; j < d.n; j++) {
-                const Part z = get(d.past + j * d.stride + row + c);
-                const float f = __ldg(d.c + j);
+            const float* past = d.past + row + c;
+            for (int j0 = 0; j0 < d.n; j0 += kAhead, past += kAhead * d.stride) {
+                Part z[kAhead];
+                float f[kAhead];
 #pragma unroll
-                for (int e = 0; e < VEC; e++) s.v[e] = fmaf(f, z.v[e], s.v[e]);
+                for (int u = 0; u < kAhead; u++) {
+                    const bool there = j0 + u < d.n;
+                    f[u] = there ? __ldg(d.c + j0 + u) : 0.0f;
+                    if (there) z[u] = get(past + u * d.stride);
+                    else
+#pragma unroll
+                        for (int e = 0; e < VEC; e++) z[u].v[e] = 0.0f;
+                }
+#pragma unroll
+                for (int u = 0; u < kAhead; u++)
+#pragma unroll
+                    for (int e = 0; e < VEC; e++) s.v[e] = fmaf(f[u], z[u].v[e], s.v[e]);
             }
+            put(d.keep + row + c, result);
         }
         put(xr + c, s);
         return s;
@@ -562,13 +615,52 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaArgs a) {
     if (blockIdx.z == 0) delta_keep_inputs<A>(a, run, h, threadIdx.x, 128);
 }
 
+__device__ __forceinline__ int head_norm_row(const HeadNormArgs& a) {
+    if (!a.runs) return blockIdx.x;
+    const SeqRun r = a.runs[blockIdx.x / a.longest];
+    const int i = blockIdx.x % a.longest;
+    return i < r.n ? r.tok0 + i : -1;
+}
+// G lanes per (token, head), four elements each: heads of up to 4 G elements, a multiple of four
+template <typename A, int G>
+__global__ void __launch_bounds__(256) head_norm4_kernel(const HeadNormArgs a) {
+    constexpr int kItems = 2, kPer = 256 / G;  // heads per group of lanes
+    pdl_launch_dependents();
+    pdl_wait();
+    const int row = head_norm_row(a);
+    if (row < 0) return;
+    const size_t t = row;
+    const int group = threadIdx.x / G, c = (threadIdx.x % G) * 4;
+    float4 o[kItems], gate[kItems], w[kItems];
+#pragma unroll
+    for (int i = 0; i < kItems; i++) {
+        const int h = blockIdx.y * kPer * kItems + i * kPer + group;
+        o[i] = gate[i] = w[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (h < a.heads && c < a.n) {
+            o[i] = *(const float4*)(a.o + (t * a.heads + h) * a.n + c);
+            gate[i] = load4<A>((const A*)a.gate + t * a.ld_gate + (size_t)h * a.n + c);
+            w[i] = *(const float4*)(a.w + (size_t)h * a.w_stride + c);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < kItems; i++) {
+        const int h = blockIdx.y * kPer * kItems + i * kPer + group;
+        float ss = sq4(o[i], 0.0f);
+#pragma unroll
+        for (int m = 1; m < G; m *= 2) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+        const float r = 1.0f / sqrtf(ss / (float)a.n + a.eps);
+        if (h < a.heads && c < a.n)
+            store4<A>((A*)a.out + t * a.ldo + (size_t)h * a.n + c, make_float4(o[i].x * r * w[i].x * sigmoid_f(gate[i].x), o[i].y * r * w[i].y * sigmoid_f(gate[i].y),
+                                                                              o[i].z * r * w[i].z * sigmoid_f(gate[i].z), o[i].w * r * w[i].w * sigmoid_f(gate[i].w)));
+    }
+}
 // One warp per (token, head)
 template <typename A>
 __global__ void __launch_bounds__(256) head_norm_kernel(const HeadNormArgs a) {
     pdl_launch_dependents();
     pdl_wait();
-    const int t = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (h >= a.heads) return;
+    const int t = head_norm_row(a), h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (t < 0 || h >= a.heads) return;
     const float *o = a.o + ((size_t)t * a.heads + h) * a.n, *w = a.w + (size_t)h * a.w_stride;
     const A* gate = (const A*)a.gate + (size_t)t * a.ld_gate + (size_t)h * a.n;
     float ss = 0.0f;
@@ -850,15 +942,20 @@ int32_t launch_pack(const __nv_bfloat16* src, int rows, int cols, __nv_bfloat16*
 int32_t launch_embed_rows(const EmbedArgs& a, cudaStream_t s) {
     const dim3 grid((unsigned)a.T), block(256);
     auto go = [&](auto kern) -> int32_t {
-        LC_CUDA(launch_pdl(kern, grid, block, 0, s, a));
+        LC_CUDA(launch_pdl(kern, grid, dim3(a.T <= sm_count() ? 512 : 256), 0, s, a));
         return LC_OK;
     };
-    if (a.pair.table) return a.f32 ? go(embed_norm_kernel<float, true>) : go(embed_norm_kernel<bf16, true>);
+    const bool vec = a.width % 8 == 0 && a.ld_act % 8 == 0;
+    if (a.pair.table) {
+        if (a.f32) return vec ? go(embed_norm_kernel<float, true, 8>) : go(embed_norm_kernel<float, true, 1>);
+        return vec ? go(embed_norm_kernel<bf16, true, 8>) : go(embed_norm_kernel<bf16, true, 1>);
+    }
     if (a.scale == 1.0f && !a.w && !a.copy && !(a.f32 && a.act)) {
         LC_CUDA(launch_pdl(embed_rows_kernel, grid, block, 0, s, a.table, a.rows, a.width, a.ids, a.x, (bf16*)a.act, a.ld_act));
         return LC_OK;
     }
-    return a.f32 ? go(embed_norm_kernel<float, false>) : go(embed_norm_kernel<bf16, false>);
+    if (a.f32) return vec ? go(embed_norm_kernel<float, false, 8>) : go(embed_norm_kernel<float, false, 1>);
+    return vec ? go(embed_norm_kernel<bf16, false, 8>) : go(embed_norm_kernel<bf16, false, 1>);
 }
 int32_t launch_keep_tokens(const SeqRun* runs, int n_runs, const int64_t* ids, int32_t* last, cudaStream_t s) {
     LC_CUDA(launch_pdl(keep_tokens_kernel, dim3((unsigned)((n_runs + 127) / 128)), dim3(128), 0, s, runs, n_runs, ids, last));
@@ -873,17 +970,21 @@ int32_t launch_residual(const ResidualArgs& a, cudaStream_t s) {
     const bool moe = a.moe.rows != nullptr, pair = a.pair.y2 != nullptr;
     const bool vec = a.width % 4 == 0 && ((uintptr_t)a.pair.w0 | (uintptr_t)a.pair.w1) % 16 == 0 && (uintptr_t)a.w % 16 == 0 && (uintptr_t)a.w_next % 16 == 0 && (a.moe.ld_rows | a.moe.ld_h | a.ld_act) % 4 == 0;
     LC_CHECK(a.moe.top <= kMaxChoices && (!a.w_next || a.act), LC_ERR_INVALID, "residual sum: bad argument");
-    auto go = [&](auto kern) -> int32_t {
-        LC_CUDA(launch_pdl(kern, grid, block, 0, s, a));
+    auto go = [&](auto kern, unsigned threads = 0) -> int32_t {
+        LC_CUDA(launch_pdl(kern, grid, threads ? dim3(threads) : block, 0, s, a));
         return LC_OK;
     };
     if (!a.w) {
         LC_CHECK(!moe && !pair, LC_ERR_UNSUPPORTED, "residual sum: a mixture or a pair without an output norm");
         const bool deep = a.depth.keep != nullptr;
-        if (a.f32) return deep ? (vec ? go(plain_residual_kernel<float, 4, true>) : go(plain_residual_kernel<float, 1, true>))
-                               : (vec ? go(plain_residual_kernel<float, 4, false>) : go(plain_residual_kernel<float, 1, false>));
-        return deep ? (vec ? go(plain_residual_kernel<bf16, 4, true>) : go(plain_residual_kernel<bf16, 1, true>))
-                    : (vec ? go(plain_residual_kernel<bf16, 4, false>) : go(plain_residual_kernel<bf16, 1, false>));
+        // few rows: a row by twice the threads
+        auto plain = [&](auto act) -> int32_t {
+            typedef decltype(act) A;
+            const bool wide = vec && a.T <= sm_count() && a.width >= 4096;
+            if (deep) return wide ? go(plain_residual_kernel<A, 4, true, 1024>, 1024) : vec ? go(plain_residual_kernel<A, 4, true, 512>) : go(plain_residual_kernel<A, 1, true, 512>);
+            return wide ? go(plain_residual_kernel<A, 4, false, 1024>, 1024) : vec ? go(plain_residual_kernel<A, 4, false, 512>) : go(plain_residual_kernel<A, 1, false, 512>);
+        };
+        return a.f32 ? plain(0.0f) : plain(bf16());
     }
     LC_CHECK(!a.depth.keep, LC_ERR_UNSUPPORTED, "residual sum: a sum over depth behind an output norm");
     if (a.f32) {
@@ -908,7 +1009,18 @@ int32_t launch_delta_prep(const DeltaArgs& a, cudaStream_t s) {
 int32_t launch_delta_scan(const DeltaArgs& a, cudaStream_t s) { return a.f32 ? scan_dispatch<float>(a, s) : scan_dispatch<__nv_bfloat16>(a, s); }
 int32_t launch_delta_step(const DeltaArgs& a, cudaStream_t s) { return a.f32 ? step_dispatch<float>(a, s) : step_dispatch<__nv_bfloat16>(a, s); }
 int32_t launch_head_norm(const HeadNormArgs& a, cudaStream_t s) {
-    const dim3 grid((unsigned)a.T, (unsigned)((a.heads + 7) / 8));
+    const bool vec = a.n % 4 == 0 && a.n <= 128 && (a.ld_gate | a.ldo | a.w_stride) % 4 == 0 && ((uintptr_t)a.w % 16) == 0 && ((uintptr_t)a.gate % 16) == 0;
+    const unsigned rows = (unsigned)(a.runs ? a.n_runs * a.longest : a.T);
+    if (vec) {
+        const int lanes = a.n <= 32 ? 8 : a.n <= 64 ? 16 : 32, per = 256 / lanes * 2;
+        auto go = [&](auto kern) -> int32_t {
+            LC_CUDA(launch_pdl(kern, dim3(rows, (unsigned)((a.heads + per - 1) / per)), dim3(256), 0, s, a));
+            return LC_OK;
+        };
+        if (a.f32) return lanes == 8 ? go(head_norm4_kernel<float, 8>) : lanes == 16 ? go(head_norm4_kernel<float, 16>) : go(head_norm4_kernel<float, 32>);
+        return lanes == 8 ? go(head_norm4_kernel<bf16, 8>) : lanes == 16 ? go(head_norm4_kernel<bf16, 16>) : go(head_norm4_kernel<bf16, 32>);
+    }
+    const dim3 grid(rows, (unsigned)((a.heads + 7) / 8));
     if (a.f32) LC_CUDA(launch_pdl(head_norm_kernel<float>, grid, dim3(256), 0, s, a));
     else LC_CUDA(launch_pdl(head_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, s, a));
     return LC_OK;
