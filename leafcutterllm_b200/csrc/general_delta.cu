@@ -42,7 +42,7 @@ __global__ void __launch_bounds__(128) general_scan_kernel(const GeneralArgs a) 
     pdl_wait();
     const GeneralShape& g = a.g;
     const SeqRun run = a.runs[blockIdx.x];
-    const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r4 = lane & 3, col = warp * 8 + (lane >> 2), e = blockIdx.z * 32 + col, n = g.heads * g.dim;
+    const int h = blockIdx.y, warp = warp_index(), lane = threadIdx.x & 31, r4 = lane & 3, col = warp * 8 + (lane >> 2), e = blockIdx.z * 32 + col, n = g.heads * g.dim;
     float* st = a.state + ((size_t)run.seq * g.heads + h) * g.dim * g.dim;
     float S[DPL];
 #pragma unroll
@@ -240,7 +240,7 @@ __global__ void __launch_bounds__(chunk_threads(DP), chunk_ctas(DP)) general_chu
     constexpr int kColBlocks = DP / 4 / cols_per_warp(DP);
     extern __shared__ __align__(16) float sm[];
     // channel-major [DP][kPitch]: u e^(G_(t-1) - G_m), r e^(G_t - G_m), k e^(G_m - G_t), b e^(G_m - G_t); the first two are read side by side
-    float *s_u = sm, *s_r = s_u + DP * kPitch + 8, *s_k = s_r + DP * kPitch, *s_b = s_k + DP * kPitch;
+    float *s_u = sm, *s_r = s_u + DP * kPitch + 16, *s_k = s_r + DP * kPitch, *s_b = s_k + DP * kPitch;
     float *s_v = s_b + DP * kPitch, *s_y = s_v + kT * DP, *s_w = s_u;                 // [kT][DP] v, Y, W (in place of u)
     float *s_auk = s_y + kT * DP, *s_aub = s_auk + kT * kPitch, *s_brk = s_aub + kT * kPitch, *s_brb = s_brk + kT * kPitch;
     float *s_cm = s_brb + kT * kPitch, *s_ce = s_cm + DP, *s_ge = s_ce + DP;          // e^G_m, e^(G_end - G_m), e^G_end
@@ -249,41 +249,60 @@ __global__ void __launch_bounds__(chunk_threads(DP), chunk_ctas(DP)) general_chu
     pdl_wait();
     const GeneralShape& g = a.g;
     const DeltaChunk ck = a.chunks[blockIdx.x / kHalves];
-    const int sub = blockIdx.x % kHalves, n = min(kT, ck.n - sub * kT), h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, dim = g.dim;
+    const int sub = blockIdx.x % kHalves, n = min(kT, ck.n - sub * kT), h = blockIdx.y, tid = threadIdx.x, warp = warp_index(), lane = tid & 31, dim = g.dim;
     if (n <= 0) return;
     const size_t tok0 = (size_t)ck.tok0 + sub * kT;
     const ItemLayout L{DP};
     float* out = scratch + ((size_t)blockIdx.x * g.heads + h) * L.size();
     const bool vec = dim % 4 == 0;
-    auto four = [&](const float* p, int d, bool ok, float (&x)[4]) {
-        if (vec) {
-            const float4 f = ok && d < dim ? *(const float4*)(p + d) : make_float4(0.f, 0.f, 0.f, 0.f);
-            x[0] = f.x; x[1] = f.y; x[2] = f.z; x[3] = f.w;
-        } else {
+    {
+        // the operands' rows as they lie, [kT][kStage] in the places that their channel-major forms take afterwards
+        constexpr int kStage = DP + 4;
+        const float *p = a.proj + tok0 * g.ld + h * dim, *l = a.log_decay + tok0 * g.heads * dim + h * dim, *ab = a.a_bias + h * dim;
+        const size_t ld_l = (size_t)g.heads * dim;
+        for (int i = tid; i < kT * DP / 4; i += kThreads) {
+            const int t = i / (DP / 4), d = (i - t * (DP / 4)) * 4, at = t * kStage + d;
+            const float *row = p + (size_t)t * g.ld + d, *lrow = l + t * ld_l + d;
+            if (vec) {
+                const int bytes = t < n && d < dim ? 16 : 0;  // 0: zeros
+                const size_t o = bytes ? 0 : (size_t)t * g.ld + d, ol = bytes ? 0 : t * ld_l + d;
+                cp16(smem_u32(s_k + at), row - o + g.off_k, bytes);
+                cp16(smem_u32(s_u + at), lrow - ol, bytes);
+                cp16(smem_u32(s_r + at), row - o, bytes);
+                cp16(smem_u32(s_b + at), row - o + g.off_a, bytes);
+                cp16(smem_u32(s_v + t * DP + d), row - o + g.off_v, bytes);
+            } else {
 #pragma unroll
-            for (int j = 0; j < 4; j++) x[j] = ok && d + j < dim ? p[d + j] : 0.0f;
+                for (int j = 0; j < 4; j++) {
+                    const bool ok = t < n && d + j < dim;
+                    s_k[at + j] = ok ? row[g.off_k + j] : 0.0f;
+                    s_u[at + j] = ok ? lrow[j] : 0.0f;
+                    s_r[at + j] = ok ? row[j] : 0.0f;
+                    s_b[at + j] = ok ? row[g.off_a + j] : 0.0f;
+                    s_v[t * DP + d + j] = ok ? row[g.off_v + j] : 0.0f;
+                }
+            }
         }
-    };
-    {  // a lane per token
-        const bool ok = lane < n;
-        const size_t tok = tok0 + (ok ? lane : 0);
-        const float *p = a.proj + tok * g.ld + h * dim, *l = a.log_decay + tok * g.heads * dim + h * dim, *ab = a.a_bias + h * dim;
-        float k[kQuads][4], ld[kQuads][4], ss = 0.0f;
+        cp_commit();
+        float k[kQuads][4], G[kQuads][4], r[kQuads][4], ra[kQuads][4], ss = 0.0f;  // a lane per token, fours of channels per warp
 #pragma unroll
         for (int i = 0; i < kQuads; i++) {
-            const int d = 4 * (warp + i * kWarps);
-            if (d < DP) { four(p + g.off_k, d, ok, k[i]); four(l, d, ok, ld[i]); }
-            else k[i][0] = k[i][1] = k[i][2] = k[i][3] = 0.0f;
+            const int d0 = 4 * (warp + i * kWarps);
 #pragma unroll
-            for (int j = 0; j < 4; j++) ss = fmaf(k[i][j], k[i][j], ss);
+            for (int j = 0; j < 4; j++) ra[i][j] = d0 + j < dim ? __ldg(ab + d0 + j) : 0.0f;
+        }
+        cp_wait<0>();
+        __syncthreads();
+#pragma unroll
+        for (int i = 0; i < kQuads; i++) {
+            const int d0 = 4 * (warp + i * kWarps), at = lane * kStage + d0;
+            if (d0 >= DP) break;
+            float z[4];
+            get4(k[i], s_k + at); get4(G[i], s_u + at); get4(r[i], s_r + at); get4(z, s_b + at);
+#pragma unroll
+            for (int j = 0; j < 4; j++) { ss = fmaf(k[i][j], k[i][j], ss); ra[i][j] += z[j]; }
         }
         s_len[warp * 32 + lane] = ss;
-        for (int i = tid; i < kT * DP / 4; i += kThreads) {
-            const int t = i / (DP / 4), e = (i - t * (DP / 4)) * 4;
-            float v[4];
-            four(a.proj + (tok0 + (t < n ? t : 0)) * g.ld + g.off_v + h * dim, e, t < n, v);
-            *(float4*)(s_v + t * DP + e) = make_float4(v[0], v[1], v[2], v[3]);
-        }
         __syncthreads();
         ss = g.unit_eps;
 #pragma unroll
@@ -293,29 +312,25 @@ __global__ void __launch_bounds__(chunk_threads(DP), chunk_ctas(DP)) general_chu
         for (int i = 0; i < kQuads; i++) {
             const int d0 = 4 * (warp + i * kWarps);
             if (d0 >= DP) break;
-            float r[4], ra[4], bias[4], G[4];
-            four(p, d0, ok, r);
-            four(p + g.off_a, d0, ok, ra);
-            four(ab, d0, true, bias);
 #pragma unroll
-            for (int j = 0; j < 4; j++) G[j] = ld[i][j] * kLog2e;
+            for (int j = 0; j < 4; j++) G[i][j] *= kLog2e;
 #pragma unroll
             for (int o = 1; o < 32; o *= 2)
 #pragma unroll
                 for (int j = 0; j < 4; j++) {
-                    const float y = __shfl_up_sync(0xffffffffu, G[j], o);
-                    if (lane >= o) G[j] += y;
+                    const float y = __shfl_up_sync(0xffffffffu, G[i][j], o);
+                    if (lane >= o) G[i][j] += y;
                 }
 #pragma unroll
             for (int j = 0; j < 4; j++) {
-                const float up = __shfl_up_sync(0xffffffffu, G[j], 1), gp = lane > 0 ? up : 0.0f, gm = __shfl_sync(0xffffffffu, G[j], kT / 2 - 1),
-                            ge = __shfl_sync(0xffffffffu, G[j], 31);
-                const float u = k[i][j] * rk, back = exp2f(gm - G[j]);
+                const float up = __shfl_up_sync(0xffffffffu, G[i][j], 1), gp = lane > 0 ? up : 0.0f, gm = __shfl_sync(0xffffffffu, G[i][j], kT / 2 - 1),
+                            ge = __shfl_sync(0xffffffffu, G[i][j], 31);
+                const float u = k[i][j] * rk, back = exp2f(gm - G[i][j]);
                 const int d = d0 + j, at = d * kPitch + lane;
                 s_u[at] = u * exp2f(gp - gm);
-                s_r[at] = r[j] * exp2f(G[j] - gm);
+                s_r[at] = r[i][j] * exp2f(G[i][j] - gm);
                 s_k[at] = k[i][j] * back;
-                s_b[at] = __fdividef(u, 1.0f + __expf(-(ra[j] + bias[j]))) * back;
+                s_b[at] = __fdividef(u, 1.0f + __expf(-ra[i][j])) * back;
                 if (lane == 0) { s_cm[d] = exp2f(gm); s_ce[d] = exp2f(ge - gm); s_ge[d] = exp2f(ge); }
             }
         }
@@ -495,7 +510,7 @@ __global__ void __launch_bounds__(4 * DP) general_carry_kernel(const GeneralArgs
     extern __shared__ __align__(128) float sm[];
     __shared__ uint64_t full[2];
     float *s_m = sm, *s_c = s_m + 2 * kM, *s_S = s_c + 2 * kC, *s_part = s_S + kC;
-    const int tid = threadIdx.x, lane = tid & 31, group = tid / (2 * DP), warp = (tid >> 5) - group * (DP / 16), d0 = 16 * warp + 4 * Lanes::row(lane), e = 4 * Lanes::col(lane);
+    const int tid = threadIdx.x, lane = tid & 31, group = warp_index() / (DP / 16), warp = warp_index() - group * (DP / 16), d0 = 16 * warp + 4 * Lanes::row(lane), e = 4 * Lanes::col(lane);
     if (tid == 0) {
         mbar_init(&full[0], 1);
         mbar_init(&full[1], 1);
@@ -593,7 +608,7 @@ __global__ void __launch_bounds__(2 * DP) general_read_kernel(const GeneralArgs 
     __shared__ uint64_t full;
     __shared__ float s_ss[kColBlocks][kT];
     float *s_S = sm, *s_R = sm + DP * DP;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cb = warp % kColBlocks;
+    const int tid = threadIdx.x, warp = warp_index(), lane = tid & 31, cb = warp % kColBlocks;
     const int t0 = 4 * (warp / kColBlocks * Lanes::kRows + Lanes::row(lane)), e0 = 4 * (cb * cols_per_warp(DP) + Lanes::col(lane));
     if (tid == 0) {
         mbar_init(&full, 1);
@@ -679,7 +694,7 @@ __global__ void __launch_bounds__(2 * DP) general_read_kernel(const GeneralArgs 
 }
 
 int padded_dim(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : 128; }
-size_t chunk_smem(int dp) { return ((size_t)4 * dp * kPitch + 8 + 2 * kT * dp + 4 * kT * kPitch + 3 * dp + chunk_threads(dp)) * sizeof(float); }
+size_t chunk_smem(int dp) { return ((size_t)4 * dp * kPitch + 16 + 2 * kT * dp + 4 * kT * kPitch + 3 * dp + chunk_threads(dp)) * sizeof(float); }
 size_t carry_smem(int dp) { return ((size_t)2 * dp * dp + 4 * dp * 32) * sizeof(float); }
 size_t read_smem(int dp) { return ((size_t)dp * dp + dp * kT) * sizeof(float); }
 

@@ -173,7 +173,7 @@ __global__ void __launch_bounds__(256, NQ > 1 ? 1 : TAPS == 0 ? 4 : 3) attn_head
     pdl_launch_dependents();
     pdl_wait();
     const AttnShape& g = a.g;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, unit = blockIdx.y * 8 + warp;
+    const int warp = warp_index(), lane = threadIdx.x & 31, unit = blockIdx.y * 8 + warp;
     if (unit >= g.heads + (a.off_k >= 0 ? 2 * g.kv_heads : 0)) return;
     const bool is_q = unit < g.heads, is_v = unit >= g.heads + g.kv_heads;
     const int h = is_q ? unit : is_v ? unit - g.heads - g.kv_heads : unit - g.heads, n = is_v ? g.vdim : g.dim, half = g.rot_dims / 2;
@@ -469,7 +469,7 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
     __shared__ int s_last;
     const AttnShape& g = a.g;
     const int d16 = (g.dp + 15) & ~15, qp = d16 + 8, qb = qp * 2, kb_row = g.k_pitch * 2, vb_row = g.v_pitch * 2;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+    const int tid = threadIdx.x, warp = warp_index(), lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
     const int rep = g.heads / g.kv_heads, blocks = (rep + 15) / 16, t = blockIdx.x, kvh = blockIdx.y / blocks, r0 = (blockIdx.y % blocks) * 16, nh = min(16, rep - r0),
               h0 = kvh * rep + r0, pieces = gridDim.z;
     bf16 *s_q = (bf16*)smem, *s_k = s_q + 16 * qp + (size_t)warp * kDecStages * kDecKeys * (g.k_pitch + g.v_pitch), *s_v = s_k + kDecStages * kDecKeys * g.k_pitch;
@@ -669,7 +669,7 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
     const AttnShape& g = a.g;
     const int d16 = (g.dp + 15) & ~15, qp = d16 + 8, qb = qp * 2, kb_row = g.k_pitch * 2, vb_row = g.v_pitch * 2;
     bf16 *s_q = (bf16*)smem, *s_k = s_q + 64 * qp, *s_v = s_k + 2 * kKeys * g.k_pitch;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+    const int tid = threadIdx.x, warp = warp_index(), lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
     if (tid == 0) {
         mbar_init(&full[0], 1);
         mbar_init(&full[1], 1);

@@ -14,6 +14,9 @@ template <> __device__ __forceinline__ float act_f<bf16>(bf16 v) { return __bflo
 template <typename A> __device__ __forceinline__ A to_act(float v);
 template <> __device__ __forceinline__ float to_act<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 to_act<bf16>(float v) { return __float2bfloat16_rn(v); }
+// The warp's index as a value that the compiler knows to be the same in all lanes: collective instructions behind a branch on it
+// need no reconvergence.
+__device__ __forceinline__ int warp_index() { return __shfl_sync(0xffffffffu, (int)(threadIdx.x >> 5), 0); }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 __device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {

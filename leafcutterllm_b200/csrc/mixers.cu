@@ -451,7 +451,7 @@ __global__ void __launch_bounds__(256, CPL > 4 ? 2 : 3) delta_prep_kernel(const 
     pdl_launch_dependents();
     pdl_wait();
     const DeltaShape& g = a.g;
-    const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int unit = blockIdx.y * 8 + warp_index(), lane = threadIdx.x & 31;
     if (unit >= 2 * g.kv_heads + g.heads) return;
     const A* proj = (const A*)a.proj;
     const A* ring = (const A*)a.ring;
@@ -659,7 +659,7 @@ template <typename A>
 __global__ void __launch_bounds__(256) head_norm_kernel(const HeadNormArgs a) {
     pdl_launch_dependents();
     pdl_wait();
-    const int t = head_norm_row(a), h = blockIdx.y * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int t = head_norm_row(a), h = blockIdx.y * 8 + warp_index(), lane = threadIdx.x & 31;
     if (t < 0 || h >= a.heads) return;
     const float *o = a.o + ((size_t)t * a.heads + h) * a.n, *w = a.w + (size_t)h * a.w_stride;
     const A* gate = (const A*)a.gate + (size_t)t * a.ld_gate + (size_t)h * a.n;
@@ -974,7 +974,7 @@ int32_t launch_residual(const ResidualArgs& a, cudaStream_t s) {
         LC_CUDA(launch_pdl(kern, grid, threads ? dim3(threads) : block, 0, s, a));
         return LC_OK;
     };
-    if (!a.w) {
+    if (!a.w && a.x) {
         LC_CHECK(!moe && !pair, LC_ERR_UNSUPPORTED, "residual sum: a mixture or a pair without an output norm");
         const bool deep = a.depth.keep != nullptr;
         // few rows: a row by twice the threads
