@@ -244,7 +244,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32) attention_staged_kernel(AttnP
             if (tid == 0) p.counters[item] = 0;
         }
     }
-    if (!ok && tid == 0 && p.error_flag) atomicExch(p.error_flag, 1);
+    if (!ok && tid == 0 && p.error_flag) atomicCAS(p.error_flag, 0, 1);
 }
 
 // ---------------------------------------------------------------------------

@@ -139,7 +139,7 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap ktm, const __grid_co
             __threadfence_block();      // the arming above is visible before the count below
             armed[st] = i / S + 1;
         }
-        if (!ok && p.error_flag) atomicExch(p.error_flag, 1);
+        if (!ok && p.error_flag) atomicCAS(p.error_flag, 0, 1);
         return;  // the producer takes no part in the barriers below (they count the consumer threads)
     }
 
@@ -603,7 +603,7 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap ktm, const __grid_co
     }
     if (rg) rg[4] = gtime();
     if (P.ring && tid == 0) atomicMax(P.ring + (size_t)P.ring_slot * 16 + 6, gtime());
-    if (!ok && lane == 0 && p.error_flag) atomicExch(p.error_flag, 1);
+    if (!ok && lane == 0 && p.error_flag) atomicCAS(p.error_flag, 0, 1);
 }
 
 unsigned long long* g_aring = nullptr;

@@ -55,6 +55,12 @@ struct DenseParams {
     int list_stride;
 };
 
+// Raises the error word unless something did before; the words behind it tell which wait of which product.
+__device__ void raise_wait(const DenseParams& p, int code, int tile, int grouped, int item, int at) {
+    if (atomicCAS(p.error_flag, 0, code) != 0) return;
+    const int words[kErrorWords - 1] = {p.n, p.kblocks, p.T, tile, grouped, item, at};
+    for (int i = 0; i < kErrorWords - 1; i++) p.error_flag[1 + i] = words[i];
+}
 __device__ __forceinline__ float softplus_f(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 // The epilogue is a template parameter of the kernels; kEpiAny stands for the rarer elementwise ones, told apart at run time.
 constexpr int kEpiAny = -1;
@@ -167,7 +173,7 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
     unsigned* last_share = (unsigned*)(tmem_slot + 2);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
-        for (int i = 0; i < p.stages; i++) { mbar_init(&full[i], 1); mbar_init(&empty[i], 1); }
+        for (int i = 0; i < p.stages; i++) { mbar_init(&full[i], GROUPED && p.lists ? 3 : 1); mbar_init(&empty[i], 1); }
         for (int i = 0; i < 2; i++) { mbar_init(&acc_full[i], 1); mbar_init(&acc_empty[i], 32 * kEpiWarps); }
         *stop = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -224,9 +230,13 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
                 for (int kb = r.k0; kb < r.k1; kb++, wb += kABytes) {
                     unsigned char* a = smem + (size_t)st * kStage;
                     if (issued >= p.stages && !mbar_wait(&empty[st], phase)) { ok = false; break; }
+                    // every issuing warp arrives, also one without a gather: a warp that fell two rounds of the ring behind would take an old phase
+                    // of "empty" for the one that it waits for
                     if (warp == 0) {
                         mbar_expect_tx(&full[st], tx_bytes);
                         bulk_load(a, wb, kABytes, &full[st]);
+                    } else {
+                        mbar_arrive(&full[st]);
                     }
                     if (p.lists) {
 #pragma unroll 4
@@ -243,7 +253,7 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
         }
         if (!ok && warp == 0 && lane == 0) {
             *stop = 1;
-            atomicExch(p.error_flag, 11);
+            raise_wait(p, 11, NT, 1, blockIdx.x, issued);
             for (int i = max(0, issued - p.stages); i < issued; i++) mbar_wait(&full[i % p.stages], (uint32_t)(i / p.stages) & 1);
         }
         __syncwarp();
@@ -279,7 +289,7 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
         }
         if (!ok) {
             *stop = 1;
-            atomicExch(p.error_flag, 11);
+            raise_wait(p, 11, NT, 0, blockIdx.x, issued);
             for (int i = max(0, issued - p.stages); i < issued; i++) mbar_wait(&full[i % p.stages], (uint32_t)(i / p.stages) & 1);
         }
     } else if (warp == 1 && lane == 0) {
@@ -308,7 +318,7 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
             }
             if (ok) umma_commit(&acc_full[set]);
         }
-        if (!ok) { *stop = 1; atomicExch(p.error_flag, 12); }
+        if (!ok) { *stop = 1; raise_wait(p, 12, NT, GROUPED, blockIdx.x, tile * 65536 + st); }
     } else if (warp >= 4) {
         pdl_wait();  // earlier kernels may still read what this one overwrites
         constexpr int kHalf = NT >= 32 ? NT / 2 : NT;  // tokens of one warp; a 16-token tile leaves the second half idle
@@ -328,7 +338,7 @@ dense_umma_kernel(const unsigned char* __restrict__ w, const __grid_constant__ C
                     if (id >= 0 && id < p.table_rows) asm volatile("prefetch.global.L2 [%0];" ::"l"(p.table + (size_t)id * p.table_ld + row - lane));
                 }
             }
-            if (!mbar_wait(&acc_full[set], (uint32_t)(tile / 2) & 1)) { *stop = 1; if (lane == 0) atomicExch(p.error_flag, 13); break; }
+            if (!mbar_wait(&acc_full[set], (uint32_t)(tile / 2) & 1)) { *stop = 1; if (lane == 0) raise_wait(p, 13, NT, GROUPED, it, tile); break; }
             tc_fence_after();
             const uint32_t base = tmem + (uint32_t)set * kCols + ((uint32_t)(quarter * 32) << 16);
             const size_t plane = (size_t)NT * kM;

@@ -194,7 +194,7 @@ __global__ void __launch_bounds__(256) peer_ll_kernel(LLParams P, const void* __
         if (KEYS) reinterpret_cast<long long*>(dst)[i] = best;
         else reinterpret_cast<float*>(dst)[i] = acc;
     }
-    if (!ok && P.error_flag) atomicExch(P.error_flag, 3);
+    if (!ok && P.error_flag) atomicCAS(P.error_flag, 0, 3);
     __syncthreads();
     if (threadIdx.x == 0) {
         const unsigned t = atomicAdd(P.ticket, 1u);

@@ -506,15 +506,18 @@ static int32_t queue_flag_read(lc_model* m) {
     if (f) LC_CUDA(cudaMemcpyAsync(dst, f, sizeof(int), cudaMemcpyDeviceToHost, m->stream));
     return LC_OK;
 }
+static int32_t raised_error(lc_model* m) {
+    int w[kErrorWords] = {};
+    int* f = gemv_error_flag_dev();
+    cudaMemcpyAsync(w, f, sizeof w, cudaMemcpyDeviceToHost, m->stream);
+    cudaMemsetAsync(f, 0, sizeof w, m->stream);
+    cudaStreamSynchronize(m->stream);
+    set_error("a device-side check failed (code %d: %s; %d %d %d %d %d %d %d); the results of this call are not valid", w[0],
+              w[0] >= 20 ? "an index outside its range" : "a bounded wait ran out", w[1], w[2], w[3], w[4], w[5], w[6], w[7]);
+    return LC_ERR_CUDA;
+}
 static int32_t flag_result(lc_model* m) {
-    const int v = *reinterpret_cast<const int*>(m->pin_next + m->head_rows);
-    if (v != 0) {
-        cudaMemsetAsync(gemv_error_flag_dev(), 0, sizeof(int), m->stream);
-        set_error("a device-side check failed (code %d: %s); the results of this call are not valid", v,
-                  v >= 20 ? "an index outside its range" : "a bounded wait ran out");
-        return LC_ERR_CUDA;
-    }
-    return LC_OK;
+    return *reinterpret_cast<const int*>(m->pin_next + m->head_rows) != 0 ? raised_error(m) : LC_OK;
 }
 
 static int32_t check_device_flag(lc_model* m) {
@@ -523,13 +526,7 @@ static int32_t check_device_flag(lc_model* m) {
     int v = 0;
     LC_CUDA(cudaMemcpyAsync(&v, f, sizeof(int), cudaMemcpyDeviceToHost, m->stream));
     LC_CUDA(cudaStreamSynchronize(m->stream));
-    if (v != 0) {
-        cudaMemsetAsync(f, 0, sizeof(int), m->stream);
-        set_error("a device-side check failed (code %d: %s); the results of this call are not valid", v,
-                  v >= 20 ? "an index outside its range" : "a bounded wait ran out");
-        return LC_ERR_CUDA;
-    }
-    return LC_OK;
+    return v != 0 ? raised_error(m) : LC_OK;
 }
 
 extern "C" {

@@ -553,7 +553,7 @@ __global__ void __launch_bounds__(4 * DP) general_carry_kernel(const GeneralArgs
     __syncthreads();
     for (int c = 0; c < chunks; c++) {
         const float *mp = s_m + (c & 1) * kM + d0 + group * (DP / 2) * DP, *sp = s_S + e + group * (DP / 2) * 32;
-        if (!mbar_wait(&full[c & 1], (uint32_t)(c >> 1) & 1) && tid == 0) atomicExch(error_flag, 17);
+        if (!mbar_wait(&full[c & 1], (uint32_t)(c >> 1) & 1) && tid == 0) atomicCAS(error_flag, 0, 18);
         float acc[4][4] = {};
         if (group == 0) {
             float* keep = item(c) + L.c() + (size_t)blockIdx.z * kC + e;
@@ -645,7 +645,7 @@ __global__ void __launch_bounds__(2 * DP) general_read_kernel(const GeneralArgs 
     }
 #pragma unroll
     for (int j = 0; j < 4; j++) w[j] = e0 + j < g.dim ? a.norm_w[h * g.dim + e0 + j] : 0.0f;
-    if (!mbar_wait(&full, 0) && tid == 0) atomicExch(error_flag, 18);
+    if (!mbar_wait(&full, 0) && tid == 0) atomicCAS(error_flag, 0, 19);
     const float *rp = s_R + t0, *sp = s_S + (e0 / 32) * DP * 32 + e0 % 32;
 #pragma unroll 8
     for (int d = 0; d < DP; d++) {

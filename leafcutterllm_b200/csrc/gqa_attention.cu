@@ -512,7 +512,7 @@ __global__ void __launch_bounds__(32 * kDecWarps) attn_tokens_kernel(const AttnA
     const int krow = (lane & 7) + ((lane >> 4) << 3), kx = krow & g.k_swz, kc = (lane >> 3) & 1, vx = lane & 15 & g.v_swz, vc = lane >> 4;
     for (int j = 0; j < mine; j++) {
         const int st = j % kDecStages, key0 = tl.at(i0 + warp + j * kDecWarps) * kDecKeys;
-        if (!mbar_wait(&full[st], (uint32_t)(j / kDecStages) & 1)) atomicExch(error_flag, 15);
+        if (!mbar_wait(&full[st], (uint32_t)(j / kDecStages) & 1)) atomicCAS(error_flag, 0, 15);
         if (key0 + kDecKeys > pos + 1) {  // the rows behind the token: their weights are zero, the values have to be finite
             for (int i = lane; i < (key0 + kDecKeys - pos - 1) * (g.v_pitch / 8); i += 32) *(uint4*)(s_v + (st * kDecKeys + pos + 1 - key0) * g.v_pitch + i * 8) = make_uint4(0u, 0u, 0u, 0u);
             __syncwarp();
@@ -715,7 +715,7 @@ __global__ void __launch_bounds__(128) attn_tiles_kernel(const AttnArgs a, const
     const int krow = (lane & 7) + ((lane >> 4) << 3), kx = krow & g.k_swz, kc = (lane >> 3) & 1, vx = lane & 15 & g.v_swz, vc = lane >> 4;
     for (int i = 0; i < kt.n; i++) {
         const int buf = i & 1, key0 = kt.at(i) * kKeys;
-        if (!mbar_wait(&full[buf], (uint32_t)(i >> 1) & 1)) atomicExch(error_flag, 16);
+        if (!mbar_wait(&full[buf], (uint32_t)(i >> 1) & 1)) atomicCAS(error_flag, 0, 16);
         if (key0 + kKeys > last + 1) {  // the rows behind the last query: their weights are zero, the values have to be finite
             for (int c = tid; c < (key0 + kKeys - last - 1) * (g.v_pitch / 8); c += 128) *(uint4*)(s_v + (buf * kKeys + last + 1 - key0) * g.v_pitch + c * 8) = make_uint4(0u, 0u, 0u, 0u);
             __syncthreads();

@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 1) latent_decode_kernel(const 
         for (int i = tid; i < nh; i += kDecodeThreads) { pc.ml[(out_row + h0 + i) * 2] = -INFINITY; pc.ml[(out_row + h0 + i) * 2 + 1] = 0.0f; }
         return;
     }
-    auto wait = [&](uint64_t* bar, int phase) { if (!mbar_wait(bar, (uint32_t)phase & 1)) atomicExch(error_flag, 14); };
+    auto wait = [&](uint64_t* bar, int phase) { if (!mbar_wait(bar, (uint32_t)phase & 1)) atomicCAS(error_flag, 0, 14); };
     const uint32_t q_sm = smem_u32(s_q), k_sm = smem_u32(s_k), p_sm = smem_u32(s_p);
     // queries: the part carried through the key projection as it is, the other part rotated; zeros behind every row
     for (int i = tid; i < ROWS * (g.cp / 8); i += kDecodeThreads) {

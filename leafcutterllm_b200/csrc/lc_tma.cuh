@@ -128,7 +128,8 @@ static cudaError_t launch_pdl(void (*kern)(KArgs...), dim3 grid, dim3 block, siz
     return cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
 }
 
-int* gemv_error_flag_dev();
+int* gemv_error_flag_dev();  // kErrorWords words: the first check that failed (0: none), then what its kernel tells about it
+constexpr int kErrorWords = 8;
 constexpr size_t kMaxSmem = 227 * 1024;
 
 // qgemv_mma.cu: Q4_K through int8 tensor-core MMAs; *launched = false when the shape does not fit.

@@ -615,7 +615,7 @@ __global__ void __launch_bounds__(kRingThreads, 1) linear_ring_kernel(const Line
         }
         if (lane == 0) {
             if (!ok) {
-                atomicExch(error_flag, 17);
+                atomicCAS(error_flag, 0, 17);
                 for (int j = stored; j < loaded; j++) mbar_wait(&s_full[j % rs.stages], (uint32_t)(j / rs.stages) & 1);
             }
             bulk_wait<0>();
@@ -639,7 +639,7 @@ __global__ void __launch_bounds__(kRingThreads, 1) linear_ring_kernel(const Line
         int pos_next = pos;
         fetch(j + 1, bl_next, pos_next);
         const float2 decay = pos > 0 ? decay_of(a, h, bl.y) : make_float2(0.0f, 0.0f);
-        if (ok && !mbar_wait(&s_full[st], (uint32_t)(j / rs.stages) & 1)) { ok = false; atomicExch(error_flag, 17); }  // every thread goes on to the barriers
+        if (ok && !mbar_wait(&s_full[st], (uint32_t)(j / rs.stages) & 1)) { ok = false; atomicCAS(error_flag, 0, 17); }  // every thread goes on to the barriers
         float* S = (float*)(ring_smem + (size_t)st * rs.stage_bytes);
         const A *q = (const A*)(S + state_elems), *k = q + g.dim, *v = k + g.dim;
         float* so = s_o + (j & 1) * groups * g.vdim;

@@ -610,7 +610,7 @@ qgemm_umma_q4k_kernel(const __grid_constant__ CUtensorMap tmw0, const __grid_con
             }
         }
     }
-    if (!ok && p.error_flag) atomicExch(p.error_flag, 3);
+    if (!ok && p.error_flag) atomicCAS(p.error_flag, 0, 3);
     tc_fence_before();
     __syncthreads();
     pdl_launch_dependents();

@@ -460,7 +460,7 @@ qgemv_tma_kernel(const __grid_constant__ CUtensorMap tm0, const __grid_constant_
             }
         }
     }
-    if (!ok && lane == 0 && p.error_flag) atomicExch(p.error_flag, 1);
+    if (!ok && lane == 0 && p.error_flag) atomicCAS(p.error_flag, 0, 1);
 }
 
 // ---------------------------------------------------------------------------
@@ -521,7 +521,7 @@ bool pdl_enabled() {
 }
 // The word kernels raise when a bounded wait runs out.  It lives in the library image (zero when the image is loaded on a
 // device), so looking it up allocates nothing: entry points that promise not to allocate can use every kernel.
-static __device__ int g_error_flag_word;
+static __device__ int g_error_flag_word[kErrorWords];
 static int* g_error_flag[16] = {};
 int* gemv_error_flag_dev() {
     int dev = 0;

@@ -581,7 +581,7 @@ qgemv_mma_q4k_kernel(const __grid_constant__ CUtensorMap tm0, const __grid_const
     }
     if (rg) rg[3] = gtime();
     if (p.ring && threadIdx.x == 0) atomicMax(p.ring + 6, gtime());  // the last CTA to finish
-    if (!ok && lane == 0 && p.error_flag) atomicExch(p.error_flag, 1);
+    if (!ok && lane == 0 && p.error_flag) atomicCAS(p.error_flag, 0, 1);
 }
 
 // The activations of a grouped launch, once per call: row r of x (RMS-normalised with gains when norm_w is given,
